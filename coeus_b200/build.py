@@ -1,10 +1,13 @@
 """In-tree builder for the native libraries.
 
-Two shared objects are produced under ``coeus_b200/lib/``:
+These shared objects are produced under ``coeus_b200/lib/``:
 
 * ``libcoeus_kernels.so`` – every ``.cu`` file of ``coeus_b200/csrc`` compiled by ``nvcc`` for
   ``sm_100a`` only (``-gencode arch=compute_100a,code=sm_100a``); plain ``extern "C"`` entry
   points that take raw device pointers and a stream, loaded through ``ctypes``.
+* ``libcoeus_serving.so`` – the subset of the same sources that a model served through the ragged
+  step needs (``SERVING_SOURCES``); built only where the full library is absent, so that a fresh
+  checkout compiles what it is about to run and nothing else.
 * ``_coeus_host*.so`` – the host-side C++ components of ``csrc/host`` (``tokenizers.cpp``,
   ``io.cpp`` checkpoint formats, ``pipeline.cpp`` data loader / suffix array / bloom filter /
   arena, ``oracle.cpp`` CPU oracle) as a pybind11 module.
@@ -36,6 +39,9 @@ NVCC_FLAGS = [
 ]
 
 
+SERVING_SOURCES = ("gemm", "ragged_rows", "shortconv", "delta_scan", "linear_f32", "ragged_attn")
+
+
 def _nvcc() -> str:
     for cand in (os.environ.get("NVCC"), shutil.which("nvcc"), "/usr/local/cuda/bin/nvcc"):
         if cand and os.path.exists(cand):
@@ -55,19 +61,48 @@ def kernels_lib_path() -> Path:
     return LIB / "libcoeus_kernels.so"
 
 
+def serving_lib_path() -> Path:
+    return LIB / "libcoeus_serving.so"
+
+
 def host_lib_path() -> Path:
     suffix = sysconfig.get_config_var("EXT_SUFFIX") or ".so"
     return LIB / f"_coeus_host{suffix}"
 
 
+def _sources(names=None):
+    cus = sorted(CSRC.glob("*.cu"))
+    return cus if names is None else [p for p in cus if p.stem in names]
+
+
+def _headers():
+    return sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+
+
+def kernels_current() -> bool:
+    """Whether the full kernel library exists and was built from the sources as they are."""
+    stamp = LIB / "kernels.sha256"
+    return kernels_lib_path().exists() and stamp.exists() and \
+        stamp.read_text() == _digest(_sources() + _headers())
+
+
+def build_serving(force: bool = False) -> Path:
+    """The library with the kernels of the ragged serving step: the full one where it is current,
+    else ``libcoeus_serving.so``."""
+    if not force and kernels_current():
+        return kernels_lib_path()
+    return _build_lib(serving_lib_path(), LIB / "serving.sha256", _sources(SERVING_SOURCES), force,
+                      False)
+
+
 def build_kernels(force: bool = False, verbose: bool = False) -> Path:
+    return _build_lib(kernels_lib_path(), LIB / "kernels.sha256", _sources(), force, verbose)
+
+
+def _build_lib(out: Path, stamp: Path, cus, force: bool, verbose: bool) -> Path:
     LIB.mkdir(exist_ok=True)
     OBJ.mkdir(exist_ok=True)
-    out = kernels_lib_path()
-    cus = sorted(CSRC.glob("*.cu"))
-    hdrs = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    stamp = LIB / "kernels.sha256"
-    digest = _digest(cus + hdrs)
+    digest = _digest(cus + _headers())
     if not force and out.exists() and stamp.exists() and stamp.read_text() == digest:
         return out
     nvcc = _nvcc()

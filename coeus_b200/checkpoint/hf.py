@@ -75,13 +75,13 @@ def config_from_hf(hf_config: Any) -> DecoderConfig:
 
 
 def load_hf_llama(state: Mapping[str, torch.Tensor], hf_config: Any, device="cuda",
-                  training: bool = False):
+                  training: bool = False, dtype: torch.dtype = None):
     """A :class:`coeus_b200.models.decoder.DecoderLM` holding the weights of ``state``."""
     from ..models.decoder import DecoderLM
     cfg = config_from_hf(hf_config)
     dev = torch.device(device)
     lm = DecoderLM(cfg, dev, init="zeros", training=training,
-                   dtype=torch.bfloat16 if dev.type == "cuda" else torch.float32)
+                   dtype=dtype or (torch.bfloat16 if dev.type == "cuda" else torch.float32))
     V = cfg.vocab_size
     n1, n2, fn = lm.layout.norm_names
 
@@ -141,7 +141,7 @@ def config_from_hf_gpt2(hf_config: Any) -> DecoderConfig:
 
 
 def load_hf_gpt2(state: Mapping[str, torch.Tensor], hf_config: Any, device="cuda",
-                 training: bool = False):
+                 training: bool = False, dtype: torch.dtype = None):
     """A :class:`coeus_b200.models.decoder.DecoderLM` holding a ``GPT2LMHeadModel`` state dict.
     GPT-2 stores its projections as ``[in, out]`` already (its ``Conv1D``), which is the layout
     used here, so nothing is transposed."""
@@ -149,7 +149,7 @@ def load_hf_gpt2(state: Mapping[str, torch.Tensor], hf_config: Any, device="cuda
     cfg = config_from_hf_gpt2(hf_config)
     dev = torch.device(device)
     lm = DecoderLM(cfg, dev, init="zeros", training=training,
-                   dtype=torch.bfloat16 if dev.type == "cuda" else torch.float32)
+                   dtype=dtype or (torch.bfloat16 if dev.type == "cuda" else torch.float32))
     V = cfg.vocab_size
     n1, n2, fn = lm.layout.norm_names
 
@@ -254,36 +254,14 @@ def to_hf_llama(lm) -> Tuple[Dict[str, torch.Tensor], Dict[str, Any]]:
     return out, hf
 
 
-def load_hf_dir(path: str, device="cuda", training: bool = False):
-    """A model directory in the Hugging Face layout: ``config.json`` plus one ``.safetensors``
-    file or several with ``model.safetensors.index.json``."""
-    import glob
-    import json
-    import os
-
-    from .formats import load_safetensors
-    with open(os.path.join(path, "config.json")) as f:
-        hf_config = json.load(f)
-    files = sorted(glob.glob(os.path.join(path, "*.safetensors")))
-    if not files:
-        raise ProcessingError.invalid_input(f"no .safetensors file in {path}")
-    state: Dict[str, torch.Tensor] = {}
-    for fpath in files:
-        tensors, _ = load_safetensors(fpath)
-        state.update(tensors)
-    if hf_config.get("model_type") == "gpt2":
-        return load_hf_gpt2(state, hf_config, device=device, training=training)
-    return load_hf_llama(state, hf_config, device=device, training=training)
+def load_hf_dir(path: str, device="cuda", training: bool = False, dtype=None):
+    """A model directory: ``config.json`` plus one ``.safetensors`` file or several.  The model
+    registry (:mod:`coeus_b200.models.registry`) picks the architecture by ``config.json``."""
+    from ..models.registry import load_dir
+    return load_dir(path, device=device, training=training, dtype=dtype)
 
 
 def save_hf_dir(lm, path: str) -> None:
-    """Write ``config.json`` and ``model.safetensors`` in the Hugging Face naming."""
-    import json
-    import os
-
-    from .formats import save_safetensors
-    os.makedirs(path, exist_ok=True)
-    state, fields = to_hf_gpt2(lm) if lm.cfg.pos == "learned" else to_hf_llama(lm)
-    save_safetensors(os.path.join(path, "model.safetensors"), state, {"format": "pt"})
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(fields, f, indent=1)
+    """Write ``config.json`` and ``model.safetensors`` in the naming of the model's architecture."""
+    from ..models.registry import save_dir
+    save_dir(lm, path)

@@ -1,0 +1,232 @@
+// Gated delta rule with one decay per key channel, over a ragged batch, in fp32.  Per head, with
+// the state S [dim, vdim] carried from token to token:
+//   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+// The columns of S are independent, so a block takes one (entry, head) and 8 columns per warp and
+// keeps its part of S in registers from the first token of the entry to the last.  Eight lanes
+// share a column pair, each holding R of the key channels.  Both products of a token use the
+// decayed state (o = S^T q + (k . q) u), so one reduction over the eight lanes serves them; the
+// arithmetic is two-wide packed fp32.  Tokens are staged in shared memory a few ahead.
+#include "ragged.cuh"
+
+namespace cb {
+
+using f2 = unsigned long long;     // two packed fp32 values
+__device__ __forceinline__ f2 mul_f2(f2 a, f2 b) {
+  f2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f2 fma_f2(f2 a, f2 b, f2 c) {
+  f2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f2 pack_f2(float lo, float hi) {
+  f2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 unpack_f2(f2 a) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a));
+  return r;
+}
+__device__ __forceinline__ float hsum_f2(f2 a) {
+  const float2 r = unpack_f2(a);
+  return r.x + r.y;
+}
+__device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory");
+}
+
+constexpr int SCAN_WARPS = 4;
+constexpr int SCAN_COLS = SCAN_WARPS * 8;
+constexpr int SCAN_TB = 8;         // tokens per stage
+
+struct ScanArgs {
+  const float* q;      // [rows, kv_heads, dim4]
+  const float* k;      // [rows, kv_heads, dim4]
+  const float* kq;     // [rows, kv_heads]
+  const float* v;      // [rows, heads, vdim]
+  const float* g;      // [rows, heads, dim4]
+  const float* beta;   // [rows, heads]
+  float* state;        // [slots, heads, dim, vdim]
+  float* o;            // out [rows, heads, vdim]
+  int heads, kv_heads, dim, dim4, vdim;
+  Entries e;
+};
+
+template <int R>       // key channels per lane; 8 R >= dim, R a multiple of 4
+__global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanArgs p) {
+  constexpr int DP = 8 * R;                                  // channels, padded with zeros
+  constexpr int STAGE = SCAN_TB * (3 * DP + SCAN_COLS + 4);  // floats
+  extern __shared__ __align__(16) float sm[];
+  const int e = blockIdx.y, h = blockIdx.x % p.heads, slab = blockIdx.x / p.heads;
+  const int hk = h / (p.heads / p.kv_heads);
+  const int row0 = p.e.row0[e], len = p.e.len[e], slot = p.e.slot[e];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ld = lane & 7;
+  const int col_base = slab * SCAN_COLS;
+  const int c0 = warp * 8 + (lane >> 3) * 2;                 // first of this lane's two columns
+  float* st = p.state + (static_cast<size_t>(slot) * p.heads + h) * p.dim * p.vdim;
+
+  auto fetch = [&](int stage, int t0) {
+    const uint32_t base = smem_u32(sm + stage * STAGE);
+    const int n = min(SCAN_TB, len - t0);
+    constexpr int CH = DP / 4;
+    for (int i = threadIdx.x; i < n * 3 * CH; i += SCAN_WARPS * 32) {
+      const int t = i / (3 * CH), w = (i / CH) % 3, c = i % CH;
+      const int row = row0 + t0 + t;
+      const bool in = c * 4 < p.dim4;
+      const float* src = w == 2 ? p.g + (static_cast<size_t>(row) * p.heads + h) * p.dim4
+                                : (w == 0 ? p.q : p.k) +
+                                      (static_cast<size_t>(row) * p.kv_heads + hk) * p.dim4;
+      cp_async16_zfill(base + ((t * 3 + w) * DP + c * 4) * 4, src + (in ? c * 4 : 0), in ? 16 : 0);
+    }
+    const uint32_t vb = base + SCAN_TB * 3 * DP * 4;
+    for (int i = threadIdx.x; i < n * SCAN_COLS; i += SCAN_WARPS * 32) {
+      const int t = i / SCAN_COLS, c = i % SCAN_COLS;
+      if (col_base + c < p.vdim)
+        cp_async4(vb + i * 4, p.v + (static_cast<size_t>(row0 + t0 + t) * p.heads + h) * p.vdim +
+                                  col_base + c);
+    }
+    const uint32_t sb = vb + SCAN_TB * SCAN_COLS * 4;
+    for (int i = threadIdx.x; i < n * 2; i += SCAN_WARPS * 32) {
+      const int row = row0 + t0 + (i >> 1);
+      cp_async4(sb + i * 4, (i & 1) ? p.kq + static_cast<size_t>(row) * p.kv_heads + hk
+                                    : p.beta + static_cast<size_t>(row) * p.heads + h);
+    }
+    cp_async_commit();
+  };
+
+  fetch(0, 0);
+  f2 s[2][R / 2];
+  const bool has_state = p.e.pos0[e] > 0;
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    const int col = col_base + c0 + c;
+#pragma unroll
+    for (int i = 0; i < R / 2; ++i) {
+      const int d = (i / 2) * 32 + ld * 4 + (i % 2) * 2;
+      float x = 0.f, y = 0.f;
+      if (has_state && col < p.vdim) {
+        if (d < p.dim) x = st[static_cast<size_t>(d) * p.vdim + col];
+        if (d + 1 < p.dim) y = st[static_cast<size_t>(d + 1) * p.vdim + col];
+      }
+      s[c][i] = pack_f2(x, y);
+    }
+  }
+  const int my = c0 + ((ld >> 1) & 1);                       // the column this lane finishes
+  int stage = 0;
+  for (int t0 = 0; t0 < len; t0 += SCAN_TB, stage ^= 1) {
+    const bool more = t0 + SCAN_TB < len;
+    if (more) {
+      fetch(stage ^ 1, t0 + SCAN_TB);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const float* sb = sm + stage * STAGE;
+    const float* sv = sb + SCAN_TB * 3 * DP;
+    const float* ss = sv + SCAN_TB * SCAN_COLS;
+    const int n = min(SCAN_TB, len - t0);
+    for (int t = 0; t < n; ++t) {
+      const float* tq = sb + t * 3 * DP + ld * 4;
+      f2 a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull;
+      f2 kk[R / 2];
+#pragma unroll
+      for (int j = 0; j < R / 4; ++j) {
+        const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(tq + j * 32);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(tq + DP + j * 32);
+        const ulonglong2 g2 = *reinterpret_cast<const ulonglong2*>(tq + 2 * DP + j * 32);
+        kk[2 * j] = k2.x;
+        kk[2 * j + 1] = k2.y;
+        s[0][2 * j] = mul_f2(s[0][2 * j], g2.x);
+        s[0][2 * j + 1] = mul_f2(s[0][2 * j + 1], g2.y);
+        s[1][2 * j] = mul_f2(s[1][2 * j], g2.x);
+        s[1][2 * j + 1] = mul_f2(s[1][2 * j + 1], g2.y);
+        a0 = fma_f2(s[0][2 * j], k2.x, a0);
+        a1 = fma_f2(s[1][2 * j], k2.x, a1);
+        b0 = fma_f2(s[0][2 * j], q2.x, b0);
+        b1 = fma_f2(s[1][2 * j], q2.x, b1);
+        a0 = fma_f2(s[0][2 * j + 1], k2.y, a0);
+        a1 = fma_f2(s[1][2 * j + 1], k2.y, a1);
+        b0 = fma_f2(s[0][2 * j + 1], q2.y, b0);
+        b1 = fma_f2(s[1][2 * j + 1], q2.y, b1);
+      }
+      // sum over the eight lanes, ending with one value per lane: bit 0 of ld picks S^T k or
+      // S^T q, bit 1 the column
+      const float fa0 = hsum_f2(a0), fa1 = hsum_f2(a1), fb0 = hsum_f2(b0), fb1 = hsum_f2(b1);
+      const bool odd = ld & 1, hi = ld & 2;
+      float x0 = (odd ? fb0 : fa0) + __shfl_xor_sync(0xffffffffu, odd ? fa0 : fb0, 1);
+      float x1 = (odd ? fb1 : fa1) + __shfl_xor_sync(0xffffffffu, odd ? fa1 : fb1, 1);
+      float y = (hi ? x1 : x0) + __shfl_xor_sync(0xffffffffu, hi ? x0 : x1, 2);
+      y += __shfl_xor_sync(0xffffffffu, y, 4);
+      const float beta = ss[t * 2], kq = ss[t * 2 + 1];
+      const float un = beta * (sv[t * SCAN_COLS + my] - y);  // of use on even lanes
+      const float u0 = __shfl_sync(0xffffffffu, un, lane & 24);
+      const float u1 = __shfl_sync(0xffffffffu, un, (lane & 24) | 2);
+      const f2 p0 = pack_f2(u0, u0), p1 = pack_f2(u1, u1);
+#pragma unroll
+      for (int i = 0; i < R / 2; ++i) {
+        s[0][i] = fma_f2(kk[i], p0, s[0][i]);
+        s[1][i] = fma_f2(kk[i], p1, s[1][i]);
+      }
+      if (odd && ld < 4 && col_base + my < p.vdim)
+        p.o[(static_cast<size_t>(row0 + t0 + t) * p.heads + h) * p.vdim + col_base + my] =
+            y + kq * (hi ? u1 : u0);
+    }
+    __syncthreads();                                         // the stage may be refilled
+  }
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    const int col = col_base + c0 + c;
+    if (col >= p.vdim) continue;
+#pragma unroll
+    for (int i = 0; i < R / 2; ++i) {
+      const int d = (i / 2) * 32 + ld * 4 + (i % 2) * 2;
+      const float2 x = unpack_f2(s[c][i]);
+      if (d < p.dim) st[static_cast<size_t>(d) * p.vdim + col] = x.x;
+      if (d + 1 < p.dim) st[static_cast<size_t>(d + 1) * p.vdim + col] = x.y;
+    }
+  }
+}
+
+template <int R>
+static int launch_scan(const ScanArgs& a, int entries, cudaStream_t st) {
+  const int smem = 2 * SCAN_TB * (3 * 8 * R + SCAN_COLS + 4) * 4;
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             smem) != cudaSuccess)
+      return -4;
+    set = true;
+  }
+  dim3 grid(a.heads * ((a.vdim + SCAN_COLS - 1) / SCAN_COLS), entries);
+  delta_scan_kernel<R><<<grid, SCAN_WARPS * 32, smem, st>>>(a);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+}  // namespace cb
+
+using namespace cb;
+
+extern "C" int cb_delta_scan(const float* q, const float* k, const float* kq, const float* v,
+                             const float* g, const float* beta, float* state, float* o, int heads,
+                             int kv_heads, int dim, int dim4, int vdim, const int* slot,
+                             const int* row0, const int* len, const int* pos0, int entries,
+                             void* stream) {
+  if (entries <= 0 || entries > 65535 || heads % kv_heads != 0) return -1;
+  if (dim > 256 || dim4 < dim || dim4 % 4 != 0) return -2;
+  ScanArgs a;
+  a.q = q; a.k = k; a.kq = kq; a.v = v; a.g = g; a.beta = beta; a.state = state; a.o = o;
+  a.heads = heads; a.kv_heads = kv_heads; a.dim = dim; a.dim4 = dim4; a.vdim = vdim;
+  a.e.slot = slot; a.e.row0 = row0; a.e.len = len; a.e.pos0 = pos0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dim <= 32) return launch_scan<4>(a, entries, st);
+  if (dim <= 64) return launch_scan<8>(a, entries, st);
+  if (dim <= 96) return launch_scan<12>(a, entries, st);
+  if (dim <= 128) return launch_scan<16>(a, entries, st);
+  if (dim <= 192) return launch_scan<24>(a, entries, st);
+  return launch_scan<32>(a, entries, st);
+}

@@ -12,8 +12,8 @@
 //   dgrad    dX[M,K] = dY[M,N]  . W[K,N]^T    A K-major,  B K-major
 //   wgrad    dW[K,N] = X[M,K]^T . dY[M,N]     A MN-major, B MN-major (split along tokens,
 //                                             fp32 atomic accumulation)
-// Fused epilogues: alpha scale, +bias[N], GELU(tanh) with the pre-activation kept, dGELU,
-// +residual, bf16 / fp32 / fp32-atomic-add output.
+// Fused epilogues: alpha scale, +bias[N], GELU(tanh) with the pre-activation kept, dGELU, squared
+// ReLU, +residual, bf16 / fp32 / fp32-atomic-add output.
 #include <cudaTypedefs.h>
 
 #include <cstring>
@@ -30,7 +30,7 @@ constexpr int AG_PARTS = 8;   // row groups a pulled tile is split into
 constexpr int MAX_TP = 8;
 enum : int { COMM_NONE = 0, COMM_AG = 1, COMM_RS = 2 };
 
-enum : int { EPI_NONE = 0, EPI_GELU = 1, EPI_DGELU = 2, EPI_SWIGLU_BWD = 3 };
+enum : int { EPI_NONE = 0, EPI_GELU = 1, EPI_DGELU = 2, EPI_SWIGLU_BWD = 3, EPI_RELU2 = 4 };
 enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_F32_ATOMIC = 2, OUT_DISCARD = 3 };
 
 struct GemmArgs {
@@ -125,6 +125,12 @@ __device__ __forceinline__ void epilogue_math(const GemmArgs& p, float* v, float
     for (int j = 0; j < 32; ++j) {
       u[j] = v[j];
       v[j] = gelu_tanh(v[j]);
+    }
+  } else if (p.epi == EPI_RELU2) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+      v[j] = fmaxf(v[j], 0.f);
+      v[j] *= v[j];
     }
   } else if (p.epi == EPI_DGELU && row_ok) {
     const __nv_bfloat16* ap = p.aux_in + static_cast<size_t>(row) * p.ldaux + col0;

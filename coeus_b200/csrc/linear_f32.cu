@@ -1,0 +1,72 @@
+// fp32 linear layer Y[M, N] = act(X[M, K] . W[N, K]^T) on the FMA units, for serving a model in
+// full 32-bit precision: 64 x 64 tiles, 4 x 4 outputs per thread, operands staged in shared memory.
+#include "ragged.cuh"
+
+namespace cb {
+
+constexpr int LT = 64, LK = 16;
+enum : int { ACT_NONE = 0, ACT_RELU2 = 4, ACT_SOFTCAP = 5 };
+
+__global__ void __launch_bounds__(256)
+linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw,
+                  float* __restrict__ y, int ldy, int M, int N, int K, int act, float act_arg,
+                  int accumulate) {
+  __shared__ float sx[LK][LT + 4], sw[LK][LT + 4];
+  const int m0 = blockIdx.y * LT, n0 = blockIdx.x * LT;
+  const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+  const int lr = threadIdx.x / 4, lc = (threadIdx.x % 4) * 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += LK) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+    if (k0 + lc < K) {                              // K is a multiple of 4
+      if (m0 + lr < M) a = *reinterpret_cast<const float4*>(x + static_cast<size_t>(m0 + lr) * ldx + k0 + lc);
+      if (n0 + lr < N) b = *reinterpret_cast<const float4*>(w + static_cast<size_t>(n0 + lr) * ldw + k0 + lc);
+    }
+    __syncthreads();
+    sx[lc][lr] = a.x; sx[lc + 1][lr] = a.y; sx[lc + 2][lr] = a.z; sx[lc + 3][lr] = a.w;
+    sw[lc][lr] = b.x; sw[lc + 1][lr] = b.y; sw[lc + 2][lr] = b.z; sw[lc + 3][lr] = b.w;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < LK; ++k) {
+      const float4 u = *reinterpret_cast<const float4*>(&sx[k][ty * 4]);
+      const float4 v = *reinterpret_cast<const float4*>(&sw[k][tx * 4]);
+      const float uu[4] = {u.x, u.y, u.z, u.w}, vv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += uu[i] * vv[j];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) continue;
+      float v = acc[i][j];
+      if (act == ACT_RELU2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      } else if (act == ACT_SOFTCAP) {
+        v = act_arg * tanhf(v / act_arg);
+      }
+      float* dst = y + static_cast<size_t>(m) * ldy + n;
+      *dst = accumulate ? *dst + v : v;
+    }
+  }
+}
+
+}  // namespace cb
+
+extern "C" int cb_linear_f32(const float* x, int ldx, const float* w, int ldw, float* y, int ldy,
+                             int M, int N, int K, int act, float act_arg, int accumulate,
+                             void* stream) {
+  if (M <= 0 || N <= 0 || K <= 0 || K % 4 || ldx % 4 || ldw % 4) return -1;
+  dim3 grid((N + cb::LT - 1) / cb::LT, (M + cb::LT - 1) / cb::LT);
+  if (grid.y > 65535) return -1;
+  cb::linear_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      x, ldx, w, ldw, y, ldy, M, N, K, act, act_arg, accumulate);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}

@@ -1,0 +1,85 @@
+// Shared pieces of the kernels that run a ragged batch: every step brings a number of sequences
+// ("entries"), each with its own count of new tokens, laid out one after the other in the rows
+// of the activations.  Activations are bf16 or fp32 (template parameter); arithmetic is fp32.
+#pragma once
+#include "common.cuh"
+#include "ptx.cuh"
+
+namespace cb {
+
+int sm_count();
+
+// The entries of one step.  Entry e owns rows row0[e] .. row0[e] + len[e] - 1, its first row is
+// the token at position pos0[e] of its sequence, and its cache pages and recurrent state are
+// those of slot[e].  A sequence whose pos0 is 0 starts from an empty state whatever its slot
+// holds, so slots need no clearing between requests.
+struct Entries {
+  const int* slot;
+  const int* row0;
+  const int* len;
+  const int* pos0;
+};
+
+constexpr int RAGGED_PAGE = 64;   // tokens per cache page
+
+template <typename T>
+__device__ __forceinline__ float to_f32(T v);
+template <>
+__device__ __forceinline__ float to_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ float to_f32<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_f32(float v);
+template <>
+__device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+// V (1 or 8) consecutive values; the 8-wide form needs 16-byte (bf16) / 32-byte-multiple rows.
+template <int V>
+__device__ __forceinline__ void load_vec(const __nv_bfloat16* p, float* f) {
+  if constexpr (V == 8) load8(p, f);
+  else f[0] = __bfloat162float(*p);
+}
+template <int V>
+__device__ __forceinline__ void load_vec(const float* p, float* f) {
+  if constexpr (V == 8) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_vec(__nv_bfloat16* p, const float* f) {
+  if constexpr (V == 8) store8(p, f);
+  else *p = __float2bfloat16(f[0]);
+}
+template <int V>
+__device__ __forceinline__ void store_vec(float* p, const float* f) {
+  if constexpr (V == 8) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+  } else {
+    *p = f[0];
+  }
+}
+
+__device__ __forceinline__ float sigmoidf_(float x) { return 1.0f / (1.0f + expf(-x)); }
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+// copies `bytes` (0 or 16) and zero-fills the rest of the 16 bytes
+__device__ __forceinline__ void cp_async16_zfill(uint32_t dst, const void* src, int bytes) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes)
+               : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+
+}  // namespace cb

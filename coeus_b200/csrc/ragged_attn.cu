@@ -1,0 +1,568 @@
+// Attention of a ragged batch over the paged cache: every query row sits at its own position of
+// its own sequence and sees the cached keys of its chunk up to itself (chunk = 0: all of them).
+// The softmax may have a sink per head (a logit in the denominator only) and the head's output a
+// gate (a sigmoid of a projected number).  Query head h reads key/value head h / (heads / kv_heads);
+// query/key width and value width are independent.
+//
+//   rows kernel    one CTA per (query row, key/value head, split): the query heads of the group
+//                  share every key and value that is loaded.  Decoding, and everything in fp32.
+//   tiles kernel   64 query rows of one head on the tensor cores (mma m16n8k16), one cache page
+//                  per step through a double-buffered shared-memory ring.  The weights enter the
+//                  second product as the sum of two bf16 numbers, so they keep 16 mantissa bits.
+#include "ragged.cuh"
+
+namespace cb {
+
+constexpr float LOG2E = 1.4426950408889634f;
+
+struct RaggedAttn {
+  const void* q;           // [rows, heads * dim]
+  const void* k_cache;     // [pages, PAGE, kv_heads, dim_p]
+  const void* v_cache;     // [pages, PAGE, kv_heads, vdim_p]
+  const int* page_table;   // [slots, max_pages]
+  int max_pages, num_pages;
+  int heads, kv_heads, dim, vdim, dim_p, vdim_p;
+  int chunk;
+  float scale;
+  const float* sink;       // [heads] or null
+  const void* gate;        // [rows, ldg] or null: column h gates head h
+  int ldg;
+  void* out;               // [rows, ldo]
+  int ldo;
+  int* status;
+};
+
+__device__ __forceinline__ int chunk_start(int pos, int chunk) {
+  return chunk > 0 ? pos / chunk * chunk : 0;
+}
+template <typename T>
+__device__ __forceinline__ float exp2_t(float x) {
+  if constexpr (sizeof(T) == 4) return exp2f(x);
+  else return fast_exp2(x);
+}
+template <typename T>
+__device__ __forceinline__ float gate_of(const RaggedAttn& p, int row, int h) {
+  if (p.gate == nullptr) return 1.f;
+  return sigmoidf_(to_f32(static_cast<const T*>(p.gate)[static_cast<size_t>(row) * p.ldg + h]));
+}
+// Softmax denominator with the sink, in units of 2^m.
+template <typename T>
+__device__ __forceinline__ float denom(const RaggedAttn& p, int h, float m, float l) {
+  return p.sink != nullptr ? l + exp2_t<T>(p.sink[h] * LOG2E - m) : l;
+}
+
+// ------------------------------------------------------------------------------ rows kernel
+constexpr int RA_WARPS = 4;
+
+struct RowsArgs {
+  RaggedAttn a;
+  const int* rows;         // [n] query rows, or null: row i
+  const int* row_slot;     // [rows of the batch]
+  const int* row_pos;
+  int splits;
+  float* part_o;           // [n, heads, splits, vdim]
+  float* part_ml;          // [n, heads, splits, 2]
+};
+
+template <typename T, int KIT, int GM>    // dim <= 64 KIT, GM query heads at a time
+__global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const RowsArgs ra) {
+  const RaggedAttn& p = ra.a;
+  constexpr int DC = 64 * KIT;
+  __shared__ __align__(16) float sq[GM][DC];
+  __shared__ __align__(16) float sp[RA_WARPS][32][GM];     // scores, then weights, [key][head]
+  __shared__ float sm_m[RA_WARPS][GM], sm_l[RA_WARPS][GM];
+  __shared__ __align__(16) float red[RA_WARPS * 32 * 8];
+  const int i = blockIdx.x, split = blockIdx.z;
+  const int per = p.heads / p.kv_heads, subs = (per + GM - 1) / GM;
+  const int hk = blockIdx.y / subs, h0 = hk * per + (blockIdx.y % subs) * GM;
+  const int ng = min(GM, (hk + 1) * per - h0);
+  const int row = ra.rows != nullptr ? ra.rows[i] : i;
+  const int slot = ra.row_slot[row], pos = ra.row_pos[row];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
+  const T* qp = static_cast<const T*>(p.q) + static_cast<size_t>(row) * p.heads * p.dim;
+  for (int j = threadIdx.x; j < GM * DC; j += RA_WARPS * 32) {
+    const int g = j / DC, d = j % DC;
+    sq[g][d] = (g < ng && d < p.dim) ? to_f32(qp[(h0 + g) * p.dim + d]) * (p.scale * LOG2E) : 0.f;
+  }
+  __syncthreads();
+  const int lo = chunk_start(pos, p.chunk), n = pos + 1 - lo;
+  const int piece = (n + ra.splits - 1) / ra.splits;
+  const int t0 = lo + split * piece, t1 = min(pos + 1, t0 + piece);
+  const T* kc = static_cast<const T*>(p.k_cache);
+  const T* vc = static_cast<const T*>(p.v_cache);
+  const int nchunk = p.vdim_p / 8, ngroups = 32 / nchunk;
+  const int kg = lane / nchunk, vch = lane % nchunk;
+  float m[GM], l[GM], acc[GM][8];
+#pragma unroll
+  for (int g = 0; g < GM; ++g) {
+    m[g] = -INFINITY;
+    l[g] = 0.f;
+#pragma unroll
+    for (int x = 0; x < 8; ++x) acc[g][x] = 0.f;
+  }
+  for (int tb = t0 + warp * 32; tb < t1; tb += RA_WARPS * 32) {
+    // scores of 32 keys: eight lanes per key, four keys at a time
+    const int my_t = tb + lane;
+    int my_page = 0;
+    if (my_t < t1) {
+      const int lp = my_t / RAGGED_PAGE;
+      my_page = lp < p.max_pages ? pt[lp] : -1;
+      if (my_page < 0 || my_page >= p.num_pages) {
+        record_status(p.status, ST_BOUNDS, row);
+        my_page = 0;
+      }
+    }
+#pragma unroll 4
+    for (int r = 0; r < 8; ++r) {
+      const int key = r * 4 + (lane >> 3), t = tb + key;
+      const int page = __shfl_sync(0xffffffffu, my_page, key);
+      float s[GM];
+#pragma unroll
+      for (int g = 0; g < GM; ++g) s[g] = 0.f;
+      if (t < t1) {
+        const T* kp = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + t % RAGGED_PAGE) * p.kv_heads + hk) * p.dim_p;
+#pragma unroll
+        for (int c = 0; c < KIT; ++c) {
+          const int d = ((lane & 7) + 8 * c) * 8;
+          if (d < p.dim_p) {
+            float f[8];
+            load_vec<8>(kp + d, f);
+#pragma unroll
+            for (int g = 0; g < GM; ++g) {
+              const float4 a = *reinterpret_cast<const float4*>(&sq[g][d]);
+              const float4 b = *reinterpret_cast<const float4*>(&sq[g][d + 4]);
+              s[g] += f[0] * a.x + f[1] * a.y + f[2] * a.z + f[3] * a.w + f[4] * b.x + f[5] * b.y +
+                      f[6] * b.z + f[7] * b.w;
+            }
+          }
+        }
+      }
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+        for (int g = 0; g < GM; ++g) s[g] += __shfl_xor_sync(0xffffffffu, s[g], o);
+#pragma unroll
+      for (int g = 0; g < GM; ++g)
+        if ((lane & 7) == (g & 7)) sp[warp][key][g] = s[g];
+    }
+    __syncwarp();
+    // weights: one key per lane
+#pragma unroll
+    for (int g = 0; g < GM; ++g) {
+      const float s = my_t < t1 ? sp[warp][lane][g] : -INFINITY;
+      const float mn = fmaxf(m[g], warp_max(s));          // finite: the block has a key
+      const float c = exp2_t<T>(m[g] - mn), w = exp2_t<T>(s - mn);
+      m[g] = mn;
+      l[g] = l[g] * c + warp_sum(w);
+#pragma unroll
+      for (int x = 0; x < 8; ++x) acc[g][x] *= c;
+      sp[warp][lane][g] = w;
+    }
+    __syncwarp();
+    // weighted values: lane (kg, vch) takes every ngroups-th key and eight value channels
+    const int nk = min(32, t1 - tb);
+#pragma unroll 4
+    for (int k0 = 0; k0 < nk; k0 += ngroups) {
+      const int key = k0 + kg, t = tb + key;
+      const int page = __shfl_sync(0xffffffffu, my_page, key & 31);
+      if (kg < ngroups && key < nk) {
+        const T* vp = vc + ((static_cast<size_t>(page) * RAGGED_PAGE + t % RAGGED_PAGE) * p.kv_heads + hk) * p.vdim_p;
+        float f[8];
+        load_vec<8>(vp + vch * 8, f);
+#pragma unroll
+        for (int g = 0; g < GM; ++g) {
+          const float w = sp[warp][key][g];
+#pragma unroll
+          for (int x = 0; x < 8; ++x) acc[g][x] += w * f[x];
+        }
+      }
+    }
+    __syncwarp();
+  }
+#pragma unroll
+  for (int g = 0; g < GM; ++g)
+    if (lane == 0) {
+      sm_m[warp][g] = m[g];
+      sm_l[warp][g] = l[g];
+    }
+  __syncthreads();
+  // merge the warps and their key groups, one query head after the other
+  const int parts = ngroups * RA_WARPS;
+#pragma unroll
+  for (int g = 0; g < GM; ++g) {
+    if (g >= ng) break;
+    float gm = -INFINITY, gl = 0.f;
+#pragma unroll
+    for (int w = 0; w < RA_WARPS; ++w) gm = fmaxf(gm, sm_m[w][g]);
+#pragma unroll
+    for (int w = 0; w < RA_WARPS; ++w)
+      gl += sm_m[w][g] == -INFINITY ? 0.f : sm_l[w][g] * exp2_t<T>(sm_m[w][g] - gm);
+    const float c = m[g] == -INFINITY ? 0.f : exp2_t<T>(m[g] - gm);
+    if (kg < ngroups) {
+#pragma unroll
+      for (int x = 0; x < 8; ++x)
+        red[(warp * ngroups + kg) * p.vdim_p + vch * 8 + x] = acc[g][x] * c;
+    }
+    __syncthreads();
+    const int h = h0 + g;
+    const float dn = ra.splits == 1 ? gate_of<T>(p, row, h) / denom<T>(p, h, gm, gl) : 1.f;
+    for (int d = threadIdx.x; d < p.vdim; d += RA_WARPS * 32) {
+      float o = 0.f;
+      for (int w = 0; w < parts; ++w) o += red[w * p.vdim_p + d];
+      if (ra.splits == 1)
+        static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] = from_f32<T>(o * dn);
+      else
+        ra.part_o[((static_cast<size_t>(i) * p.heads + h) * ra.splits + split) * p.vdim + d] = o;
+    }
+    if (ra.splits > 1 && threadIdx.x == 0) {
+      float* ml = ra.part_ml + ((static_cast<size_t>(i) * p.heads + h) * ra.splits + split) * 2;
+      ml[0] = gm;
+      ml[1] = gl;
+    }
+    __syncthreads();
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(64) ragged_attn_merge_kernel(const RowsArgs ra) {
+  const RaggedAttn& p = ra.a;
+  const int i = blockIdx.x, h = blockIdx.y;
+  const int row = ra.rows != nullptr ? ra.rows[i] : i;
+  const size_t base = (static_cast<size_t>(i) * p.heads + h) * ra.splits;
+  float gm = -INFINITY, gl = 0.f;
+  for (int s = 0; s < ra.splits; ++s) gm = fmaxf(gm, ra.part_ml[(base + s) * 2]);
+  for (int s = 0; s < ra.splits; ++s) {
+    const float ms = ra.part_ml[(base + s) * 2];
+    gl += ms == -INFINITY ? 0.f : ra.part_ml[(base + s) * 2 + 1] * exp2_t<T>(ms - gm);
+  }
+  const float dn = gate_of<T>(p, row, h) / denom<T>(p, h, gm, gl);
+  for (int d = threadIdx.x; d < p.vdim; d += 64) {
+    float o = 0.f;
+    for (int s = 0; s < ra.splits; ++s) {
+      const float ms = ra.part_ml[(base + s) * 2];
+      if (ms != -INFINITY) o += ra.part_o[(base + s) * p.vdim + d] * exp2_t<T>(ms - gm);
+    }
+    static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] = from_f32<T>(o * dn);
+  }
+}
+
+// ------------------------------------------------------------------------------ tiles kernel
+constexpr int TA_WARPS = 4;
+constexpr int TA_ROWS = 16 * TA_WARPS;
+
+__device__ __forceinline__ void ldsm4(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, "
+               "{%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+struct TilesArgs {
+  RaggedAttn a;
+  Entries e;
+  const int* tile_entry;   // [tiles]
+  const int* tile_off;     // [tiles] first token of the tile inside its entry
+};
+
+template <int DC, int VC>   // dim <= DC, vdim <= VC, multiples of 32
+__global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const TilesArgs ta) {
+  using bf16 = __nv_bfloat16;
+  const RaggedAttn& p = ta.a;
+  constexpr int KS = DC + 8, VS = VC + 8;       // padded rows (elements): conflict-free ldmatrix
+  extern __shared__ __align__(16) unsigned char smem[];
+  bf16* sK = reinterpret_cast<bf16*>(smem);                      // [2][PAGE][KS]
+  bf16* sV = sK + 2 * RAGGED_PAGE * KS;                          // [2][PAGE][VS]
+  bf16* sQ = sV + 2 * RAGGED_PAGE * VS;                          // [TA_ROWS][KS]
+  const int e = ta.tile_entry[blockIdx.x], off = ta.tile_off[blockIdx.x], h = blockIdx.y;
+  const int hk = h / (p.heads / p.kv_heads);
+  const int row0 = ta.e.row0[e] + off, len = min(TA_ROWS, ta.e.len[e] - off);
+  const int pos0 = ta.e.pos0[e] + off, slot = ta.e.slot[e];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
+  const bf16* q = static_cast<const bf16*>(p.q);
+  const bf16* kc = static_cast<const bf16*>(p.k_cache);
+  const bf16* vc = static_cast<const bf16*>(p.v_cache);
+  // padding columns of the rings are zero once and for all
+  for (int i = tid; i < 2 * RAGGED_PAGE * (KS - p.dim_p); i += TA_WARPS * 32)
+    sK[(i / (KS - p.dim_p)) * KS + p.dim_p + i % (KS - p.dim_p)] = __float2bfloat16(0.f);
+  for (int i = tid; i < 2 * RAGGED_PAGE * (VS - p.vdim_p); i += TA_WARPS * 32)
+    sV[(i / (VS - p.vdim_p)) * VS + p.vdim_p + i % (VS - p.vdim_p)] = __float2bfloat16(0.f);
+  const int last = pos0 + len - 1;
+  const int pg0 = chunk_start(pos0, p.chunk) / RAGGED_PAGE, pg1 = last / RAGGED_PAGE;
+  auto fetch = [&](int pg, int st) {
+    int page = pg < p.max_pages ? pt[pg] : -1;
+    if (page < 0 || page >= p.num_pages) {
+      if (tid == 0) record_status(p.status, ST_BOUNDS, row0);
+      page = 0;
+    }
+    const int base = pg * RAGGED_PAGE;
+    const int kch = p.dim_p / 8, vch = p.vdim_p / 8;
+    for (int i = tid; i < RAGGED_PAGE * kch; i += TA_WARPS * 32) {
+      const int t = i / kch, c = i % kch;
+      const bf16* src = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + t) * p.kv_heads + hk) * p.dim_p + c * 8;
+      cp_async16_zfill(smem_u32(sK + (st * RAGGED_PAGE + t) * KS + c * 8), src, base + t <= last ? 16 : 0);
+    }
+    for (int i = tid; i < RAGGED_PAGE * vch; i += TA_WARPS * 32) {
+      const int t = i / vch, c = i % vch;
+      const bf16* src = vc + ((static_cast<size_t>(page) * RAGGED_PAGE + t) * p.kv_heads + hk) * p.vdim_p + c * 8;
+      cp_async16_zfill(smem_u32(sV + (st * RAGGED_PAGE + t) * VS + c * 8), src, base + t <= last ? 16 : 0);
+    }
+    cp_async_commit();
+  };
+  fetch(pg0, 0);
+  if (p.dim % 8 == 0) {
+    for (int i = tid; i < TA_ROWS * (DC / 8); i += TA_WARPS * 32) {
+      const int t = i / (DC / 8), c = (i % (DC / 8)) * 8;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (t < len && c < p.dim)
+        v = *reinterpret_cast<const uint4*>(q + (static_cast<size_t>(row0 + t) * p.heads + h) * p.dim + c);
+      *reinterpret_cast<uint4*>(sQ + t * KS + c) = v;
+    }
+  } else {
+    for (int i = tid; i < TA_ROWS * DC; i += TA_WARPS * 32) {
+      const int t = i / DC, c = i % DC;
+      sQ[t * KS + c] = (t < len && c < p.dim)
+                           ? q[(static_cast<size_t>(row0 + t) * p.heads + h) * p.dim + c]
+                           : __float2bfloat16(0.f);
+    }
+  }
+  __syncthreads();
+  uint32_t qf[DC / 16][4];
+#pragma unroll
+  for (int k = 0; k < DC / 16; ++k)
+    ldsm4(qf[k], smem_u32(sQ + (warp * 16 + (lane & 15)) * KS + k * 16 + (lane >> 4) * 8));
+  float o[VC / 8][4];
+#pragma unroll
+  for (int i = 0; i < VC / 8; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const int r0 = warp * 16 + (lane >> 2);
+  const int qpos[2] = {pos0 + r0, pos0 + r0 + 8};
+  const int qlo[2] = {chunk_start(qpos[0], p.chunk), chunk_start(qpos[1], p.chunk)};
+  const float sl2 = p.scale * LOG2E;
+  const int w_first = pos0 + warp * 16, w_last = min(w_first + 15, last);
+  for (int pg = pg0; pg <= pg1; ++pg) {
+    const int st = (pg - pg0) & 1, base = pg * RAGGED_PAGE;
+    if (pg < pg1) {
+      fetch(pg + 1, st ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    // skip pages that no row of this warp sees
+    if (w_first <= last && base <= w_last && base + RAGGED_PAGE > chunk_start(w_first, p.chunk)) {
+      float s[8][4];
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+      const bf16* kb = sK + st * RAGGED_PAGE * KS;
+#pragma unroll
+      for (int k = 0; k < DC / 16; ++k) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {       // 16 keys: two n-tiles
+          uint32_t b[4];
+          ldsm4(b, smem_u32(kb + (i * 16 + (lane & 7) + (lane >> 4) * 8) * KS + k * 16 + ((lane >> 3) & 1) * 8));
+          mma_bf16(s[2 * i], qf[k], b[0], b[1]);
+          mma_bf16(s[2 * i + 1], qf[k], b[2], b[3]);
+        }
+      }
+      const bool full = base >= chunk_start(w_last, p.chunk) && base + RAGGED_PAGE - 1 <= w_first;
+      float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int r = j >> 1, t = base + i * 8 + (lane & 3) * 2 + (j & 1);
+          s[i][j] = (full || (t <= qpos[r] && t >= qlo[r])) ? s[i][j] * sl2 : -INFINITY;
+          mx[r] = fmaxf(mx[r], s[i][j]);
+        }
+      float c[2], sum[2] = {0.f, 0.f};
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+        const float mn = fmaxf(m[r], mx[r]);
+        c[r] = m[r] == -INFINITY ? 0.f : fast_exp2(m[r] - mn);
+        m[r] = mn;
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int r = j >> 1;
+          s[i][j] = s[i][j] == -INFINITY ? 0.f : fast_exp2(s[i][j] - m[r]);
+          sum[r] += s[i][j];
+        }
+      l[0] = l[0] * c[0] + sum[0];          // this lane's keys; the lanes are added at the end
+      l[1] = l[1] * c[1] + sum[1];
+#pragma unroll
+      for (int i = 0; i < VC / 8; ++i) {
+        o[i][0] *= c[0];
+        o[i][1] *= c[0];
+        o[i][2] *= c[1];
+        o[i][3] *= c[1];
+      }
+      const bf16* vb = sV + st * RAGGED_PAGE * VS;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {         // 16 keys
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const float u = s[2 * k + (x >> 1)][(x & 1) * 2], w = s[2 * k + (x >> 1)][(x & 1) * 2 + 1];
+          ph[x] = pack_bf16x2(u, w);
+          const float2 b = unpack_bf16x2(ph[x]);
+          pl[x] = pack_bf16x2(u - b.x, w - b.y);
+        }
+#pragma unroll
+        for (int i = 0; i < VC / 16; ++i) {
+          uint32_t b[4];
+          ldsm4_t(b, smem_u32(vb + (k * 16 + (lane & 15)) * VS + i * 16 + (lane >> 4) * 8));
+          mma_bf16(o[2 * i], ph, b[0], b[1]);
+          mma_bf16(o[2 * i + 1], ph, b[2], b[3]);
+          mma_bf16(o[2 * i], pl, b[0], b[1]);
+          mma_bf16(o[2 * i + 1], pl, b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+    const int t = r0 + r * 8;
+    if (t >= len) continue;
+    const int row = row0 + t;
+    const float dn = gate_of<bf16>(p, row, h) / denom<bf16>(p, h, m[r], l[r]);
+    bf16* dst = static_cast<bf16*>(p.out) + static_cast<size_t>(row) * p.ldo + h * p.vdim;
+    const bool pairs = (p.vdim & 1) == 0 && (p.ldo & 1) == 0;
+#pragma unroll
+    for (int i = 0; i < VC / 8; ++i) {
+      const int d = i * 8 + (lane & 3) * 2;
+      const float u = o[i][r * 2] * dn, w = o[i][r * 2 + 1] * dn;
+      if (pairs) {
+        if (d < p.vdim) *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(u, w);
+      } else {
+        if (d < p.vdim) dst[d] = __float2bfloat16(u);
+        if (d + 1 < p.vdim) dst[d + 1] = __float2bfloat16(w);
+      }
+    }
+  }
+}
+
+template <int DC, int VC>
+static int launch_tiles(const TilesArgs& a, int tiles, cudaStream_t st) {
+  const int smem = (2 * RAGGED_PAGE * (DC + 8) + 2 * RAGGED_PAGE * (VC + 8) + TA_ROWS * (DC + 8)) * 2;
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(ragged_attn_tiles_kernel<DC, VC>,
+                             cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      return -4;
+    set = true;
+  }
+  dim3 grid(tiles, a.a.heads);
+  ragged_attn_tiles_kernel<DC, VC><<<grid, TA_WARPS * 32, smem, st>>>(a);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+template <int DC>
+static int launch_tiles_v(const TilesArgs& a, int tiles, cudaStream_t st) {
+  if (a.a.vdim <= 64) return launch_tiles<DC, 64>(a, tiles, st);
+  if (a.a.vdim <= 128) return launch_tiles<DC, 128>(a, tiles, st);
+  return launch_tiles<DC, 256>(a, tiles, st);
+}
+
+template <typename T, int KIT>
+static int launch_rows(const RowsArgs& a, int n, cudaStream_t st) {
+  const int per = a.a.heads / a.a.kv_heads;
+#define CB_ROWS(GM_)                                                                         \
+  do {                                                                                       \
+    dim3 grid(n, a.a.kv_heads * ((per + GM_ - 1) / GM_), a.splits);                          \
+    ragged_attn_rows_kernel<T, KIT, GM_><<<grid, RA_WARPS * 32, 0, st>>>(a);                 \
+  } while (0)
+  if (per == 1) CB_ROWS(1);
+  else if (per == 2) CB_ROWS(2);
+  else if (per <= 4) CB_ROWS(4);
+  else CB_ROWS(8);
+#undef CB_ROWS
+  if (a.splits > 1) {
+    dim3 g2(n, a.a.heads);
+    ragged_attn_merge_kernel<T><<<g2, 64, 0, st>>>(a);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+template <typename T>
+static int launch_rows_d(const RowsArgs& a, int n, cudaStream_t st) {
+  if (a.a.dim <= 64) return launch_rows<T, 1>(a, n, st);
+  if (a.a.dim <= 128) return launch_rows<T, 2>(a, n, st);
+  return launch_rows<T, 4>(a, n, st);
+}
+
+}  // namespace cb
+
+using namespace cb;
+
+static int fill_attn(RaggedAttn& p, const void* q, const void* k_cache, const void* v_cache,
+                     const int* page_table, int max_pages, int num_pages, int heads, int kv_heads,
+                     int dim, int vdim, int dim_p, int vdim_p, int chunk, float scale,
+                     const float* sink, const void* gate, int ldg, void* out, int ldo, int* status) {
+  if (kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || dim > 256 || vdim > 256) return -1;
+  if (dim_p % 8 != 0 || vdim_p % 8 != 0 || dim_p < dim || vdim_p < vdim || dim_p > 256 || vdim_p > 256)
+    return -2;
+  p.q = q; p.k_cache = k_cache; p.v_cache = v_cache; p.page_table = page_table;
+  p.max_pages = max_pages; p.num_pages = num_pages; p.heads = heads; p.kv_heads = kv_heads;
+  p.dim = dim; p.vdim = vdim; p.dim_p = dim_p; p.vdim_p = vdim_p; p.chunk = chunk; p.scale = scale;
+  p.sink = sink; p.gate = gate; p.ldg = ldg; p.out = out; p.ldo = ldo; p.status = status;
+  return 0;
+}
+
+extern "C" int cb_ragged_attn_tile() { return TA_ROWS; }
+
+extern "C" int cb_ragged_attn_rows(const void* q, const void* k_cache, const void* v_cache,
+                                   const int* page_table, int max_pages, int num_pages, int heads,
+                                   int kv_heads, int dim, int vdim, int dim_p, int vdim_p, int chunk,
+                                   float scale, const float* sink, const void* gate, int ldg,
+                                   void* out, int ldo, const int* rows, const int* row_slot,
+                                   const int* row_pos, int n, int splits, float* part_o,
+                                   float* part_ml, int f32, int* status, void* stream) {
+  RowsArgs a;
+  const int rc = fill_attn(a.a, q, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
+                           dim, vdim, dim_p, vdim_p, chunk, scale, sink, gate, ldg, out, ldo, status);
+  if (rc != 0) return rc;
+  if (n <= 0 || splits < 1 || (splits > 1 && (part_o == nullptr || part_ml == nullptr))) return -5;
+  a.rows = rows; a.row_slot = row_slot; a.row_pos = row_pos; a.splits = splits;
+  a.part_o = part_o; a.part_ml = part_ml;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return f32 ? launch_rows_d<float>(a, n, st) : launch_rows_d<__nv_bfloat16>(a, n, st);
+}
+
+extern "C" int cb_ragged_attn_tiles(const void* q, const void* k_cache, const void* v_cache,
+                                    const int* page_table, int max_pages, int num_pages, int heads,
+                                    int kv_heads, int dim, int vdim, int dim_p, int vdim_p, int chunk,
+                                    float scale, const float* sink, const void* gate, int ldg,
+                                    void* out, int ldo, const int* slot, const int* row0,
+                                    const int* len, const int* pos0, const int* tile_entry,
+                                    const int* tile_off, int tiles, int* status, void* stream) {
+  TilesArgs a;
+  const int rc = fill_attn(a.a, q, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
+                           dim, vdim, dim_p, vdim_p, chunk, scale, sink, gate, ldg, out, ldo, status);
+  if (rc != 0) return rc;
+  if (tiles <= 0) return -5;
+  a.e.slot = slot; a.e.row0 = row0; a.e.len = len; a.e.pos0 = pos0;
+  a.tile_entry = tile_entry; a.tile_off = tile_off;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dim <= 64) return launch_tiles_v<64>(a, tiles, st);
+  if (dim <= 128) return launch_tiles_v<128>(a, tiles, st);
+  return launch_tiles_v<256>(a, tiles, st);
+}

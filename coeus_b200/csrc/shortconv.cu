@@ -1,0 +1,348 @@
+// Short causal convolutions over time in front of a mixer, for a ragged batch, together with what
+// follows them element by element:
+//   shortconv_attn   q, k, v of an attention layer: convolution, rotary embedding of q and k,
+//                    value mixing, and the write of k and v into the cache pages
+//   shortconv_delta  q, k, v of a gated delta layer: convolution, SiLU, unit norm of q and k,
+//                    the decay of every key channel and the step size
+// The convolution of a channel with n taps needs the n - 1 projected values before the current
+// one.  Inside a step they are earlier rows of the projection; at the start of an entry they come
+// from the slot's state, [n - 1, channels] projected values in time order.  The block that owns
+// an entry's first tile is the only one that reads the state, so it alone replaces it, after its
+// last read.
+#include "ragged.cuh"
+
+namespace cb {
+
+constexpr int CONV_TILE = 16;      // tokens per block
+constexpr int CONV_THREADS = 128;
+
+struct ConvIn {
+  const void* raw;        // [rows, ld] projections: q at column 0, k at koff, v at voff
+  int ld, koff, voff;
+  const float* taps_w;    // [taps, channels], channels = q | k | v without gaps
+  int taps;
+  void* state;            // [slots, taps - 1, channels] in the activation type
+  int heads, kv_heads, dim, vdim;
+  Entries e;
+  const int* tile_entry;  // [tiles]
+  const int* tile_off;    // [tiles] first token of the tile inside its entry
+};
+
+// Column of channel c (q | k | v numbering) in the projection buffer.
+__device__ __forceinline__ int raw_col(const ConvIn& p, int c) {
+  const int qc = p.heads * p.dim, kc = p.kv_heads * p.dim;
+  return c < qc ? c : (c < qc + kc ? p.koff + (c - qc) : p.voff + (c - qc - kc));
+}
+// The delta layer has kv_heads query heads.
+__device__ __forceinline__ int raw_col_delta(const ConvIn& p, int c) {
+  const int qc = p.kv_heads * p.dim;
+  return c < qc ? c : (c < 2 * qc ? p.koff + (c - qc) : p.voff + (c - 2 * qc));
+}
+
+// V consecutive channels from c (columns from col) of the token at offset t of the entry.
+template <typename T, int V>
+__device__ __forceinline__ void conv_at(const ConvIn& p, int c, int col, int channels, int row0,
+                                        int t, int slot, bool has_state, float* y) {
+#pragma unroll
+  for (int i = 0; i < V; ++i) y[i] = 0.f;
+  const T* raw = static_cast<const T*>(p.raw);
+  const T* st = static_cast<const T*>(p.state);
+  const int n1 = p.taps - 1;
+  for (int j = 0; j <= n1; ++j) {
+    const int o = t - n1 + j;
+    float u[V], w[V];
+    if (o >= 0) {
+      load_vec<V>(raw + static_cast<size_t>(row0 + o) * p.ld + col, u);
+    } else {
+      if (!has_state) continue;
+      load_vec<V>(st + (static_cast<size_t>(slot) * n1 + (n1 + o)) * channels + c, u);
+    }
+    load_vec<V>(p.taps_w + static_cast<size_t>(j) * channels + c, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[i] += u[i] * w[i];
+  }
+}
+
+// The state of channel c after the entry's len tokens.
+template <typename T>
+__device__ __forceinline__ void conv_advance(const ConvIn& p, int c, int col, int channels,
+                                             int row0, int len, int slot, bool has_state) {
+  const int n1 = p.taps - 1;
+  const T* raw = static_cast<const T*>(p.raw);
+  T* st = static_cast<T*>(p.state) + static_cast<size_t>(slot) * n1 * channels + c;
+  for (int j = 0; j < n1; ++j) {          // ascending: st[j + len] is read before it is replaced
+    const int o = len - n1 + j;
+    T v;
+    if (o >= 0) v = raw[static_cast<size_t>(row0 + o) * p.ld + col];
+    else v = has_state ? st[static_cast<size_t>(n1 + o) * channels] : from_f32<T>(0.f);
+    st[static_cast<size_t>(j) * channels] = v;
+  }
+}
+
+struct AttnPre {
+  ConvIn c;
+  int half;                // rotated pairs per head (0: no rotation)
+  const float2* rope;      // [rows, half] (cos, sin)
+  void* q;                 // out [rows, heads * dim]
+  void* k_cache;           // [pages, PAGE, kv_heads, dim_p]
+  void* v_cache;           // [pages, PAGE, kv_heads, vdim_p]
+  int dim_p, vdim_p;
+  const int* page_table;   // [slots, max_pages]
+  int max_pages, num_pages;
+  void* v_first;           // [rows, kv_heads * vdim]: written when mix_mode = 1, read when 2
+  const float* lambda;
+  int mix_mode;
+  int* status;
+};
+
+// grid (tiles, kv_heads): the block's channels are its key/value head and the query heads on it.
+template <typename T, int V>
+__global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const AttnPre p) {
+  const ConvIn& ci = p.c;
+  const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
+  const int row0 = ci.e.row0[e], len = ci.e.len[e], pos0 = ci.e.pos0[e], slot = ci.e.slot[e];
+  const bool has_state = pos0 > 0;
+  const int per = ci.heads / ci.kv_heads, dim = ci.dim, vdim = ci.vdim;
+  const int qc = ci.heads * dim, kc = ci.kv_heads * dim;
+  const int channels = qc + kc + ci.kv_heads * vdim;
+  const int nt = min(CONV_TILE, len - off);
+  // per head: half / V units that make two rotated vectors, then plain units
+  const int pair_u = p.half / V, plain_u = (dim - 2 * p.half) / V, head_u = pair_u + plain_u;
+  const int v_u = vdim / V, units = (per + 1) * head_u + v_u;
+  const float lam = p.mix_mode == 2 ? *p.lambda : 0.f;
+  for (int i = threadIdx.x; i < nt * units; i += CONV_THREADS) {
+    const int t = off + i / units, u = i % units, row = row0 + t, pos = pos0 + t;
+    const int lp = pos / RAGGED_PAGE;
+    const bool in_table = lp < p.max_pages;
+    const int page = in_table ? p.page_table[static_cast<size_t>(slot) * p.max_pages + lp] : -1;
+    if (page < 0 || page >= p.num_pages) {
+      record_status(p.status, ST_BOUNDS, row);
+      continue;
+    }
+    const size_t cell = (static_cast<size_t>(page) * RAGGED_PAGE + pos % RAGGED_PAGE) * ci.kv_heads + g;
+    if (u < (per + 1) * head_u) {
+      const int hi = u / head_u, k = u % head_u;       // hi < per: query head, else the key head
+      const bool is_q = hi < per;
+      const int base = is_q ? (g * per + hi) * dim : qc + g * dim;
+      const int colb = is_q ? base : ci.koff + g * dim;
+      T* dst = is_q ? static_cast<T*>(p.q) + static_cast<size_t>(row) * qc + base
+                    : static_cast<T*>(p.k_cache) + cell * p.dim_p;
+      if (k < pair_u) {
+        const int d = k * V;
+        float a[V], b[V], oa[V], ob[V];
+        conv_at<T, V>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
+        conv_at<T, V>(ci, base + p.half + d, colb + p.half + d, channels, row0, t, slot, has_state, b);
+#pragma unroll
+        for (int x = 0; x < V; ++x) {
+          const float2 cs = p.rope[static_cast<size_t>(row) * p.half + d + x];
+          oa[x] = a[x] * cs.x - b[x] * cs.y;
+          ob[x] = b[x] * cs.x + a[x] * cs.y;
+        }
+        store_vec<V>(dst + d, oa);
+        store_vec<V>(dst + p.half + d, ob);
+      } else {
+        const int d = 2 * p.half + (k - pair_u) * V;
+        float a[V];
+        conv_at<T, V>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
+        store_vec<V>(dst + d, a);
+      }
+    } else {
+      const int d = (u - (per + 1) * head_u) * V;
+      float a[V];
+      conv_at<T, V>(ci, qc + kc + g * vdim + d, ci.voff + g * vdim + d, channels, row0, t, slot,
+                    has_state, a);
+      if (p.mix_mode != 0) {
+        T* vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d;
+        if (p.mix_mode == 1) {
+          store_vec<V>(vf, a);
+        } else {
+          float f[V];
+          load_vec<V>(vf, f);
+#pragma unroll
+          for (int x = 0; x < V; ++x) a[x] = (1.f - lam) * a[x] + lam * f[x];
+        }
+      }
+      store_vec<V>(static_cast<T*>(p.v_cache) + cell * p.vdim_p + d, a);
+    }
+  }
+  if (off == 0 && ci.taps > 1) {
+    __syncthreads();
+    const int mine = (per + 1) * dim + vdim;
+    for (int i = threadIdx.x; i < mine; i += CONV_THREADS) {
+      const int c = i < per * dim ? g * per * dim + i
+                  : (i < (per + 1) * dim ? qc + g * dim + (i - per * dim)
+                                         : qc + kc + g * vdim + (i - (per + 1) * dim));
+      conv_advance<T>(ci, c, raw_col(ci, c), channels, row0, len, slot, has_state);
+    }
+  }
+}
+
+struct DeltaPre {
+  ConvIn c;                // heads value heads, kv_heads query/key heads
+  int boff;                // column of the step-size projection in raw
+  const float* a;          // [rows, heads * dim] decay projection, fp32
+  int lda;
+  const float* A_log;      // [heads]
+  const float* dt_bias;    // [heads * dim]
+  float* q;                // out [rows, kv_heads, dim4] unit norm, scaled by dim^-1/2
+  float* k;                // out [rows, kv_heads, dim4] unit norm
+  float* kq;               // out [rows, kv_heads] their dot product
+  float* v;                // out [rows, heads, vdim]
+  float* g;                // out [rows, heads, dim4] decay factors
+  float* beta;             // out [rows, heads]
+  int dim4;                // dim rounded up to a multiple of 4; the padding is zero
+};
+
+__device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus_exact(float x) {
+  return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+}
+
+// grid (tiles, kv_heads): one query/key head and the value heads on it.
+template <typename T>
+__global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_kernel(const DeltaPre p) {
+  const ConvIn& ci = p.c;
+  const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
+  const int row0 = ci.e.row0[e], len = ci.e.len[e], slot = ci.e.slot[e];
+  const bool has_state = ci.e.pos0[e] > 0;
+  const int per = ci.heads / ci.kv_heads, dim = ci.dim, vdim = ci.vdim;
+  const int qc = ci.kv_heads * dim;
+  const int channels = 2 * qc + ci.heads * vdim;
+  const int nt = min(CONV_TILE, len - off);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float qscale = 1.0f / sqrtf(static_cast<float>(dim));
+  // q and k: a warp per token
+  for (int t = off + warp; t < off + nt; t += CONV_THREADS / 32) {
+    constexpr int MAXD = 8;                      // dim <= 256
+    float qv[MAXD], kv[MAXD], sq = 0.f, sk = 0.f, dot = 0.f;
+#pragma unroll
+    for (int i = 0; i < MAXD; ++i) {
+      const int d = lane + 32 * i;
+      qv[i] = kv[i] = 0.f;
+      if (d < dim) {
+        conv_at<T, 1>(ci, g * dim + d, g * dim + d, channels, row0, t, slot, has_state, &qv[i]);
+        conv_at<T, 1>(ci, qc + g * dim + d, ci.koff + g * dim + d, channels, row0, t, slot, has_state, &kv[i]);
+        qv[i] = silu_exact(qv[i]);
+        kv[i] = silu_exact(kv[i]);
+      }
+      sq += qv[i] * qv[i];
+      sk += kv[i] * kv[i];
+    }
+    const float rq = qscale / sqrtf(warp_sum(sq) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f);
+    const size_t cell = static_cast<size_t>(row0 + t) * ci.kv_heads + g;
+#pragma unroll
+    for (int i = 0; i < MAXD; ++i) {
+      const int d = lane + 32 * i;
+      const float a = qv[i] * rq, b = kv[i] * rk;
+      dot += a * b;
+      if (d < p.dim4) {
+        p.q[cell * p.dim4 + d] = a;
+        p.k[cell * p.dim4 + d] = b;
+      }
+    }
+    dot = warp_sum(dot);
+    if (lane == 0) p.kq[cell] = dot;
+  }
+  const T* raw = static_cast<const T*>(ci.raw);
+  for (int i = threadIdx.x; i < nt * per * vdim; i += CONV_THREADS) {
+    const int t = off + i / (per * vdim), c = g * per * vdim + i % (per * vdim);
+    float y;
+    conv_at<T, 1>(ci, 2 * qc + c, ci.voff + c, channels, row0, t, slot, has_state, &y);
+    p.v[static_cast<size_t>(row0 + t) * ci.heads * vdim + c] = silu_exact(y);
+  }
+  for (int i = threadIdx.x; i < nt * per * p.dim4; i += CONV_THREADS) {
+    const int t = off + i / (per * p.dim4), x = i % (per * p.dim4);
+    const int h = g * per + x / p.dim4, d = x % p.dim4;
+    float f = 0.f;
+    if (d < dim) {
+      const float a = p.a[static_cast<size_t>(row0 + t) * p.lda + h * dim + d] + p.dt_bias[h * dim + d];
+      f = expf(-expf(p.A_log[h]) * softplus_exact(a));
+    }
+    p.g[(static_cast<size_t>(row0 + t) * ci.heads + h) * p.dim4 + d] = f;
+  }
+  for (int i = threadIdx.x; i < nt * per; i += CONV_THREADS) {
+    const int row = row0 + off + i / per, h = g * per + i % per;
+    p.beta[static_cast<size_t>(row) * ci.heads + h] =
+        sigmoidf_(to_f32(raw[static_cast<size_t>(row) * ci.ld + p.boff + h]));
+  }
+  if (off == 0 && ci.taps > 1) {
+    __syncthreads();
+    const int mine = 2 * dim + per * vdim;
+    for (int i = threadIdx.x; i < mine; i += CONV_THREADS) {
+      const int c = i < dim ? g * dim + i
+                  : (i < 2 * dim ? qc + g * dim + (i - dim) : 2 * qc + g * per * vdim + (i - 2 * dim));
+      conv_advance<T>(ci, c, raw_col_delta(ci, c), channels, row0, len, slot, has_state);
+    }
+  }
+}
+
+}  // namespace cb
+
+using namespace cb;
+
+static ConvIn conv_in(const void* raw, int ld, int koff, int voff, const float* taps_w, int taps,
+                      void* state, int heads, int kv_heads, int dim, int vdim, const int* slot,
+                      const int* row0, const int* len, const int* pos0, const int* tile_entry,
+                      const int* tile_off) {
+  ConvIn c;
+  c.raw = raw; c.ld = ld; c.koff = koff; c.voff = voff; c.taps_w = taps_w; c.taps = taps;
+  c.state = state; c.heads = heads; c.kv_heads = kv_heads; c.dim = dim; c.vdim = vdim;
+  c.e.slot = slot; c.e.row0 = row0; c.e.len = len; c.e.pos0 = pos0;
+  c.tile_entry = tile_entry; c.tile_off = tile_off;
+  return c;
+}
+
+extern "C" int cb_conv_tile() { return CONV_TILE; }
+
+extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, const float* taps_w,
+                                 int taps, void* state, int heads, int kv_heads, int dim, int vdim,
+                                 const int* slot, const int* row0, const int* len, const int* pos0,
+                                 const int* tile_entry, const int* tile_off, int tiles, int half,
+                                 const void* rope, void* q, void* k_cache, void* v_cache, int dim_p,
+                                 int vdim_p, const int* page_table, int max_pages, int num_pages,
+                                 void* v_first, const float* lambda, int mix_mode, int f32,
+                                 int* status, void* stream) {
+  if (tiles <= 0 || taps < 1 || kv_heads < 1 || heads % kv_heads != 0 || 2 * half > dim) return -1;
+  if (mix_mode != 0 && v_first == nullptr) return -2;
+  AttnPre p;
+  p.c = conv_in(raw, ld, koff, voff, taps_w, taps, state, heads, kv_heads, dim, vdim, slot, row0, len,
+                pos0, tile_entry, tile_off);
+  p.half = half; p.rope = static_cast<const float2*>(rope); p.q = q; p.k_cache = k_cache;
+  p.v_cache = v_cache; p.dim_p = dim_p; p.vdim_p = vdim_p; p.page_table = page_table;
+  p.max_pages = max_pages; p.num_pages = num_pages; p.v_first = v_first; p.lambda = lambda;
+  p.mix_mode = mix_mode; p.status = status;
+  const bool vec = dim % 8 == 0 && vdim % 8 == 0 && half % 8 == 0 && ld % 8 == 0 && koff % 8 == 0 &&
+                   voff % 8 == 0;
+  dim3 grid(tiles, kv_heads);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) {
+    if (vec) shortconv_attn_kernel<float, 8><<<grid, CONV_THREADS, 0, st>>>(p);
+    else shortconv_attn_kernel<float, 1><<<grid, CONV_THREADS, 0, st>>>(p);
+  } else {
+    if (vec) shortconv_attn_kernel<__nv_bfloat16, 8><<<grid, CONV_THREADS, 0, st>>>(p);
+    else shortconv_attn_kernel<__nv_bfloat16, 1><<<grid, CONV_THREADS, 0, st>>>(p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, int boff,
+                                  const float* taps_w, int taps, void* state, int heads,
+                                  int kv_heads, int dim, int vdim, const int* slot, const int* row0,
+                                  const int* len, const int* pos0, const int* tile_entry,
+                                  const int* tile_off, int tiles, const float* a, int lda,
+                                  const float* A_log, const float* dt_bias, float* q, float* k,
+                                  float* kq, float* v, float* g, float* beta, int dim4, int f32,
+                                  void* stream) {
+  if (tiles <= 0 || taps < 1 || kv_heads < 1 || heads % kv_heads != 0) return -1;
+  if (dim > 256 || dim4 < dim || dim4 % 4 != 0 || dim4 > dim + 3) return -2;
+  DeltaPre p;
+  p.c = conv_in(raw, ld, koff, voff, taps_w, taps, state, heads, kv_heads, dim, vdim, slot, row0, len,
+                pos0, tile_entry, tile_off);
+  p.boff = boff; p.a = a; p.lda = lda; p.A_log = A_log; p.dt_bias = dt_bias; p.q = q; p.k = k;
+  p.kq = kq; p.v = v; p.g = g; p.beta = beta; p.dim4 = dim4;
+  dim3 grid(tiles, kv_heads);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) shortconv_delta_kernel<float><<<grid, CONV_THREADS, 0, st>>>(p);
+  else shortconv_delta_kernel<__nv_bfloat16><<<grid, CONV_THREADS, 0, st>>>(p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}

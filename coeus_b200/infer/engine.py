@@ -23,7 +23,15 @@ from .kv_cache import PagedKVCache
 from .sampler import select
 
 
+def make_engine(model, **kw) -> "InferenceEngine":
+    """The engine that serves ``model``: its own (``model.make_engine``) or the decoder's."""
+    make = getattr(model, "make_engine", None)
+    return make(**kw) if make is not None else InferenceEngine(model, **kw)
+
+
 class InferenceEngine:
+    ragged = False       # whether step() runs unequal entries as one batch
+
     def __init__(self, model: DecoderLM, max_batch: int = 64, max_len: Optional[int] = None,
                  decode_splits: int = 0, use_graph: Optional[bool] = None) -> None:
         """``use_graph``: capture the decode step in a CUDA graph and replay it per token (default:

@@ -1,9 +1,13 @@
 """Paged KV cache: fixed-size pages of 64 tokens handed out from a free list, one page table row
 per sequence, so the context is bounded by device memory and not by a dense ``[B, S_max]``
-allocation.  One pair of ``[num_pages, 64, heads, dh]`` bf16 tensors per layer."""
+allocation.  One pair of ``[num_pages, 64, heads, dh]`` tensors per layer (bf16 unless the caller
+says otherwise).
+
+:class:`SequenceState` adds what recurrent layers and short convolutions carry from token to
+token: one slot per sequence, addressed like the page-table rows."""
 from __future__ import annotations
 
-from typing import Dict, List
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -13,13 +17,19 @@ from ..ops.decode import PAGE
 
 class PagedKVCache:
     def __init__(self, num_layers: int, num_heads: int, head_dim: int, num_pages: int,
-                 max_seqs: int, max_pages_per_seq: int, device, dtype=torch.bfloat16) -> None:
+                 max_seqs: int, max_pages_per_seq: int, device, dtype=torch.bfloat16,
+                 layer_dims: Optional[Sequence[Tuple[int, int, int]]] = None) -> None:
+        """``layer_dims``: ``(heads, key size, value size)`` of every cached layer where they
+        differ between layers or between keys and values (``num_layers`` entries)."""
         self.num_layers, self.nh, self.dh = num_layers, num_heads, head_dim
         self.num_pages = num_pages
         self.device = torch.device(device)
-        shape = (num_pages, PAGE, num_heads, head_dim)
-        self.k = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
+        dims = list(layer_dims) if layer_dims is not None else \
+            [(num_heads, head_dim, head_dim)] * num_layers
+        self.k = [torch.zeros((num_pages, PAGE, h, dk), dtype=dtype, device=self.device)
+                  for h, dk, _ in dims]
+        self.v = [torch.zeros((num_pages, PAGE, h, dv), dtype=dtype, device=self.device)
+                  for h, _, dv in dims]
         self.page_table = torch.zeros((max_seqs, max_pages_per_seq), dtype=torch.int32,
                                       device=self.device)
         self.free: List[int] = list(range(num_pages - 1, -1, -1))
@@ -91,3 +101,23 @@ class PagedKVCache:
 
     def pages_in_use(self) -> int:
         return self.num_pages - len(self.free)
+
+
+class SequenceState:
+    """Recurrent state of ``slots`` sequences: named tensors per layer with the slot as their
+    first dimension.  A slot needs no clearing when it changes hands: a sequence's first tokens
+    (position 0) are computed from an empty state whatever the slot holds."""
+
+    def __init__(self, slots: int, device) -> None:
+        self.slots, self.device = slots, torch.device(device)
+        self.tensors: Dict[Tuple[int, str], torch.Tensor] = {}
+
+    def add(self, layer: int, name: str, shape: Sequence[int], dtype: torch.dtype) -> None:
+        self.tensors[(layer, name)] = torch.zeros((self.slots, *shape), dtype=dtype,
+                                                  device=self.device)
+
+    def __getitem__(self, key: Tuple[int, str]) -> torch.Tensor:
+        return self.tensors[key]
+
+    def bytes_per_slot(self) -> int:
+        return sum(t[0].numel() * t.element_size() for t in self.tensors.values())

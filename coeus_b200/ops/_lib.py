@@ -13,7 +13,7 @@ from typing import Optional
 
 import torch
 
-from ..build import build_kernels, kernels_lib_path
+from ..build import build_kernels, build_serving, kernels_lib_path
 
 _lock = threading.Lock()
 _lib: Optional[ctypes.CDLL] = None
@@ -38,6 +38,26 @@ def lib() -> ctypes.CDLL:
                         ) from e
                 _lib = ctypes.CDLL(str(path))
     return _traced if _traced is not None else _lib
+
+
+_serving: Optional[ctypes.CDLL] = None
+
+
+def serving_lib() -> ctypes.CDLL:
+    """The library with the kernels of the ragged serving step: the full library when it is loaded
+    or built from the current sources, else the serving subset, built on first use."""
+    global _serving
+    if _lib is not None:
+        return lib()
+    if _serving is None:
+        with _lock:
+            if _serving is None:
+                try:
+                    path = build_serving()
+                except Exception as e:  # pragma: no cover - depends on toolchain
+                    raise KernelLibraryError(f"the serving kernels could not be built: {e}") from e
+                _serving = ctypes.CDLL(str(path))
+    return _serving
 
 
 class _TracedLib:

@@ -88,6 +88,11 @@ def argmax_rows(logits: torch.Tensor) -> torch.Tensor:
         return logits.float().argmax(-1)
     B, V = logits.shape
     out = torch.empty(B, dtype=torch.int64, device=logits.device)
+    if logits.dtype == torch.float32:
+        rc = _lib.serving_lib().cb_argmax_f32(_lib.ptr(logits), logits.stride(0), B, V, _lib.ptr(out),
+                                              _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_argmax_f32")
+        return out
     rc = _lib.lib().cb_argmax(_lib.ptr(logits), logits.stride(0), B, V, _lib.ptr(out),
                               _lib.stream_ptr())
     _lib.check_rc(rc, "cb_argmax")

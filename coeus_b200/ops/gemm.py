@@ -18,7 +18,7 @@ import torch
 
 from . import _lib
 
-EPI = {"none": 0, "gelu": 1, "dgelu": 2}
+EPI = {"none": 0, "gelu": 1, "dgelu": 2, "relu2": 4}
 _OUT_BF16, _OUT_F32, _OUT_F32_ATOMIC = 0, 1, 2
 
 
@@ -117,6 +117,8 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
             v = _gelu_ref(v)
         elif epi == "dgelu":
             v = v * _gelu_grad_ref(aux_in.float())
+        elif epi == "relu2":
+            v = torch.relu(v).square()
         if dropout is not None and dropout[0] > 0:
             from .elementwise import dropout_mask
             keep = dropout_mask(M, N, dropout[0], dropout[1], v.device)
@@ -253,3 +255,42 @@ def linear_wgrad(x: torch.Tensor, dy: torch.Tensor, grad_w: torch.Tensor, *,
             ksplit = _pick_ksplit(tiles, (T + 63) // 64)
     return gemm(x, dy, a_mn=True, b_mn=True, out=grad_w, accumulate=True, ksplit=ksplit,
                 max_ctas=max_ctas)
+
+
+def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "none",
+           softcap: Optional[float] = None, accumulate: bool = False) -> torch.Tensor:
+    """``out[M, N] (+)= epi(x[M, K] @ w[N, K]^T)`` for a serving step: the weight is stored
+    ``[out, in]``, rows of ``x`` and ``out`` may be strided.  bf16 operands run on the tensor cores
+    with a bf16 or fp32 ``out``; fp32 operands are multiplied in full fp32 (``cb_linear_f32``).
+    ``accumulate`` adds into an fp32 ``out`` (the residual stream); ``softcap`` maps the result
+    ``z`` to ``softcap * tanh(z / softcap)`` (fp32 ``out``)."""
+    M, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K or out.shape[0] != M or out.shape[1] != N:
+        raise ValueError(f"linear: shapes {tuple(x.shape)} {tuple(w.shape)} {tuple(out.shape)}")
+    if not x.is_cuda:
+        v = x.float() @ w.float().t()
+        if epi == "relu2":
+            v = torch.relu(v).square()
+        if softcap is not None:
+            v = softcap * torch.tanh(v / softcap)
+        return out.add_(v) if accumulate else out.copy_(v.to(out.dtype))
+    if x.dtype == torch.float32:
+        act = 5 if softcap is not None else EPI[epi]
+        rc = _lib.serving_lib().cb_linear_f32(
+            _lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(out), out.stride(0), M, N,
+            K, act, ctypes.c_float(softcap or 0.0), int(accumulate), _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_linear_f32")
+        return out
+    out_mode = _OUT_BF16 if out.dtype == torch.bfloat16 else (
+        _OUT_F32_ATOMIC if accumulate else _OUT_F32)
+    rc = _lib.serving_lib().cb_gemm_bf16(
+        _lib.ptr(x), _lib.ptr(w), _lib.ptr(out), M, N, K, x.stride(0), w.stride(0), out.stride(0),
+        0, 0, None, None, 0, None, None, 0, EPI[epi], out_mode, ctypes.c_float(1.0), 1,
+        _pick_bn(M, N), _lib.ptr(_lib.status_buffer(x.device)), 0, _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_gemm_bf16")
+    if softcap is not None:
+        rc = _lib.serving_lib().cb_softcap(_lib.ptr(out), out.stride(0), M, N,
+                                           ctypes.c_float(softcap), _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_softcap")
+    return out

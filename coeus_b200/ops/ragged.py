@@ -1,0 +1,367 @@
+"""Ops of the ragged serving step (``csrc/ragged_rows.cu``, ``shortconv.cu``, ``delta_scan.cu``,
+``ragged_attn.cu``): one batch holds portions of prompts beside single decoded tokens, each at its
+own position of its own sequence, and recurrent and cached state is addressed by slot.
+
+CPU tensors take a PyTorch restatement of the same math; CUDA tensors always run the kernels, in
+bf16 or (for a model held in fp32) in full fp32.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import List, Optional, Sequence, Tuple
+
+import numpy as np
+import torch
+
+from . import _lib
+from .decode import PAGE
+
+CONV_TILE = 16        # tokens per block of the convolution kernels
+ATTN_TILE = 64        # query rows per block of the tensor-core attention kernel
+ROWS_MAX = 4          # entries of at most this many tokens take the row kernel
+_F = ctypes.c_float
+
+
+def _p(t):
+    return _lib.ptr(t)
+
+
+@dataclass
+class Entry:
+    """The next ``tokens`` of the sequence in ``slot``, which already holds ``pos0`` tokens;
+    ``want`` lists the places among them whose logits are asked for."""
+
+    slot: int
+    pos0: int
+    tokens: Sequence[int]
+    want: Sequence[int] = ()
+
+
+class RaggedBatch:
+    """Index arrays of one step, in one int32 buffer (one host-to-device copy).  ``tile_rows``
+    says whether long entries may take the tensor-core attention kernel (bf16 models on CUDA);
+    otherwise every row is listed for the row kernel."""
+
+    def __init__(self, entries: List[Entry], device, tile_rows: bool = True,
+                 into: Optional["RaggedBatch"] = None) -> None:
+        n = len(entries)
+        lens = [len(e.tokens) for e in entries]
+        if not n or min(lens) < 1:
+            raise ValueError("a step needs entries of at least one token")
+        self.n, self.T, self.lens = n, sum(lens), lens
+        self.pos0_host = [e.pos0 for e in entries]
+        self.slots_host = [e.slot for e in entries]
+        self.max_ctx = max(e.pos0 + m for e, m in zip(entries, lens))
+        row0 = np.concatenate([[0], np.cumsum(lens)]).astype(np.int32)
+        tokens = np.concatenate([np.asarray(e.tokens, dtype=np.int32) for e in entries])
+        pos = np.concatenate([np.arange(e.pos0, e.pos0 + m, dtype=np.int32)
+                              for e, m in zip(entries, lens)])
+        row_slot = np.repeat(np.asarray([e.slot for e in entries], dtype=np.int32), lens)
+        ct = [(i, o) for i, m in enumerate(lens) for o in range(0, m, CONV_TILE)]
+        big = [i for i, m in enumerate(lens) if tile_rows and m > ROWS_MAX]
+        # tiles with the most keys first
+        at = sorted(((i, o) for i in big for o in range(0, lens[i], ATTN_TILE)),
+                    key=lambda t: -(entries[t[0]].pos0 + t[1]))
+        small = [i for i in range(n) if i not in set(big)]
+        rows = np.concatenate([np.arange(row0[i], row0[i + 1], dtype=np.int32) for i in small]) \
+            if small else np.zeros(0, np.int32)
+        want = np.asarray([row0[i] + k for i, e in enumerate(entries) for k in e.want],
+                          dtype=np.int32)
+        parts = [pos, np.asarray(self.pos0_host, np.int32), tokens, row_slot,
+                 np.asarray(self.slots_host, np.int32), row0[:n], np.asarray(lens, np.int32),
+                 np.asarray([c[0] for c in ct], np.int32), np.asarray([c[1] for c in ct], np.int32),
+                 rows, np.asarray([c[0] for c in at], np.int32),
+                 np.asarray([c[1] for c in at], np.int32), want]
+        host = torch.from_numpy(np.concatenate(parts).astype(np.int32, copy=False))
+        if into is None:
+            self.buf = host.to(device)
+        else:
+            if into.buf.numel() != host.numel():
+                raise ValueError("the batch does not fit the captured one")
+            self.buf = into.buf
+            self.buf.copy_(host)
+        views, o = [], 0
+        for part in parts:
+            views.append(self.buf[o:o + len(part)])
+            o += len(part)
+        (self.pos, self.pos0, self.tokens, self.row_slot, self.slot, self.row0, self.len,
+         self.conv_entry, self.conv_off, self.rows, self.attn_entry, self.attn_off,
+         self.want) = views
+        self.positions = self.buf[:self.T + n]       # pos and pos0: what a decode step advances
+        self.n_conv, self.n_rows, self.n_attn, self.n_want = len(ct), len(rows), len(at), len(want)
+
+    def entry_args(self):
+        return _p(self.slot), _p(self.row0), _p(self.len), _p(self.pos0)
+
+
+def embed_norm(tokens: torch.Tensor, embed: torch.Tensor, weight: Optional[torch.Tensor],
+               width: int, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """Rows of ``embed`` (RMS-normalised with ``weight`` when given) as the fp32 residual stream;
+    columns ``width ..`` of ``out`` are zero."""
+    if not out.is_cuda:
+        x = embed[tokens.long(), :width].float()
+        if weight is not None:
+            x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * weight[:width]
+        out.zero_()
+        out[:, :width] = x
+        return out
+    rc = _lib.serving_lib().cb_embed_norm(
+        _p(tokens), _p(embed), embed.stride(0), embed.shape[0], _p(weight), _p(out), out.stride(0),
+        out.shape[0], width, _F(eps), int(embed.dtype == torch.float32),
+        _p(_lib.status_buffer(out.device)), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_embed_norm")
+    return out
+
+
+def rms_rows(x: torch.Tensor, w1: torch.Tensor, width: int, eps: float, dtype: torch.dtype,
+             w2: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None
+             ) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """RMS norm of the fp32 stream (of its ``rows`` only, when given) in the activation type,
+    with one weight or, in the same pass, with two."""
+    n = x.shape[0] if rows is None else rows.shape[0]
+    if not x.is_cuda:
+        v = x if rows is None else x[rows.long()]
+        r = v * torch.rsqrt((v[:, :width] ** 2).mean(-1, keepdim=True) + eps)
+        return (r * w1).to(dtype), None if w2 is None else (r * w2).to(dtype)
+    y1 = torch.empty((n, x.shape[1]), dtype=dtype, device=x.device)
+    y2 = torch.empty_like(y1) if w2 is not None else None
+    rc = _lib.serving_lib().cb_rms_rows(
+        _p(x), x.stride(0), _p(rows), _p(w1), _p(y1), _p(w2), _p(y2), y1.stride(0), n, width,
+        _F(eps), int(dtype == torch.float32), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_rms_rows")
+    return y1, y2
+
+
+def rope_table(pos: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+    """``[rows, half, 2]`` fp32 (cos, sin) of ``pos * inv_freq``."""
+    n, half = pos.shape[0], inv_freq.shape[0]
+    if not pos.is_cuda:
+        a = pos.float()[:, None] * inv_freq[None]
+        return torch.stack([a.cos(), a.sin()], -1)
+    out = torch.empty((n, half, 2), dtype=torch.float32, device=pos.device)
+    rc = _lib.serving_lib().cb_rope_table(_p(pos), _p(inv_freq), n, half, _p(out),
+                                          _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_rope_table")
+    return out
+
+
+def _conv_ref(raw: torch.Tensor, taps_w: torch.Tensor, state: torch.Tensor, batch: RaggedBatch
+              ) -> torch.Tensor:
+    """Convolution of ``raw [rows, C]`` entry by entry; advances ``state [slots, taps-1, C]``."""
+    n1 = taps_w.shape[0] - 1
+    out = torch.empty(raw.shape, dtype=torch.float32)
+    r = 0
+    for i, m in enumerate(batch.lens):
+        s = batch.slots_host[i]
+        prev = state[s].float() if int(batch.pos0[i]) > 0 else torch.zeros(n1, raw.shape[1])
+        u = torch.cat([prev, raw[r:r + m].float()])
+        out[r:r + m] = sum(u[j:j + m] * taps_w[j] for j in range(n1 + 1))
+        if n1:
+            state[s] = u[-n1:].to(state.dtype)
+        r += m
+    return out
+
+
+def _cells(page_table: torch.Tensor, batch: RaggedBatch):
+    pos, slot = batch.pos.long(), batch.row_slot.long()
+    return page_table[slot, pos // PAGE].long(), pos % PAGE
+
+
+def shortconv_attn(raw: torch.Tensor, koff: int, voff: int, taps_w: torch.Tensor,
+                   state: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
+                   batch: RaggedBatch, rope: Optional[torch.Tensor], k_cache: torch.Tensor,
+                   v_cache: torch.Tensor, page_table: torch.Tensor,
+                   v_first: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                   write_first: bool = False) -> torch.Tensor:
+    """What stands between the projections and the scores of an attention layer: a causal
+    convolution over time on every channel of q, k and v (``taps_w [taps, channels]``), rotary
+    embedding of the first ``2 * rope.shape[1]`` entries of the q and k heads in the rotate-half
+    layout, value mixing ``v <- (1 - mix) v + mix v_first`` (or, with ``write_first``, keeping v as
+    ``v_first``), and the write of k and v into the cache pages.  Returns ``q [rows, heads*dim]``."""
+    T = raw.shape[0]
+    half = rope.shape[1] if rope is not None else 0
+    mode = 1 if write_first else (2 if mix is not None else 0)
+    qc, kc, vc = heads * dim, kv_heads * dim, kv_heads * vdim
+    if not raw.is_cuda:
+        u = torch.cat([raw[:, :qc], raw[:, koff:koff + kc], raw[:, voff:voff + vc]], 1)
+        y = _conv_ref(u, taps_w, state, batch)
+        q, k = y[:, :qc].view(T, heads, dim), y[:, qc:qc + kc].view(T, kv_heads, dim)
+        v = y[:, qc + kc:].view(T, kv_heads, vdim)
+        if half:
+            c, s = rope[:, None, :, 0], rope[:, None, :, 1]
+
+            def rot(x):
+                a, b = x[..., :half], x[..., half:2 * half]
+                return torch.cat([a * c - b * s, b * c + a * s, x[..., 2 * half:]], -1)
+            q, k = rot(q), rot(k)
+        if mode == 1:
+            v_first.copy_(v.reshape(T, -1))
+        elif mode == 2:
+            v = (1 - mix) * v + mix * v_first.float().view(T, kv_heads, vdim)
+        page, at = _cells(page_table, batch)
+        k_cache[page, at, :, :dim] = k.to(k_cache.dtype)
+        v_cache[page, at, :, :vdim] = v.to(v_cache.dtype)
+        return q.reshape(T, qc).to(raw.dtype)
+    q = torch.empty((T, qc), dtype=raw.dtype, device=raw.device)
+    rc = _lib.serving_lib().cb_shortconv_attn(
+        _p(raw), raw.stride(0), koff, voff, _p(taps_w), taps_w.shape[0], _p(state), heads, kv_heads,
+        dim, vdim, *batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off), batch.n_conv, half,
+        _p(rope), _p(q), _p(k_cache), _p(v_cache), k_cache.shape[-1], v_cache.shape[-1],
+        _p(page_table), page_table.shape[1], k_cache.shape[0], _p(v_first), _p(mix), mode,
+        int(raw.dtype == torch.float32), _p(_lib.status_buffer(raw.device)), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_shortconv_attn")
+    return q
+
+
+def shortconv_delta(raw: torch.Tensor, koff: int, voff: int, boff: int, taps_w: torch.Tensor,
+                    state: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
+                    batch: RaggedBatch, a: torch.Tensor, A_log: torch.Tensor,
+                    dt_bias: torch.Tensor):
+    """Inputs of the gated delta recurrence, fp32: convolution and SiLU of q, k and v, unit norm of
+    q and k (q also times ``dim ** -0.5``), the decay ``exp(-exp(A_log) softplus(a + dt_bias))`` of
+    every key channel, the step size ``sigmoid(raw[:, boff + h])``.  Returns
+    ``(q, k, kq, v, g, beta)``; q, k, g are padded with zeros to a multiple of four channels."""
+    T = raw.shape[0]
+    dim4 = (dim + 3) // 4 * 4
+    qc, vc = kv_heads * dim, heads * vdim
+    f32 = dict(dtype=torch.float32, device=raw.device)
+    alloc = torch.zeros if not raw.is_cuda else torch.empty
+    q, k = alloc((T, kv_heads, dim4), **f32), alloc((T, kv_heads, dim4), **f32)
+    kq, v = alloc((T, kv_heads), **f32), alloc((T, heads, vdim), **f32)
+    g, beta = alloc((T, heads, dim4), **f32), alloc((T, heads), **f32)
+    if not raw.is_cuda:
+        u = torch.cat([raw[:, :qc], raw[:, koff:koff + qc], raw[:, voff:voff + vc]], 1)
+        y = torch.nn.functional.silu(_conv_ref(u, taps_w, state, batch))
+
+        def unit(x):
+            return x * torch.rsqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+        q[..., :dim] = unit(y[:, :qc].view(T, kv_heads, dim)) * dim ** -0.5
+        k[..., :dim] = unit(y[:, qc:2 * qc].view(T, kv_heads, dim))
+        kq.copy_((q * k).sum(-1))
+        v.copy_(y[:, 2 * qc:].view(T, heads, vdim))
+        z = torch.nn.functional.softplus(a[:, :heads * dim].float() + dt_bias, threshold=100.0)
+        g[..., :dim] = torch.exp(-torch.exp(A_log)[None, :, None] * z.view(T, heads, dim))
+        beta.copy_(torch.sigmoid(raw[:, boff:boff + heads].float()))
+        return q, k, kq, v, g, beta
+    rc = _lib.serving_lib().cb_shortconv_delta(
+        _p(raw), raw.stride(0), koff, voff, boff, _p(taps_w), taps_w.shape[0], _p(state), heads,
+        kv_heads, dim, vdim, *batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off),
+        batch.n_conv, _p(a), a.stride(0), _p(A_log), _p(dt_bias), _p(q), _p(k), _p(kq), _p(v), _p(g),
+        _p(beta), dim4, int(raw.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_shortconv_delta")
+    return q, k, kq, v, g, beta
+
+
+def delta_scan(q: torch.Tensor, k: torch.Tensor, kq: torch.Tensor, v: torch.Tensor,
+               g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor, batch: RaggedBatch
+               ) -> torch.Tensor:
+    """The gated delta rule over every entry, from and into ``state [slots, heads, dim, vdim]``
+    (fp32).  Returns the read-outs ``[rows, heads, vdim]``, fp32."""
+    T, heads, vdim = v.shape
+    kv_heads, dim, dim4 = q.shape[1], state.shape[2], q.shape[2]
+    o = torch.empty_like(v)
+    if not v.is_cuda:
+        per, r = heads // kv_heads, 0
+        for i, m in enumerate(batch.lens):
+            s = batch.slots_host[i]
+            S = state[s].clone() if int(batch.pos0[i]) > 0 else torch.zeros_like(state[s])
+            for t in range(r, r + m):
+                kk, qq = (x[t, :, :dim].repeat_interleave(per, 0) for x in (k, q))
+                S = S * g[t, :, :dim, None]
+                w = beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, kk))
+                S = S + kk[:, :, None] * w[:, None, :]
+                o[t] = torch.einsum("hdv,hd->hv", S, qq)
+            state[s] = S
+            r += m
+        return o
+    rc = _lib.serving_lib().cb_delta_scan(
+        _p(q), _p(k), _p(kq), _p(v), _p(g), _p(beta), _p(state), _p(o), heads, kv_heads, dim, dim4,
+        vdim, *batch.entry_args(), batch.n, _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_delta_scan")
+    return o
+
+
+def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float,
+                    out: torch.Tensor) -> torch.Tensor:
+    """``out = o / rms(o) * weight * sigmoid(gate)`` per head; ``o [rows, heads, vdim]`` fp32,
+    ``gate`` and ``out`` ``[rows, heads * vdim]`` views."""
+    T, heads, vdim = o.shape
+    if not o.is_cuda:
+        y = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps) * weight
+        y = y * torch.sigmoid(gate[:, :heads * vdim].float()).view(T, heads, vdim)
+        return out.copy_(y.reshape(T, -1).to(out.dtype))
+    rc = _lib.serving_lib().cb_gated_head_norm(
+        _p(o), _p(gate), gate.stride(0), _p(weight), _p(out), out.stride(0), T, heads, vdim, _F(eps),
+        int(out.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_gated_head_norm")
+    return out
+
+
+def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                     page_table: torch.Tensor, batch: RaggedBatch, heads: int, kv_heads: int,
+                     dim: int, vdim: int, scale: float, out: torch.Tensor, *,
+                     chunk: Optional[int] = None, sink: Optional[torch.Tensor] = None,
+                     gate: Optional[torch.Tensor] = None, max_ctx: Optional[int] = None
+                     ) -> torch.Tensor:
+    """Causal attention of every query row over the cached keys of its own sequence, restricted to
+    the row's chunk (positions with the same ``pos // chunk``) when ``chunk`` is given.  ``sink``
+    (fp32 ``[heads]``) is a logit that enters the softmax denominator only; ``gate`` (a view whose
+    column ``h`` belongs to head ``h``) multiplies head ``h``'s output by its sigmoid.  Query head
+    ``h`` reads key/value head ``h // (heads // kv_heads)``.  ``out`` is a ``[rows, heads * vdim]``
+    view; ``max_ctx`` bounds the keys of any row (it only chooses how many CTAs share a row)."""
+    T = q.shape[0]
+    if not q.is_cuda:
+        per = heads // kv_heads
+        r = 0
+        for i, m in enumerate(batch.lens):
+            pos = batch.pos[r:r + m].long()
+            n = int(pos[-1]) + 1
+            pages = page_table[batch.slots_host[i], :(n + PAGE - 1) // PAGE].long()
+            K = k_cache[pages].reshape(-1, kv_heads, k_cache.shape[-1])[:n, :, :dim].float()
+            V = v_cache[pages].reshape(-1, kv_heads, v_cache.shape[-1])[:n, :, :vdim].float()
+            K, V = K.repeat_interleave(per, 1), V.repeat_interleave(per, 1)
+            s = torch.einsum("thd,nhd->htn", q[r:r + m].float().view(m, heads, dim), K) * scale
+            j = torch.arange(n)
+            lo = pos // chunk * chunk if chunk else torch.zeros_like(pos)
+            ok = (j[None] <= pos[:, None]) & (j[None] >= lo[:, None])
+            s = s.masked_fill(~ok, float("-inf"))
+            top = s.amax(-1, keepdim=True)
+            if sink is not None:
+                top = torch.maximum(top, sink.view(-1, 1, 1))
+            w = torch.exp(s - top)
+            den = w.sum(-1, keepdim=True)
+            if sink is not None:
+                den = den + torch.exp(sink.view(-1, 1, 1) - top)
+            o = torch.einsum("htn,nhd->thd", w / den, V)
+            if gate is not None:
+                o = o * torch.sigmoid(gate[r:r + m, :heads].float())[:, :, None]
+            out[r:r + m] = o.reshape(m, -1).to(out.dtype)
+            r += m
+        return out
+    st = _p(_lib.status_buffer(q.device))
+    lib = _lib.serving_lib()
+    common = (_p(q), _p(k_cache), _p(v_cache), _p(page_table), page_table.shape[1],
+              k_cache.shape[0], heads, kv_heads, dim, vdim, k_cache.shape[-1], v_cache.shape[-1],
+              chunk or 0, _F(scale), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0,
+              _p(out), out.stride(0))
+    if batch.n_attn:
+        rc = lib.cb_ragged_attn_tiles(*common, *batch.entry_args(), _p(batch.attn_entry),
+                                      _p(batch.attn_off), batch.n_attn, st, _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_ragged_attn_tiles")
+    n = batch.n_rows
+    if n:
+        per = heads // kv_heads
+        ctas = n * kv_heads * (1 if per <= 8 else (per + 7) // 8)
+        ctx = max_ctx or batch.max_ctx
+        ctx = min(ctx, chunk) if chunk else ctx
+        splits = max(1, min(16, (4 * 148 + ctas - 1) // ctas, ctx // 256))
+        part_o = part_ml = None
+        if splits > 1:
+            part_o = torch.empty((n, heads, splits, vdim), dtype=torch.float32, device=q.device)
+            part_ml = torch.empty((n, heads, splits, 2), dtype=torch.float32, device=q.device)
+        rc = lib.cb_ragged_attn_rows(*common, _p(batch.rows), _p(batch.row_slot), _p(batch.pos), n,
+                                     splits, _p(part_o), _p(part_ml), int(q.dtype == torch.float32),
+                                     st, _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_ragged_attn_rows", launches=2 if splits > 1 else 1)
+    return out
