@@ -5,7 +5,8 @@ Commands
     generate   load a model file and continue a prompt
     eval       load a model file and report loss / perplexity on text or token files
     serve      load a model file (or build a random one) and serve completions over HTTP
-    info       print the resolved configuration and the parameter count
+    info       print the resolved configuration and the parameter count (of ``--weights``, when a
+               model directory is given)
 
 Configuration comes, lowest priority first, from the built-in defaults, the given ``.yaml`` /
 ``.json`` files, ``COEUS_*`` environment variables (``COEUS_TRAIN__LR=1e-4`` sets ``train.lr``)
@@ -232,11 +233,11 @@ def cmd_train(store) -> dict:
 
 
 def _load_weights(weights: str, device: str, training: bool = False):
-    """A model file (``.safetensors`` / ``.gguf`` / ``.rustllm``) or a Hugging Face style
-    directory (``config.json`` + ``*.safetensors``, Llama naming)."""
+    """A model file (``.safetensors`` / ``.gguf`` / ``.rustllm``) or a model directory
+    (``config.json`` + ``*.safetensors``) of a registered architecture."""
     if os.path.isdir(weights):
-        from .checkpoint.hf import load_hf_dir
-        return load_hf_dir(weights, device=device, training=training)
+        from .models.registry import load_dir
+        return load_dir(weights, device=device, training=training)
     from .checkpoint.formats import load_model
     return load_model(weights, device=device, training=training)[0]
 
@@ -259,7 +260,7 @@ def _load_tokenizer(store, weights: str):
 def cmd_generate(store, rest: List[str]) -> dict:
     import torch
 
-    from .infer.engine import InferenceEngine
+    from .infer.engine import make_engine
     device = _device(store)
     weights = _get(store, "weights")
     if not weights:
@@ -275,7 +276,7 @@ def cmd_generate(store, rest: List[str]) -> dict:
         raise SystemExit("generate needs --prompt_ids=1,2,3, or --prompt=text with a tokenizer "
                          "file (<weights>.tokenizer.json or --tokenizer=...)")
     n = int(_get(store, "max_tokens") or 16)
-    out = InferenceEngine(model, max_batch=1).generate(
+    out = make_engine(model, max_batch=1).generate(
         torch.tensor(ids, device=device)[None], n,
         temperature=float(_get(store, "temperature") or 0.0))
     res = {"prompt_ids": ids, "token_ids": out[0, len(ids):].tolist()}
@@ -340,8 +341,10 @@ def cmd_serve(store) -> int:
         model = DecoderLM(_model_config(store), device if world == 1 else "cpu",
                           dtype=dtype if world == 1 else torch.float32, training=False)
     max_seqs = int(_get(store, "max_seqs") or 16)
-    kw = dict(max_seqs=max_seqs, max_len=model.cfg.max_seq_len)
+    kw = dict(max_seqs=max_seqs, max_len=int(_get(store, "max_len") or model.cfg.max_seq_len))
     engine = group = None
+    if world > 1 and not isinstance(model, DecoderLM):
+        raise SystemExit(f"{model.cfg.architecture} models are served by one process")
     if world > 1:
         import torch.distributed as dist
 
@@ -366,6 +369,15 @@ def cmd_serve(store) -> int:
 
 def cmd_info(store) -> dict:
     from .models.decoder import ParamLayout
+    weights = _get(store, "weights")
+    if weights and os.path.isdir(str(weights)):
+        from .models.registry import read_config, resolve
+        config = read_config(str(weights))
+        model = _load_weights(str(weights), "cpu")
+        out = {"architecture": resolve(config).name, "model": model.cfg.to_dict(),
+               "parameters": model.num_parameters()}
+        print(json.dumps(out))
+        return out
     cfg = _model_config(store)
     out = {"model": cfg.to_dict(), "parameters": ParamLayout(cfg).num_parameters(),
            "config": {k: _get(store, k) for k in sorted(store.keys())}}

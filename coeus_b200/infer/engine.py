@@ -179,11 +179,17 @@ class InferenceEngine:
         return self._logits(last)
 
     # ------------------------------------------------------------------ slot-wise API (serving)
-    def open_slots(self, max_seqs: int, max_len: int) -> PagedKVCache:
+    def open_slots(self, max_seqs: int, max_len: int, num_pages: Optional[int] = None
+                   ) -> PagedKVCache:
         """A cache whose rows are independent request slots (see
-        :class:`coeus_b200.infer.scheduler.ContinuousBatcher`); pages are handed out per slot."""
-        c = PagedKVCache.for_model(self.cfg, max_seqs, max(max_len, D.PAGE) + D.PAGE,
-                                   self.m.device)
+        :class:`coeus_b200.infer.scheduler.ContinuousBatcher`); pages are handed out per slot, from
+        a pool of ``num_pages`` (default: enough for every slot to grow to ``max_len``)."""
+        if num_pages is None:
+            c = PagedKVCache.for_model(self.cfg, max_seqs, max(max_len, D.PAGE) + D.PAGE,
+                                       self.m.device)
+        else:
+            c = PagedKVCache(self.cfg.num_layers, self.cfg.kv_heads, self.cfg.head_dim, num_pages,
+                             max_seqs, max(1, (max_len + D.PAGE - 1) // D.PAGE), self.m.device)
         if self.m.p16.dtype != torch.bfloat16:       # CPU oracle runs keep their precision
             c.k = [t.to(self.m.p16.dtype) for t in c.k]
             c.v = [t.to(self.m.p16.dtype) for t in c.v]
@@ -264,6 +270,29 @@ class InferenceEngine:
                          pos_dev=positions if cfg.pos == "rope" else None, page_table=table,
                          ctx=ctx)
         return self._logits(x)
+
+    def step(self, entries) -> Optional[torch.Tensor]:
+        """The next tokens of several sequences (:class:`coeus_b200.ops.ragged.Entry`), cut anywhere;
+        the logits ``[wanted, V]`` of the wanted places in order.  This decoder's kernels want one
+        token per sequence, so an entry's tokens take one decode batch each."""
+        for e in entries:
+            self.cache.reserve(e.slot, e.pos0 + len(e.tokens))
+        got = {}
+        for k in range(max(len(e.tokens) for e in entries)):
+            live = [(i, e) for i, e in enumerate(entries) if k < len(e.tokens)]
+            logits = self.decode_slots(
+                torch.tensor([e.slot for _, e in live], dtype=torch.int64, device=self.m.device),
+                torch.tensor([e.tokens[k] for _, e in live], dtype=torch.int64,
+                             device=self.m.device),
+                torch.tensor([e.pos0 + k for _, e in live], dtype=torch.int32,
+                             device=self.m.device))
+            for row, (i, e) in enumerate(live):
+                if k in e.want:
+                    got[i, k] = logits[row]
+        for e in entries:
+            self.cache.set_length(e.slot, e.pos0 + len(e.tokens))
+        rows = [got[i, k] for i, e in enumerate(entries) for k in e.want]
+        return torch.stack(rows) if rows else None
 
     def _decode_body(self, tokens: torch.Tensor) -> torch.Tensor:
         """One token per sequence at the device-side position; advances the positions."""

@@ -156,6 +156,9 @@ class HybridEngine(InferenceEngine):
             if e.pos0 != c.length(e.slot):
                 raise ProcessingError.invalid_input(
                     f"slot {e.slot} holds {c.length(e.slot)} tokens, the entry starts at {e.pos0}")
+            if min(e.tokens) < 0 or max(e.tokens) >= self.cfg.vocab_size:
+                raise ProcessingError.invalid_input(
+                    f"token ids must lie in [0, {self.cfg.vocab_size})")
         for e in entries:
             c.reserve(e.slot, e.pos0 + len(e.tokens))
         if self.use_graph and layer_out is None and \
@@ -272,3 +275,7 @@ class HybridEngine(InferenceEngine):
                      ) -> torch.Tensor:
         return self.step([Entry(s, p, [t], [0]) for s, t, p in
                           zip(slots.tolist(), tokens.tolist(), positions.tolist())])
+
+    def prefill_slot_paged(self, slot, ids, total_len, prefix_pages):
+        raise ProcessingError.unsupported("a prompt on cached prefix pages",
+                                          "the layers' state at that point is not in the pages")

@@ -7,6 +7,10 @@ per active slot through the model in a single decode batch whose rows sit at dif
 and retires the rows that are done, returning their pages to the free list.  The reference's
 ``InferenceRequest{tokens, max_length}`` / ``InferenceResult{predictions}``
 (src/domain/inference/mod.rs:6-32) name a request and a result; it has no batching or cache.
+
+Engines that run ragged batches (``engine.ragged``) get one step for everything: the next token of
+every decoding request and portions of the prompts that are still being read, up to
+``step_tokens`` rows, go through the model together.
 """
 from __future__ import annotations
 
@@ -16,7 +20,8 @@ from typing import Callable, Deque, Dict, List, Optional
 
 import torch
 
-from ..foundation.error import Error, ProcessingError
+from ..foundation.error import ProcessingError, ResourceError
+from ..ops.ragged import Entry
 from .engine import InferenceEngine
 from .sampler import select
 
@@ -35,6 +40,7 @@ class Request:
     stop_ids: tuple = ()                 # further token ids that end the request like eos_id
     output: List[int] = field(default_factory=list)
     slot: int = -1
+    read: int = 0                        # prompt tokens that have been through the model
     on_token: Optional[Callable[[int], None]] = None      # called with every new token
     error: Optional[BaseException] = None                  # set when the request failed alone
 
@@ -126,17 +132,22 @@ class PrefixCache:
 class ContinuousBatcher:
     def __init__(self, engine: InferenceEngine, max_seqs: int = 64, max_len: Optional[int] = None,
                  token_chunk: Optional[int] = None, seed: int = 0,
-                 prefix_cache: bool = False) -> None:
+                 prefix_cache: bool = False, step_tokens: int = 2048) -> None:
         """``max_seqs`` rows decode together; ``max_len`` bounds prompt + generated tokens of one
         request; ``token_chunk`` prefills long prompts in pieces; ``prefix_cache`` reuses the
         cache pages of prompt prefixes that earlier requests already computed (shared system
-        prompts), in units of whole pages."""
+        prompts), in units of whole pages; ``step_tokens`` bounds the rows of a ragged step."""
         self.engine = engine
         self.max_seqs = max_seqs
         self.max_len = max_len or engine.max_len
         self.token_chunk = token_chunk
         self.device = engine.m.device
         engine.open_slots(max_seqs, self.max_len)
+        self.step_tokens = max(1, step_tokens)
+        if prefix_cache and engine.ragged:
+            raise ProcessingError.unsupported(
+                "prefix caching with this model",
+                "its layers carry state that the cached pages do not hold")
         self.prefix = PrefixCache(engine.cache) if prefix_cache and hasattr(
             engine, "prefill_slot_paged") else None
         self.waiting: Deque[Request] = deque()
@@ -188,6 +199,8 @@ class ContinuousBatcher:
     def step(self) -> List[Request]:
         """Admit, decode one token per active request, retire; returns the requests that finished
         in this step."""
+        if self.engine.ragged:
+            return self._step_ragged()
         eng, cache = self.engine, self.engine.cache
         finished: List[Request] = []
         # a request's first token comes from its prefill
@@ -250,13 +263,78 @@ class ContinuousBatcher:
                 out[r.id] = r.output
         return out
 
+    # ------------------------------------------------------------------ ragged steps
+    def _admit(self, finished: List[Request]) -> None:
+        """Waiting requests into free slots while the page pool can hold them to their end; a
+        request that has to wait for pages keeps its place at the head of the queue."""
+        cache = self.engine.cache
+        while self.waiting and self.free_slots:
+            r = self.waiting[0]
+            slot = self.free_slots[-1]
+            try:
+                cache.reserve(slot, len(r.prompt) + r.max_new_tokens)
+            except ResourceError as e:
+                cache.release(slot)
+                if self.active:
+                    return
+                self.waiting.popleft()          # not even an empty pool is enough
+                r.error = e
+                finished.append(r)
+                continue
+            self.waiting.popleft()
+            self.free_slots.pop()
+            r.slot = slot
+            self.active[slot] = r
+
+    def _step_ragged(self) -> List[Request]:
+        eng = self.engine
+        finished: List[Request] = []
+        self._admit(finished)
+        entries, reqs = [], []
+        room = self.step_tokens
+        order = sorted(self.active.values(), key=lambda r: (r.read < len(r.prompt), r.id))
+        for r in order:                         # decoding requests first, then the oldest prompts
+            if r.read >= len(r.prompt):
+                entries.append(Entry(r.slot, len(r.prompt) + len(r.output) - 1, [r.output[-1]], [0]))
+                reqs.append((r, True))
+                room -= 1
+                continue
+            n = min(len(r.prompt) - r.read, max(room, 0) if entries else max(room, 1),
+                    self.token_chunk or self.step_tokens)
+            if n <= 0:
+                break
+            last = r.read + n == len(r.prompt)
+            entries.append(Entry(r.slot, r.read, r.prompt[r.read:r.read + n], [n - 1] if last else []))
+            reqs.append((r, last))
+            room -= n
+        self.stats["steps"] += 1
+        if not entries:
+            return finished
+        logits = eng.step(entries)
+        decoded = sum(r.read >= len(r.prompt) for r, _ in reqs)
+        for e, (r, _) in zip(entries, reqs):
+            r.read = max(r.read, min(len(r.prompt), e.pos0 + len(e.tokens)))
+        sampled = [r for r, wanted in reqs if wanted]
+        if sampled:
+            V = eng.cfg.vocab_size
+            greedy = all(not r.temperature and r.repetition_penalty == 1.0 for r in sampled)
+            nxt = select(logits[:, :V], 0.0, None, None, None).tolist() if greedy else None
+            for i, r in enumerate(sampled):
+                if not r.output:
+                    self.stats["prefills"] += 1
+                r.push(int(nxt[i] if greedy else self._sample(logits[i:i + 1], r)[0]))
+                if r.done:
+                    self._retire(r, finished)
+        self.stats["decoded_tokens"] += decoded
+        self.stats["max_active"] = max(self.stats["max_active"], decoded)
+        return finished
+
     # ------------------------------------------------------------------ internals
     def _prefill(self, r: Request, ids: torch.Tensor) -> torch.Tensor:
         eng, total = self.engine, len(r.prompt) + r.max_new_tokens
         if self.prefix is None:
             return eng.prefill_slot(r.slot, ids, total, token_chunk=self.token_chunk)
         from ..ops.decode import PAGE
-        from ..foundation.error import ResourceError
         for attempt in range(2):
             pages = self.prefix.match(r.prompt, PAGE)
             try:

@@ -30,6 +30,8 @@ from .kv_cache import PagedKVCache
 
 
 class TPInferenceEngine:
+    ragged = False
+
     def __init__(self, model: TPDecoderLM, max_batch: int = 64, use_graph: Optional[bool] = None,
                  ar_backend: Optional[str] = None, decode_splits: int = 0) -> None:
         self.m, self.cfg, self.tp = model, model.cfg, model.tp

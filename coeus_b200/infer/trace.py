@@ -60,7 +60,13 @@ def main(argv=None) -> int:
     from ..models.registry import load_dir
     from .engine import make_engine
     torch.backends.cuda.matmul.allow_tf32 = False
-    model = load_dir(a.model, device=a.device, dtype=getattr(torch, a.dtype))
+    try:
+        model = load_dir(a.model, device=a.device, dtype=getattr(torch, a.dtype))
+    except ProcessingError as e:
+        if a.dtype == "float32":
+            print(e, file=sys.stderr)
+            return 3
+        raise
     runner = TraceRunner(make_engine(model, max_batch=SLOTS), a.max_tokens)
     for line in sys.stdin:
         if not line.strip():

@@ -112,11 +112,11 @@ class HybridConfig:
                 if m.chunk is not None and m.chunk < 1:
                     raise ConfigError.invalid(where, m.chunk, "A chunk has at least one position")
                 if m.v_mix:
-                    shape = (m.kv_heads, m.vdim)
-                    if mixing not in (None, shape):
-                        raise ConfigError.invalid(where, shape,
+                    size = m.kv_heads * m.vdim
+                    if mixing not in (None, size):
+                        raise ConfigError.invalid(where, size,
                                                   "Layers that mix values must agree in their size")
-                    mixing = shape
+                    mixing = size
             if layer.mlp is not None and layer.mlp.kind != "dense":
                 raise ConfigError.invalid(f"layers[{i}].mlp", layer.mlp.kind,
                                           "Feed-forward kind must be 'dense'")

@@ -17,7 +17,7 @@ from typing import Dict, List, Optional
 
 from ..core.traits import HealthCheck, Metrics
 from ..foundation.error import ProcessingError
-from ..infer.engine import InferenceEngine
+from ..infer.engine import make_engine
 from ..infer.scheduler import ContinuousBatcher
 
 try:        # the request schema lives at module level so that FastAPI can resolve its annotation
@@ -51,8 +51,7 @@ class ServingLoop(Metrics, HealthCheck):
         tensor-parallel engine; every rank of it runs a loop, rank 0 of the group takes the
         requests and sends each iteration's submissions and cancellations to the others, so all
         ranks feed their batcher the same events in the same order and step together."""
-        self.engine = engine if engine is not None else InferenceEngine(
-            model, max_batch=max_seqs, use_graph=False)
+        self.engine = engine if engine is not None else make_engine(model, max_batch=max_seqs)
         self.group = group
         self.leader = True
         if group is not None:

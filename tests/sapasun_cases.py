@@ -1,0 +1,466 @@
+"""Small Sapasun configurations, weights and checks shared by the CPU and the GPU tests.  The
+oracle is :mod:`plain_sapasun`; the configurations are chosen so that sizes differ from one
+another (heads, key and value widths, taps, chunks, ranks), with and without each option."""
+import torch
+
+import plain_sapasun as plain
+from coeus_b200.infer.engine import make_engine
+from coeus_b200.infer.scheduler import ContinuousBatcher
+from coeus_b200.models import hybrid as H
+from coeus_b200.ops import gemm as G
+from coeus_b200.ops import ragged as R
+from coeus_b200.ops.decode import PAGE
+
+A, D, M, L = H.AttentionSpec, H.ChannelDeltaSpec, H.MlpSpec, H.LayerSpec
+
+
+def config(kind):
+    if kind == "odd":         # nothing is a multiple of eight
+        return H.HybridConfig(
+            vocab_size=83, hidden_dim=44, norm_eps=2e-5, logit_softcap=9.0, layers=(
+                L(D(6, 3, 10, 7, 2, 5, 3), M(50)),
+                L(A(6, 3, 12, 5, 5, 0.4, 9, 6, 300.0, False), None),
+                L(A(2, 1, 10, 6, 2, 0.3, 31, 10, 5000.0, True), M(21)),
+                L(D(2, 2, 5, 9, 1, 4, 6), None),
+                L(A(4, 1, 14, 6, 1, 0.2, 70, 4, 70.0, True), M(36)),
+            ))
+    if kind == "wide":        # vectorised paths, several pages per chunk, groups of 1, 3 and 8
+        return H.HybridConfig(
+            vocab_size=264, hidden_dim=96, norm_eps=1e-6, logit_softcap=20.0, layers=(
+                L(A(8, 1, 80, 40, 4, 0.11, 150, 48, 1e4, True), M(128)),
+                L(A(3, 1, 128, 40, 2, 0.09, 77, 64, 1e5, True), M(64)),
+                L(D(4, 2, 72, 40, 3, 16, 8), M(64)),
+                L(A(2, 2, 24, 136, 3, 0.2, 64, 16, 50.0, False), M(72)),
+                L(D(1, 1, 130, 16, 4, 8, 24), M(40)),
+            ))
+    if kind == "delta":       # recurrence only
+        return H.HybridConfig(
+            vocab_size=40, hidden_dim=24, norm_eps=1e-5, logit_softcap=5.0, layers=(
+                L(D(3, 1, 16, 8, 3, 4, 4), M(24)), L(D(2, 2, 8, 12, 2, 3, 5), M(16))))
+    return H.HybridConfig(    # "attn": attention only, without rotation, mask or cap
+        vocab_size=40, hidden_dim=32, norm_eps=1e-5, logit_softcap=None, layers=(
+            L(A(4, 2, 8, 8, 3, 0.35, None, 0, 1.0, True), M(24)),
+            L(A(6, 2, 6, 8, 2, 0.5, 16, 2, 10.0, True), M(24))))
+
+
+def weights(cfg, seed=0):
+    """Random weights under which old tokens matter: peaked attention, slow decay, sinks of some
+    weight, mixing far from 0 and 1."""
+    w = H.random_state(cfg, seed, dtype=torch.float32)
+    for i, layer in enumerate(cfg.layers):
+        p = f"l{i}.mix."
+        if isinstance(layer.mixer, A):
+            w[p + "q"] *= 2.5
+            if p + "vmix" in w:
+                w[p + "vmix"] = torch.tensor(0.35 + 0.1 * i)
+            w[p + "sink"] += 1.0
+        else:
+            w[p + "dt_bias"] -= 3.0
+    return {n: t.bfloat16() for n, t in w.items()}
+
+
+def plain_config(cfg):
+    d = H.config_to_json(cfg)
+    for layer in d["layers"]:
+        if layer["type"] == "attention":
+            layer["mixer"].setdefault("mask", {"size": 1 << 30})
+            layer["mixer"].setdefault("rot", {"dims": 0, "base": 1.0})
+    if d["logit_softcap"] is None:
+        d["logit_softcap"] = 1e9
+    return d
+
+
+_memo = {}
+
+
+def oracle(cfg, seed, ids):
+    """Logits of every position from the plain implementation, kept between tests."""
+    key = (cfg, seed, tuple(ids))
+    if key not in _memo:
+        _memo[key] = plain.forward(plain_config(cfg), weights(cfg, seed), list(ids))
+    return _memo[key]
+
+
+def tokens(cfg, n, seed):
+    g = torch.Generator().manual_seed(seed)
+    return torch.randint(0, cfg.vocab_size, (n,), generator=g).tolist()
+
+
+class Bench:
+    """One model on one device with its tolerance."""
+
+    def __init__(self, kind, device, dtype, seed=1):
+        self.cfg, self.seed = config(kind), seed
+        self.device, self.dtype = torch.device(device), dtype
+        self.lm = H.HybridLM(self.cfg, weights(self.cfg, seed), device, dtype)
+        self.tol = 2e-5 if dtype == torch.float32 else 0.05
+
+    def engine(self, slots=4, max_len=512, num_pages=None, **kw):
+        eng = make_engine(self.lm, max_batch=slots, **kw)
+        eng.open_slots(slots, max_len, num_pages=num_pages)
+        return eng
+
+    def close(self, got, want, tol=None):
+        """Root-mean-square difference over the vocabulary, relative to the oracle's spread."""
+        got = got[..., :self.cfg.vocab_size].double().cpu()
+        err = (got - want).square().mean(-1).sqrt() / want.std()
+        assert torch.isfinite(got).all()
+        assert float(err.max()) < (tol or self.tol), (float(err.max()), int(err.argmax()))
+
+    def whole(self, ids, eng=None):
+        eng = eng or self.engine(1)
+        return eng.step([R.Entry(0, 0, ids, range(len(ids)))]).clone()
+
+
+def feed(eng, slot, ids, cuts):
+    """Feeds ``ids`` in portions of the sizes ``cuts`` (repeated); all logits."""
+    out, at, i = [], 0, 0
+    while at < len(ids):
+        n = min(cuts[i % len(cuts)], len(ids) - at)
+        out.append(eng.step([R.Entry(slot, at, ids[at:at + n], range(n))]).clone())
+        at, i = at + n, i + 1
+    return torch.cat(out)
+
+
+# ------------------------------------------------------------------------------- model checks
+def check_whole_prompt(b):
+    for n, s in ((1, 2), (2, 3), (7, 4), (140, 5)):
+        ids = tokens(b.cfg, n, s)
+        b.close(b.whole(ids), oracle(b.cfg, b.seed, ids))
+
+
+def check_token_by_token(b):
+    ids = tokens(b.cfg, 140, 5)
+    b.close(feed(b.engine(1), 0, ids, [1]), oracle(b.cfg, b.seed, ids))
+
+
+def check_portions(b):
+    ids = tokens(b.cfg, 140, 5)
+    want = oracle(b.cfg, b.seed, ids)
+    for cuts in ([2], [3, 2], [63, 2, 1], [64], [17, 5, 31]):
+        b.close(feed(b.engine(1), 0, ids, cuts), want)
+
+
+def check_mixed_batches(b):
+    """Four unequal requests advance together, portions beside single tokens, one of them left out
+    of some steps; each gets what it gets alone."""
+    seqs = [tokens(b.cfg, n, 5 if n == 140 else n) for n in (140, 33, 90, 5)]
+    want = [oracle(b.cfg, b.seed, s) for s in seqs]
+    eng, at = b.engine(4), [0] * 4
+    plan = [(40, 3, 1, 2), (0, 1, 64, 1), (1, 1, 1, 1), (2, 0, 3, 0), (30, 28, 0, 1), (1, 1, 21, 1)]
+    k = 0
+    while any(a < len(s) for a, s in zip(at, seqs)):
+        takes = plan[k] if k < len(plan) else (7, 1, 1, 1)
+        k += 1
+        entries = []
+        for i, n in enumerate(takes):
+            part = seqs[i][at[i]:at[i] + n]
+            if part:
+                entries.append((i, R.Entry(i, at[i], part, range(len(part)))))
+        if not entries:
+            continue
+        out, r = eng.step([e for _, e in entries]), 0
+        for i, e in entries:
+            n = len(e.tokens)
+            b.close(out[r:r + n], want[i][at[i]:at[i] + n])
+            r, at[i] = r + n, at[i] + n
+
+
+def check_reuse(b):
+    """A pool of few pages and two slots: requests come and go, every page and slot changes hands,
+    in another order each time."""
+    eng = b.engine(2, max_len=192, num_pages=5)
+    seqs = [tokens(b.cfg, n, s) for n, s in ((140, 5), (33, 33), (70, 8), (140, 5), (90, 90), (1, 2))]
+    waiting, live, used = list(range(len(seqs))), {}, set()
+    free = [0, 1]
+    while waiting or live:
+        while waiting and free and (len(eng.cache.free) >= -(-len(seqs[waiting[0]]) // PAGE)):
+            i = waiting.pop(0)
+            slot = free.pop()
+            eng.cache.reserve(slot, len(seqs[i]))
+            used |= set(eng.cache.owned[slot])
+            live[i] = slot
+        entries = []
+        for i, slot in live.items():
+            at = eng.cache.length(slot)
+            entries.append((i, R.Entry(slot, at, seqs[i][at:at + 29 + 7 * i],
+                                       [len(seqs[i][at:at + 29 + 7 * i]) - 1])))
+        out = eng.step([e for _, e in entries]).clone()
+        for r, (i, e) in enumerate(entries):
+            end = e.pos0 + len(e.tokens)
+            b.close(out[r], oracle(b.cfg, b.seed, seqs[i])[end - 1])
+            if end == len(seqs[i]):
+                eng.release_slot(live[i])
+                free.append(live.pop(i))
+    assert len(used) == 5 and eng.cache.pages_in_use() == 0
+
+
+def check_long_decode(b):
+    ids = tokens(b.cfg, 330, 9)
+    want = oracle(b.cfg, b.seed, ids)
+    eng = b.engine(3)
+    first = eng.step([R.Entry(1, 0, ids[:10], range(10))])
+    b.close(first, want[:10])
+    got = torch.cat([eng.step([R.Entry(1, p, [ids[p]], [0])]).clone() for p in range(10, 330)])
+    b.close(got, want[10:])
+
+
+def plain_greedy(b, prompt, n):
+    ids = list(prompt)
+    for _ in range(n):
+        z = plain.forward(plain_config(b.cfg), weights(b.cfg, b.seed), ids)[-1]
+        ids.append(int(z.argmax()))
+    return ids[len(prompt):]
+
+
+def agrees(b, prompt, got):
+    """Greedy tokens: each is the oracle's arg-max after the tokens before it, up to the error the
+    logits may have."""
+    z = plain.forward(plain_config(b.cfg), weights(b.cfg, b.seed), list(prompt) + list(got))
+    for i, t in enumerate(got):
+        row = z[len(prompt) - 1 + i]
+        assert float(row.max() - row[t]) <= 3 * b.tol * float(z.std()), (i, t)
+
+
+def check_generate(b):
+    prompts = torch.tensor([tokens(b.cfg, 21, 11), tokens(b.cfg, 21, 12)], device=b.device)
+    eng = make_engine(b.lm, max_batch=2)
+    out = eng.generate(prompts, 12)
+    for row, p in zip(out.tolist(), prompts.tolist()):
+        assert row[:21] == p
+        agrees(b, p, row[21:])
+    again = eng.generate(prompts, 12, token_chunk=5, seq_chunk=1)     # other cuts, used slots
+    for row, p in zip(again.tolist(), prompts.tolist()):
+        agrees(b, p, row[21:])
+
+
+def check_batcher(b):
+    """More requests than slots through the scheduler, prompts read in portions beside decoding."""
+    cb = ContinuousBatcher(make_engine(b.lm, max_batch=3), max_seqs=3, max_len=128, token_chunk=9,
+                           step_tokens=16)
+    reqs = [(tokens(b.cfg, n, 20 + n), k) for n, k in ((5, 7), (40, 3), (1, 9), (23, 1), (17, 6))]
+    ids = {cb.submit(p, k): (p, k) for p, k in reqs}
+    out = cb.run()
+    for rid, (p, k) in ids.items():
+        assert len(out[rid]) == k
+        agrees(b, p, out[rid])
+    assert cb.engine.cache.pages_in_use() == 0 and cb.stats["prefills"] == len(reqs)
+
+
+# --------------------------------------------------------------------------- mechanism checks
+def rel(got, want):
+    got, want = got.double().cpu(), want.double()
+    return float((got - want).abs().max() / want.abs().max().clamp_min(1e-30))
+
+
+def rnd(shape, seed, device, dtype=torch.float32):
+    g = torch.Generator().manual_seed(seed)
+    return torch.randn(shape, generator=g).to(dtype).to(device)
+
+
+def batch_of(entries, device, tiles):
+    return R.RaggedBatch([R.Entry(s, p, [0] * n) for s, p, n in entries], device, tile_rows=tiles)
+
+
+def check_norms(device, dtype, tol):
+    x = rnd((5, 56), 1, device)
+    x[:, 50:] = 0
+    w1, w2 = (torch.nn.functional.pad(1 + rnd((50,), s, device), (0, 6)) for s in (2, 3))
+    y1, y2 = R.rms_rows(x, w1, 50, 3e-4, dtype, w2=w2)
+    xd = x[:, :50].cpu().double()
+    for y, w in ((y1, w1), (y2, w2)):
+        assert rel(y[:, :50], plain.rms_norm(xd, w[:50].cpu().double(), 3e-4)) < tol
+        assert float(y[:, 50:].abs().max()) == 0
+    rows = torch.tensor([4, 0, 2], dtype=torch.int32, device=device)
+    y, _ = R.rms_rows(x, w1, 50, 3e-4, dtype, rows=rows)
+    assert rel(y[:, :50], plain.rms_norm(xd[[4, 0, 2]], w1[:50].cpu().double(), 3e-4)) < tol
+    emb = torch.nn.functional.pad(rnd((9, 50), 4, device, dtype), (0, 6))
+    tok = torch.tensor([8, 0, 3], dtype=torch.int32, device=device)
+    out = torch.full((3, 56), 7.0, device=device)
+    R.embed_norm(tok, emb, w1, 50, 1e-5, out)
+    e = emb[[8, 0, 3], :50].cpu().double()
+    assert rel(out[:, :50], plain.rms_norm(e, w1[:50].cpu().double(), 1e-5)) < 1e-5
+    assert float(out[:, 50:].abs().max()) == 0
+
+
+def check_linear(device, dtype, tol):
+    for M_, N_, K_ in ((1, 8, 24), (3, 40, 8), (17, 136, 72), (70, 200, 136), (300, 520, 264)):
+        x, w = rnd((M_, K_), 1, device, dtype), rnd((N_, K_), 2, device, dtype)
+        z = x.cpu().double() @ w.cpu().double().T
+        y = torch.empty((M_, N_), dtype=dtype, device=device)
+        assert rel(G.linear(x, w, y), z) < tol
+        assert rel(G.linear(x, w, y, epi="relu2"), torch.relu(z).square()) < tol
+        f = rnd((M_, N_), 3, device)
+        start = f.cpu().double()
+        assert rel(G.linear(x, w, f, accumulate=True), start + z) < tol
+        assert rel(G.linear(x, w, torch.empty_like(f), softcap=4.0), plain.soft_cap(z, 4.0)) < tol
+
+
+def check_attention_inputs(device, dtype, tol):
+    """Convolution, rotation, value mixing and cache writes against the plain functions, one
+    sequence cut at several places, in two slots at once."""
+    for (H_, Gk, d, dv, taps, half, seed) in ((4, 2, 16, 8, 4, 8, 1), (3, 1, 10, 7, 2, 3, 2),
+                                              (2, 2, 24, 16, 1, 0, 3), (5, 1, 8, 12, 6, 4, 4)):
+        qc, kc, vc = H_ * d, Gk * d, Gk * dv
+        koff = (qc + 7) // 8 * 8
+        voff = koff + (kc + 7) // 8 * 8
+        ld = voff + (vc + 7) // 8 * 8
+        T = 75
+        raws = [rnd((T, ld), seed * 10 + s, device, dtype) for s in (0, 1)]
+        wt = rnd((taps, qc + kc + vc), seed + 50, device)
+        f = torch.tensor([300.0 ** (-2.0 * i / max(1, 2 * half)) for i in range(half)], device=device)
+        pages, table = 9, torch.tensor([[3, 1, 0], [7, 2, 8], [5, 4, 6]], dtype=torch.int32)
+        table = table.to(device)
+        kcache = torch.zeros((pages, PAGE, Gk, (d + 7) // 8 * 8), dtype=dtype, device=device)
+        vcache = torch.zeros((pages, PAGE, Gk, (dv + 7) // 8 * 8), dtype=dtype, device=device)
+        state = torch.full((3, taps - 1, qc + kc + vc), 9.0, dtype=dtype, device=device)
+        firsts = [rnd((T, vc), seed + 60 + s, device, dtype) for s in (0, 1)]
+        mix = torch.tensor([0.3], device=device)
+        qs = [[], []]
+        at = [0, 0]
+        for cut in ((1, 40), (2, 1), (1, 1), (30, 2), (40, 1), (1, 30)):
+            b = batch_of([(2, at[0], cut[0]), (0, at[1], cut[1])], device, False)
+            raw = torch.cat([raws[s][at[s]:at[s] + cut[s]] for s in (0, 1)])
+            vf = torch.cat([firsts[s][at[s]:at[s] + cut[s]] for s in (0, 1)])
+            rope = R.rope_table(b.pos, f) if half else None
+            q = R.shortconv_attn(raw, koff, voff, wt, state, H_, Gk, d, dv, b, rope, kcache, vcache,
+                                 table, v_first=vf, mix=mix)
+            qs[0].append(q[:cut[0]])
+            qs[1].append(q[cut[0]:])
+            at = [at[0] + cut[0], at[1] + cut[1]]
+        for s, slot in ((0, 2), (1, 0)):
+            raw = raws[s].cpu().double()
+            w = wt.cpu().double().T
+            u = torch.cat([raw[:, :qc], raw[:, koff:koff + kc], raw[:, voff:voff + vc]], 1)
+            y = plain.causal_conv(u, w)
+            want_q = plain.rotate_half(y[:, :qc].view(T, H_, d), 2 * half, 300.0) if half \
+                else y[:, :qc].view(T, H_, d)
+            want_k = y[:, qc:qc + kc].view(T, Gk, d)
+            want_k = plain.rotate_half(want_k, 2 * half, 300.0) if half else want_k
+            want_v = 0.7 * y[:, qc + kc:] + 0.3 * firsts[s].cpu().double()
+            assert rel(torch.cat(qs[s]), want_q.reshape(T, -1)) < tol
+            got_k = kcache[table[slot].long()].reshape(-1, Gk, kcache.shape[-1])[:T, :, :d]
+            got_v = vcache[table[slot].long()].reshape(-1, Gk, vcache.shape[-1])[:T, :, :dv]
+            assert rel(got_k, want_k) < tol
+            assert rel(got_v, want_v.view(T, Gk, dv)) < tol
+            if taps > 1:
+                assert torch.equal(state[slot].cpu().double(), u[-(taps - 1):])
+        # keeping v as the later layers' v_first
+        b = batch_of([(1, 0, 5)], device, False)
+        vf = torch.zeros((5, vc), dtype=dtype, device=device)
+        R.shortconv_attn(raws[0][:5], koff, voff, wt, state, H_, Gk, d, dv, b,
+                         R.rope_table(b.pos, f) if half else None, kcache, vcache, table, v_first=vf,
+                         write_first=True)
+        raw = raws[0][:5, voff:voff + vc].cpu().double()
+        assert rel(vf, plain.causal_conv(raw, wt[:, qc + kc:].cpu().double().T)) < tol
+
+
+def check_attention(device, dtype, tol):
+    """Rows at the edges of pages and chunks, with one key that stands out placed far away, just
+    inside and just outside; sinks from none to dominating; several group sizes and widths."""
+    g = torch.Generator().manual_seed(0)
+    for H_, Gk, d, dv, chunk in ((4, 1, 64, 48, 120), (6, 2, 40, 24, 50), (2, 2, 10, 7, 9),
+                                 (9, 1, 72, 128, 200), (3, 3, 136, 200, 64), (4, 4, 128, 64, None),
+                                 (2, 1, 16, 16, 1)):
+        n = 260
+        k = torch.randn((n, Gk, d), generator=g).to(dtype)
+        v = torch.randn((n, Gk, dv), generator=g).to(dtype)
+        table = torch.randperm(7, generator=g)[:5].int()[None].to(device)
+        dp, dvp = (d + 7) // 8 * 8, (dv + 7) // 8 * 8
+        kc = torch.zeros((7, PAGE, Gk, dp), dtype=dtype)
+        vc = torch.zeros((7, PAGE, Gk, dvp), dtype=dtype)
+        for t in range(n):
+            page = int(table[0, t // PAGE])
+            kc[page, t % PAGE, :, :d], vc[page, t % PAGE, :, :dv] = k[t], v[t]
+        kc, vc = kc.to(device), vc.to(device)
+        size = chunk or 1 << 30
+        scale = 0.7 / d ** 0.5
+        sink = torch.linspace(-3.0, 4.0, H_)
+        span = [p for c in (chunk or 64, 64) for e in range(c, n, c) for p in (e - 1, e, e + 1)]
+        pos = sorted({0, 1, n - 1, *[p for p in span if p < n]})[:40]
+        for start, m in [(p, 1) for p in pos] + [(0, 70), (50, 100), (117, 66), (n - 6, 6)]:
+            m = min(m, n - start)
+            q = torch.randn((m, H_, d), generator=g)
+            # each row points at one key: its chunk's first, the one before it, itself, or a far one
+            for r in range(m):
+                i = start + r
+                lo = i // size * size
+                j = [lo, max(lo - 1, 0), i, (i * 7) % (i + 1)][r % 4 if m > 1 else i % 4]
+                q[r] += 3.0 * k[j].double().repeat_interleave(H_ // Gk, 0)
+            q = q.to(dtype)
+            gate = torch.randn((m, H_ + 3), generator=g).to(dtype)
+            b = batch_of([(0, start, m)], device, tiles=dtype == torch.bfloat16)
+            out = torch.full((m, H_ * dv + 8), 5.0, dtype=dtype, device=device)
+            R.ragged_attention(q.reshape(m, -1).to(device), kc, vc, table, b, H_, Gk, d, dv, scale,
+                               out[:, :H_ * dv], chunk=chunk, sink=sink.to(device),
+                               gate=gate.to(device)[:, 2:])
+            want = torch.zeros(m, H_, dv, dtype=torch.float64)
+            for r in range(m):
+                i = start + r
+                js = [j for j in range(i + 1) if plain.chunk_visible(i, j, size)]
+                for h in range(H_):
+                    s = (k[js, h // (H_ // Gk)].double() @ q[r, h].double()) * scale
+                    want[r, h] = plain.sink_softmax(s, sink[h].double()) @ v[js, h // (H_ // Gk)].double()
+            want *= torch.sigmoid(gate[:, 2:2 + H_].double())[:, :, None]
+            assert rel(out[:, :H_ * dv], want.reshape(m, -1)) < tol, (H_, d, chunk, start, m)
+            assert float((out[:, H_ * dv:].float() - 5.0).abs().max()) == 0
+
+
+def check_delta(device, dtype, tol):
+    """Inputs of the recurrence, the recurrence and the gated norm, cut at several places."""
+    for H_, Gk, d, dv, taps, seed in ((4, 2, 16, 24, 3, 1), (3, 1, 10, 7, 1, 2), (2, 2, 70, 40, 4, 3),
+                                      (1, 1, 130, 9, 2, 4), (2, 1, 200, 33, 2, 5)):
+        qc, vc = Gk * d, H_ * dv
+        koff = (qc + 7) // 8 * 8
+        voff = koff + koff
+        boff = voff + (vc + 7) // 8 * 8
+        ld = boff + 8
+        T = 60
+        raws = [rnd((T, ld), seed * 10 + s, device, dtype) for s in (0, 1)]
+        avs = [rnd((T, H_ * d), seed * 10 + 5 + s, device) for s in (0, 1)]
+        wt = rnd((taps, 2 * qc + vc), seed + 50, device)
+        A_log, dt = rnd((H_,), seed + 51, device), rnd((H_ * d,), seed + 52, device) - 2.0
+        nw = 1 + rnd((dv,), seed + 53, device)
+        conv = torch.full((3, taps - 1, 2 * qc + vc), 9.0, dtype=dtype, device=device)
+        state = torch.full((3, H_, d, dv), 9.0, device=device)
+        gates = [rnd((T, H_ * dv), seed + 54 + s, device, dtype) for s in (0, 1)]
+        outs, at = [[], []], [0, 0]
+        for cut in ((1, 20), (2, 1), (1, 1), (16, 2), (39, 1), (1, 35)):
+            b = batch_of([(2, at[0], cut[0]), (0, at[1], cut[1])], device, False)
+            raw = torch.cat([raws[s][at[s]:at[s] + cut[s]] for s in (0, 1)])
+            a = torch.cat([avs[s][at[s]:at[s] + cut[s]] for s in (0, 1)])
+            gt = torch.cat([gates[s][at[s]:at[s] + cut[s]] for s in (0, 1)])
+            x = R.shortconv_delta(raw, koff, voff, boff, wt, conv, H_, Gk, d, dv, b, a, A_log, dt)
+            o = R.delta_scan(*x, state, b)
+            y = torch.zeros((sum(cut), H_ * dv), dtype=dtype, device=device)
+            R.gated_head_norm(o, gt, nw, 1e-4, y)
+            outs[0].append((o[:cut[0]], y[:cut[0]]))
+            outs[1].append((o[cut[0]:], y[cut[0]:]))
+            at = [at[0] + cut[0], at[1] + cut[1]]
+        for s, slot in ((0, 2), (1, 0)):
+            raw = raws[s].cpu().double()
+            u = torch.cat([raw[:, :qc], raw[:, koff:koff + qc], raw[:, voff:voff + vc]], 1)
+            y = plain.silu(plain.causal_conv(u, wt.cpu().double().T))
+            q = plain.unit(y[:, :qc].view(T, Gk, d)) * d ** -0.5
+            k = plain.unit(y[:, qc:2 * qc].view(T, Gk, d))
+            v = y[:, 2 * qc:].view(T, H_, dv)
+            beta = torch.sigmoid(raw[:, boff:boff + H_])
+            g = plain.channel_decay(avs[s].cpu().double().view(T, H_, d), A_log.cpu().double(),
+                                    dt.cpu().double())
+            per = H_ // Gk
+            want = torch.empty(T, H_, dv, dtype=torch.float64)
+            for h in range(H_):
+                want[:, h], S = plain.delta_scan(q[:, h // per], k[:, h // per], v[:, h], g[:, h],
+                                                 beta[:, h])
+                assert rel(state[slot, h], S) < 5e-5
+            assert rel(torch.cat([o for o, _ in outs[s]]), want) < 5e-5
+            n = plain.rms_norm(want, nw.cpu().double(), 1e-4) * \
+                torch.sigmoid(gates[s].cpu().double()).view(T, H_, dv)
+            assert rel(torch.cat([y for _, y in outs[s]]), n.reshape(T, -1)) < tol
+            if taps > 1:
+                assert torch.equal(conv[slot].cpu().double(), u[-(taps - 1):])
+
+
+MODEL_CHECKS = [check_whole_prompt, check_token_by_token, check_portions, check_mixed_batches,
+                check_reuse, check_long_decode, check_generate, check_batcher]
+MECHANISM_CHECKS = [check_norms, check_linear, check_attention_inputs, check_attention, check_delta]
