@@ -39,7 +39,8 @@ NVCC_FLAGS = [
 ]
 
 
-SERVING_SOURCES = ("gemm", "ragged_rows", "shortconv", "delta_scan", "linear_f32", "ragged_attn")
+SERVING_SOURCES = ("gemm", "ragged_rows", "shortconv", "delta_scan", "linear_f32", "linear_skinny",
+                   "ragged_attn")
 
 
 def _nvcc() -> str:

@@ -42,24 +42,26 @@ __device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
 constexpr int SCAN_WARPS = 4;
 constexpr int SCAN_COLS = SCAN_WARPS * 8;
 constexpr int SCAN_TB = 8;         // tokens per stage
+constexpr int SCAN_STAGES = 3;
 
 struct ScanArgs {
-  const float* q;      // [rows, kv_heads, dim4]
-  const float* k;      // [rows, kv_heads, dim4]
-  const float* kq;     // [rows, kv_heads]
+  const float* q;      // [kv_heads, rows, DP], DP = dim rounded up to a multiple of 32
+  const float* k;      // [kv_heads, rows, DP]
+  const float* kq;     // [kv_heads, rows]
   const float* v;      // [rows, heads, vdim]
-  const float* g;      // [rows, heads, dim4]
-  const float* beta;   // [rows, heads]
+  const float* g;      // [heads, rows, DP]
+  const float* beta;   // [heads, rows]
   float* state;        // [slots, heads, dim, vdim]
   float* o;            // out [rows, heads, vdim]
-  int heads, kv_heads, dim, dim4, vdim;
+  int rows, heads, kv_heads, dim, vdim;
   Entries e;
 };
 
-template <int R>       // key channels per lane; 8 R >= dim, R a multiple of 4
+template <int R>       // key channels per lane, a multiple of 4; DP = 8 R
 __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanArgs p) {
-  constexpr int DP = 8 * R;                                  // channels, padded with zeros
-  constexpr int STAGE = SCAN_TB * (3 * DP + SCAN_COLS + 4);  // floats
+  constexpr int DP = 8 * R;
+  constexpr int STAGE = SCAN_TB * (3 * DP + SCAN_COLS + 2);  // floats
+  constexpr int THREADS = SCAN_WARPS * 32;
   extern __shared__ __align__(16) float sm[];
   const int e = blockIdx.y, h = blockIdx.x % p.heads, slab = blockIdx.x / p.heads;
   const int hk = h / (p.heads / p.kv_heads);
@@ -68,37 +70,47 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
   const int col_base = slab * SCAN_COLS;
   const int c0 = warp * 8 + (lane >> 3) * 2;                 // first of this lane's two columns
   float* st = p.state + (static_cast<size_t>(slot) * p.heads + h) * p.dim * p.vdim;
+  const float* gq = p.q + (static_cast<size_t>(hk) * p.rows + row0) * DP;
+  const float* gk = p.k + (static_cast<size_t>(hk) * p.rows + row0) * DP;
+  const float* gg = p.g + (static_cast<size_t>(h) * p.rows + row0) * DP;
+  const float* gv = p.v + (static_cast<size_t>(row0) * p.heads + h) * p.vdim + col_base;
+  const float* gb = p.beta + static_cast<size_t>(h) * p.rows + row0;
+  const float* gkq = p.kq + static_cast<size_t>(hk) * p.rows + row0;
+  const int vstride = p.heads * p.vdim;
 
+  // tokens t0 .. t0 + SCAN_TB - 1 into a stage: q, k and g are contiguous blocks
   auto fetch = [&](int stage, int t0) {
     const uint32_t base = smem_u32(sm + stage * STAGE);
     const int n = min(SCAN_TB, len - t0);
-    constexpr int CH = DP / 4;
-    for (int i = threadIdx.x; i < n * 3 * CH; i += SCAN_WARPS * 32) {
-      const int t = i / (3 * CH), w = (i / CH) % 3, c = i % CH;
-      const int row = row0 + t0 + t;
-      const bool in = c * 4 < p.dim4;
-      const float* src = w == 2 ? p.g + (static_cast<size_t>(row) * p.heads + h) * p.dim4
-                                : (w == 0 ? p.q : p.k) +
-                                      (static_cast<size_t>(row) * p.kv_heads + hk) * p.dim4;
-      cp_async16_zfill(base + ((t * 3 + w) * DP + c * 4) * 4, src + (in ? c * 4 : 0), in ? 16 : 0);
+    const int at = t0 * DP;
+#pragma unroll
+    for (int i = threadIdx.x; i < SCAN_TB * DP / 4; i += THREADS) {
+      if (i < n * (DP / 4)) {
+        cp_async16(base + i * 16, gq + at + i * 4);
+        cp_async16(base + (SCAN_TB * DP + i * 4) * 4, gk + at + i * 4);
+        cp_async16(base + (2 * SCAN_TB * DP + i * 4) * 4, gg + at + i * 4);
+      }
     }
     const uint32_t vb = base + SCAN_TB * 3 * DP * 4;
-    for (int i = threadIdx.x; i < n * SCAN_COLS; i += SCAN_WARPS * 32) {
+#pragma unroll
+    for (int i = threadIdx.x; i < SCAN_TB * SCAN_COLS; i += THREADS) {
       const int t = i / SCAN_COLS, c = i % SCAN_COLS;
-      if (col_base + c < p.vdim)
-        cp_async4(vb + i * 4, p.v + (static_cast<size_t>(row0 + t0 + t) * p.heads + h) * p.vdim +
-                                  col_base + c);
+      if (t < n && col_base + c < p.vdim)
+        cp_async4(vb + i * 4, gv + static_cast<size_t>(t0 + t) * vstride + c);
     }
-    const uint32_t sb = vb + SCAN_TB * SCAN_COLS * 4;
-    for (int i = threadIdx.x; i < n * 2; i += SCAN_WARPS * 32) {
-      const int row = row0 + t0 + (i >> 1);
-      cp_async4(sb + i * 4, (i & 1) ? p.kq + static_cast<size_t>(row) * p.kv_heads + hk
-                                    : p.beta + static_cast<size_t>(row) * p.heads + h);
+    if (threadIdx.x < 2 * SCAN_TB) {
+      const int t = threadIdx.x % SCAN_TB;
+      if (t < n)
+        cp_async4(vb + (SCAN_TB * SCAN_COLS + threadIdx.x) * 4,
+                  (threadIdx.x < SCAN_TB ? gb : gkq) + t0 + t);
     }
     cp_async_commit();
   };
 
-  fetch(0, 0);
+  for (int i = 0; i < SCAN_STAGES - 1; ++i) {
+    if (i * SCAN_TB < len) fetch(i, i * SCAN_TB);
+    else cp_async_commit();
+  }
   f2 s[2][R / 2];
   const bool has_state = p.e.pos0[e] > 0;
 #pragma unroll
@@ -117,28 +129,26 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
   }
   const int my = c0 + ((ld >> 1) & 1);                       // the column this lane finishes
   int stage = 0;
-  for (int t0 = 0; t0 < len; t0 += SCAN_TB, stage ^= 1) {
-    const bool more = t0 + SCAN_TB < len;
-    if (more) {
-      fetch(stage ^ 1, t0 + SCAN_TB);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
+  for (int t0 = 0; t0 < len; t0 += SCAN_TB) {
+    cp_async_wait<SCAN_STAGES - 2>();
+    __syncthreads();                       // the stage is filled, and the one before it is free
+    const int ahead = t0 + (SCAN_STAGES - 1) * SCAN_TB;
+    if (ahead < len) fetch((stage + SCAN_STAGES - 1) % SCAN_STAGES, ahead);
+    else cp_async_commit();
     const float* sb = sm + stage * STAGE;
     const float* sv = sb + SCAN_TB * 3 * DP;
     const float* ss = sv + SCAN_TB * SCAN_COLS;
     const int n = min(SCAN_TB, len - t0);
+    stage = (stage + 1) % SCAN_STAGES;
     for (int t = 0; t < n; ++t) {
-      const float* tq = sb + t * 3 * DP + ld * 4;
+      const float* tq = sb + t * DP + ld * 4;
       f2 a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull;
       f2 kk[R / 2];
 #pragma unroll
       for (int j = 0; j < R / 4; ++j) {
         const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(tq + j * 32);
-        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(tq + DP + j * 32);
-        const ulonglong2 g2 = *reinterpret_cast<const ulonglong2*>(tq + 2 * DP + j * 32);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(tq + SCAN_TB * DP + j * 32);
+        const ulonglong2 g2 = *reinterpret_cast<const ulonglong2*>(tq + 2 * SCAN_TB * DP + j * 32);
         kk[2 * j] = k2.x;
         kk[2 * j + 1] = k2.y;
         s[0][2 * j] = mul_f2(s[0][2 * j], g2.x);
@@ -162,7 +172,7 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
       float x1 = (odd ? fb1 : fa1) + __shfl_xor_sync(0xffffffffu, odd ? fa1 : fb1, 1);
       float y = (hi ? x1 : x0) + __shfl_xor_sync(0xffffffffu, hi ? x0 : x1, 2);
       y += __shfl_xor_sync(0xffffffffu, y, 4);
-      const float beta = ss[t * 2], kq = ss[t * 2 + 1];
+      const float beta = ss[t], kq = ss[SCAN_TB + t];
       const float un = beta * (sv[t * SCAN_COLS + my] - y);  // of use on even lanes
       const float u0 = __shfl_sync(0xffffffffu, un, lane & 24);
       const float u1 = __shfl_sync(0xffffffffu, un, (lane & 24) | 2);
@@ -176,7 +186,6 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
         p.o[(static_cast<size_t>(row0 + t0 + t) * p.heads + h) * p.vdim + col_base + my] =
             y + kq * (hi ? u1 : u0);
     }
-    __syncthreads();                                         // the stage may be refilled
   }
 #pragma unroll
   for (int c = 0; c < 2; ++c) {
@@ -194,7 +203,7 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
 
 template <int R>
 static int launch_scan(const ScanArgs& a, int entries, cudaStream_t st) {
-  const int smem = 2 * SCAN_TB * (3 * 8 * R + SCAN_COLS + 4) * 4;
+  const int smem = SCAN_STAGES * SCAN_TB * (3 * 8 * R + SCAN_COLS + 2) * 4;
   static bool set = false;
   if (!set) {
     if (cudaFuncSetAttribute(delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -212,21 +221,25 @@ static int launch_scan(const ScanArgs& a, int entries, cudaStream_t st) {
 using namespace cb;
 
 extern "C" int cb_delta_scan(const float* q, const float* k, const float* kq, const float* v,
-                             const float* g, const float* beta, float* state, float* o, int heads,
-                             int kv_heads, int dim, int dim4, int vdim, const int* slot,
+                             const float* g, const float* beta, float* state, float* o, int rows,
+                             int heads, int kv_heads, int dim, int dim_p, int vdim, const int* slot,
                              const int* row0, const int* len, const int* pos0, int entries,
                              void* stream) {
-  if (entries <= 0 || entries > 65535 || heads % kv_heads != 0) return -1;
-  if (dim > 256 || dim4 < dim || dim4 % 4 != 0) return -2;
+  if (entries <= 0 || entries > 65535 || kv_heads < 1 || heads % kv_heads != 0) return -1;
+  if (dim < 1 || dim > 256 || dim_p != (dim + 31) / 32 * 32) return -2;
   ScanArgs a;
   a.q = q; a.k = k; a.kq = kq; a.v = v; a.g = g; a.beta = beta; a.state = state; a.o = o;
-  a.heads = heads; a.kv_heads = kv_heads; a.dim = dim; a.dim4 = dim4; a.vdim = vdim;
+  a.rows = rows; a.heads = heads; a.kv_heads = kv_heads; a.dim = dim; a.vdim = vdim;
   a.e.slot = slot; a.e.row0 = row0; a.e.len = len; a.e.pos0 = pos0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dim <= 32) return launch_scan<4>(a, entries, st);
-  if (dim <= 64) return launch_scan<8>(a, entries, st);
-  if (dim <= 96) return launch_scan<12>(a, entries, st);
-  if (dim <= 128) return launch_scan<16>(a, entries, st);
-  if (dim <= 192) return launch_scan<24>(a, entries, st);
-  return launch_scan<32>(a, entries, st);
+  switch (dim_p / 32) {
+    case 1: return launch_scan<4>(a, entries, st);
+    case 2: return launch_scan<8>(a, entries, st);
+    case 3: return launch_scan<12>(a, entries, st);
+    case 4: return launch_scan<16>(a, entries, st);
+    case 5: return launch_scan<20>(a, entries, st);
+    case 6: return launch_scan<24>(a, entries, st);
+    case 7: return launch_scan<28>(a, entries, st);
+    default: return launch_scan<32>(a, entries, st);
+  }
 }

@@ -35,11 +35,16 @@ __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 
-// V (1 or 8) consecutive values; the 8-wide form needs 16-byte (bf16) / 32-byte-multiple rows.
+// V (1, 4 or 8) consecutive values, aligned to the vector (fp32: to 16 bytes).
 template <int V>
 __device__ __forceinline__ void load_vec(const __nv_bfloat16* p, float* f) {
-  if constexpr (V == 8) load8(p, f);
-  else f[0] = __bfloat162float(*p);
+  if constexpr (V == 8) {
+    load8(p, f);
+  } else if constexpr (V == 4) {
+    const uint2 x = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(x.x), b = unpack_bf16x2(x.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else f[0] = __bfloat162float(*p);
 }
 template <int V>
 __device__ __forceinline__ void load_vec(const float* p, float* f) {
@@ -47,6 +52,9 @@ __device__ __forceinline__ void load_vec(const float* p, float* f) {
     const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
     f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
     f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  } else if constexpr (V == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
   } else {
     f[0] = *p;
   }

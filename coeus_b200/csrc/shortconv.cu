@@ -39,27 +39,46 @@ __device__ __forceinline__ int raw_col_delta(const ConvIn& p, int c) {
   return c < qc ? c : (c < 2 * qc ? p.koff + (c - qc) : p.voff + (c - 2 * qc));
 }
 
-// V consecutive channels from c (columns from col) of the token at offset t of the entry.
-template <typename T, int V>
+// V consecutive channels from c (columns from col) of the token at offset t of the entry.  TAPS > 0
+// is the number of taps, known at compile time so that all loads are issued together; 0: any.
+template <typename T, int V, int TAPS>
 __device__ __forceinline__ void conv_at(const ConvIn& p, int c, int col, int channels, int row0,
                                         int t, int slot, bool has_state, float* y) {
+  const T* raw = static_cast<const T*>(p.raw) + static_cast<ptrdiff_t>(row0) * p.ld + col;
+  const int n1 = (TAPS > 0 ? TAPS : p.taps) - 1;
+  const T* st = static_cast<const T*>(p.state) + static_cast<ptrdiff_t>(slot) * n1 * channels + c;
 #pragma unroll
   for (int i = 0; i < V; ++i) y[i] = 0.f;
-  const T* raw = static_cast<const T*>(p.raw);
-  const T* st = static_cast<const T*>(p.state);
-  const int n1 = p.taps - 1;
-  for (int j = 0; j <= n1; ++j) {
-    const int o = t - n1 + j;
-    float u[V], w[V];
-    if (o >= 0) {
-      load_vec<V>(raw + static_cast<size_t>(row0 + o) * p.ld + col, u);
-    } else {
-      if (!has_state) continue;
-      load_vec<V>(st + (static_cast<size_t>(slot) * n1 + (n1 + o)) * channels + c, u);
-    }
-    load_vec<V>(p.taps_w + static_cast<size_t>(j) * channels + c, w);
+  if constexpr (TAPS > 0) {
+    float u[TAPS][V], w[TAPS][V];
 #pragma unroll
-    for (int i = 0; i < V; ++i) y[i] += u[i] * w[i];
+    for (int j = 0; j < TAPS; ++j) {
+      const int o = t - (TAPS - 1) + j;
+      const bool ok = o >= 0 || has_state;
+      const T* src = o >= 0 || !ok ? raw + static_cast<ptrdiff_t>(max(o, 0)) * p.ld
+                                   : st + static_cast<ptrdiff_t>(n1 + o) * channels;
+      load_vec<V>(src, u[j]);
+      load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * channels + c, w[j]);
+      if (!ok) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) u[j][i] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[i] += u[j][i] * w[j][i];
+  } else {
+    for (int j = 0; j <= n1; ++j) {
+      const int o = t - n1 + j;
+      float u[V], w[V];
+      if (o < 0 && !has_state) continue;
+      load_vec<V>(o >= 0 ? raw + static_cast<ptrdiff_t>(o) * p.ld
+                         : st + static_cast<ptrdiff_t>(n1 + o) * channels, u);
+      load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * channels + c, w);
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[i] += u[i] * w[i];
+    }
   }
 }
 
@@ -96,7 +115,7 @@ struct AttnPre {
 };
 
 // grid (tiles, kv_heads): the block's channels are its key/value head and the query heads on it.
-template <typename T, int V>
+template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const AttnPre p) {
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -130,8 +149,8 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
       if (k < pair_u) {
         const int d = k * V;
         float a[V], b[V], oa[V], ob[V];
-        conv_at<T, V>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
-        conv_at<T, V>(ci, base + p.half + d, colb + p.half + d, channels, row0, t, slot, has_state, b);
+        conv_at<T, V, TAPS>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
+        conv_at<T, V, TAPS>(ci, base + p.half + d, colb + p.half + d, channels, row0, t, slot, has_state, b);
 #pragma unroll
         for (int x = 0; x < V; ++x) {
           const float2 cs = p.rope[static_cast<size_t>(row) * p.half + d + x];
@@ -143,13 +162,13 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
       } else {
         const int d = 2 * p.half + (k - pair_u) * V;
         float a[V];
-        conv_at<T, V>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
+        conv_at<T, V, TAPS>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
         store_vec<V>(dst + d, a);
       }
     } else {
       const int d = (u - (per + 1) * head_u) * V;
       float a[V];
-      conv_at<T, V>(ci, qc + kc + g * vdim + d, ci.voff + g * vdim + d, channels, row0, t, slot,
+      conv_at<T, V, TAPS>(ci, qc + kc + g * vdim + d, ci.voff + g * vdim + d, channels, row0, t, slot,
                     has_state, a);
       if (p.mix_mode != 0) {
         T* vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d;
@@ -184,22 +203,37 @@ struct DeltaPre {
   int lda;
   const float* A_log;      // [heads]
   const float* dt_bias;    // [heads * dim]
-  float* q;                // out [rows, kv_heads, dim4] unit norm, scaled by dim^-1/2
-  float* k;                // out [rows, kv_heads, dim4] unit norm
-  float* kq;               // out [rows, kv_heads] their dot product
+  float* q;                // out [kv_heads, rows, dim_p] unit norm, scaled by dim^-1/2
+  float* k;                // out [kv_heads, rows, dim_p] unit norm
+  float* kq;               // out [kv_heads, rows] their dot product
   float* v;                // out [rows, heads, vdim]
-  float* g;                // out [rows, heads, dim4] decay factors
-  float* beta;             // out [rows, heads]
-  int dim4;                // dim rounded up to a multiple of 4; the padding is zero
+  float* g;                // out [heads, rows, dim_p] decay factors
+  float* beta;             // out [heads, rows]
+  int rows, dim_p;         // dim_p: dim rounded up to a multiple of 32; the padding is zero
 };
 
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_exact(float x) {
   return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
 }
+template <int V>
+__device__ __forceinline__ void load_f32(const float* p, float* f) {
+  if constexpr (V == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_f32(float* p, const float* f) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
 
-// grid (tiles, kv_heads): one query/key head and the value heads on it.
-template <typename T>
+// grid (tiles, kv_heads): one query/key head and the value heads on it.  V consecutive channels
+// per thread (4 when dim and vdim are multiples of four).
+template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_kernel(const DeltaPre p) {
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -213,56 +247,73 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_kernel(const Del
   const float qscale = 1.0f / sqrtf(static_cast<float>(dim));
   // q and k: a warp per token
   for (int t = off + warp; t < off + nt; t += CONV_THREADS / 32) {
-    constexpr int MAXD = 8;                      // dim <= 256
-    float qv[MAXD], kv[MAXD], sq = 0.f, sk = 0.f, dot = 0.f;
+    constexpr int NI = 256 / (32 * V);           // dim <= 256
+    float qv[NI][V], kv[NI][V], sq = 0.f, sk = 0.f, dot = 0.f;
 #pragma unroll
-    for (int i = 0; i < MAXD; ++i) {
-      const int d = lane + 32 * i;
-      qv[i] = kv[i] = 0.f;
+    for (int i = 0; i < NI; ++i) {
+      const int d = (lane + 32 * i) * V;
+#pragma unroll
+      for (int x = 0; x < V; ++x) qv[i][x] = kv[i][x] = 0.f;
       if (d < dim) {
-        conv_at<T, 1>(ci, g * dim + d, g * dim + d, channels, row0, t, slot, has_state, &qv[i]);
-        conv_at<T, 1>(ci, qc + g * dim + d, ci.koff + g * dim + d, channels, row0, t, slot, has_state, &kv[i]);
-        qv[i] = silu_exact(qv[i]);
-        kv[i] = silu_exact(kv[i]);
+        conv_at<T, V, TAPS>(ci, g * dim + d, g * dim + d, channels, row0, t, slot, has_state, qv[i]);
+        conv_at<T, V, TAPS>(ci, qc + g * dim + d, ci.koff + g * dim + d, channels, row0, t, slot, has_state, kv[i]);
+#pragma unroll
+        for (int x = 0; x < V; ++x) {
+          qv[i][x] = silu_exact(qv[i][x]);
+          kv[i][x] = silu_exact(kv[i][x]);
+          sq += qv[i][x] * qv[i][x];
+          sk += kv[i][x] * kv[i][x];
+        }
       }
-      sq += qv[i] * qv[i];
-      sk += kv[i] * kv[i];
     }
     const float rq = qscale / sqrtf(warp_sum(sq) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f);
-    const size_t cell = static_cast<size_t>(row0 + t) * ci.kv_heads + g;
+    const size_t cell = static_cast<size_t>(g) * p.rows + row0 + t;
 #pragma unroll
-    for (int i = 0; i < MAXD; ++i) {
-      const int d = lane + 32 * i;
-      const float a = qv[i] * rq, b = kv[i] * rk;
-      dot += a * b;
-      if (d < p.dim4) {
-        p.q[cell * p.dim4 + d] = a;
-        p.k[cell * p.dim4 + d] = b;
+    for (int i = 0; i < NI; ++i) {
+      const int d = (lane + 32 * i) * V;
+#pragma unroll
+      for (int x = 0; x < V; ++x) {
+        qv[i][x] *= rq;
+        kv[i][x] *= rk;
+        dot += qv[i][x] * kv[i][x];
+      }
+      if (d < p.dim_p) {
+        store_f32<V>(p.q + cell * p.dim_p + d, qv[i]);
+        store_f32<V>(p.k + cell * p.dim_p + d, kv[i]);
       }
     }
     dot = warp_sum(dot);
     if (lane == 0) p.kq[cell] = dot;
   }
   const T* raw = static_cast<const T*>(ci.raw);
-  for (int i = threadIdx.x; i < nt * per * vdim; i += CONV_THREADS) {
-    const int t = off + i / (per * vdim), c = g * per * vdim + i % (per * vdim);
-    float y;
-    conv_at<T, 1>(ci, 2 * qc + c, ci.voff + c, channels, row0, t, slot, has_state, &y);
-    p.v[static_cast<size_t>(row0 + t) * ci.heads * vdim + c] = silu_exact(y);
+  const int vn = per * vdim / V;
+  for (int i = threadIdx.x; i < nt * vn; i += CONV_THREADS) {
+    const int t = off + i / vn, c = g * per * vdim + (i % vn) * V;
+    float y[V];
+    conv_at<T, V, TAPS>(ci, 2 * qc + c, ci.voff + c, channels, row0, t, slot, has_state, y);
+#pragma unroll
+    for (int x = 0; x < V; ++x) y[x] = silu_exact(y[x]);
+    store_f32<V>(p.v + static_cast<size_t>(row0 + t) * ci.heads * vdim + c, y);
   }
-  for (int i = threadIdx.x; i < nt * per * p.dim4; i += CONV_THREADS) {
-    const int t = off + i / (per * p.dim4), x = i % (per * p.dim4);
-    const int h = g * per + x / p.dim4, d = x % p.dim4;
-    float f = 0.f;
+  const int gn = p.dim_p / V;
+  for (int i = threadIdx.x; i < nt * per * gn; i += CONV_THREADS) {
+    const int h = g * per + (i / gn) % per, row = row0 + off + i / (gn * per), d = (i % gn) * V;
+    float f[V];
+#pragma unroll
+    for (int x = 0; x < V; ++x) f[x] = 0.f;
     if (d < dim) {
-      const float a = p.a[static_cast<size_t>(row0 + t) * p.lda + h * dim + d] + p.dt_bias[h * dim + d];
-      f = expf(-expf(p.A_log[h]) * softplus_exact(a));
+      float a[V], b[V];
+      load_f32<V>(p.a + static_cast<size_t>(row) * p.lda + h * dim + d, a);
+      load_f32<V>(p.dt_bias + h * dim + d, b);
+      const float rate = expf(p.A_log[h]);
+#pragma unroll
+      for (int x = 0; x < V; ++x) f[x] = expf(-rate * softplus_exact(a[x] + b[x]));
     }
-    p.g[(static_cast<size_t>(row0 + t) * ci.heads + h) * p.dim4 + d] = f;
+    store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row) * p.dim_p + d, f);
   }
   for (int i = threadIdx.x; i < nt * per; i += CONV_THREADS) {
-    const int row = row0 + off + i / per, h = g * per + i % per;
-    p.beta[static_cast<size_t>(row) * ci.heads + h] =
+    const int h = g * per + i / nt, row = row0 + off + i % nt;
+    p.beta[static_cast<size_t>(h) * p.rows + row] =
         sigmoidf_(to_f32(raw[static_cast<size_t>(row) * ci.ld + p.boff + h]));
   }
   if (off == 0 && ci.taps > 1) {
@@ -274,6 +325,27 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_kernel(const Del
       conv_advance<T>(ci, c, raw_col_delta(ci, c), channels, row0, len, slot, has_state);
     }
   }
+}
+
+template <typename T, int V>
+static int launch_conv_attn(const AttnPre& p, dim3 grid, cudaStream_t st) {
+  switch (p.c.taps) {
+    case 2: shortconv_attn_kernel<T, V, 2><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    case 3: shortconv_attn_kernel<T, V, 3><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    case 4: shortconv_attn_kernel<T, V, 4><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    default: shortconv_attn_kernel<T, V, 0><<<grid, CONV_THREADS, 0, st>>>(p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+template <typename T, int V>
+static int launch_conv_delta(const DeltaPre& p, dim3 grid, cudaStream_t st) {
+  switch (p.c.taps) {
+    case 2: shortconv_delta_kernel<T, V, 2><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    case 3: shortconv_delta_kernel<T, V, 3><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    case 4: shortconv_delta_kernel<T, V, 4><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    default: shortconv_delta_kernel<T, V, 0><<<grid, CONV_THREADS, 0, st>>>(p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
 }  // namespace cb
@@ -315,14 +387,10 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
                    voff % 8 == 0;
   dim3 grid(tiles, kv_heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) {
-    if (vec) shortconv_attn_kernel<float, 8><<<grid, CONV_THREADS, 0, st>>>(p);
-    else shortconv_attn_kernel<float, 1><<<grid, CONV_THREADS, 0, st>>>(p);
-  } else {
-    if (vec) shortconv_attn_kernel<__nv_bfloat16, 8><<<grid, CONV_THREADS, 0, st>>>(p);
-    else shortconv_attn_kernel<__nv_bfloat16, 1><<<grid, CONV_THREADS, 0, st>>>(p);
-  }
-  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  if (f32)
+    return vec ? launch_conv_attn<float, 8>(p, grid, st) : launch_conv_attn<float, 1>(p, grid, st);
+  return vec ? launch_conv_attn<__nv_bfloat16, 8>(p, grid, st)
+             : launch_conv_attn<__nv_bfloat16, 1>(p, grid, st);
 }
 
 extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, int boff,
@@ -331,18 +399,23 @@ extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, i
                                   const int* len, const int* pos0, const int* tile_entry,
                                   const int* tile_off, int tiles, const float* a, int lda,
                                   const float* A_log, const float* dt_bias, float* q, float* k,
-                                  float* kq, float* v, float* g, float* beta, int dim4, int f32,
+                                  float* kq, float* v, float* g, float* beta, int rows, int dim_p,
+                                  int f32,
                                   void* stream) {
   if (tiles <= 0 || taps < 1 || kv_heads < 1 || heads % kv_heads != 0) return -1;
-  if (dim > 256 || dim4 < dim || dim4 % 4 != 0 || dim4 > dim + 3) return -2;
+  if (dim > 256 || dim_p % 32 != 0 || dim_p < dim || dim_p > 256) return -2;
   DeltaPre p;
   p.c = conv_in(raw, ld, koff, voff, taps_w, taps, state, heads, kv_heads, dim, vdim, slot, row0, len,
                 pos0, tile_entry, tile_off);
   p.boff = boff; p.a = a; p.lda = lda; p.A_log = A_log; p.dt_bias = dt_bias; p.q = q; p.k = k;
-  p.kq = kq; p.v = v; p.g = g; p.beta = beta; p.dim4 = dim4;
+  p.kq = kq; p.v = v; p.g = g; p.beta = beta; p.rows = rows;
+  p.dim_p = dim_p;
   dim3 grid(tiles, kv_heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) shortconv_delta_kernel<float><<<grid, CONV_THREADS, 0, st>>>(p);
-  else shortconv_delta_kernel<__nv_bfloat16><<<grid, CONV_THREADS, 0, st>>>(p);
-  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && lda % 4 == 0 && ld % 8 == 0 && koff % 8 == 0 &&
+                   voff % 8 == 0;
+  if (f32)
+    return vec ? launch_conv_delta<float, 4>(p, grid, st) : launch_conv_delta<float, 1>(p, grid, st);
+  return vec ? launch_conv_delta<__nv_bfloat16, 4>(p, grid, st)
+             : launch_conv_delta<__nv_bfloat16, 1>(p, grid, st);
 }

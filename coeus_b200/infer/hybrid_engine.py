@@ -79,12 +79,13 @@ class HybridEngine(InferenceEngine):
         buffer, the feed-forward's activation."""
         T, m = h1.shape[0], self.m
         raw = torch.empty((T, layer.w_in.shape[0]), dtype=m.dtype, device=m.device)
-        G.linear(h1, layer.w_in, raw)
         cat = torch.empty((T, layer.w_out.shape[1]), dtype=m.dtype, device=m.device)
         if layer.out_dim != layer.act_off:
             cat[:, layer.out_dim:layer.act_off].zero_()
+        up = None
         if layer.w_up is not None:
-            G.linear(h2, layer.w_up, cat[:, layer.act_off:], epi="relu2")
+            up = (h2, layer.w_up, cat[:, layer.act_off:], "relu2", None, False)
+        G.linear_pair((h1, layer.w_in, raw, "none", None, False), up)
         return raw, cat
 
     def _attention(self, l: int, layer, raw: torch.Tensor, cat: torch.Tensor, b: R.RaggedBatch,
@@ -107,9 +108,10 @@ class HybridEngine(InferenceEngine):
         s, m, seg = layer.spec.mixer, self.m, layer.seg
         T = raw.shape[0]
         a = torch.empty((T, layer.w_a2.shape[0]), dtype=torch.float32, device=m.device)
-        G.linear(raw[:, seg["a1"]:seg["a1"] + layer.w_a2.shape[1]], layer.w_a2, a)
         gate = torch.empty((T, layer.w_g2.shape[0]), dtype=m.dtype, device=m.device)
-        G.linear(raw[:, seg["g1"]:seg["g1"] + layer.w_g2.shape[1]], layer.w_g2, gate)
+        a1, g1 = raw[:, seg["a1"]:], raw[:, seg["g1"]:]
+        G.linear_pair((a1[:, :layer.w_a2.shape[1]], layer.w_a2, a, "none", None, False),
+                      (g1[:, :layer.w_g2.shape[1]], layer.w_g2, gate, "none", None, False))
         qkvg = R.shortconv_delta(raw, seg["k"], seg["v"], seg["b"], layer.conv,
                                  self.state[l, "conv"], s.heads, s.kv_heads, s.dim, s.vdim, b, a,
                                  layer.A_log, layer.dt_bias)

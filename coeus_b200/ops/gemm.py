@@ -282,6 +282,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
             K, act, ctypes.c_float(softcap or 0.0), int(accumulate), _lib.stream_ptr())
         _lib.check_rc(rc, "cb_linear_f32")
         return out
+    if M <= SKINNY_MAX:
+        return linear_pair((x, w, out, epi, softcap, accumulate))[0]
     out_mode = _OUT_BF16 if out.dtype == torch.bfloat16 else (
         _OUT_F32_ATOMIC if accumulate else _OUT_F32)
     rc = _lib.serving_lib().cb_gemm_bf16(
@@ -294,3 +296,30 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
                                            ctypes.c_float(softcap), _lib.stream_ptr())
         _lib.check_rc(rc, "cb_softcap")
     return out
+
+
+SKINNY_MAX = 64       # rows up to which a bf16 product runs on the weight-streaming kernel
+
+
+def _skinny_args(x, w, out, epi, softcap, accumulate):
+    f32 = out.dtype == torch.float32
+    return (_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(out), out.stride(0),
+            w.shape[0], w.shape[1], 5 if softcap is not None else EPI[epi],
+            ctypes.c_float(softcap or 0.0), int(f32), int(accumulate))
+
+
+def linear_pair(first: tuple, second: Optional[tuple] = None):
+    """One or two independent products of the same few rows, each given as the arguments
+    ``(x, w, out, epi, softcap, accumulate)`` of :func:`linear`; in one launch where the rows are
+    few enough for the weight-streaming kernel (``cb_linear_skinny``), else one after the other."""
+    x = first[0]
+    M = x.shape[0]
+    todo = [first] if second is None else [first, second]
+    if not x.is_cuda or x.dtype != torch.bfloat16 or M > SKINNY_MAX:
+        return [linear(a[0], a[1], a[2], epi=a[3], softcap=a[4], accumulate=a[5]) for a in todo]
+    empty = (None, 0, None, 0, None, 0, 0, 0, 0, ctypes.c_float(0.0), 0, 0)
+    rc = _lib.serving_lib().cb_linear_skinny(
+        *_skinny_args(*first), *(empty if second is None else _skinny_args(*second)), M,
+        _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_linear_skinny")
+    return [a[2] for a in todo]

@@ -221,34 +221,36 @@ def shortconv_delta(raw: torch.Tensor, koff: int, voff: int, boff: int, taps_w: 
     """Inputs of the gated delta recurrence, fp32: convolution and SiLU of q, k and v, unit norm of
     q and k (q also times ``dim ** -0.5``), the decay ``exp(-exp(A_log) softplus(a + dt_bias))`` of
     every key channel, the step size ``sigmoid(raw[:, boff + h])``.  Returns
-    ``(q, k, kq, v, g, beta)``; q, k, g are padded with zeros to a multiple of four channels."""
+    ``(q [kv_heads, rows, P], k, kq [kv_heads, rows], v [rows, heads, vdim], g [heads, rows, P],
+    beta [heads, rows])``, the channels of q, k and g padded with zeros to a multiple of 32."""
     T = raw.shape[0]
-    dim4 = (dim + 3) // 4 * 4
+    P = (dim + 31) // 32 * 32
     qc, vc = kv_heads * dim, heads * vdim
     f32 = dict(dtype=torch.float32, device=raw.device)
     alloc = torch.zeros if not raw.is_cuda else torch.empty
-    q, k = alloc((T, kv_heads, dim4), **f32), alloc((T, kv_heads, dim4), **f32)
-    kq, v = alloc((T, kv_heads), **f32), alloc((T, heads, vdim), **f32)
-    g, beta = alloc((T, heads, dim4), **f32), alloc((T, heads), **f32)
+    q, k = alloc((kv_heads, T, P), **f32), alloc((kv_heads, T, P), **f32)
+    kq, v = alloc((kv_heads, T), **f32), alloc((T, heads, vdim), **f32)
+    g, beta = alloc((heads, T, P), **f32), alloc((heads, T), **f32)
     if not raw.is_cuda:
         u = torch.cat([raw[:, :qc], raw[:, koff:koff + qc], raw[:, voff:voff + vc]], 1)
         y = torch.nn.functional.silu(_conv_ref(u, taps_w, state, batch))
 
         def unit(x):
             return x * torch.rsqrt((x * x).sum(-1, keepdim=True) + 1e-6)
-        q[..., :dim] = unit(y[:, :qc].view(T, kv_heads, dim)) * dim ** -0.5
-        k[..., :dim] = unit(y[:, qc:2 * qc].view(T, kv_heads, dim))
+        q[..., :dim] = (unit(y[:, :qc].view(T, kv_heads, dim)) * dim ** -0.5).transpose(0, 1)
+        k[..., :dim] = unit(y[:, qc:2 * qc].view(T, kv_heads, dim)).transpose(0, 1)
         kq.copy_((q * k).sum(-1))
         v.copy_(y[:, 2 * qc:].view(T, heads, vdim))
         z = torch.nn.functional.softplus(a[:, :heads * dim].float() + dt_bias, threshold=100.0)
-        g[..., :dim] = torch.exp(-torch.exp(A_log)[None, :, None] * z.view(T, heads, dim))
-        beta.copy_(torch.sigmoid(raw[:, boff:boff + heads].float()))
+        g[..., :dim] = torch.exp(-torch.exp(A_log)[:, None, None]
+                                 * z.view(T, heads, dim).transpose(0, 1))
+        beta.copy_(torch.sigmoid(raw[:, boff:boff + heads].float()).t())
         return q, k, kq, v, g, beta
     rc = _lib.serving_lib().cb_shortconv_delta(
         _p(raw), raw.stride(0), koff, voff, boff, _p(taps_w), taps_w.shape[0], _p(state), heads,
         kv_heads, dim, vdim, *batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off),
         batch.n_conv, _p(a), a.stride(0), _p(A_log), _p(dt_bias), _p(q), _p(k), _p(kq), _p(v), _p(g),
-        _p(beta), dim4, int(raw.dtype == torch.float32), _lib.stream_ptr())
+        _p(beta), T, P, int(raw.dtype == torch.float32), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_shortconv_delta")
     return q, k, kq, v, g, beta
 
@@ -259,7 +261,7 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, kq: torch.Tensor, v: torch.Tens
     """The gated delta rule over every entry, from and into ``state [slots, heads, dim, vdim]``
     (fp32).  Returns the read-outs ``[rows, heads, vdim]``, fp32."""
     T, heads, vdim = v.shape
-    kv_heads, dim, dim4 = q.shape[1], state.shape[2], q.shape[2]
+    kv_heads, dim, P = q.shape[0], state.shape[2], q.shape[2]
     o = torch.empty_like(v)
     if not v.is_cuda:
         per, r = heads // kv_heads, 0
@@ -267,17 +269,17 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, kq: torch.Tensor, v: torch.Tens
             s = batch.slots_host[i]
             S = state[s].clone() if int(batch.pos0[i]) > 0 else torch.zeros_like(state[s])
             for t in range(r, r + m):
-                kk, qq = (x[t, :, :dim].repeat_interleave(per, 0) for x in (k, q))
-                S = S * g[t, :, :dim, None]
-                w = beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, kk))
+                kk, qq = (x[:, t, :dim].repeat_interleave(per, 0) for x in (k, q))
+                S = S * g[:, t, :dim, None]
+                w = beta[:, t, None] * (v[t] - torch.einsum("hdv,hd->hv", S, kk))
                 S = S + kk[:, :, None] * w[:, None, :]
                 o[t] = torch.einsum("hdv,hd->hv", S, qq)
             state[s] = S
             r += m
         return o
     rc = _lib.serving_lib().cb_delta_scan(
-        _p(q), _p(k), _p(kq), _p(v), _p(g), _p(beta), _p(state), _p(o), heads, kv_heads, dim, dim4,
-        vdim, *batch.entry_args(), batch.n, _lib.stream_ptr())
+        _p(q), _p(k), _p(kq), _p(v), _p(g), _p(beta), _p(state), _p(o), T, heads, kv_heads, dim,
+        P, vdim, *batch.entry_args(), batch.n, _lib.stream_ptr())
     _lib.check_rc(rc, "cb_delta_scan")
     return o
 
