@@ -1,9 +1,10 @@
 // Gated delta rule with one decay per key channel, over a ragged batch, in fp32.  Per head, with
 // the state S [dim, vdim] carried from token to token:
 //   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
-// The columns of S are independent, so a block takes one (entry, head) and 8 columns per warp and
+// The columns of S are independent, so a block takes one (entry, head) and 4 C columns per warp and
 // keeps its part of S in registers from the first token of the entry to the last.  Eight lanes
-// share a column pair, each holding R of the key channels.  Both products of a token use the
+// share C (2 or 4) columns, each holding R of the key channels; more columns per lane save reads
+// of shared memory, fewer give more warps.  Both products of a token use the
 // decayed state (o = S^T q + (k . q) u), so one reduction over the eight lanes serves them; the
 // arithmetic is two-wide packed fp32.  Tokens are staged in shared memory a few ahead.
 #include "ragged.cuh"
@@ -40,7 +41,6 @@ __device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
 }
 
 constexpr int SCAN_WARPS = 4;
-constexpr int SCAN_COLS = SCAN_WARPS * 8;
 constexpr int SCAN_TB = 8;         // tokens per stage
 constexpr int SCAN_STAGES = 3;
 
@@ -57,9 +57,9 @@ struct ScanArgs {
   Entries e;
 };
 
-template <int R>       // key channels per lane, a multiple of 4; DP = 8 R
+template <int R, int C>   // R key channels per lane, a multiple of 4; DP = 8 R
 __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanArgs p) {
-  constexpr int DP = 8 * R;
+  constexpr int DP = 8 * R, SCAN_COLS = SCAN_WARPS * 4 * C;
   constexpr int STAGE = SCAN_TB * (3 * DP + SCAN_COLS + 2);  // floats
   constexpr int THREADS = SCAN_WARPS * 32;
   extern __shared__ __align__(16) float sm[];
@@ -68,7 +68,7 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
   const int row0 = p.e.row0[e], len = p.e.len[e], slot = p.e.slot[e];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ld = lane & 7;
   const int col_base = slab * SCAN_COLS;
-  const int c0 = warp * 8 + (lane >> 3) * 2;                 // first of this lane's two columns
+  const int c0 = (warp * 4 + (lane >> 3)) * C;               // first of this lane's columns
   float* st = p.state + (static_cast<size_t>(slot) * p.heads + h) * p.dim * p.vdim;
   const float* gq = p.q + (static_cast<size_t>(hk) * p.rows + row0) * DP;
   const float* gk = p.k + (static_cast<size_t>(hk) * p.rows + row0) * DP;
@@ -111,10 +111,10 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
     if (i * SCAN_TB < len) fetch(i, i * SCAN_TB);
     else cp_async_commit();
   }
-  f2 s[2][R / 2];
+  f2 s[C][R / 2];
   const bool has_state = p.e.pos0[e] > 0;
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
+  for (int c = 0; c < C; ++c) {
     const int col = col_base + c0 + c;
 #pragma unroll
     for (int i = 0; i < R / 2; ++i) {
@@ -127,7 +127,9 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
       s[c][i] = pack_f2(x, y);
     }
   }
-  const int my = c0 + ((ld >> 1) & 1);                       // the column this lane finishes
+  // the column this lane finishes, and whether it ends with S^T q (else S^T k); see below
+  const int my_c = C == 4 ? ((ld >> 1) & 1) * 2 + ((ld >> 2) & 1) : (ld >> 1) & 1;
+  const int my = c0 + my_c;
   int stage = 0;
   for (int t0 = 0; t0 < len; t0 += SCAN_TB) {
     cp_async_wait<SCAN_STAGES - 2>();
@@ -142,7 +144,9 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
     stage = (stage + 1) % SCAN_STAGES;
     for (int t = 0; t < n; ++t) {
       const float* tq = sb + t * DP + ld * 4;
-      f2 a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull;
+      f2 a[C], b[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) a[c] = b[c] = 0ull;
       f2 kk[R / 2];
 #pragma unroll
       for (int j = 0; j < R / 4; ++j) {
@@ -151,44 +155,52 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
         const ulonglong2 g2 = *reinterpret_cast<const ulonglong2*>(tq + 2 * SCAN_TB * DP + j * 32);
         kk[2 * j] = k2.x;
         kk[2 * j + 1] = k2.y;
-        s[0][2 * j] = mul_f2(s[0][2 * j], g2.x);
-        s[0][2 * j + 1] = mul_f2(s[0][2 * j + 1], g2.y);
-        s[1][2 * j] = mul_f2(s[1][2 * j], g2.x);
-        s[1][2 * j + 1] = mul_f2(s[1][2 * j + 1], g2.y);
-        a0 = fma_f2(s[0][2 * j], k2.x, a0);
-        a1 = fma_f2(s[1][2 * j], k2.x, a1);
-        b0 = fma_f2(s[0][2 * j], q2.x, b0);
-        b1 = fma_f2(s[1][2 * j], q2.x, b1);
-        a0 = fma_f2(s[0][2 * j + 1], k2.y, a0);
-        a1 = fma_f2(s[1][2 * j + 1], k2.y, a1);
-        b0 = fma_f2(s[0][2 * j + 1], q2.y, b0);
-        b1 = fma_f2(s[1][2 * j + 1], q2.y, b1);
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          s[c][2 * j] = mul_f2(s[c][2 * j], g2.x);
+          s[c][2 * j + 1] = mul_f2(s[c][2 * j + 1], g2.y);
+          a[c] = fma_f2(s[c][2 * j], k2.x, a[c]);
+          b[c] = fma_f2(s[c][2 * j], q2.x, b[c]);
+          a[c] = fma_f2(s[c][2 * j + 1], k2.y, a[c]);
+          b[c] = fma_f2(s[c][2 * j + 1], q2.y, b[c]);
+        }
       }
-      // sum over the eight lanes, ending with one value per lane: bit 0 of ld picks S^T k or
-      // S^T q, bit 1 the column
-      const float fa0 = hsum_f2(a0), fa1 = hsum_f2(a1), fb0 = hsum_f2(b0), fb1 = hsum_f2(b1);
-      const bool odd = ld & 1, hi = ld & 2;
-      float x0 = (odd ? fb0 : fa0) + __shfl_xor_sync(0xffffffffu, odd ? fa0 : fb0, 1);
-      float x1 = (odd ? fb1 : fa1) + __shfl_xor_sync(0xffffffffu, odd ? fa1 : fb1, 1);
-      float y = (hi ? x1 : x0) + __shfl_xor_sync(0xffffffffu, hi ? x0 : x1, 2);
-      y += __shfl_xor_sync(0xffffffffu, y, 4);
+      // Sum over the eight lanes, ending with one value per lane: in the first exchange a lane
+      // keeps S^T q (odd ld) or S^T k (even), in the next ones a half of the columns it still has.
+      const bool odd = ld & 1, hi = ld & 2, top = ld & 4;
+      float x[C], y;
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        const float fa = hsum_f2(a[c]), fb = hsum_f2(b[c]);
+        x[c] = (odd ? fb : fa) + __shfl_xor_sync(0xffffffffu, odd ? fa : fb, 1);
+      }
+      if constexpr (C == 4) {
+        const float z0 = (hi ? x[2] : x[0]) + __shfl_xor_sync(0xffffffffu, hi ? x[0] : x[2], 2);
+        const float z1 = (hi ? x[3] : x[1]) + __shfl_xor_sync(0xffffffffu, hi ? x[1] : x[3], 2);
+        y = (top ? z1 : z0) + __shfl_xor_sync(0xffffffffu, top ? z0 : z1, 4);
+      } else {
+        y = (hi ? x[1] : x[0]) + __shfl_xor_sync(0xffffffffu, hi ? x[0] : x[1], 2);
+        y += __shfl_xor_sync(0xffffffffu, y, 4);
+      }
       const float beta = ss[t], kq = ss[SCAN_TB + t];
       const float un = beta * (sv[t * SCAN_COLS + my] - y);  // of use on even lanes
-      const float u0 = __shfl_sync(0xffffffffu, un, lane & 24);
-      const float u1 = __shfl_sync(0xffffffffu, un, (lane & 24) | 2);
-      const f2 p0 = pack_f2(u0, u0), p1 = pack_f2(u1, u1);
+      float u_my = 0.f;
 #pragma unroll
-      for (int i = 0; i < R / 2; ++i) {
-        s[0][i] = fma_f2(kk[i], p0, s[0][i]);
-        s[1][i] = fma_f2(kk[i], p1, s[1][i]);
+      for (int c = 0; c < C; ++c) {
+        // the even lane that finished column c
+        const int src = C == 4 ? ((c >> 1) << 1) | ((c & 1) << 2) : c << 1;
+        const float u = __shfl_sync(0xffffffffu, un, (lane & 24) | src);
+        if (c == my_c) u_my = u;
+        const f2 uu = pack_f2(u, u);
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) s[c][i] = fma_f2(kk[i], uu, s[c][i]);
       }
-      if (odd && ld < 4 && col_base + my < p.vdim)
-        p.o[(static_cast<size_t>(row0 + t0 + t) * p.heads + h) * p.vdim + col_base + my] =
-            y + kq * (hi ? u1 : u0);
+      if (odd && (C == 4 || ld < 4) && col_base + my < p.vdim)
+        p.o[(static_cast<size_t>(row0 + t0 + t) * p.heads + h) * p.vdim + col_base + my] = y + kq * u_my;
     }
   }
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
+  for (int c = 0; c < C; ++c) {
     const int col = col_base + c0 + c;
     if (col >= p.vdim) continue;
 #pragma unroll
@@ -201,19 +213,28 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanA
   }
 }
 
-template <int R>
-static int launch_scan(const ScanArgs& a, int entries, cudaStream_t st) {
-  const int smem = SCAN_STAGES * SCAN_TB * (3 * 8 * R + SCAN_COLS + 2) * 4;
+template <int R, int C>
+static int launch_scan_c(const ScanArgs& a, int entries, cudaStream_t st) {
+  constexpr int cols = SCAN_WARPS * 4 * C;
+  const int smem = SCAN_STAGES * SCAN_TB * (3 * 8 * R + cols + 2) * 4;
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(delta_scan_kernel<R, C>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              smem) != cudaSuccess)
       return -4;
     set = true;
   }
-  dim3 grid(a.heads * ((a.vdim + SCAN_COLS - 1) / SCAN_COLS), entries);
-  delta_scan_kernel<R><<<grid, SCAN_WARPS * 32, smem, st>>>(a);
+  dim3 grid(a.heads * ((a.vdim + cols - 1) / cols), entries);
+  delta_scan_kernel<R, C><<<grid, SCAN_WARPS * 32, smem, st>>>(a);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+template <int R>
+static int launch_scan(const ScanArgs& a, int entries, cudaStream_t st) {
+  if constexpr (R <= 16) {
+    const int wide = a.heads * ((a.vdim + 63) / 64) * entries;   // blocks with four columns a lane
+    if (a.vdim > 32 && wide >= sm_count()) return launch_scan_c<R, 4>(a, entries, st);
+  }
+  return launch_scan_c<R, 2>(a, entries, st);
 }
 
 }  // namespace cb

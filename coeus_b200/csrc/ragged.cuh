@@ -62,6 +62,8 @@ __device__ __forceinline__ void load_vec(const float* p, float* f) {
 template <int V>
 __device__ __forceinline__ void store_vec(__nv_bfloat16* p, const float* f) {
   if constexpr (V == 8) store8(p, f);
+  else if constexpr (V == 4)
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
   else *p = __float2bfloat16(f[0]);
 }
 template <int V>
@@ -69,6 +71,8 @@ __device__ __forceinline__ void store_vec(float* p, const float* f) {
   if constexpr (V == 8) {
     *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
     *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
   } else {
     *p = f[0];
   }

@@ -111,17 +111,43 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 gated_head_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int ldg,
                        const float* __restrict__ w, T* __restrict__ y, int ldy, int rows, int heads,
-                       int vdim, float eps) {
+                       int vdim, float eps, bool vec) {
   const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (unit >= rows * heads) return;
   const int r = unit / heads, h = unit % heads;
   const float* src = o + static_cast<size_t>(unit) * vdim;
+  const T* gp = gate + static_cast<size_t>(r) * ldg + h * vdim;
+  T* dst = y + static_cast<size_t>(r) * ldy + h * vdim;
   float s = 0.f;
+  if (vec) {                                  // four channels per lane, at most 256 in all
+    float f[2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int c = (lane + 32 * i) * 4;
+      if (c < vdim) {
+        load_vec<4>(src + c, f[i]);
+        s += f[i][0] * f[i][0] + f[i][1] * f[i][1] + f[i][2] * f[i][2] + f[i][3] * f[i][3];
+      }
+    }
+    s = warp_sum(s);
+    const float rs = 1.0f / sqrtf(s / vdim + eps);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int c = (lane + 32 * i) * 4;
+      if (c < vdim) {
+        float g[4], k[4];
+        load_vec<4>(gp + c, g);
+        load_vec<4>(w + c, k);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) f[i][x] = f[i][x] * rs * k[x] * sigmoidf_(g[x]);
+        store_vec<4>(dst + c, f[i]);
+      }
+    }
+    return;
+  }
   for (int c = lane; c < vdim; c += 32) s += src[c] * src[c];
   s = warp_sum(s);
   const float rs = 1.0f / sqrtf(s / vdim + eps);
-  const T* gp = gate + static_cast<size_t>(r) * ldg + h * vdim;
-  T* dst = y + static_cast<size_t>(r) * ldy + h * vdim;
   for (int c = lane; c < vdim; c += 32)
     dst[c] = from_f32<T>(src[c] * rs * w[c] * sigmoidf_(to_f32(gp[c])));
 }
@@ -211,14 +237,16 @@ extern "C" int cb_gated_head_norm(const float* o, const void* gate, int ldg, con
                                   void* stream) {
   if (rows <= 0) return -1;
   const int blocks = (rows * heads + 3) / 4;
+  const bool vec = vdim % 4 == 0 && vdim <= 256 && ldg % 4 == 0 && ldy % 4 == 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     gated_head_norm_kernel<float><<<blocks, 128, 0, st>>>(
-        o, static_cast<const float*>(gate), ldg, w, static_cast<float*>(y), ldy, rows, heads, vdim, eps);
+        o, static_cast<const float*>(gate), ldg, w, static_cast<float*>(y), ldy, rows, heads, vdim, eps,
+        vec);
   else
     gated_head_norm_kernel<__nv_bfloat16><<<blocks, 128, 0, st>>>(
         o, static_cast<const __nv_bfloat16*>(gate), ldg, w, static_cast<__nv_bfloat16*>(y), ldy, rows,
-        heads, vdim, eps);
+        heads, vdim, eps, vec);
   return CB_RC();
 }
 

@@ -111,6 +111,8 @@ struct AttnPre {
   void* v_first;           // [rows, kv_heads * vdim]: written when mix_mode = 1, read when 2
   const float* lambda;
   int mix_mode;
+  void* k_rows;            // out [rows, kv_heads * dim]: k once more, row by row (or null)
+  void* v_rows;            // out [rows, kv_heads * vdim]
   int* status;
 };
 
@@ -159,11 +161,18 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
         }
         store_vec<V>(dst + d, oa);
         store_vec<V>(dst + p.half + d, ob);
+        if (!is_q && p.k_rows != nullptr) {
+          T* kr = static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d;
+          store_vec<V>(kr, oa);
+          store_vec<V>(kr + p.half, ob);
+        }
       } else {
         const int d = 2 * p.half + (k - pair_u) * V;
         float a[V];
         conv_at<T, V, TAPS>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
         store_vec<V>(dst + d, a);
+        if (!is_q && p.k_rows != nullptr)
+          store_vec<V>(static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d, a);
       }
     } else {
       const int d = (u - (per + 1) * head_u) * V;
@@ -182,12 +191,161 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
         }
       }
       store_vec<V>(static_cast<T*>(p.v_cache) + cell * p.vdim_p + d, a);
+      if (p.v_rows != nullptr)
+        store_vec<V>(static_cast<T*>(p.v_rows) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d, a);
     }
   }
   if (off == 0 && ci.taps > 1) {
     __syncthreads();
     const int mine = (per + 1) * dim + vdim;
     for (int i = threadIdx.x; i < mine; i += CONV_THREADS) {
+      const int c = i < per * dim ? g * per * dim + i
+                  : (i < (per + 1) * dim ? qc + g * dim + (i - per * dim)
+                                         : qc + kc + g * vdim + (i - (per + 1) * dim));
+      conv_advance<T>(ci, c, raw_col(ci, c), channels, row0, len, slot, has_state);
+    }
+  }
+}
+
+// The same with V = 4 consecutive channels per thread for a whole tile of tokens: the taps of a
+// thread's channels stay in registers and every projected row is loaded once.  dim, vdim and half
+// are multiples of four.  The threads of a block are its units (see above), nothing else.
+template <typename T, int TAPS>
+struct Window {
+  static constexpr int V = 4;
+  float w[TAPS][V], u[TAPS][V];
+  // loads the taps of channels c.. and the TAPS - 1 rows before token t
+  __device__ __forceinline__ void start(const ConvIn& p, int c, int col, int channels, int row0,
+                                        int t, int slot, bool has_state) {
+    const T* raw = static_cast<const T*>(p.raw) + static_cast<ptrdiff_t>(row0) * p.ld + col;
+    const T* st = static_cast<const T*>(p.state) + static_cast<ptrdiff_t>(slot) * (TAPS - 1) * channels + c;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * channels + c, w[j]);
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) {
+      const int o = t - TAPS + j;
+#pragma unroll
+      for (int i = 0; i < V; ++i) u[j][i] = 0.f;
+      if (o >= 0) load_vec<V>(raw + static_cast<ptrdiff_t>(o) * p.ld, u[j]);
+      else if (has_state) load_vec<V>(st + static_cast<ptrdiff_t>(TAPS - 1 + o) * channels, u[j]);
+    }
+  }
+  // takes the next row in, y = convolution at its token
+  __device__ __forceinline__ void next(const T* row, float* y) {
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < V; ++i) u[j][i] = u[j + 1][i];
+    load_vec<V>(row, u[TAPS - 1]);
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[i] = 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[i] += u[j][i] * w[j][i];
+  }
+};
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(512) shortconv_attn_tile_kernel(const AttnPre p) {
+  constexpr int V = 4;
+  const ConvIn& ci = p.c;
+  const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
+  const int row0 = ci.e.row0[e], len = ci.e.len[e], pos0 = ci.e.pos0[e], slot = ci.e.slot[e];
+  const bool has_state = pos0 > 0;
+  const int per = ci.heads / ci.kv_heads, dim = ci.dim, vdim = ci.vdim;
+  const int qc = ci.heads * dim, kc = ci.kv_heads * dim;
+  const int channels = qc + kc + ci.kv_heads * vdim;
+  const int t1 = min(off + CONV_TILE, len);
+  const int pair_u = p.half / V, head_u = (dim - p.half) / V;
+  const int heads_u = (per + 1) * head_u;
+  const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
+  __shared__ int s_page[2];
+  if (threadIdx.x < 2) {                     // a tile of 16 tokens touches at most two pages
+    const int lp = (pos0 + off) / RAGGED_PAGE + threadIdx.x;
+    int page = lp < p.max_pages ? p.page_table[static_cast<size_t>(slot) * p.max_pages + lp] : -1;
+    const bool used = lp <= (pos0 + t1 - 1) / RAGGED_PAGE;
+    if (used && (page < 0 || page >= p.num_pages)) record_status(p.status, ST_BOUNDS, row0 + off);
+    s_page[threadIdx.x] = used && page >= 0 && page < p.num_pages ? page : -1;
+  }
+  __syncthreads();
+  const int lp0 = (pos0 + off) / RAGGED_PAGE;
+  for (int u = threadIdx.x; u < heads_u + vdim / V; u += blockDim.x) {
+    const bool is_v = u >= heads_u;
+    const int hi = is_v ? 0 : u / head_u, k = is_v ? 0 : u % head_u;
+    const bool is_q = !is_v && hi < per, pair = !is_v && k < pair_u;
+    int c, col, d;
+    if (is_v) {
+      d = (u - heads_u) * V;
+      c = qc + kc + g * vdim + d;
+      col = ci.voff + g * vdim + d;
+    } else {
+      d = pair ? k * V : p.half + k * V;     // plain units start behind the second half
+      const int base = is_q ? (g * per + hi) * dim : g * dim;
+      c = (is_q ? 0 : qc) + base + d;
+      col = (is_q ? 0 : ci.koff) + base + d;
+    }
+    Window<T, TAPS> wa, wb;
+    wa.start(ci, c, col, channels, row0, off, slot, has_state);
+    if (pair) wb.start(ci, c + p.half, col + p.half, channels, row0, off, slot, has_state);
+    const float lam = is_v && p.mix_mode == 2 ? *p.lambda : 0.f;
+#pragma unroll 2
+    for (int t = off; t < t1; ++t) {
+      const int row = row0 + t, pos = pos0 + t;
+      const int page = s_page[pos / RAGGED_PAGE - lp0];
+      const T* src = raw + static_cast<ptrdiff_t>(t) * ci.ld + col;
+      float a[V];
+      wa.next(src, a);
+      const size_t cell = (static_cast<size_t>(max(page, 0)) * RAGGED_PAGE + pos % RAGGED_PAGE) * ci.kv_heads + g;
+      T* dst = is_q ? static_cast<T*>(p.q) + static_cast<size_t>(row) * qc + c
+                    : (is_v ? static_cast<T*>(p.v_cache) + cell * p.vdim_p + d
+                            : static_cast<T*>(p.k_cache) + cell * p.dim_p + d);
+      const bool ok = is_q || page >= 0;
+      if (pair) {
+        float b[V], oa[V], ob[V];
+        wb.next(src + p.half, b);
+        const float4* cs = reinterpret_cast<const float4*>(p.rope + static_cast<size_t>(row) * p.half + d);
+        const float4 x = cs[0], y = cs[1];
+        const float cc[V] = {x.x, x.z, y.x, y.z}, ss[V] = {x.y, x.w, y.y, y.w};
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+          oa[i] = a[i] * cc[i] - b[i] * ss[i];
+          ob[i] = b[i] * cc[i] + a[i] * ss[i];
+        }
+        if (ok) {
+          store_vec<V>(dst, oa);
+          store_vec<V>(dst + p.half, ob);
+        }
+        if (!is_q && p.k_rows != nullptr) {
+          T* kr = static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d;
+          store_vec<V>(kr, oa);
+          store_vec<V>(kr + p.half, ob);
+        }
+        continue;
+      }
+      if (is_v && p.mix_mode != 0) {
+        T* vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d;
+        if (p.mix_mode == 1) {
+          store_vec<V>(vf, a);
+        } else {
+          float f[V];
+          load_vec<V>(vf, f);
+#pragma unroll
+          for (int i = 0; i < V; ++i) a[i] = (1.f - lam) * a[i] + lam * f[i];
+        }
+      }
+      if (ok) store_vec<V>(dst, a);
+      if (!is_q && p.k_rows != nullptr) {
+        T* kr = is_v ? static_cast<T*>(p.v_rows) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d
+                     : static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d;
+        store_vec<V>(kr, a);
+      }
+    }
+  }
+  if (off == 0) {
+    __syncthreads();
+    const int mine = (per + 1) * dim + vdim;
+    for (int i = threadIdx.x; i < mine; i += blockDim.x) {
       const int c = i < per * dim ? g * per * dim + i
                   : (i < (per + 1) * dim ? qc + g * dim + (i - per * dim)
                                          : qc + kc + g * vdim + (i - (per + 1) * dim));
@@ -327,23 +485,194 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_kernel(const Del
   }
 }
 
-template <typename T, int V>
-static int launch_conv_attn(const AttnPre& p, dim3 grid, cudaStream_t st) {
-  switch (p.c.taps) {
-    case 2: shortconv_attn_kernel<T, V, 2><<<grid, CONV_THREADS, 0, st>>>(p); break;
-    case 3: shortconv_attn_kernel<T, V, 3><<<grid, CONV_THREADS, 0, st>>>(p); break;
-    case 4: shortconv_attn_kernel<T, V, 4><<<grid, CONV_THREADS, 0, st>>>(p); break;
-    default: shortconv_attn_kernel<T, V, 0><<<grid, CONV_THREADS, 0, st>>>(p);
+// SiLU of a convolution's output (an activation: the fast form where activations are bf16).
+template <typename T>
+__device__ __forceinline__ float silu_act(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-x));
+  else return silu_exact(x);
+}
+
+// The same with four channels per thread over a tile of tokens.  Work of a block, dealt to its
+// warps: q and k of the two halves of the tile (a token's 128 or 256 channels are one warp's, the
+// norms are warp sums), the values and the decays in pieces of 128 channels.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(const DeltaPre p) {
+  constexpr int V = 4;
+  const ConvIn& ci = p.c;
+  const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
+  const int row0 = ci.e.row0[e], len = ci.e.len[e], slot = ci.e.slot[e];
+  const bool has_state = ci.e.pos0[e] > 0;
+  const int per = ci.heads / ci.kv_heads, dim = ci.dim, vdim = ci.vdim;
+  const int qc = ci.kv_heads * dim;
+  const int channels = 2 * qc + ci.heads * vdim;
+  const int t1 = min(off + CONV_TILE, len);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float qscale = 1.0f / sqrtf(static_cast<float>(dim));
+  const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
+  const int half_t = t1 - off > CONV_TILE / 2 ? CONV_TILE / 2 : CONV_TILE;
+  const int n_qk = t1 - off > half_t ? 2 : 1;
+  const int n_v = (per * vdim + 127) / 128, n_g = per * ((p.dim_p + 127) / 128);
+  for (int u = warp; u < n_qk + n_v + n_g; u += CONV_THREADS / 32) {
+    if (u < n_qk) {
+      const int ta = off + u * half_t, tb = min(ta + half_t, t1);
+      if (dim <= 128) {
+        const int d = lane * V;
+        const bool in = d < dim;
+        Window<T, TAPS> wq, wk;
+        const int cq = g * dim + (in ? d : 0);
+        wq.start(ci, cq, cq, channels, row0, ta, slot, has_state);
+        wk.start(ci, qc + cq, ci.koff + cq, channels, row0, ta, slot, has_state);
+#pragma unroll 2
+        for (int t = ta; t < tb; ++t) {
+          const T* src = raw + static_cast<ptrdiff_t>(t) * ci.ld + cq;
+          float q[V], k[V], sq = 0.f, sk = 0.f, dot = 0.f;
+          wq.next(src, q);
+          wk.next(src + ci.koff, k);
+#pragma unroll
+          for (int x = 0; x < V; ++x) {
+            q[x] = in ? silu_act<T>(q[x]) : 0.f;
+            k[x] = in ? silu_act<T>(k[x]) : 0.f;
+            sq += q[x] * q[x];
+            sk += k[x] * k[x];
+            dot += q[x] * k[x];
+          }
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) {
+            sq += __shfl_xor_sync(0xffffffffu, sq, o);
+            sk += __shfl_xor_sync(0xffffffffu, sk, o);
+            dot += __shfl_xor_sync(0xffffffffu, dot, o);
+          }
+          const float rq = qscale / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f);
+          const size_t cell = static_cast<size_t>(g) * p.rows + row0 + t;
+#pragma unroll
+          for (int x = 0; x < V; ++x) {
+            q[x] *= rq;
+            k[x] *= rk;
+          }
+          if (d < p.dim_p) {
+            store_f32<V>(p.q + cell * p.dim_p + d, q);
+            store_f32<V>(p.k + cell * p.dim_p + d, k);
+          }
+          if (lane == 0) p.kq[cell] = dot * rq * rk;
+        }
+      } else {
+        for (int t = ta; t < tb; ++t) {
+          float q[2][V], k[2][V], sq = 0.f, sk = 0.f, dot = 0.f;
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const int d = (lane + 32 * i) * V;
+#pragma unroll
+            for (int x = 0; x < V; ++x) q[i][x] = k[i][x] = 0.f;
+            if (d < dim) {
+              conv_at<T, V, TAPS>(ci, g * dim + d, g * dim + d, channels, row0, t, slot, has_state, q[i]);
+              conv_at<T, V, TAPS>(ci, qc + g * dim + d, ci.koff + g * dim + d, channels, row0, t, slot, has_state, k[i]);
+            }
+#pragma unroll
+            for (int x = 0; x < V; ++x) {
+              q[i][x] = silu_act<T>(q[i][x]);
+              k[i][x] = silu_act<T>(k[i][x]);
+              sq += q[i][x] * q[i][x];
+              sk += k[i][x] * k[i][x];
+              dot += q[i][x] * k[i][x];
+            }
+          }
+          const float rq = qscale / sqrtf(warp_sum(sq) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f);
+          dot = warp_sum(dot);
+          const size_t cell = static_cast<size_t>(g) * p.rows + row0 + t;
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const int d = (lane + 32 * i) * V;
+#pragma unroll
+            for (int x = 0; x < V; ++x) {
+              q[i][x] *= rq;
+              k[i][x] *= rk;
+            }
+            if (d < p.dim_p) {
+              store_f32<V>(p.q + cell * p.dim_p + d, q[i]);
+              store_f32<V>(p.k + cell * p.dim_p + d, k[i]);
+            }
+          }
+          if (lane == 0) p.kq[cell] = dot * rq * rk;
+        }
+      }
+    } else if (u < n_qk + n_v) {
+      const int i = ((u - n_qk) * 32 + lane) * V;
+      if (i < per * vdim) {
+        const int c = g * per * vdim + i;
+        Window<T, TAPS> w;
+        w.start(ci, 2 * qc + c, ci.voff + c, channels, row0, off, slot, has_state);
+#pragma unroll 4
+        for (int t = off; t < t1; ++t) {
+          float y[V];
+          w.next(raw + static_cast<ptrdiff_t>(t) * ci.ld + ci.voff + c, y);
+#pragma unroll
+          for (int x = 0; x < V; ++x) y[x] = silu_act<T>(y[x]);
+          store_f32<V>(p.v + static_cast<size_t>(row0 + t) * ci.heads * vdim + c, y);
+        }
+      }
+    } else {
+      const int pieces = (p.dim_p + 127) / 128, i = u - n_qk - n_v;
+      const int h = g * per + i / pieces, d = ((i % pieces) * 32 + lane) * V;
+      if (d < p.dim_p) {
+        const bool in = d < dim;
+        const float rate = expf(p.A_log[h]);
+        float b[V] = {};
+        if (in) load_f32<V>(p.dt_bias + h * dim + d, b);
+#pragma unroll 4
+        for (int t = off; t < t1; ++t) {
+          float f[V] = {};
+          if (in) {
+            float a[V];
+            load_f32<V>(p.a + static_cast<size_t>(row0 + t) * p.lda + h * dim + d, a);
+#pragma unroll
+            for (int x = 0; x < V; ++x) f[x] = expf(-rate * softplus_exact(a[x] + b[x]));
+          }
+          store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row0 + t) * p.dim_p + d, f);
+        }
+      }
+    }
+  }
+  for (int i = threadIdx.x; i < (t1 - off) * per; i += CONV_THREADS) {
+    const int h = g * per + i / (t1 - off), t = off + i % (t1 - off);
+    p.beta[static_cast<size_t>(h) * p.rows + row0 + t] =
+        sigmoidf_(to_f32(raw[static_cast<ptrdiff_t>(t) * ci.ld + p.boff + h]));
+  }
+  if (off == 0) {
+    __syncthreads();
+    const int mine = 2 * dim + per * vdim;
+    for (int i = threadIdx.x; i < mine; i += CONV_THREADS) {
+      const int c = i < dim ? g * dim + i
+                  : (i < 2 * dim ? qc + g * dim + (i - dim) : 2 * qc + g * per * vdim + (i - 2 * dim));
+      conv_advance<T>(ci, c, raw_col_delta(ci, c), channels, row0, len, slot, has_state);
+    }
+  }
+}
+
+template <typename T>
+static int launch_conv_attn(const AttnPre& p, dim3 grid, bool vec, cudaStream_t st) {
+  if (vec) {
+    const int units = (p.c.heads / p.c.kv_heads + 1) * ((p.c.dim - p.half) / 4) + p.c.vdim / 4;
+    const int threads = min(512, (units + 31) / 32 * 32);
+    switch (p.c.taps) {
+      case 2: shortconv_attn_tile_kernel<T, 2><<<grid, threads, 0, st>>>(p); break;
+      case 3: shortconv_attn_tile_kernel<T, 3><<<grid, threads, 0, st>>>(p); break;
+      default: shortconv_attn_tile_kernel<T, 4><<<grid, threads, 0, st>>>(p);
+    }
+  } else {
+    shortconv_attn_kernel<T, 1, 0><<<grid, CONV_THREADS, 0, st>>>(p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
-template <typename T, int V>
-static int launch_conv_delta(const DeltaPre& p, dim3 grid, cudaStream_t st) {
-  switch (p.c.taps) {
-    case 2: shortconv_delta_kernel<T, V, 2><<<grid, CONV_THREADS, 0, st>>>(p); break;
-    case 3: shortconv_delta_kernel<T, V, 3><<<grid, CONV_THREADS, 0, st>>>(p); break;
-    case 4: shortconv_delta_kernel<T, V, 4><<<grid, CONV_THREADS, 0, st>>>(p); break;
-    default: shortconv_delta_kernel<T, V, 0><<<grid, CONV_THREADS, 0, st>>>(p);
+template <typename T>
+static int launch_conv_delta(const DeltaPre& p, dim3 grid, bool vec, cudaStream_t st) {
+  if (vec) {
+    switch (p.c.taps) {
+      case 2: shortconv_delta_tile_kernel<T, 2><<<grid, CONV_THREADS, 0, st>>>(p); break;
+      case 3: shortconv_delta_tile_kernel<T, 3><<<grid, CONV_THREADS, 0, st>>>(p); break;
+      default: shortconv_delta_tile_kernel<T, 4><<<grid, CONV_THREADS, 0, st>>>(p);
+    }
+  } else {
+    shortconv_delta_kernel<T, 1, 0><<<grid, CONV_THREADS, 0, st>>>(p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
@@ -372,8 +701,8 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
                                  const int* tile_entry, const int* tile_off, int tiles, int half,
                                  const void* rope, void* q, void* k_cache, void* v_cache, int dim_p,
                                  int vdim_p, const int* page_table, int max_pages, int num_pages,
-                                 void* v_first, const float* lambda, int mix_mode, int f32,
-                                 int* status, void* stream) {
+                                 void* v_first, const float* lambda, int mix_mode, void* k_rows,
+                                 void* v_rows, int f32, int* status, void* stream) {
   if (tiles <= 0 || taps < 1 || kv_heads < 1 || heads % kv_heads != 0 || 2 * half > dim) return -1;
   if (mix_mode != 0 && v_first == nullptr) return -2;
   AttnPre p;
@@ -383,14 +712,13 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
   p.v_cache = v_cache; p.dim_p = dim_p; p.vdim_p = vdim_p; p.page_table = page_table;
   p.max_pages = max_pages; p.num_pages = num_pages; p.v_first = v_first; p.lambda = lambda;
   p.mix_mode = mix_mode; p.status = status;
-  const bool vec = dim % 8 == 0 && vdim % 8 == 0 && half % 8 == 0 && ld % 8 == 0 && koff % 8 == 0 &&
-                   voff % 8 == 0;
+  p.k_rows = k_rows; p.v_rows = v_rows;
+  const bool vec = taps >= 2 && taps <= 4 && dim % 4 == 0 && vdim % 4 == 0 && half % 4 == 0 &&
+                   ld % 8 == 0 && koff % 8 == 0 && voff % 8 == 0;
   dim3 grid(tiles, kv_heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32)
-    return vec ? launch_conv_attn<float, 8>(p, grid, st) : launch_conv_attn<float, 1>(p, grid, st);
-  return vec ? launch_conv_attn<__nv_bfloat16, 8>(p, grid, st)
-             : launch_conv_attn<__nv_bfloat16, 1>(p, grid, st);
+  return f32 ? launch_conv_attn<float>(p, grid, vec, st)
+             : launch_conv_attn<__nv_bfloat16>(p, grid, vec, st);
 }
 
 extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, int boff,
@@ -412,10 +740,8 @@ extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, i
   p.dim_p = dim_p;
   dim3 grid(tiles, kv_heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && lda % 4 == 0 && ld % 8 == 0 && koff % 8 == 0 &&
+  const bool vec = taps >= 2 && taps <= 4 && dim % 4 == 0 && vdim % 4 == 0 && lda % 4 == 0 && ld % 8 == 0 && koff % 8 == 0 &&
                    voff % 8 == 0;
-  if (f32)
-    return vec ? launch_conv_delta<float, 4>(p, grid, st) : launch_conv_delta<float, 1>(p, grid, st);
-  return vec ? launch_conv_delta<__nv_bfloat16, 4>(p, grid, st)
-             : launch_conv_delta<__nv_bfloat16, 1>(p, grid, st);
+  return f32 ? launch_conv_delta<float>(p, grid, vec, st)
+             : launch_conv_delta<__nv_bfloat16>(p, grid, vec, st);
 }

@@ -173,12 +173,14 @@ def shortconv_attn(raw: torch.Tensor, koff: int, voff: int, taps_w: torch.Tensor
                    batch: RaggedBatch, rope: Optional[torch.Tensor], k_cache: torch.Tensor,
                    v_cache: torch.Tensor, page_table: torch.Tensor,
                    v_first: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
-                   write_first: bool = False) -> torch.Tensor:
+                   write_first: bool = False, k_rows: Optional[torch.Tensor] = None,
+                   v_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
     """What stands between the projections and the scores of an attention layer: a causal
     convolution over time on every channel of q, k and v (``taps_w [taps, channels]``), rotary
     embedding of the first ``2 * rope.shape[1]`` entries of the q and k heads in the rotate-half
     layout, value mixing ``v <- (1 - mix) v + mix v_first`` (or, with ``write_first``, keeping v as
-    ``v_first``), and the write of k and v into the cache pages.  Returns ``q [rows, heads*dim]``."""
+    ``v_first``), and the write of k and v into the cache pages (and, when given, row by row into
+    ``k_rows [rows, kv_heads*dim]`` and ``v_rows``).  Returns ``q [rows, heads*dim]``."""
     T = raw.shape[0]
     half = rope.shape[1] if rope is not None else 0
     mode = 1 if write_first else (2 if mix is not None else 0)
@@ -202,6 +204,9 @@ def shortconv_attn(raw: torch.Tensor, koff: int, voff: int, taps_w: torch.Tensor
         page, at = _cells(page_table, batch)
         k_cache[page, at, :, :dim] = k.to(k_cache.dtype)
         v_cache[page, at, :, :vdim] = v.to(v_cache.dtype)
+        if k_rows is not None:
+            k_rows.copy_(k.reshape(T, -1))
+            v_rows.copy_(v.reshape(T, -1))
         return q.reshape(T, qc).to(raw.dtype)
     q = torch.empty((T, qc), dtype=raw.dtype, device=raw.device)
     rc = _lib.serving_lib().cb_shortconv_attn(
@@ -209,7 +214,7 @@ def shortconv_attn(raw: torch.Tensor, koff: int, voff: int, taps_w: torch.Tensor
         dim, vdim, *batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off), batch.n_conv, half,
         _p(rope), _p(q), _p(k_cache), _p(v_cache), k_cache.shape[-1], v_cache.shape[-1],
         _p(page_table), page_table.shape[1], k_cache.shape[0], _p(v_first), _p(mix), mode,
-        int(raw.dtype == torch.float32), _p(_lib.status_buffer(raw.device)), _lib.stream_ptr())
+        _p(k_rows), _p(v_rows), int(raw.dtype == torch.float32), _p(_lib.status_buffer(raw.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_shortconv_attn")
     return q
 
@@ -357,7 +362,8 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         ctas = n * kv_heads * (1 if per <= 8 else (per + 7) // 8)
         ctx = max_ctx or batch.max_ctx
         ctx = min(ctx, chunk) if chunk else ctx
-        splits = max(1, min(16, (4 * 148 + ctas - 1) // ctas, ctx // 256))
+        # a CTA takes 128 keys at a time
+        splits = max(1, min(16, (4 * 148 + ctas - 1) // ctas, (ctx + 127) // 128))
         part_o = part_ml = None
         if splits > 1:
             part_o = torch.empty((n, heads, splits, vdim), dtype=torch.float32, device=q.device)
