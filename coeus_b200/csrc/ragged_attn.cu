@@ -5,7 +5,9 @@
 // query/key width and value width are independent.
 //
 //   rows kernel    one CTA per (query row, key/value head, split): the query heads of the group
-//                  share every key and value that is loaded.  Decoding, and everything in fp32.
+//                  share every key and value that is loaded.  Everything in fp32, and decoding
+//                  of heads wider than 128.
+//   group kernel   decoding in bf16: the same split of the work, on the tensor cores.
 //   tiles kernel   64 query rows of one head on the tensor cores (mma m16n8k16), one cache page
 //                  per step through a double-buffered shared-memory ring.  The weights enter the
 //                  second product as the sum of two bf16 numbers, so they keep 16 mantissa bits.
@@ -462,6 +464,246 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
   }
 }
 
+// ------------------------------------------------------------------------------ group kernel
+// Decoding in bf16: one query row, the (up to 16) query heads of one key/value head as the rows
+// of the tensor-core tile.  The warps of a CTA take blocks of 32 keys in turn, each through its
+// own double-buffered ring, and their partial softmaxes are merged at the end.
+constexpr int GA_WARPS = 4;
+constexpr int GA_KEYS = 32;
+
+template <int DC, int VC>
+__global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const RowsArgs ra) {
+  using bf16 = __nv_bfloat16;
+  const RaggedAttn& p = ra.a;
+  constexpr int KS = DC + 8, VS = VC + 8;
+  constexpr int STAGE = GA_KEYS * (KS + VS);            // elements of one stage of one warp
+  extern __shared__ __align__(16) unsigned char smem[];
+  bf16* ring = reinterpret_cast<bf16*>(smem);           // [GA_WARPS][2][STAGE]
+  bf16* sQ = ring + GA_WARPS * 2 * STAGE;               // [16][KS]
+  __shared__ float sm_m[GA_WARPS][16], sm_l[GA_WARPS][16];
+  const int i = blockIdx.x, split = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int per = p.heads / p.kv_heads, subs = (per + 15) / 16;
+  const int hk = blockIdx.y / subs, h0 = hk * per + (blockIdx.y % subs) * 16;
+  const int ng = min(16, (hk + 1) * per - h0);
+  const int row = ra.rows != nullptr ? ra.rows[i] : i;
+  const int slot = ra.row_slot[row], pos = ra.row_pos[row];
+  const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
+  const bf16* kc = static_cast<const bf16*>(p.k_cache) + hk * p.dim_p;
+  const bf16* vc = static_cast<const bf16*>(p.v_cache) + hk * p.vdim_p;
+  const int lo = chunk_start(pos, p.chunk), n = pos + 1 - lo;
+  const int piece = (n + ra.splits - 1) / ra.splits;
+  const int t0 = lo + split * piece, t1 = min(pos + 1, t0 + piece);
+  bf16* mine = ring + warp * 2 * STAGE;
+  const int kch = p.dim_p / 8, vch = p.vdim_p / 8;
+  auto fetch = [&](int tb, int st) {                    // keys tb .. tb + 31 into a stage
+    const int t = tb + lane;
+    int page = 0;
+    if (t < t1) {
+      const int lp = t / RAGGED_PAGE;
+      page = lp < p.max_pages ? pt[lp] : -1;
+      if (page < 0 || page >= p.num_pages) {
+        record_status(p.status, ST_BOUNDS, row);
+        page = 0;
+      }
+    }
+    bf16* kd = mine + st * STAGE;
+    bf16* vd = kd + GA_KEYS * KS;
+    for (int x = lane; x < GA_KEYS * kch; x += 32) {
+      const int key = x / kch, c = x % kch;
+      const int pg = __shfl_sync(0xffffffffu, page, key);
+      const size_t cell = static_cast<size_t>(pg) * RAGGED_PAGE + (tb + key) % RAGGED_PAGE;
+      cp_async16_zfill(smem_u32(kd + key * KS + c * 8), kc + cell * p.kv_heads * p.dim_p + c * 8,
+                       tb + key < t1 ? 16 : 0);
+    }
+    for (int x = lane; x < GA_KEYS * vch; x += 32) {
+      const int key = x / vch, c = x % vch;
+      const int pg = __shfl_sync(0xffffffffu, page, key);
+      const size_t cell = static_cast<size_t>(pg) * RAGGED_PAGE + (tb + key) % RAGGED_PAGE;
+      cp_async16_zfill(smem_u32(vd + key * VS + c * 8), vc + cell * p.kv_heads * p.vdim_p + c * 8,
+                       tb + key < t1 ? 16 : 0);
+    }
+    cp_async_commit();
+  };
+  // zero the padding columns of this warp's ring, then start loading
+  for (int x = lane; x < 2 * GA_KEYS * (DC - p.dim_p); x += 32) {
+    const int r = x / (DC - p.dim_p), c = p.dim_p + x % (DC - p.dim_p);
+    mine[(r / GA_KEYS) * STAGE + (r % GA_KEYS) * KS + c] = __float2bfloat16(0.f);
+  }
+  for (int x = lane; x < 2 * GA_KEYS * (VC - p.vdim_p); x += 32) {
+    const int r = x / (VC - p.vdim_p), c = p.vdim_p + x % (VC - p.vdim_p);
+    mine[(r / GA_KEYS) * STAGE + GA_KEYS * KS + (r % GA_KEYS) * VS + c] = __float2bfloat16(0.f);
+  }
+  int tb = t0 + warp * GA_KEYS;
+  if (tb < t1) fetch(tb, 0);
+  const bf16* q = static_cast<const bf16*>(p.q) + (static_cast<size_t>(row) * p.heads + h0) * p.dim;
+  for (int x = tid; x < 16 * DC; x += GA_WARPS * 32) {
+    const int g = x / DC, d = x % DC;
+    sQ[g * KS + d] = g < ng && d < p.dim ? q[g * p.dim + d] : __float2bfloat16(0.f);
+  }
+  __syncthreads();
+  uint32_t qf[DC / 16][4];
+#pragma unroll
+  for (int k = 0; k < DC / 16; ++k)
+    ldsm4(qf[k], smem_u32(sQ + (lane & 15) * KS + k * 16 + (lane >> 4) * 8));
+  float o[VC / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+  for (int x = 0; x < VC / 8; ++x)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[x][j] = 0.f;
+  const float sl2 = p.scale * LOG2E;
+  for (int st = 0; tb < t1; tb += GA_WARPS * GA_KEYS, st ^= 1) {
+    if (tb + GA_WARPS * GA_KEYS < t1) {
+      fetch(tb + GA_WARPS * GA_KEYS, st ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncwarp();
+    const bf16* kb = mine + st * STAGE;
+    const bf16* vb = kb + GA_KEYS * KS;
+    float s[4][4];
+#pragma unroll
+    for (int x = 0; x < 4; ++x)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[x][j] = 0.f;
+#pragma unroll
+    for (int k = 0; k < DC / 16; ++k)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        uint32_t b[4];
+        ldsm4(b, smem_u32(kb + (x * 16 + (lane & 7) + (lane >> 4) * 8) * KS + k * 16 + ((lane >> 3) & 1) * 8));
+        mma_bf16(s[2 * x], qf[k], b[0], b[1]);
+        mma_bf16(s[2 * x + 1], qf[k], b[2], b[3]);
+      }
+    float mx[2] = {-INFINITY, -INFINITY}, c[2];
+#pragma unroll
+    for (int x = 0; x < 4; ++x)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int t = tb + x * 8 + (lane & 3) * 2 + (j & 1);
+        s[x][j] = t < t1 ? s[x][j] * sl2 : -INFINITY;
+        mx[j >> 1] = fmaxf(mx[j >> 1], s[x][j]);
+      }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+      const float mn = fmaxf(m[r], mx[r]);              // finite: the block has a key
+      c[r] = fast_exp2(m[r] - mn);
+      m[r] = mn;
+      l[r] *= c[r];
+    }
+#pragma unroll
+    for (int x = 0; x < 4; ++x)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        s[x][j] = fast_exp2(s[x][j] - m[j >> 1]);
+        l[j >> 1] += s[x][j];
+      }
+#pragma unroll
+    for (int x = 0; x < VC / 8; ++x)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[x][j] *= c[j >> 1];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      uint32_t ph[4], pl[4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const float u = s[2 * k + (x >> 1)][(x & 1) * 2], w = s[2 * k + (x >> 1)][(x & 1) * 2 + 1];
+        ph[x] = pack_bf16x2(u, w);
+        const float2 f = unpack_bf16x2(ph[x]);
+        pl[x] = pack_bf16x2(u - f.x, w - f.y);
+      }
+#pragma unroll
+      for (int x = 0; x < VC / 16; ++x) {
+        uint32_t b[4];
+        ldsm4_t(b, smem_u32(vb + (k * 16 + (lane & 15)) * VS + x * 16 + (lane >> 4) * 8));
+        mma_bf16(o[2 * x], ph, b[0], b[1]);
+        mma_bf16(o[2 * x + 1], ph, b[2], b[3]);
+        mma_bf16(o[2 * x], pl, b[0], b[1]);
+        mma_bf16(o[2 * x + 1], pl, b[2], b[3]);
+      }
+    }
+    __syncwarp();                                       // before the stage is filled again
+  }
+  // merge the warps through shared memory (the rings are free): [GA_WARPS][16][VC]
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+    if ((lane & 3) == 0) {
+      sm_m[warp][(lane >> 2) + 8 * r] = m[r];
+      sm_l[warp][(lane >> 2) + 8 * r] = l[r];
+    }
+  }
+  __syncthreads();
+  float* red = reinterpret_cast<float*>(smem);
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int g = (lane >> 2) + 8 * r;
+    float gm = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < GA_WARPS; ++w) gm = fmaxf(gm, sm_m[w][g]);
+    const float c = m[r] == -INFINITY ? 0.f : fast_exp2(m[r] - gm);
+#pragma unroll
+    for (int x = 0; x < VC / 8; ++x)
+      *reinterpret_cast<float2*>(red + (warp * 16 + g) * VC + x * 8 + (lane & 3) * 2) =
+          make_float2(o[x][2 * r] * c, o[x][2 * r + 1] * c);
+  }
+  __syncthreads();
+  for (int g = warp; g < ng; g += GA_WARPS) {
+    const int h = h0 + g;
+    float gm = -INFINITY, gl = 0.f;
+#pragma unroll
+    for (int w = 0; w < GA_WARPS; ++w) gm = fmaxf(gm, sm_m[w][g]);
+#pragma unroll
+    for (int w = 0; w < GA_WARPS; ++w)
+      gl += sm_m[w][g] == -INFINITY ? 0.f : sm_l[w][g] * fast_exp2(sm_m[w][g] - gm);
+    const size_t part = (static_cast<size_t>(i) * p.heads + h) * ra.splits + split;
+    const float dn = ra.splits == 1 ? gate_of<bf16>(p, row, h) / denom<bf16>(p, h, gm, gl) : 1.f;
+    for (int d = lane; d < p.vdim; d += 32) {
+      float v = 0.f;
+#pragma unroll
+      for (int w = 0; w < GA_WARPS; ++w) v += red[(w * 16 + g) * VC + d];
+      if (ra.splits == 1)
+        static_cast<bf16*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] = __float2bfloat16(v * dn);
+      else
+        ra.part_o[part * p.vdim + d] = v;
+    }
+    if (ra.splits > 1 && lane == 0) {
+      ra.part_ml[part * 2] = gm;
+      ra.part_ml[part * 2 + 1] = gl;
+    }
+  }
+}
+
+template <int DC, int VC>
+static int launch_group(const RowsArgs& a, int n, cudaStream_t st) {
+  constexpr int ring = GA_WARPS * 2 * GA_KEYS * (DC + 8 + VC + 8) * 2 + 16 * (DC + 8) * 2;
+  constexpr int merge = GA_WARPS * 16 * VC * 4;
+  constexpr int smem = ring > merge ? ring : merge;
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(ragged_attn_group_kernel<DC, VC>,
+                             cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      return -4;
+    set = true;
+  }
+  const int per = a.a.heads / a.a.kv_heads;
+  dim3 grid(n, a.a.kv_heads * ((per + 15) / 16), a.splits);
+  ragged_attn_group_kernel<DC, VC><<<grid, GA_WARPS * 32, smem, st>>>(a);
+  if (a.splits > 1) {
+    dim3 g2(n, a.a.heads);
+    ragged_attn_merge_kernel<__nv_bfloat16><<<g2, 64, 0, st>>>(a);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+template <int DC>
+static int launch_group_v(const RowsArgs& a, int n, cudaStream_t st) {
+  if (a.a.vdim <= 64) return launch_group<DC, 64>(a, n, st);
+  return launch_group<DC, 128>(a, n, st);
+}
+
 template <int DC, int VC>
 static int launch_tiles(const TilesArgs& a, int tiles, cudaStream_t st) {
   const int smem = (2 * RAGGED_PAGE * (DC + 8) + 2 * RAGGED_PAGE * (VC + 8) + TA_ROWS * (DC + 8)) * 2;
@@ -544,7 +786,9 @@ extern "C" int cb_ragged_attn_rows(const void* q, const void* k_cache, const voi
   a.rows = rows; a.row_slot = row_slot; a.row_pos = row_pos; a.splits = splits;
   a.part_o = part_o; a.part_ml = part_ml;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return f32 ? launch_rows_d<float>(a, n, st) : launch_rows_d<__nv_bfloat16>(a, n, st);
+  if (f32) return launch_rows_d<float>(a, n, st);
+  if (dim > 128 || vdim > 128) return launch_rows<__nv_bfloat16, 4>(a, n, st);
+  return dim <= 64 ? launch_group_v<64>(a, n, st) : launch_group_v<128>(a, n, st);
 }
 
 extern "C" int cb_ragged_attn_tiles(const void* q, const void* k_cache, const void* v_cache,

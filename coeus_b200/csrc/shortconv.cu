@@ -210,6 +210,26 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
 // The same with V = 4 consecutive channels per thread for a whole tile of tokens: the taps of a
 // thread's channels stay in registers and every projected row is loaded once.  dim, vdim and half
 // are multiples of four.  The threads of a block are its units (see above), nothing else.
+constexpr int CONV_AHEAD = 8;      // rows loaded before the first of them is used
+
+template <typename T>
+struct Packed4;
+template <>
+struct Packed4<float> {
+  float4 v;
+  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ void get(float* f) const { f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
+};
+template <>
+struct Packed4<__nv_bfloat16> {
+  uint2 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ void get(float* f) const {
+    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+};
+
 template <typename T, int TAPS>
 struct Window {
   static constexpr int V = 4;
@@ -231,12 +251,12 @@ struct Window {
     }
   }
   // takes the next row in, y = convolution at its token
-  __device__ __forceinline__ void next(const T* row, float* y) {
+  __device__ __forceinline__ void next(const Packed4<T>& row, float* y) {
 #pragma unroll
     for (int j = 0; j + 1 < TAPS; ++j)
 #pragma unroll
       for (int i = 0; i < V; ++i) u[j][i] = u[j + 1][i];
-    load_vec<V>(row, u[TAPS - 1]);
+    row.get(u[TAPS - 1]);
 #pragma unroll
     for (int i = 0; i < V; ++i) y[i] = 0.f;
 #pragma unroll
@@ -247,7 +267,7 @@ struct Window {
 };
 
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(512) shortconv_attn_tile_kernel(const AttnPre p) {
+__global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre p) {
   constexpr int V = 4;
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -261,6 +281,9 @@ __global__ void __launch_bounds__(512) shortconv_attn_tile_kernel(const AttnPre 
   const int heads_u = (per + 1) * head_u;
   const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
   __shared__ int s_page[2];
+  __shared__ __align__(16) float2 s_rope[CONV_TILE * 128];    // half <= 128
+  for (int i = threadIdx.x; i < (t1 - off) * p.half; i += blockDim.x)
+    s_rope[i] = p.rope[static_cast<size_t>(row0 + off) * p.half + i];
   if (threadIdx.x < 2) {                     // a tile of 16 tokens touches at most two pages
     const int lp = (pos0 + off) / RAGGED_PAGE + threadIdx.x;
     int page = lp < p.max_pages ? p.page_table[static_cast<size_t>(slot) * p.max_pages + lp] : -1;
@@ -289,13 +312,26 @@ __global__ void __launch_bounds__(512) shortconv_attn_tile_kernel(const AttnPre 
     wa.start(ci, c, col, channels, row0, off, slot, has_state);
     if (pair) wb.start(ci, c + p.half, col + p.half, channels, row0, off, slot, has_state);
     const float lam = is_v && p.mix_mode == 2 ? *p.lambda : 0.f;
-#pragma unroll 2
-    for (int t = off; t < t1; ++t) {
+    const bool mixes = is_v && p.mix_mode == 2;
+    T* vf0 = static_cast<T*>(p.v_first) + static_cast<size_t>(row0) * ci.kv_heads * vdim + g * vdim + d;
+    for (int tb = off; tb < t1; tb += CONV_AHEAD) {
+    Packed4<T> ra[CONV_AHEAD], rb[CONV_AHEAD];
+#pragma unroll
+    for (int i = 0; i < CONV_AHEAD; ++i) {
+      const int t = min(tb + i, t1 - 1);
+      const T* src = raw + static_cast<ptrdiff_t>(t) * ci.ld + col;
+      ra[i].load(src);
+      if (pair) rb[i].load(src + p.half);
+      else if (mixes) rb[i].load(vf0 + static_cast<size_t>(t) * ci.kv_heads * vdim);
+    }
+#pragma unroll
+    for (int i = 0; i < CONV_AHEAD; ++i) {
+      const int t = tb + i;
+      if (t >= t1) break;
       const int row = row0 + t, pos = pos0 + t;
       const int page = s_page[pos / RAGGED_PAGE - lp0];
-      const T* src = raw + static_cast<ptrdiff_t>(t) * ci.ld + col;
       float a[V];
-      wa.next(src, a);
+      wa.next(ra[i], a);
       const size_t cell = (static_cast<size_t>(max(page, 0)) * RAGGED_PAGE + pos % RAGGED_PAGE) * ci.kv_heads + g;
       T* dst = is_q ? static_cast<T*>(p.q) + static_cast<size_t>(row) * qc + c
                     : (is_v ? static_cast<T*>(p.v_cache) + cell * p.vdim_p + d
@@ -303,14 +339,14 @@ __global__ void __launch_bounds__(512) shortconv_attn_tile_kernel(const AttnPre 
       const bool ok = is_q || page >= 0;
       if (pair) {
         float b[V], oa[V], ob[V];
-        wb.next(src + p.half, b);
-        const float4* cs = reinterpret_cast<const float4*>(p.rope + static_cast<size_t>(row) * p.half + d);
+        wb.next(rb[i], b);
+        const float4* cs = reinterpret_cast<const float4*>(&s_rope[(t - off) * p.half + d]);
         const float4 x = cs[0], y = cs[1];
         const float cc[V] = {x.x, x.z, y.x, y.z}, ss[V] = {x.y, x.w, y.y, y.w};
 #pragma unroll
-        for (int i = 0; i < V; ++i) {
-          oa[i] = a[i] * cc[i] - b[i] * ss[i];
-          ob[i] = b[i] * cc[i] + a[i] * ss[i];
+        for (int x = 0; x < V; ++x) {
+          oa[x] = a[x] * cc[x] - b[x] * ss[x];
+          ob[x] = b[x] * cc[x] + a[x] * ss[x];
         }
         if (ok) {
           store_vec<V>(dst, oa);
@@ -323,16 +359,13 @@ __global__ void __launch_bounds__(512) shortconv_attn_tile_kernel(const AttnPre 
         }
         continue;
       }
-      if (is_v && p.mix_mode != 0) {
-        T* vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d;
-        if (p.mix_mode == 1) {
-          store_vec<V>(vf, a);
-        } else {
-          float f[V];
-          load_vec<V>(vf, f);
+      if (mixes) {
+        float f[V];
+        rb[i].get(f);
 #pragma unroll
-          for (int i = 0; i < V; ++i) a[i] = (1.f - lam) * a[i] + lam * f[i];
-        }
+        for (int x = 0; x < V; ++x) a[x] = (1.f - lam) * a[x] + lam * f[x];
+      } else if (is_v && p.mix_mode == 1) {
+        store_vec<V>(vf0 + static_cast<size_t>(t) * ci.kv_heads * vdim, a);
       }
       if (ok) store_vec<V>(dst, a);
       if (!is_q && p.k_rows != nullptr) {
@@ -340,6 +373,7 @@ __global__ void __launch_bounds__(512) shortconv_attn_tile_kernel(const AttnPre 
                      : static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d;
         store_vec<V>(kr, a);
       }
+    }
     }
   }
   if (off == 0) {
@@ -509,7 +543,8 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(cons
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float qscale = 1.0f / sqrtf(static_cast<float>(dim));
   const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
-  const int half_t = t1 - off > CONV_TILE / 2 ? CONV_TILE / 2 : CONV_TILE;
+  constexpr int half_t = CONV_TILE / 2;
+  static_assert(half_t == CONV_AHEAD, "a warp loads its rows in one go");
   const int n_qk = t1 - off > half_t ? 2 : 1;
   const int n_v = (per * vdim + 127) / 128, n_g = per * ((p.dim_p + 127) / 128);
   for (int u = warp; u < n_qk + n_v + n_g; u += CONV_THREADS / 32) {
@@ -522,12 +557,20 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(cons
         const int cq = g * dim + (in ? d : 0);
         wq.start(ci, cq, cq, channels, row0, ta, slot, has_state);
         wk.start(ci, qc + cq, ci.koff + cq, channels, row0, ta, slot, has_state);
-#pragma unroll 2
-        for (int t = ta; t < tb; ++t) {
-          const T* src = raw + static_cast<ptrdiff_t>(t) * ci.ld + cq;
+        Packed4<T> rq4[CONV_AHEAD], rk4[CONV_AHEAD];
+#pragma unroll
+        for (int i = 0; i < CONV_AHEAD; ++i) {
+          const T* src = raw + static_cast<ptrdiff_t>(min(ta + i, tb - 1)) * ci.ld + cq;
+          rq4[i].load(src);
+          rk4[i].load(src + ci.koff);
+        }
+#pragma unroll
+        for (int i = 0; i < CONV_AHEAD; ++i) {
+          const int t = ta + i;
+          if (t >= tb) break;
           float q[V], k[V], sq = 0.f, sk = 0.f, dot = 0.f;
-          wq.next(src, q);
-          wk.next(src + ci.koff, k);
+          wq.next(rq4[i], q);
+          wk.next(rk4[i], k);
 #pragma unroll
           for (int x = 0; x < V; ++x) {
             q[x] = in ? silu_act<T>(q[x]) : 0.f;
@@ -601,13 +644,20 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(cons
         const int c = g * per * vdim + i;
         Window<T, TAPS> w;
         w.start(ci, 2 * qc + c, ci.voff + c, channels, row0, off, slot, has_state);
-#pragma unroll 4
-        for (int t = off; t < t1; ++t) {
-          float y[V];
-          w.next(raw + static_cast<ptrdiff_t>(t) * ci.ld + ci.voff + c, y);
+        for (int tb = off; tb < t1; tb += CONV_AHEAD) {
+          Packed4<T> rv[CONV_AHEAD];
 #pragma unroll
-          for (int x = 0; x < V; ++x) y[x] = silu_act<T>(y[x]);
-          store_f32<V>(p.v + static_cast<size_t>(row0 + t) * ci.heads * vdim + c, y);
+          for (int j = 0; j < CONV_AHEAD; ++j)
+            rv[j].load(raw + static_cast<ptrdiff_t>(min(tb + j, t1 - 1)) * ci.ld + ci.voff + c);
+#pragma unroll
+          for (int j = 0; j < CONV_AHEAD; ++j) {
+            if (tb + j >= t1) break;
+            float y[V];
+            w.next(rv[j], y);
+#pragma unroll
+            for (int x = 0; x < V; ++x) y[x] = silu_act<T>(y[x]);
+            store_f32<V>(p.v + static_cast<size_t>(row0 + tb + j) * ci.heads * vdim + c, y);
+          }
         }
       }
     } else {
@@ -618,16 +668,24 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(cons
         const float rate = expf(p.A_log[h]);
         float b[V] = {};
         if (in) load_f32<V>(p.dt_bias + h * dim + d, b);
-#pragma unroll 4
-        for (int t = off; t < t1; ++t) {
-          float f[V] = {};
-          if (in) {
-            float a[V];
-            load_f32<V>(p.a + static_cast<size_t>(row0 + t) * p.lda + h * dim + d, a);
+        for (int tb = off; tb < t1; tb += CONV_AHEAD) {
+          float4 ra[CONV_AHEAD];
 #pragma unroll
-            for (int x = 0; x < V; ++x) f[x] = expf(-rate * softplus_exact(a[x] + b[x]));
+          for (int j = 0; j < CONV_AHEAD; ++j) {
+            ra[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (in)
+              ra[j] = *reinterpret_cast<const float4*>(
+                  p.a + static_cast<size_t>(row0 + min(tb + j, t1 - 1)) * p.lda + h * dim + d);
           }
-          store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row0 + t) * p.dim_p + d, f);
+#pragma unroll
+          for (int j = 0; j < CONV_AHEAD; ++j) {
+            if (tb + j >= t1) break;
+            const float a[V] = {ra[j].x, ra[j].y, ra[j].z, ra[j].w};
+            float f[V];
+#pragma unroll
+            for (int x = 0; x < V; ++x) f[x] = in ? expf(-rate * softplus_exact(a[x] + b[x])) : 0.f;
+            store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row0 + tb + j) * p.dim_p + d, f);
+          }
         }
       }
     }
@@ -652,7 +710,7 @@ template <typename T>
 static int launch_conv_attn(const AttnPre& p, dim3 grid, bool vec, cudaStream_t st) {
   if (vec) {
     const int units = (p.c.heads / p.c.kv_heads + 1) * ((p.c.dim - p.half) / 4) + p.c.vdim / 4;
-    const int threads = min(512, (units + 31) / 32 * 32);
+    const int threads = min(256, (units + 31) / 32 * 32);
     switch (p.c.taps) {
       case 2: shortconv_attn_tile_kernel<T, 2><<<grid, threads, 0, st>>>(p); break;
       case 3: shortconv_attn_tile_kernel<T, 3><<<grid, threads, 0, st>>>(p); break;
@@ -714,7 +772,7 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
   p.mix_mode = mix_mode; p.status = status;
   p.k_rows = k_rows; p.v_rows = v_rows;
   const bool vec = taps >= 2 && taps <= 4 && dim % 4 == 0 && vdim % 4 == 0 && half % 4 == 0 &&
-                   ld % 8 == 0 && koff % 8 == 0 && voff % 8 == 0;
+                   half <= 128 && ld % 8 == 0 && koff % 8 == 0 && voff % 8 == 0;
   dim3 grid(tiles, kv_heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return f32 ? launch_conv_attn<float>(p, grid, vec, st)

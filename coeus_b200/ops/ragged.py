@@ -359,7 +359,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     n = batch.n_rows
     if n:
         per = heads // kv_heads
-        ctas = n * kv_heads * (1 if per <= 8 else (per + 7) // 8)
+        ctas = n * kv_heads * ((per + 15) // 16)
         ctx = max_ctx or batch.max_ctx
         ctx = min(ctx, chunk) if chunk else ctx
         # a CTA takes 128 keys at a time
