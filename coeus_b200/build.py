@@ -40,7 +40,7 @@ NVCC_FLAGS = [
 
 
 SERVING_SOURCES = ("gemm", "ragged_rows", "shortconv", "delta_scan", "linear_f32", "linear_skinny",
-                   "ragged_attn")
+                   "ragged_attn", "attention_fwd")
 
 
 def _nvcc() -> str:

@@ -47,6 +47,12 @@ struct AttnFwdArgs {
   int drop_thr;
   uint32_t drop_key;
   float drop_scale;
+  // pieces of unequal length instead of B sequences of S rows: piece b is the rows pieces[b].x ..
+  // pieces[b].x + pieces[b].y - 1 (at most S), which attend to one another only; null: none
+  const int2* pieces;
+  const float* sink;           // [nh] logits that enter the denominator only, or null
+  const __nv_bfloat16* gate;   // [rows, ldg], column h: head h's output times its sigmoid; or null
+  int ldg;
 };
 
 // Optional device timeline of CTA 0 (clock64 stamps; see cb_attn_fwd_set_trace): softmax warp 0
@@ -105,6 +111,8 @@ struct AFWalk {
   // position
   int wave, j, t;
   int b, h, qa;          // batch, head, first query tile of the pair
+  int row0, len;         // first row and rows of the sequence (or piece)
+  const int2* pieces;
   int n0, n1, nmax;      // key tiles of tile A / B (0: the tile does not exist)
   int kv_seq;            // how many (item, j) groups came before this one: the K/V ring position
   bool valid;
@@ -118,6 +126,8 @@ struct AFWalk {
     n_bh = p.B * p.nh;
     n_items = n_pairs * n_bh;
     causal = p.causal;
+    pieces = p.pieces;
+    len = p.S;
     n_waves = (n_items + gridDim.x - 1) / gridDim.x;
     wave = -1;
     kv_seq = -1;
@@ -137,6 +147,16 @@ struct AFWalk {
       b = bh / nh;
       h = bh % nh;
       qa = 2 * pair;
+      if (pieces != nullptr) {
+        const int2 pc = pieces[b];
+        row0 = pc.x;
+        len = pc.y;
+        n_q_tiles = (len + AF_BM - 1) / AF_BM;
+        n_kv_tiles = (len + bkv - 1) / bkv;
+        if (qa >= n_q_tiles) continue;             // a shorter piece ends before this pair
+      } else {
+        row0 = b * len;
+      }
       n0 = causal ? min(n_kv_tiles, ((qa + 1) * AF_BM + bkv - 1) / bkv) : n_kv_tiles;
       n1 = qa + 1 >= n_q_tiles ? 0
            : (causal ? min(n_kv_tiles, ((qa + 2) * AF_BM + bkv - 1) / bkv) : n_kv_tiles);
@@ -234,7 +254,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       AFWalk w;
       w.init(p, BKV);
       while (w.valid && ok) {
-        const int row0 = w.b * p.S;
+        const int row0 = w.row0;
         const int h = w.h, hk = w.h / group, qa = w.qa;
         const int n0 = w.n0, n1 = w.n1, nmax = w.nmax;
         auto load_q = [&](int t) {
@@ -488,8 +508,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (tr) tr[tri] = clock64();
       tc_fence_after();
       const int kv0 = j * BKV;
-      const bool need_mask = (p.causal && kv0 + BKV - 1 > q0) || (kv0 + BKV > p.S);
-      const int kv_limit = p.causal ? min(q_idx, p.S - 1) : (p.S - 1);  // last visible key
+      const bool need_mask = (p.causal && kv0 + BKV - 1 > q0) || (kv0 + BKV > w.len);
+      const int kv_limit = p.causal ? min(q_idx, w.len - 1) : (w.len - 1);  // last visible key
       uint32_t v[BKV];
 #pragma unroll
       for (int c = 0; c < BKV / 32; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v + c * 32);
@@ -610,10 +630,14 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       }
       tc_fence_after();
       const float lsum = (l[0] + l[1]) + (l[2] + l[3]);
-      const float inv_l = lsum > 0.f ? 1.0f / lsum : 0.f;
-      const bool row_ok = q_idx < p.S;
-      __nv_bfloat16* orow =
-          p.O + (static_cast<size_t>(w.b) * p.S + q_idx) * p.ldo + static_cast<size_t>(w.h) * DH;
+      float inv_l = lsum > 0.f ? 1.0f / lsum : 0.f;
+      const bool row_ok = q_idx < w.len;
+      const size_t out_row = static_cast<size_t>(w.row0) + q_idx;
+      if (p.sink != nullptr)
+        inv_l = 1.0f / (lsum + exp2f(p.sink[w.h] * 1.4426950408889634f - m_used));
+      if (p.gate != nullptr && row_ok)
+        inv_l /= 1.0f + expf(-__bfloat162float(p.gate[out_row * p.ldg + w.h]));
+      __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * DH;
 #pragma unroll 1
       for (int c = 0; c < DH / 32; ++c) {
         uint32_t o[32];
@@ -705,6 +729,10 @@ extern "C" int cb_attn_fwd_dropout(const void* q, const void* k, const void* v, 
   a.scale_log2 = scale * 1.4426950408889634f;
   a.causal = causal;
   a.status = status;
+  a.pieces = nullptr;
+  a.sink = nullptr;
+  a.gate = nullptr;
+  a.ldg = 0;
   a.drop_thr = drop_thr;
   a.drop_key = drop_key;
   a.drop_scale = 256.0f / static_cast<float>(256 - drop_thr);
@@ -725,4 +753,40 @@ extern "C" int cb_attn_fwd(const void* q, const void* k, const void* v, void* o,
                            void* stream) {
   return cb_attn_fwd_dropout(q, k, v, o, lse, B, S, nh, nkv, dh, ldq, ldk, ldv, ldo, scale, causal,
                              poly, 0, 0u, status, max_ctas, stream);
+}
+
+// Causal attention inside every piece of a ragged batch: n_pieces (first row, rows) pairs over the
+// `rows` rows of q, k, v and o, none longer than max_len.  sink (fp32 [nh]) is a logit per head that
+// enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view) multiplies head
+// h's output by its sigmoid; both may be null.  scale > 0.
+extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, void* o, int rows,
+                                  const void* pieces, int n_pieces, int max_len, int nh, int nkv,
+                                  int dh, int ldq, int ldk, int ldv, int ldo, float scale,
+                                  const float* sink, const void* gate, int ldg, int* status,
+                                  void* stream) {
+  using namespace cb;
+  if (dh != 64 && dh != 128) return -1;
+  if (rows <= 0 || n_pieces <= 0 || max_len <= 0 || nh <= 0 || nkv <= 0 || (nh % nkv) != 0 ||
+      (ldo % 8) != 0 || !(scale > 0.f))
+    return -2;
+  CUtensorMap tq, tk, tv;
+  const uint32_t bkv = dh == 64 ? AFCfg<64>::BKV : AFCfg<128>::BKV;
+  if (make_tmap_bf16_2d(&tq, q, static_cast<uint64_t>(nh) * dh, rows, ldq, 64, AF_BM) != 0) return -3;
+  if (make_tmap_bf16_2d(&tk, k, static_cast<uint64_t>(nkv) * dh, rows, ldk, 64, bkv) != 0) return -4;
+  if (make_tmap_bf16_2d(&tv, v, static_cast<uint64_t>(nkv) * dh, rows, ldv, 64, bkv) != 0) return -5;
+  AttnFwdArgs a = {};
+  a.B = n_pieces; a.S = max_len; a.nh = nh; a.nkv = nkv;
+  a.O = static_cast<__nv_bfloat16*>(o);
+  a.ldo = ldo;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.causal = 1;
+  a.status = status;
+  a.drop_scale = 1.0f;
+  a.pieces = static_cast<const int2*>(pieces);
+  a.sink = sink;
+  a.gate = static_cast<const __nv_bfloat16*>(gate);
+  a.ldg = ldg;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dh == 64 ? launch_attn_fwd<64, false>(tq, tk, tv, a, 0, st)
+                  : launch_attn_fwd<128, false>(tq, tk, tv, a, 0, st);
 }

@@ -273,6 +273,7 @@ struct TilesArgs {
   Entries e;
   const int* tile_entry;   // [tiles]
   const int* tile_off;     // [tiles] first token of the tile inside its entry
+  const int* tile_len;     // [tiles] its tokens, at most TA_ROWS
 };
 
 template <int DC, int VC>   // dim <= DC, vdim <= VC, multiples of 32
@@ -286,7 +287,7 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
   bf16* sQ = sV + 2 * RAGGED_PAGE * VS;                          // [TA_ROWS][KS]
   const int e = ta.tile_entry[blockIdx.x], off = ta.tile_off[blockIdx.x], h = blockIdx.y;
   const int hk = h / (p.heads / p.kv_heads);
-  const int row0 = ta.e.row0[e] + off, len = min(TA_ROWS, ta.e.len[e] - off);
+  const int row0 = ta.e.row0[e] + off, len = min(TA_ROWS, ta.tile_len[blockIdx.x]);
   const int pos0 = ta.e.pos0[e] + off, slot = ta.e.slot[e];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
@@ -797,14 +798,14 @@ extern "C" int cb_ragged_attn_tiles(const void* q, const void* k_cache, const vo
                                     float scale, const float* sink, const void* gate, int ldg,
                                     void* out, int ldo, const int* slot, const int* row0,
                                     const int* len, const int* pos0, const int* tile_entry,
-                                    const int* tile_off, int tiles, int* status, void* stream) {
+                                    const int* tile_off, const int* tile_len, int tiles, int* status, void* stream) {
   TilesArgs a;
   const int rc = fill_attn(a.a, q, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
                            dim, vdim, dim_p, vdim_p, chunk, scale, sink, gate, ldg, out, ldo, status);
   if (rc != 0) return rc;
   if (tiles <= 0) return -5;
   a.e.slot = slot; a.e.row0 = row0; a.e.len = len; a.e.pos0 = pos0;
-  a.tile_entry = tile_entry; a.tile_off = tile_off;
+  a.tile_entry = tile_entry; a.tile_off = tile_off; a.tile_len = tile_len;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (dim <= 64) return launch_tiles_v<64>(a, tiles, st);
   if (dim <= 128) return launch_tiles_v<128>(a, tiles, st);

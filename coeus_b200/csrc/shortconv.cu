@@ -210,7 +210,7 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
 // The same with V = 4 consecutive channels per thread for a whole tile of tokens: the taps of a
 // thread's channels stay in registers and every projected row is loaded once.  dim, vdim and half
 // are multiples of four.  The threads of a block are its units (see above), nothing else.
-constexpr int CONV_AHEAD = 8;      // rows loaded before the first of them is used
+constexpr int CONV_AHEAD = 4;      // rows loaded before the first of them is used
 
 template <typename T>
 struct Packed4;
@@ -267,7 +267,7 @@ struct Window {
 };
 
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre p) {
+__global__ void __launch_bounds__(256, 2) shortconv_attn_tile_kernel(const AttnPre p) {
   constexpr int V = 4;
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -277,11 +277,13 @@ __global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre 
   const int qc = ci.heads * dim, kc = ci.kv_heads * dim;
   const int channels = qc + kc + ci.kv_heads * vdim;
   const int t1 = min(off + CONV_TILE, len);
-  const int pair_u = p.half / V, head_u = (dim - p.half) / V;
-  const int heads_u = (per + 1) * head_u;
+  // units: the rotated pairs of all heads, then their other vectors, then the values, so that
+  // the threads of a warp mostly do the same
+  const int pair_u = p.half / V, plain_u = (dim - 2 * p.half) / V;
+  const int pairs_u = (per + 1) * pair_u, heads_u = pairs_u + (per + 1) * plain_u;
   const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
   __shared__ int s_page[2];
-  __shared__ __align__(16) float2 s_rope[CONV_TILE * 128];    // half <= 128
+  extern __shared__ __align__(16) float2 s_rope[];           // [CONV_TILE][half]
   for (int i = threadIdx.x; i < (t1 - off) * p.half; i += blockDim.x)
     s_rope[i] = p.rope[static_cast<size_t>(row0 + off) * p.half + i];
   if (threadIdx.x < 2) {                     // a tile of 16 tokens touches at most two pages
@@ -294,20 +296,20 @@ __global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre 
   __syncthreads();
   const int lp0 = (pos0 + off) / RAGGED_PAGE;
   for (int u = threadIdx.x; u < heads_u + vdim / V; u += blockDim.x) {
-    const bool is_v = u >= heads_u;
-    const int hi = is_v ? 0 : u / head_u, k = is_v ? 0 : u % head_u;
-    const bool is_q = !is_v && hi < per, pair = !is_v && k < pair_u;
-    int c, col, d;
+    const bool is_v = u >= heads_u, pair = u < pairs_u;
+    int c, col, d, hi = 0;
     if (is_v) {
       d = (u - heads_u) * V;
       c = qc + kc + g * vdim + d;
       col = ci.voff + g * vdim + d;
     } else {
-      d = pair ? k * V : p.half + k * V;     // plain units start behind the second half
-      const int base = is_q ? (g * per + hi) * dim : g * dim;
-      c = (is_q ? 0 : qc) + base + d;
-      col = (is_q ? 0 : ci.koff) + base + d;
+      hi = pair ? u / pair_u : (u - pairs_u) / plain_u;
+      d = pair ? u % pair_u * V : 2 * p.half + (u - pairs_u) % plain_u * V;
+      const int base = hi < per ? (g * per + hi) * dim : g * dim;
+      c = (hi < per ? 0 : qc) + base + d;
+      col = (hi < per ? 0 : ci.koff) + base + d;
     }
+    const bool is_q = !is_v && hi < per;
     Window<T, TAPS> wa, wb;
     wa.start(ci, c, col, channels, row0, off, slot, has_state);
     if (pair) wb.start(ci, c + p.half, col + p.half, channels, row0, off, slot, has_state);
@@ -530,7 +532,7 @@ __device__ __forceinline__ float silu_act(float x) {
 // warps: q and k of the two halves of the tile (a token's 128 or 256 channels are one warp's, the
 // norms are warp sums), the values and the decays in pieces of 128 channels.
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(const DeltaPre p) {
+__global__ void __launch_bounds__(CONV_THREADS, 4) shortconv_delta_tile_kernel(const DeltaPre p) {
   constexpr int V = 4;
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -544,7 +546,6 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(cons
   const float qscale = 1.0f / sqrtf(static_cast<float>(dim));
   const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
   constexpr int half_t = CONV_TILE / 2;
-  static_assert(half_t == CONV_AHEAD, "a warp loads its rows in one go");
   const int n_qk = t1 - off > half_t ? 2 : 1;
   const int n_v = (per * vdim + 127) / 128, n_g = per * ((p.dim_p + 127) / 128);
   for (int u = warp; u < n_qk + n_v + n_g; u += CONV_THREADS / 32) {
@@ -557,16 +558,17 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(cons
         const int cq = g * dim + (in ? d : 0);
         wq.start(ci, cq, cq, channels, row0, ta, slot, has_state);
         wk.start(ci, qc + cq, ci.koff + cq, channels, row0, ta, slot, has_state);
+        for (int t0 = ta; t0 < tb; t0 += CONV_AHEAD) {
         Packed4<T> rq4[CONV_AHEAD], rk4[CONV_AHEAD];
 #pragma unroll
         for (int i = 0; i < CONV_AHEAD; ++i) {
-          const T* src = raw + static_cast<ptrdiff_t>(min(ta + i, tb - 1)) * ci.ld + cq;
+          const T* src = raw + static_cast<ptrdiff_t>(min(t0 + i, tb - 1)) * ci.ld + cq;
           rq4[i].load(src);
           rk4[i].load(src + ci.koff);
         }
 #pragma unroll
         for (int i = 0; i < CONV_AHEAD; ++i) {
-          const int t = ta + i;
+          const int t = t0 + i;
           if (t >= tb) break;
           float q[V], k[V], sq = 0.f, sk = 0.f, dot = 0.f;
           wq.next(rq4[i], q);
@@ -597,6 +599,7 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_tile_kernel(cons
             store_f32<V>(p.k + cell * p.dim_p + d, k);
           }
           if (lane == 0) p.kq[cell] = dot * rq * rk;
+        }
         }
       } else {
         for (int t = ta; t < tb; ++t) {
@@ -710,11 +713,12 @@ template <typename T>
 static int launch_conv_attn(const AttnPre& p, dim3 grid, bool vec, cudaStream_t st) {
   if (vec) {
     const int units = (p.c.heads / p.c.kv_heads + 1) * ((p.c.dim - p.half) / 4) + p.c.vdim / 4;
+    const int smem = CONV_TILE * p.half * static_cast<int>(sizeof(float2));
     const int threads = min(256, (units + 31) / 32 * 32);
     switch (p.c.taps) {
-      case 2: shortconv_attn_tile_kernel<T, 2><<<grid, threads, 0, st>>>(p); break;
-      case 3: shortconv_attn_tile_kernel<T, 3><<<grid, threads, 0, st>>>(p); break;
-      default: shortconv_attn_tile_kernel<T, 4><<<grid, threads, 0, st>>>(p);
+      case 2: shortconv_attn_tile_kernel<T, 2><<<grid, threads, smem, st>>>(p); break;
+      case 3: shortconv_attn_tile_kernel<T, 3><<<grid, threads, smem, st>>>(p); break;
+      default: shortconv_attn_tile_kernel<T, 4><<<grid, threads, smem, st>>>(p);
     }
   } else {
     shortconv_attn_kernel<T, 1, 0><<<grid, CONV_THREADS, 0, st>>>(p);

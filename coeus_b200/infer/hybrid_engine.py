@@ -45,6 +45,15 @@ class HybridEngine(InferenceEngine):
         self.use_graph = (model.device.type == "cuda") if use_graph is None else use_graph
         self._graphs: Dict[int, tuple] = {}
         self._tiles = model.device.type == "cuda" and model.dtype == torch.bfloat16
+        mixers = [self.cfg.layers[l].mixer for l in self.cfg.attention_layers()]
+        self._plans = [R.AttnPlan(a.chunk, self._pieces(a)) for a in mixers]
+
+    def _pieces(self, a: AttentionSpec) -> bool:
+        return self._tiles and R.pieces_allowed(a.dim, a.vdim, a.chunk, a.scale)
+
+    def _batch(self, entries: List[Entry], into: Optional[R.RaggedBatch] = None) -> R.RaggedBatch:
+        return R.RaggedBatch(entries, self.m.device, tile_rows=self._tiles, into=into,
+                             plans=self._plans)
 
     # ------------------------------------------------------------------ cache and state
     def open_slots(self, max_seqs: int, max_len: int, num_pages: Optional[int] = None
@@ -94,14 +103,19 @@ class HybridEngine(InferenceEngine):
         first = s.v_mix and v_first is None
         if first:
             v_first = torch.empty((b.T, s.kv_heads * s.vdim), dtype=raw.dtype, device=raw.device)
+        k_rows = v_rows = None
+        if b.n_big and self._pieces(s):
+            k_rows = torch.empty((b.T, s.kv_heads * s.dim), dtype=raw.dtype, device=raw.device)
+            v_rows = torch.empty((b.T, s.kv_heads * s.vdim), dtype=raw.dtype, device=raw.device)
         q = R.shortconv_attn(
             raw, layer.seg["k"], layer.seg["v"], layer.conv, self.state[l, "conv"], s.heads,
             s.kv_heads, s.dim, s.vdim, b, rope.get(layer.rope_key), c.k[i], c.v[i], c.page_table,
             v_first=v_first if s.v_mix else None, mix=layer.mix if s.v_mix and not first else None,
-            write_first=first)
+            write_first=first, k_rows=k_rows, v_rows=v_rows)
         R.ragged_attention(q, c.k[i], c.v[i], c.page_table, b, s.heads, s.kv_heads, s.dim, s.vdim,
                            s.scale, cat[:, :layer.out_dim], chunk=s.chunk, sink=layer.sink,
-                           gate=raw[:, layer.seg["g"]:], max_ctx=max_ctx)
+                           gate=raw[:, layer.seg["g"]:], max_ctx=max_ctx,
+                           k_rows=k_rows, v_rows=v_rows)
         return v_first
 
     def _delta(self, l: int, layer, raw: torch.Tensor, cat: torch.Tensor, b: R.RaggedBatch) -> None:
@@ -167,7 +181,7 @@ class HybridEngine(InferenceEngine):
                 all(len(e.tokens) == 1 and len(e.want) == 1 and e.pos0 > 0 for e in entries):
             out = self._decode_graph(entries)
         else:
-            b = R.RaggedBatch(entries, self.m.device, tile_rows=self._tiles)
+            b = self._batch(entries)
             out = self._forward(b, b.max_ctx, layer_out)
         for e in entries:
             c.set_length(e.slot, e.pos0 + len(e.tokens))
@@ -178,7 +192,7 @@ class HybridEngine(InferenceEngine):
         the entries themselves: they write the same cache cells and would advance the recurrent
         state, which is put back."""
         n = len(entries)
-        b = R.RaggedBatch(entries, self.m.device, tile_rows=self._tiles)
+        b = self._batch(entries)
         ctx = self.cache.page_table.shape[1] * PAGE
         idx = b.slot.long()
         keep = {k: t[idx].clone() for k, t in self.state.tensors.items()}
@@ -201,7 +215,7 @@ class HybridEngine(InferenceEngine):
         if g is None:
             g = self._capture(entries)
         else:
-            R.RaggedBatch(entries, self.m.device, tile_rows=self._tiles, into=g[1])
+            self._batch(entries, into=g[1])
             g[1].slots_host = [e.slot for e in entries]
         self._graph_pos = None
         g[0].replay()

@@ -20,6 +20,7 @@ from .decode import PAGE
 CONV_TILE = 16        # tokens per block of the convolution kernels
 ATTN_TILE = 64        # query rows per block of the tensor-core attention kernel
 ROWS_MAX = 4          # entries of at most this many tokens take the row kernel
+MIN_PIECE = 64        # chunks from this size on are worth a piece of their own
 _F = ctypes.c_float
 
 
@@ -38,13 +39,40 @@ class Entry:
     want: Sequence[int] = ()
 
 
+@dataclass(frozen=True)
+class AttnPlan:
+    """How the long entries of a batch go through attention under one mask.  A piece is a run of
+    rows that starts at a chunk's start (or at position 0), so that its rows see one another and
+    nothing else: it needs no cache and takes the piece kernel.  What comes before an entry's
+    first piece sees cached keys too and goes in tiles of ``ATTN_TILE`` rows."""
+
+    chunk: Optional[int]
+    pieces: bool              # whether the layer's sizes allow the piece kernel
+
+
+def pieces_allowed(dim: int, vdim: int, chunk: Optional[int], scale: float) -> bool:
+    return dim == vdim and dim in (64, 128) and scale > 0 and (chunk is None or chunk >= MIN_PIECE)
+
+
+def _cut(plan: AttnPlan, pos0: int, n: int):
+    """``(rows before the first piece, [(offset, rows), ...])`` of an entry of ``n`` tokens."""
+    if not plan.pieces:
+        return n, []
+    if plan.chunk is None:
+        return (n, []) if pos0 else (0, [(0, n)])
+    head = min(n, -pos0 % plan.chunk)
+    return head, [(o, min(plan.chunk, n - o)) for o in range(head, n, plan.chunk)]
+
+
 class RaggedBatch:
     """Index arrays of one step, in one int32 buffer (one host-to-device copy).  ``tile_rows``
-    says whether long entries may take the tensor-core attention kernel (bf16 models on CUDA);
-    otherwise every row is listed for the row kernel."""
+    says whether long entries may take the tensor-core attention kernels (bf16 models on CUDA);
+    otherwise every row is listed for the row kernel.  ``plans`` are the attention plans the
+    model's layers will ask for."""
 
     def __init__(self, entries: List[Entry], device, tile_rows: bool = True,
-                 into: Optional["RaggedBatch"] = None) -> None:
+                 into: Optional["RaggedBatch"] = None,
+                 plans: Sequence[AttnPlan] = (AttnPlan(None, False),)) -> None:
         n = len(entries)
         lens = [len(e.tokens) for e in entries]
         if not n or min(lens) < 1:
@@ -60,9 +88,6 @@ class RaggedBatch:
         row_slot = np.repeat(np.asarray([e.slot for e in entries], dtype=np.int32), lens)
         ct = [(i, o) for i, m in enumerate(lens) for o in range(0, m, CONV_TILE)]
         big = [i for i, m in enumerate(lens) if tile_rows and m > ROWS_MAX]
-        # tiles with the most keys first
-        at = sorted(((i, o) for i in big for o in range(0, lens[i], ATTN_TILE)),
-                    key=lambda t: -(entries[t[0]].pos0 + t[1]))
         small = [i for i in range(n) if i not in set(big)]
         rows = np.concatenate([np.arange(row0[i], row0[i + 1], dtype=np.int32) for i in small]) \
             if small else np.zeros(0, np.int32)
@@ -71,8 +96,22 @@ class RaggedBatch:
         parts = [pos, np.asarray(self.pos0_host, np.int32), tokens, row_slot,
                  np.asarray(self.slots_host, np.int32), row0[:n], np.asarray(lens, np.int32),
                  np.asarray([c[0] for c in ct], np.int32), np.asarray([c[1] for c in ct], np.int32),
-                 rows, np.asarray([c[0] for c in at], np.int32),
-                 np.asarray([c[1] for c in at], np.int32), want]
+                 rows, want]
+        self.plans, cols = {}, len(parts)
+        for plan in dict.fromkeys(plans):
+            tiles, pieces = [], []
+            for i in big:
+                head, ps = _cut(plan, entries[i].pos0, lens[i])
+                tiles += [(i, o, min(ATTN_TILE, head - o)) for o in range(0, head, ATTN_TILE)]
+                pieces += [(int(row0[i]) + o, m) for o, m in ps]
+            tiles.sort(key=lambda t: -(entries[t[0]].pos0 + t[1]))     # the most keys first
+            pieces.sort(key=lambda t: -t[1])
+            if pieces and sum(len(x) for x in parts) % 2:              # pairs are read as int2
+                parts.append(np.zeros(1, np.int32))
+            self.plans[plan] = (len(tiles), len(pieces), max([m for _, m in pieces], default=0),
+                                len(parts))
+            parts += [np.asarray(pieces, np.int32).reshape(-1),
+                      *np.asarray(tiles, np.int32).reshape(-1, 3).T]
         host = torch.from_numpy(np.concatenate(parts).astype(np.int32, copy=False))
         if into is None:
             self.buf = host.to(device)
@@ -86,10 +125,16 @@ class RaggedBatch:
             views.append(self.buf[o:o + len(part)])
             o += len(part)
         (self.pos, self.pos0, self.tokens, self.row_slot, self.slot, self.row0, self.len,
-         self.conv_entry, self.conv_off, self.rows, self.attn_entry, self.attn_off,
-         self.want) = views
+         self.conv_entry, self.conv_off, self.rows, self.want) = views[:cols]
+        self._views = views
         self.positions = self.buf[:self.T + n]       # pos and pos0: what a decode step advances
-        self.n_conv, self.n_rows, self.n_attn, self.n_want = len(ct), len(rows), len(at), len(want)
+        self.n_conv, self.n_rows, self.n_want = len(ct), len(rows), len(want)
+        self.n_big = len(big)
+
+    def plan(self, plan: AttnPlan):
+        """``(tiles, pieces, longest piece, piece array, tile entries, offsets, lengths)``."""
+        n_tiles, n_pieces, longest, at = self.plans[plan]
+        return (n_tiles, n_pieces, longest, *self._views[at:at + 4])
 
     def entry_args(self):
         return _p(self.slot), _p(self.row0), _p(self.len), _p(self.pos0)
@@ -309,14 +354,17 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      page_table: torch.Tensor, batch: RaggedBatch, heads: int, kv_heads: int,
                      dim: int, vdim: int, scale: float, out: torch.Tensor, *,
                      chunk: Optional[int] = None, sink: Optional[torch.Tensor] = None,
-                     gate: Optional[torch.Tensor] = None, max_ctx: Optional[int] = None
-                     ) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, max_ctx: Optional[int] = None,
+                     k_rows: Optional[torch.Tensor] = None,
+                     v_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of every query row over the cached keys of its own sequence, restricted to
     the row's chunk (positions with the same ``pos // chunk``) when ``chunk`` is given.  ``sink``
     (fp32 ``[heads]``) is a logit that enters the softmax denominator only; ``gate`` (a view whose
     column ``h`` belongs to head ``h``) multiplies head ``h``'s output by its sigmoid.  Query head
     ``h`` reads key/value head ``h // (heads // kv_heads)``.  ``out`` is a ``[rows, heads * vdim]``
-    view; ``max_ctx`` bounds the keys of any row (it only chooses how many CTAs share a row)."""
+    view; ``max_ctx`` bounds the keys of any row (it only chooses how many CTAs share a row).  With
+    this step's ``k_rows`` and ``v_rows`` at hand, runs of rows that see no earlier step go through
+    the tcgen05 kernel (:class:`AttnPlan`; the batch must have been built with the layer's plan)."""
     T = q.shape[0]
     if not q.is_cuda:
         per = heads // kv_heads
@@ -352,10 +400,20 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
               k_cache.shape[0], heads, kv_heads, dim, vdim, k_cache.shape[-1], v_cache.shape[-1],
               chunk or 0, _F(scale), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0,
               _p(out), out.stride(0))
-    if batch.n_attn:
-        rc = lib.cb_ragged_attn_tiles(*common, *batch.entry_args(), _p(batch.attn_entry),
-                                      _p(batch.attn_off), batch.n_attn, st, _lib.stream_ptr())
-        _lib.check_rc(rc, "cb_ragged_attn_tiles")
+    if batch.n_big:
+        n_tiles, n_pieces, longest, pieces, t_entry, t_off, t_len = batch.plan(
+            AttnPlan(chunk, k_rows is not None))
+        if n_tiles:
+            rc = lib.cb_ragged_attn_tiles(*common, *batch.entry_args(), _p(t_entry), _p(t_off),
+                                          _p(t_len), n_tiles, st, _lib.stream_ptr())
+            _lib.check_rc(rc, "cb_ragged_attn_tiles")
+        if n_pieces:
+            rc = lib.cb_attn_fwd_pieces(
+                _p(q), _p(k_rows), _p(v_rows), _p(out), T, _p(pieces), n_pieces, longest, heads,
+                kv_heads, dim, q.stride(0), k_rows.stride(0), v_rows.stride(0), out.stride(0),
+                _F(scale), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0, st,
+                _lib.stream_ptr())
+            _lib.check_rc(rc, "cb_attn_fwd_pieces")
     n = batch.n_rows
     if n:
         per = heads // kv_heads

@@ -33,6 +33,14 @@ def config(kind):
                 L(A(2, 2, 24, 136, 3, 0.2, 64, 16, 50.0, False), M(72)),
                 L(D(1, 1, 130, 16, 4, 8, 24), M(40)),
             ))
+    if kind == "square":      # key and value heads of one size: prompts in pieces
+        return H.HybridConfig(
+            vocab_size=120, hidden_dim=72, norm_eps=1e-5, logit_softcap=15.0, layers=(
+                L(A(4, 2, 64, 64, 4, 0.15, 96, 32, 1e4, True), M(96)),
+                L(D(2, 1, 32, 48, 4, 8, 8), M(40)),
+                L(A(2, 2, 64, 64, 3, 0.12, 64, 64, 1e3, True), M(96)),
+                L(A(1, 1, 128, 128, 2, 0.1, None, 128, 1e5, False), None),
+            ))
     if kind == "delta":       # recurrence only
         return H.HybridConfig(
             vocab_size=40, hidden_dim=24, norm_eps=1e-5, logit_softcap=5.0, layers=(
@@ -258,8 +266,9 @@ def rnd(shape, seed, device, dtype=torch.float32):
     return torch.randn(shape, generator=g).to(dtype).to(device)
 
 
-def batch_of(entries, device, tiles):
-    return R.RaggedBatch([R.Entry(s, p, [0] * n) for s, p, n in entries], device, tile_rows=tiles)
+def batch_of(entries, device, tiles, chunk=None):
+    return R.RaggedBatch([R.Entry(s, p, [0] * n) for s, p, n in entries], device, tile_rows=tiles,
+                         plans=[R.AttnPlan(chunk, x) for x in (False, True)])
 
 
 def check_norms(device, dtype, tol):
@@ -361,7 +370,8 @@ def check_attention(device, dtype, tol):
     g = torch.Generator().manual_seed(0)
     for H_, Gk, d, dv, chunk in ((4, 1, 64, 48, 120), (6, 2, 40, 24, 50), (2, 2, 10, 7, 9),
                                  (9, 1, 72, 128, 200), (3, 3, 136, 200, 64), (4, 4, 128, 64, None),
-                                 (2, 1, 16, 16, 1)):
+                                 (2, 1, 16, 16, 1), (20, 1, 24, 32, 90), (4, 2, 64, 64, 100),
+                                 (2, 1, 128, 128, 64), (3, 1, 64, 64, None), (2, 2, 128, 128, 300)):
         n = 260
         k = torch.randn((n, Gk, d), generator=g).to(dtype)
         v = torch.randn((n, Gk, dv), generator=g).to(dtype)
@@ -378,7 +388,8 @@ def check_attention(device, dtype, tol):
         sink = torch.linspace(-3.0, 4.0, H_)
         span = [p for c in (chunk or 64, 64) for e in range(c, n, c) for p in (e - 1, e, e + 1)]
         pos = sorted({0, 1, n - 1, *[p for p in span if p < n]})[:40]
-        for start, m in [(p, 1) for p in pos] + [(0, 70), (50, 100), (117, 66), (n - 6, 6)]:
+        rows_too = dtype == torch.bfloat16 and R.pieces_allowed(d, dv, chunk, scale)
+        for start, m in [(p, 1) for p in pos] + [(0, 70), (0, 260), (50, 100), (117, 66), (n - 6, 6)]:
             m = min(m, n - start)
             q = torch.randn((m, H_, d), generator=g)
             # each row points at one key: its chunk's first, the one before it, itself, or a far one
@@ -389,11 +400,12 @@ def check_attention(device, dtype, tol):
                 q[r] += 3.0 * k[j].double().repeat_interleave(H_ // Gk, 0)
             q = q.to(dtype)
             gate = torch.randn((m, H_ + 3), generator=g).to(dtype)
-            b = batch_of([(0, start, m)], device, tiles=dtype == torch.bfloat16)
+            b = batch_of([(0, start, m)], device, dtype == torch.bfloat16, chunk)
             out = torch.full((m, H_ * dv + 8), 5.0, dtype=dtype, device=device)
-            R.ragged_attention(q.reshape(m, -1).to(device), kc, vc, table, b, H_, Gk, d, dv, scale,
-                               out[:, :H_ * dv], chunk=chunk, sink=sink.to(device),
-                               gate=gate.to(device)[:, 2:])
+            args = (q.reshape(m, -1).to(device), kc, vc, table, b, H_, Gk, d, dv, scale,
+                    out[:, :H_ * dv])
+            kw = dict(chunk=chunk, sink=sink.to(device), gate=gate.to(device)[:, 2:])
+            R.ragged_attention(*args, **kw)
             want = torch.zeros(m, H_, dv, dtype=torch.float64)
             for r in range(m):
                 i = start + r
@@ -403,6 +415,11 @@ def check_attention(device, dtype, tol):
                     want[r, h] = plain.sink_softmax(s, sink[h].double()) @ v[js, h // (H_ // Gk)].double()
             want *= torch.sigmoid(gate[:, 2:2 + H_].double())[:, :, None]
             assert rel(out[:, :H_ * dv], want.reshape(m, -1)) < tol, (H_, d, chunk, start, m)
+            if rows_too:       # the same with this step's keys and values at hand, row by row
+                out.fill_(5.0)
+                R.ragged_attention(*args, **kw, k_rows=k[start:start + m].reshape(m, -1).to(device),
+                                   v_rows=v[start:start + m].reshape(m, -1).to(device))
+                assert rel(out[:, :H_ * dv], want.reshape(m, -1)) < tol, (H_, d, chunk, start, m)
             assert float((out[:, H_ * dv:].float() - 5.0).abs().max()) == 0
 
 

@@ -32,7 +32,7 @@ def test_mechanism(check, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=["fp32", "bf16"])
-@pytest.mark.parametrize("kind", ["odd", "wide", "delta", "attn"])
+@pytest.mark.parametrize("kind", ["odd", "wide", "square", "delta", "attn"])
 @pytest.mark.parametrize("check", cases.MODEL_CHECKS, ids=lambda c: c.__name__[6:])
 def test_model(kind, check, dtype):
     check(bench(kind, dtype))
