@@ -207,56 +207,62 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
   }
 }
 
-// The same with V = 4 consecutive channels per thread for a whole tile of tokens: the taps of a
-// thread's channels stay in registers and every projected row is loaded once.  dim, vdim and half
-// are multiples of four.  The threads of a block are its units (see above), nothing else.
-constexpr int CONV_AHEAD = 4;      // rows loaded before the first of them is used
-
+// The tile kernels do the same with V = 4 consecutive channels per thread for a whole tile of
+// tokens.  The projected rows of the tile and the TAPS - 1 before it are staged in shared memory in
+// one go, and the taps of a thread's channels stay in registers.  dim, vdim and half are multiples
+// of four.
 template <typename T>
-struct Packed4;
-template <>
-struct Packed4<float> {
-  float4 v;
-  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float4*>(p); }
-  __device__ __forceinline__ void get(float* f) const { f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
-};
-template <>
-struct Packed4<__nv_bfloat16> {
-  uint2 v;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint2*>(p); }
-  __device__ __forceinline__ void get(float* f) const {
-    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
-    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+__device__ __forceinline__ void cp_async_quad(uint32_t dst, const T* src, bool in) {
+  if constexpr (sizeof(T) == 2)
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(dst), "l"(src), "r"(in ? 8 : 0)
+                 : "memory");
+  else
+    cp_async16_zfill(dst, src, in ? 16 : 0);
+}
+
+// Four channels of one thread: projection column col (state channel c) for the rows off - (TAPS-1)
+// .. off + nt - 1 of an entry, to shared memory at dst with a pitch of `pitch` elements.
+template <typename T, int TAPS>
+__device__ __forceinline__ void stage_quad(const ConvIn& p, int c, int col, int channels, int row0,
+                                           int off, int nt, int slot, bool has_state, T* dst,
+                                           int pitch) {
+  const T* raw = static_cast<const T*>(p.raw) + static_cast<ptrdiff_t>(row0) * p.ld + col;
+  const T* st = static_cast<const T*>(p.state) + static_cast<ptrdiff_t>(slot) * (TAPS - 1) * channels + c;
+  const uint32_t d = smem_u32(dst);
+#pragma unroll
+  for (int j = 0; j < TAPS - 1; ++j) {
+    const int o = off - (TAPS - 1) + j;
+    const bool in = o >= 0 || has_state;
+    const T* src = o >= 0 ? raw + static_cast<ptrdiff_t>(o) * p.ld
+                          : (in ? st + static_cast<ptrdiff_t>(TAPS - 1 + o) * channels : raw);
+    cp_async_quad<T>(d + j * pitch * sizeof(T), src, in);
   }
-};
+#pragma unroll 4
+  for (int j = 0; j < nt; ++j)
+    cp_async_quad<T>(d + (TAPS - 1 + j) * pitch * sizeof(T),
+                     raw + static_cast<ptrdiff_t>(off + j) * p.ld, true);
+}
 
 template <typename T, int TAPS>
 struct Window {
   static constexpr int V = 4;
   float w[TAPS][V], u[TAPS][V];
-  // loads the taps of channels c.. and the TAPS - 1 rows before token t
-  __device__ __forceinline__ void start(const ConvIn& p, int c, int col, int channels, int row0,
-                                        int t, int slot, bool has_state) {
-    const T* raw = static_cast<const T*>(p.raw) + static_cast<ptrdiff_t>(row0) * p.ld + col;
-    const T* st = static_cast<const T*>(p.state) + static_cast<ptrdiff_t>(slot) * (TAPS - 1) * channels + c;
+  __device__ __forceinline__ void taps(const ConvIn& p, int c, int channels) {
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * channels + c, w[j]);
-#pragma unroll
-    for (int j = 1; j < TAPS; ++j) {
-      const int o = t - TAPS + j;
-#pragma unroll
-      for (int i = 0; i < V; ++i) u[j][i] = 0.f;
-      if (o >= 0) load_vec<V>(raw + static_cast<ptrdiff_t>(o) * p.ld, u[j]);
-      else if (has_state) load_vec<V>(st + static_cast<ptrdiff_t>(TAPS - 1 + o) * channels, u[j]);
-    }
   }
-  // takes the next row in, y = convolution at its token
-  __device__ __forceinline__ void next(const Packed4<T>& row, float* y) {
+  // the rows before the first token t: rows t .. t + TAPS - 2 of the staged tile
+  __device__ __forceinline__ void start(const T* s, int pitch) {
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) load_vec<V>(s + (j - 1) * pitch, u[j]);
+  }
+  // takes the next staged row in, y = convolution at its token
+  __device__ __forceinline__ void next(const T* row, float* y) {
 #pragma unroll
     for (int j = 0; j + 1 < TAPS; ++j)
 #pragma unroll
       for (int i = 0; i < V; ++i) u[j][i] = u[j + 1][i];
-    row.get(u[TAPS - 1]);
+    load_vec<V>(row, u[TAPS - 1]);
 #pragma unroll
     for (int i = 0; i < V; ++i) y[i] = 0.f;
 #pragma unroll
@@ -267,7 +273,7 @@ struct Window {
 };
 
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256, 2) shortconv_attn_tile_kernel(const AttnPre p) {
+__global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre p) {
   constexpr int V = 4;
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -281,101 +287,118 @@ __global__ void __launch_bounds__(256, 2) shortconv_attn_tile_kernel(const AttnP
   // the threads of a warp mostly do the same
   const int pair_u = p.half / V, plain_u = (dim - 2 * p.half) / V;
   const int pairs_u = (per + 1) * pair_u, heads_u = pairs_u + (per + 1) * plain_u;
-  const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
+  const int nt = t1 - off, cols = (per + 1) * dim + vdim;   // staged columns: q heads | k | v
+  extern __shared__ __align__(16) unsigned char conv_smem[];
+  float2* s_rope = reinterpret_cast<float2*>(conv_smem);     // [CONV_TILE][half]
+  T* s_raw = reinterpret_cast<T*>(s_rope + CONV_TILE * p.half);
   __shared__ int s_page[2];
-  extern __shared__ __align__(16) float2 s_rope[];           // [CONV_TILE][half]
-  for (int i = threadIdx.x; i < (t1 - off) * p.half; i += blockDim.x)
+  for (int i = threadIdx.x * V; i < cols; i += blockDim.x * V) {
+    const int c = i < per * dim ? g * per * dim + i
+                : (i < (per + 1) * dim ? qc + g * dim + (i - per * dim)
+                                       : qc + kc + g * vdim + (i - (per + 1) * dim));
+    stage_quad<T, TAPS>(ci, c, raw_col(ci, c), channels, row0, off, nt, slot, has_state, s_raw + i, cols);
+  }
+  cp_async_commit();
+  for (int i = threadIdx.x; i < nt * p.half; i += blockDim.x)
     s_rope[i] = p.rope[static_cast<size_t>(row0 + off) * p.half + i];
+  const int lp0 = (pos0 + off) / RAGGED_PAGE;
   if (threadIdx.x < 2) {                     // a tile of 16 tokens touches at most two pages
-    const int lp = (pos0 + off) / RAGGED_PAGE + threadIdx.x;
+    const int lp = lp0 + threadIdx.x;
     int page = lp < p.max_pages ? p.page_table[static_cast<size_t>(slot) * p.max_pages + lp] : -1;
     const bool used = lp <= (pos0 + t1 - 1) / RAGGED_PAGE;
     if (used && (page < 0 || page >= p.num_pages)) record_status(p.status, ST_BOUNDS, row0 + off);
     s_page[threadIdx.x] = used && page >= 0 && page < p.num_pages ? page : -1;
   }
+  cp_async_wait<0>();
   __syncthreads();
-  const int lp0 = (pos0 + off) / RAGGED_PAGE;
   for (int u = threadIdx.x; u < heads_u + vdim / V; u += blockDim.x) {
     const bool is_v = u >= heads_u, pair = u < pairs_u;
-    int c, col, d, hi = 0;
+    int c, d, i, hi = 0;                     // channel, place in the head, staged column
     if (is_v) {
       d = (u - heads_u) * V;
       c = qc + kc + g * vdim + d;
-      col = ci.voff + g * vdim + d;
+      i = (per + 1) * dim + d;
     } else {
       hi = pair ? u / pair_u : (u - pairs_u) / plain_u;
       d = pair ? u % pair_u * V : 2 * p.half + (u - pairs_u) % plain_u * V;
-      const int base = hi < per ? (g * per + hi) * dim : g * dim;
-      c = (hi < per ? 0 : qc) + base + d;
-      col = (hi < per ? 0 : ci.koff) + base + d;
+      c = (hi < per ? (g * per + hi) * dim : qc + g * dim) + d;
+      i = hi * dim + d;
     }
     const bool is_q = !is_v && hi < per;
+    const T* src = s_raw + i;
     Window<T, TAPS> wa, wb;
-    wa.start(ci, c, col, channels, row0, off, slot, has_state);
-    if (pair) wb.start(ci, c + p.half, col + p.half, channels, row0, off, slot, has_state);
-    const float lam = is_v && p.mix_mode == 2 ? *p.lambda : 0.f;
-    const bool mixes = is_v && p.mix_mode == 2;
-    T* vf0 = static_cast<T*>(p.v_first) + static_cast<size_t>(row0) * ci.kv_heads * vdim + g * vdim + d;
-    for (int tb = off; tb < t1; tb += CONV_AHEAD) {
-    Packed4<T> ra[CONV_AHEAD], rb[CONV_AHEAD];
-#pragma unroll
-    for (int i = 0; i < CONV_AHEAD; ++i) {
-      const int t = min(tb + i, t1 - 1);
-      const T* src = raw + static_cast<ptrdiff_t>(t) * ci.ld + col;
-      ra[i].load(src);
-      if (pair) rb[i].load(src + p.half);
-      else if (mixes) rb[i].load(vf0 + static_cast<size_t>(t) * ci.kv_heads * vdim);
+    wa.taps(ci, c, channels);
+    wa.start(src, cols);
+    if (pair) {
+      wb.taps(ci, c + p.half, channels);
+      wb.start(src + p.half, cols);
     }
-#pragma unroll
-    for (int i = 0; i < CONV_AHEAD; ++i) {
-      const int t = tb + i;
-      if (t >= t1) break;
-      const int row = row0 + t, pos = pos0 + t;
-      const int page = s_page[pos / RAGGED_PAGE - lp0];
+    src += (TAPS - 1) * cols;
+    // where the first token goes, and how far apart the tokens of a page are
+    T* kr = nullptr;
+    T* vf = nullptr;
+    T* dst = nullptr;
+    int step = qc, row_step = kc;
+    if (is_q) {
+      dst = static_cast<T*>(p.q) + static_cast<size_t>(row0 + off) * qc + c;
+    } else if (is_v) {
+      step = ci.kv_heads * p.vdim_p;
+      row_step = ci.kv_heads * vdim;
+      if (p.k_rows != nullptr) kr = static_cast<T*>(p.v_rows) + static_cast<size_t>(row0 + off) * row_step + g * vdim + d;
+      if (p.mix_mode != 0) vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row0 + off) * row_step + g * vdim + d;
+    } else {
+      step = ci.kv_heads * p.dim_p;
+      if (p.k_rows != nullptr) kr = static_cast<T*>(p.k_rows) + static_cast<size_t>(row0 + off) * kc + g * dim + d;
+    }
+    T* cache = static_cast<T*>(is_v ? p.v_cache : p.k_cache);
+    const int in_cell = is_v ? g * p.vdim_p + d : g * p.dim_p + d;
+    const float lam = is_v && p.mix_mode == 2 ? *p.lambda : 0.f;
+#pragma unroll 2
+    for (int t = 0; t < nt; ++t, src += cols) {
+      if (!is_q) {
+        const int pos = pos0 + off + t;
+        const int page = s_page[pos / RAGGED_PAGE - lp0];
+        dst = page < 0 ? nullptr
+                       : cache + (static_cast<size_t>(page) * RAGGED_PAGE + pos % RAGGED_PAGE) * step + in_cell;
+      }
       float a[V];
-      wa.next(ra[i], a);
-      const size_t cell = (static_cast<size_t>(max(page, 0)) * RAGGED_PAGE + pos % RAGGED_PAGE) * ci.kv_heads + g;
-      T* dst = is_q ? static_cast<T*>(p.q) + static_cast<size_t>(row) * qc + c
-                    : (is_v ? static_cast<T*>(p.v_cache) + cell * p.vdim_p + d
-                            : static_cast<T*>(p.k_cache) + cell * p.dim_p + d);
-      const bool ok = is_q || page >= 0;
+      wa.next(src, a);
       if (pair) {
         float b[V], oa[V], ob[V];
-        wb.next(rb[i], b);
-        const float4* cs = reinterpret_cast<const float4*>(&s_rope[(t - off) * p.half + d]);
+        wb.next(src + p.half, b);
+        const float4* cs = reinterpret_cast<const float4*>(s_rope + t * p.half + d);
         const float4 x = cs[0], y = cs[1];
         const float cc[V] = {x.x, x.z, y.x, y.z}, ss[V] = {x.y, x.w, y.y, y.w};
 #pragma unroll
-        for (int x = 0; x < V; ++x) {
-          oa[x] = a[x] * cc[x] - b[x] * ss[x];
-          ob[x] = b[x] * cc[x] + a[x] * ss[x];
+        for (int k = 0; k < V; ++k) {
+          oa[k] = a[k] * cc[k] - b[k] * ss[k];
+          ob[k] = b[k] * cc[k] + a[k] * ss[k];
         }
-        if (ok) {
+        if (dst != nullptr) {
           store_vec<V>(dst, oa);
           store_vec<V>(dst + p.half, ob);
         }
-        if (!is_q && p.k_rows != nullptr) {
-          T* kr = static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d;
+        if (kr != nullptr) {
           store_vec<V>(kr, oa);
           store_vec<V>(kr + p.half, ob);
         }
-        continue;
-      }
-      if (mixes) {
-        float f[V];
-        rb[i].get(f);
+      } else {
+        if (vf != nullptr) {
+          if (p.mix_mode == 1) {
+            store_vec<V>(vf, a);
+          } else {
+            float f[V];
+            load_vec<V>(vf, f);
 #pragma unroll
-        for (int x = 0; x < V; ++x) a[x] = (1.f - lam) * a[x] + lam * f[x];
-      } else if (is_v && p.mix_mode == 1) {
-        store_vec<V>(vf0 + static_cast<size_t>(t) * ci.kv_heads * vdim, a);
+            for (int k = 0; k < V; ++k) a[k] = (1.f - lam) * a[k] + lam * f[k];
+          }
+          vf += row_step;
+        }
+        if (dst != nullptr) store_vec<V>(dst, a);
+        if (kr != nullptr) store_vec<V>(kr, a);
       }
-      if (ok) store_vec<V>(dst, a);
-      if (!is_q && p.k_rows != nullptr) {
-        T* kr = is_v ? static_cast<T*>(p.v_rows) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d
-                     : static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d;
-        store_vec<V>(kr, a);
-      }
-    }
+      if (is_q) dst += qc;
+      if (kr != nullptr) kr += row_step;
     }
   }
   if (off == 0) {
@@ -532,7 +555,7 @@ __device__ __forceinline__ float silu_act(float x) {
 // warps: q and k of the two halves of the tile (a token's 128 or 256 channels are one warp's, the
 // norms are warp sums), the values and the decays in pieces of 128 channels.
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(CONV_THREADS, 4) shortconv_delta_tile_kernel(const DeltaPre p) {
+__global__ void __launch_bounds__(CONV_THREADS, 6) shortconv_delta_tile_kernel(const DeltaPre p) {
   constexpr int V = 4;
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -545,152 +568,120 @@ __global__ void __launch_bounds__(CONV_THREADS, 4) shortconv_delta_tile_kernel(c
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float qscale = 1.0f / sqrtf(static_cast<float>(dim));
   const T* raw = static_cast<const T*>(ci.raw) + static_cast<ptrdiff_t>(row0) * ci.ld;
-  constexpr int half_t = CONV_TILE / 2;
-  const int n_qk = t1 - off > half_t ? 2 : 1;
-  const int n_v = (per * vdim + 127) / 128, n_g = per * ((p.dim_p + 127) / 128);
-  for (int u = warp; u < n_qk + n_v + n_g; u += CONV_THREADS / 32) {
-    if (u < n_qk) {
-      const int ta = off + u * half_t, tb = min(ta + half_t, t1);
-      if (dim <= 128) {
-        const int d = lane * V;
-        const bool in = d < dim;
-        Window<T, TAPS> wq, wk;
-        const int cq = g * dim + (in ? d : 0);
-        wq.start(ci, cq, cq, channels, row0, ta, slot, has_state);
-        wk.start(ci, qc + cq, ci.koff + cq, channels, row0, ta, slot, has_state);
-        for (int t0 = ta; t0 < tb; t0 += CONV_AHEAD) {
-        Packed4<T> rq4[CONV_AHEAD], rk4[CONV_AHEAD];
-#pragma unroll
-        for (int i = 0; i < CONV_AHEAD; ++i) {
-          const T* src = raw + static_cast<ptrdiff_t>(min(t0 + i, tb - 1)) * ci.ld + cq;
-          rq4[i].load(src);
-          rk4[i].load(src + ci.koff);
-        }
-#pragma unroll
-        for (int i = 0; i < CONV_AHEAD; ++i) {
-          const int t = t0 + i;
-          if (t >= tb) break;
-          float q[V], k[V], sq = 0.f, sk = 0.f, dot = 0.f;
-          wq.next(rq4[i], q);
-          wk.next(rk4[i], k);
-#pragma unroll
-          for (int x = 0; x < V; ++x) {
-            q[x] = in ? silu_act<T>(q[x]) : 0.f;
-            k[x] = in ? silu_act<T>(k[x]) : 0.f;
-            sq += q[x] * q[x];
-            sk += k[x] * k[x];
-            dot += q[x] * k[x];
-          }
-#pragma unroll
-          for (int o = 16; o > 0; o >>= 1) {
-            sq += __shfl_xor_sync(0xffffffffu, sq, o);
-            sk += __shfl_xor_sync(0xffffffffu, sk, o);
-            dot += __shfl_xor_sync(0xffffffffu, dot, o);
-          }
-          const float rq = qscale / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f);
-          const size_t cell = static_cast<size_t>(g) * p.rows + row0 + t;
-#pragma unroll
-          for (int x = 0; x < V; ++x) {
-            q[x] *= rq;
-            k[x] *= rk;
-          }
-          if (d < p.dim_p) {
-            store_f32<V>(p.q + cell * p.dim_p + d, q);
-            store_f32<V>(p.k + cell * p.dim_p + d, k);
-          }
-          if (lane == 0) p.kq[cell] = dot * rq * rk;
-        }
-        }
-      } else {
-        for (int t = ta; t < tb; ++t) {
-          float q[2][V], k[2][V], sq = 0.f, sk = 0.f, dot = 0.f;
-#pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            const int d = (lane + 32 * i) * V;
-#pragma unroll
-            for (int x = 0; x < V; ++x) q[i][x] = k[i][x] = 0.f;
-            if (d < dim) {
-              conv_at<T, V, TAPS>(ci, g * dim + d, g * dim + d, channels, row0, t, slot, has_state, q[i]);
-              conv_at<T, V, TAPS>(ci, qc + g * dim + d, ci.koff + g * dim + d, channels, row0, t, slot, has_state, k[i]);
-            }
-#pragma unroll
-            for (int x = 0; x < V; ++x) {
-              q[i][x] = silu_act<T>(q[i][x]);
-              k[i][x] = silu_act<T>(k[i][x]);
-              sq += q[i][x] * q[i][x];
-              sk += k[i][x] * k[i][x];
-              dot += q[i][x] * k[i][x];
-            }
-          }
-          const float rq = qscale / sqrtf(warp_sum(sq) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f);
-          dot = warp_sum(dot);
-          const size_t cell = static_cast<size_t>(g) * p.rows + row0 + t;
-#pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            const int d = (lane + 32 * i) * V;
-#pragma unroll
-            for (int x = 0; x < V; ++x) {
-              q[i][x] *= rq;
-              k[i][x] *= rk;
-            }
-            if (d < p.dim_p) {
-              store_f32<V>(p.q + cell * p.dim_p + d, q[i]);
-              store_f32<V>(p.k + cell * p.dim_p + d, k[i]);
-            }
-          }
-          if (lane == 0) p.kq[cell] = dot * rq * rk;
-        }
-      }
-    } else if (u < n_qk + n_v) {
-      const int i = ((u - n_qk) * 32 + lane) * V;
-      if (i < per * vdim) {
-        const int c = g * per * vdim + i;
-        Window<T, TAPS> w;
-        w.start(ci, 2 * qc + c, ci.voff + c, channels, row0, off, slot, has_state);
-        for (int tb = off; tb < t1; tb += CONV_AHEAD) {
-          Packed4<T> rv[CONV_AHEAD];
-#pragma unroll
-          for (int j = 0; j < CONV_AHEAD; ++j)
-            rv[j].load(raw + static_cast<ptrdiff_t>(min(tb + j, t1 - 1)) * ci.ld + ci.voff + c);
-#pragma unroll
-          for (int j = 0; j < CONV_AHEAD; ++j) {
-            if (tb + j >= t1) break;
-            float y[V];
-            w.next(rv[j], y);
-#pragma unroll
-            for (int x = 0; x < V; ++x) y[x] = silu_act<T>(y[x]);
-            store_f32<V>(p.v + static_cast<size_t>(row0 + tb + j) * ci.heads * vdim + c, y);
-          }
-        }
-      }
-    } else {
-      const int pieces = (p.dim_p + 127) / 128, i = u - n_qk - n_v;
+  const int nt = t1 - off, cols = 2 * dim + per * vdim;      // staged columns: q | k | values
+  extern __shared__ __align__(16) unsigned char conv_smem[];
+  T* s_raw = reinterpret_cast<T*>(conv_smem);
+  for (int i = threadIdx.x * V; i < cols; i += CONV_THREADS * V) {
+    const int c = i < dim ? g * dim + i
+                : (i < 2 * dim ? qc + g * dim + (i - dim) : 2 * qc + g * per * vdim + (i - 2 * dim));
+    stage_quad<T, TAPS>(ci, c, raw_col_delta(ci, c), channels, row0, off, nt, slot, has_state, s_raw + i, cols);
+  }
+  cp_async_commit();
+  // the decays meanwhile, in pieces of 128 channels
+  {
+    const int pieces = (p.dim_p + 127) / 128;
+    for (int u = warp; u < per * pieces * 4; u += CONV_THREADS / 32) {   // a quarter of the tile each
+      const int i = u / 4, ta = (u & 3) * (CONV_TILE / 4), tb = min(ta + CONV_TILE / 4, nt);
       const int h = g * per + i / pieces, d = ((i % pieces) * 32 + lane) * V;
-      if (d < p.dim_p) {
-        const bool in = d < dim;
-        const float rate = expf(p.A_log[h]);
-        float b[V] = {};
-        if (in) load_f32<V>(p.dt_bias + h * dim + d, b);
-        for (int tb = off; tb < t1; tb += CONV_AHEAD) {
-          float4 ra[CONV_AHEAD];
+      if (ta >= tb || d >= p.dim_p) continue;
+      const bool in = d < dim;
+      const float rate = expf(p.A_log[h]);
+      float b[V] = {};
+      if (in) load_f32<V>(p.dt_bias + h * dim + d, b);
+      float4 ra[CONV_TILE / 4];
 #pragma unroll
-          for (int j = 0; j < CONV_AHEAD; ++j) {
-            ra[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (in)
-              ra[j] = *reinterpret_cast<const float4*>(
-                  p.a + static_cast<size_t>(row0 + min(tb + j, t1 - 1)) * p.lda + h * dim + d);
-          }
+      for (int j = 0; j < CONV_TILE / 4; ++j) {
+        ra[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (in)
+          ra[j] = *reinterpret_cast<const float4*>(
+              p.a + static_cast<size_t>(row0 + off + min(ta + j, tb - 1)) * p.lda + h * dim + d);
+      }
 #pragma unroll
-          for (int j = 0; j < CONV_AHEAD; ++j) {
-            if (tb + j >= t1) break;
-            const float a[V] = {ra[j].x, ra[j].y, ra[j].z, ra[j].w};
-            float f[V];
+      for (int j = 0; j < CONV_TILE / 4; ++j) {
+        if (ta + j >= tb) break;
+        const float a[V] = {ra[j].x, ra[j].y, ra[j].z, ra[j].w};
+        float f[V];
 #pragma unroll
-            for (int x = 0; x < V; ++x) f[x] = in ? expf(-rate * softplus_exact(a[x] + b[x])) : 0.f;
-            store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row0 + tb + j) * p.dim_p + d, f);
-          }
+        for (int x = 0; x < V; ++x) f[x] = in ? expf(-rate * softplus_exact(a[x] + b[x])) : 0.f;
+        store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row0 + off + ta + j) * p.dim_p + d, f);
+      }
+    }
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // q and k: a quarter of the tile per warp, the norms are warp sums (dim <= 256)
+  {
+    const int ta = warp * (CONV_TILE / 4), tb = min(ta + CONV_TILE / 4, nt);
+    constexpr int NI = 2;
+    for (int t = ta; t < tb; ++t) {
+      float k[NI][V], sq = 0.f, sk = 0.f, dot = 0.f;
+      float qq[NI][V];
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int d = (lane + 32 * i) * V;
+#pragma unroll
+        for (int x = 0; x < V; ++x) qq[i][x] = k[i][x] = 0.f;
+        if (d >= dim) continue;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+          float u[V], w[V];
+          load_vec<V>(s_raw + (t + j) * cols + d, u);
+          load_vec<V>(ci.taps_w + static_cast<ptrdiff_t>(j) * channels + g * dim + d, w);
+#pragma unroll
+          for (int x = 0; x < V; ++x) qq[i][x] += u[x] * w[x];
+          load_vec<V>(s_raw + (t + j) * cols + dim + d, u);
+          load_vec<V>(ci.taps_w + static_cast<ptrdiff_t>(j) * channels + qc + g * dim + d, w);
+#pragma unroll
+          for (int x = 0; x < V; ++x) k[i][x] += u[x] * w[x];
+        }
+#pragma unroll
+        for (int x = 0; x < V; ++x) {
+          qq[i][x] = silu_act<T>(qq[i][x]);
+          k[i][x] = silu_act<T>(k[i][x]);
+          sq += qq[i][x] * qq[i][x];
+          sk += k[i][x] * k[i][x];
+          dot += qq[i][x] * k[i][x];
         }
       }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        dot += __shfl_xor_sync(0xffffffffu, dot, o);
+      }
+      const float rq = qscale / sqrtf(sq + 1e-6f), rk = 1.0f / sqrtf(sk + 1e-6f);
+      const size_t cell = static_cast<size_t>(g) * p.rows + row0 + off + t;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int d = (lane + 32 * i) * V;
+        if (d >= p.dim_p) continue;
+#pragma unroll
+        for (int x = 0; x < V; ++x) {
+          qq[i][x] *= rq;
+          k[i][x] *= rk;
+        }
+        store_f32<V>(p.q + cell * p.dim_p + d, qq[i]);
+        store_f32<V>(p.k + cell * p.dim_p + d, k[i]);
+      }
+      if (lane == 0) p.kq[cell] = dot * rq * rk;
+    }
+  }
+  // values: four channels per thread
+  for (int i = threadIdx.x * V; i < per * vdim; i += CONV_THREADS * V) {
+    const int c = g * per * vdim + i;
+    Window<T, TAPS> w;
+    w.taps(ci, 2 * qc + c, channels);
+    const T* src = s_raw + 2 * dim + i;
+    w.start(src, cols);
+    src += (TAPS - 1) * cols;
+    float* dst = p.v + static_cast<size_t>(row0 + off) * ci.heads * vdim + c;
+#pragma unroll 4
+    for (int t = 0; t < nt; ++t, src += cols, dst += ci.heads * vdim) {
+      float y[V];
+      w.next(src, y);
+#pragma unroll
+      for (int x = 0; x < V; ++x) y[x] = silu_act<T>(y[x]);
+      store_f32<V>(dst, y);
     }
   }
   for (int i = threadIdx.x; i < (t1 - off) * per; i += CONV_THREADS) {
@@ -709,34 +700,67 @@ __global__ void __launch_bounds__(CONV_THREADS, 4) shortconv_delta_tile_kernel(c
   }
 }
 
+constexpr int CONV_SMEM_MAX = 200 * 1024;
+
+template <typename T, int TAPS>
+static int launch_attn_tile(const AttnPre& p, dim3 grid, int threads, int smem, cudaStream_t st) {
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(shortconv_attn_tile_kernel<T, TAPS>,
+                             cudaFuncAttributeMaxDynamicSharedMemorySize, CONV_SMEM_MAX) != cudaSuccess)
+      return -4;
+    set = true;
+  }
+  shortconv_attn_tile_kernel<T, TAPS><<<grid, threads, smem, st>>>(p);
+  return 0;
+}
+template <typename T, int TAPS>
+static int launch_delta_tile(const DeltaPre& p, dim3 grid, int smem, cudaStream_t st) {
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(shortconv_delta_tile_kernel<T, TAPS>,
+                             cudaFuncAttributeMaxDynamicSharedMemorySize, CONV_SMEM_MAX) != cudaSuccess)
+      return -4;
+    set = true;
+  }
+  shortconv_delta_tile_kernel<T, TAPS><<<grid, CONV_THREADS, smem, st>>>(p);
+  return 0;
+}
+
 template <typename T>
 static int launch_conv_attn(const AttnPre& p, dim3 grid, bool vec, cudaStream_t st) {
-  if (vec) {
-    const int units = (p.c.heads / p.c.kv_heads + 1) * ((p.c.dim - p.half) / 4) + p.c.vdim / 4;
-    const int smem = CONV_TILE * p.half * static_cast<int>(sizeof(float2));
+  const int per = p.c.heads / p.c.kv_heads, cols = (per + 1) * p.c.dim + p.c.vdim;
+  const int smem = CONV_TILE * p.half * static_cast<int>(sizeof(float2)) +
+                   (CONV_TILE + p.c.taps - 1) * cols * static_cast<int>(sizeof(T));
+  int rc = 0;
+  if (vec && smem <= CONV_SMEM_MAX) {
+    const int units = (per + 1) * ((p.c.dim - p.half) / 4) + p.c.vdim / 4;
     const int threads = min(256, (units + 31) / 32 * 32);
     switch (p.c.taps) {
-      case 2: shortconv_attn_tile_kernel<T, 2><<<grid, threads, smem, st>>>(p); break;
-      case 3: shortconv_attn_tile_kernel<T, 3><<<grid, threads, smem, st>>>(p); break;
-      default: shortconv_attn_tile_kernel<T, 4><<<grid, threads, smem, st>>>(p);
+      case 2: rc = launch_attn_tile<T, 2>(p, grid, threads, smem, st); break;
+      case 3: rc = launch_attn_tile<T, 3>(p, grid, threads, smem, st); break;
+      default: rc = launch_attn_tile<T, 4>(p, grid, threads, smem, st);
     }
   } else {
     shortconv_attn_kernel<T, 1, 0><<<grid, CONV_THREADS, 0, st>>>(p);
   }
-  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  return rc != 0 ? rc : (cudaGetLastError() == cudaSuccess ? 0 : -3);
 }
 template <typename T>
 static int launch_conv_delta(const DeltaPre& p, dim3 grid, bool vec, cudaStream_t st) {
-  if (vec) {
+  const int cols = 2 * p.c.dim + p.c.heads / p.c.kv_heads * p.c.vdim;
+  const int smem = (CONV_TILE + p.c.taps - 1) * cols * static_cast<int>(sizeof(T));
+  int rc = 0;
+  if (vec && smem <= CONV_SMEM_MAX) {
     switch (p.c.taps) {
-      case 2: shortconv_delta_tile_kernel<T, 2><<<grid, CONV_THREADS, 0, st>>>(p); break;
-      case 3: shortconv_delta_tile_kernel<T, 3><<<grid, CONV_THREADS, 0, st>>>(p); break;
-      default: shortconv_delta_tile_kernel<T, 4><<<grid, CONV_THREADS, 0, st>>>(p);
+      case 2: rc = launch_delta_tile<T, 2>(p, grid, smem, st); break;
+      case 3: rc = launch_delta_tile<T, 3>(p, grid, smem, st); break;
+      default: rc = launch_delta_tile<T, 4>(p, grid, smem, st);
     }
   } else {
     shortconv_delta_kernel<T, 1, 0><<<grid, CONV_THREADS, 0, st>>>(p);
   }
-  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  return rc != 0 ? rc : (cudaGetLastError() == cudaSuccess ? 0 : -3);
 }
 
 }  // namespace cb

@@ -12,6 +12,7 @@ from __future__ import annotations
 
 from typing import Dict, List, Optional
 
+import numpy as np
 import torch
 
 from ..foundation.error import ProcessingError
@@ -172,7 +173,8 @@ class HybridEngine(InferenceEngine):
             if e.pos0 != c.length(e.slot):
                 raise ProcessingError.invalid_input(
                     f"slot {e.slot} holds {c.length(e.slot)} tokens, the entry starts at {e.pos0}")
-            if min(e.tokens) < 0 or max(e.tokens) >= self.cfg.vocab_size:
+            ids = np.asarray(e.tokens)
+            if ids.min() < 0 or ids.max() >= self.cfg.vocab_size:
                 raise ProcessingError.invalid_input(
                     f"token ids must lie in [0, {self.cfg.vocab_size})")
         for e in entries:
@@ -237,7 +239,7 @@ class HybridEngine(InferenceEngine):
             c.release(b)
         for b in range(B):
             c.reserve(b, total_len)
-        rows = ids.tolist()
+        rows = ids.cpu().numpy()
         nb = max(1, min(B, int(seq_chunk or B)))
         step = max(1, min(S, int(token_chunk or S), max(1, self.prefill_tokens // nb)))
         out: List[torch.Tensor] = []
