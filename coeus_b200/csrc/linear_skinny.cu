@@ -1,4 +1,4 @@
-// bf16 linear layers of a decode step: Y[M, N] = act(X[M, K] . W[N, K]^T) with few rows (M <= 64),
+// bf16 linear layers of a decode step: Y[M, N] = act(X[M, K] . W[N, K]^T) with few rows (M <= 16),
 // bound by streaming the weights.  The weights are the 16-row operand of mma m16n8k16 and the
 // tokens its 8 columns; every lane reads 32 consecutive bytes of a weight row per 64-wide slice
 // of K (the contraction index is permuted the same way on both sides, so fragments come straight
@@ -164,15 +164,13 @@ static int skinny_problem(SkinnyProblem& p, const void* x, int ldx, const void* 
   return 0;
 }
 
-extern "C" int cb_linear_skinny_max() { return 64; }
-
 // The second problem is skipped when x1 is null.
 extern "C" int cb_linear_skinny(const void* x0, int ldx0, const void* w0, int ldw0, void* y0,
                                 int ldy0, int N0, int K0, int act0, float arg0, int f32_0, int acc0,
                                 const void* x1, int ldx1, const void* w1, int ldw1, void* y1,
                                 int ldy1, int N1, int K1, int act1, float arg1, int f32_1, int acc1,
                                 int M, void* stream) {
-  if (M <= 0 || M > 64) return -1;
+  if (M <= 0 || M > 16) return -1;
   SkinnyArgs a = {};
   a.M = M;
   int rc = skinny_problem(a.p[0], x0, ldx0, w0, ldw0, y0, ldy0, N0, K0, act0, arg0, f32_0, acc0);
@@ -186,7 +184,5 @@ extern "C" int cb_linear_skinny(const void* x0, int ldx0, const void* w0, int ld
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const bool deep = K0 >= 4096 && count == 1;
   if (M <= 8) return deep ? launch_skinny<1, 1, 16>(a, count, st) : launch_skinny<1, 1, 8>(a, count, st);
-  if (M <= 16) return deep ? launch_skinny<1, 2, 16>(a, count, st) : launch_skinny<1, 2, 8>(a, count, st);
-  if (M <= 32) return deep ? launch_skinny<1, 4, 16>(a, count, st) : launch_skinny<2, 4, 8>(a, count, st);
-  return deep ? launch_skinny<1, 8, 16>(a, count, st) : launch_skinny<2, 8, 8>(a, count, st);
+  return deep ? launch_skinny<1, 2, 16>(a, count, st) : launch_skinny<1, 2, 8>(a, count, st);
 }

@@ -273,7 +273,7 @@ struct Window {
 };
 
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre p) {
+__global__ void __launch_bounds__(256, 3) shortconv_attn_tile_kernel(const AttnPre p) {
   constexpr int V = 4;
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -326,14 +326,13 @@ __global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre 
     }
     const bool is_q = !is_v && hi < per;
     const T* src = s_raw + i;
-    Window<T, TAPS> wa, wb;
-    wa.taps(ci, c, channels);
-    wa.start(src, cols);
-    if (pair) {
-      wb.taps(ci, c + p.half, channels);
-      wb.start(src + p.half, cols);
+    float wa[TAPS][V], wb[TAPS][V];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const float* w = ci.taps_w + static_cast<ptrdiff_t>(j) * channels + c;
+      load_vec<V>(w, wa[j]);
+      if (pair) load_vec<V>(w + p.half, wb[j]);
     }
-    src += (TAPS - 1) * cols;
     // where the first token goes, and how far apart the tokens of a page are
     T* kr = nullptr;
     T* vf = nullptr;
@@ -353,6 +352,17 @@ __global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre 
     T* cache = static_cast<T*>(is_v ? p.v_cache : p.k_cache);
     const int in_cell = is_v ? g * p.vdim_p + d : g * p.dim_p + d;
     const float lam = is_v && p.mix_mode == 2 ? *p.lambda : 0.f;
+    auto conv = [&](const T* at, const float (*w)[V], float* y) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) y[k] = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        float f[V];
+        load_vec<V>(at + j * cols, f);
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] += f[k] * w[j][k];
+      }
+    };
 #pragma unroll 2
     for (int t = 0; t < nt; ++t, src += cols) {
       if (!is_q) {
@@ -362,10 +372,10 @@ __global__ void __launch_bounds__(256) shortconv_attn_tile_kernel(const AttnPre 
                        : cache + (static_cast<size_t>(page) * RAGGED_PAGE + pos % RAGGED_PAGE) * step + in_cell;
       }
       float a[V];
-      wa.next(src, a);
+      conv(src, wa, a);
       if (pair) {
         float b[V], oa[V], ob[V];
-        wb.next(src + p.half, b);
+        conv(src + p.half, wb, b);
         const float4* cs = reinterpret_cast<const float4*>(s_rope + t * p.half + d);
         const float4 x = cs[0], y = cs[1];
         const float cc[V] = {x.x, x.z, y.x, y.z}, ss[V] = {x.y, x.w, y.y, y.w};

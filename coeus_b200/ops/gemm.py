@@ -282,14 +282,19 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
             K, act, ctypes.c_float(softcap or 0.0), int(accumulate), _lib.stream_ptr())
         _lib.check_rc(rc, "cb_linear_f32")
         return out
-    if M <= SKINNY_MAX:
+    if M <= SKINNY_MAX and not (accumulate and (M > 8 or K >= 16384)):
         return linear_pair((x, w, out, epi, softcap, accumulate))[0]
     out_mode = _OUT_BF16 if out.dtype == torch.bfloat16 else (
         _OUT_F32_ATOMIC if accumulate else _OUT_F32)
+    # Few tiles: narrower ones spread the weights over more SMs, and a product that is added to
+    # the stream can be cut along the contraction until every SM streams a share of them.
+    tiles = ((M + 127) // 128) * ((N + 127) // 128)
+    bn, ksplit = (128 if tiles <= 148 or M <= 128 else _pick_bn(M, N)), 1
+    if accumulate:
+        ksplit = max(1, min(16, 148 // tiles, (K + 63) // 64 // 4))
     rc = _lib.serving_lib().cb_gemm_bf16(
         _lib.ptr(x), _lib.ptr(w), _lib.ptr(out), M, N, K, x.stride(0), w.stride(0), out.stride(0),
-        0, 0, None, None, 0, None, None, 0, EPI[epi], out_mode, ctypes.c_float(1.0), 1,
-        _pick_bn(M, N), _lib.ptr(_lib.status_buffer(x.device)), 0, _lib.stream_ptr())
+        0, 0, None, None, 0, None, None, 0, EPI[epi], out_mode, ctypes.c_float(1.0), ksplit, bn, _lib.ptr(_lib.status_buffer(x.device)), 0, _lib.stream_ptr())
     _lib.check_rc(rc, "cb_gemm_bf16")
     if softcap is not None:
         rc = _lib.serving_lib().cb_softcap(_lib.ptr(out), out.stride(0), M, N,
@@ -298,7 +303,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
     return out
 
 
-SKINNY_MAX = 64       # rows up to which a bf16 product runs on the weight-streaming kernel
+SKINNY_MAX = 16       # rows up to which a bf16 product runs on the weight-streaming kernel
 
 
 def _skinny_args(x, w, out, epi, softcap, accumulate):

@@ -421,7 +421,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         ctx = max_ctx or batch.max_ctx
         ctx = min(ctx, chunk) if chunk else ctx
         # a CTA takes 128 keys at a time
-        splits = max(1, min(16, (4 * 148 + ctas - 1) // ctas, (ctx + 127) // 128))
+        splits = max(1, min(16, (2 * 148 + ctas - 1) // ctas, (ctx + 127) // 128))
         part_o = part_ml = None
         if splits > 1:
             part_o = torch.empty((n, heads, splits, vdim), dtype=torch.float32, device=q.device)
