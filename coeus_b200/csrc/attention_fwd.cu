@@ -47,9 +47,11 @@ struct AttnFwdArgs {
   int drop_thr;
   uint32_t drop_key;
   float drop_scale;
-  // pieces of unequal length instead of B sequences of S rows: piece b is the rows pieces[b].x ..
-  // pieces[b].x + pieces[b].y - 1 (at most S), which attend to one another only; null: none
-  const int2* pieces;
+  // Pieces of unequal length instead of B sequences of S rows.  Piece b has y = pieces[b].y query
+  // rows (at most S) from row pieces[b].x on and w + y keys from row pieces[b].z of K and V on; its
+  // query i sees the first w + i + 1 of them (causal).  null: none
+  const int4* pieces;
+  int vdim;                    // columns of a head that are stored, vdim apart in O
   const float* sink;           // [nh] logits that enter the denominator only, or null
   const __nv_bfloat16* gate;   // [rows, ldg], column h: head h's output times its sigmoid; or null
   int ldg;
@@ -112,7 +114,8 @@ struct AFWalk {
   int wave, j, t;
   int b, h, qa;          // batch, head, first query tile of the pair
   int row0, len;         // first row and rows of the sequence (or piece)
-  const int2* pieces;
+  int kv_row0, ahead;    // first key row, keys before the first query's own
+  const int4* pieces;
   int n0, n1, nmax;      // key tiles of tile A / B (0: the tile does not exist)
   int kv_seq;            // how many (item, j) groups came before this one: the K/V ring position
   bool valid;
@@ -128,6 +131,7 @@ struct AFWalk {
     causal = p.causal;
     pieces = p.pieces;
     len = p.S;
+    ahead = 0;
     n_waves = (n_items + gridDim.x - 1) / gridDim.x;
     wave = -1;
     kv_seq = -1;
@@ -148,18 +152,20 @@ struct AFWalk {
       h = bh % nh;
       qa = 2 * pair;
       if (pieces != nullptr) {
-        const int2 pc = pieces[b];
+        const int4 pc = pieces[b];
         row0 = pc.x;
         len = pc.y;
+        kv_row0 = pc.z;
+        ahead = pc.w;
         n_q_tiles = (len + AF_BM - 1) / AF_BM;
-        n_kv_tiles = (len + bkv - 1) / bkv;
+        n_kv_tiles = (ahead + len + bkv - 1) / bkv;
         if (qa >= n_q_tiles) continue;             // a shorter piece ends before this pair
       } else {
-        row0 = b * len;
+        row0 = kv_row0 = b * len;
       }
-      n0 = causal ? min(n_kv_tiles, ((qa + 1) * AF_BM + bkv - 1) / bkv) : n_kv_tiles;
+      n0 = causal ? min(n_kv_tiles, (ahead + (qa + 1) * AF_BM + bkv - 1) / bkv) : n_kv_tiles;
       n1 = qa + 1 >= n_q_tiles ? 0
-           : (causal ? min(n_kv_tiles, ((qa + 2) * AF_BM + bkv - 1) / bkv) : n_kv_tiles);
+           : (causal ? min(n_kv_tiles, (ahead + (qa + 2) * AF_BM + bkv - 1) / bkv) : n_kv_tiles);
       nmax = max(n0, n1);
       j = 0;
       t = 0;
@@ -254,7 +260,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       AFWalk w;
       w.init(p, BKV);
       while (w.valid && ok) {
-        const int row0 = w.row0;
+        const int row0 = w.row0, kv_row0 = w.kv_row0;
         const int h = w.h, hk = w.h / group, qa = w.qa;
         const int n0 = w.n0, n1 = w.n1, nmax = w.nmax;
         auto load_q = [&](int t) {
@@ -282,7 +288,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int c = 0; c < DH / 64; ++c)
             tma_load_2d(sK(s) + c * (BKV * 128), &tmK, bar(Cfg::B_KF + s), hk * DH + c * 64,
-                        row0 + j * BKV);
+                        kv_row0 + j * BKV);
           ++kcnt;
         };
         auto load_v = [&](int j) {
@@ -296,7 +302,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int c = 0; c < DH / 64; ++c)
             tma_load_2d(sV(s) + c * (BKV * 128), &tmV, bar(Cfg::B_VF + s), hk * DH + c * 64,
-                        row0 + j * BKV);
+                        kv_row0 + j * BKV);
           ++vcnt;
         };
         load_q(0);
@@ -508,8 +514,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (tr) tr[tri] = clock64();
       tc_fence_after();
       const int kv0 = j * BKV;
-      const bool need_mask = (p.causal && kv0 + BKV - 1 > q0) || (kv0 + BKV > w.len);
-      const int kv_limit = p.causal ? min(q_idx, w.len - 1) : (w.len - 1);  // last visible key
+      const bool need_mask = (p.causal && kv0 + BKV - 1 > q0 + w.ahead) || (kv0 + BKV > w.ahead + w.len);
+      const int kv_limit = w.ahead + (p.causal ? min(q_idx, w.len - 1) : (w.len - 1));  // last visible key
       uint32_t v[BKV];
 #pragma unroll
       for (int c = 0; c < BKV / 32; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v + c * 32);
@@ -637,7 +643,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         inv_l = 1.0f / (lsum + exp2f(p.sink[w.h] * 1.4426950408889634f - m_used));
       if (p.gate != nullptr && row_ok)
         inv_l /= 1.0f + expf(-__bfloat162float(p.gate[out_row * p.ldg + w.h]));
-      __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * DH;
+      __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * p.vdim;
 #pragma unroll 1
       for (int c = 0; c < DH / 32; ++c) {
         uint32_t o[32];
@@ -651,7 +657,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
             wv.y = pack_bf16x2(__uint_as_float(o[8 * gq + 2]) * inv_l, __uint_as_float(o[8 * gq + 3]) * inv_l);
             wv.z = pack_bf16x2(__uint_as_float(o[8 * gq + 4]) * inv_l, __uint_as_float(o[8 * gq + 5]) * inv_l);
             wv.w = pack_bf16x2(__uint_as_float(o[8 * gq + 6]) * inv_l, __uint_as_float(o[8 * gq + 7]) * inv_l);
-            *reinterpret_cast<uint4*>(orow + c * 32 + gq * 8) = wv;
+            const int d0 = c * 32 + gq * 8;
+            if (d0 + 8 <= p.vdim && (p.vdim & 7) == 0) {
+              *reinterpret_cast<uint4*>(orow + d0) = wv;
+            } else {
+#pragma unroll
+              for (int x = 0; x < 8; ++x)
+                if (d0 + x < p.vdim)
+                  orow[d0 + x] = __float2bfloat16(__uint_as_float(o[8 * gq + x]) * inv_l);
+            }
           }
         }
       }
@@ -730,6 +744,7 @@ extern "C" int cb_attn_fwd_dropout(const void* q, const void* k, const void* v, 
   a.causal = causal;
   a.status = status;
   a.pieces = nullptr;
+  a.vdim = dh;
   a.sink = nullptr;
   a.gate = nullptr;
   a.ldg = 0;
@@ -755,34 +770,36 @@ extern "C" int cb_attn_fwd(const void* q, const void* k, const void* v, void* o,
                              poly, 0, 0u, status, max_ctas, stream);
 }
 
-// Causal attention inside every piece of a ragged batch: n_pieces (first row, rows) pairs over the
-// `rows` rows of q, k, v and o, none longer than max_len.  sink (fp32 [nh]) is a logit per head that
-// enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view) multiplies head
-// h's output by its sigmoid; both may be null.  scale > 0.
+// Causal attention of a ragged batch in pieces (see AttnFwdArgs): n_pieces quadruples over `rows`
+// query rows and `kv_rows` key rows, none with more than max_len queries.  Heads of q, k and v are
+// dh apart (64 or 128, padded with zeros), heads of o vdim <= dh.  sink (fp32 [nh]) is a logit per head
+// that enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view) multiplies
+// head h's output by its sigmoid; both may be null.  scale > 0.
 extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, void* o, int rows,
-                                  const void* pieces, int n_pieces, int max_len, int nh, int nkv,
-                                  int dh, int ldq, int ldk, int ldv, int ldo, float scale,
-                                  const float* sink, const void* gate, int ldg, int* status,
-                                  void* stream) {
+                                  int kv_rows, const void* pieces, int n_pieces, int max_len, int nh,
+                                  int nkv, int dh, int vdim, int ldq, int ldk, int ldv, int ldo,
+                                  float scale, const float* sink, const void* gate, int ldg,
+                                  int* status, void* stream) {
   using namespace cb;
   if (dh != 64 && dh != 128) return -1;
-  if (rows <= 0 || n_pieces <= 0 || max_len <= 0 || nh <= 0 || nkv <= 0 || (nh % nkv) != 0 ||
-      (ldo % 8) != 0 || !(scale > 0.f))
+  if (rows <= 0 || kv_rows <= 0 || n_pieces <= 0 || max_len <= 0 || nh <= 0 || nkv <= 0 ||
+      (nh % nkv) != 0 || (ldo % 8) != 0 || vdim < 1 || vdim > dh || !(scale > 0.f))
     return -2;
   CUtensorMap tq, tk, tv;
   const uint32_t bkv = dh == 64 ? AFCfg<64>::BKV : AFCfg<128>::BKV;
   if (make_tmap_bf16_2d(&tq, q, static_cast<uint64_t>(nh) * dh, rows, ldq, 64, AF_BM) != 0) return -3;
-  if (make_tmap_bf16_2d(&tk, k, static_cast<uint64_t>(nkv) * dh, rows, ldk, 64, bkv) != 0) return -4;
-  if (make_tmap_bf16_2d(&tv, v, static_cast<uint64_t>(nkv) * dh, rows, ldv, 64, bkv) != 0) return -5;
+  if (make_tmap_bf16_2d(&tk, k, static_cast<uint64_t>(nkv) * dh, kv_rows, ldk, 64, bkv) != 0) return -4;
+  if (make_tmap_bf16_2d(&tv, v, static_cast<uint64_t>(nkv) * dh, kv_rows, ldv, 64, bkv) != 0) return -5;
   AttnFwdArgs a = {};
   a.B = n_pieces; a.S = max_len; a.nh = nh; a.nkv = nkv;
   a.O = static_cast<__nv_bfloat16*>(o);
   a.ldo = ldo;
+  a.vdim = vdim;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.causal = 1;
   a.status = status;
   a.drop_scale = 1.0f;
-  a.pieces = static_cast<const int2*>(pieces);
+  a.pieces = static_cast<const int4*>(pieces);
   a.sink = sink;
   a.gate = static_cast<const __nv_bfloat16*>(gate);
   a.ldg = ldg;

@@ -18,7 +18,8 @@ namespace cb {
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct RaggedAttn {
-  const void* q;           // [rows, heads * dim]
+  const void* q;           // [rows, heads, q_head]
+  int q_head;
   const void* k_cache;     // [pages, PAGE, kv_heads, dim_p]
   const void* v_cache;     // [pages, PAGE, kv_heads, vdim_p]
   const int* page_table;   // [slots, max_pages]
@@ -82,10 +83,10 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
   const int slot = ra.row_slot[row], pos = ra.row_pos[row];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
-  const T* qp = static_cast<const T*>(p.q) + static_cast<size_t>(row) * p.heads * p.dim;
+  const T* qp = static_cast<const T*>(p.q) + static_cast<size_t>(row) * p.heads * p.q_head;
   for (int j = threadIdx.x; j < GM * DC; j += RA_WARPS * 32) {
     const int g = j / DC, d = j % DC;
-    sq[g][d] = (g < ng && d < p.dim) ? to_f32(qp[(h0 + g) * p.dim + d]) * (p.scale * LOG2E) : 0.f;
+    sq[g][d] = (g < ng && d < p.dim) ? to_f32(qp[(h0 + g) * p.q_head + d]) * (p.scale * LOG2E) : 0.f;
   }
   __syncthreads();
   const int lo = chunk_start(pos, p.chunk), n = pos + 1 - lo;
@@ -322,19 +323,19 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
     cp_async_commit();
   };
   fetch(pg0, 0);
-  if (p.dim % 8 == 0) {
+  if (p.dim % 8 == 0 && p.q_head % 8 == 0) {
     for (int i = tid; i < TA_ROWS * (DC / 8); i += TA_WARPS * 32) {
       const int t = i / (DC / 8), c = (i % (DC / 8)) * 8;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (t < len && c < p.dim)
-        v = *reinterpret_cast<const uint4*>(q + (static_cast<size_t>(row0 + t) * p.heads + h) * p.dim + c);
+        v = *reinterpret_cast<const uint4*>(q + (static_cast<size_t>(row0 + t) * p.heads + h) * p.q_head + c);
       *reinterpret_cast<uint4*>(sQ + t * KS + c) = v;
     }
   } else {
     for (int i = tid; i < TA_ROWS * DC; i += TA_WARPS * 32) {
       const int t = i / DC, c = i % DC;
       sQ[t * KS + c] = (t < len && c < p.dim)
-                           ? q[(static_cast<size_t>(row0 + t) * p.heads + h) * p.dim + c]
+                           ? q[(static_cast<size_t>(row0 + t) * p.heads + h) * p.q_head + c]
                            : __float2bfloat16(0.f);
     }
   }
@@ -536,10 +537,10 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
   }
   int tb = t0 + warp * GA_KEYS;
   if (tb < t1) fetch(tb, 0);
-  const bf16* q = static_cast<const bf16*>(p.q) + (static_cast<size_t>(row) * p.heads + h0) * p.dim;
+  const bf16* q = static_cast<const bf16*>(p.q) + (static_cast<size_t>(row) * p.heads + h0) * p.q_head;
   for (int x = tid; x < 16 * DC; x += GA_WARPS * 32) {
     const int g = x / DC, d = x % DC;
-    sQ[g * KS + d] = g < ng && d < p.dim ? q[g * p.dim + d] : __float2bfloat16(0.f);
+    sQ[g * KS + d] = g < ng && d < p.dim ? q[g * p.q_head + d] : __float2bfloat16(0.f);
   }
   __syncthreads();
   uint32_t qf[DC / 16][4];
@@ -756,14 +757,14 @@ static int launch_rows_d(const RowsArgs& a, int n, cudaStream_t st) {
 
 using namespace cb;
 
-static int fill_attn(RaggedAttn& p, const void* q, const void* k_cache, const void* v_cache,
+static int fill_attn(RaggedAttn& p, const void* q, int q_head, const void* k_cache, const void* v_cache,
                      const int* page_table, int max_pages, int num_pages, int heads, int kv_heads,
                      int dim, int vdim, int dim_p, int vdim_p, int chunk, float scale,
                      const float* sink, const void* gate, int ldg, void* out, int ldo, int* status) {
   if (kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || dim > 256 || vdim > 256) return -1;
   if (dim_p % 8 != 0 || vdim_p % 8 != 0 || dim_p < dim || vdim_p < vdim || dim_p > 256 || vdim_p > 256)
     return -2;
-  p.q = q; p.k_cache = k_cache; p.v_cache = v_cache; p.page_table = page_table;
+  p.q = q; p.q_head = q_head; p.k_cache = k_cache; p.v_cache = v_cache; p.page_table = page_table;
   p.max_pages = max_pages; p.num_pages = num_pages; p.heads = heads; p.kv_heads = kv_heads;
   p.dim = dim; p.vdim = vdim; p.dim_p = dim_p; p.vdim_p = vdim_p; p.chunk = chunk; p.scale = scale;
   p.sink = sink; p.gate = gate; p.ldg = ldg; p.out = out; p.ldo = ldo; p.status = status;
@@ -772,7 +773,7 @@ static int fill_attn(RaggedAttn& p, const void* q, const void* k_cache, const vo
 
 extern "C" int cb_ragged_attn_tile() { return TA_ROWS; }
 
-extern "C" int cb_ragged_attn_rows(const void* q, const void* k_cache, const void* v_cache,
+extern "C" int cb_ragged_attn_rows(const void* q, int q_head, const void* k_cache, const void* v_cache,
                                    const int* page_table, int max_pages, int num_pages, int heads,
                                    int kv_heads, int dim, int vdim, int dim_p, int vdim_p, int chunk,
                                    float scale, const float* sink, const void* gate, int ldg,
@@ -780,7 +781,7 @@ extern "C" int cb_ragged_attn_rows(const void* q, const void* k_cache, const voi
                                    const int* row_pos, int n, int splits, float* part_o,
                                    float* part_ml, int f32, int* status, void* stream) {
   RowsArgs a;
-  const int rc = fill_attn(a.a, q, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
+  const int rc = fill_attn(a.a, q, q_head, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
                            dim, vdim, dim_p, vdim_p, chunk, scale, sink, gate, ldg, out, ldo, status);
   if (rc != 0) return rc;
   if (n <= 0 || splits < 1 || (splits > 1 && (part_o == nullptr || part_ml == nullptr))) return -5;
@@ -792,7 +793,7 @@ extern "C" int cb_ragged_attn_rows(const void* q, const void* k_cache, const voi
   return dim <= 64 ? launch_group_v<64>(a, n, st) : launch_group_v<128>(a, n, st);
 }
 
-extern "C" int cb_ragged_attn_tiles(const void* q, const void* k_cache, const void* v_cache,
+extern "C" int cb_ragged_attn_tiles(const void* q, int q_head, const void* k_cache, const void* v_cache,
                                     const int* page_table, int max_pages, int num_pages, int heads,
                                     int kv_heads, int dim, int vdim, int dim_p, int vdim_p, int chunk,
                                     float scale, const float* sink, const void* gate, int ldg,
@@ -800,7 +801,7 @@ extern "C" int cb_ragged_attn_tiles(const void* q, const void* k_cache, const vo
                                     const int* len, const int* pos0, const int* tile_entry,
                                     const int* tile_off, const int* tile_len, int tiles, int* status, void* stream) {
   TilesArgs a;
-  const int rc = fill_attn(a.a, q, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
+  const int rc = fill_attn(a.a, q, q_head, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
                            dim, vdim, dim_p, vdim_p, chunk, scale, sink, gate, ldg, out, ldo, status);
   if (rc != 0) return rc;
   if (tiles <= 0) return -5;

@@ -102,7 +102,8 @@ struct AttnPre {
   ConvIn c;
   int half;                // rotated pairs per head (0: no rotation)
   const float2* rope;      // [rows, half] (cos, sin)
-  void* q;                 // out [rows, heads * dim]
+  void* q;                 // out [rows, heads, q_head]
+  int q_head, row_head;    // distance of the heads in q, and in k_rows and v_rows
   void* k_cache;           // [pages, PAGE, kv_heads, dim_p]
   void* v_cache;           // [pages, PAGE, kv_heads, vdim_p]
   int dim_p, vdim_p;
@@ -111,8 +112,8 @@ struct AttnPre {
   void* v_first;           // [rows, kv_heads * vdim]: written when mix_mode = 1, read when 2
   const float* lambda;
   int mix_mode;
-  void* k_rows;            // out [rows, kv_heads * dim]: k once more, row by row (or null)
-  void* v_rows;            // out [rows, kv_heads * vdim]
+  void* k_rows;            // out [rows, kv_heads, row_head]: k once more, row by row (or null)
+  void* v_rows;            // out [rows, kv_heads, row_head]
   int* status;
 };
 
@@ -146,7 +147,7 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
       const bool is_q = hi < per;
       const int base = is_q ? (g * per + hi) * dim : qc + g * dim;
       const int colb = is_q ? base : ci.koff + g * dim;
-      T* dst = is_q ? static_cast<T*>(p.q) + static_cast<size_t>(row) * qc + base
+      T* dst = is_q ? static_cast<T*>(p.q) + (static_cast<size_t>(row) * ci.heads + g * per + hi) * p.q_head
                     : static_cast<T*>(p.k_cache) + cell * p.dim_p;
       if (k < pair_u) {
         const int d = k * V;
@@ -162,7 +163,7 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
         store_vec<V>(dst + d, oa);
         store_vec<V>(dst + p.half + d, ob);
         if (!is_q && p.k_rows != nullptr) {
-          T* kr = static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d;
+          T* kr = static_cast<T*>(p.k_rows) + (static_cast<size_t>(row) * ci.kv_heads + g) * p.row_head + d;
           store_vec<V>(kr, oa);
           store_vec<V>(kr + p.half, ob);
         }
@@ -172,7 +173,7 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
         conv_at<T, V, TAPS>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
         store_vec<V>(dst + d, a);
         if (!is_q && p.k_rows != nullptr)
-          store_vec<V>(static_cast<T*>(p.k_rows) + static_cast<size_t>(row) * kc + g * dim + d, a);
+          store_vec<V>(static_cast<T*>(p.k_rows) + (static_cast<size_t>(row) * ci.kv_heads + g) * p.row_head + d, a);
       }
     } else {
       const int d = (u - (per + 1) * head_u) * V;
@@ -192,7 +193,7 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
       }
       store_vec<V>(static_cast<T*>(p.v_cache) + cell * p.vdim_p + d, a);
       if (p.v_rows != nullptr)
-        store_vec<V>(static_cast<T*>(p.v_rows) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d, a);
+        store_vec<V>(static_cast<T*>(p.v_rows) + (static_cast<size_t>(row) * ci.kv_heads + g) * p.row_head + d, a);
     }
   }
   if (off == 0 && ci.taps > 1) {
@@ -337,17 +338,17 @@ __global__ void __launch_bounds__(256, 3) shortconv_attn_tile_kernel(const AttnP
     T* kr = nullptr;
     T* vf = nullptr;
     T* dst = nullptr;
-    int step = qc, row_step = kc;
+    int step = 0;
+    const int q_step = ci.heads * p.q_head, kr_step = ci.kv_heads * p.row_head, vf_step = ci.kv_heads * vdim;
     if (is_q) {
-      dst = static_cast<T*>(p.q) + static_cast<size_t>(row0 + off) * qc + c;
-    } else if (is_v) {
-      step = ci.kv_heads * p.vdim_p;
-      row_step = ci.kv_heads * vdim;
-      if (p.k_rows != nullptr) kr = static_cast<T*>(p.v_rows) + static_cast<size_t>(row0 + off) * row_step + g * vdim + d;
-      if (p.mix_mode != 0) vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row0 + off) * row_step + g * vdim + d;
+      dst = static_cast<T*>(p.q) + static_cast<size_t>(row0 + off) * q_step + (g * per + hi) * p.q_head + d;
     } else {
-      step = ci.kv_heads * p.dim_p;
-      if (p.k_rows != nullptr) kr = static_cast<T*>(p.k_rows) + static_cast<size_t>(row0 + off) * kc + g * dim + d;
+      step = ci.kv_heads * (is_v ? p.vdim_p : p.dim_p);
+      if (p.k_rows != nullptr)
+        kr = static_cast<T*>(is_v ? p.v_rows : p.k_rows) + static_cast<size_t>(row0 + off) * kr_step +
+             g * p.row_head + d;
+      if (is_v && p.mix_mode != 0)
+        vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row0 + off) * vf_step + g * vdim + d;
     }
     T* cache = static_cast<T*>(is_v ? p.v_cache : p.k_cache);
     const int in_cell = is_v ? g * p.vdim_p + d : g * p.dim_p + d;
@@ -402,13 +403,13 @@ __global__ void __launch_bounds__(256, 3) shortconv_attn_tile_kernel(const AttnP
 #pragma unroll
             for (int k = 0; k < V; ++k) a[k] = (1.f - lam) * a[k] + lam * f[k];
           }
-          vf += row_step;
+          vf += vf_step;
         }
         if (dst != nullptr) store_vec<V>(dst, a);
         if (kr != nullptr) store_vec<V>(kr, a);
       }
-      if (is_q) dst += qc;
-      if (kr != nullptr) kr += row_step;
+      if (is_q) dst += q_step;
+      if (kr != nullptr) kr += kr_step;
     }
   }
   if (off == 0) {
@@ -710,6 +711,29 @@ __global__ void __launch_bounds__(CONV_THREADS, 6) shortconv_delta_tile_kernel(c
   }
 }
 
+// One block per row, vectors of eight bf16; the padding of a head is zero.
+__global__ void kv_gather_kernel(const uint4* __restrict__ k_cache, const uint4* __restrict__ v_cache,
+                                 int kv_heads, int kw, int vw, const int* __restrict__ page_table,
+                                 int max_pages, int num_pages, const int2* __restrict__ where,
+                                 uint4* __restrict__ k_rows, uint4* __restrict__ v_rows, int row_w,
+                                 int* status) {
+  const int2 at = where[blockIdx.x];
+  const int lp = at.y / RAGGED_PAGE;
+  int page = lp < max_pages ? page_table[static_cast<size_t>(at.x) * max_pages + lp] : -1;
+  if (page < 0 || page >= num_pages) {
+    if (threadIdx.x == 0) record_status(status, ST_BOUNDS, blockIdx.x);
+    return;
+  }
+  const size_t cell = static_cast<size_t>(page) * RAGGED_PAGE + at.y % RAGGED_PAGE;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  for (int i = threadIdx.x; i < kv_heads * row_w; i += blockDim.x) {
+    const int g = i / row_w, c = i % row_w;
+    const size_t dst = static_cast<size_t>(blockIdx.x) * kv_heads * row_w + i;
+    k_rows[dst] = c < kw ? k_cache[(cell * kv_heads + g) * kw + c] : zero;
+    v_rows[dst] = c < vw ? v_cache[(cell * kv_heads + g) * vw + c] : zero;
+  }
+}
+
 constexpr int CONV_SMEM_MAX = 200 * 1024;
 
 template <typename T, int TAPS>
@@ -795,10 +819,10 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
                                  int taps, void* state, int heads, int kv_heads, int dim, int vdim,
                                  const int* slot, const int* row0, const int* len, const int* pos0,
                                  const int* tile_entry, const int* tile_off, int tiles, int half,
-                                 const void* rope, void* q, void* k_cache, void* v_cache, int dim_p,
+                                 const void* rope, void* q, int q_head, void* k_cache, void* v_cache, int dim_p,
                                  int vdim_p, const int* page_table, int max_pages, int num_pages,
                                  void* v_first, const float* lambda, int mix_mode, void* k_rows,
-                                 void* v_rows, int f32, int* status, void* stream) {
+                                 void* v_rows, int row_head, int f32, int* status, void* stream) {
   if (tiles <= 0 || taps < 1 || kv_heads < 1 || heads % kv_heads != 0 || 2 * half > dim) return -1;
   if (mix_mode != 0 && v_first == nullptr) return -2;
   AttnPre p;
@@ -808,13 +832,27 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
   p.v_cache = v_cache; p.dim_p = dim_p; p.vdim_p = vdim_p; p.page_table = page_table;
   p.max_pages = max_pages; p.num_pages = num_pages; p.v_first = v_first; p.lambda = lambda;
   p.mix_mode = mix_mode; p.status = status;
-  p.k_rows = k_rows; p.v_rows = v_rows;
+  p.k_rows = k_rows; p.v_rows = v_rows; p.q_head = q_head; p.row_head = row_head;
   const bool vec = taps >= 2 && taps <= 4 && dim % 4 == 0 && vdim % 4 == 0 && half % 4 == 0 &&
-                   half <= 128 && ld % 8 == 0 && koff % 8 == 0 && voff % 8 == 0;
+                   half <= 128 && q_head % 4 == 0 && row_head % 4 == 0 && ld % 8 == 0 && koff % 8 == 0 && voff % 8 == 0;
   dim3 grid(tiles, kv_heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return f32 ? launch_conv_attn<float>(p, grid, vec, st)
              : launch_conv_attn<__nv_bfloat16>(p, grid, vec, st);
+}
+
+// Rows gathered from the cache pages: row i of k_rows / v_rows ([n, kv_heads, row_head]) is the token
+// at position where[2 i + 1] of slot where[2 i].
+extern "C" int cb_kv_gather(const void* k_cache, const void* v_cache, int kv_heads, int dim_p,
+                            int vdim_p, const int* page_table, int max_pages, int num_pages,
+                            const void* where, int n, void* k_rows, void* v_rows, int row_head,
+                            int* status, void* stream) {
+  if (n <= 0 || dim_p % 8 || vdim_p % 8 || row_head % 8 || dim_p > row_head || vdim_p > row_head) return -1;
+  kv_gather_kernel<<<n, 128, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const uint4*>(k_cache), static_cast<const uint4*>(v_cache), kv_heads, dim_p / 8,
+      vdim_p / 8, page_table, max_pages, num_pages, static_cast<const int2*>(where),
+      static_cast<uint4*>(k_rows), static_cast<uint4*>(v_rows), row_head / 8, status);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
 extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, int boff,

@@ -104,19 +104,24 @@ class HybridEngine(InferenceEngine):
         first = s.v_mix and v_first is None
         if first:
             v_first = torch.empty((b.T, s.kv_heads * s.vdim), dtype=raw.dtype, device=raw.device)
-        k_rows = v_rows = None
-        if b.n_big and self._pieces(s):
-            k_rows = torch.empty((b.T, s.kv_heads * s.dim), dtype=raw.dtype, device=raw.device)
-            v_rows = torch.empty((b.T, s.kv_heads * s.vdim), dtype=raw.dtype, device=raw.device)
+        q = k_rows = v_rows = None
+        plan = R.AttnPlan(s.chunk, self._pieces(s))
+        n = b.kv_rows(plan)
+        if n:       # head sizes the kernel does not have are padded with zeros
+            P = R.row_head(s.dim, s.vdim)
+            new = torch.empty if s.dim == s.vdim == P else torch.zeros
+            k_rows, v_rows = (new((n, s.kv_heads, P), dtype=raw.dtype, device=raw.device)
+                              for _ in range(2))
+            q = new((b.T, s.heads, P), dtype=raw.dtype, device=raw.device)
         q = R.shortconv_attn(
             raw, layer.seg["k"], layer.seg["v"], layer.conv, self.state[l, "conv"], s.heads,
             s.kv_heads, s.dim, s.vdim, b, rope.get(layer.rope_key), c.k[i], c.v[i], c.page_table,
             v_first=v_first if s.v_mix else None, mix=layer.mix if s.v_mix and not first else None,
-            write_first=first, k_rows=k_rows, v_rows=v_rows)
+            write_first=first, k_rows=k_rows, v_rows=v_rows, q=q)
         R.ragged_attention(q, c.k[i], c.v[i], c.page_table, b, s.heads, s.kv_heads, s.dim, s.vdim,
                            s.scale, cat[:, :layer.out_dim], chunk=s.chunk, sink=layer.sink,
                            gate=raw[:, layer.seg["g"]:], max_ctx=max_ctx,
-                           k_rows=k_rows, v_rows=v_rows)
+                           k_rows=k_rows, v_rows=v_rows, plan=plan)
         return v_first
 
     def _delta(self, l: int, layer, raw: torch.Tensor, cat: torch.Tensor, b: R.RaggedBatch) -> None:

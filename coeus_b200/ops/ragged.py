@@ -41,27 +41,33 @@ class Entry:
 
 @dataclass(frozen=True)
 class AttnPlan:
-    """How the long entries of a batch go through attention under one mask.  A piece is a run of
-    rows that starts at a chunk's start (or at position 0), so that its rows see one another and
-    nothing else: it needs no cache and takes the piece kernel.  What comes before an entry's
-    first piece sees cached keys too and goes in tiles of ``ATTN_TILE`` rows."""
+    """How the long entries of a batch go through attention under one mask.  The rows of an entry
+    that lie in one chunk form a piece for the tcgen05 kernel.  A piece that starts at its chunk's
+    start (or at position 0) needs only this step's keys and values; one that continues a chunk
+    also needs the cached ones, which are gathered into rows for it.  A continued chunk of few
+    rows is not worth that and goes in tiles of ``ATTN_TILE`` rows that read the cache."""
 
     chunk: Optional[int]
     pieces: bool              # whether the layer's sizes allow the piece kernel
 
 
 def pieces_allowed(dim: int, vdim: int, chunk: Optional[int], scale: float) -> bool:
-    return dim == vdim and dim in (64, 128) and scale > 0 and (chunk is None or chunk >= MIN_PIECE)
+    return max(dim, vdim) <= 128 and scale > 0 and (chunk is None or chunk >= MIN_PIECE)
+
+
+def row_head(dim: int, vdim: int) -> int:
+    """Distance of the heads in the row-wise q, k and v of the piece kernel."""
+    return 64 if max(dim, vdim) <= 64 else 128
 
 
 def _cut(plan: AttnPlan, pos0: int, n: int):
-    """``(rows before the first piece, [(offset, rows), ...])`` of an entry of ``n`` tokens."""
-    if not plan.pieces:
-        return n, []
+    """``(rows that continue a chunk, positions of that chunk before them, [(offset, rows), ...])``
+    of an entry of ``n`` tokens."""
     if plan.chunk is None:
-        return (n, []) if pos0 else (0, [(0, n)])
+        return (n, pos0, []) if pos0 else (0, 0, [(0, n)])
     head = min(n, -pos0 % plan.chunk)
-    return head, [(o, min(plan.chunk, n - o)) for o in range(head, n, plan.chunk)]
+    return head, pos0 % plan.chunk, [(o, min(plan.chunk, n - o))
+                                     for o in range(head, n, plan.chunk)]
 
 
 class RaggedBatch:
@@ -99,18 +105,27 @@ class RaggedBatch:
                  rows, want]
         self.plans, cols = {}, len(parts)
         for plan in dict.fromkeys(plans):
-            tiles, pieces = [], []
+            tiles, pieces, where = [], [], []
+            extra = 0
             for i in big:
-                head, ps = _cut(plan, entries[i].pos0, lens[i])
-                tiles += [(i, o, min(ATTN_TILE, head - o)) for o in range(0, head, ATTN_TILE)]
-                pieces += [(int(row0[i]) + o, m) for o, m in ps]
+                p0, r0 = entries[i].pos0, int(row0[i])
+                head, ahead, ps = _cut(plan, p0, lens[i]) if plan.pieces else (lens[i], 0, [])
+                if plan.pieces and head > MIN_PIECE:
+                    keys = np.arange(p0 - ahead, p0 + head, dtype=np.int32)
+                    where.append(np.stack([np.full_like(keys, entries[i].slot), keys], 1))
+                    pieces.append((r0, head, self.T + extra, ahead))
+                    extra += len(keys)
+                else:
+                    tiles += [(i, o, min(ATTN_TILE, head - o)) for o in range(0, head, ATTN_TILE)]
+                pieces += [(r0 + o, m, r0 + o, 0) for o, m in ps]
             tiles.sort(key=lambda t: -(entries[t[0]].pos0 + t[1]))     # the most keys first
-            pieces.sort(key=lambda t: -t[1])
-            if pieces and sum(len(x) for x in parts) % 2:              # pairs are read as int2
-                parts.append(np.zeros(1, np.int32))
-            self.plans[plan] = (len(tiles), len(pieces), max([m for _, m in pieces], default=0),
-                                len(parts))
+            pieces.sort(key=lambda t: -t[1] * (t[1] + 2 * t[3]))
+            if pieces:                                                 # read four at a time
+                parts.append(np.zeros(-sum(len(x) for x in parts) % 4, np.int32))
+            self.plans[plan] = (len(tiles), len(pieces), max([t[1] for t in pieces], default=0),
+                                extra, len(parts))
             parts += [np.asarray(pieces, np.int32).reshape(-1),
+                      np.concatenate(where).reshape(-1) if where else np.zeros(0, np.int32),
                       *np.asarray(tiles, np.int32).reshape(-1, 3).T]
         host = torch.from_numpy(np.concatenate(parts).astype(np.int32, copy=False))
         if into is None:
@@ -132,9 +147,16 @@ class RaggedBatch:
         self.n_big = len(big)
 
     def plan(self, plan: AttnPlan):
-        """``(tiles, pieces, longest piece, piece array, tile entries, offsets, lengths)``."""
-        n_tiles, n_pieces, longest, at = self.plans[plan]
-        return (n_tiles, n_pieces, longest, *self._views[at:at + 4])
+        """``(tiles, pieces, longest piece, gathered rows, piece array, (slot, position) of the
+        gathered rows, tile entries, offsets, lengths)``."""
+        n_tiles, n_pieces, longest, extra, at = self.plans[plan]
+        return (n_tiles, n_pieces, longest, extra, *self._views[at:at + 5])
+
+    def kv_rows(self, plan: AttnPlan) -> int:
+        """Rows of the ``k_rows`` / ``v_rows`` buffers under ``plan``: this step's, then gathered
+        ones (0: no piece, no buffers)."""
+        _, n_pieces, _, extra, _ = self.plans[plan]
+        return self.T + extra if n_pieces else 0
 
     def entry_args(self):
         return _p(self.slot), _p(self.row0), _p(self.len), _p(self.pos0)
@@ -219,13 +241,15 @@ def shortconv_attn(raw: torch.Tensor, koff: int, voff: int, taps_w: torch.Tensor
                    v_cache: torch.Tensor, page_table: torch.Tensor,
                    v_first: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
                    write_first: bool = False, k_rows: Optional[torch.Tensor] = None,
-                   v_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   v_rows: Optional[torch.Tensor] = None, q: Optional[torch.Tensor] = None
+                   ) -> torch.Tensor:
     """What stands between the projections and the scores of an attention layer: a causal
     convolution over time on every channel of q, k and v (``taps_w [taps, channels]``), rotary
     embedding of the first ``2 * rope.shape[1]`` entries of the q and k heads in the rotate-half
     layout, value mixing ``v <- (1 - mix) v + mix v_first`` (or, with ``write_first``, keeping v as
     ``v_first``), and the write of k and v into the cache pages (and, when given, row by row into
-    ``k_rows [rows, kv_heads*dim]`` and ``v_rows``).  Returns ``q [rows, heads*dim]``."""
+    the first rows of ``k_rows [.., kv_heads, P]`` and ``v_rows``).  Returns ``q [rows, heads, dim]``, or
+    fills the ``q [rows, heads, Q >= dim]`` it is given; padding is left alone."""
     T = raw.shape[0]
     half = rope.shape[1] if rope is not None else 0
     mode = 1 if write_first else (2 if mix is not None else 0)
@@ -249,17 +273,15 @@ def shortconv_attn(raw: torch.Tensor, koff: int, voff: int, taps_w: torch.Tensor
         page, at = _cells(page_table, batch)
         k_cache[page, at, :, :dim] = k.to(k_cache.dtype)
         v_cache[page, at, :, :vdim] = v.to(v_cache.dtype)
-        if k_rows is not None:
-            k_rows.copy_(k.reshape(T, -1))
-            v_rows.copy_(v.reshape(T, -1))
-        return q.reshape(T, qc).to(raw.dtype)
-    q = torch.empty((T, qc), dtype=raw.dtype, device=raw.device)
+        return q.to(raw.dtype)
+    if q is None:
+        q = torch.empty((T, heads, dim), dtype=raw.dtype, device=raw.device)
     rc = _lib.serving_lib().cb_shortconv_attn(
         _p(raw), raw.stride(0), koff, voff, _p(taps_w), taps_w.shape[0], _p(state), heads, kv_heads,
         dim, vdim, *batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off), batch.n_conv, half,
-        _p(rope), _p(q), _p(k_cache), _p(v_cache), k_cache.shape[-1], v_cache.shape[-1],
+        _p(rope), _p(q), q.shape[2], _p(k_cache), _p(v_cache), k_cache.shape[-1], v_cache.shape[-1],
         _p(page_table), page_table.shape[1], k_cache.shape[0], _p(v_first), _p(mix), mode,
-        _p(k_rows), _p(v_rows), int(raw.dtype == torch.float32), _p(_lib.status_buffer(raw.device)), _lib.stream_ptr())
+        _p(k_rows), _p(v_rows), k_rows.shape[2] if k_rows is not None else dim, int(raw.dtype == torch.float32), _p(_lib.status_buffer(raw.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_shortconv_attn")
     return q
 
@@ -356,15 +378,17 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      chunk: Optional[int] = None, sink: Optional[torch.Tensor] = None,
                      gate: Optional[torch.Tensor] = None, max_ctx: Optional[int] = None,
                      k_rows: Optional[torch.Tensor] = None,
-                     v_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     v_rows: Optional[torch.Tensor] = None,
+                     plan: Optional[AttnPlan] = None) -> torch.Tensor:
     """Causal attention of every query row over the cached keys of its own sequence, restricted to
     the row's chunk (positions with the same ``pos // chunk``) when ``chunk`` is given.  ``sink``
     (fp32 ``[heads]``) is a logit that enters the softmax denominator only; ``gate`` (a view whose
     column ``h`` belongs to head ``h``) multiplies head ``h``'s output by its sigmoid.  Query head
-    ``h`` reads key/value head ``h // (heads // kv_heads)``.  ``out`` is a ``[rows, heads * vdim]``
+    ``h`` reads key/value head ``h // (heads // kv_heads)``.  ``q`` is ``[rows, heads, Q >= dim]``, ``out`` a ``[rows, heads * vdim]``
     view; ``max_ctx`` bounds the keys of any row (it only chooses how many CTAs share a row).  With
-    this step's ``k_rows`` and ``v_rows`` at hand, runs of rows that see no earlier step go through
-    the tcgen05 kernel (:class:`AttnPlan`; the batch must have been built with the layer's plan)."""
+    row-wise ``k_rows`` and ``v_rows`` at hand (:meth:`RaggedBatch.kv_rows` rows of ``[kv_heads, P]``,
+    this step's filled in; q then has the same head distance P), the pieces of ``plan`` go through
+    the tcgen05 kernel; the default plan has pieces when the buffers are given."""
     T = q.shape[0]
     if not q.is_cuda:
         per = heads // kv_heads
@@ -376,7 +400,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             K = k_cache[pages].reshape(-1, kv_heads, k_cache.shape[-1])[:n, :, :dim].float()
             V = v_cache[pages].reshape(-1, kv_heads, v_cache.shape[-1])[:n, :, :vdim].float()
             K, V = K.repeat_interleave(per, 1), V.repeat_interleave(per, 1)
-            s = torch.einsum("thd,nhd->htn", q[r:r + m].float().view(m, heads, dim), K) * scale
+            s = torch.einsum("thd,nhd->htn", q[r:r + m].float(), K) * scale
             j = torch.arange(n)
             lo = pos // chunk * chunk if chunk else torch.zeros_like(pos)
             ok = (j[None] <= pos[:, None]) & (j[None] >= lo[:, None])
@@ -396,23 +420,29 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         return out
     st = _p(_lib.status_buffer(q.device))
     lib = _lib.serving_lib()
-    common = (_p(q), _p(k_cache), _p(v_cache), _p(page_table), page_table.shape[1],
+    common = (_p(q), q.shape[2], _p(k_cache), _p(v_cache), _p(page_table), page_table.shape[1],
               k_cache.shape[0], heads, kv_heads, dim, vdim, k_cache.shape[-1], v_cache.shape[-1],
               chunk or 0, _F(scale), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0,
               _p(out), out.stride(0))
     if batch.n_big:
-        n_tiles, n_pieces, longest, pieces, t_entry, t_off, t_len = batch.plan(
-            AttnPlan(chunk, k_rows is not None))
+        n_tiles, n_pieces, longest, extra, pieces, where, t_entry, t_off, t_len = batch.plan(
+            plan or AttnPlan(chunk, k_rows is not None))
         if n_tiles:
             rc = lib.cb_ragged_attn_tiles(*common, *batch.entry_args(), _p(t_entry), _p(t_off),
                                           _p(t_len), n_tiles, st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_ragged_attn_tiles")
+        if extra:
+            rc = lib.cb_kv_gather(_p(k_cache), _p(v_cache), kv_heads, k_cache.shape[-1],
+                                  v_cache.shape[-1], _p(page_table), page_table.shape[1],
+                                  k_cache.shape[0], _p(where), extra, _p(k_rows[T:]), _p(v_rows[T:]),
+                                  k_rows.shape[2], st, _lib.stream_ptr())
+            _lib.check_rc(rc, "cb_kv_gather")
         if n_pieces:
             rc = lib.cb_attn_fwd_pieces(
-                _p(q), _p(k_rows), _p(v_rows), _p(out), T, _p(pieces), n_pieces, longest, heads,
-                kv_heads, dim, q.stride(0), k_rows.stride(0), v_rows.stride(0), out.stride(0),
-                _F(scale), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0, st,
-                _lib.stream_ptr())
+                _p(q), _p(k_rows), _p(v_rows), _p(out), T, k_rows.shape[0], _p(pieces), n_pieces,
+                longest, heads, kv_heads, k_rows.shape[2], vdim, q.stride(0), k_rows.stride(0),
+                v_rows.stride(0), out.stride(0), _F(scale), _p(sink), _p(gate),
+                gate.stride(0) if gate is not None else 0, st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_attn_fwd_pieces")
     n = batch.n_rows
     if n:

@@ -147,8 +147,8 @@ def kernel_table(size: str = "1b-layers") -> List[Dict]:
                 (h1, la.w_up, out1[:, la.act_off:], "relu2", None, False)), bytes_=wb(n_in, W))
         rope = R.rope_table(batch.pos, lm.inv_freq[la.rope_key])
         st, c = eng.state, eng.cache
-        kr = t(T, kv * d) if S > 1 else None
-        vr = t(T, kv * d) if S > 1 else None
+        kr = t(T, kv, d) if S > 1 else None
+        vr = t(T, kv, d) if S > 1 else None
         vf = t(T, kv * d)
         qkv = (nh + 2 * kv) * d
         rec("shortconv_attn", phase, lambda: R.shortconv_attn(
@@ -156,7 +156,7 @@ def kernel_table(size: str = "1b-layers") -> List[Dict]:
             c.v[0], c.page_table, v_first=vf, mix=la.mix, k_rows=kr, v_rows=vr),
             bytes_=T * (2 * qkv + 2 * kv * d * (2 if S > 1 else 0) + kv * d) * 2
             + (0 if S > 1 else T * 2 * 3 * qkv * 2))
-        q = t(T, nh * d)
+        q = t(T, nh, d)
         gate = raw[:, la.seg["g"]:]
         attn = lambda: R.ragged_attention(                              # noqa: E731
             q, c.k[0], c.v[0], c.page_table, batch, nh, kv, d, d, d ** -0.5, out[:, :nh * d],
@@ -166,12 +166,13 @@ def kernel_table(size: str = "1b-layers") -> List[Dict]:
             rec("attention (prompt pieces)", phase, attn, flops=4 * pairs * nh * d)
             for b in range(B):
                 eng.cache.reserve(b, 1024)
-            pairs = B * (512 * 512 + 512 * 512 / 2)
+            pairs = B * (512 * 512 + 512 * 512 / 2)      # half a chunk behind the cached other half
             part = eng._batch([R.Entry(b, 512, [0] * 512) for b in range(B)])
+            k2, v2 = (t(part.kv_rows(R.AttnPlan(CHUNK, True)), kv, d) for _ in range(2))
             rec("attention (rest of a chunk, cached keys)", phase, lambda: R.ragged_attention(
                 q[:B * 512], c.k[0], c.v[0], c.page_table, part, nh, kv, d, d, d ** -0.5,
                 out[:B * 512, :nh * d], chunk=CHUNK, sink=la.sink, gate=gate[:B * 512],
-                k_rows=kr[:B * 512], v_rows=vr[:B * 512]), flops=4 * pairs * nh * d)
+                k_rows=k2, v_rows=v2), flops=4 * pairs * nh * d)
         else:
             rec("attention (decode)", phase, attn,
                 bytes_=B * (at % CHUNK + 1) * kv * d * 2 * 2)
@@ -199,7 +200,7 @@ def kernel_table(size: str = "1b-layers") -> List[Dict]:
         if S > 1:
             rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), flops=2 * T * W * qkv)
             kk, vv = t(T, kv * d), t(T, kv * d)
-            rec("closest: attention", phase, lambda: A.attention_fwd(q, kk, vv, B, S, nh, d, causal=True),
+            rec("closest: attention", phase, lambda: A.attention_fwd(q.view(T, -1), kk, vv, B, S, nh, d, causal=True),
                 flops=4 * B * S * S / 2 * nh * d)
         else:
             rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), bytes_=wb(W, qkv))
@@ -207,7 +208,7 @@ def kernel_table(size: str = "1b-layers") -> List[Dict]:
             pages = (CONTEXT + 63) // 64
             kc, vc = t(B * pages, 64, kv, d), t(B * pages, 64, kv, d)
             pt = torch.arange(B * pages, dtype=torch.int32, device=dev).view(B, pages)
-            rec("closest: attention", phase, lambda: D.decode_attention(q, kc, vc, pt, ctx, nh, d, nkv=kv),
+            rec("closest: attention", phase, lambda: D.decode_attention(q.view(T, -1), kc, vc, pt, ctx, nh, d, nkv=kv),
                 bytes_=B * CONTEXT * kv * d * 2 * 2)
         buf = t(T, qkv)
         pos = torch.full((B,), at, dtype=torch.int32, device=dev)

@@ -347,7 +347,7 @@ def check_attention_inputs(device, dtype, tol):
             want_k = y[:, qc:qc + kc].view(T, Gk, d)
             want_k = plain.rotate_half(want_k, 2 * half, 300.0) if half else want_k
             want_v = 0.7 * y[:, qc + kc:] + 0.3 * firsts[s].cpu().double()
-            assert rel(torch.cat(qs[s]), want_q.reshape(T, -1)) < tol
+            assert rel(torch.cat(qs[s]), want_q) < tol
             got_k = kcache[table[slot].long()].reshape(-1, Gk, kcache.shape[-1])[:T, :, :d]
             got_v = vcache[table[slot].long()].reshape(-1, Gk, vcache.shape[-1])[:T, :, :dv]
             assert rel(got_k, want_k) < tol
@@ -402,7 +402,7 @@ def check_attention(device, dtype, tol):
             gate = torch.randn((m, H_ + 3), generator=g).to(dtype)
             b = batch_of([(0, start, m)], device, dtype == torch.bfloat16, chunk)
             out = torch.full((m, H_ * dv + 8), 5.0, dtype=dtype, device=device)
-            args = (q.reshape(m, -1).to(device), kc, vc, table, b, H_, Gk, d, dv, scale,
+            args = (q.to(device), kc, vc, table, b, H_, Gk, d, dv, scale,
                     out[:, :H_ * dv])
             kw = dict(chunk=chunk, sink=sink.to(device), gate=gate.to(device)[:, 2:])
             R.ragged_attention(*args, **kw)
@@ -417,8 +417,15 @@ def check_attention(device, dtype, tol):
             assert rel(out[:, :H_ * dv], want.reshape(m, -1)) < tol, (H_, d, chunk, start, m)
             if rows_too:       # the same with this step's keys and values at hand, row by row
                 out.fill_(5.0)
-                R.ragged_attention(*args, **kw, k_rows=k[start:start + m].reshape(m, -1).to(device),
-                                   v_rows=v[start:start + m].reshape(m, -1).to(device))
+                P, rows = R.row_head(d, dv), b.kv_rows(R.AttnPlan(chunk, True))
+                kr, vr = (torch.zeros((max(rows, 1), Gk, P), dtype=dtype, device=device)
+                          for _ in range(2))
+                qp = torch.zeros((m, H_, P), dtype=dtype, device=device)
+                if rows:
+                    kr[:m, :, :d], vr[:m, :, :dv] = k[start:start + m], v[start:start + m]
+                qp[:, :, :d] = q
+                R.ragged_attention(qp, *args[1:], **kw, k_rows=kr, v_rows=vr,
+                                   plan=R.AttnPlan(chunk, True))
                 assert rel(out[:, :H_ * dv], want.reshape(m, -1)) < tol, (H_, d, chunk, start, m)
             assert float((out[:, H_ * dv:].float() - 5.0).abs().max()) == 0
 
