@@ -20,7 +20,6 @@ from .decode import PAGE
 CONV_TILE = 16        # tokens per block of the convolution kernels
 ATTN_TILE = 64        # query rows per block of the tensor-core attention kernel
 ROWS_MAX = 4          # entries of at most this many tokens take the row kernel
-SCAN_SINGLE = 2       # longest entry up to which the recurrence takes tokens one by one
 MIN_PIECE = 64        # chunks from this size on are worth a piece of their own
 _F = ctypes.c_float
 
@@ -103,7 +102,6 @@ class RaggedBatch:
         parts = [pos, np.asarray(self.pos0_host, np.int32), tokens, row_slot,
                  np.asarray(self.slots_host, np.int32), row0[:n], np.asarray(lens, np.int32),
                  np.asarray([c[0] for c in ct], np.int32), np.asarray([c[1] for c in ct], np.int32),
-                 np.cumsum([0] + [-(-m // CONV_TILE) for m in lens[:-1]]).astype(np.int32),
                  rows, want]
         self.plans, cols = {}, len(parts)
         for plan in dict.fromkeys(plans):
@@ -142,7 +140,7 @@ class RaggedBatch:
             views.append(self.buf[o:o + len(part)])
             o += len(part)
         (self.pos, self.pos0, self.tokens, self.row_slot, self.slot, self.row0, self.len,
-         self.conv_entry, self.conv_off, self.conv_first, self.rows, self.want) = views[:cols]
+         self.conv_entry, self.conv_off, self.rows, self.want) = views[:cols]
         self._views = views
         self.positions = self.buf[:self.T + n]       # pos and pos0: what a decode step advances
         self.n_conv, self.n_rows, self.n_want = len(ct), len(rows), len(want)
@@ -350,17 +348,6 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, kq: torch.Tensor, v: torch.Tens
                 o[t] = torch.einsum("hdv,hd->hv", S, qq)
             state[s] = S
             r += m
-        return o
-    if max(batch.lens) > SCAN_SINGLE:
-        # four tokens at a time; scratch for the vectors and coefficients of every block
-        groups = 4 * batch.n_conv
-        vecs = torch.empty((heads, groups, 13, P), dtype=torch.float32, device=v.device)
-        scal = torch.empty((heads, groups, 20), dtype=torch.float32, device=v.device)
-        rc = _lib.serving_lib().cb_delta_scan_blocks(
-            _p(q), _p(k), _p(v), _p(g), _p(beta), _p(state), _p(o), _p(vecs), _p(scal), T, heads,
-            kv_heads, dim, P, vdim, *batch.entry_args(), batch.n, _p(batch.conv_entry),
-            _p(batch.conv_off), _p(batch.conv_first), batch.n_conv, _lib.stream_ptr())
-        _lib.check_rc(rc, "cb_delta_scan_blocks", launches=2)
         return o
     rc = _lib.serving_lib().cb_delta_scan(
         _p(q), _p(k), _p(kq), _p(v), _p(g), _p(beta), _p(state), _p(o), T, heads, kv_heads, dim,
