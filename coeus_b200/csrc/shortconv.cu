@@ -8,7 +8,8 @@
 // one.  Inside a step they are earlier rows of the projection; at the start of an entry they come
 // from the slot's state, [n - 1, channels] projected values in time order.  The block that owns
 // an entry's first tile is the only one that reads the state, so it alone replaces it, after its
-// last read.
+// last read.  (A convolution may have at most CONV_TILE + 1 taps, so that no other
+// tile reaches back to the state.)
 #include "ragged.cuh"
 
 namespace cb {
@@ -39,47 +40,22 @@ __device__ __forceinline__ int raw_col_delta(const ConvIn& p, int c) {
   return c < qc ? c : (c < 2 * qc ? p.koff + (c - qc) : p.voff + (c - 2 * qc));
 }
 
-// V consecutive channels from c (columns from col) of the token at offset t of the entry.  TAPS > 0
-// is the number of taps, known at compile time so that all loads are issued together; 0: any.
-template <typename T, int V, int TAPS>
-__device__ __forceinline__ void conv_at(const ConvIn& p, int c, int col, int channels, int row0,
-                                        int t, int slot, bool has_state, float* y) {
+// Channel c (column col) of the token at offset t of the entry, any number of taps.
+template <typename T>
+__device__ __forceinline__ float conv_at(const ConvIn& p, int c, int col, int channels, int row0,
+                                         int t, int slot, bool has_state) {
   const T* raw = static_cast<const T*>(p.raw) + static_cast<ptrdiff_t>(row0) * p.ld + col;
-  const int n1 = (TAPS > 0 ? TAPS : p.taps) - 1;
+  const int n1 = p.taps - 1;
   const T* st = static_cast<const T*>(p.state) + static_cast<ptrdiff_t>(slot) * n1 * channels + c;
-#pragma unroll
-  for (int i = 0; i < V; ++i) y[i] = 0.f;
-  if constexpr (TAPS > 0) {
-    float u[TAPS][V], w[TAPS][V];
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) {
-      const int o = t - (TAPS - 1) + j;
-      const bool ok = o >= 0 || has_state;
-      const T* src = o >= 0 || !ok ? raw + static_cast<ptrdiff_t>(max(o, 0)) * p.ld
-                                   : st + static_cast<ptrdiff_t>(n1 + o) * channels;
-      load_vec<V>(src, u[j]);
-      load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * channels + c, w[j]);
-      if (!ok) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) u[j][i] = 0.f;
-      }
-    }
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j)
-#pragma unroll
-      for (int i = 0; i < V; ++i) y[i] += u[j][i] * w[j][i];
-  } else {
-    for (int j = 0; j <= n1; ++j) {
-      const int o = t - n1 + j;
-      float u[V], w[V];
-      if (o < 0 && !has_state) continue;
-      load_vec<V>(o >= 0 ? raw + static_cast<ptrdiff_t>(o) * p.ld
-                         : st + static_cast<ptrdiff_t>(n1 + o) * channels, u);
-      load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * channels + c, w);
-#pragma unroll
-      for (int i = 0; i < V; ++i) y[i] += u[i] * w[i];
-    }
+  float y = 0.f;
+  for (int j = 0; j <= n1; ++j) {
+    const int o = t - n1 + j;
+    if (o < 0 && !has_state) continue;
+    const float u = to_f32(o >= 0 ? raw[static_cast<ptrdiff_t>(o) * p.ld]
+                                  : st[static_cast<ptrdiff_t>(n1 + o) * channels]);
+    y += u * p.taps_w[static_cast<ptrdiff_t>(j) * channels + c];
   }
+  return y;
 }
 
 // The state of channel c after the entry's len tokens.
@@ -118,7 +94,8 @@ struct AttnPre {
 };
 
 // grid (tiles, kv_heads): the block's channels are its key/value head and the query heads on it.
-template <typename T, int V, int TAPS>
+// One channel (or rotated pair) at a time, for sizes and taps that the tile kernel does not take.
+template <typename T>
 __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const AttnPre p) {
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -128,72 +105,49 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_attn_kernel(const Attn
   const int qc = ci.heads * dim, kc = ci.kv_heads * dim;
   const int channels = qc + kc + ci.kv_heads * vdim;
   const int nt = min(CONV_TILE, len - off);
-  // per head: half / V units that make two rotated vectors, then plain units
-  const int pair_u = p.half / V, plain_u = (dim - 2 * p.half) / V, head_u = pair_u + plain_u;
-  const int v_u = vdim / V, units = (per + 1) * head_u + v_u;
+  const int head_u = dim - p.half;           // per head: rotated pairs, then single channels
+  const int heads_u = (per + 1) * head_u, units = heads_u + vdim;
   const float lam = p.mix_mode == 2 ? *p.lambda : 0.f;
   for (int i = threadIdx.x; i < nt * units; i += CONV_THREADS) {
     const int t = off + i / units, u = i % units, row = row0 + t, pos = pos0 + t;
     const int lp = pos / RAGGED_PAGE;
-    const bool in_table = lp < p.max_pages;
-    const int page = in_table ? p.page_table[static_cast<size_t>(slot) * p.max_pages + lp] : -1;
+    const int page = lp < p.max_pages ? p.page_table[static_cast<size_t>(slot) * p.max_pages + lp] : -1;
     if (page < 0 || page >= p.num_pages) {
       record_status(p.status, ST_BOUNDS, row);
       continue;
     }
     const size_t cell = (static_cast<size_t>(page) * RAGGED_PAGE + pos % RAGGED_PAGE) * ci.kv_heads + g;
-    if (u < (per + 1) * head_u) {
+    const size_t row_cell = (static_cast<size_t>(row) * ci.kv_heads + g) * p.row_head;
+    if (u < heads_u) {
       const int hi = u / head_u, k = u % head_u;       // hi < per: query head, else the key head
       const bool is_q = hi < per;
       const int base = is_q ? (g * per + hi) * dim : qc + g * dim;
       const int colb = is_q ? base : ci.koff + g * dim;
       T* dst = is_q ? static_cast<T*>(p.q) + (static_cast<size_t>(row) * ci.heads + g * per + hi) * p.q_head
                     : static_cast<T*>(p.k_cache) + cell * p.dim_p;
-      if (k < pair_u) {
-        const int d = k * V;
-        float a[V], b[V], oa[V], ob[V];
-        conv_at<T, V, TAPS>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
-        conv_at<T, V, TAPS>(ci, base + p.half + d, colb + p.half + d, channels, row0, t, slot, has_state, b);
-#pragma unroll
-        for (int x = 0; x < V; ++x) {
-          const float2 cs = p.rope[static_cast<size_t>(row) * p.half + d + x];
-          oa[x] = a[x] * cs.x - b[x] * cs.y;
-          ob[x] = b[x] * cs.x + a[x] * cs.y;
-        }
-        store_vec<V>(dst + d, oa);
-        store_vec<V>(dst + p.half + d, ob);
-        if (!is_q && p.k_rows != nullptr) {
-          T* kr = static_cast<T*>(p.k_rows) + (static_cast<size_t>(row) * ci.kv_heads + g) * p.row_head + d;
-          store_vec<V>(kr, oa);
-          store_vec<V>(kr + p.half, ob);
-        }
-      } else {
-        const int d = 2 * p.half + (k - pair_u) * V;
-        float a[V];
-        conv_at<T, V, TAPS>(ci, base + d, colb + d, channels, row0, t, slot, has_state, a);
-        store_vec<V>(dst + d, a);
-        if (!is_q && p.k_rows != nullptr)
-          store_vec<V>(static_cast<T*>(p.k_rows) + (static_cast<size_t>(row) * ci.kv_heads + g) * p.row_head + d, a);
+      T* kr = !is_q && p.k_rows != nullptr ? static_cast<T*>(p.k_rows) + row_cell : nullptr;
+      const int d = k < p.half ? k : k + p.half;
+      float a = conv_at<T>(ci, base + d, colb + d, channels, row0, t, slot, has_state);
+      if (k < p.half) {
+        const float b = conv_at<T>(ci, base + p.half + d, colb + p.half + d, channels, row0, t, slot, has_state);
+        const float2 cs = p.rope[static_cast<size_t>(row) * p.half + d];
+        const T hi_half = from_f32<T>(b * cs.x + a * cs.y);
+        a = a * cs.x - b * cs.y;
+        dst[p.half + d] = hi_half;
+        if (kr != nullptr) kr[p.half + d] = hi_half;
       }
+      dst[d] = from_f32<T>(a);
+      if (kr != nullptr) kr[d] = from_f32<T>(a);
     } else {
-      const int d = (u - (per + 1) * head_u) * V;
-      float a[V];
-      conv_at<T, V, TAPS>(ci, qc + kc + g * vdim + d, ci.voff + g * vdim + d, channels, row0, t, slot,
-                    has_state, a);
+      const int d = u - heads_u;
+      float a = conv_at<T>(ci, qc + kc + g * vdim + d, ci.voff + g * vdim + d, channels, row0, t, slot, has_state);
       if (p.mix_mode != 0) {
         T* vf = static_cast<T*>(p.v_first) + static_cast<size_t>(row) * ci.kv_heads * vdim + g * vdim + d;
-        if (p.mix_mode == 1) {
-          store_vec<V>(vf, a);
-        } else {
-          float f[V];
-          load_vec<V>(vf, f);
-#pragma unroll
-          for (int x = 0; x < V; ++x) a[x] = (1.f - lam) * a[x] + lam * f[x];
-        }
+        if (p.mix_mode == 1) *vf = from_f32<T>(a);
+        else a = (1.f - lam) * a + lam * to_f32(*vf);
       }
-      store_vec<V>(static_cast<T*>(p.v_cache) + cell * p.vdim_p + d, a);
-      if (p.v_rows != nullptr)
-        store_vec<V>(static_cast<T*>(p.v_rows) + (static_cast<size_t>(row) * ci.kv_heads + g) * p.row_head + d, a);
+      static_cast<T*>(p.v_cache)[cell * p.vdim_p + d] = from_f32<T>(a);
+      if (p.v_rows != nullptr) static_cast<T*>(p.v_rows)[row_cell + d] = from_f32<T>(a);
     }
   }
   if (off == 0 && ci.taps > 1) {
@@ -444,24 +398,8 @@ __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-
 __device__ __forceinline__ float softplus_exact(float x) {
   return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
 }
-template <int V>
-__device__ __forceinline__ void load_f32(const float* p, float* f) {
-  if constexpr (V == 4) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
-  } else {
-    f[0] = *p;
-  }
-}
-template <int V>
-__device__ __forceinline__ void store_f32(float* p, const float* f) {
-  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  else *p = f[0];
-}
-
-// grid (tiles, kv_heads): one query/key head and the value heads on it.  V consecutive channels
-// per thread (4 when dim and vdim are multiples of four).
-template <typename T, int V, int TAPS>
+// grid (tiles, kv_heads): one query/key head and the value heads on it; one channel at a time.
+template <typename T>
 __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_kernel(const DeltaPre p) {
   const ConvIn& ci = p.c;
   const int e = ci.tile_entry[blockIdx.x], off = ci.tile_off[blockIdx.x], g = blockIdx.y;
@@ -475,69 +413,48 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_delta_kernel(const Del
   const float qscale = 1.0f / sqrtf(static_cast<float>(dim));
   // q and k: a warp per token
   for (int t = off + warp; t < off + nt; t += CONV_THREADS / 32) {
-    constexpr int NI = 256 / (32 * V);           // dim <= 256
-    float qv[NI][V], kv[NI][V], sq = 0.f, sk = 0.f, dot = 0.f;
+    constexpr int NI = 8;                        // dim <= 256
+    float qv[NI], kv[NI], sq = 0.f, sk = 0.f, dot = 0.f;
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int d = (lane + 32 * i) * V;
-#pragma unroll
-      for (int x = 0; x < V; ++x) qv[i][x] = kv[i][x] = 0.f;
+      const int d = lane + 32 * i;
+      qv[i] = kv[i] = 0.f;
       if (d < dim) {
-        conv_at<T, V, TAPS>(ci, g * dim + d, g * dim + d, channels, row0, t, slot, has_state, qv[i]);
-        conv_at<T, V, TAPS>(ci, qc + g * dim + d, ci.koff + g * dim + d, channels, row0, t, slot, has_state, kv[i]);
-#pragma unroll
-        for (int x = 0; x < V; ++x) {
-          qv[i][x] = silu_exact(qv[i][x]);
-          kv[i][x] = silu_exact(kv[i][x]);
-          sq += qv[i][x] * qv[i][x];
-          sk += kv[i][x] * kv[i][x];
-        }
+        qv[i] = silu_exact(conv_at<T>(ci, g * dim + d, g * dim + d, channels, row0, t, slot, has_state));
+        kv[i] = silu_exact(conv_at<T>(ci, qc + g * dim + d, ci.koff + g * dim + d, channels, row0, t, slot, has_state));
       }
+      sq += qv[i] * qv[i];
+      sk += kv[i] * kv[i];
     }
     const float rq = qscale / sqrtf(warp_sum(sq) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f);
     const size_t cell = static_cast<size_t>(g) * p.rows + row0 + t;
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int d = (lane + 32 * i) * V;
-#pragma unroll
-      for (int x = 0; x < V; ++x) {
-        qv[i][x] *= rq;
-        kv[i][x] *= rk;
-        dot += qv[i][x] * kv[i][x];
-      }
+      const int d = lane + 32 * i;
+      qv[i] *= rq;
+      kv[i] *= rk;
+      dot += qv[i] * kv[i];
       if (d < p.dim_p) {
-        store_f32<V>(p.q + cell * p.dim_p + d, qv[i]);
-        store_f32<V>(p.k + cell * p.dim_p + d, kv[i]);
+        p.q[cell * p.dim_p + d] = qv[i];
+        p.k[cell * p.dim_p + d] = kv[i];
       }
     }
     dot = warp_sum(dot);
     if (lane == 0) p.kq[cell] = dot;
   }
   const T* raw = static_cast<const T*>(ci.raw);
-  const int vn = per * vdim / V;
-  for (int i = threadIdx.x; i < nt * vn; i += CONV_THREADS) {
-    const int t = off + i / vn, c = g * per * vdim + (i % vn) * V;
-    float y[V];
-    conv_at<T, V, TAPS>(ci, 2 * qc + c, ci.voff + c, channels, row0, t, slot, has_state, y);
-#pragma unroll
-    for (int x = 0; x < V; ++x) y[x] = silu_exact(y[x]);
-    store_f32<V>(p.v + static_cast<size_t>(row0 + t) * ci.heads * vdim + c, y);
+  for (int i = threadIdx.x; i < nt * per * vdim; i += CONV_THREADS) {
+    const int t = off + i / (per * vdim), c = g * per * vdim + i % (per * vdim);
+    p.v[static_cast<size_t>(row0 + t) * ci.heads * vdim + c] =
+        silu_exact(conv_at<T>(ci, 2 * qc + c, ci.voff + c, channels, row0, t, slot, has_state));
   }
-  const int gn = p.dim_p / V;
-  for (int i = threadIdx.x; i < nt * per * gn; i += CONV_THREADS) {
-    const int h = g * per + (i / gn) % per, row = row0 + off + i / (gn * per), d = (i % gn) * V;
-    float f[V];
-#pragma unroll
-    for (int x = 0; x < V; ++x) f[x] = 0.f;
-    if (d < dim) {
-      float a[V], b[V];
-      load_f32<V>(p.a + static_cast<size_t>(row) * p.lda + h * dim + d, a);
-      load_f32<V>(p.dt_bias + h * dim + d, b);
-      const float rate = expf(p.A_log[h]);
-#pragma unroll
-      for (int x = 0; x < V; ++x) f[x] = expf(-rate * softplus_exact(a[x] + b[x]));
-    }
-    store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row) * p.dim_p + d, f);
+  for (int i = threadIdx.x; i < nt * per * p.dim_p; i += CONV_THREADS) {
+    const int h = g * per + (i / p.dim_p) % per, row = row0 + off + i / (p.dim_p * per), d = i % p.dim_p;
+    float f = 0.f;
+    if (d < dim)
+      f = expf(-expf(p.A_log[h]) *
+               softplus_exact(p.a[static_cast<size_t>(row) * p.lda + h * dim + d] + p.dt_bias[h * dim + d]));
+    p.g[(static_cast<size_t>(h) * p.rows + row) * p.dim_p + d] = f;
   }
   for (int i = threadIdx.x; i < nt * per; i += CONV_THREADS) {
     const int h = g * per + i / nt, row = row0 + off + i % nt;
@@ -598,7 +515,7 @@ __global__ void __launch_bounds__(CONV_THREADS, 6) shortconv_delta_tile_kernel(c
       const bool in = d < dim;
       const float rate = expf(p.A_log[h]);
       float b[V] = {};
-      if (in) load_f32<V>(p.dt_bias + h * dim + d, b);
+      if (in) load_vec<V>(p.dt_bias + h * dim + d, b);
       float4 ra[CONV_TILE / 4];
 #pragma unroll
       for (int j = 0; j < CONV_TILE / 4; ++j) {
@@ -614,7 +531,7 @@ __global__ void __launch_bounds__(CONV_THREADS, 6) shortconv_delta_tile_kernel(c
         float f[V];
 #pragma unroll
         for (int x = 0; x < V; ++x) f[x] = in ? expf(-rate * softplus_exact(a[x] + b[x])) : 0.f;
-        store_f32<V>(p.g + (static_cast<size_t>(h) * p.rows + row0 + off + ta + j) * p.dim_p + d, f);
+        store_vec<V>(p.g + (static_cast<size_t>(h) * p.rows + row0 + off + ta + j) * p.dim_p + d, f);
       }
     }
   }
@@ -671,8 +588,8 @@ __global__ void __launch_bounds__(CONV_THREADS, 6) shortconv_delta_tile_kernel(c
           qq[i][x] *= rq;
           k[i][x] *= rk;
         }
-        store_f32<V>(p.q + cell * p.dim_p + d, qq[i]);
-        store_f32<V>(p.k + cell * p.dim_p + d, k[i]);
+        store_vec<V>(p.q + cell * p.dim_p + d, qq[i]);
+        store_vec<V>(p.k + cell * p.dim_p + d, k[i]);
       }
       if (lane == 0) p.kq[cell] = dot * rq * rk;
     }
@@ -692,7 +609,7 @@ __global__ void __launch_bounds__(CONV_THREADS, 6) shortconv_delta_tile_kernel(c
       w.next(src, y);
 #pragma unroll
       for (int x = 0; x < V; ++x) y[x] = silu_act<T>(y[x]);
-      store_f32<V>(dst, y);
+      store_vec<V>(dst, y);
     }
   }
   for (int i = threadIdx.x; i < (t1 - off) * per; i += CONV_THREADS) {
@@ -776,7 +693,7 @@ static int launch_conv_attn(const AttnPre& p, dim3 grid, bool vec, cudaStream_t 
       default: rc = launch_attn_tile<T, 4>(p, grid, threads, smem, st);
     }
   } else {
-    shortconv_attn_kernel<T, 1, 0><<<grid, CONV_THREADS, 0, st>>>(p);
+    shortconv_attn_kernel<T><<<grid, CONV_THREADS, 0, st>>>(p);
   }
   return rc != 0 ? rc : (cudaGetLastError() == cudaSuccess ? 0 : -3);
 }
@@ -792,7 +709,7 @@ static int launch_conv_delta(const DeltaPre& p, dim3 grid, bool vec, cudaStream_
       default: rc = launch_delta_tile<T, 4>(p, grid, smem, st);
     }
   } else {
-    shortconv_delta_kernel<T, 1, 0><<<grid, CONV_THREADS, 0, st>>>(p);
+    shortconv_delta_kernel<T><<<grid, CONV_THREADS, 0, st>>>(p);
   }
   return rc != 0 ? rc : (cudaGetLastError() == cudaSuccess ? 0 : -3);
 }
@@ -823,7 +740,7 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
                                  int vdim_p, const int* page_table, int max_pages, int num_pages,
                                  void* v_first, const float* lambda, int mix_mode, void* k_rows,
                                  void* v_rows, int row_head, int f32, int* status, void* stream) {
-  if (tiles <= 0 || taps < 1 || kv_heads < 1 || heads % kv_heads != 0 || 2 * half > dim) return -1;
+  if (tiles <= 0 || taps < 1 || taps > CONV_TILE + 1 || kv_heads < 1 || heads % kv_heads != 0 || 2 * half > dim) return -1;
   if (mix_mode != 0 && v_first == nullptr) return -2;
   AttnPre p;
   p.c = conv_in(raw, ld, koff, voff, taps_w, taps, state, heads, kv_heads, dim, vdim, slot, row0, len,
@@ -864,7 +781,7 @@ extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, i
                                   float* kq, float* v, float* g, float* beta, int rows, int dim_p,
                                   int f32,
                                   void* stream) {
-  if (tiles <= 0 || taps < 1 || kv_heads < 1 || heads % kv_heads != 0) return -1;
+  if (tiles <= 0 || taps < 1 || taps > CONV_TILE + 1 || kv_heads < 1 || heads % kv_heads != 0) return -1;
   if (dim > 256 || dim_p % 32 != 0 || dim_p < dim || dim_p > 256) return -2;
   DeltaPre p;
   p.c = conv_in(raw, ld, koff, voff, taps_w, taps, state, heads, kv_heads, dim, vdim, slot, row0, len,

@@ -20,6 +20,7 @@ from ..foundation.error import ConfigError, ProcessingError
 
 ARCHITECTURES = ("Sapasun",)
 MAX_HEAD_DIM = 256           # the attention and recurrence kernels' limit per head
+MAX_TAPS = 17                # and of the convolution kernels
 DEFAULT_MAX_SEQ_LEN = 8192   # serving default; the design itself has no length limit
 
 
@@ -103,8 +104,8 @@ class HybridConfig:
             if not (1 <= m.dim <= MAX_HEAD_DIM and 1 <= m.vdim <= MAX_HEAD_DIM):
                 raise ConfigError.invalid(where, f"{m.dim}/{m.vdim}",
                                           f"Head sizes must lie in 1..{MAX_HEAD_DIM}")
-            if m.conv < 1:
-                raise ConfigError.invalid(where, m.conv, "A convolution has at least one tap")
+            if not 1 <= m.conv <= MAX_TAPS:
+                raise ConfigError.invalid(where, m.conv, f"A convolution has 1 to {MAX_TAPS} taps")
             if isinstance(m, AttentionSpec):
                 if m.rot_dims % 2 or not 0 <= m.rot_dims <= m.dim:
                     raise ConfigError.invalid(where, m.rot_dims,
