@@ -107,19 +107,23 @@ __device__ __forceinline__ float exp2_poly(float x) {
 // item of every wave of gridDim.x items, counted from the front of even waves and from the back
 // of odd ones, so that the heavy and the light ends of the sorted list meet in one CTA), within
 // an item key tile by key tile, tile A before tile B.
+template <bool PIECES>
 struct AFWalk {
   // problem
   int n_items, n_bh, n_pairs, n_q_tiles, n_kv_tiles, nh, causal, bkv, n_waves;
   // position
   int wave, j, t;
   int b, h, qa;          // batch, head, first query tile of the pair
-  int row0, len;         // first row and rows of the sequence (or piece)
-  int kv_row0, ahead;    // first key row, keys before the first query's own
+  int4 piece;            // PIECES: the entry of AttnFwdArgs::pieces
   const int4* pieces;
   int n0, n1, nmax;      // key tiles of tile A / B (0: the tile does not exist)
   int kv_seq;            // how many (item, j) groups came before this one: the K/V ring position
   bool valid;
 
+  __device__ int first_row(const AttnFwdArgs& p) const { return PIECES ? piece.x : b * p.S; }
+  __device__ int first_key(const AttnFwdArgs& p) const { return PIECES ? piece.z : b * p.S; }
+  __device__ int rows(const AttnFwdArgs& p) const { return PIECES ? piece.y : p.S; }
+  __device__ int keys_ahead() const { return PIECES ? piece.w : 0; }   // keys before query 0's own
   __device__ void init(const AttnFwdArgs& p, int bkv_) {
     bkv = bkv_;
     n_q_tiles = (p.S + AF_BM - 1) / AF_BM;
@@ -130,8 +134,6 @@ struct AFWalk {
     n_items = n_pairs * n_bh;
     causal = p.causal;
     pieces = p.pieces;
-    len = p.S;
-    ahead = 0;
     n_waves = (n_items + gridDim.x - 1) / gridDim.x;
     wave = -1;
     kv_seq = -1;
@@ -151,18 +153,13 @@ struct AFWalk {
       b = bh / nh;
       h = bh % nh;
       qa = 2 * pair;
-      if (pieces != nullptr) {
-        const int4 pc = pieces[b];
-        row0 = pc.x;
-        len = pc.y;
-        kv_row0 = pc.z;
-        ahead = pc.w;
-        n_q_tiles = (len + AF_BM - 1) / AF_BM;
-        n_kv_tiles = (ahead + len + bkv - 1) / bkv;
+      if constexpr (PIECES) {
+        piece = pieces[b];
+        n_q_tiles = (piece.y + AF_BM - 1) / AF_BM;
+        n_kv_tiles = (piece.w + piece.y + bkv - 1) / bkv;
         if (qa >= n_q_tiles) continue;             // a shorter piece ends before this pair
-      } else {
-        row0 = kv_row0 = b * len;
       }
+      const int ahead = keys_ahead();
       n0 = causal ? min(n_kv_tiles, (ahead + (qa + 1) * AF_BM + bkv - 1) / bkv) : n_kv_tiles;
       n1 = qa + 1 >= n_q_tiles ? 0
            : (causal ? min(n_kv_tiles, (ahead + (qa + 2) * AF_BM + bkv - 1) / bkv) : n_kv_tiles);
@@ -187,7 +184,7 @@ struct AFWalk {
   __device__ bool last_of_tile() const { return j == (t ? n1 : n0) - 1; }
 };
 
-template <int DH, bool POLY, bool DROP>
+template <int DH, bool POLY, bool DROP, bool PIECES>
 __global__ void __launch_bounds__(AF_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const AttnFwdArgs p) {
@@ -257,10 +254,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       uint32_t qcnt[2] = {0u, 0u};     // uses of each query buffer so far
       uint32_t kcnt = 0, vcnt = 0;     // K / V tiles loaded so far
       bool ok = true;
-      AFWalk w;
+      AFWalk<PIECES> w;
       w.init(p, BKV);
       while (w.valid && ok) {
-        const int row0 = w.row0, kv_row0 = w.kv_row0;
+        const int row0 = w.first_row(p), kv_row0 = w.first_key(p);
         const int h = w.h, hk = w.h / group, qa = w.qa;
         const int n0 = w.n0, n1 = w.n1, nmax = w.nmax;
         auto load_q = [&](int t) {
@@ -346,7 +343,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem_base, 0);
       bool ok = true;
       int v_waited = -1;
-      AFWalk wp;
+      AFWalk<PIECES> wp;
       wp.init(p, BKV);
       for (uint32_t gp = 0; wp.valid && ok; wp.advance(), ++gp) {
         const uint32_t buf = gp % NBUF;
@@ -401,7 +398,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
         return ok;
       };
-      AFWalk ws;
+      AFWalk<PIECES> ws;
       ws.init(p, BKV);
       for (uint32_t gs = 0; ws.valid && ok; ws.advance(), ++gs) {
         const int t = ws.t;
@@ -453,7 +450,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     bool ok = true;
     float m_used = -INFINITY;
     float l[4] = {0.f, 0.f, 0.f, 0.f};           // the row sum is kept as four partial sums
-    AFWalk w;
+    AFWalk<PIECES> w;
     w.init(p, BKV);
     for (; w.valid && ok; w.advance(), ++g) {
       if (w.t != t) continue;
@@ -514,8 +511,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (tr) tr[tri] = clock64();
       tc_fence_after();
       const int kv0 = j * BKV;
-      const bool need_mask = (p.causal && kv0 + BKV - 1 > q0 + w.ahead) || (kv0 + BKV > w.ahead + w.len);
-      const int kv_limit = w.ahead + (p.causal ? min(q_idx, w.len - 1) : (w.len - 1));  // last visible key
+      const bool need_mask = (p.causal && kv0 + BKV - 1 > q0 + w.keys_ahead()) ||
+                             (kv0 + BKV > w.keys_ahead() + w.rows(p));
+      const int kv_limit = w.keys_ahead() + (p.causal ? min(q_idx, w.rows(p) - 1) : (w.rows(p) - 1));  // last visible key
       uint32_t v[BKV];
 #pragma unroll
       for (int c = 0; c < BKV / 32; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v + c * 32);
@@ -637,13 +635,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       tc_fence_after();
       const float lsum = (l[0] + l[1]) + (l[2] + l[3]);
       float inv_l = lsum > 0.f ? 1.0f / lsum : 0.f;
-      const bool row_ok = q_idx < w.len;
-      const size_t out_row = static_cast<size_t>(w.row0) + q_idx;
-      if (p.sink != nullptr)
-        inv_l = 1.0f / (lsum + exp2f(p.sink[w.h] * 1.4426950408889634f - m_used));
-      if (p.gate != nullptr && row_ok)
-        inv_l /= 1.0f + expf(-__bfloat162float(p.gate[out_row * p.ldg + w.h]));
-      __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * p.vdim;
+      const bool row_ok = q_idx < w.rows(p);
+      const size_t out_row = static_cast<size_t>(w.first_row(p)) + q_idx;
+      if constexpr (PIECES) {
+        if (p.sink != nullptr)
+          inv_l = 1.0f / (lsum + exp2f(p.sink[w.h] * 1.4426950408889634f - m_used));
+        if (p.gate != nullptr && row_ok)
+          inv_l /= 1.0f + expf(-__bfloat162float(p.gate[out_row * p.ldg + w.h]));
+      }
+      __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * (PIECES ? p.vdim : DH);
 #pragma unroll 1
       for (int c = 0; c < DH / 32; ++c) {
         uint32_t o[32];
@@ -658,7 +658,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
             wv.z = pack_bf16x2(__uint_as_float(o[8 * gq + 4]) * inv_l, __uint_as_float(o[8 * gq + 5]) * inv_l);
             wv.w = pack_bf16x2(__uint_as_float(o[8 * gq + 6]) * inv_l, __uint_as_float(o[8 * gq + 7]) * inv_l);
             const int d0 = c * 32 + gq * 8;
-            if (d0 + 8 <= p.vdim && (p.vdim & 7) == 0) {
+            if (!PIECES || (d0 + 8 <= p.vdim && (p.vdim & 7) == 0)) {
               *reinterpret_cast<uint4*>(orow + d0) = wv;
             } else {
 #pragma unroll
@@ -686,13 +686,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
-template <int DH, bool POLY, bool DROP = false>
+template <int DH, bool POLY, bool DROP = false, bool PIECES = false>
 static int launch_attn_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
                               const AttnFwdArgs& a, int max_ctas, cudaStream_t st) {
   using Cfg = AFCfg<DH>;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attn_fwd_kernel<DH, POLY, DROP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attn_fwd_kernel<DH, POLY, DROP, PIECES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              Cfg::SMEM_BYTES) != cudaSuccess)
       return -10;
     configured = true;
@@ -702,7 +702,7 @@ static int launch_attn_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const C
   int grid = sm_count();
   if (max_ctas > 0 && max_ctas < grid) grid = max_ctas;
   if (items < grid) grid = items;
-  attn_fwd_kernel<DH, POLY, DROP><<<grid, AF_THREADS, Cfg::SMEM_BYTES, st>>>(tq, tk, tv, a);
+  attn_fwd_kernel<DH, POLY, DROP, PIECES><<<grid, AF_THREADS, Cfg::SMEM_BYTES, st>>>(tq, tk, tv, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
 }
 
@@ -804,6 +804,6 @@ extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, v
   a.gate = static_cast<const __nv_bfloat16*>(gate);
   a.ldg = ldg;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return dh == 64 ? launch_attn_fwd<64, false>(tq, tk, tv, a, 0, st)
-                  : launch_attn_fwd<128, false>(tq, tk, tv, a, 0, st);
+  return dh == 64 ? launch_attn_fwd<64, false, false, true>(tq, tk, tv, a, 0, st)
+                  : launch_attn_fwd<128, false, false, true>(tq, tk, tv, a, 0, st);
 }

@@ -83,7 +83,7 @@ def throughput(model, steps: int, warmup: int) -> List[Dict]:
     return out
 
 
-def kernel_table(size: str = "1b-layers") -> List[Dict]:
+def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> List[Dict]:
     """Every kernel of the design and the like kernels of the closest model on the shapes of
     ``size``: a prompt batch of 8 x 2048 tokens and a decode step of 64 sequences.  ``bound`` names
     the roofline (measured copy bandwidth, measured bf16 throughput, or fp32 FMA issue at the
@@ -102,7 +102,9 @@ def kernel_table(size: str = "1b-layers") -> List[Dict]:
     rows: List[Dict] = []
 
     def rec(name, phase, fn, bytes_=0, flops=0, fma=0):
-        us = timeit(fn, 3, 10, True) * 1e3
+        if only not in f"{name}, {phase}":
+            return
+        us = timeit(fn, min(3, iters), iters, True) * 1e3
         kind, best = ("bytes", bytes_ / hbm / 1e3) if bytes_ else (
             ("bf16", flops / tensor / 1e6) if flops else ("fp32", fma / fp32 * 1e6))
         rows.append({"kernel": name, "phase": phase, "us": round(us, 1), "bound": kind,
@@ -256,3 +258,22 @@ def run(steps: int = 20, warmup: int = 3, kernels: bool = False, sampler=None) -
     if kernels:
         for row in kernel_table():
             print(json.dumps(row), flush=True)
+
+
+def main(argv=None) -> int:
+    """``python -m coeus_b200.utils.serving_bench --kernel delta_scan``: the kernel table alone, or the
+    rows whose ``name, phase`` contains the text (with ``--iters 1`` a small case for a profiler)."""
+    import argparse
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--size", default="1b-layers", choices=list(SIZES))
+    ap.add_argument("--kernel", default="")
+    ap.add_argument("--iters", type=int, default=10)
+    a = ap.parse_args(argv)
+    for row in kernel_table(a.size, a.kernel, a.iters):
+        print(json.dumps(row), flush=True)
+    return 0
+
+
+if __name__ == "__main__":
+    import sys
+    sys.exit(main())
