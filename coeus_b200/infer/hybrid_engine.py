@@ -255,7 +255,6 @@ class HybridEngine(InferenceEngine):
                 want = [s1 - s0 - 1] if s1 == S else []
                 got = self.step([Entry(b, s0, rows[b][s0:s1], want) for b in group])
             out.append(got.clone())
-        self._B = B
         return torch.cat(out)
 
     def decode_step(self, tokens: torch.Tensor) -> torch.Tensor:
