@@ -58,7 +58,8 @@ def _worker(rank, world, port, batch, out):
     losses = [float(tr.train_step(mine[:, :-1], mine[:, 1:])) for _ in range(3)]
     full = dp.gather_master()
     if rank == 0:
-        out.put((losses, full.clone(), model.p16.float().clone()))
+        # plain arrays: shared tensors would need this process alive until they are taken
+        out.put((losses, full.numpy().copy(), model.p16.float().numpy().copy()))
     dist.barrier()
     dist.destroy_process_group()
 
@@ -75,7 +76,8 @@ def test_two_ranks_match_one_rank():
     procs = [ctx.Process(target=_worker, args=(r, 2, port, batch, q)) for r in range(2)]
     for p in procs:
         p.start()
-    losses, master, p16 = q.get(timeout=300)
+    losses, *arrays = q.get(timeout=300)
+    master, p16 = (torch.from_numpy(a) for a in arrays)
     for p in procs:
         p.join(timeout=60)
         assert p.exitcode == 0
