@@ -39,8 +39,9 @@ NVCC_FLAGS = [
 ]
 
 
-SERVING_SOURCES = ("gemm", "ragged_rows", "shortconv", "delta_scan", "linear_f32", "linear_skinny",
-                   "ragged_attn", "attention_fwd")
+SERVING_SOURCES = ("gemm", "ragged_rows", "residual", "shortconv", "delta_scan", "ssd", "mingru",
+                   "linear_f32", "linear_skinny", "linear_heads", "ragged_attn", "latent_attn",
+                   "attention_fwd")
 
 
 def _nvcc() -> str:

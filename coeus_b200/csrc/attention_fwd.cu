@@ -49,12 +49,14 @@ struct AttnFwdArgs {
   float drop_scale;
   // Pieces of unequal length instead of B sequences of S rows.  Piece b has y = pieces[b].y query
   // rows (at most S) from row pieces[b].x on and w + y keys from row pieces[b].z of K and V on; its
-  // query i sees the first w + i + 1 of them (causal).  null: none
+  // query i sees the first w + i + 1 of them (causal), or of those the last `window`.  null: none
   const int4* pieces;
   int vdim;                    // columns of a head that are stored, vdim apart in O
   const float* sink;           // [nh] logits that enter the denominator only, or null
-  const __nv_bfloat16* gate;   // [rows, ldg], column h: head h's output times its sigmoid; or null
-  int ldg;
+  const __nv_bfloat16* gate;   // [rows, ldg] or null: the output times its sigmoid, column h for all
+  int ldg;                     // of head h, or (gate_wide) column h * vdim + d for its column d
+  int gate_wide;
+  int window;                  // 0: no window
 };
 
 // Optional device timeline of CTA 0 (clock64 stamps; see cb_attn_fwd_set_trace): softmax warp 0
@@ -511,8 +513,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (tr) tr[tri] = clock64();
       tc_fence_after();
       const int kv0 = j * BKV;
+      const bool below = PIECES && p.window > 0;
       const bool need_mask = (p.causal && kv0 + BKV - 1 > q0 + w.keys_ahead()) ||
-                             (kv0 + BKV > w.keys_ahead() + w.rows(p));
+                             (kv0 + BKV > w.keys_ahead() + w.rows(p)) ||
+                             (below && kv0 < q0 + AF_BM + w.keys_ahead() - p.window);
       const int kv_limit = w.keys_ahead() + (p.causal ? min(q_idx, w.rows(p) - 1) : (w.rows(p) - 1));  // last visible key
       uint32_t v[BKV];
 #pragma unroll
@@ -521,10 +525,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (tr) tr[tri + 1] = clock64();
       if (need_mask) {
         // hidden keys get a score of -inf, after which the step takes the common path (their
-        // exponential is an exact zero); with causal masking every row sees at least key 0
+        // exponential is an exact zero); with causal masking every row sees at least key 0, with
+        // a window at least its own key
+        const int kv_low = below ? kv_limit - p.window : -1;
 #pragma unroll
         for (int e = 0; e < BKV; ++e)
-          if (kv0 + e > kv_limit) v[e] = 0xff800000u;
+          if (kv0 + e > kv_limit || (PIECES && kv0 + e <= kv_low)) v[e] = 0xff800000u;
       }
       float mx;
       {
@@ -566,7 +572,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         for (int a = 0; a < 4; ++a) l[a] *= f;
       }
       g_prev = g;
+      // a row that has seen no key yet (below its window) keeps a maximum under every score
       if (grow) m_used = (m_new == -INFINITY) ? 0.f : m_new;
+      else if (PIECES && m_used == -INFINITY) m_used = -1e30f;
       // P = exp2(s * scale - m) as packed bf16 over the first half of the score buffer; row sum
       const float sc = p.scale_log2, nm = -m_used;
       if (tr) tr[tri + 2] = clock64();
@@ -640,7 +648,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if constexpr (PIECES) {
         if (p.sink != nullptr)
           inv_l = 1.0f / (lsum + exp2f(p.sink[w.h] * 1.4426950408889634f - m_used));
-        if (p.gate != nullptr && row_ok)
+        if (p.gate != nullptr && row_ok && !p.gate_wide)
           inv_l /= 1.0f + expf(-__bfloat162float(p.gate[out_row * p.ldg + w.h]));
       }
       __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * (PIECES ? p.vdim : DH);
@@ -650,6 +658,26 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         tmem_ld_32x32b_x32(o_addr + c * 32, o);
         tmem_ld_wait();
         if (row_ok) {
+          if constexpr (PIECES) {
+            if (p.gate != nullptr && p.gate_wide) {
+              const __nv_bfloat16* gp = p.gate + out_row * p.ldg + static_cast<size_t>(w.h) * p.vdim + c * 32;
+              const bool vec = (p.vdim & 7) == 0;
+#pragma unroll
+              for (int gq = 0; gq < 4; ++gq) {
+                float f[8];
+                if (vec && c * 32 + gq * 8 < p.vdim) {
+                  load8(gp + gq * 8, f);
+                } else {
+#pragma unroll
+                  for (int x = 0; x < 8; ++x)
+                    f[x] = c * 32 + gq * 8 + x < p.vdim ? __bfloat162float(gp[gq * 8 + x]) : 0.f;
+                }
+#pragma unroll
+                for (int x = 0; x < 8; ++x)
+                  o[8 * gq + x] = __float_as_uint(__fdividef(__uint_as_float(o[8 * gq + x]), 1.0f + __expf(-f[x])));
+              }
+            }
+          }
 #pragma unroll
           for (int gq = 0; gq < 4; ++gq) {
             uint4 wv;
@@ -748,6 +776,8 @@ extern "C" int cb_attn_fwd_dropout(const void* q, const void* k, const void* v, 
   a.sink = nullptr;
   a.gate = nullptr;
   a.ldg = 0;
+  a.gate_wide = 0;
+  a.window = 0;
   a.drop_thr = drop_thr;
   a.drop_key = drop_key;
   a.drop_scale = 256.0f / static_cast<float>(256 - drop_thr);
@@ -773,15 +803,18 @@ extern "C" int cb_attn_fwd(const void* q, const void* k, const void* v, void* o,
 // Causal attention of a ragged batch in pieces (see AttnFwdArgs): n_pieces quadruples over `rows`
 // query rows and `kv_rows` key rows, none with more than max_len queries.  Heads of q, k and v are
 // dh apart (64 or 128, padded with zeros), heads of o vdim <= dh.  sink (fp32 [nh]) is a logit per head
-// that enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view) multiplies
-// head h's output by its sigmoid; both may be null.  scale > 0.
+// that enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view, or with
+// gate_wide column h * vdim + d) multiplies head h's output by its sigmoid; both may be null.  A
+// query sees the last `window` of its keys (0: all).  scale > 0.
 extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, void* o, int rows,
                                   int kv_rows, const void* pieces, int n_pieces, int max_len, int nh,
                                   int nkv, int dh, int vdim, int ldq, int ldk, int ldv, int ldo,
                                   float scale, const float* sink, const void* gate, int ldg,
-                                  int* status, void* stream) {
+                                  int gate_wide, int window, int* status, void* stream) {
   using namespace cb;
   if (dh != 64 && dh != 128) return -1;
+  if (gate_wide && vdim % 8 == 0 && ((reinterpret_cast<uintptr_t>(gate) & 15u) || ldg % 8)) return -6;
+  if (window < 0) return -2;
   if (rows <= 0 || kv_rows <= 0 || n_pieces <= 0 || max_len <= 0 || nh <= 0 || nkv <= 0 ||
       (nh % nkv) != 0 || (ldo % 8) != 0 || vdim < 1 || vdim > dh || !(scale > 0.f))
     return -2;
@@ -803,6 +836,8 @@ extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, v
   a.sink = sink;
   a.gate = static_cast<const __nv_bfloat16*>(gate);
   a.ldg = ldg;
+  a.gate_wide = gate_wide;
+  a.window = window;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dh == 64 ? launch_attn_fwd<64, false, false, true>(tq, tk, tv, a, 0, st)
                   : launch_attn_fwd<128, false, false, true>(tq, tk, tv, a, 0, st);

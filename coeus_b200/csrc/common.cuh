@@ -18,6 +18,21 @@ __device__ __forceinline__ float gelu_tanh(float x) {
   const float u = 0.7978845608028654f * x * (1.0f + 0.044715f * x * x);
   return 0.5f * x * (1.0f + tanh_fast(u));
 }
+__device__ __forceinline__ float gelu_erf(float x) {
+  return 0.5f * x * (1.0f + erff(x * 0.7071067811865476f));
+}
+// The same for results that are rounded to bf16: erf by formula 7.1.26 of Abramowitz and Stegun's
+// Handbook of Mathematical Functions (absolute error below 1.5e-7) with the fast exponential.
+__device__ __forceinline__ float gelu_erf_bf16(float x) {
+  const float a = fabsf(x) * 0.7071067811865476f;
+  const float t = __fdividef(1.0f, fmaf(0.3275911f, a, 1.0f));
+  float q = fmaf(1.061405429f, t, -1.453152027f);
+  q = fmaf(q, t, 1.421413741f);
+  q = fmaf(q, t, -0.284496736f);
+  q = fmaf(q, t, 0.254829592f);
+  const float tail = 0.5f * q * t * __expf(-a * a);      // half of erfc(a)
+  return x * (x >= 0.f ? 1.0f - tail : tail);
+}
 __device__ __forceinline__ float gelu_tanh_grad(float x) {
   const float x2 = x * x;
   const float u = 0.7978845608028654f * x * (1.0f + 0.044715f * x2);

@@ -13,7 +13,7 @@
 //   wgrad    dW[K,N] = X[M,K]^T . dY[M,N]     A MN-major, B MN-major (split along tokens,
 //                                             fp32 atomic accumulation)
 // Fused epilogues: alpha scale, +bias[N], GELU(tanh) with the pre-activation kept, dGELU, squared
-// ReLU, +residual, bf16 / fp32 / fp32-atomic-add output.
+// ReLU, GELU(erf), +residual, bf16 / fp32 / fp32-atomic-add output.
 #include <cudaTypedefs.h>
 
 #include <cstring>
@@ -30,7 +30,8 @@ constexpr int AG_PARTS = 8;   // row groups a pulled tile is split into
 constexpr int MAX_TP = 8;
 enum : int { COMM_NONE = 0, COMM_AG = 1, COMM_RS = 2 };
 
-enum : int { EPI_NONE = 0, EPI_GELU = 1, EPI_DGELU = 2, EPI_SWIGLU_BWD = 3, EPI_RELU2 = 4 };
+enum : int { EPI_NONE = 0, EPI_GELU = 1, EPI_DGELU = 2, EPI_SWIGLU_BWD = 3, EPI_RELU2 = 4,
+             EPI_GELU_ERF = 6 };
 enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_F32_ATOMIC = 2, OUT_DISCARD = 3 };
 
 struct GemmArgs {
@@ -132,6 +133,9 @@ __device__ __forceinline__ void epilogue_math(const GemmArgs& p, float* v, float
       v[j] = fmaxf(v[j], 0.f);
       v[j] *= v[j];
     }
+  } else if (p.epi == EPI_GELU_ERF) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = gelu_erf_bf16(v[j]);
   } else if (p.epi == EPI_DGELU && row_ok) {
     const __nv_bfloat16* ap = p.aux_in + static_cast<size_t>(row) * p.ldaux + col0;
 #pragma unroll

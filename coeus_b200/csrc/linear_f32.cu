@@ -1,16 +1,16 @@
-// fp32 linear layer Y[M, N] = act(X[M, K] . W[N, K]^T) on the FMA units, for serving a model in
+// fp32 linear layer Y[M, N] = act(X[M, K] . W[N, K]^T + bias[N]) on the FMA units, for serving a model in
 // full 32-bit precision: 64 x 64 tiles, 4 x 4 outputs per thread, operands staged in shared memory.
 #include "ragged.cuh"
 
 namespace cb {
 
 constexpr int LT = 64, LK = 16;
-enum : int { ACT_NONE = 0, ACT_RELU2 = 4, ACT_SOFTCAP = 5 };
+enum : int { ACT_NONE = 0, ACT_RELU2 = 4, ACT_SOFTCAP = 5, ACT_GELU_ERF = 6 };
 
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw,
-                  float* __restrict__ y, int ldy, int M, int N, int K, int act, float act_arg,
-                  int accumulate) {
+                  const float* __restrict__ bias, float* __restrict__ y, int ldy, int M, int N,
+                  int K, int act, float act_arg, int accumulate) {
   __shared__ float sx[LK][LT + 4], sw[LK][LT + 4];
   const int m0 = blockIdx.y * LT, n0 = blockIdx.x * LT;
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
@@ -46,7 +46,10 @@ linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict_
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       float v = acc[i][j];
-      if (act == ACT_RELU2) {
+      if (bias != nullptr) v += bias[n];
+      if (act == ACT_GELU_ERF) {
+        v = gelu_erf(v);
+      } else if (act == ACT_RELU2) {
         v = fmaxf(v, 0.f);
         v *= v;
       } else if (act == ACT_SOFTCAP) {
@@ -60,13 +63,13 @@ linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict_
 
 }  // namespace cb
 
-extern "C" int cb_linear_f32(const float* x, int ldx, const float* w, int ldw, float* y, int ldy,
-                             int M, int N, int K, int act, float act_arg, int accumulate,
+extern "C" int cb_linear_f32(const float* x, int ldx, const float* w, int ldw,
+                             const float* bias, float* y, int ldy, int M, int N, int K, int act, float act_arg, int accumulate,
                              void* stream) {
   if (M <= 0 || N <= 0 || K <= 0 || K % 4 || ldx % 4 || ldw % 4) return -1;
   dim3 grid((N + cb::LT - 1) / cb::LT, (M + cb::LT - 1) / cb::LT);
   if (grid.y > 65535) return -1;
   cb::linear_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      x, ldx, w, ldw, y, ldy, M, N, K, act, act_arg, accumulate);
+      x, ldx, w, ldw, bias, y, ldy, M, N, K, act, act_arg, accumulate);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

@@ -1,5 +1,5 @@
-// bf16 linear layers of a decode step: Y[M, N] = act(X[M, K] . W[N, K]^T) with few rows (M <= 16),
-// bound by streaming the weights.  The weights are the 16-row operand of mma m16n8k16 and the
+// bf16 linear layers of a decode step: Y[M, N] = act(X[M, K] . W[N, K]^T + bias[N]) with few rows
+// (M <= 16), bound by streaming the weights.  The weights are the 16-row operand of mma m16n8k16 and the
 // tokens its 8 columns; every lane reads 32 consecutive bytes of a weight row per 64-wide slice
 // of K (the contraction index is permuted the same way on both sides, so fragments come straight
 // from global memory).  The warps of a CTA split K and add their results through shared memory.
@@ -9,11 +9,12 @@
 
 namespace cb {
 
-enum : int { SK_NONE = 0, SK_RELU2 = 4, SK_SOFTCAP = 5 };
+enum : int { SK_NONE = 0, SK_RELU2 = 4, SK_SOFTCAP = 5, SK_GELU_ERF = 6 };
 
 struct SkinnyProblem {
   const __nv_bfloat16* x;   // [M, ldx]
   const __nv_bfloat16* w;   // [N, ldw]
+  const __nv_bfloat16* bias;   // [N] or null
   void* y;                  // [M, ldy] bf16 or fp32
   int ldx, ldw, ldy, N, K, act, f32, accumulate;
   float act_arg;
@@ -117,7 +118,10 @@ __global__ void __launch_bounds__(WARPS * 32) linear_skinny_kernel(const SkinnyA
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) v += red[(w * NT * 8 + m) * LD + c];
-    if (p.act == SK_RELU2) {
+    if (p.bias != nullptr) v += __bfloat162float(p.bias[n]);
+    if (p.act == SK_GELU_ERF) {
+      v = gelu_erf(v);
+    } else if (p.act == SK_RELU2) {
       v = fmaxf(v, 0.f);
       v *= v;
     } else if (p.act == SK_SOFTCAP) {
@@ -153,31 +157,32 @@ static int launch_skinny(SkinnyArgs a, int count, cudaStream_t st) {
 
 using namespace cb;
 
-static int skinny_problem(SkinnyProblem& p, const void* x, int ldx, const void* w, int ldw, void* y,
-                          int ldy, int N, int K, int act, float act_arg, int f32, int accumulate) {
+static int skinny_problem(SkinnyProblem& p, const void* x, int ldx, const void* w, int ldw,
+                          const void* bias, void* y, int ldy, int N, int K, int act, float act_arg, int f32, int accumulate) {
   if (N <= 0 || K <= 0 || K % 8 || ldx % 8 || ldw % 8 || (accumulate && !f32)) return -1;
   if ((reinterpret_cast<uintptr_t>(x) & 15u) || (reinterpret_cast<uintptr_t>(w) & 15u)) return -2;
   p.x = static_cast<const __nv_bfloat16*>(x);
   p.w = static_cast<const __nv_bfloat16*>(w);
+  p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.y = y; p.ldx = ldx; p.ldw = ldw; p.ldy = ldy; p.N = N; p.K = K; p.act = act; p.f32 = f32;
   p.accumulate = accumulate; p.act_arg = act_arg;
   return 0;
 }
 
 // The second problem is skipped when x1 is null.
-extern "C" int cb_linear_skinny(const void* x0, int ldx0, const void* w0, int ldw0, void* y0,
-                                int ldy0, int N0, int K0, int act0, float arg0, int f32_0, int acc0,
-                                const void* x1, int ldx1, const void* w1, int ldw1, void* y1,
-                                int ldy1, int N1, int K1, int act1, float arg1, int f32_1, int acc1,
+extern "C" int cb_linear_skinny(const void* x0, int ldx0, const void* w0, int ldw0,
+                                const void* b0, void* y0, int ldy0, int N0, int K0, int act0, float arg0, int f32_0, int acc0,
+                                const void* x1, int ldx1, const void* w1, int ldw1,
+                                const void* b1, void* y1, int ldy1, int N1, int K1, int act1, float arg1, int f32_1, int acc1,
                                 int M, void* stream) {
   if (M <= 0 || M > 16) return -1;
   SkinnyArgs a = {};
   a.M = M;
-  int rc = skinny_problem(a.p[0], x0, ldx0, w0, ldw0, y0, ldy0, N0, K0, act0, arg0, f32_0, acc0);
+  int rc = skinny_problem(a.p[0], x0, ldx0, w0, ldw0, b0, y0, ldy0, N0, K0, act0, arg0, f32_0, acc0);
   if (rc != 0) return rc;
   int count = 1;
   if (x1 != nullptr) {
-    rc = skinny_problem(a.p[1], x1, ldx1, w1, ldw1, y1, ldy1, N1, K1, act1, arg1, f32_1, acc1);
+    rc = skinny_problem(a.p[1], x1, ldx1, w1, ldw1, b1, y1, ldy1, N1, K1, act1, arg1, f32_1, acc1);
     if (rc != 0) return rc;
     count = 2;
   }

@@ -1,0 +1,157 @@
+// The minGRU recurrence over a ragged batch, element by element in fp32:
+//   z = sigmoid(zl);  c = u >= 0 ? u + 1/2 : sigmoid(u);  S <- (1 - z) S + z c;  out = S silu(g)
+// with zl, u and g the projections.  A step is S <- a S + b, which composes: (a1, b1) then (a2, b2)
+// is (a1 a2, a2 b1 + b2).  A block owns 32 channels of one entry and goes through its tokens 128 at
+// a time: 16 threads side by side hold two channels each, 16 groups of them take eight tokens each,
+// compose them, and learn the state in front of their tokens from the groups before them.
+#include "ragged.cuh"
+
+namespace cb {
+
+constexpr int MG_CH = 32, MG_SEG = 16, MG_TOK = 8, MG_BLOCK = MG_SEG * MG_TOK;
+
+struct MinGru {
+  const void* raw;        // [rows, ld]: zl at zoff, u at uoff, g at goff
+  int ld, zoff, uoff, goff;
+  float* state;           // [slots, width]
+  void* out;              // [rows, ldo]
+  int ldo, width;         // width: even
+  Entries e;
+};
+
+__device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) {
+  return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
+}
+__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(a, b);
+}
+__device__ __forceinline__ void store_pair(float* p, float a, float b) {
+  *reinterpret_cast<float2*>(p) = make_float2(a, b);
+}
+// a and b of one step
+__device__ __forceinline__ void mg_step(float zl, float u, float& a, float& b) {
+  const float ez = expf(-fabsf(zl)), r = 1.0f / (1.0f + ez);
+  const float z = zl >= 0.f ? r : ez * r;
+  a = zl >= 0.f ? ez * r : r;                            // 1 - z without cancellation
+  b = z * (u >= 0.f ? u + 0.5f : sigmoidf_(u));
+}
+template <typename T>
+__device__ __forceinline__ float mg_silu(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-x));
+  else return x / (1.0f + expf(-x));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(MG_CH / 2 * MG_SEG) mingru_kernel(const MinGru p) {
+  __shared__ float2 sa[MG_SEG][MG_CH / 2], sb[MG_SEG][MG_CH / 2];
+  __shared__ float2 carry[2][MG_CH / 2];
+  const int e = blockIdx.y, row0 = p.e.row0[e], len = p.e.len[e], slot = p.e.slot[e];
+  const int cp = threadIdx.x % (MG_CH / 2), seg = threadIdx.x / (MG_CH / 2);
+  const int ch = blockIdx.x * MG_CH + cp * 2;
+  const bool in = ch < p.width;
+  float* st = p.state + static_cast<size_t>(slot) * p.width + ch;
+  const T* raw = static_cast<const T*>(p.raw) + static_cast<size_t>(row0) * p.ld + (in ? ch : 0);
+  T* out = static_cast<T*>(p.out) + static_cast<size_t>(row0) * p.ldo + ch;
+  if (seg == 0)
+    carry[0][cp] = in && p.e.pos0[e] > 0 ? *reinterpret_cast<const float2*>(st) : make_float2(0.f, 0.f);
+  float2 z[MG_TOK], u[MG_TOK], g[MG_TOK];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < MG_TOK; ++i) {
+      const int t = t0 + seg * MG_TOK + i;
+      if (t >= len) continue;
+      const T* r = raw + static_cast<size_t>(t) * p.ld;
+      z[i] = load_pair(r + p.zoff);
+      u[i] = load_pair(r + p.uoff);
+      g[i] = load_pair(r + p.goff);
+    }
+  };
+  fetch(0);
+  int turn = 0;
+  for (int t0 = 0; t0 < len; t0 += MG_BLOCK, turn ^= 1) {
+    const int n = min(MG_TOK, len - t0 - seg * MG_TOK);  // may be <= 0
+    float2 a[MG_TOK], b[MG_TOK], ta = make_float2(1.f, 1.f), tb = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < MG_TOK; ++i) {
+      a[i] = make_float2(1.f, 1.f);
+      b[i] = make_float2(0.f, 0.f);
+      if (i < n) {
+        mg_step(z[i].x, u[i].x, a[i].x, b[i].x);
+        mg_step(z[i].y, u[i].y, a[i].y, b[i].y);
+      }
+      tb = make_float2(a[i].x * tb.x + b[i].x, a[i].y * tb.y + b[i].y);
+      ta = make_float2(ta.x * a[i].x, ta.y * a[i].y);
+    }
+    float2 act[MG_TOK];
+#pragma unroll
+    for (int i = 0; i < MG_TOK; ++i)
+      act[i] = i < n ? make_float2(mg_silu<T>(g[i].x), mg_silu<T>(g[i].y)) : make_float2(0.f, 0.f);
+    if (t0 + MG_BLOCK < len) fetch(t0 + MG_BLOCK);
+    sa[seg][cp] = ta;
+    sb[seg][cp] = tb;
+    __syncthreads();
+    float2 s = carry[turn][cp];
+    for (int k = 0; k < seg; ++k) {
+      const float2 ka = sa[k][cp], kb = sb[k][cp];
+      s = make_float2(ka.x * s.x + kb.x, ka.y * s.y + kb.y);
+    }
+#pragma unroll
+    for (int i = 0; i < MG_TOK; ++i) {
+      s = make_float2(a[i].x * s.x + b[i].x, a[i].y * s.y + b[i].y);
+      if (i < n && in)
+        store_pair(out + static_cast<size_t>(t0 + seg * MG_TOK + i) * p.ldo, s.x * act[i].x, s.y * act[i].y);
+    }
+    if (seg == MG_SEG - 1) carry[turn ^ 1][cp] = s;      // identity steps behind the entry's end
+    __syncthreads();
+  }
+  if (seg == 0 && in) *reinterpret_cast<float2*>(st) = carry[turn][cp];
+}
+
+// Entries of a few tokens: a thread per channel pair.
+template <typename T>
+__global__ void __launch_bounds__(128) mingru_short_kernel(const MinGru p) {
+  const int e = blockIdx.y, row0 = p.e.row0[e], len = p.e.len[e], slot = p.e.slot[e];
+  const int ch = (blockIdx.x * 128 + threadIdx.x) * 2;
+  if (ch >= p.width) return;
+  float2* st = reinterpret_cast<float2*>(p.state + static_cast<size_t>(slot) * p.width + ch);
+  float2 s = p.e.pos0[e] > 0 ? *st : make_float2(0.f, 0.f);
+  for (int t = 0; t < len; ++t) {
+    const T* r = static_cast<const T*>(p.raw) + static_cast<size_t>(row0 + t) * p.ld + ch;
+    const float2 z = load_pair(r + p.zoff), u = load_pair(r + p.uoff), g = load_pair(r + p.goff);
+    float2 a, b;
+    mg_step(z.x, u.x, a.x, b.x);
+    mg_step(z.y, u.y, a.y, b.y);
+    s = make_float2(a.x * s.x + b.x, a.y * s.y + b.y);
+    store_pair(static_cast<T*>(p.out) + static_cast<size_t>(row0 + t) * p.ldo + ch, s.x * mg_silu<T>(g.x),
+               s.y * mg_silu<T>(g.y));
+  }
+  *st = s;
+}
+
+template <typename T>
+static int launch_mingru(const MinGru& p, int entries, int longest, cudaStream_t st) {
+  if (longest <= MG_TOK)
+    mingru_short_kernel<T><<<dim3((p.width + 255) / 256, entries), 128, 0, st>>>(p);
+  else
+    mingru_kernel<T><<<dim3((p.width + MG_CH - 1) / MG_CH, entries), MG_CH / 2 * MG_SEG, 0, st>>>(p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+}  // namespace cb
+
+using namespace cb;
+
+extern "C" int cb_mingru(const void* raw, int ld, int zoff, int uoff, int goff, float* state, void* out,
+                         int ldo, int width, const int* slot, const int* row0, const int* len,
+                         const int* pos0, int entries, int longest, int f32, void* stream) {
+  if (entries <= 0 || entries > 65535 || width <= 0 || width % 2) return -1;
+  if (ld % 2 || zoff % 2 || uoff % 2 || goff % 2 || ldo % 2) return -2;
+  MinGru p;
+  p.raw = raw; p.ld = ld; p.zoff = zoff; p.uoff = uoff; p.goff = goff; p.state = state; p.out = out;
+  p.ldo = ldo; p.width = width;
+  p.e.slot = slot; p.e.row0 = row0; p.e.len = len; p.e.pos0 = pos0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return f32 ? launch_mingru<float>(p, entries, longest, st)
+             : launch_mingru<__nv_bfloat16>(p, entries, longest, st);
+}

@@ -4,6 +4,7 @@
 //                    value mixing, and the write of k and v into the cache pages
 //   shortconv_delta  q, k, v of a gated delta layer: convolution, SiLU, unit norm of q and k,
 //                    the decay of every key channel and the step size
+//   shortconv_act    any channels: convolution, bias, SiLU (in front of a state-space layer)
 // The convolution of a channel with n taps needs the n - 1 projected values before the current
 // one.  Inside a step they are earlier rows of the projection; at the start of an entry they come
 // from the slot's state, [n - 1, channels] projected values in time order.  The block that owns
@@ -628,7 +629,100 @@ __global__ void __launch_bounds__(CONV_THREADS, 6) shortconv_delta_tile_kernel(c
   }
 }
 
-// One block per row, vectors of eight bf16; the padding of a head is zero.
+struct ConvAct {
+  const void* raw;         // [rows, ld], the channels from column off on
+  int ld, off;
+  const float* taps_w;     // [taps, channels], channels a multiple of eight
+  const float* bias;       // [channels]
+  int taps, channels;
+  void* state;             // [slots, taps - 1, channels]
+  void* out;               // [rows, channels]
+  Entries e;
+  const int* tile_entry;
+  const int* tile_off;
+};
+
+// Eight channels per thread over a tile of tokens, the last TAPS values in registers (TAPS = 0: any
+// number of taps, read again for every token).
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(CONV_THREADS) shortconv_act_kernel(const ConvAct p) {
+  constexpr int V = 8, W = TAPS > 0 ? TAPS : 1;
+  const int e = p.tile_entry[blockIdx.x], off = p.tile_off[blockIdx.x];
+  const int c = (blockIdx.y * CONV_THREADS + threadIdx.x) * V;
+  if (c >= p.channels) return;
+  const int row0 = p.e.row0[e], len = p.e.len[e], slot = p.e.slot[e], n1 = p.taps - 1;
+  const bool has_state = p.e.pos0[e] > 0;
+  const T* raw = static_cast<const T*>(p.raw) + static_cast<ptrdiff_t>(row0) * p.ld + p.off + c;
+  T* st = static_cast<T*>(p.state) + static_cast<ptrdiff_t>(slot) * n1 * p.channels + c;
+  T* out = static_cast<T*>(p.out) + static_cast<ptrdiff_t>(row0) * p.channels + c;
+  auto at = [&](int o, float* f) {                       // the value at offset o, which may be negative
+    if (o >= 0) {
+      load_vec<V>(raw + static_cast<ptrdiff_t>(o) * p.ld, f);
+    } else if (has_state) {
+      load_vec<V>(st + static_cast<ptrdiff_t>(n1 + o) * p.channels, f);
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k) f[k] = 0.f;
+    }
+  };
+  float w[W][V], u[W][V], b[V];
+  load_vec<V>(p.bias + c, b);
+  if constexpr (TAPS > 0) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * p.channels + c, w[j]);
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) at(off - TAPS + j, u[j]);
+  }
+  const int t1 = min(off + CONV_TILE, len);
+#pragma unroll 4
+  for (int t = off; t < t1; ++t) {
+    float y[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) y[k] = b[k];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) u[j][k] = u[j + 1][k];
+      load_vec<V>(raw + static_cast<ptrdiff_t>(t) * p.ld, u[W - 1]);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] += u[j][k] * w[j][k];
+    } else {
+      for (int j = 0; j <= n1; ++j) {
+        at(t - n1 + j, u[0]);
+        load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * p.channels + c, w[0]);
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] += u[0][k] * w[0][k];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) y[k] = silu_act<T>(y[k]);
+    store_vec<V>(out + static_cast<ptrdiff_t>(t) * p.channels, y);
+  }
+  if (off == 0)
+    for (int j = 0; j < n1; ++j) {        // ascending: row j + len is read before it is replaced
+      float f[V];
+      at(len - n1 + j, f);
+      store_vec<V>(st + static_cast<ptrdiff_t>(j) * p.channels, f);
+    }
+}
+
+template <typename T>
+static int launch_conv_act(const ConvAct& p, int tiles, cudaStream_t st) {
+  dim3 grid(tiles, (p.channels / 8 + CONV_THREADS - 1) / CONV_THREADS);
+  switch (p.taps) {
+    case 1: shortconv_act_kernel<T, 1><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    case 2: shortconv_act_kernel<T, 2><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    case 3: shortconv_act_kernel<T, 3><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    case 4: shortconv_act_kernel<T, 4><<<grid, CONV_THREADS, 0, st>>>(p); break;
+    default: shortconv_act_kernel<T, 0><<<grid, CONV_THREADS, 0, st>>>(p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+// One block per row, vectors of eight bf16; the padding of a head is zero.  v may be absent.
 __global__ void kv_gather_kernel(const uint4* __restrict__ k_cache, const uint4* __restrict__ v_cache,
                                  int kv_heads, int kw, int vw, const int* __restrict__ page_table,
                                  int max_pages, int num_pages, const int2* __restrict__ where,
@@ -647,7 +741,7 @@ __global__ void kv_gather_kernel(const uint4* __restrict__ k_cache, const uint4*
     const int g = i / row_w, c = i % row_w;
     const size_t dst = static_cast<size_t>(blockIdx.x) * kv_heads * row_w + i;
     k_rows[dst] = c < kw ? k_cache[(cell * kv_heads + g) * kw + c] : zero;
-    v_rows[dst] = c < vw ? v_cache[(cell * kv_heads + g) * vw + c] : zero;
+    if (v_rows != nullptr) v_rows[dst] = c < vw ? v_cache[(cell * kv_heads + g) * vw + c] : zero;
   }
 }
 
@@ -795,4 +889,20 @@ extern "C" int cb_shortconv_delta(const void* raw, int ld, int koff, int voff, i
                    voff % 8 == 0;
   return f32 ? launch_conv_delta<float>(p, grid, vec, st)
              : launch_conv_delta<__nv_bfloat16>(p, grid, vec, st);
+}
+
+extern "C" int cb_shortconv_act(const void* raw, int ld, int off, const float* taps_w, const float* bias,
+                                int taps, int channels, void* state, void* out, const int* slot,
+                                const int* row0, const int* len, const int* pos0,
+                                const int* tile_entry, const int* tile_off, int tiles, int f32,
+                                void* stream) {
+  if (tiles <= 0 || taps < 1 || taps > CONV_TILE + 1 || channels <= 0 || channels % 8 || ld % 8 || off % 8)
+    return -1;
+  ConvAct p;
+  p.raw = raw; p.ld = ld; p.off = off; p.taps_w = taps_w; p.bias = bias; p.taps = taps;
+  p.channels = channels; p.state = state; p.out = out;
+  p.e.slot = slot; p.e.row0 = row0; p.e.len = len; p.e.pos0 = pos0;
+  p.tile_entry = tile_entry; p.tile_off = tile_off;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return f32 ? launch_conv_act<float>(p, tiles, st) : launch_conv_act<__nv_bfloat16>(p, tiles, st);
 }

@@ -16,9 +16,11 @@ import numpy as np
 import torch
 
 from ..foundation.error import ProcessingError
-from ..models.hybrid import AttentionSpec, HybridLM
+from ..models.hybrid import CACHED, AttentionSpec, HybridLM, LatentAttentionSpec
 from ..ops import gemm as G
+from ..ops import latent as L
 from ..ops import ragged as R
+from ..ops import recurrence as RC
 from ..ops.decode import PAGE
 from .engine import InferenceEngine
 from .kv_cache import PagedKVCache, SequenceState
@@ -46,11 +48,15 @@ class HybridEngine(InferenceEngine):
         self.use_graph = (model.device.type == "cuda") if use_graph is None else use_graph
         self._graphs: Dict[int, tuple] = {}
         self._tiles = model.device.type == "cuda" and model.dtype == torch.bfloat16
-        mixers = [self.cfg.layers[l].mixer for l in self.cfg.attention_layers()]
-        self._plans = [R.AttnPlan(a.chunk, self._pieces(a)) for a in mixers]
+        self._runs = self.cfg.runs()
+        self._plans = [self._plan(layer.mixer) for layer in self.cfg.layers
+                       if isinstance(layer.mixer, CACHED)]
 
-    def _pieces(self, a: AttentionSpec) -> bool:
-        return self._tiles and R.pieces_allowed(a.dim, a.vdim, a.chunk, a.scale)
+    def _plan(self, a) -> R.AttnPlan:
+        if isinstance(a, AttentionSpec):
+            return R.AttnPlan(a.chunk, self._tiles and R.pieces_allowed(a.dim, a.vdim, a.chunk, a.scale))
+        return R.AttnPlan(None, self._tiles and L.pieces_allowed(a.dim + a.rot_dim, a.vdim, a.scale),
+                          a.window or 1 << 30)
 
     def _batch(self, entries: List[Entry], into: Optional[R.RaggedBatch] = None) -> R.RaggedBatch:
         return R.RaggedBatch(entries, self.m.device, tile_rows=self._tiles, into=into,
@@ -60,23 +66,34 @@ class HybridEngine(InferenceEngine):
     def open_slots(self, max_seqs: int, max_len: int, num_pages: Optional[int] = None
                    ) -> PagedKVCache:
         """Cache and state for ``max_seqs`` sequences of up to ``max_len`` tokens.  ``num_pages``
-        sizes the shared page pool (default: every slot can grow to ``max_len``)."""
-        cfg, m = self.cfg, self.m
+        sizes the shared page pool (default: every slot can grow to ``max_len``).  Every run of a
+        layer has a cache or state of its own."""
+        m = self.m
         per_seq = max(1, (max_len + PAGE - 1) // PAGE)
         dims = []
         self._cache_index: Dict[int, int] = {}
-        for l in cfg.attention_layers():
-            a = cfg.layers[l].mixer
-            self._cache_index[l] = len(dims)
-            dims.append((a.kv_heads, _up8(a.dim), _up8(a.vdim)))
+        for n, run in enumerate(self._runs):
+            a = m.layers[run.layer].spec.mixer
+            if isinstance(a, CACHED):
+                self._cache_index[n] = len(dims)
+                dims.append((a.kv_heads, _up8(a.dim), _up8(a.vdim)) if isinstance(a, AttentionSpec)
+                            else (1, _up8(a.latent), 0))
         self.cache = PagedKVCache(len(dims), 0, 0, num_pages or max_seqs * per_seq, max_seqs,
                                   per_seq, m.device, m.dtype, layer_dims=dims)
         self.state = SequenceState(max_seqs, m.device)
-        for l, layer in enumerate(m.layers):
+        for n, run in enumerate(self._runs):
+            layer = m.layers[run.layer]
             s = layer.spec.mixer
-            self.state.add(l, "conv", (s.conv - 1, layer.channels), m.dtype)
-            if not isinstance(s, AttentionSpec):
-                self.state.add(l, "delta", (s.heads, s.dim, s.vdim), torch.float32)
+            if hasattr(s, "conv"):
+                self.state.add(n, "conv", (s.conv - 1, layer.channels), m.dtype)
+            if s.kind == "channel_delta":
+                self.state.add(n, "delta", (s.heads, s.dim, s.vdim), torch.float32)
+            elif s.kind == "mamba2":
+                self.state.add(n, "ssd", (s.heads, s.state, (s.vdim + 3) // 4 * 4), torch.float32)
+            elif s.kind == "mingru":
+                self.state.add(n, "gru", (_up8(s.width),), torch.float32)
+            if layer.shift is not None:
+                self.state.add(n, "before", (self.cfg.width_padded,), torch.float32)
         self._graphs.clear()
         return self.cache
 
@@ -98,23 +115,23 @@ class HybridEngine(InferenceEngine):
         G.linear_pair((h1, layer.w_in, raw, "none", None, False), up)
         return raw, cat
 
-    def _attention(self, l: int, layer, raw: torch.Tensor, cat: torch.Tensor, b: R.RaggedBatch,
+    def _attention(self, n: int, layer, raw: torch.Tensor, cat: torch.Tensor, b: R.RaggedBatch,
                    rope: dict, v_first: Optional[torch.Tensor], max_ctx: int):
-        s, c, i = layer.spec.mixer, self.cache, self._cache_index[l]
+        s, c, i = layer.spec.mixer, self.cache, self._cache_index[n]
         first = s.v_mix and v_first is None
         if first:
             v_first = torch.empty((b.T, s.kv_heads * s.vdim), dtype=raw.dtype, device=raw.device)
         q = k_rows = v_rows = None
-        plan = R.AttnPlan(s.chunk, self._pieces(s))
-        n = b.kv_rows(plan)
-        if n:       # head sizes the kernel does not have are padded with zeros
+        plan = self._plan(s)
+        key_rows = b.kv_rows(plan)
+        if key_rows:       # head sizes the kernel does not have are padded with zeros
             P = R.row_head(s.dim, s.vdim)
             new = torch.empty if s.dim == s.vdim == P else torch.zeros
-            k_rows, v_rows = (new((n, s.kv_heads, P), dtype=raw.dtype, device=raw.device)
+            k_rows, v_rows = (new((key_rows, s.kv_heads, P), dtype=raw.dtype, device=raw.device)
                               for _ in range(2))
             q = new((b.T, s.heads, P), dtype=raw.dtype, device=raw.device)
         q = R.shortconv_attn(
-            raw, layer.seg["k"], layer.seg["v"], layer.conv, self.state[l, "conv"], s.heads,
+            raw, layer.seg["k"], layer.seg["v"], layer.conv, self.state[n, "conv"], s.heads,
             s.kv_heads, s.dim, s.vdim, b, rope.get(layer.rope_key), c.k[i], c.v[i], c.page_table,
             v_first=v_first if s.v_mix else None, mix=layer.mix if s.v_mix and not first else None,
             write_first=first, k_rows=k_rows, v_rows=v_rows, q=q)
@@ -124,7 +141,7 @@ class HybridEngine(InferenceEngine):
                            k_rows=k_rows, v_rows=v_rows, plan=plan)
         return v_first
 
-    def _delta(self, l: int, layer, raw: torch.Tensor, cat: torch.Tensor, b: R.RaggedBatch) -> None:
+    def _delta(self, n: int, layer, raw: torch.Tensor, cat: torch.Tensor, b: R.RaggedBatch) -> None:
         s, m, seg = layer.spec.mixer, self.m, layer.seg
         T = raw.shape[0]
         a = torch.empty((T, layer.w_a2.shape[0]), dtype=torch.float32, device=m.device)
@@ -133,36 +150,138 @@ class HybridEngine(InferenceEngine):
         G.linear_pair((a1[:, :layer.w_a2.shape[1]], layer.w_a2, a, "none", None, False),
                       (g1[:, :layer.w_g2.shape[1]], layer.w_g2, gate, "none", None, False))
         qkvg = R.shortconv_delta(raw, seg["k"], seg["v"], seg["b"], layer.conv,
-                                 self.state[l, "conv"], s.heads, s.kv_heads, s.dim, s.vdim, b, a,
+                                 self.state[n, "conv"], s.heads, s.kv_heads, s.dim, s.vdim, b, a,
                                  layer.A_log, layer.dt_bias)
-        o = R.delta_scan(*qkvg, self.state[l, "delta"], b)
+        o = R.delta_scan(*qkvg, self.state[n, "delta"], b)
         R.gated_head_norm(o, gate, layer.head_norm, self.cfg.norm_eps, cat[:, :layer.out_dim])
+
+    # the mixers of a sequential block fill ``out``, the columns in front of their output projection
+    def _latent(self, n: int, layer, raw: torch.Tensor, out: torch.Tensor, b: R.RaggedBatch,
+                rope: dict, max_ctx: int) -> None:
+        s, m, seg = layer.spec.mixer, self.m, layer.seg
+        cache, table = self.cache.k[self._cache_index[n]], self.cache.page_table
+        plan, H = self._plan(s), s.heads
+        P, row_p = layer.w_kv.shape[2], cache.shape[-1]
+        pieces = b.plans[plan][1]
+        lat = None
+        if pieces:
+            lat = torch.empty((b.kv_rows(plan), row_p), dtype=raw.dtype, device=raw.device)
+        q = L.latent_prep(raw, seg["dkv"], H, s.dim, s.rot_dim, s.kv_rank, layer.latent_norm,
+                          self.cfg.norm_eps, rope[layer.rope_key], P, b, cache, table, rows_out=lat)
+        gate = raw[:, seg["g"]:]
+        if pieces:
+            extra, where = b.plan(plan)[3], b.plan(plan)[5]
+            if extra:
+                L.gather_rows(cache, table, where, extra, lat[b.T:])
+            kv = torch.empty((lat.shape[0], 2 * H * P), dtype=raw.dtype, device=raw.device)
+            G.linear(lat, layer.w_kv.view(2 * H * P, row_p), kv)
+            L.piece_attention(q, kv, b, plan, s.vdim, s.scale, gate, out)
+        rows = b.rows if pieces or not b.n_big else b.every_row
+        if rows.shape[0]:
+            ql = torch.empty((rows.shape[0], H, row_p), dtype=raw.dtype, device=raw.device)
+            L.linear_heads(q, layer.w_absorb, ql.view(-1, H * row_p), row_p, x_rows=rows)
+            o = L.latent_attention(ql, cache, table, b, rows, s.kv_rank, s.rot_dim, s.scale, s.window,
+                                   max_ctx)
+            L.linear_heads(o, layer.w_value[:, :, :o.shape[2]], out, s.vdim, y_rows=rows, gate=gate)
+
+    def _mamba2(self, n: int, layer, raw: torch.Tensor, out: torch.Tensor, b: R.RaggedBatch) -> None:
+        s, seg = layer.spec.mixer, layer.seg
+        u = RC.shortconv_act(raw, seg["x"], layer.conv, layer.conv_b, self.state[n, "conv"], b)
+        y = torch.empty((b.T, _up8(s.out_dim)), dtype=raw.dtype, device=raw.device)
+        RC.ssd_scan(u, layer.boff, layer.coff, raw[:, seg["dt"]:], layer.dt_bias, layer.A_log, layer.D,
+                    self.state[n, "ssd"], s.groups, s.vdim, b, y)
+        RC.gated_group_norm(y, raw[:, seg["z"]:], layer.out_norm, s.norm_groups, self.cfg.norm_eps, out)
+
+    def _mingru(self, n: int, layer, raw: torch.Tensor, out: torch.Tensor, b: R.RaggedBatch) -> None:
+        seg = layer.seg
+        RC.mingru_scan(raw, seg["z"], seg["x"], seg["g"], self.state[n, "gru"], b, out)
+
+    def _product(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        """``x @ w^T`` on its way into the residual stream: fp32 where that costs nothing or the
+        contraction has to be cut to occupy the SMs, else in the working type."""
+        M, N = x.shape[0], w.shape[0]
+        if not x.is_cuda or x.dtype == torch.float32 or M <= G.SKINNY_MAX:
+            return G.linear(x, w, torch.empty((M, N), dtype=torch.float32, device=x.device))
+        if ((M + 127) // 128) * ((N + 127) // 128) <= 74:
+            return G.linear(x, w, torch.zeros((M, N), dtype=torch.float32, device=x.device),
+                            accumulate=True)
+        return G.linear(x, w, torch.empty((M, N), dtype=x.dtype, device=x.device))
 
     def _forward(self, b: R.RaggedBatch, max_ctx: int, layer_out: Optional[list] = None
                  ) -> Optional[torch.Tensor]:
         """All layers over the batch; logits ``[wanted, vocab_padded]`` (fp32) of the wanted rows,
         None when there are none.  ``layer_out`` collects the residual stream after every layer."""
         m, cfg = self.m, self.cfg
-        W, eps = cfg.hidden_dim, cfg.norm_eps
-        x = torch.empty((b.T, cfg.width_padded), dtype=torch.float32, device=m.device)
-        R.embed_norm(b.tokens, m.embed, m.embed_norm, W, eps, x)
         rope = {k: R.rope_table(b.pos, f) for k, f in m.inv_freq.items()}
+        x = torch.empty((b.T, cfg.width_padded), dtype=torch.float32, device=m.device)
+        R.embed_norm(b.tokens, m.embed, m.embed_norm, cfg.hidden_dim, cfg.norm_eps, x)
+        blocks = self._parallel if cfg.design.parallel else self._sequential
+        xf = blocks(x, b, rope, max_ctx, layer_out)
+        if xf is None:
+            return None
+        logits = torch.empty((b.n_want, cfg.vocab_padded), dtype=torch.float32, device=m.device)
+        return G.linear(xf, m.head, logits, softcap=cfg.logit_softcap)
+
+    def _parallel(self, x: torch.Tensor, b: R.RaggedBatch, rope: dict, max_ctx: int,
+                  layer_out: Optional[list]) -> Optional[torch.Tensor]:
+        """Blocks whose mixer and feed-forward read the same stream."""
+        m, W, eps = self.m, self.cfg.hidden_dim, self.cfg.norm_eps
         v_first = None
-        for l, layer in enumerate(m.layers):
+        for n, run in enumerate(self._runs):
+            layer = m.layers[run.layer]
             h1, h2 = R.rms_rows(x, layer.norm1, W, eps, m.dtype, w2=layer.norm2)
             raw, cat = self._mixer_in(layer, h1, h2)
             if isinstance(layer.spec.mixer, AttentionSpec):
-                v_first = self._attention(l, layer, raw, cat, b, rope, v_first, max_ctx)
+                v_first = self._attention(n, layer, raw, cat, b, rope, v_first, max_ctx)
             else:
-                self._delta(l, layer, raw, cat, b)
+                self._delta(n, layer, raw, cat, b)
             G.linear(cat, layer.w_out, x, accumulate=True)
             if layer_out is not None:
                 layer_out.append(x[:, :W].clone())
         if not b.n_want:
             return None
-        xf, _ = R.rms_rows(x, m.final_norm, W, eps, m.dtype, rows=b.want)
-        logits = torch.empty((b.n_want, cfg.vocab_padded), dtype=torch.float32, device=m.device)
-        return G.linear(xf, m.head, logits, softcap=cfg.logit_softcap)
+        return R.rms_rows(x, m.final_gain, W, eps, m.dtype, rows=b.want)[0]
+
+    def _sequential(self, x: torch.Tensor, b: R.RaggedBatch, rope: dict, max_ctx: int,
+                    layer_out: Optional[list]) -> Optional[torch.Tensor]:
+        """Blocks of one sublayer after the other, norms before and after each.  A sublayer's result
+        stays pending (``add``) until the pass in front of the next one."""
+        m, cfg = self.m, self.cfg
+        W, wp, eps, dt = cfg.hidden_dim, cfg.width_padded, cfg.norm_eps, m.dtype
+        add: dict = {}
+        both = None
+        if cfg.loop is not None:           # operand [x | x0] of the product in front of every pass
+            both = torch.empty((b.T, 2 * wp), dtype=dt, device=m.device)
+            R.add_norm(x, W, eps, dt, casts=[both[:, wp:]])
+        for n, run in enumerate(self._runs):
+            layer = m.layers[run.layer]
+            if run.starts is not None:
+                R.add_norm(x, W, eps, dt, casts=[both[:, :wp]], keep=False, **add)
+                x, add = None, dict(y=self._product(both, m.loop_in), bias=m.loop_step[run.starts])
+            shift = {} if layer.shift is None else dict(shift=layer.shift, before=self.state[n, "before"],
+                                                        batch=b)
+            x, h = R.add_norm(x, W, eps, dt, gain=layer.norm1, **shift, **add)
+            raw = torch.empty((b.T, layer.w_in.shape[0]), dtype=dt, device=m.device)
+            G.linear(h, layer.w_in, raw, bias=layer.b_in)
+            out = torch.empty((b.T, layer.act_off), dtype=dt, device=m.device)
+            if layer.out_dim != layer.act_off:
+                out[:, layer.out_dim:].zero_()
+            if isinstance(layer.spec.mixer, LatentAttentionSpec):
+                self._latent(n, layer, raw, out, b, rope, max_ctx)
+            else:
+                {"mamba2": self._mamba2, "mingru": self._mingru}[layer.spec.mixer.kind](n, layer, raw, out, b)
+            add = dict(y=self._product(out, layer.w_out), post=layer.norm1b)
+            if layer.w_up is not None:
+                x, h = R.add_norm(x, W, eps, dt, gain=layer.norm2, **add)
+                act = torch.empty((b.T, layer.ff_padded), dtype=dt, device=m.device)
+                G.linear(h, layer.w_up, act, epi=cfg.design.act, bias=layer.b_up)
+                add = dict(y=self._product(act, layer.w_down), bias=layer.b_down, post=layer.norm2b)
+            if layer_out is not None:
+                x, add = R.add_norm(x, W, eps, dt, **add)[0], {}
+                layer_out.append(x[:, :W].clone())
+        if not b.n_want:
+            return None
+        return R.add_norm(x, W, eps, dt, gain=m.final_gain, rows=b.want, **add)[1]
 
     def step(self, entries: List[Entry], layer_out: Optional[list] = None
              ) -> Optional[torch.Tensor]:

@@ -5,27 +5,73 @@ recurrence, with its own sizes and constants) and a feed-forward or none.  A
 :class:`HybridLM` holds the weights the way the serving step wants them; the step itself, with the
 cache and the recurrent state, is :class:`coeus_b200.infer.hybrid_engine.HybridEngine`.
 
-The design served this way is Sapasun: a parallel block (mixer and feed-forward read the same
-residual stream through two norms), chunked attention with short convolutions, sinks, value mixing
-and head gates, and a gated delta rule with per-channel decay.
+What a design fixes for all its models is a :class:`Design`; the mixers are open to every design:
+
+* Sapasun: a parallel block (mixer and feed-forward read the same residual stream through two
+  norms), chunked attention with short convolutions, sinks, value mixing and head gates, and a
+  gated delta rule with per-channel decay.
+* Bananex: norms before and after each sublayer, a token shift in front of every mixer, a run of
+  layers that is looped with the embedding fed in again, and latent attention under a sliding
+  window, Mamba-2 and minGRU layers.
 """
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Mapping, Optional, Tuple, Union
+from typing import Any, ClassVar, Dict, List, Mapping, NamedTuple, Optional, Tuple, Union
 
 import torch
 
 from ..foundation.error import ConfigError, ProcessingError
 
-ARCHITECTURES = ("Sapasun",)
 MAX_HEAD_DIM = 256           # the attention and recurrence kernels' limit per head
+MAX_LATENT = 640             # and per cached latent row
 MAX_TAPS = 17                # and of the convolution kernels
-DEFAULT_MAX_SEQ_LEN = 8192   # serving default; the design itself has no length limit
+DEFAULT_MAX_SEQ_LEN = 8192   # serving default; the designs themselves have no length limit
+
+Shapes = Dict[str, Tuple[int, ...]]
+
+
+@dataclass(frozen=True)
+class Design:
+    """The constants of a design."""
+
+    name: str
+    mixers: Tuple[str, ...]
+    parallel: bool           # mixer and feed-forward side by side on one stream, else one by one
+    post_norms: bool         # sublayer results are normalised before they are added
+    scalar_norms: bool       # the gain of a norm of the stream is one number
+    embed_norm: bool
+    token_shift: bool
+    act: str                 # of the feed-forward
+    mlp_bias: bool
+
+
+DESIGNS = {d.name: d for d in (
+    Design("Sapasun", ("attention", "channel_delta"), parallel=True, post_norms=False,
+           scalar_norms=False, embed_norm=True, token_shift=False, act="relu2", mlp_bias=False),
+    Design("Bananex", ("latent_attention", "mamba2", "mingru"), parallel=False, post_norms=True,
+           scalar_norms=True, embed_norm=False, token_shift=True, act="gelu_erf", mlp_bias=True),
+)}
+ARCHITECTURES = tuple(DESIGNS)
+
+
+def _refuse(where: str, value, why: str) -> None:
+    raise ConfigError.invalid(where, value, why)
+
+
+def _heads_ok(where: str, *dims: int) -> None:
+    if not all(1 <= d <= MAX_HEAD_DIM for d in dims):
+        _refuse(where, "/".join(map(str, dims)), f"Head sizes must lie in 1..{MAX_HEAD_DIM}")
+
+
+def _taps_ok(where: str, taps: int) -> None:
+    if not 1 <= taps <= MAX_TAPS:
+        _refuse(where, taps, f"A convolution has 1 to {MAX_TAPS} taps")
 
 
 @dataclass(frozen=True)
 class AttentionSpec:
+    kind: ClassVar[str] = "attention"
     heads: int
     kv_heads: int
     dim: int                 # per-head query/key size
@@ -37,9 +83,53 @@ class AttentionSpec:
     rot_base: float
     v_mix: bool
 
+    @classmethod
+    def read(cls, m: Mapping[str, Any], shapes: Mapping[str, Any], p: str) -> "AttentionSpec":
+        rot, mask = m.get("rot"), m.get("mask")
+        return cls(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                   vdim=int(m["vdim"]), conv=int(m["conv"]), scale=float(m["scale"]),
+                   chunk=int(mask["size"]) if mask else None,
+                   rot_dims=int(rot["dims"]) if rot else 0,
+                   rot_base=float(rot["base"]) if rot else 1.0, v_mix=bool(m.get("v_mix", False)))
+
+    def to_json(self) -> Dict[str, Any]:
+        out: Dict[str, Any] = dict(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim,
+                                   vdim=self.vdim, conv=self.conv, scale=self.scale, v_mix=self.v_mix)
+        if self.chunk is not None:
+            out["mask"] = {"size": self.chunk}
+        if self.rot_dims:
+            out["rot"] = {"base": self.rot_base, "dims": self.rot_dims}
+        return out
+
+    def check(self, where: str) -> None:
+        if self.kv_heads < 1 or self.heads < 1 or self.heads % self.kv_heads:
+            _refuse(where, f"{self.heads}/{self.kv_heads}",
+                    "Key/value heads must divide the number of heads")
+        _heads_ok(where, self.dim, self.vdim)
+        _taps_ok(where, self.conv)
+        if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim:
+            _refuse(where, self.rot_dims, "Rotated dimensions must be even and fit the head")
+        if self.chunk is not None and self.chunk < 1:
+            _refuse(where, self.chunk, "A chunk has at least one position")
+
+    def tensors(self, W: int) -> Shapes:
+        rows = {"q": self.heads * self.dim, "k": self.kv_heads * self.dim,
+                "v": self.kv_heads * self.vdim}
+        out: Shapes = {"sink": (self.heads,), "g": (self.heads, W)}
+        if self.v_mix:
+            out["vmix"] = ()
+        for n, r in rows.items():
+            out[n], out[n + ".conv"] = (r, W), (r, self.conv)
+        return out
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
 
 @dataclass(frozen=True)
 class ChannelDeltaSpec:
+    kind: ClassVar[str] = "channel_delta"
     heads: int               # value heads
     kv_heads: int            # query/key heads
     dim: int
@@ -48,17 +138,191 @@ class ChannelDeltaSpec:
     decay_rank: int          # width between the two factors of the decay projection
     gate_rank: int           # and of the output-gate projection
 
+    @classmethod
+    def read(cls, m: Mapping[str, Any], shapes: Mapping[str, Any], p: str) -> "ChannelDeltaSpec":
+        return cls(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                   vdim=int(m["vdim"]), conv=int(m["conv"]), decay_rank=_rank(shapes, p + "a1"),
+                   gate_rank=_rank(shapes, p + "g1"))
+
+    def to_json(self) -> Dict[str, Any]:
+        return dict(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim,
+                    conv=self.conv)
+
+    def check(self, where: str) -> None:
+        if self.kv_heads < 1 or self.heads < 1 or self.heads % self.kv_heads:
+            _refuse(where, f"{self.heads}/{self.kv_heads}",
+                    "Key/value heads must divide the number of heads")
+        _heads_ok(where, self.dim, self.vdim)
+        _taps_ok(where, self.conv)
+
+    def tensors(self, W: int) -> Shapes:
+        H, qk, v = self.heads, self.kv_heads * self.dim, self.heads * self.vdim
+        out: Shapes = {"b": (H, W), "A_log": (H,), "norm": (self.vdim,), "a1": (self.decay_rank, W),
+                       "a2": (H * self.dim, self.decay_rank), "dt_bias": (H * self.dim,),
+                       "g1": (self.gate_rank, W), "g2": (v, self.gate_rank)}
+        for n, r in (("q", qk), ("k", qk), ("v", v)):
+            out[n], out[n + ".conv"] = (r, W), (r, self.conv)
+        return out
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    kind: ClassVar[str] = "latent_attention"
+    heads: int
+    dim: int                 # unrotated query/key size per head
+    rot_dim: int             # rotated query/key size per head; the key's is shared by all heads
+    vdim: int
+    kv_rank: int             # numbers per token that keys and values are made from
+    scale: float
+    window: Optional[int]    # a position sees itself and window - 1 before it
+    rot_base: float
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any], shapes: Mapping[str, Any], p: str) -> "LatentAttentionSpec":
+        rot, mask = m.get("rot"), m.get("mask")
+        if rot and int(rot.get("dims", m["rot_dim"])) != int(m["rot_dim"]):
+            _refuse(p + "rot", rot["dims"], "The rotated part is rotated as a whole")
+        return cls(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]),
+                   vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
+                   window=int(mask["size"]) if mask else None,
+                   rot_base=float(rot["base"]) if rot else 1.0)
+
+    def to_json(self) -> Dict[str, Any]:
+        out: Dict[str, Any] = dict(heads=self.heads, dim=self.dim, rot_dim=self.rot_dim,
+                                   vdim=self.vdim, kv_rank=self.kv_rank, scale=self.scale,
+                                   rot={"base": self.rot_base, "dims": self.rot_dim})
+        if self.window is not None:
+            out["mask"] = {"size": self.window}
+        return out
+
+    def check(self, where: str) -> None:
+        if self.heads < 1:
+            _refuse(where, self.heads, "Attention needs a head")
+        _heads_ok(where, self.dim + self.rot_dim, self.dim, self.vdim)
+        if self.rot_dim % 2 or self.rot_dim < 2:
+            _refuse(where, self.rot_dim, "Rotated dimensions must be even")
+        if self.kv_rank < 1 or self.latent > MAX_LATENT:
+            _refuse(where, self.kv_rank, f"A cached row holds 1 to {MAX_LATENT} numbers")
+        if self.window is not None and self.window < 1:
+            _refuse(where, self.window, "A window has at least one position")
+
+    def tensors(self, W: int) -> Shapes:
+        H, r = self.heads, self.kv_rank
+        return {"q": (H * (self.dim + self.rot_dim), W), "dkv": (r + self.rot_dim, W), "dkv.norm": (r,),
+                "uk": (H * self.dim, r), "uv": (H * self.vdim, r), "g": (H * self.vdim, W)}
+
+    @property
+    def latent(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class Mamba2Spec:
+    kind: ClassVar[str] = "mamba2"
+    heads: int
+    vdim: int
+    state: int
+    groups: int              # of heads that share B and C
+    conv: int
+    norm_groups: int         # equal parts of the output norm
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any], shapes: Mapping[str, Any], p: str) -> "Mamba2Spec":
+        return cls(**{k: int(m[k]) for k in ("heads", "vdim", "state", "groups", "conv", "norm_groups")})
+
+    def to_json(self) -> Dict[str, Any]:
+        return dict(heads=self.heads, vdim=self.vdim, state=self.state, groups=self.groups,
+                    conv=self.conv, norm_groups=self.norm_groups)
+
+    def check(self, where: str) -> None:
+        if self.heads < 1 or self.groups < 1 or self.heads % self.groups:
+            _refuse(where, f"{self.heads}/{self.groups}", "Groups must divide the number of heads")
+        if self.norm_groups < 1 or self.out_dim % self.norm_groups:
+            _refuse(where, self.norm_groups, "The parts of the output norm must be equal")
+        if self.vdim < 1:
+            _refuse(where, self.vdim, "Heads have at least one column")
+        _heads_ok(where, self.state)
+        _taps_ok(where, self.conv)
+
+    @property
+    def channels(self) -> int:
+        return self.out_dim + 2 * self.groups * self.state
+
+    def tensors(self, W: int) -> Shapes:
+        H, c = self.heads, self.channels
+        return {"in": (self.out_dim + c + H, W), "conv": (c, self.conv), "conv.b": (c,),
+                "dt_bias": (H,), "A_log": (H,), "D": (H,), "norm": (self.out_dim,)}
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class MinGruSpec:
+    kind: ClassVar[str] = "mingru"
+    width: int
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any], shapes: Mapping[str, Any], p: str) -> "MinGruSpec":
+        return cls(width=int(m["width"]))
+
+    def to_json(self) -> Dict[str, Any]:
+        return dict(width=self.width)
+
+    def check(self, where: str) -> None:
+        if self.width < 1:
+            _refuse(where, self.width, "A recurrence has at least one channel")
+
+    def tensors(self, W: int) -> Shapes:
+        n = self.width
+        return {"z": (n, W), "z.b": (n,), "x": (n, W), "x.b": (n,), "g": (n, W)}
+
+    @property
+    def out_dim(self) -> int:
+        return self.width
+
+
+MixerSpec = Union[AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, Mamba2Spec, MinGruSpec]
+MIXERS = {c.kind: c for c in (AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, Mamba2Spec,
+                              MinGruSpec)}
+CACHED = (AttentionSpec, LatentAttentionSpec)    # mixers that look back through the paged cache
+
 
 @dataclass(frozen=True)
 class MlpSpec:
     ff: int
-    kind: str = "dense"      # down(relu(up)^2)
+    kind: str = "dense"      # down(act(up))
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, ChannelDeltaSpec]
+    mixer: MixerSpec
     mlp: Optional[MlpSpec]
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights."""
+
+    start: int
+    stop: int
+    times: int
+
+
+class Run(NamedTuple):
+    """One run of a layer; every run has its own cache or state."""
+
+    layer: int
+    starts: Optional[int]    # the number of the pass this run begins, if it begins one
 
 
 @dataclass(frozen=True)
@@ -67,10 +331,16 @@ class HybridConfig:
     hidden_dim: int
     layers: Tuple[LayerSpec, ...]
     norm_eps: float
-    logit_softcap: Optional[float]
+    logit_softcap: Optional[float] = None
     architecture: str = "Sapasun"
     max_seq_len: int = DEFAULT_MAX_SEQ_LEN
+    logit_scale: float = 1.0
+    loop: Optional[LoopSpec] = None
     pos: str = field(default="rope", init=False)   # positions need no table of trained rows
+
+    @property
+    def design(self) -> Design:
+        return DESIGNS[self.architecture]
 
     @property
     def num_layers(self) -> int:
@@ -84,43 +354,38 @@ class HybridConfig:
     def vocab_padded(self) -> int:
         return _up8(self.vocab_size)
 
-    def attention_layers(self) -> List[int]:
-        return [i for i, l in enumerate(self.layers) if isinstance(l.mixer, AttentionSpec)]
-
-    def first_v_mix(self) -> Optional[int]:
-        return next((i for i in self.attention_layers() if self.layers[i].mixer.v_mix), None)
+    def runs(self) -> List[Run]:
+        """The layers in the order they run."""
+        a, b, n = (self.loop.start, self.loop.stop, self.loop.times) if self.loop else (0, 0, 0)
+        return [Run(i, None) for i in range(a)] + \
+            [Run(i, t if i == a else None) for t in range(n) for i in range(a, b)] + \
+            [Run(i, None) for i in range(b, self.num_layers)]
 
     def validate(self) -> None:
+        if self.architecture not in DESIGNS:
+            _refuse("architecture", self.architecture, f"Known designs: {', '.join(DESIGNS)}")
         if self.vocab_size < 1 or self.hidden_dim < 1 or not self.layers:
-            raise ConfigError.invalid("layers", self.num_layers,
-                                      "A model needs a vocabulary, a width and layers")
+            _refuse("layers", self.num_layers, "A model needs a vocabulary, a width and layers")
         mixing = None
         for i, layer in enumerate(self.layers):
             m = layer.mixer
             where = f"layers[{i}].mixer"
-            if m.kv_heads < 1 or m.heads < 1 or m.heads % m.kv_heads:
-                raise ConfigError.invalid(where, f"{m.heads}/{m.kv_heads}",
-                                          "Key/value heads must divide the number of heads")
-            if not (1 <= m.dim <= MAX_HEAD_DIM and 1 <= m.vdim <= MAX_HEAD_DIM):
-                raise ConfigError.invalid(where, f"{m.dim}/{m.vdim}",
-                                          f"Head sizes must lie in 1..{MAX_HEAD_DIM}")
-            if not 1 <= m.conv <= MAX_TAPS:
-                raise ConfigError.invalid(where, m.conv, f"A convolution has 1 to {MAX_TAPS} taps")
-            if isinstance(m, AttentionSpec):
-                if m.rot_dims % 2 or not 0 <= m.rot_dims <= m.dim:
-                    raise ConfigError.invalid(where, m.rot_dims,
-                                              "Rotated dimensions must be even and fit the head")
-                if m.chunk is not None and m.chunk < 1:
-                    raise ConfigError.invalid(where, m.chunk, "A chunk has at least one position")
-                if m.v_mix:
-                    size = m.kv_heads * m.vdim
-                    if mixing not in (None, size):
-                        raise ConfigError.invalid(where, size,
-                                                  "Layers that mix values must agree in their size")
-                    mixing = size
-            if layer.mlp is not None and layer.mlp.kind != "dense":
-                raise ConfigError.invalid(f"layers[{i}].mlp", layer.mlp.kind,
-                                          "Feed-forward kind must be 'dense'")
+            if m.kind not in self.design.mixers:
+                _refuse(where, m.kind, f"{self.architecture} has {', '.join(self.design.mixers)}")
+            m.check(where)
+            if getattr(m, "v_mix", False):
+                size = m.kv_heads * m.vdim
+                if mixing not in (None, size):
+                    _refuse(where, size, "Layers that mix values must agree in their size")
+                mixing = size
+            if layer.mlp is not None and (layer.mlp.kind != "dense" or layer.mlp.ff < 1):
+                _refuse(f"layers[{i}].mlp", layer.mlp.kind, "Feed-forward kind must be 'dense'")
+        if self.loop is not None:
+            lo = self.loop
+            if self.design.parallel:
+                _refuse("loop", lo, f"{self.architecture} has no loop")
+            if not 0 <= lo.start < lo.stop <= self.num_layers or lo.times < 1:
+                _refuse("loop", f"{lo.start}..{lo.stop} x {lo.times}", "The loop must be a run of layers")
 
     def to_dict(self) -> Dict[str, Any]:
         return config_to_json(self)
@@ -141,85 +406,63 @@ def config_from_json(config: Mapping[str, Any], shapes: Mapping[str, Any]) -> Hy
     sizes the file does not name (the inner widths of the factored projections)."""
     layers = []
     for i, entry in enumerate(config["layers"]):
-        m, p = entry["mixer"], f"l{i}.mix."
-        if entry["type"] == "attention":
-            rot, mask = m.get("rot"), m.get("mask")
-            mixer = AttentionSpec(
-                heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
-                vdim=int(m["vdim"]), conv=int(m["conv"]), scale=float(m["scale"]),
-                chunk=int(mask["size"]) if mask else None,
-                rot_dims=int(rot["dims"]) if rot else 0,
-                rot_base=float(rot["base"]) if rot else 1.0, v_mix=bool(m.get("v_mix", False)))
-        elif entry["type"] == "channel_delta":
-            mixer = ChannelDeltaSpec(
-                heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
-                vdim=int(m["vdim"]), conv=int(m["conv"]), decay_rank=_rank(shapes, p + "a1"),
-                gate_rank=_rank(shapes, p + "g1"))
-        else:
-            raise ProcessingError.unsupported(f"mixer type '{entry['type']}'",
-                                              "attention and channel_delta")
+        if entry["type"] not in MIXERS:
+            raise ProcessingError.unsupported(f"mixer type '{entry['type']}'", ", ".join(MIXERS))
+        mixer = MIXERS[entry["type"]].read(entry["mixer"], shapes, f"l{i}.mix.")
         mlp = entry.get("mlp")
         layers.append(LayerSpec(mixer, None if mlp is None else
                                 MlpSpec(ff=int(mlp["ff"]), kind=str(mlp["kind"]))))
-    cap = config.get("logit_softcap")
+    cap, loop = config.get("logit_softcap"), config.get("loop")
     cfg = HybridConfig(
         vocab_size=int(config["vocab"]), hidden_dim=int(config["width"]), layers=tuple(layers),
         norm_eps=float(config["norm"]["eps"]), logit_softcap=None if cap is None else float(cap),
-        architecture=str(config.get("architecture", "Sapasun")))
+        architecture=str(config.get("architecture", "Sapasun")),
+        logit_scale=float(config.get("logit_scale", 1.0)),
+        loop=None if not loop else LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"])))
     cfg.validate()
     return cfg
 
 
 def config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
-    layers = []
-    for layer in cfg.layers:
-        m = layer.mixer
-        mixer: Dict[str, Any] = dict(heads=m.heads, kv_heads=m.kv_heads, dim=m.dim, vdim=m.vdim,
-                                     conv=m.conv)
-        if isinstance(m, AttentionSpec):
-            kind = "attention"
-            mixer.update(scale=m.scale, v_mix=m.v_mix)
-            if m.chunk is not None:
-                mixer["mask"] = {"size": m.chunk}
-            if m.rot_dims:
-                mixer["rot"] = {"base": m.rot_base, "dims": m.rot_dims}
-        else:
-            kind = "channel_delta"
-        layers.append({"type": kind, "mixer": mixer, "mlp": None if layer.mlp is None else
-                       {"kind": layer.mlp.kind, "ff": layer.mlp.ff}})
-    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_dim,
-            "norm": {"eps": cfg.norm_eps}, "logit_softcap": cfg.logit_softcap, "layers": layers}
+    layers = [{"type": layer.mixer.kind, "mixer": layer.mixer.to_json(),
+               "mlp": None if layer.mlp is None else {"kind": layer.mlp.kind, "ff": layer.mlp.ff}}
+              for layer in cfg.layers]
+    out = {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_dim,
+           "norm": {"eps": cfg.norm_eps}, "layers": layers}
+    if cfg.design.parallel:
+        out["logit_softcap"] = cfg.logit_softcap
+    else:
+        out["logit_scale"] = cfg.logit_scale
+    if cfg.loop is not None:
+        out["loop"] = {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times}
+    return out
 
 
-def tensor_shapes(cfg: HybridConfig) -> Dict[str, Tuple[int, ...]]:
+def tensor_shapes(cfg: HybridConfig) -> Shapes:
     """Every tensor of a checkpoint and its shape (linear weights ``[out, in]``)."""
-    W, V = cfg.hidden_dim, cfg.vocab_size
-    out: Dict[str, Tuple[int, ...]] = {"embed": (V, W), "embed.norm": (W,)}
+    W, V, d = cfg.hidden_dim, cfg.vocab_size, cfg.design
+    norm: Tuple[int, ...] = () if d.scalar_norms else (W,)
+    out: Shapes = {"embed": (V, W)}
+    if d.embed_norm:
+        out["embed.norm"] = norm
+    if cfg.loop is not None:
+        out.update({"loop.in": (W, 2 * W), "loop.step": (cfg.loop.times, W)})
     for i, layer in enumerate(cfg.layers):
-        m, p = layer.mixer, f"l{i}."
-        out[p + "norm1"] = (W,)
-        if layer.mlp is not None:
-            out[p + "norm2"] = (W,)
-        x = p + "mix."
-        if isinstance(m, AttentionSpec):
-            rows = {"q": m.heads * m.dim, "k": m.kv_heads * m.dim, "v": m.kv_heads * m.vdim}
-            out.update({x + "sink": (m.heads,), x + "g": (m.heads, W)})
-            if m.v_mix:
-                out[x + "vmix"] = ()
-        else:
-            rows = {"q": m.kv_heads * m.dim, "k": m.kv_heads * m.dim, "v": m.heads * m.vdim}
-            out.update({x + "b": (m.heads, W), x + "A_log": (m.heads,), x + "norm": (m.vdim,),
-                        x + "a1": (m.decay_rank, W), x + "a2": (m.heads * m.dim, m.decay_rank),
-                        x + "dt_bias": (m.heads * m.dim,), x + "g1": (m.gate_rank, W),
-                        x + "g2": (m.heads * m.vdim, m.gate_rank)})
-        for n, r in rows.items():
-            out[x + n] = (r, W)
-            out[x + n + ".conv"] = (r, m.conv)
-        out[x + "o"] = (W, m.heads * m.vdim)
+        p = f"l{i}."
+        for n in ("norm1", "norm2")[:1 if layer.mlp is None else 2]:
+            out[p + n] = norm
+            if d.post_norms:
+                out[p + n + "b"] = norm
+        if d.token_shift:
+            out[p + "shift"] = (W,)
+        out.update({f"{p}mix.{n}": s for n, s in layer.mixer.tensors(W).items()})
+        out[p + "mix.o"] = (W, layer.mixer.out_dim)
         if layer.mlp is not None:
             out[p + "mlp.up"] = (layer.mlp.ff, W)
             out[p + "mlp.down"] = (W, layer.mlp.ff)
-    out.update({"final.norm": (W,), "head": (V, W)})
+            if d.mlp_bias:
+                out.update({p + "mlp.up.b": (layer.mlp.ff,), p + "mlp.down.b": (W,)})
+    out.update({"final.norm": norm, "head": (V, W)})
     return out
 
 
@@ -239,10 +482,14 @@ def random_state(cfg: HybridConfig, seed: int = 0, device="cpu",
         elif leaf == "conv":
             t = normal(shape, 0.3)
             t[:, -1] += 1.0
-        elif leaf == "embed":
+        elif leaf in ("embed", "D"):
             t = normal(shape, 1.0)
         elif leaf in ("sink", "vmix", "A_log", "dt_bias"):
             t = normal(shape, 0.5)
+        elif leaf == "step" or (leaf == "b" and len(shape) == 1):
+            t = normal(shape, 0.2)
+        elif leaf == "shift":
+            t = torch.sigmoid(normal(shape, 1.0))
         else:
             t = normal(shape, shape[-1] ** -0.5)
         out[name] = t.to(dtype)
@@ -256,59 +503,182 @@ def _pad(t: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
 
 
 class HybridLayer:
-    """Device weights of one layer.  ``w_in`` stacks every projection of the normalised stream
-    (each segment starts at a multiple of eight rows, ``seg[name]`` is its first output column),
-    ``w_out`` puts the mixer's output projection and the feed-forward's down projection side by
-    side: both are added to the same stream, so they are one product over
-    ``[mixer output | activation]``, the activation starting at column ``act_off``."""
+    """Device weights of one layer.  ``w_in`` stacks every projection of the mixer's input (each
+    segment starts at a multiple of eight rows, ``seg[name]`` is its first output column; ``b_in``
+    the biases, where a segment has one).  In a parallel block ``w_out`` puts the mixer's output
+    projection and the feed-forward's down projection side by side: both are added to the same
+    stream, so they are one product over ``[mixer output | activation]``, the activation starting at
+    column ``act_off``.  Otherwise ``w_out`` is the mixer's output projection and ``w_down`` the
+    feed-forward's."""
 
-    def __init__(self, spec: LayerSpec, w_get, width: int, dtype: torch.dtype) -> None:
-        self.spec = spec
-        m = spec.mixer
-        attn = isinstance(m, AttentionSpec)
-        wp = _up8(width)
-
-        def mat(name):
-            return w_get(name).to(dtype)
-
-        def vec(name, pad=0):
-            t = w_get(name).float()
-            return torch.nn.functional.pad(t, (0, pad - t.numel())).contiguous() if pad \
-                else t.contiguous()
-        self.norm1 = vec("norm1", wp)
-        parts = ["q", "k", "v", "g"] if attn else ["q", "k", "v", "b", "a1", "g1"]
+    def __init__(self, spec: LayerSpec, design: Design, w_get, width: int, dtype: torch.dtype) -> None:
+        self.spec, self.dtype = spec, dtype
+        self._get = w_get
+        self.wp = _up8(width)
+        self.norm1 = self._gain("norm1", design)
+        self.norm1b = self._gain("norm1b", design) if design.post_norms else None
+        self.shift = self._vec("shift", self.wp) if design.token_shift else None
         self.seg: Dict[str, int] = {}
-        blocks, at = [], 0
-        for n in parts:
-            t = mat("mix." + n)
-            self.seg[n] = at
-            blocks.append(_pad(t, _up8(t.shape[0]), wp))
-            at += blocks[-1].shape[0]
-        self.w_in = torch.cat(blocks).contiguous()
-        # taps-major, channels q | k | v
-        self.conv = torch.cat([w_get(f"mix.{n}.conv").float() for n in "qkv"]).t().contiguous()
-        self.channels = self.conv.shape[1]
-        if attn:
-            self.sink = vec("mix.sink")
-            self.mix = vec("mix.vmix").reshape(1) if m.v_mix else None
-            half = m.rot_dims // 2
-            self.rope_key = (m.rot_base, m.rot_dims) if half else None
-        else:
-            self.A_log, self.dt_bias = vec("mix.A_log"), vec("mix.dt_bias")
-            self.head_norm = vec("mix.norm")
-            self.w_a2 = _pad(mat("mix.a2"), _up8(m.heads * m.dim), _up8(m.decay_rank))
-            self.w_g2 = _pad(mat("mix.g2"), _up8(m.heads * m.vdim), _up8(m.gate_rank))
-        self.out_dim = m.heads * m.vdim
+        {"attention": self._attention, "channel_delta": self._channel_delta,
+         "latent_attention": self._latent, "mamba2": self._mamba2,
+         "mingru": self._mingru}[spec.mixer.kind](spec.mixer)
+        self.out_dim = spec.mixer.out_dim
         self.act_off = _up8(self.out_dim)
-        outs = [_pad(mat("mix.o"), wp, self.act_off)]
-        self.norm2 = self.w_up = None
+        outs = [_pad(self._mat("mix.o"), self.wp, self.act_off)]
+        self.norm2 = self.norm2b = self.w_up = self.b_up = self.w_down = self.b_down = None
         self.ff = self.ff_padded = 0
         if spec.mlp is not None:
-            self.norm2 = vec("norm2", wp)
+            self.norm2 = self._gain("norm2", design)
+            self.norm2b = self._gain("norm2b", design) if design.post_norms else None
             self.ff, self.ff_padded = spec.mlp.ff, _up8(spec.mlp.ff)
-            self.w_up = _pad(mat("mlp.up"), self.ff_padded, wp)
-            outs.append(_pad(mat("mlp.down"), wp, self.ff_padded))
+            self.w_up = _pad(self._mat("mlp.up"), self.ff_padded, self.wp)
+            down = _pad(self._mat("mlp.down"), self.wp, self.ff_padded)
+            if design.parallel:
+                outs.append(down)
+            else:
+                self.w_down = down
+            if design.mlp_bias:
+                self.b_up = self._vec("mlp.up.b", self.ff_padded).to(dtype)
+                self.b_down = self._vec("mlp.down.b", self.wp)
         self.w_out = torch.cat(outs, 1).contiguous()
+        del self._get
+
+    def _mat(self, name: str) -> torch.Tensor:
+        return self._get(name).to(self.dtype)
+
+    def _vec(self, name: str, pad: int = 0) -> torch.Tensor:
+        t = self._get(name).float()
+        return torch.nn.functional.pad(t, (0, pad - t.numel())).contiguous() if pad else t.contiguous()
+
+    def _gain(self, name: str, design: Design) -> torch.Tensor:
+        return self._vec(name).reshape(1) if design.scalar_norms else self._vec(name, self.wp)
+
+    def _stack(self, parts: Mapping[str, torch.Tensor], biases: Optional[Mapping[str, torch.Tensor]] = None
+               ) -> None:
+        blocks, at = [], 0
+        for n, t in parts.items():
+            self.seg[n] = at
+            blocks.append(_pad(t, _up8(t.shape[0]), self.wp))
+            at += blocks[-1].shape[0]
+        self.w_in = torch.cat(blocks).contiguous()
+        self.b_in = None
+        if biases:
+            self.b_in = torch.zeros(at, dtype=self.dtype, device=self.w_in.device)
+            for n, b in biases.items():
+                self.b_in[self.seg[n]:self.seg[n] + b.numel()] = b.to(self.dtype)
+
+    def _conv_qkv(self) -> None:      # taps-major, channels q | k | v
+        self.conv = torch.cat([self._get(f"mix.{n}.conv").float() for n in "qkv"]).t().contiguous()
+        self.channels = self.conv.shape[1]
+
+    def _attention(self, m: AttentionSpec) -> None:
+        self._stack({n: self._mat("mix." + n) for n in ("q", "k", "v", "g")})
+        self._conv_qkv()
+        self.sink = self._vec("mix.sink")
+        self.mix = self._vec("mix.vmix").reshape(1) if m.v_mix else None
+        self.rope_key = (m.rot_base, m.rot_dims) if m.rot_dims else None
+
+    def _channel_delta(self, m: ChannelDeltaSpec) -> None:
+        self._stack({n: self._mat("mix." + n) for n in ("q", "k", "v", "b", "a1", "g1")})
+        self._conv_qkv()
+        self.A_log, self.dt_bias = self._vec("mix.A_log"), self._vec("mix.dt_bias")
+        self.head_norm = self._vec("mix.norm")
+        self.w_a2 = _pad(self._mat("mix.a2"), _up8(m.heads * m.dim), _up8(m.decay_rank))
+        self.w_g2 = _pad(self._mat("mix.g2"), _up8(m.heads * m.vdim), _up8(m.gate_rank))
+
+    def _latent(self, m: LatentAttentionSpec) -> None:
+        """``w_kv [2, heads, P, latent]`` makes every head's key (its rotated part copied from the
+        cached row by unit rows) and value from cached rows; ``w_absorb [heads, latent, P]`` is its
+        key part transposed, which brings a query to the cached rows instead."""
+        from ..ops.latent import head_pitch
+        self._stack({n: self._mat("mix." + n) for n in ("q", "dkv", "g")})
+        self.latent_norm = self._vec("mix.dkv.norm")
+        self.rope_key = (m.rot_base, m.rot_dim)
+        H, r, P = m.heads, m.kv_rank, head_pitch(m.dim + m.rot_dim, m.vdim)
+        w = torch.zeros((2, H, P, _up8(m.latent)), dtype=self.dtype, device=self.w_in.device)
+        w[0, :, :m.dim, :r] = self._mat("mix.uk").view(H, m.dim, r)
+        for i in range(m.rot_dim):
+            w[0, :, m.dim + i, r + i] = 1.0
+        w[1, :, :m.vdim, :r] = self._mat("mix.uv").view(H, m.vdim, r)
+        self.w_kv = w
+        self.w_absorb = w[0].transpose(1, 2).contiguous()
+        self.w_value = w[1, :, :m.vdim].contiguous()
+
+    def _mamba2(self, m: Mamba2Spec) -> None:
+        """The convolved channels are ``x | B | C``, each starting at a multiple of eight."""
+        bc = m.groups * m.state
+        sizes = dict(z=m.out_dim, x=m.out_dim, B=bc, C=bc, dt=m.heads)
+        self._stack(dict(zip(sizes, torch.split(self._mat("mix.in"), list(sizes.values())))))
+        pads = [(n, _up8(sizes[n])) for n in ("x", "B", "C")]
+        self.boff, self.coff = pads[0][1], pads[0][1] + pads[1][1]
+        self.channels = sum(p for _, p in pads)
+
+        def spread(t: torch.Tensor) -> torch.Tensor:
+            parts = torch.split(t, [sizes[n] for n, _ in pads])
+            return torch.cat([_pad(x, p, t.shape[1]) for x, (_, p) in zip(parts, pads)])
+        self.conv = spread(self._get("mix.conv").float()).t().contiguous()
+        self.conv_b = spread(self._vec("mix.conv.b")[:, None])[:, 0].contiguous()
+        self.dt_bias, self.A_log, self.D = (self._vec("mix." + n) for n in ("dt_bias", "A_log", "D"))
+        self.out_norm = self._vec("mix.norm")
+
+    def _mingru(self, m: MinGruSpec) -> None:
+        self._stack({n: self._mat("mix." + n) for n in ("z", "x", "g")},
+                    {n: self._get(f"mix.{n}.b") for n in ("z", "x")})
+
+    # ------------------------------------------------------------------ taken apart again
+    def tensors(self, width: int) -> Dict[str, torch.Tensor]:
+        """The layer's tensors under their names in a checkpoint (without the layer's prefix)."""
+        m, W = self.spec.mixer, width
+        shapes = m.tensors(W)
+        out = {"norm1": self.norm1, "mix.o": self.w_out[:W, :self.out_dim]}
+
+        def stacked(names):
+            for n in names:
+                out["mix." + n] = self.w_in[self.seg[n]:self.seg[n] + shapes[n][0], :W]
+        if isinstance(m, (AttentionSpec, ChannelDeltaSpec)):
+            c = 0
+            for n in "qkv":
+                r = shapes[n][0]
+                out[f"mix.{n}.conv"] = self.conv[:, c:c + r].t()
+                c += r
+        if isinstance(m, AttentionSpec):
+            stacked(("q", "k", "v", "g"))
+            out["mix.sink"] = self.sink
+            if self.mix is not None:
+                out["mix.vmix"] = self.mix
+        elif isinstance(m, ChannelDeltaSpec):
+            stacked(("q", "k", "v", "b", "a1", "g1"))
+            out.update({"mix.A_log": self.A_log, "mix.dt_bias": self.dt_bias, "mix.norm": self.head_norm})
+            for n, t in (("a2", self.w_a2), ("g2", self.w_g2)):
+                out["mix." + n] = t[:shapes[n][0], :shapes[n][1]]
+        elif isinstance(m, LatentAttentionSpec):
+            stacked(("q", "dkv", "g"))
+            out["mix.dkv.norm"] = self.latent_norm
+            out["mix.uk"] = self.w_kv[0, :, :m.dim, :m.kv_rank].reshape(shapes["uk"])
+            out["mix.uv"] = self.w_kv[1, :, :m.vdim, :m.kv_rank].reshape(shapes["uv"])
+        elif isinstance(m, Mamba2Spec):
+            bc = m.groups * m.state
+            sizes = dict(z=m.out_dim, x=m.out_dim, B=bc, C=bc, dt=m.heads)
+            out["mix.in"] = torch.cat([self.w_in[self.seg[n]:self.seg[n] + r, :W] for n, r in sizes.items()])
+            at = {"x": 0, "B": self.boff, "C": self.coff}
+            idx = torch.cat([torch.arange(at[n], at[n] + sizes[n]) for n in at]).to(self.conv.device)
+            out.update({"mix.conv": self.conv[:, idx].t(), "mix.conv.b": self.conv_b[idx],
+                        "mix.dt_bias": self.dt_bias, "mix.A_log": self.A_log, "mix.D": self.D,
+                        "mix.norm": self.out_norm})
+        else:
+            stacked(("z", "x", "g"))
+            for n in ("z", "x"):
+                out[f"mix.{n}.b"] = self.b_in[self.seg[n]:self.seg[n] + m.width]
+        for n in ("norm1b", "norm2", "norm2b", "shift"):
+            if getattr(self, n) is not None:
+                out[n] = getattr(self, n)
+        if self.w_up is not None:
+            out["mlp.up"] = self.w_up[:self.ff, :W]
+            out["mlp.down"] = self.w_out[:W, self.act_off:self.act_off + self.ff] \
+                if self.w_down is None else self.w_down[:W, :self.ff]
+            if self.b_up is not None:
+                out["mlp.up.b"], out["mlp.down.b"] = self.b_up[:self.ff], self.b_down[:W]
+        return out
 
 
 class HybridLM:
@@ -332,15 +702,24 @@ class HybridLM:
                 raise ProcessingError.invalid_input(
                     f"tensor '{name}' has shape {tuple(t.shape)}, expected {shapes[name]}")
             return t.to(self.device)
-        W, wp = cfg.hidden_dim, cfg.width_padded
+        W, wp, design = cfg.hidden_dim, cfg.width_padded, cfg.design
 
-        def vec(name):
-            return torch.nn.functional.pad(get(name).float(), (0, wp - W)).contiguous()
+        def gain(name):
+            t = get(name).float()
+            return t.reshape(1) if design.scalar_norms else \
+                torch.nn.functional.pad(t, (0, wp - W)).contiguous()
         self.embed = _pad(get("embed").to(self.dtype), cfg.vocab_size, wp)
-        self.embed_norm = vec("embed.norm")
-        self.layers = [HybridLayer(spec, lambda n, i=i: get(f"l{i}.{n}"), W, self.dtype)
+        self.embed_norm = gain("embed.norm") if design.embed_norm else None
+        self.loop_in = self.loop_step = None
+        if cfg.loop is not None:       # [W, 2 W] with the padding of each half behind it
+            a, b = get("loop.in").to(self.dtype).split(W, 1)
+            self.loop_in = torch.cat([_pad(a, wp, wp), _pad(b, wp, wp)], 1).contiguous()
+            self.loop_step = _pad(get("loop.step").float(), cfg.loop.times, wp)
+        self.layers = [HybridLayer(spec, design, lambda n, i=i: get(f"l{i}.{n}"), W, self.dtype)
                        for i, spec in enumerate(cfg.layers)]
-        self.final_norm = vec("final.norm")
+        self.final_norm = gain("final.norm")
+        # the logits' factor rides on the last norm's gain
+        self.final_gain = self.final_norm * cfg.logit_scale
         self.head = _pad(get("head").to(self.dtype), cfg.vocab_padded, wp)
         # rotary frequencies base^(-2i/dims), one table per distinct (base, dims)
         self.inv_freq: Dict[Tuple[float, int], torch.Tensor] = {}
@@ -358,13 +737,7 @@ class HybridLM:
         return cls(cfg, random_state(cfg, seed, device), device, dtype)
 
     def num_parameters(self) -> int:
-        n = 0
-        for shape in self._shapes.values():
-            k = 1
-            for s in shape:
-                k *= s
-            n += k
-        return n
+        return sum(_size(shape) for shape in self._shapes.values())
 
     def make_engine(self, **kw):
         from ..infer.hybrid_engine import HybridEngine
@@ -373,34 +746,26 @@ class HybridLM:
     def state_dict(self) -> Dict[str, torch.Tensor]:
         """The checkpoint's tensors, taken apart again."""
         cfg, W = self.cfg, self.cfg.hidden_dim
-        out = {"embed": self.embed[:, :W], "embed.norm": self.embed_norm[:W],
-               "final.norm": self.final_norm[:W], "head": self.head[:cfg.vocab_size, :W]}
-        for i, (layer, spec) in enumerate(zip(self.layers, cfg.layers)):
-            p, x = f"l{i}.", f"l{i}.mix."
-            out[p + "norm1"] = layer.norm1[:W]
-            c = 0
-            for n, at in layer.seg.items():
-                rows = self._shapes[x + n][0]
-                out[x + n] = layer.w_in[at:at + rows, :W]
-                if n in "qkv":
-                    out[f"{x}{n}.conv"] = layer.conv[:, c:c + rows].t()
-                    c += rows
-            if isinstance(spec.mixer, AttentionSpec):
-                out[x + "sink"] = layer.sink
-                if layer.mix is not None:
-                    out[x + "vmix"] = layer.mix.reshape(())
-            else:
-                out.update({x + "A_log": layer.A_log, x + "dt_bias": layer.dt_bias,
-                            x + "norm": layer.head_norm})
-                for n, t in (("a2", layer.w_a2), ("g2", layer.w_g2)):
-                    r, k = self._shapes[x + n]
-                    out[x + n] = t[:r, :k]
-            out[x + "o"] = layer.w_out[:W, :layer.out_dim]
-            if layer.w_up is not None:
-                out[p + "norm2"] = layer.norm2[:W]
-                out[p + "mlp.up"] = layer.w_up[:layer.ff, :W]
-                out[p + "mlp.down"] = layer.w_out[:W, layer.act_off:layer.act_off + layer.ff]
-        return {n: t.detach().cpu().contiguous().clone() for n, t in out.items()}
+        out = {"embed": self.embed[:, :W], "final.norm": self.final_norm[:W],
+               "head": self.head[:cfg.vocab_size, :W]}
+        if self.embed_norm is not None:
+            out["embed.norm"] = self.embed_norm[:W]
+        if self.loop_in is not None:
+            wp = cfg.width_padded
+            out["loop.in"] = torch.cat([self.loop_in[:W, :W], self.loop_in[:W, wp:wp + W]], 1)
+            out["loop.step"] = self.loop_step[:, :W]
+        for i, layer in enumerate(self.layers):
+            out.update({f"l{i}.{n}": t for n, t in layer.tensors(W).items()})
+        return {n: t.detach().flatten()[:_size(self._shapes[n])].reshape(self._shapes[n]).cpu()
+                .contiguous().clone() if t.dim() < 2 else t.detach().cpu().contiguous().clone()
+                for n, t in out.items()}
+
+
+def _size(shape: Tuple[int, ...]) -> int:
+    n = 1
+    for s in shape:
+        n *= s
+    return n
 
 
 def load_hybrid(state: Mapping[str, torch.Tensor], config: Mapping[str, Any], device="cuda",

@@ -18,7 +18,7 @@ import torch
 
 from . import _lib
 
-EPI = {"none": 0, "gelu": 1, "dgelu": 2, "relu2": 4}
+EPI = {"none": 0, "gelu": 1, "dgelu": 2, "relu2": 4, "gelu_erf": 6}
 _OUT_BF16, _OUT_F32, _OUT_F32_ATOMIC = 0, 1, 2
 
 
@@ -119,6 +119,8 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
             v = v * _gelu_grad_ref(aux_in.float())
         elif epi == "relu2":
             v = torch.relu(v).square()
+        elif epi == "gelu_erf":
+            v = torch.nn.functional.gelu(v)
         if dropout is not None and dropout[0] > 0:
             from .elementwise import dropout_mask
             keep = dropout_mask(M, N, dropout[0], dropout[1], v.device)
@@ -258,9 +260,11 @@ def linear_wgrad(x: torch.Tensor, dy: torch.Tensor, grad_w: torch.Tensor, *,
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "none",
-           softcap: Optional[float] = None, accumulate: bool = False) -> torch.Tensor:
-    """``out[M, N] (+)= epi(x[M, K] @ w[N, K]^T)`` for a serving step: the weight is stored
-    ``[out, in]``, rows of ``x`` and ``out`` may be strided.  bf16 operands run on the tensor cores
+           softcap: Optional[float] = None, accumulate: bool = False,
+           bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[M, N] (+)= epi(x[M, K] @ w[N, K]^T + bias)`` for a serving step: the weight is stored
+    ``[out, in]``, rows of ``x`` and ``out`` may be strided, ``bias`` has the weight's type.  bf16
+    operands run on the tensor cores
     with a bf16 or fp32 ``out``; fp32 operands are multiplied in full fp32 (``cb_linear_f32``).
     ``accumulate`` adds into an fp32 ``out`` (the residual stream); ``softcap`` maps the result
     ``z`` to ``softcap * tanh(z / softcap)`` (fp32 ``out``)."""
@@ -268,22 +272,29 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
     N = w.shape[0]
     if w.shape[1] != K or out.shape[0] != M or out.shape[1] != N:
         raise ValueError(f"linear: shapes {tuple(x.shape)} {tuple(w.shape)} {tuple(out.shape)}")
+    if bias is not None and (bias.dtype != w.dtype or bias.shape != (N,) or accumulate):
+        raise ValueError("linear: the bias needs the weight's type, one entry per output, no accumulation")
     if not x.is_cuda:
         v = x.float() @ w.float().t()
+        if bias is not None:
+            v = v + bias.float()
         if epi == "relu2":
             v = torch.relu(v).square()
+        elif epi == "gelu_erf":
+            v = torch.nn.functional.gelu(v)
         if softcap is not None:
             v = softcap * torch.tanh(v / softcap)
         return out.add_(v) if accumulate else out.copy_(v.to(out.dtype))
     if x.dtype == torch.float32:
         act = 5 if softcap is not None else EPI[epi]
         rc = _lib.serving_lib().cb_linear_f32(
-            _lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(out), out.stride(0), M, N,
-            K, act, ctypes.c_float(softcap or 0.0), int(accumulate), _lib.stream_ptr())
+            _lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(bias), _lib.ptr(out),
+            out.stride(0), M, N, K, act, ctypes.c_float(softcap or 0.0), int(accumulate),
+            _lib.stream_ptr())
         _lib.check_rc(rc, "cb_linear_f32")
         return out
     if M <= SKINNY_MAX and not (accumulate and (M > 8 or K >= 16384)):
-        return linear_pair((x, w, out, epi, softcap, accumulate))[0]
+        return linear_pair((x, w, out, epi, softcap, accumulate, bias))[0]
     out_mode = _OUT_BF16 if out.dtype == torch.bfloat16 else (
         _OUT_F32_ATOMIC if accumulate else _OUT_F32)
     # Few tiles: narrower ones spread the weights over more SMs, and a product that is added to
@@ -294,7 +305,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
         ksplit = max(1, min(16, 148 // tiles, (K + 63) // 64 // 4))
     rc = _lib.serving_lib().cb_gemm_bf16(
         _lib.ptr(x), _lib.ptr(w), _lib.ptr(out), M, N, K, x.stride(0), w.stride(0), out.stride(0),
-        0, 0, None, None, 0, None, None, 0, EPI[epi], out_mode, ctypes.c_float(1.0), ksplit, bn, _lib.ptr(_lib.status_buffer(x.device)), 0, _lib.stream_ptr())
+        0, 0, _lib.ptr(bias), None, 0, None, None, 0, EPI[epi], out_mode, ctypes.c_float(1.0), ksplit,
+        bn, _lib.ptr(_lib.status_buffer(x.device)), 0, _lib.stream_ptr())
     _lib.check_rc(rc, "cb_gemm_bf16")
     if softcap is not None:
         rc = _lib.serving_lib().cb_softcap(_lib.ptr(out), out.stride(0), M, N,
@@ -306,23 +318,24 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
 SKINNY_MAX = 16       # rows up to which a bf16 product runs on the weight-streaming kernel
 
 
-def _skinny_args(x, w, out, epi, softcap, accumulate):
+def _skinny_args(x, w, out, epi, softcap, accumulate, bias=None):
     f32 = out.dtype == torch.float32
-    return (_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(out), out.stride(0),
-            w.shape[0], w.shape[1], 5 if softcap is not None else EPI[epi],
+    return (_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(bias), _lib.ptr(out),
+            out.stride(0), w.shape[0], w.shape[1], 5 if softcap is not None else EPI[epi],
             ctypes.c_float(softcap or 0.0), int(f32), int(accumulate))
 
 
 def linear_pair(first: tuple, second: Optional[tuple] = None):
     """One or two independent products of the same few rows, each given as the arguments
-    ``(x, w, out, epi, softcap, accumulate)`` of :func:`linear`; in one launch where the rows are
-    few enough for the weight-streaming kernel (``cb_linear_skinny``), else one after the other."""
+    ``(x, w, out, epi, softcap, accumulate[, bias])`` of :func:`linear`; in one launch where the rows
+    are few enough for the weight-streaming kernel (``cb_linear_skinny``), else one after the other."""
     x = first[0]
     M = x.shape[0]
     todo = [first] if second is None else [first, second]
     if not x.is_cuda or x.dtype != torch.bfloat16 or M > SKINNY_MAX:
-        return [linear(a[0], a[1], a[2], epi=a[3], softcap=a[4], accumulate=a[5]) for a in todo]
-    empty = (None, 0, None, 0, None, 0, 0, 0, 0, ctypes.c_float(0.0), 0, 0)
+        return [linear(a[0], a[1], a[2], epi=a[3], softcap=a[4], accumulate=a[5],
+                       bias=a[6] if len(a) > 6 else None) for a in todo]
+    empty = (None, 0, None, 0, None, None, 0, 0, 0, 0, ctypes.c_float(0.0), 0, 0)
     rc = _lib.serving_lib().cb_linear_skinny(
         *_skinny_args(*first), *(empty if second is None else _skinny_args(*second)), M,
         _lib.stream_ptr())

@@ -1,5 +1,6 @@
-"""Ops of the ragged serving step (``csrc/ragged_rows.cu``, ``shortconv.cu``, ``delta_scan.cu``,
-``ragged_attn.cu``): one batch holds portions of prompts beside single decoded tokens, each at its
+"""Ops of the ragged serving step (``csrc/ragged_rows.cu``, ``residual.cu``, ``shortconv.cu``,
+``delta_scan.cu``, ``ragged_attn.cu``; latent attention and further recurrences have modules of their
+own): one batch holds portions of prompts beside single decoded tokens, each at its
 own position of its own sequence, and recurrent and cached state is addressed by slot.
 
 CPU tensors take a PyTorch restatement of the same math; CUDA tensors always run the kernels, in
@@ -21,6 +22,7 @@ CONV_TILE = 16        # tokens per block of the convolution kernels
 ATTN_TILE = 64        # query rows per block of the tensor-core attention kernel
 ROWS_MAX = 4          # entries of at most this many tokens take the row kernel
 MIN_PIECE = 64        # chunks from this size on are worth a piece of their own
+WINDOW_PIECE = 256    # query rows of a piece under a sliding window
 _F = ctypes.c_float
 
 
@@ -45,10 +47,15 @@ class AttnPlan:
     that lie in one chunk form a piece for the tcgen05 kernel.  A piece that starts at its chunk's
     start (or at position 0) needs only this step's keys and values; one that continues a chunk
     also needs the cached ones, which are gathered into rows for it.  A continued chunk of few
-    rows is not worth that and goes in tiles of ``ATTN_TILE`` rows that read the cache."""
+    rows is not worth that and goes in tiles of ``ATTN_TILE`` rows that read the cache.
+
+    Under a sliding ``window`` a piece is a run of at most ``WINDOW_PIECE`` rows together with the
+    keys its first row sees before it; an entry that continues a sequence gathers its own keys and
+    those of the window before it."""
 
     chunk: Optional[int]
     pieces: bool              # whether the layer's sizes allow the piece kernel
+    window: Optional[int] = None
 
 
 def pieces_allowed(dim: int, vdim: int, chunk: Optional[int], scale: float) -> bool:
@@ -102,13 +109,25 @@ class RaggedBatch:
         parts = [pos, np.asarray(self.pos0_host, np.int32), tokens, row_slot,
                  np.asarray(self.slots_host, np.int32), row0[:n], np.asarray(lens, np.int32),
                  np.asarray([c[0] for c in ct], np.int32), np.asarray([c[1] for c in ct], np.int32),
-                 rows, want]
+                 rows, want, np.arange(self.T, dtype=np.int32)]
         self.plans, cols = {}, len(parts)
         for plan in dict.fromkeys(plans):
             tiles, pieces, where = [], [], []
             extra = 0
             for i in big:
                 p0, r0 = entries[i].pos0, int(row0[i])
+                if plan.window is not None:
+                    ahead = min(p0, plan.window - 1)
+                    first = r0                             # key row of the entry's first token
+                    if p0:
+                        keys = np.arange(p0 - ahead, p0 + lens[i], dtype=np.int32)
+                        where.append(np.stack([np.full_like(keys, entries[i].slot), keys], 1))
+                        first = self.T + extra + ahead
+                        extra += len(keys)
+                    for o in range(0, lens[i], WINDOW_PIECE):
+                        before = min(ahead + o, plan.window - 1)
+                        pieces.append((r0 + o, min(WINDOW_PIECE, lens[i] - o), first + o - before, before))
+                    continue
                 head, ahead, ps = _cut(plan, p0, lens[i]) if plan.pieces else (lens[i], 0, [])
                 if plan.pieces and head > MIN_PIECE:
                     keys = np.arange(p0 - ahead, p0 + head, dtype=np.int32)
@@ -140,7 +159,7 @@ class RaggedBatch:
             views.append(self.buf[o:o + len(part)])
             o += len(part)
         (self.pos, self.pos0, self.tokens, self.row_slot, self.slot, self.row0, self.len,
-         self.conv_entry, self.conv_off, self.rows, self.want) = views[:cols]
+         self.conv_entry, self.conv_off, self.rows, self.want, self.every_row) = views[:cols]
         self._views = views
         self.positions = self.buf[:self.T + n]       # pos and pos0: what a decode step advances
         self.n_conv, self.n_rows, self.n_want = len(ct), len(rows), len(want)
@@ -198,6 +217,67 @@ def rms_rows(x: torch.Tensor, w1: torch.Tensor, width: int, eps: float, dtype: t
         _F(eps), int(dtype == torch.float32), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_rms_rows")
     return y1, y2
+
+
+def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dtype, *,
+             y: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+             post: Optional[torch.Tensor] = None, gain: Optional[torch.Tensor] = None,
+             shift: Optional[torch.Tensor] = None, before: Optional[torch.Tensor] = None,
+             batch: Optional["RaggedBatch"] = None, rows: Optional[torch.Tensor] = None,
+             keep: bool = True, casts: Sequence[torch.Tensor] = ()
+             ) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
+    """One pass between two sublayers, ``(x', h)``: ``v = y + bias``, RMS-normed with gain ``post`` when
+    given; ``x' = x + v`` in fp32 (``v`` alone without ``x``, ``x`` itself without ``y``); ``h`` the RMS
+    norm of ``x'`` with ``gain`` in the activation type, shifted by ``h + (h_before - h) * shift`` with
+    the previous token's h (``before [slots, ld]`` at an entry's start, which is advanced).  Gains are
+    one number or a vector.  ``rows`` restricts the pass to some rows (``x'`` is not returned then),
+    ``keep=False`` drops ``x'``; ``casts`` are up to two views that get ``x'`` in the activation type."""
+    src = x if x is not None else y
+    ld, n = src.shape[1], src.shape[0] if rows is None else rows.shape[0]
+    if rows is not None:
+        keep = False
+    if not src.is_cuda:
+        pick = (lambda t: t) if rows is None else (lambda t: t[rows.long()])
+
+        def norm(v, g):
+            return v * torch.rsqrt((v[:, :width] ** 2).mean(-1, keepdim=True) + eps) * g
+        out = None if x is None else pick(x)
+        if y is not None:
+            v = pick(y).float()
+            v = v if bias is None else v + bias
+            v = v if post is None else norm(v, post)
+            out = v if out is None else out + v
+        for c in casts:
+            c.copy_(out.to(c.dtype))
+        h = None
+        if gain is not None:
+            h = norm(out, gain)
+            if shift is not None:
+                prev, r = torch.zeros_like(h), 0
+                prev[1:] = h[:-1]
+                for i, m in enumerate(batch.lens):
+                    s = batch.slots_host[i]
+                    prev[r] = before[s] if int(batch.pos0[i]) > 0 else 0.0
+                    before[s] = h[r + m - 1]
+                    r += m
+                h = h + (prev - h) * shift
+            h = h.to(dtype)
+        return (out if keep else None), h
+    x_out = torch.empty((n, ld), dtype=torch.float32, device=src.device) \
+        if keep and (y is not None or x is None) else None
+    h = torch.empty((n, ld), dtype=dtype, device=src.device) if gain is not None else None
+    shifted = shift is not None
+    none = (None,) * 6
+    ents = (*batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off)) if shifted else none
+    cast = list(casts) + [None] * (2 - len(casts))
+    rc = _lib.serving_lib().cb_add_norm(
+        _p(x), _p(y), _p(bias), _p(post), int(post is not None and post.numel() > 1), _p(x_out), ld,
+        y.stride(0) if y is not None else 0, _p(gain), int(gain is not None and gain.numel() > 1), _p(h),
+        ld, _p(cast[0]), _p(cast[1]), casts[0].stride(0) if casts else 0, _p(shift), _p(before),
+        _p(rows), *ents, batch.n_conv if shifted else n, width, _F(eps), int(dtype == torch.float32),
+        int(y is not None and y.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_add_norm")
+    return (x_out if x_out is not None else (x if keep else None)), h
 
 
 def rope_table(pos: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
@@ -442,7 +522,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                 _p(q), _p(k_rows), _p(v_rows), _p(out), T, k_rows.shape[0], _p(pieces), n_pieces,
                 longest, heads, kv_heads, k_rows.shape[2], vdim, q.stride(0), k_rows.stride(0),
                 v_rows.stride(0), out.stride(0), _F(scale), _p(sink), _p(gate),
-                gate.stride(0) if gate is not None else 0, st, _lib.stream_ptr())
+                gate.stride(0) if gate is not None else 0, 0, 0, st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_attn_fwd_pieces")
     n = batch.n_rows
     if n:
