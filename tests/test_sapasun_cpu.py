@@ -51,7 +51,7 @@ def test_directory_round_trip_and_registry(tmp_path):
     assert registry.resolve(config).name == "Sapasun" and "Sapasun" in registry.architectures()
     lm = registry.load_dir(str(tmp_path), device="cpu", dtype=torch.float32)
     assert lm.cfg == b.cfg and lm.num_parameters() == b.lm.num_parameters()
-    w = cases.weights(b.cfg, b.seed)
+    w = b.w
     got = lm.state_dict()
     assert set(got) == set(w)
     for n in w:
@@ -166,7 +166,7 @@ def test_trace_runner(tmp_path):
             lo = at.get(i, 0)
             ids = seqs[i.split("#")[0]]
             es.append({"id": i, "tokens": ids[lo:lo + m], "want": w})
-            rows += [cases.oracle(b.cfg, b.seed, ids)[lo + k] for k in w]
+            rows += [b.oracle(ids)[lo + k] for k in w]
             at[i] = lo + m
         lines.append(json.dumps({"step": n, "entries": es, "end": end}))
         if rows:
