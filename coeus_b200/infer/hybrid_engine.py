@@ -190,7 +190,8 @@ class HybridEngine(InferenceEngine):
         y = torch.empty((b.T, _up8(s.out_dim)), dtype=raw.dtype, device=raw.device)
         RC.ssd_scan(u, layer.boff, layer.coff, raw[:, seg["dt"]:], layer.dt_bias, layer.A_log, layer.D,
                     self.state[n, "ssd"], s.groups, s.vdim, b, y)
-        RC.gated_group_norm(y, raw[:, seg["z"]:], layer.out_norm, s.norm_groups, self.cfg.norm_eps, out)
+        RC.gated_group_norm(y, raw[:, seg["z"]:], layer.out_norm, s.norm_groups, self.cfg.norm_eps,
+                            out[:, :s.out_dim])
 
     def _mingru(self, n: int, layer, raw: torch.Tensor, out: torch.Tensor, b: R.RaggedBatch) -> None:
         seg = layer.seg
