@@ -39,7 +39,7 @@ NVCC_FLAGS = [
 ]
 
 
-SERVING_SOURCES = ("gemm", "ragged_rows", "residual", "shortconv", "delta_scan", "ssd", "mingru",
+SERVING_SOURCES = ("gemm", "ragged_rows", "residual", "shortconv", "delta_scan", "ssd", "ssd_chunk", "mingru",
                    "linear_f32", "linear_skinny", "linear_heads", "ragged_attn", "latent_attn",
                    "attention_fwd")
 

@@ -3,37 +3,11 @@
 //   dt = softplus(dt_raw + dt_bias);   S <- exp(-exp(A_log) dt) S + dt B x^T;   y = S^T C + D x
 //
 //   step kernel    token by token on the FMA units: everything in fp32, and short entries
-//   chunk kernel   bf16 prompts: 64 tokens at a time as matrix products (below)
+//   chunk kernel   bf16 prompts: 64 tokens at a time as matrix products (ssd_chunk.cu)
 //   gated norm     y silu(z), RMS norm in equal parts, weight
-#include "ragged.cuh"
+#include "ssd.cuh"
 
 namespace cb {
-
-struct Ssd {
-  const void* u;           // [rows, ldu]: x at 0, B at boff, C at coff (behind the convolution)
-  int ldu, boff, coff;
-  const void* dt;          // [rows, lddt], column h: head h
-  int lddt;
-  const float* dt_bias;    // [heads]
-  const float* A_log;
-  const float* D;
-  float* state;            // [slots, heads, N, Pp]
-  void* y;                 // out [rows, ldy], head h at h * P
-  int ldy;
-  int heads, groups, N, P, Pp;
-  Entries e;
-  const int* entry;        // entries this launch works on: [n]
-  // segments of long entries (chunk kernel)
-  const int* seg_off;      // [n] first token inside the entry
-  const int* seg_len;      // [n]
-  float* seg_state;        // [n, heads, N, Pp], or null: one segment per entry, straight from the slot
-  float* seg_decay;        // [n, heads]
-};
-
-__device__ __forceinline__ float ssd_dt(float raw, float bias) {
-  const float x = raw + bias;
-  return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
-}
 
 // ------------------------------------------------------------------------------ step kernel
 // A block takes one (entry, head) and 64 columns: a thread has four columns and NR = N / 8 rows.
@@ -198,18 +172,6 @@ static int launch_norm(const void* y, int ldy, const void* z, int ldz, const flo
 }  // namespace cb
 
 using namespace cb;
-
-static int fill_ssd(Ssd& p, const void* u, int ldu, int boff, int coff, const void* dt, int lddt,
-                    const float* dt_bias, const float* A_log, const float* D, float* state, void* y,
-                    int ldy, int heads, int groups, int N, int P, int Pp, const int* slot, const int* row0,
-                    const int* len, const int* pos0, const int* entry) {
-  if (heads < 1 || groups < 1 || heads % groups || N < 1 || N > 256 || P < 1 || Pp < P || Pp % 4) return -1;
-  p.u = u; p.ldu = ldu; p.boff = boff; p.coff = coff; p.dt = dt; p.lddt = lddt; p.dt_bias = dt_bias;
-  p.A_log = A_log; p.D = D; p.state = state; p.y = y; p.ldy = ldy; p.heads = heads; p.groups = groups;
-  p.N = N; p.P = P; p.Pp = Pp; p.e.slot = slot; p.e.row0 = row0; p.e.len = len; p.e.pos0 = pos0;
-  p.entry = entry; p.seg_off = p.seg_len = nullptr; p.seg_state = p.seg_decay = nullptr;
-  return 0;
-}
 
 extern "C" int cb_ssd_step(const void* u, int ldu, int boff, int coff, const void* dt, int lddt,
                            const float* dt_bias, const float* A_log, const float* D, float* state,

@@ -16,7 +16,7 @@ import numpy as np
 import torch
 
 from ..foundation.error import ProcessingError
-from ..models.hybrid import CACHED, AttentionSpec, HybridLM, LatentAttentionSpec
+from ..models.hybrid import CACHED, AttentionSpec, HybridLM, LatentAttentionSpec, Mamba2Spec
 from ..ops import gemm as G
 from ..ops import latent as L
 from ..ops import ragged as R
@@ -51,6 +51,8 @@ class HybridEngine(InferenceEngine):
         self._runs = self.cfg.runs()
         self._plans = [self._plan(layer.mixer) for layer in self.cfg.layers
                        if isinstance(layer.mixer, CACHED)]
+        self._plans += [RC.ssd_plan(a.heads, a.vdim, a.state) for a in
+                        (layer.mixer for layer in self.cfg.layers) if isinstance(a, Mamba2Spec)]
 
     def _plan(self, a) -> R.AttnPlan:
         if isinstance(a, AttentionSpec):

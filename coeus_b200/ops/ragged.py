@@ -58,6 +58,34 @@ class AttnPlan:
     window: Optional[int] = None
 
 
+SCAN_MIN = 16         # entries of more tokens than this take the chunked recurrence
+SCAN_SEGMENT = 256    # and are cut into segments of at least this many
+SCAN_BLOCKS = 2 * 148
+
+
+@dataclass(frozen=True)
+class ScanPlan:
+    """How the entries of a batch go through a recurrence of ``blocks`` independent parts per entry
+    (heads): short ones token by token, long ones 64 tokens at a time, cut into segments where
+    there are fewer parts than the GPU has room for."""
+
+    blocks: int
+    chunks: bool              # whether the layer's sizes allow the chunked kernel
+
+
+def _segments(plan: ScanPlan, long: List[int], lens: List[int]):
+    """``([(entry, offset, tokens, 0)], [(entry, first segment, segments, 0)])``."""
+    want = SCAN_BLOCKS // max(1, plan.blocks * len(long))
+    segs, runs = [], []
+    for i in long:
+        n = max(1, min(want, lens[i] // SCAN_SEGMENT))
+        size = -(-lens[i] // (64 * n)) * 64
+        cut = [(i, o, min(size, lens[i] - o), 0) for o in range(0, lens[i], size)]
+        runs.append((i, len(segs), len(cut), 0))
+        segs += cut
+    return segs, runs
+
+
 def pieces_allowed(dim: int, vdim: int, chunk: Optional[int], scale: float) -> bool:
     return max(dim, vdim) <= 128 and scale > 0 and (chunk is None or chunk >= MIN_PIECE)
 
@@ -80,12 +108,12 @@ def _cut(plan: AttnPlan, pos0: int, n: int):
 class RaggedBatch:
     """Index arrays of one step, in one int32 buffer (one host-to-device copy).  ``tile_rows``
     says whether long entries may take the tensor-core attention kernels (bf16 models on CUDA);
-    otherwise every row is listed for the row kernel.  ``plans`` are the attention plans the
-    model's layers will ask for."""
+    otherwise every row is listed for the row kernel.  ``plans`` are the attention and
+    recurrence plans the model's layers will ask for."""
 
     def __init__(self, entries: List[Entry], device, tile_rows: bool = True,
                  into: Optional["RaggedBatch"] = None,
-                 plans: Sequence[AttnPlan] = (AttnPlan(None, False),)) -> None:
+                 plans: Sequence = (AttnPlan(None, False),)) -> None:
         n = len(entries)
         lens = [len(e.tokens) for e in entries]
         if not n or min(lens) < 1:
@@ -111,12 +139,24 @@ class RaggedBatch:
                  np.asarray([c[0] for c in ct], np.int32), np.asarray([c[1] for c in ct], np.int32),
                  rows, want, np.arange(self.T, dtype=np.int32)]
         self.plans, cols = {}, len(parts)
+        def align():                                               # read four at a time
+            parts.append(np.zeros(-sum(len(x) for x in parts) % 4, np.int32))
         for plan in dict.fromkeys(plans):
+            if isinstance(plan, ScanPlan):
+                long = [i for i, m in enumerate(lens) if tile_rows and plan.chunks and m > SCAN_MIN]
+                segs, runs = _segments(plan, long, lens)
+                align()
+                self.plans[plan] = (n - len(long), len(segs), len(runs), len(parts))
+                parts += [np.asarray(segs, np.int32).reshape(-1), np.asarray(runs, np.int32).reshape(-1),
+                          np.asarray([i for i in range(n) if i not in set(long)], np.int32)]
+                continue
             tiles, pieces, where = [], [], []
             extra = 0
             for i in big:
                 p0, r0 = entries[i].pos0, int(row0[i])
                 if plan.window is not None:
+                    if not plan.pieces:
+                        continue
                     ahead = min(p0, plan.window - 1)
                     first = r0                             # key row of the entry's first token
                     if p0:
@@ -139,8 +179,8 @@ class RaggedBatch:
                 pieces += [(r0 + o, m, r0 + o, 0) for o, m in ps]
             tiles.sort(key=lambda t: -(entries[t[0]].pos0 + t[1]))     # the most keys first
             pieces.sort(key=lambda t: -t[1] * (t[1] + 2 * t[3]))
-            if pieces:                                                 # read four at a time
-                parts.append(np.zeros(-sum(len(x) for x in parts) % 4, np.int32))
+            if pieces:
+                align()
             self.plans[plan] = (len(tiles), len(pieces), max([t[1] for t in pieces], default=0),
                                 extra, len(parts))
             parts += [np.asarray(pieces, np.int32).reshape(-1),
@@ -170,6 +210,11 @@ class RaggedBatch:
         gathered rows, tile entries, offsets, lengths)``."""
         n_tiles, n_pieces, longest, extra, at = self.plans[plan]
         return (n_tiles, n_pieces, longest, extra, *self._views[at:at + 5])
+
+    def scan(self, plan: ScanPlan):
+        """``(short entries, segments, entries in segments, segment array, run array, short array)``."""
+        n_short, n_segs, n_runs, at = self.plans[plan]
+        return (n_short, n_segs, n_runs, *self._views[at:at + 3])
 
     def kv_rows(self, plan: AttnPlan) -> int:
         """Rows of the ``k_rows`` / ``v_rows`` buffers under ``plan``: this step's, then gathered

@@ -11,9 +11,17 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
-from .ragged import RaggedBatch, _conv_ref, _p
+from .ragged import RaggedBatch, ScanPlan, _conv_ref, _p
 
 _F = ctypes.c_float
+
+
+SCAN_COLS = 64       # columns of a head per block
+CHUNK_STATE = 128    # largest state the chunked kernel takes
+
+
+def ssd_plan(heads: int, vdim: int, N: int) -> ScanPlan:
+    return ScanPlan(heads * ((vdim + SCAN_COLS - 1) // SCAN_COLS), N <= CHUNK_STATE)
 
 
 def shortconv_act(raw: torch.Tensor, off: int, taps_w: torch.Tensor, bias: torch.Tensor,
@@ -62,8 +70,18 @@ def ssd_scan(u: torch.Tensor, boff: int, coff: int, dt: torch.Tensor, dt_bias: t
     common = (_p(u), u.stride(0), boff, coff, _p(dt), dt.stride(0), _p(dt_bias), _p(A_log), _p(D),
               _p(state), _p(y), y.stride(0), heads, groups, N, vdim, state.shape[3],
               *batch.entry_args())
-    rc = lib.cb_ssd_step(*common, _p(batch.every_row), batch.n, int(f32), _lib.stream_ptr())
-    _lib.check_rc(rc, "cb_ssd_step")
+    n_short, n_segs, n_runs, segs, runs, short = batch.scan(ssd_plan(heads, vdim, N))
+    if n_short:
+        rc = lib.cb_ssd_step(*common, _p(short), n_short, int(f32), _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_ssd_step")
+    if n_segs:
+        kept = decay = None
+        if n_segs > n_runs:
+            kept = torch.empty((n_segs, *state.shape[1:]), dtype=torch.float32, device=u.device)
+            decay = torch.empty((n_segs, heads), dtype=torch.float32, device=u.device)
+        rc = lib.cb_ssd_chunk(*common, _p(segs), n_segs, _p(runs), n_runs, _p(kept), _p(decay),
+                              _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_ssd_chunk", launches=1 if kept is None else 3)
     return y
 
 
