@@ -1,5 +1,6 @@
-"""Serving throughput of the Sapasun design beside the framework's closest model at equal size, and
-its kernels one by one against the roofline (``python bench.py --serving sapasun [--kernels]``).
+"""Serving throughput of a design of mixed layers beside the framework's closest model at equal size,
+and its kernels one by one against the roofline (``python bench.py --serving sapasun|bananex
+[--kernels]``; the kernels of Bananex are in :mod:`coeus_b200.utils.bananex_bench`).
 
 The closest model is the RMSNorm / SwiGLU / rotary decoder with grouped-query attention: same
 width, depth, heads and vocabulary, the feed-forward as wide as gives the same parameters per
@@ -83,33 +84,76 @@ def throughput(model, steps: int, warmup: int) -> List[Dict]:
     return out
 
 
-def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> List[Dict]:
-    """Every kernel of the design and the like kernels of the closest model on the shapes of
-    ``size``: a prompt batch of 8 x 2048 tokens and a decode step of 64 sequences.  ``bound`` names
-    the roofline (measured copy bandwidth, measured bf16 throughput, or fp32 FMA issue at the
-    maximum clock), ``fraction`` is algorithmic work / time / roofline."""
-    from ..ops import attention as A
-    from ..ops import decode as D
-    from ..ops import elementwise as E
-    from ..ops import gemm as G
-    from ..ops import norm as N
-    from ..ops import ragged as R
+def recorder(rows: List[Dict], only: str, iters: int) -> Callable:
+    """``rec(name, phase, fn, bytes_ | flops | fma)``: times ``fn`` with L2 flushed in between and adds a
+    row; the bound is the largest of the times its bytes, bf16 operations and fp32 FMAs need."""
     from .kernel_bench import peaks, timeit
     hbm, tensor, source = peaks()
     fp32 = 148 * 128 * 1.965e9          # FMA issue slots per second
-    W, _, nh, kv = SIZES[size]
-    d, dev, bf = HEAD, "cuda", torch.bfloat16
-    rows: List[Dict] = []
 
     def rec(name, phase, fn, bytes_=0, flops=0, fma=0):
         if only not in f"{name}, {phase}":
             return
         us = timeit(fn, min(3, iters), iters, True) * 1e3
-        kind, best = ("bytes", bytes_ / hbm / 1e3) if bytes_ else (
-            ("bf16", flops / tensor / 1e6) if flops else ("fp32", fma / fp32 * 1e6))
+        best, kind = max((bytes_ / hbm / 1e3, "bytes"), (flops / tensor / 1e6, "bf16"),
+                         (fma / fp32 * 1e6, "fp32"))
         rows.append({"kernel": name, "phase": phase, "us": round(us, 1), "bound": kind,
                      "roofline_us": round(best, 1), "fraction": round(best / us, 3),
                      "peaks": source})
+    return rec
+
+
+def closest_kernels(rec, phase: str, B: int, S: int, at: int, W: int, nh: int, kv: int, c) -> None:
+    """The closest model's kernels at width ``W``; ``c`` is a cache of ``kv`` heads of ``HEAD``."""
+    from ..ops import attention as A
+    from ..ops import decode as D
+    from ..ops import elementwise as E
+    from ..ops import gemm as G
+    from ..ops import norm as N
+    T, d, dev = B * S, HEAD, "cuda"
+    qkv = (nh + 2 * kv) * d
+
+    def t(*shape):
+        return torch.randn(shape, device=dev, dtype=torch.float32).to(torch.bfloat16)
+    q = t(T, nh, d)
+    hx, wn = t(T, W), t(W)
+    rec("closest: norm_fwd", phase, lambda: N.norm_fwd(hx, wn, None, 1e-5, True), bytes_=T * W * 4)
+    w1 = t(W, qkv)
+    if S > 1:
+        rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), flops=2 * T * W * qkv)
+        kk, vv = t(T, kv * d), t(T, kv * d)
+        rec("closest: attention", phase, lambda: A.attention_fwd(q.view(T, -1), kk, vv, B, S, nh, d, causal=True),
+            flops=4 * B * S * S / 2 * nh * d)
+    else:
+        rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), bytes_=W * qkv * 2)
+        ctx = torch.full((B,), CONTEXT, dtype=torch.int32, device=dev)
+        pages = (CONTEXT + 63) // 64
+        kc, vc = t(B * pages, 64, kv, d), t(B * pages, 64, kv, d)
+        pt = torch.arange(B * pages, dtype=torch.int32, device=dev).view(B, pages)
+        rec("closest: attention", phase, lambda: D.decode_attention(q.view(T, -1), kc, vc, pt, ctx, nh, d, nkv=kv),
+            bytes_=B * CONTEXT * kv * d * 2 * 2)
+    buf = t(T, qkv)
+    pos = torch.full((B,), at, dtype=torch.int32, device=dev)
+    rec("closest: rope", phase, lambda: E.rope_(buf, nh + kv, d, S, pos_dev=pos if S == 1 else None),
+        bytes_=T * (nh + kv) * d * 4)
+    rec("closest: kv_write", phase, lambda: D.kv_write(
+        buf[:, nh * d:(nh + kv) * d], buf[:, (nh + kv) * d:], c.k[0], c.v[0], c.page_table, pos, S,
+        kv, d), bytes_=T * kv * d * 2 * 4)
+    gu = t(T, 2 * (8 * W // 3 // 128 * 128))
+    rec("closest: swiglu", phase, lambda: E.swiglu_fwd(gu), bytes_=gu.numel() * 3)
+
+
+def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> List[Dict]:
+    """Every kernel of the design and the like kernels of the closest model on the shapes of
+    ``size``: a prompt batch of 8 x 2048 tokens and a decode step of 64 sequences.  ``bound`` names
+    the roofline (measured copy bandwidth, measured bf16 throughput, or fp32 FMA issue at the
+    maximum clock), ``fraction`` is algorithmic work / time / roofline."""
+    from ..ops import gemm as G
+    from ..ops import ragged as R
+    W, _, nh, kv = SIZES[size]
+    d, dev, bf = HEAD, "cuda", torch.bfloat16
+    rows: List[Dict] = []
+    rec = recorder(rows, only, iters)
 
     def t(*shape, dtype=bf):
         return torch.randn(shape, device=dev, dtype=torch.float32).to(dtype)
@@ -195,43 +239,21 @@ def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> Li
         rec("gated_head_norm", phase, lambda: R.gated_head_norm(o, g2, ld.head_norm, 1e-5,
                                                                 out[:, :nh * d]),
             bytes_=T * nh * d * 8)
-        # ---- the closest model's kernels
-        hx, wn = t(T, W), t(W)
-        rec("closest: norm_fwd", phase, lambda: N.norm_fwd(hx, wn, None, 1e-5, True), bytes_=T * W * 4)
-        w1 = t(W, qkv)
-        if S > 1:
-            rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), flops=2 * T * W * qkv)
-            kk, vv = t(T, kv * d), t(T, kv * d)
-            rec("closest: attention", phase, lambda: A.attention_fwd(q.view(T, -1), kk, vv, B, S, nh, d, causal=True),
-                flops=4 * B * S * S / 2 * nh * d)
-        else:
-            rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), bytes_=wb(W, qkv))
-            ctx = torch.full((B,), CONTEXT, dtype=torch.int32, device=dev)
-            pages = (CONTEXT + 63) // 64
-            kc, vc = t(B * pages, 64, kv, d), t(B * pages, 64, kv, d)
-            pt = torch.arange(B * pages, dtype=torch.int32, device=dev).view(B, pages)
-            rec("closest: attention", phase, lambda: D.decode_attention(q.view(T, -1), kc, vc, pt, ctx, nh, d, nkv=kv),
-                bytes_=B * CONTEXT * kv * d * 2 * 2)
-        buf = t(T, qkv)
-        pos = torch.full((B,), at, dtype=torch.int32, device=dev)
-        rec("closest: rope", phase, lambda: E.rope_(buf, nh + kv, d, S, pos_dev=pos if S == 1 else None),
-            bytes_=T * (nh + kv) * d * 4)
-        rec("closest: kv_write", phase, lambda: D.kv_write(
-            buf[:, nh * d:(nh + kv) * d], buf[:, (nh + kv) * d:], c.k[0], c.v[0], c.page_table, pos, S,
-            kv, d), bytes_=T * kv * d * 2 * 4)
-        gu = t(T, 2 * (8 * W // 3 // 128 * 128))
-        rec("closest: swiglu", phase, lambda: E.swiglu_fwd(gu), bytes_=gu.numel() * 3)
+        closest_kernels(rec, phase, B, S, at, W, nh, kv, c)
         del eng, z
     return rows
 
 
-def run(steps: int = 20, warmup: int = 3, kernels: bool = False, sampler=None) -> None:
+def run(design: str, steps: int = 20, warmup: int = 3, kernels: bool = False, sampler=None) -> None:
     """One JSON line per size and model, then (``kernels``) one per kernel."""
     from ..ops import _lib
+    from . import bananex_bench
+    config, table = {"sapasun": (sapasun_config, kernel_table),
+                     "bananex": (bananex_bench.config, bananex_bench.kernel_table)}[design]
     for name, size in SIZES.items():
-        for which in ("sapasun", "closest"):
-            if which == "sapasun":
-                cfg = sapasun_config(*size)
+        for which in (design, "closest"):
+            if which == design:
+                cfg = config(*size)
                 model = H.HybridLM.random(cfg)
             else:
                 cfg = closest_config(*size)
@@ -256,20 +278,23 @@ def run(steps: int = 20, warmup: int = 3, kernels: bool = False, sampler=None) -
             del model
             torch.cuda.empty_cache()
     if kernels:
-        for row in kernel_table():
+        for row in table():
             print(json.dumps(row), flush=True)
 
 
 def main(argv=None) -> int:
-    """``python -m coeus_b200.utils.serving_bench --kernel delta_scan``: the kernel table alone, or the
+    """``python -m coeus_b200.utils.serving_bench --kernel delta_scan``: a kernel table alone, or its
     rows whose ``name, phase`` contains the text (with ``--iters 1`` a small case for a profiler)."""
     import argparse
     ap = argparse.ArgumentParser()
+    ap.add_argument("--design", default="sapasun", choices=["sapasun", "bananex"])
     ap.add_argument("--size", default="1b-layers", choices=list(SIZES))
     ap.add_argument("--kernel", default="")
     ap.add_argument("--iters", type=int, default=10)
     a = ap.parse_args(argv)
-    for row in kernel_table(a.size, a.kernel, a.iters):
+    from . import bananex_bench
+    table = kernel_table if a.design == "sapasun" else bananex_bench.kernel_table
+    for row in table(a.size, a.kernel, a.iters):
         print(json.dumps(row), flush=True)
     return 0
 
