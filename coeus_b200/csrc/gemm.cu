@@ -135,7 +135,7 @@ __device__ __forceinline__ void epilogue_math(const GemmArgs& p, float* v, float
     }
   } else if (p.epi == EPI_GELU_ERF) {
 #pragma unroll
-    for (int j = 0; j < 32; ++j) v[j] = gelu_erf_bf16(v[j]);
+    for (int j = 0; j < 32; j += 2) gelu_erf_pair(v[j], v[j + 1]);
   } else if (p.epi == EPI_DGELU && row_ok) {
     const __nv_bfloat16* ap = p.aux_in + static_cast<size_t>(row) * p.ldaux + col0;
 #pragma unroll

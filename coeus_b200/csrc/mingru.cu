@@ -1,14 +1,14 @@
 // The minGRU recurrence over a ragged batch, element by element in fp32:
 //   z = sigmoid(zl);  c = u >= 0 ? u + 1/2 : sigmoid(u);  S <- (1 - z) S + z c;  out = S silu(g)
 // with zl, u and g the projections.  A step is S <- a S + b, which composes: (a1, b1) then (a2, b2)
-// is (a1 a2, a2 b1 + b2).  A block owns 32 channels of one entry and goes through its tokens 128 at
-// a time: 16 threads side by side hold two channels each, 16 groups of them take eight tokens each,
+// is (a1 a2, a2 b1 + b2).  A block owns 32 channels of one entry and goes through its tokens 64 at
+// a time: 16 threads side by side hold two channels each, 16 groups of them take four tokens each,
 // compose them, and learn the state in front of their tokens from the groups before them.
 #include "ragged.cuh"
 
 namespace cb {
 
-constexpr int MG_CH = 32, MG_SEG = 16, MG_TOK = 8, MG_BLOCK = MG_SEG * MG_TOK;
+constexpr int MG_CH = 32, MG_SEG = 16, MG_TOK = 4, MG_BLOCK = MG_SEG * MG_TOK;
 
 struct MinGru {
   const void* raw;        // [rows, ld]: zl at zoff, u at uoff, g at goff
@@ -29,17 +29,26 @@ __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
 __device__ __forceinline__ void store_pair(float* p, float a, float b) {
   *reinterpret_cast<float2*>(p) = make_float2(a, b);
 }
-// a and b of one step
-__device__ __forceinline__ void mg_step(float zl, float u, float& a, float& b) {
-  const float ez = expf(-fabsf(zl)), r = 1.0f / (1.0f + ez);
-  const float z = zl >= 0.f ? r : ez * r;
-  a = zl >= 0.f ? ez * r : r;                            // 1 - z without cancellation
-  b = z * (u >= 0.f ? u + 0.5f : sigmoidf_(u));
-}
+// a and b of one step, and silu(g).  With e_v = exp(-|v|), every sigmoid here is 1 / (1 + e_v) or
+// e_v / (1 + e_v), so one reciprocal of the product of the three denominators (in 1..8) serves all.
+// bf16 projections take the fast exponential and reciprocal (a few units in the last place of fp32).
 template <typename T>
-__device__ __forceinline__ float mg_silu(float x) {
-  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-x));
-  else return x / (1.0f + expf(-x));
+__device__ __forceinline__ void mg_step(float zl, float u, float g, float& a, float& b, float& act) {
+  float ez, eu, eg;
+  if constexpr (sizeof(T) == 2) {
+    ez = __expf(-fabsf(zl)); eu = __expf(-fabsf(u)); eg = __expf(-fabsf(g));
+  } else {
+    ez = expf(-fabsf(zl)); eu = expf(-fabsf(u)); eg = expf(-fabsf(g));
+  }
+  const float pz = 1.f + ez, pu = 1.f + eu, pg = 1.f + eg, zu = pz * pu;
+  float r;
+  if constexpr (sizeof(T) == 2) r = __fdividef(1.0f, zu * pg);
+  else r = 1.0f / (zu * pg);
+  const float rz = pu * pg * r;                          // 1 / (1 + ez)
+  const float z = zl >= 0.f ? rz : ez * rz;
+  a = zl >= 0.f ? ez * rz : rz;                          // 1 - z without cancellation
+  b = z * (u >= 0.f ? u + 0.5f : eu * (pz * pg * r));
+  act = (g >= 0.f ? g : g * eg) * (zu * r);
 }
 
 template <typename T>
@@ -71,22 +80,18 @@ __global__ void __launch_bounds__(MG_CH / 2 * MG_SEG) mingru_kernel(const MinGru
   int turn = 0;
   for (int t0 = 0; t0 < len; t0 += MG_BLOCK, turn ^= 1) {
     const int n = min(MG_TOK, len - t0 - seg * MG_TOK);  // may be <= 0
-    float2 a[MG_TOK], b[MG_TOK], ta = make_float2(1.f, 1.f), tb = make_float2(0.f, 0.f);
+    float2 a[MG_TOK], b[MG_TOK], act[MG_TOK], ta = make_float2(1.f, 1.f), tb = make_float2(0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < MG_TOK; ++i) {
       a[i] = make_float2(1.f, 1.f);
-      b[i] = make_float2(0.f, 0.f);
+      b[i] = act[i] = make_float2(0.f, 0.f);
       if (i < n) {
-        mg_step(z[i].x, u[i].x, a[i].x, b[i].x);
-        mg_step(z[i].y, u[i].y, a[i].y, b[i].y);
+        mg_step<T>(z[i].x, u[i].x, g[i].x, a[i].x, b[i].x, act[i].x);
+        mg_step<T>(z[i].y, u[i].y, g[i].y, a[i].y, b[i].y, act[i].y);
       }
       tb = make_float2(a[i].x * tb.x + b[i].x, a[i].y * tb.y + b[i].y);
       ta = make_float2(ta.x * a[i].x, ta.y * a[i].y);
     }
-    float2 act[MG_TOK];
-#pragma unroll
-    for (int i = 0; i < MG_TOK; ++i)
-      act[i] = i < n ? make_float2(mg_silu<T>(g[i].x), mg_silu<T>(g[i].y)) : make_float2(0.f, 0.f);
     if (t0 + MG_BLOCK < len) fetch(t0 + MG_BLOCK);
     sa[seg][cp] = ta;
     sb[seg][cp] = tb;
@@ -119,12 +124,12 @@ __global__ void __launch_bounds__(128) mingru_short_kernel(const MinGru p) {
   for (int t = 0; t < len; ++t) {
     const T* r = static_cast<const T*>(p.raw) + static_cast<size_t>(row0 + t) * p.ld + ch;
     const float2 z = load_pair(r + p.zoff), u = load_pair(r + p.uoff), g = load_pair(r + p.goff);
-    float2 a, b;
-    mg_step(z.x, u.x, a.x, b.x);
-    mg_step(z.y, u.y, a.y, b.y);
+    float2 a, b, act;
+    mg_step<T>(z.x, u.x, g.x, a.x, b.x, act.x);
+    mg_step<T>(z.y, u.y, g.y, a.y, b.y, act.y);
     s = make_float2(a.x * s.x + b.x, a.y * s.y + b.y);
-    store_pair(static_cast<T*>(p.out) + static_cast<size_t>(row0 + t) * p.ldo + ch, s.x * mg_silu<T>(g.x),
-               s.y * mg_silu<T>(g.y));
+    store_pair(static_cast<T*>(p.out) + static_cast<size_t>(row0 + t) * p.ldo + ch, s.x * act.x,
+               s.y * act.y);
   }
   *st = s;
 }

@@ -674,32 +674,56 @@ __global__ void __launch_bounds__(CONV_THREADS) shortconv_act_kernel(const ConvA
     for (int j = 1; j < TAPS; ++j) at(off - TAPS + j, u[j]);
   }
   const int t1 = min(off + CONV_TILE, len);
-#pragma unroll 4
-  for (int t = off; t < t1; ++t) {
-    float y[V];
+  auto finish = [&](int t, float* y) {
 #pragma unroll
-    for (int k = 0; k < V; ++k) y[k] = b[k];
-    if constexpr (TAPS > 0) {
+    for (int k = 0; k < V; ++k) y[k] = silu_act<T>(y[k]);
+    store_vec<V>(out + static_cast<ptrdiff_t>(t) * p.channels, y);
+  };
+  if constexpr (TAPS > 0) {
+    auto step = [&](int t, const float* f) {
+      float y[V];
 #pragma unroll
       for (int j = 0; j + 1 < TAPS; ++j)
 #pragma unroll
         for (int k = 0; k < V; ++k) u[j][k] = u[j + 1][k];
-      load_vec<V>(raw + static_cast<ptrdiff_t>(t) * p.ld, u[W - 1]);
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        u[W - 1][k] = f[k];
+        y[k] = b[k];
+      }
 #pragma unroll
       for (int j = 0; j < TAPS; ++j)
 #pragma unroll
         for (int k = 0; k < V; ++k) y[k] += u[j][k] * w[j][k];
-    } else {
+      finish(t, y);
+    };
+    int t = off;
+    constexpr int AHEAD = 4;               // rows loaded together
+    for (; t + AHEAD <= t1; t += AHEAD) {
+      float f[AHEAD][V];
+#pragma unroll
+      for (int i = 0; i < AHEAD; ++i) load_vec<V>(raw + static_cast<ptrdiff_t>(t + i) * p.ld, f[i]);
+#pragma unroll
+      for (int i = 0; i < AHEAD; ++i) step(t + i, f[i]);
+    }
+    for (; t < t1; ++t) {
+      float f[V];
+      load_vec<V>(raw + static_cast<ptrdiff_t>(t) * p.ld, f);
+      step(t, f);
+    }
+  } else {
+    for (int t = off; t < t1; ++t) {
+      float y[V];
+#pragma unroll
+      for (int k = 0; k < V; ++k) y[k] = b[k];
       for (int j = 0; j <= n1; ++j) {
         at(t - n1 + j, u[0]);
         load_vec<V>(p.taps_w + static_cast<ptrdiff_t>(j) * p.channels + c, w[0]);
 #pragma unroll
         for (int k = 0; k < V; ++k) y[k] += u[0][k] * w[0][k];
       }
+      finish(t, y);
     }
-#pragma unroll
-    for (int k = 0; k < V; ++k) y[k] = silu_act<T>(y[k]);
-    store_vec<V>(out + static_cast<ptrdiff_t>(t) * p.channels, y);
   }
   if (off == 0)
     for (int j = 0; j < n1; ++j) {        // ascending: row j + len is read before it is replaced

@@ -2,9 +2,10 @@
 // m16n8k16).  With c_i the sum of the log-decays of a chunk's tokens up to and including i:
 //   y_i = exp(c_i) C_i . S  +  sum_{j <= i} (C_i . B_j) exp(c_i - c_j) dt_j x_j  +  D x_i
 //   S  <- exp(c_last) S  +  sum_j exp(c_last - c_j) dt_j B_j x_j^T
-// x, B and C enter as the bf16 numbers they are; what is computed in fp32 (the state, the weighted
-// scores, the weighted B) enters a product as the sum of two bf16 numbers.  The state stays in fp32
-// registers from an entry's first token to its last.
+// x, B and C enter as the bf16 numbers they are.  The state stays in fp32 registers from an entry's
+// first token to its last, and what is added to it (the weighted B) enters its product as the sum of
+// two bf16 numbers; only for reading y, which is rounded to bf16 itself, are the state and the
+// weighted scores rounded to bf16 operands.
 //
 // A block of four warps takes one head (and 64 of its columns) of one segment of an entry; a warp
 // owns 16 of the chunk's rows for y and every fourth 16-row tile of S.  Where entries and heads do
@@ -41,7 +42,7 @@ __device__ __forceinline__ void split2(float u, float v, uint32_t& hi, uint32_t&
 
 template <int NP>
 constexpr int sc_smem() {
-  return (2 * SC_TOK * (NP + 8) + SC_TOK * SC_XP + 2 * NP * SC_XP) * 2 + 4 * SC_TOK * 4;
+  return (2 * SC_TOK * (NP + 8) + SC_TOK * SC_XP + NP * SC_XP) * 2 + 4 * SC_TOK * 4;
 }
 
 enum : int { SC_WHOLE = 0, SC_STATE = 1, SC_FROM = 2 };
@@ -54,9 +55,8 @@ __global__ void __launch_bounds__(SC_THREADS, 2) ssd_chunk_kernel(const Ssd p) {
   bf16* sB = reinterpret_cast<bf16*>(sc_raw);              // [SC_TOK][LD]
   bf16* sC = sB + SC_TOK * LD;                             // [SC_TOK][LD]
   bf16* sX = sC + SC_TOK * LD;                             // [SC_TOK][SC_XP]
-  bf16* sH = sX + SC_TOK * SC_XP;                          // [NP][SC_XP] state, high part
-  bf16* sL = sH + NP * SC_XP;                              // and low part
-  float* sCum = reinterpret_cast<float*>(sL + NP * SC_XP); // [SC_TOK] c_i, in units of log 2
+  bf16* sS = sX + SC_TOK * SC_XP;                          // [NP][SC_XP] state in front of the chunk
+  float* sCum = reinterpret_cast<float*>(sS + NP * SC_XP); // [SC_TOK] c_i, in units of log 2
   float* sDt = sCum + SC_TOK;
   float* sE = sDt + SC_TOK;                                // exp(c_i)
   float* sW = sE + SC_TOK;                                 // exp(c_last - c_i) dt_i
@@ -154,10 +154,7 @@ __global__ void __launch_bounds__(SC_THREADS, 2) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
             const int at = ((warp + 4 * a) * 16 + r + c * 8) * SC_XP + b * 8 + t * 2;
-            uint32_t hi, lo;
-            split2(S[a][b][2 * c], S[a][b][2 * c + 1], hi, lo);
-            *reinterpret_cast<uint32_t*>(sH + at) = hi;
-            *reinterpret_cast<uint32_t*>(sL + at) = lo;
+            *reinterpret_cast<uint32_t*>(sS + at) = pack_bf16x2(S[a][b][2 * c], S[a][b][2 * c + 1]);
           }
     }
     cp_async_wait<0>();
@@ -185,11 +182,7 @@ __global__ void __launch_bounds__(SC_THREADS, 2) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) {                      // C . S
           uint32_t b[4];
-          const int at = (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8;
-          sc_ldsm4_t(b, smem_u32(sH + at));
-          sc_mma(y[2 * j], a, b[0], b[1]);
-          sc_mma(y[2 * j + 1], a, b[2], b[3]);
-          sc_ldsm4_t(b, smem_u32(sL + at));
+          sc_ldsm4_t(b, smem_u32(sS + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
           sc_mma(y[2 * j], a, b[0], b[1]);
           sc_mma(y[2 * j + 1], a, b[2], b[3]);
         }
@@ -207,19 +200,15 @@ __global__ void __launch_bounds__(SC_THREADS, 2) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         if (k <= warp) {
-          uint32_t hi[4], lo[4];
-          split2(G[2 * k][0], G[2 * k][1], hi[0], lo[0]);
-          split2(G[2 * k][2], G[2 * k][3], hi[1], lo[1]);
-          split2(G[2 * k + 1][0], G[2 * k + 1][1], hi[2], lo[2]);
-          split2(G[2 * k + 1][2], G[2 * k + 1][3], hi[3], lo[3]);
+          const uint32_t m[4] = {pack_bf16x2(G[2 * k][0], G[2 * k][1]), pack_bf16x2(G[2 * k][2], G[2 * k][3]),
+                                 pack_bf16x2(G[2 * k + 1][0], G[2 * k + 1][1]),
+                                 pack_bf16x2(G[2 * k + 1][2], G[2 * k + 1][3])};
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             uint32_t b[4];
             sc_ldsm4_t(b, smem_u32(sX + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
-            sc_mma(y[2 * j], hi, b[0], b[1]);
-            sc_mma(y[2 * j + 1], hi, b[2], b[3]);
-            sc_mma(y[2 * j], lo, b[0], b[1]);
-            sc_mma(y[2 * j + 1], lo, b[2], b[3]);
+            sc_mma(y[2 * j], m, b[0], b[1]);
+            sc_mma(y[2 * j + 1], m, b[2], b[3]);
           }
         }
       }
