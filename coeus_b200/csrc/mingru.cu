@@ -36,13 +36,14 @@ template <typename T>
 __device__ __forceinline__ void mg_step(float zl, float u, float g, float& a, float& b, float& act) {
   float ez, eu, eg;
   if constexpr (sizeof(T) == 2) {
-    ez = __expf(-fabsf(zl)); eu = __expf(-fabsf(u)); eg = __expf(-fabsf(g));
+    constexpr float L2E = -1.4426950408889634f;
+    ez = fast_exp2(fabsf(zl) * L2E); eu = fast_exp2(fabsf(u) * L2E); eg = fast_exp2(fabsf(g) * L2E);
   } else {
     ez = expf(-fabsf(zl)); eu = expf(-fabsf(u)); eg = expf(-fabsf(g));
   }
   const float pz = 1.f + ez, pu = 1.f + eu, pg = 1.f + eg, zu = pz * pu;
   float r;
-  if constexpr (sizeof(T) == 2) r = __fdividef(1.0f, zu * pg);
+  if constexpr (sizeof(T) == 2) asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(zu * pg));
   else r = 1.0f / (zu * pg);
   const float rz = pu * pg * r;                          // 1 / (1 + ez)
   const float z = zl >= 0.f ? rz : ez * rz;
@@ -52,34 +53,34 @@ __device__ __forceinline__ void mg_step(float zl, float u, float g, float& a, fl
 }
 
 template <typename T>
-__global__ void __launch_bounds__(MG_CH / 2 * MG_SEG) mingru_kernel(const MinGru p) {
-  __shared__ float2 sa[MG_SEG][MG_CH / 2], sb[MG_SEG][MG_CH / 2];
+__global__ void __launch_bounds__(MG_CH / 2 * MG_SEG, 4) mingru_kernel(const MinGru p) {
+  __shared__ float2 sa[MG_SEG / 2][MG_CH / 2], sb[MG_SEG / 2][MG_CH / 2];    // of two groups together
   __shared__ float2 carry[2][MG_CH / 2];
   const int e = blockIdx.y, row0 = p.e.row0[e], len = p.e.len[e], slot = p.e.slot[e];
   const int cp = threadIdx.x % (MG_CH / 2), seg = threadIdx.x / (MG_CH / 2);
   const int ch = blockIdx.x * MG_CH + cp * 2;
   const bool in = ch < p.width;
   float* st = p.state + static_cast<size_t>(slot) * p.width + ch;
-  const T* raw = static_cast<const T*>(p.raw) + static_cast<size_t>(row0) * p.ld + (in ? ch : 0);
-  T* out = static_cast<T*>(p.out) + static_cast<size_t>(row0) * p.ldo + ch;
+  const T* raw = static_cast<const T*>(p.raw) + (static_cast<size_t>(row0) + seg * MG_TOK) * p.ld + (in ? ch : 0);
+  T* out = static_cast<T*>(p.out) + (static_cast<size_t>(row0) + seg * MG_TOK) * p.ldo + ch;
+  const ptrdiff_t ahead = static_cast<ptrdiff_t>(MG_BLOCK) * p.ld, out_ahead = static_cast<ptrdiff_t>(MG_BLOCK) * p.ldo;
   if (seg == 0)
     carry[0][cp] = in && p.e.pos0[e] > 0 ? *reinterpret_cast<const float2*>(st) : make_float2(0.f, 0.f);
   float2 z[MG_TOK], u[MG_TOK], g[MG_TOK];
-  auto fetch = [&](int t0) {
+  auto fetch = [&](int n) {
+    const T* r = raw;
 #pragma unroll
-    for (int i = 0; i < MG_TOK; ++i) {
-      const int t = t0 + seg * MG_TOK + i;
-      if (t >= len) continue;
-      const T* r = raw + static_cast<size_t>(t) * p.ld;
+    for (int i = 0; i < MG_TOK; ++i, r += p.ld) {
+      if (i >= n) continue;
       z[i] = load_pair(r + p.zoff);
       u[i] = load_pair(r + p.uoff);
       g[i] = load_pair(r + p.goff);
     }
   };
-  fetch(0);
+  fetch(len - seg * MG_TOK);
   int turn = 0;
   for (int t0 = 0; t0 < len; t0 += MG_BLOCK, turn ^= 1) {
-    const int n = min(MG_TOK, len - t0 - seg * MG_TOK);  // may be <= 0
+    const int n = len - t0 - seg * MG_TOK;               // of these four; may be <= 0
     float2 a[MG_TOK], b[MG_TOK], act[MG_TOK], ta = make_float2(1.f, 1.f), tb = make_float2(0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < MG_TOK; ++i) {
@@ -92,21 +93,30 @@ __global__ void __launch_bounds__(MG_CH / 2 * MG_SEG) mingru_kernel(const MinGru
       tb = make_float2(a[i].x * tb.x + b[i].x, a[i].y * tb.y + b[i].y);
       ta = make_float2(ta.x * a[i].x, ta.y * a[i].y);
     }
-    if (t0 + MG_BLOCK < len) fetch(t0 + MG_BLOCK);
-    sa[seg][cp] = ta;
-    sb[seg][cp] = tb;
+    raw += ahead;
+    fetch(n - MG_BLOCK);
+    // the even group of the warp's two, seen from the odd one
+    const float2 ea = make_float2(__shfl_xor_sync(0xffffffffu, ta.x, 16), __shfl_xor_sync(0xffffffffu, ta.y, 16));
+    const float2 eb = make_float2(__shfl_xor_sync(0xffffffffu, tb.x, 16), __shfl_xor_sync(0xffffffffu, tb.y, 16));
+    const bool odd = seg & 1;
+    if (odd) {
+      sa[seg / 2][cp] = make_float2(ta.x * ea.x, ta.y * ea.y);
+      sb[seg / 2][cp] = make_float2(ta.x * eb.x + tb.x, ta.y * eb.y + tb.y);
+    }
     __syncthreads();
     float2 s = carry[turn][cp];
-    for (int k = 0; k < seg; ++k) {
+    for (int k = 0; k < seg / 2; ++k) {
       const float2 ka = sa[k][cp], kb = sb[k][cp];
       s = make_float2(ka.x * s.x + kb.x, ka.y * s.y + kb.y);
     }
+    if (odd) s = make_float2(ea.x * s.x + eb.x, ea.y * s.y + eb.y);
+    T* o = out;
 #pragma unroll
-    for (int i = 0; i < MG_TOK; ++i) {
+    for (int i = 0; i < MG_TOK; ++i, o += p.ldo) {
       s = make_float2(a[i].x * s.x + b[i].x, a[i].y * s.y + b[i].y);
-      if (i < n && in)
-        store_pair(out + static_cast<size_t>(t0 + seg * MG_TOK + i) * p.ldo, s.x * act[i].x, s.y * act[i].y);
+      if (i < n && in) store_pair(o, s.x * act[i].x, s.y * act[i].y);
     }
+    out += out_ahead;
     if (seg == MG_SEG - 1) carry[turn ^ 1][cp] = s;      // identity steps behind the entry's end
     __syncthreads();
   }

@@ -11,6 +11,8 @@
 // owns 16 of the chunk's rows for y and every fourth 16-row tile of S.  Where entries and heads do
 // not fill the GPU, entries are cut into segments: a first launch finds what each segment adds to an
 // empty state, a second one carries the states through, a third one runs all segments at once.
+#include <type_traits>
+
 #include "ssd.cuh"
 
 namespace cb {
@@ -48,7 +50,7 @@ constexpr int sc_smem() {
 enum : int { SC_WHOLE = 0, SC_STATE = 1, SC_FROM = 2 };
 
 template <int NP, int MODE>
-__global__ void __launch_bounds__(SC_THREADS, 2) ssd_chunk_kernel(const Ssd p) {
+__global__ void __launch_bounds__(SC_THREADS, 3) ssd_chunk_kernel(const Ssd p) {
   using bf16 = __nv_bfloat16;
   constexpr int LD = NP + 8, RT = NP / 64;                 // RT 16-row tiles of S per warp
   extern __shared__ __align__(16) unsigned char sc_raw[];
@@ -97,17 +99,21 @@ __global__ void __launch_bounds__(SC_THREADS, 2) ssd_chunk_kernel(const Ssd p) {
     const int n_tok = min(SC_TOK, len - c0);
     // ---- the chunk into shared memory; rows behind the segment's end are zero
     if (vec) {
-      const int nb = p.N / 8, xb = cols / 8, per = 2 * nb + xb;
-      for (int i = tid; i < SC_TOK * per; i += SC_THREADS) {
-        const int tok = i / per, k = i % per;
-        const size_t at = static_cast<size_t>(c0 + min(tok, n_tok - 1)) * p.ldu;
-        const bf16* src;
-        bf16* dst;
-        if (k < nb) { src = gB + k * 8; dst = sB + tok * LD + k * 8; }
-        else if (k < 2 * nb) { src = gC + (k - nb) * 8; dst = sC + tok * LD + (k - nb) * 8; }
-        else { src = gx + (k - 2 * nb) * 8; dst = sX + tok * SC_XP + (k - 2 * nb) * 8; }
-        cp_async16_zfill(smem_u32(dst), src + at, tok < n_tok ? 16 : 0);
-      }
+      auto rows_in = [&](bf16* dst, int pitch, const bf16* src, auto width, int n) {   // n of width columns
+        constexpr int C8 = decltype(width)::value / 8;
+        const int k = tid % C8;
+        if (k * 8 >= n) return;
+        const uint32_t to = smem_u32(dst + k * 8);
+#pragma unroll
+        for (int i = 0; i < SC_TOK * C8 / SC_THREADS; ++i) {
+          const int tok = tid / C8 + i * (SC_THREADS / C8);
+          cp_async16_zfill(to + tok * pitch * 2, src + static_cast<size_t>(c0 + min(tok, n_tok - 1)) * p.ldu + k * 8,
+                           tok < n_tok ? 16 : 0);
+        }
+      };
+      rows_in(sB, LD, gB, std::integral_constant<int, NP>(), p.N);
+      if (MODE != SC_STATE) rows_in(sC, LD, gC, std::integral_constant<int, NP>(), p.N);
+      rows_in(sX, SC_XP, gx, std::integral_constant<int, SC_COLS>(), cols);
       cp_async_commit();
     } else {
       const int per = 2 * p.N + cols;
@@ -161,54 +167,74 @@ __global__ void __launch_bounds__(SC_THREADS, 2) ssd_chunk_kernel(const Ssd p) {
     __syncthreads();
     if (MODE != SC_STATE) {
       // ---- scores C_i . B_j of this warp's rows, columns up to its own
-      float G[8][4], y[8][4];
+      const int i0 = warp * 16 + r;
+      const bf16* rowsC = sC + (warp * 16 + (lane & 15)) * LD + (lane >> 4) * 8;
+      uint32_t m[4][4];                                    // weighted, as operands of the product with x
+      {
+        float G[8][4];
+#pragma unroll
+        for (int b = 0; b < 8; ++b)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) G[b][c] = 0.f;
+#pragma unroll
+        for (int k = 0; k < NP / 16; ++k) {
+          uint32_t a[4];
+          sc_ldsm4(a, smem_u32(rowsC + k * 16));
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            if (j <= warp) {
+              uint32_t b[4];
+              sc_ldsm4(b, smem_u32(sB + (j * 16 + (lane & 7) + (lane >> 4) * 8) * LD + k * 16 + ((lane >> 3) & 1) * 8));
+              sc_mma(G[2 * j], a, b[0], b[1]);
+              sc_mma(G[2 * j + 1], a, b[2], b[3]);
+            }
+          }
+        }
+        const float ci[2] = {sCum[i0], sCum[i0 + 8]};
+#pragma unroll
+        for (int b = 0; b < 8; ++b) {
+          const float2 cj = *reinterpret_cast<const float2*>(sCum + b * 8 + t * 2);
+          const float2 dj = *reinterpret_cast<const float2*>(sDt + b * 8 + t * 2);
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            const int i = i0 + c * 8, j = b * 8 + t * 2;
+            const float u = j <= i ? G[b][2 * c] * fast_exp2(ci[c] - cj.x) * dj.x : 0.f;
+            const float v = j < i ? G[b][2 * c + 1] * fast_exp2(ci[c] - cj.y) * dj.y : 0.f;
+            m[b / 2][(b & 1) * 2 + c] = pack_bf16x2(u, v);
+          }
+        }
+      }
+      float y[8][4];
 #pragma unroll
       for (int b = 0; b < 8; ++b)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) G[b][c] = y[b][c] = 0.f;
+        for (int c = 0; c < 4; ++c) y[b][c] = 0.f;
 #pragma unroll
-      for (int k = 0; k < NP / 16; ++k) {
+      for (int k = 0; k < NP / 16; ++k) {                  // C . S
         uint32_t a[4];
-        sc_ldsm4(a, smem_u32(sC + (warp * 16 + (lane & 15)) * LD + k * 16 + (lane >> 4) * 8));
+        sc_ldsm4(a, smem_u32(rowsC + k * 16));
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          if (j <= warp) {
-            uint32_t b[4];
-            sc_ldsm4(b, smem_u32(sB + (j * 16 + (lane & 7) + (lane >> 4) * 8) * LD + k * 16 + ((lane >> 3) & 1) * 8));
-            sc_mma(G[2 * j], a, b[0], b[1]);
-            sc_mma(G[2 * j + 1], a, b[2], b[3]);
-          }
-        }
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {                      // C . S
           uint32_t b[4];
           sc_ldsm4_t(b, smem_u32(sS + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
           sc_mma(y[2 * j], a, b[0], b[1]);
           sc_mma(y[2 * j + 1], a, b[2], b[3]);
         }
       }
-      const int i0 = warp * 16 + r;
-      const float ci[2] = {sCum[i0], sCum[i0 + 8]}, ei[2] = {sE[i0], sE[i0 + 8]};
+      const float ei[2] = {sE[i0], sE[i0 + 8]};
 #pragma unroll
       for (int b = 0; b < 8; ++b)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          y[b][c] *= ei[c >> 1];
-          const int i = i0 + (c >> 1) * 8, j = b * 8 + t * 2 + (c & 1);
-          G[b][c] = j <= i ? G[b][c] * fast_exp2(ci[c >> 1] - sCum[j]) * sDt[j] : 0.f;
-        }
+        for (int c = 0; c < 4; ++c) y[b][c] *= ei[c >> 1];
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         if (k <= warp) {
-          const uint32_t m[4] = {pack_bf16x2(G[2 * k][0], G[2 * k][1]), pack_bf16x2(G[2 * k][2], G[2 * k][3]),
-                                 pack_bf16x2(G[2 * k + 1][0], G[2 * k + 1][1]),
-                                 pack_bf16x2(G[2 * k + 1][2], G[2 * k + 1][3])};
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             uint32_t b[4];
             sc_ldsm4_t(b, smem_u32(sX + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
-            sc_mma(y[2 * j], m, b[0], b[1]);
-            sc_mma(y[2 * j + 1], m, b[2], b[3]);
+            sc_mma(y[2 * j], m[k], b[0], b[1]);
+            sc_mma(y[2 * j + 1], m[k], b[2], b[3]);
           }
         }
       }
