@@ -36,7 +36,8 @@ struct LatentPrep {
   int* status;
 };
 
-// V = 8: dim, rot and q_head are multiples of eight; V = 1: any sizes
+// V = 8: dim, rot, rank, q_head and the row sizes are multiples of eight, rank at most 2048; V = 1:
+// any sizes
 template <typename T, int V>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrep p) {
   __shared__ float red[32];
@@ -53,26 +54,15 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrep p) {
   T* cell = page < 0 ? nullptr
                      : static_cast<T*>(p.cache) + (static_cast<size_t>(page) * RAGGED_PAGE + pos % RAGGED_PAGE) * p.lat_p;
   T* keep = p.rows_out != nullptr ? static_cast<T*>(p.rows_out) + static_cast<size_t>(row) * p.lat_p : nullptr;
-  float s = 0.f;
-  for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
-    const float v = to_f32(lat[c]);
-    s += v * v;
-  }
-  s = block_sum(s, red);
-  const float rs = 1.0f / sqrtf(s / p.rank + p.eps);
-  for (int c = threadIdx.x; c < p.lat_p; c += blockDim.x) {
-    float v = 0.f;
-    if (c < p.rank) {
-      v = to_f32(lat[c]) * rs * p.norm[c];
-    } else if (c < p.rank + p.rot) {
-      const int i = (c - p.rank) / 2, odd = (c - p.rank) & 1;
-      const float a = to_f32(lat[p.rank + 2 * i]), b = to_f32(lat[p.rank + 2 * i + 1]);
-      const float2 cs = rope[i];
-      v = odd ? b * cs.x + a * cs.y : a * cs.x - b * cs.y;
-    }
-    const T o = from_f32<T>(v);
-    if (cell != nullptr) cell[c] = o;
-    if (keep != nullptr) keep[c] = o;
+  float s = 0.f, own[V];                     // V = 8: a thread has eight numbers of the row
+  const int c8 = threadIdx.x * 8;
+  if constexpr (V == 8) {
+    if (c8 < p.rank + p.rot) load_vec<V>(lat + c8, own);
+    if (c8 < p.rank)
+#pragma unroll
+      for (int k = 0; k < V; ++k) s += own[k] * own[k];
+  } else {
+    for (int c = threadIdx.x; c < p.rank; c += blockDim.x) s += to_f32(lat[c]) * to_f32(lat[c]);
   }
   const int units = p.q_head / V, full = p.dim + p.rot;
   T* q = static_cast<T*>(p.q) + static_cast<size_t>(row) * p.heads * p.q_head;
@@ -102,6 +92,42 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrep p) {
       }
     }
     store_vec<V>(q + h * p.q_head + d, o);
+  }
+  s = block_sum(s, red);
+  const float rs = 1.0f / sqrtf(s / p.rank + p.eps);
+  if constexpr (V == 8) {
+    if (c8 >= p.lat_p) return;
+    float o[V];
+    if (c8 < p.rank) {
+      float g[V];
+      load_vec<V>(p.norm + c8, g);
+#pragma unroll
+      for (int k = 0; k < V; ++k) o[k] = own[k] * rs * g[k];
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; k += 2) {
+        const float2 cs = rope[(c8 - p.rank + k) / 2];
+        o[k] = own[k] * cs.x - own[k + 1] * cs.y;
+        o[k + 1] = own[k + 1] * cs.x + own[k] * cs.y;
+      }
+    }
+    if (cell != nullptr) store_vec<V>(cell + c8, o);
+    if (keep != nullptr) store_vec<V>(keep + c8, o);
+  } else {
+    for (int c = threadIdx.x; c < p.lat_p; c += blockDim.x) {
+      float v = 0.f;
+      if (c < p.rank) {
+        v = to_f32(lat[c]) * rs * p.norm[c];
+      } else if (c < p.rank + p.rot) {
+        const int i = (c - p.rank) / 2, odd = (c - p.rank) & 1;
+        const float a = to_f32(lat[p.rank + 2 * i]), b = to_f32(lat[p.rank + 2 * i + 1]);
+        const float2 cs = rope[i];
+        v = odd ? b * cs.x + a * cs.y : a * cs.x - b * cs.y;
+      }
+      const T o = from_f32<T>(v);
+      if (cell != nullptr) cell[c] = o;
+      if (keep != nullptr) keep[c] = o;
+    }
   }
 }
 
@@ -428,7 +454,8 @@ extern "C" int cb_latent_prep(const void* raw, int ld, int qoff, int doff, int h
   p.q_head = q_head; p.cache = cache; p.lat_p = lat_p; p.rows_out = rows_out;
   p.page_table = page_table; p.max_pages = max_pages; p.num_pages = num_pages;
   p.row_slot = row_slot; p.row_pos = row_pos; p.status = status;
-  const bool vec = dim % 8 == 0 && rot % 8 == 0 && q_head % 8 == 0 && ld % 8 == 0 && qoff % 8 == 0;
+  const bool vec = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && lat_p == rank + rot && lat_p <= 2048 &&
+                   q_head % 8 == 0 && ld % 8 == 0 && qoff % 8 == 0 && doff % 8 == 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32) {
     if (vec) latent_prep_kernel<float, 8><<<rows, 256, 0, st>>>(p);

@@ -19,10 +19,16 @@ struct MinGru {
   Entries e;
 };
 
-__device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) {
-  return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
+// two neighbouring numbers as they are stored, and as fp32
+template <typename T> struct Pair;
+template <> struct Pair<__nv_bfloat16> { using type = uint32_t; };
+template <> struct Pair<float> { using type = float2; };
+template <typename T>
+__device__ __forceinline__ typename Pair<T>::type load_pair(const T* p) {
+  return *reinterpret_cast<const typename Pair<T>::type*>(p);
 }
-__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 pair_f32(uint32_t v) { return unpack_bf16x2(v); }
+__device__ __forceinline__ float2 pair_f32(float2 v) { return v; }
 __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
   *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(a, b);
 }
@@ -66,7 +72,7 @@ __global__ void __launch_bounds__(MG_CH / 2 * MG_SEG, 4) mingru_kernel(const Min
   const ptrdiff_t ahead = static_cast<ptrdiff_t>(MG_BLOCK) * p.ld, out_ahead = static_cast<ptrdiff_t>(MG_BLOCK) * p.ldo;
   if (seg == 0)
     carry[0][cp] = in && p.e.pos0[e] > 0 ? *reinterpret_cast<const float2*>(st) : make_float2(0.f, 0.f);
-  float2 z[MG_TOK], u[MG_TOK], g[MG_TOK];
+  typename Pair<T>::type z[MG_TOK], u[MG_TOK], g[MG_TOK];
   auto fetch = [&](int n) {
     const T* r = raw;
 #pragma unroll
@@ -87,8 +93,9 @@ __global__ void __launch_bounds__(MG_CH / 2 * MG_SEG, 4) mingru_kernel(const Min
       a[i] = make_float2(1.f, 1.f);
       b[i] = act[i] = make_float2(0.f, 0.f);
       if (i < n) {
-        mg_step<T>(z[i].x, u[i].x, g[i].x, a[i].x, b[i].x, act[i].x);
-        mg_step<T>(z[i].y, u[i].y, g[i].y, a[i].y, b[i].y, act[i].y);
+        const float2 fz = pair_f32(z[i]), fu = pair_f32(u[i]), fg = pair_f32(g[i]);
+        mg_step<T>(fz.x, fu.x, fg.x, a[i].x, b[i].x, act[i].x);
+        mg_step<T>(fz.y, fu.y, fg.y, a[i].y, b[i].y, act[i].y);
       }
       tb = make_float2(a[i].x * tb.x + b[i].x, a[i].y * tb.y + b[i].y);
       ta = make_float2(ta.x * a[i].x, ta.y * a[i].y);
@@ -133,7 +140,8 @@ __global__ void __launch_bounds__(128) mingru_short_kernel(const MinGru p) {
   float2 s = p.e.pos0[e] > 0 ? *st : make_float2(0.f, 0.f);
   for (int t = 0; t < len; ++t) {
     const T* r = static_cast<const T*>(p.raw) + static_cast<size_t>(row0 + t) * p.ld + ch;
-    const float2 z = load_pair(r + p.zoff), u = load_pair(r + p.uoff), g = load_pair(r + p.goff);
+    const float2 z = pair_f32(load_pair(r + p.zoff)), u = pair_f32(load_pair(r + p.uoff)),
+                 g = pair_f32(load_pair(r + p.goff));
     float2 a, b, act;
     mg_step<T>(z.x, u.x, g.x, a.x, b.x, act.x);
     mg_step<T>(z.y, u.y, g.y, a.y, b.y, act.y);
