@@ -49,7 +49,7 @@ __global__ void __launch_bounds__(LH_WARPS * 32) linear_heads_kernel(const Heads
   }
   float acc[2][4] = {};
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll 2
+#pragma unroll 4
   for (int k0 = 0; k0 < p.K; k0 += 64) {
     uint4 a[2][2], b[2][2];
 #pragma unroll
