@@ -31,11 +31,14 @@ __device__ __forceinline__ void lh_mma(float* d, uint32_t a0, uint32_t a1, uint3
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
+// SPLIT: the warps of a block share 16 columns and take the slices of k in turn; else 16 columns each
+template <bool SPLIT>
 __global__ void __launch_bounds__(LH_WARPS * 32) linear_heads_kernel(const HeadsArgs p) {
   using bf16 = __nv_bfloat16;
+  __shared__ float red[SPLIT ? LH_WARPS : 1][8][32];
   const int h = blockIdx.y, m0 = blockIdx.z * 16, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n0 = blockIdx.x * LH_COLS + warp * 16;
-  if (n0 >= p.N) return;
+  const int n0 = SPLIT ? blockIdx.x * 16 : blockIdx.x * LH_COLS + warp * 16;
+  if (!SPLIT && n0 >= p.N) return;
   const int r = lane >> 2, t = lane & 3;
   const bf16* xp[2];
   const bf16* wp[2];
@@ -49,8 +52,9 @@ __global__ void __launch_bounds__(LH_WARPS * 32) linear_heads_kernel(const Heads
   }
   float acc[2][4] = {};
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll 4
-  for (int k0 = 0; k0 < p.K; k0 += 64) {
+  constexpr int STEP = SPLIT ? 64 * LH_WARPS : 64;
+#pragma unroll 2
+  for (int k0 = SPLIT ? warp * 64 : 0; k0 < p.K; k0 += STEP) {
     uint4 a[2][2], b[2][2];
 #pragma unroll
     for (int j = 0; j < 2; ++j)
@@ -67,6 +71,19 @@ __global__ void __launch_bounds__(LH_WARPS * 32) linear_heads_kernel(const Heads
         lh_mma(acc[j], a[0][v].x, a[1][v].x, a[0][v].y, a[1][v].y, b[j][v].x, b[j][v].y);
         lh_mma(acc[j], a[0][v].z, a[1][v].z, a[0][v].w, a[1][v].w, b[j][v].z, b[j][v].w);
       }
+  }
+  if constexpr (SPLIT) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) red[warp][j][lane] = acc[j / 4][j % 4];
+    __syncthreads();
+    if (warp != 0) return;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      float v = 0.f;
+#pragma unroll
+      for (int w = 0; w < LH_WARPS; ++w) v += red[w][j][lane];
+      acc[j / 4][j % 4] = v;
+    }
   }
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -143,7 +160,10 @@ extern "C" int cb_linear_heads(const void* x, int ldx, int x_head, const int* x_
   } else {
     const int tiles = (M + 15) / 16;
     if (tiles > 65535) return -1;
-    linear_heads_kernel<<<dim3((N + LH_COLS - 1) / LH_COLS, heads, tiles), LH_WARPS * 32, 0, st>>>(p);
+    if (K >= 64 * LH_WARPS)
+      linear_heads_kernel<true><<<dim3((N + 15) / 16, heads, tiles), LH_WARPS * 32, 0, st>>>(p);
+    else
+      linear_heads_kernel<false><<<dim3((N + LH_COLS - 1) / LH_COLS, heads, tiles), LH_WARPS * 32, 0, st>>>(p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
