@@ -164,21 +164,6 @@ __device__ __forceinline__ int latent_page(const LatentAttn& p, const int* pt, i
   return 0;
 }
 
-__device__ __forceinline__ void la_ldsm4(uint32_t* r, uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void la_ldsm4_t(uint32_t* r, uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void la_mma(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, "
-               "{%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
 constexpr int LA_WARPS = 8;
 constexpr int LA_KEYS = 8 * LA_WARPS;
 constexpr int LA_PS = LA_KEYS + 8;        // pitch of the weights (bf16)
@@ -257,11 +242,11 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_group_kernel(const Laten
 #pragma unroll 4
       for (int k = 0; k < lat32; k += 32) {
         uint32_t b[4], a[4], c[4];
-        la_ldsm4(b, smem_u32(mine + k));
-        la_ldsm4(a, smem_u32(qa + k));
-        la_ldsm4(c, smem_u32(qa + k + 16));
-        la_mma(s, a, b[0], b[1]);
-        la_mma(u, c, b[2], b[3]);
+        ldsm4(b, smem_u32(mine + k));
+        ldsm4(a, smem_u32(qa + k));
+        ldsm4(c, smem_u32(qa + k + 16));
+        mma_bf16(s, a, b[0], b[1]);
+        mma_bf16(u, c, b[2], b[3]);
       }
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
@@ -299,18 +284,18 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_group_kernel(const Laten
 #pragma unroll
     for (int k = 0; k < LA_KEYS / 16; ++k) {
       uint32_t ph[4], pl[4];
-      la_ldsm4(ph, smem_u32(sP + (lane & 15) * LA_PS + k * 16 + (lane >> 4) * 8));
-      la_ldsm4(pl, smem_u32(sP + (16 + (lane & 15)) * LA_PS + k * 16 + (lane >> 4) * 8));
+      ldsm4(ph, smem_u32(sP + (lane & 15) * LA_PS + k * 16 + (lane >> 4) * 8));
+      ldsm4(pl, smem_u32(sP + (16 + (lane & 15)) * LA_PS + k * 16 + (lane >> 4) * 8));
 #pragma unroll
       for (int a = 0; a < NV; ++a) {
         const int col = (warp * NV + a) * 16;
         if (col < p.rank) {
           uint32_t b[4];
-          la_ldsm4_t(b, smem_u32(kb + (k * 16 + (lane & 15)) * LS + col + (lane >> 4) * 8));
-          la_mma(o[a][0], ph, b[0], b[1]);
-          la_mma(o[a][1], ph, b[2], b[3]);
-          la_mma(o[a][0], pl, b[0], b[1]);
-          la_mma(o[a][1], pl, b[2], b[3]);
+          ldsm4_t(b, smem_u32(kb + (k * 16 + (lane & 15)) * LS + col + (lane >> 4) * 8));
+          mma_bf16(o[a][0], ph, b[0], b[1]);
+          mma_bf16(o[a][1], ph, b[2], b[3]);
+          mma_bf16(o[a][0], pl, b[0], b[1]);
+          mma_bf16(o[a][1], pl, b[2], b[3]);
         }
       }
     }

@@ -23,14 +23,6 @@ struct HeadsArgs {
 constexpr int LH_WARPS = 4;
 constexpr int LH_COLS = LH_WARPS * 16;
 
-__device__ __forceinline__ void lh_mma(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
-                                       uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, "
-               "{%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-
 // SPLIT: the warps of a block share 16 columns and take the slices of k in turn; else 16 columns each
 template <bool SPLIT>
 __global__ void __launch_bounds__(LH_WARPS * 32) linear_heads_kernel(const HeadsArgs p) {
@@ -68,8 +60,10 @@ __global__ void __launch_bounds__(LH_WARPS * 32) linear_heads_kernel(const Heads
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int v = 0; v < 2; ++v) {
-        lh_mma(acc[j], a[0][v].x, a[1][v].x, a[0][v].y, a[1][v].y, b[j][v].x, b[j][v].y);
-        lh_mma(acc[j], a[0][v].z, a[1][v].z, a[0][v].w, a[1][v].w, b[j][v].z, b[j][v].w);
+        const uint32_t lo[4] = {a[0][v].x, a[1][v].x, a[0][v].y, a[1][v].y};
+        const uint32_t hi[4] = {a[0][v].z, a[1][v].z, a[0][v].w, a[1][v].w};
+        mma_bf16(acc[j], lo, b[j][v].x, b[j][v].y);
+        mma_bf16(acc[j], hi, b[j][v].z, b[j][v].w);
       }
   }
   if constexpr (SPLIT) {

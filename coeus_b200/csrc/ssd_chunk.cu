@@ -21,20 +21,6 @@ constexpr int SC_TOK = 64, SC_COLS = 64, SC_WARPS = 4, SC_THREADS = SC_WARPS * 3
 constexpr int SC_XP = SC_COLS + 8;
 constexpr float SC_LOG2E = 1.4426950408889634f;
 
-__device__ __forceinline__ void sc_ldsm4(uint32_t* r, uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void sc_ldsm4_t(uint32_t* r, uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void sc_mma(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, "
-               "{%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 // (u, v) as the sum of two packed bf16 pairs
 __device__ __forceinline__ void split2(float u, float v, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(u, v);
@@ -179,14 +165,14 @@ __global__ void __launch_bounds__(SC_THREADS, 3) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
         for (int k = 0; k < NP / 16; ++k) {
           uint32_t a[4];
-          sc_ldsm4(a, smem_u32(rowsC + k * 16));
+          ldsm4(a, smem_u32(rowsC + k * 16));
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             if (j <= warp) {
               uint32_t b[4];
-              sc_ldsm4(b, smem_u32(sB + (j * 16 + (lane & 7) + (lane >> 4) * 8) * LD + k * 16 + ((lane >> 3) & 1) * 8));
-              sc_mma(G[2 * j], a, b[0], b[1]);
-              sc_mma(G[2 * j + 1], a, b[2], b[3]);
+              ldsm4(b, smem_u32(sB + (j * 16 + (lane & 7) + (lane >> 4) * 8) * LD + k * 16 + ((lane >> 3) & 1) * 8));
+              mma_bf16(G[2 * j], a, b[0], b[1]);
+              mma_bf16(G[2 * j + 1], a, b[2], b[3]);
             }
           }
         }
@@ -212,13 +198,13 @@ __global__ void __launch_bounds__(SC_THREADS, 3) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
       for (int k = 0; k < NP / 16; ++k) {                  // C . S
         uint32_t a[4];
-        sc_ldsm4(a, smem_u32(rowsC + k * 16));
+        ldsm4(a, smem_u32(rowsC + k * 16));
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           uint32_t b[4];
-          sc_ldsm4_t(b, smem_u32(sS + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
-          sc_mma(y[2 * j], a, b[0], b[1]);
-          sc_mma(y[2 * j + 1], a, b[2], b[3]);
+          ldsm4_t(b, smem_u32(sS + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
+          mma_bf16(y[2 * j], a, b[0], b[1]);
+          mma_bf16(y[2 * j + 1], a, b[2], b[3]);
         }
       }
       const float ei[2] = {sE[i0], sE[i0 + 8]};
@@ -232,9 +218,9 @@ __global__ void __launch_bounds__(SC_THREADS, 3) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             uint32_t b[4];
-            sc_ldsm4_t(b, smem_u32(sX + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
-            sc_mma(y[2 * j], m[k], b[0], b[1]);
-            sc_mma(y[2 * j + 1], m[k], b[2], b[3]);
+            ldsm4_t(b, smem_u32(sX + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
+            mma_bf16(y[2 * j], m[k], b[0], b[1]);
+            mma_bf16(y[2 * j + 1], m[k], b[2], b[3]);
           }
         }
       }
@@ -275,7 +261,7 @@ __global__ void __launch_bounds__(SC_THREADS, 3) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
       for (int a = 0; a < RT; ++a) {
         uint32_t m[4];
-        sc_ldsm4_t(m, smem_u32(sB + (k * 16 + (lane >> 4) * 8 + (lane & 7)) * LD + (warp + 4 * a) * 16 +
+        ldsm4_t(m, smem_u32(sB + (k * 16 + (lane >> 4) * 8 + (lane & 7)) * LD + (warp + 4 * a) * 16 +
                                ((lane >> 3) & 1) * 8));
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
@@ -286,13 +272,13 @@ __global__ void __launch_bounds__(SC_THREADS, 3) ssd_chunk_kernel(const Ssd p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         uint32_t b[4];
-        sc_ldsm4_t(b, smem_u32(sX + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
+        ldsm4_t(b, smem_u32(sX + (k * 16 + (lane & 15)) * SC_XP + j * 16 + (lane >> 4) * 8));
 #pragma unroll
         for (int a = 0; a < RT; ++a) {
-          sc_mma(S[a][2 * j], hi[a], b[0], b[1]);
-          sc_mma(S[a][2 * j + 1], hi[a], b[2], b[3]);
-          sc_mma(S[a][2 * j], lo[a], b[0], b[1]);
-          sc_mma(S[a][2 * j + 1], lo[a], b[2], b[3]);
+          mma_bf16(S[a][2 * j], hi[a], b[0], b[1]);
+          mma_bf16(S[a][2 * j + 1], hi[a], b[2], b[3]);
+          mma_bf16(S[a][2 * j], lo[a], b[0], b[1]);
+          mma_bf16(S[a][2 * j + 1], lo[a], b[2], b[3]);
         }
       }
     }

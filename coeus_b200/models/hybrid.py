@@ -26,6 +26,7 @@ from ..foundation.error import ConfigError, ProcessingError
 MAX_HEAD_DIM = 256           # the attention and recurrence kernels' limit per head
 MAX_LATENT = 640             # and per cached latent row
 MAX_TAPS = 17                # and of the convolution kernels
+MAX_WIDTH = 16384            # and of the pass between two sublayers
 DEFAULT_MAX_SEQ_LEN = 8192   # serving default; the designs themselves have no length limit
 
 Shapes = Dict[str, Tuple[int, ...]]
@@ -366,6 +367,8 @@ class HybridConfig:
             _refuse("architecture", self.architecture, f"Known designs: {', '.join(DESIGNS)}")
         if self.vocab_size < 1 or self.hidden_dim < 1 or not self.layers:
             _refuse("layers", self.num_layers, "A model needs a vocabulary, a width and layers")
+        if self.hidden_dim > MAX_WIDTH:
+            _refuse("width", self.hidden_dim, f"The width must not exceed {MAX_WIDTH}")
         mixing = None
         for i, layer in enumerate(self.layers):
             m = layer.mixer
