@@ -16,7 +16,9 @@ import numpy as np
 import torch
 
 from ..foundation.error import ProcessingError
-from ..models.hybrid import CACHED, AttentionSpec, HybridLM, LatentAttentionSpec, Mamba2Spec
+from ..models.hybrid import (CACHED, AttentionSpec, HeadAttentionSpec, HybridLM, LatentAttentionSpec,
+                             Mamba2Spec)
+from ..ops import experts as X
 from ..ops import gemm as G
 from ..ops import latent as L
 from ..ops import ragged as R
@@ -57,6 +59,9 @@ class HybridEngine(InferenceEngine):
     def _plan(self, a) -> R.AttnPlan:
         if isinstance(a, AttentionSpec):
             return R.AttnPlan(a.chunk, self._tiles and R.pieces_allowed(a.dim, a.vdim, a.chunk, a.scale))
+        if isinstance(a, HeadAttentionSpec):
+            return R.AttnPlan(None, self._tiles and R.pieces_allowed(a.dim, a.vdim, None, a.scale), a.window,
+                              tiles=True)
         return R.AttnPlan(None, self._tiles and L.pieces_allowed(a.dim + a.rot_dim, a.vdim, a.scale),
                           a.window or 1 << 30)
 
@@ -78,8 +83,11 @@ class HybridEngine(InferenceEngine):
             a = m.layers[run.layer].spec.mixer
             if isinstance(a, CACHED):
                 self._cache_index[n] = len(dims)
-                dims.append((a.kv_heads, _up8(a.dim), _up8(a.vdim)) if isinstance(a, AttentionSpec)
-                            else (1, _up8(a.latent), 0))
+                if isinstance(a, LatentAttentionSpec):
+                    dims.append((1, _up8(a.latent), 0))
+                else:
+                    maps = getattr(a, "maps", 1)       # every map has a key of its own, values are shared
+                    dims.append((a.kv_heads, _up8(a.dim), _up8(a.vdim), a.kv_heads * maps))
         self.cache = PagedKVCache(len(dims), 0, 0, num_pages or max_seqs * per_seq, max_seqs,
                                   per_seq, m.device, m.dtype, layer_dims=dims)
         self.state = SequenceState(max_seqs, m.device)
@@ -158,6 +166,48 @@ class HybridEngine(InferenceEngine):
         R.gated_head_norm(o, gate, layer.head_norm, self.cfg.norm_eps, cat[:, :layer.out_dim])
 
     # the mixers of a sequential block fill ``out``, the columns in front of their output projection
+    def _heads(self, n: int, layer, raw: torch.Tensor, out: torch.Tensor, b: R.RaggedBatch, rope: dict,
+               max_ctx: int) -> None:
+        s, c, i = layer.spec.mixer, self.cache, self._cache_index[n]
+        eps, plan, kh = self.cfg.norm_eps, self._plan(s), s.kv_heads * s.maps
+        key_rows, k_rows, v_rows, q_head = b.kv_rows(plan), None, None, None
+        if key_rows:        # the heads' distance in the row-wise buffers of the piece kernel
+            q_head, v_head = R.row_heads(s.dim, s.vdim, s.maps)
+            k_rows, v_rows = (torch.empty((key_rows, h, p), dtype=raw.dtype, device=raw.device)
+                              for h, p in ((kh, q_head), (s.kv_heads, v_head)))
+        q = R.head_prep(raw, layer.seg["k"], layer.seg["v"], s.heads * s.maps, kh, s.dim, s.vdim, b,
+                        rope.get(layer.rope_key), c.k[i], c.v[i], c.page_table, interleaved=s.interleaved,
+                        unit_eps=eps if s.unit_qk else None, q_head=q_head, k_rows=k_rows, v_rows=v_rows)
+        R.ragged_attention(
+            q, c.k[i], c.v[i], c.page_table, b, s.heads, s.kv_heads, s.dim, s.vdim, s.scale,
+            out[:, :layer.out_dim], window=s.window, softcap=s.softcap, maps=s.maps,
+            map_weight=layer.map_weight, map_factor=1.0 - s.diff if s.maps == 2 else 1.0, eps=eps,
+            gate=raw[:, layer.seg["g"]:] if s.gated else None, gate_wide=True, max_ctx=max_ctx,
+            k_rows=k_rows, v_rows=v_rows, plan=plan)
+
+    def _experts(self, layer, h: torch.Tensor) -> dict:
+        """The mixture of experts of ``h``, as what the next pass over the stream adds."""
+        e, m = layer.experts, layer.experts.spec
+        r = X.Routing(m.experts, m.top, m.groups, m.keep, m.scale)
+        c = X.route(h, e.router, r)
+        shared = m.shared is not None
+        if h.is_cuda and h.dtype == torch.bfloat16 and h.shape[0] <= X.FEW:
+            return dict(y=X.experts_few(h, c, r, e.w_in, e.w_down, m.expert.limit, e.s_in, e.s_down,
+                                        m.shared.limit if shared else 0.0, e.slope))
+
+        def rows(n, w):
+            return torch.empty((n, w), dtype=h.dtype, device=h.device)
+        s = X.sort_rows(h, c, r)
+        n = s.rows.shape[0]
+        act = X.grouped_linear(s.rows, e.w_in, s.block_expert, rows(n, e.w_in.shape[1] // 2),
+                               glu=(e.slope, m.expert.limit))
+        res = X.grouped_linear(act, e.w_down, s.block_expert, rows(n, e.wp))
+        add = dict(spread=R.Spread(res, s.slot, c.weight))
+        if shared:
+            act = G.linear(h, e.s_in, rows(h.shape[0], e.s_in.shape[0] // 2), glu=(e.slope, m.shared.limit))
+            add["y"] = self._product(act, e.s_down)
+        return add
+
     def _latent(self, n: int, layer, raw: torch.Tensor, out: torch.Tensor, b: R.RaggedBatch,
                 rope: dict, max_ctx: int) -> None:
         s, m, seg = layer.spec.mixer, self.m, layer.seg
@@ -269,12 +319,16 @@ class HybridEngine(InferenceEngine):
             out = torch.empty((b.T, layer.act_off), dtype=dt, device=m.device)
             if layer.out_dim != layer.act_off:
                 out[:, layer.out_dim:].zero_()
-            if isinstance(layer.spec.mixer, LatentAttentionSpec):
-                self._latent(n, layer, raw, out, b, rope, max_ctx)
+            if isinstance(layer.spec.mixer, (HeadAttentionSpec, LatentAttentionSpec)):
+                mix = self._heads if isinstance(layer.spec.mixer, HeadAttentionSpec) else self._latent
+                mix(n, layer, raw, out, b, rope, max_ctx)
             else:
                 {"mamba2": self._mamba2, "mingru": self._mingru}[layer.spec.mixer.kind](n, layer, raw, out, b)
             add = dict(y=self._product(out, layer.w_out), post=layer.norm1b)
-            if layer.w_up is not None:
+            if layer.experts is not None:
+                x, h = R.add_norm(x, W, eps, dt, gain=layer.norm2, **add)
+                add = dict(post=layer.norm2b, **self._experts(layer, h))
+            elif layer.w_up is not None:
                 x, h = R.add_norm(x, W, eps, dt, gain=layer.norm2, **add)
                 act = torch.empty((b.T, layer.ff_padded), dtype=dt, device=m.device)
                 G.linear(h, layer.w_up, act, epi=cfg.design.act, bias=layer.b_up)

@@ -18,18 +18,18 @@ from ..ops.decode import PAGE
 class PagedKVCache:
     def __init__(self, num_layers: int, num_heads: int, head_dim: int, num_pages: int,
                  max_seqs: int, max_pages_per_seq: int, device, dtype=torch.bfloat16,
-                 layer_dims: Optional[Sequence[Tuple[int, int, int]]] = None) -> None:
-        """``layer_dims``: ``(heads, key size, value size)`` of every cached layer where they
-        differ between layers or between keys and values (``num_layers`` entries)."""
+                 layer_dims: Optional[Sequence[Tuple[int, ...]]] = None) -> None:
+        """``layer_dims``: ``(heads, key size, value size[, heads of the keys])`` of every cached layer
+        where they differ between layers or between keys and values (``num_layers`` entries)."""
         self.num_layers, self.nh, self.dh = num_layers, num_heads, head_dim
         self.num_pages = num_pages
         self.device = torch.device(device)
         dims = list(layer_dims) if layer_dims is not None else \
             [(num_heads, head_dim, head_dim)] * num_layers
-        self.k = [torch.zeros((num_pages, PAGE, h, dk), dtype=dtype, device=self.device)
-                  for h, dk, _ in dims]
-        self.v = [torch.zeros((num_pages, PAGE, h, dv), dtype=dtype, device=self.device)
-                  for h, _, dv in dims]
+        self.k = [torch.zeros((num_pages, PAGE, d[3] if len(d) > 3 else d[0], d[1]), dtype=dtype,
+                              device=self.device) for d in dims]
+        self.v = [torch.zeros((num_pages, PAGE, d[0], d[2]), dtype=dtype, device=self.device)
+                  for d in dims]
         self.page_table = torch.zeros((max_seqs, max_pages_per_seq), dtype=torch.int32,
                                       device=self.device)
         self.free: List[int] = list(range(num_pages - 1, -1, -1))

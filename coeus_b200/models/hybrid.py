@@ -13,6 +13,9 @@ What a design fixes for all its models is a :class:`Design`; the mixers are open
 * Bananex: norms before and after each sublayer, a token shift in front of every mixer, a run of
   layers that is looped with the embedding fed in again, and latent attention under a sliding
   window, Mamba-2 and minGRU layers.
+* Rupasun: norms before and after each sublayer, differential attention over the whole context,
+  attention under a sliding window with normalised queries and keys, capped scores and an output
+  gate, and feed-forwards that are dense or a mixture of experts with a shared one.
 """
 from __future__ import annotations
 
@@ -27,6 +30,7 @@ MAX_HEAD_DIM = 256           # the attention and recurrence kernels' limit per h
 MAX_LATENT = 640             # and per cached latent row
 MAX_TAPS = 17                # and of the convolution kernels
 MAX_WIDTH = 16384            # and of the pass between two sublayers
+MAX_EXPERTS, MAX_TOP = 256, 16   # and of the routing kernels
 DEFAULT_MAX_SEQ_LEN = 8192   # serving default; the designs themselves have no length limit
 
 Shapes = Dict[str, Tuple[int, ...]]
@@ -37,21 +41,32 @@ class Design:
     """The constants of a design."""
 
     name: str
-    mixers: Tuple[str, ...]
+    mixers: Mapping[str, str]    # type of a layer in a configuration file -> kind of mixer
     parallel: bool           # mixer and feed-forward side by side on one stream, else one by one
     post_norms: bool         # sublayer results are normalised before they are added
     scalar_norms: bool       # the gain of a norm of the stream is one number
     embed_norm: bool
     token_shift: bool
-    act: str                 # of the feed-forward
+    act: str                 # of the dense feed-forward
     mlp_bias: bool
+    mlps: Tuple[str, ...] = ("dense",)
+    glu_slope: float = 1.0   # of the sigmoid in the experts' gated unit
+    scaled_logits: bool = False
+
+
+def _same(*kinds: str) -> Dict[str, str]:
+    return {k: k for k in kinds}
 
 
 DESIGNS = {d.name: d for d in (
-    Design("Sapasun", ("attention", "channel_delta"), parallel=True, post_norms=False,
+    Design("Sapasun", _same("attention", "channel_delta"), parallel=True, post_norms=False,
            scalar_norms=False, embed_norm=True, token_shift=False, act="relu2", mlp_bias=False),
-    Design("Bananex", ("latent_attention", "mamba2", "mingru"), parallel=False, post_norms=True,
-           scalar_norms=True, embed_norm=False, token_shift=True, act="gelu_erf", mlp_bias=True),
+    Design("Bananex", _same("latent_attention", "mamba2", "mingru"), parallel=False, post_norms=True,
+           scalar_norms=True, embed_norm=False, token_shift=True, act="gelu_erf", mlp_bias=True,
+           scaled_logits=True),
+    Design("Rupasun", {"attention": "diff_attention", "attention_2": "capped_attention"}, parallel=False,
+           post_norms=True, scalar_norms=False, embed_norm=False, token_shift=False, act="relu2",
+           mlp_bias=False, mlps=("dense", "moe"), glu_slope=1.702),
 )}
 ARCHITECTURES = tuple(DESIGNS)
 
@@ -292,22 +307,211 @@ class MinGruSpec:
         return self.width
 
 
-MixerSpec = Union[AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, Mamba2Spec, MinGruSpec]
+@dataclass(frozen=True)
+class HeadAttentionSpec:
+    """Softmax attention of rotated heads straight from the projections.  What a kind fixes are class
+    attributes, what its models choose are fields."""
+
+    kind: ClassVar[str]
+    maps: ClassVar[int] = 1             # attention maps per head, over the same values
+    interleaved: ClassVar[bool] = False  # rotated pairs are neighbours, else half a rotation apart
+    unit_qk: ClassVar[bool] = False     # rotated queries and keys are divided by their root mean square
+    gated: ClassVar[bool] = False       # the output times the sigmoid of a projection, number by number
+
+    heads: int
+    kv_heads: int
+    dim: int                 # query/key size per head and map
+    vdim: int
+    scale: float
+    rot_dims: int
+    rot_base: float
+    window: Optional[int] = None        # a position sees itself and window - 1 before it
+    softcap: Optional[float] = None     # scores s become softcap * tanh(s / softcap)
+    diff: Optional[float] = None        # two maps: what their weights add to
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any], shapes: Mapping[str, Any], p: str) -> "HeadAttentionSpec":
+        rot, mask, cap = m.get("rot"), m.get("mask"), m.get("softcap")
+        return cls(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                   vdim=int(m["vdim"]), scale=float(m["scale"]), rot_dims=int(rot["dims"]) if rot else 0,
+                   rot_base=float(rot["base"]) if rot else 1.0,
+                   window=int(mask["size"]) if mask else None,
+                   softcap=None if cap is None else float(cap),
+                   diff=float(m["diff"]) if cls.maps == 2 else None)
+
+    def to_json(self) -> Dict[str, Any]:
+        out: Dict[str, Any] = dict(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim,
+                                   vdim=self.vdim, scale=self.scale)
+        if self.rot_dims:
+            out["rot"] = {"base": self.rot_base, "dims": self.rot_dims}
+        if self.window is not None:
+            out["mask"] = {"size": self.window}
+        if self.softcap is not None:
+            out["softcap"] = self.softcap
+        if self.diff is not None:
+            out["diff"] = self.diff
+        return out
+
+    def check(self, where: str) -> None:
+        if self.kv_heads < 1 or self.heads < 1 or self.heads % self.kv_heads:
+            _refuse(where, f"{self.heads}/{self.kv_heads}",
+                    "Key/value heads must divide the number of heads")
+        _heads_ok(where, self.dim, self.vdim)
+        if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim:
+            _refuse(where, self.rot_dims, "Rotated dimensions must be even and fit the head")
+        if self.window is not None and self.window < 1:
+            _refuse(where, self.window, "A window has at least one position")
+        if self.softcap is not None and not self.softcap > 0:
+            _refuse(where, self.softcap, "A cap of scores is positive")
+        if (self.diff is not None) != (self.maps == 2):
+            _refuse(where, self.diff, "Two maps, and only two, need the constant of their difference")
+
+    def tensors(self, W: int) -> Shapes:
+        out: Shapes = {"q": (self.heads * self.maps * self.dim, W),
+                       "k": (self.kv_heads * self.maps * self.dim, W), "v": (self.kv_heads * self.vdim, W)}
+        if self.maps == 2:
+            out.update({n: (self.dim,) for n in MAP_VECTORS})
+        if self.gated:
+            out["g"] = (self.out_dim, W)
+        return out
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+MAP_VECTORS = ("lq1", "lk1", "lq2", "lk2")    # exp(lq1 . lk1) - exp(lq2 . lk2) + diff weighs the second map
+
+
+@dataclass(frozen=True)
+class DiffAttentionSpec(HeadAttentionSpec):
+    """Two maps over the same values; the head is their weighted difference, divided by its root mean
+    square, times ``1 - diff``."""
+
+    kind: ClassVar[str] = "diff_attention"
+    maps: ClassVar[int] = 2
+
+
+@dataclass(frozen=True)
+class CappedAttentionSpec(HeadAttentionSpec):
+    kind: ClassVar[str] = "capped_attention"
+    interleaved: ClassVar[bool] = True
+    unit_qk: ClassVar[bool] = True
+    gated: ClassVar[bool] = True
+
+
+MixerSpec = Union[AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, Mamba2Spec, MinGruSpec,
+                  HeadAttentionSpec]
 MIXERS = {c.kind: c for c in (AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, Mamba2Spec,
-                              MinGruSpec)}
-CACHED = (AttentionSpec, LatentAttentionSpec)    # mixers that look back through the paged cache
+                              MinGruSpec, DiffAttentionSpec, CappedAttentionSpec)}
+# mixers that look back through the paged cache
+CACHED = (AttentionSpec, LatentAttentionSpec, HeadAttentionSpec)
 
 
 @dataclass(frozen=True)
 class MlpSpec:
+    """down(act(up))."""
+
+    kind: ClassVar[str] = "dense"
     ff: int
-    kind: str = "dense"      # down(act(up))
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any]) -> "MlpSpec":
+        return cls(ff=int(m["ff"]))
+
+    def to_json(self) -> Dict[str, Any]:
+        return dict(kind=self.kind, ff=self.ff)
+
+    def check(self, where: str) -> None:
+        if self.ff < 1:
+            _refuse(where, self.ff, "A feed-forward has at least one channel")
+
+    def tensors(self, W: int, bias: bool) -> Shapes:
+        out: Shapes = {"up": (self.ff, W), "down": (W, self.ff)}
+        if bias:
+            out.update({"up.b": (self.ff,), "down.b": (W,)})
+        return out
+
+
+@dataclass(frozen=True)
+class GluSpec:
+    """An expert: ``down(g * sigmoid(slope * g) * (u + 1))``, ``g`` bounded by ``limit`` above and ``u``
+    on both sides."""
+
+    ff: int
+    limit: float
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any]) -> "GluSpec":
+        return cls(ff=int(m["ff"]), limit=float(m["limit"]))
+
+    def tensors(self, W: int, p: str) -> Shapes:
+        return {p + "gate": (self.ff, W), p + "up": (self.ff, W), p + "down": (W, self.ff)}
+
+
+@dataclass(frozen=True)
+class MoeSpec:
+    """Every token uses the ``top`` of ``experts`` with the largest sigmoid scores among the ``keep`` best
+    of ``groups`` equal groups of neighbours (a group counts the sum of its two largest), weighted by
+    their scores over the scores' sum, times ``scale``; and the shared expert, if there is one."""
+
+    kind: ClassVar[str] = "moe"
+    experts: int
+    top: int
+    expert: GluSpec
+    scale: float = 1.0
+    groups: int = 1
+    keep: int = 1
+    shared: Optional[GluSpec] = None
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any]) -> "MoeSpec":
+        r = m["router"]
+        groups = r.get("groups") or {"count": 1, "keep": 1}
+        return cls(experts=int(r["experts"]), top=int(r["top"]), expert=GluSpec.read(m["expert"]),
+                   scale=float(r.get("scale", 1.0)), groups=int(groups["count"]), keep=int(groups["keep"]),
+                   shared=GluSpec.read(m["shared"]) if m.get("shared") else None)
+
+    def to_json(self) -> Dict[str, Any]:
+        def glu(g: GluSpec) -> Dict[str, Any]:
+            return dict(ff=g.ff, limit=g.limit)
+        out: Dict[str, Any] = dict(
+            kind=self.kind, expert=glu(self.expert),
+            router=dict(experts=self.experts, top=self.top, scale=self.scale,
+                        groups=dict(count=self.groups, keep=self.keep)))
+        if self.shared is not None:
+            out["shared"] = glu(self.shared)
+        return out
+
+    def check(self, where: str) -> None:
+        if not 1 <= self.experts <= MAX_EXPERTS or not 1 <= self.top <= MAX_TOP:
+            _refuse(where, f"{self.top} of {self.experts}",
+                    f"Up to {MAX_TOP} of up to {MAX_EXPERTS} experts are chosen")
+        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            _refuse(where, f"{self.keep} of {self.groups}", "Groups must be equal, and one of them kept")
+        if self.top > self.keep * (self.experts // self.groups):
+            _refuse(where, self.top, "The kept groups must hold enough experts")
+        for g in (self.expert, self.shared):
+            if g is not None and (g.ff < 1 or not g.limit > 0):
+                _refuse(where, f"{g.ff}/{g.limit}", "An expert has a channel and a positive limit")
+
+    def tensors(self, W: int, bias: bool) -> Shapes:
+        out: Shapes = {"router": (self.experts, W)}
+        for e in range(self.experts):
+            out.update(self.expert.tensors(W, f"e{e}."))
+        if self.shared is not None:
+            out.update(self.shared.tensors(W, "shared."))
+        return out
+
+
+FeedForwardSpec = Union[MlpSpec, MoeSpec]
+MLPS = {c.kind: c for c in (MlpSpec, MoeSpec)}
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
-    mlp: Optional[MlpSpec]
+    mlp: Optional[FeedForwardSpec]
 
 
 @dataclass(frozen=True)
@@ -373,16 +577,19 @@ class HybridConfig:
         for i, layer in enumerate(self.layers):
             m = layer.mixer
             where = f"layers[{i}].mixer"
-            if m.kind not in self.design.mixers:
-                _refuse(where, m.kind, f"{self.architecture} has {', '.join(self.design.mixers)}")
+            if m.kind not in self.design.mixers.values():
+                _refuse(where, m.kind, f"{self.architecture} has {', '.join(self.design.mixers.values())}")
             m.check(where)
             if getattr(m, "v_mix", False):
                 size = m.kv_heads * m.vdim
                 if mixing not in (None, size):
                     _refuse(where, size, "Layers that mix values must agree in their size")
                 mixing = size
-            if layer.mlp is not None and (layer.mlp.kind != "dense" or layer.mlp.ff < 1):
-                _refuse(f"layers[{i}].mlp", layer.mlp.kind, "Feed-forward kind must be 'dense'")
+            if layer.mlp is not None:
+                if layer.mlp.kind not in self.design.mlps:
+                    _refuse(f"layers[{i}].mlp", layer.mlp.kind,
+                            f"Feed-forwards of {self.architecture}: {', '.join(self.design.mlps)}")
+                layer.mlp.check(f"layers[{i}].mlp")
         if self.loop is not None:
             lo = self.loop
             if self.design.parallel:
@@ -408,33 +615,38 @@ def config_from_json(config: Mapping[str, Any], shapes: Mapping[str, Any]) -> Hy
     """``config``: the parsed ``config.json``; ``shapes``: tensor name -> shape, which gives the
     sizes the file does not name (the inner widths of the factored projections)."""
     layers = []
+    architecture = str(config.get("architecture", "Sapasun"))
+    if architecture not in DESIGNS:
+        raise ProcessingError.unsupported(f"architecture '{architecture}'", ", ".join(DESIGNS))
+    kinds = DESIGNS[architecture].mixers
     for i, entry in enumerate(config["layers"]):
-        if entry["type"] not in MIXERS:
-            raise ProcessingError.unsupported(f"mixer type '{entry['type']}'", ", ".join(MIXERS))
-        mixer = MIXERS[entry["type"]].read(entry["mixer"], shapes, f"l{i}.mix.")
+        if entry["type"] not in kinds:
+            raise ProcessingError.unsupported(f"mixer type '{entry['type']}'", ", ".join(kinds))
+        mixer = MIXERS[kinds[entry["type"]]].read(entry["mixer"], shapes, f"l{i}.mix.")
         mlp = entry.get("mlp")
-        layers.append(LayerSpec(mixer, None if mlp is None else
-                                MlpSpec(ff=int(mlp["ff"]), kind=str(mlp["kind"]))))
+        if mlp and mlp["kind"] not in MLPS:
+            raise ProcessingError.unsupported(f"feed-forward '{mlp['kind']}'", ", ".join(MLPS))
+        layers.append(LayerSpec(mixer, MLPS[mlp["kind"]].read(mlp) if mlp else None))
     cap, loop = config.get("logit_softcap"), config.get("loop")
     cfg = HybridConfig(
         vocab_size=int(config["vocab"]), hidden_dim=int(config["width"]), layers=tuple(layers),
         norm_eps=float(config["norm"]["eps"]), logit_softcap=None if cap is None else float(cap),
-        architecture=str(config.get("architecture", "Sapasun")),
-        logit_scale=float(config.get("logit_scale", 1.0)),
+        architecture=architecture,
+        logit_scale=float(config.get("logit_scale", 1.0)) if DESIGNS[architecture].scaled_logits else 1.0,
         loop=None if not loop else LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"])))
     cfg.validate()
     return cfg
 
 
 def config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
-    layers = [{"type": layer.mixer.kind, "mixer": layer.mixer.to_json(),
-               "mlp": None if layer.mlp is None else {"kind": layer.mlp.kind, "ff": layer.mlp.ff}}
-              for layer in cfg.layers]
+    types = {kind: name for name, kind in cfg.design.mixers.items()}
+    layers = [{"type": types[layer.mixer.kind], "mixer": layer.mixer.to_json(),
+               "mlp": None if layer.mlp is None else layer.mlp.to_json()} for layer in cfg.layers]
     out = {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_dim,
            "norm": {"eps": cfg.norm_eps}, "layers": layers}
     if cfg.design.parallel:
         out["logit_softcap"] = cfg.logit_softcap
-    else:
+    elif cfg.design.scaled_logits:
         out["logit_scale"] = cfg.logit_scale
     if cfg.loop is not None:
         out["loop"] = {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times}
@@ -461,10 +673,7 @@ def tensor_shapes(cfg: HybridConfig) -> Shapes:
         out.update({f"{p}mix.{n}": s for n, s in layer.mixer.tensors(W).items()})
         out[p + "mix.o"] = (W, layer.mixer.out_dim)
         if layer.mlp is not None:
-            out[p + "mlp.up"] = (layer.mlp.ff, W)
-            out[p + "mlp.down"] = (W, layer.mlp.ff)
-            if d.mlp_bias:
-                out.update({p + "mlp.up.b": (layer.mlp.ff,), p + "mlp.down.b": (W,)})
+            out.update({f"{p}mlp.{n}": s for n, s in layer.mlp.tensors(W, d.mlp_bias).items()})
     out.update({"final.norm": norm, "head": (V, W)})
     return out
 
@@ -489,7 +698,7 @@ def random_state(cfg: HybridConfig, seed: int = 0, device="cpu",
             t = normal(shape, 1.0)
         elif leaf in ("sink", "vmix", "A_log", "dt_bias"):
             t = normal(shape, 0.5)
-        elif leaf == "step" or (leaf == "b" and len(shape) == 1):
+        elif leaf in MAP_VECTORS or leaf == "step" or (leaf == "b" and len(shape) == 1):
             t = normal(shape, 0.2)
         elif leaf == "shift":
             t = torch.sigmoid(normal(shape, 1.0))
@@ -503,6 +712,37 @@ def _pad(t: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
     out = torch.zeros((rows, cols), dtype=t.dtype, device=t.device)
     out[:t.shape[0], :t.shape[1]] = t
     return out
+
+
+class Experts:
+    """Device weights of a mixture of experts.  Rows of gate and up alternate (``w_in [experts, 2 ff, W]``),
+    so that a tile of the product has both numbers of a channel; ``w_down [experts, W, ff]``; the shared
+    expert's ``s_in`` and ``s_down`` likewise."""
+
+    def __init__(self, spec: MoeSpec, slope: float, mat, wp: int) -> None:
+        self.spec, self.slope, self.wp = spec, slope, wp
+        self.router = _pad(mat("mlp.router"), _up8(spec.experts), wp)
+
+        def pair(p: str, g: GluSpec):
+            n = _up8(g.ff)
+            w = torch.stack([_pad(mat(p + "gate"), n, wp), _pad(mat(p + "up"), n, wp)], 1)
+            return w.view(2 * n, wp), _pad(mat(p + "down"), wp, n)
+        ws = [pair(f"mlp.e{e}.", spec.expert) for e in range(spec.experts)]
+        self.w_in, self.w_down = (torch.stack(t).contiguous() for t in zip(*ws))
+        self.s_in, self.s_down = pair("mlp.shared.", spec.shared) if spec.shared else (None, None)
+
+    def tensors(self, W: int) -> Dict[str, torch.Tensor]:
+        s = self.spec
+        out = {"router": self.router[:s.experts, :W]}
+
+        def apart(p: str, w_in: torch.Tensor, down: torch.Tensor, ff: int) -> None:
+            out.update({p + "gate": w_in[0:2 * ff:2, :W], p + "up": w_in[1:2 * ff:2, :W],
+                        p + "down": down[:W, :ff]})
+        for e in range(s.experts):
+            apart(f"e{e}.", self.w_in[e], self.w_down[e], s.expert.ff)
+        if s.shared is not None:
+            apart("shared.", self.s_in, self.s_down, s.shared.ff)
+        return out
 
 
 class HybridLayer:
@@ -523,16 +763,20 @@ class HybridLayer:
         self.shift = self._vec("shift", self.wp) if design.token_shift else None
         self.seg: Dict[str, int] = {}
         {"attention": self._attention, "channel_delta": self._channel_delta,
-         "latent_attention": self._latent, "mamba2": self._mamba2,
-         "mingru": self._mingru}[spec.mixer.kind](spec.mixer)
+         "latent_attention": self._latent, "mamba2": self._mamba2, "mingru": self._mingru,
+         "diff_attention": self._heads, "capped_attention": self._heads}[spec.mixer.kind](spec.mixer)
         self.out_dim = spec.mixer.out_dim
         self.act_off = _up8(self.out_dim)
         outs = [_pad(self._mat("mix.o"), self.wp, self.act_off)]
         self.norm2 = self.norm2b = self.w_up = self.b_up = self.w_down = self.b_down = None
         self.ff = self.ff_padded = 0
+        self.experts: Optional[Experts] = None
         if spec.mlp is not None:
             self.norm2 = self._gain("norm2", design)
             self.norm2b = self._gain("norm2b", design) if design.post_norms else None
+        if isinstance(spec.mlp, MoeSpec):
+            self.experts = Experts(spec.mlp, design.glu_slope, self._mat, self.wp)
+        elif spec.mlp is not None:
             self.ff, self.ff_padded = spec.mlp.ff, _up8(spec.mlp.ff)
             self.w_up = _pad(self._mat("mlp.up"), self.ff_padded, self.wp)
             down = _pad(self._mat("mlp.down"), self.wp, self.ff_padded)
@@ -628,6 +872,15 @@ class HybridLayer:
         self._stack({n: self._mat("mix." + n) for n in ("z", "x", "g")},
                     {n: self._get(f"mix.{n}.b") for n in ("z", "x")})
 
+    def _heads(self, m: HeadAttentionSpec) -> None:
+        self._stack({n: self._mat("mix." + n) for n in (("q", "k", "v", "g") if m.gated else ("q", "k", "v"))})
+        self.rope_key = (m.rot_base, m.rot_dims) if m.rot_dims else None
+        self.map_vectors = self.map_weight = None
+        if m.maps == 2:
+            self.map_vectors = {n: self._vec("mix." + n) for n in MAP_VECTORS}
+            a, b, c, d = (self.map_vectors[n].double() for n in MAP_VECTORS)
+            self.map_weight = ((a * b).sum().exp() - (c * d).sum().exp() + m.diff).float().reshape(1)
+
     # ------------------------------------------------------------------ taken apart again
     def tensors(self, width: int) -> Dict[str, torch.Tensor]:
         """The layer's tensors under their names in a checkpoint (without the layer's prefix)."""
@@ -668,6 +921,9 @@ class HybridLayer:
             out.update({"mix.conv": self.conv[:, idx].t(), "mix.conv.b": self.conv_b[idx],
                         "mix.dt_bias": self.dt_bias, "mix.A_log": self.A_log, "mix.D": self.D,
                         "mix.norm": self.out_norm})
+        elif isinstance(m, HeadAttentionSpec):
+            stacked(n for n in ("q", "k", "v", "g") if n in shapes)
+            out.update({"mix." + n: t for n, t in (self.map_vectors or {}).items()})
         else:
             stacked(("z", "x", "g"))
             for n in ("z", "x"):
@@ -675,6 +931,8 @@ class HybridLayer:
         for n in ("norm1b", "norm2", "norm2b", "shift"):
             if getattr(self, n) is not None:
                 out[n] = getattr(self, n)
+        if self.experts is not None:
+            out.update({"mlp." + n: t for n, t in self.experts.tensors(W).items()})
         if self.w_up is not None:
             out["mlp.up"] = self.w_up[:self.ff, :W]
             out["mlp.down"] = self.w_out[:W, self.act_off:self.act_off + self.ff] \

@@ -1,0 +1,177 @@
+"""Mixture of experts of the serving step (``csrc/experts.cu``): routing by sigmoid scores among the best
+groups, without a capacity (every chosen expert runs), and experts whose gated unit is bounded.
+
+Few rows stream the weights of the chosen experts (:func:`experts_few`).  Larger batches are sorted by
+expert into a buffer whose experts start at multiples of ``BLOCK`` rows, and the experts' products are one
+grouped launch each (:func:`route`, :func:`sort_rows`, :func:`grouped_linear`); the results leave through
+:class:`coeus_b200.ops.ragged.Spread`.
+
+CPU tensors take a PyTorch restatement of the same math; CUDA tensors always run the kernels.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import Optional, Tuple
+
+import torch
+
+from . import _lib
+from .gemm import clamped_glu
+
+BLOCK = 128           # rows of one expert's tile
+FEW = 16              # rows up to which the experts' weights are streamed
+ROUTE_FEW = 128       # rows up to which the router's product and the choice are one launch
+ROUTE_TOKENS = 32     # tokens per block of the choice otherwise
+_F = ctypes.c_float
+
+
+def _p(t):
+    return _lib.ptr(t)
+
+
+@dataclass(frozen=True)
+class Routing:
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+
+
+@dataclass
+class Choice:
+    """``expert`` (int32) and ``weight`` (fp32) ``[tokens, top]``; on the GPU also what sorting needs: the
+    tokens of a block, the rank of a pair among its block's of the same expert, the blocks' counts."""
+
+    expert: torch.Tensor
+    weight: torch.Tensor
+    per_block: int = 0
+    rank: Optional[torch.Tensor] = None
+    counts: Optional[torch.Tensor] = None
+
+
+def choose(z: torch.Tensor, r: Routing) -> Tuple[torch.Tensor, torch.Tensor]:
+    """The choice in PyTorch, from the router's logits ``z [tokens, experts]``; ties go to the lower index."""
+    s = torch.sigmoid(z.float())
+    T, n = s.shape[0], r.experts // r.groups
+    value = s.view(T, r.groups, n).topk(min(2, n), -1).values.sum(-1)
+    kept = torch.sort(value, dim=-1, descending=True, stable=True).indices[:, :r.keep]
+    ok = torch.zeros(T, r.groups, dtype=torch.bool, device=z.device).scatter_(1, kept, True)
+    masked = s.masked_fill(~ok.repeat_interleave(n, 1), -1.0)
+    expert = torch.sort(masked, dim=-1, descending=True, stable=True).indices[:, :r.top]
+    w = s.gather(1, expert)
+    return expert.to(torch.int32), w / (w.sum(-1, keepdim=True) + 1e-20) * r.scale
+
+
+def route(h: torch.Tensor, router: torch.Tensor, r: Routing) -> Choice:
+    """The experts of every row of ``h [tokens, W]`` by the logits ``h @ router^T`` (``router [experts
+    rounded up to 8, W]``), which are fp32."""
+    T, W = h.shape
+    if not h.is_cuda:
+        return Choice(*choose(h.float() @ router[:r.experts].float().t(), r))
+    from .gemm import linear
+    few, dev = T <= ROUTE_FEW, h.device
+    logits = None
+    if not few:
+        logits = linear(h, router, torch.empty((T, router.shape[0]), dtype=torch.float32, device=dev))
+    per = 1 if few else ROUTE_TOKENS
+    blocks = (T + per - 1) // per
+    expert, rank = (torch.empty((T, r.top), dtype=torch.int32, device=dev) for _ in range(2))
+    weight = torch.empty((T, r.top), dtype=torch.float32, device=dev)
+    counts = torch.empty((blocks, r.experts), dtype=torch.int32, device=dev)
+    rc = _lib.serving_lib().cb_moe_choose(
+        _p(logits), logits.stride(0) if logits is not None else 0, _p(h), h.stride(0), _p(router),
+        router.stride(0), W, T, r.experts, r.top, r.groups, r.keep, _F(r.scale), _p(expert), _p(weight),
+        _p(rank), _p(counts), int(h.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_moe_choose")
+    return Choice(expert, weight, per, rank, counts)
+
+
+@dataclass
+class Sorted:
+    """``rows [blocks * BLOCK, W]``: every token's row once per expert it uses, sorted by expert;
+    ``slot [tokens, top]`` says where; ``block_expert [blocks]`` is the expert of a block of rows, -1 behind
+    the last one."""
+
+    rows: torch.Tensor
+    slot: torch.Tensor
+    block_expert: torch.Tensor
+
+
+def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
+    T, W = h.shape
+    pairs = T * r.top
+    blocks = pairs // BLOCK + min(r.experts, pairs)
+    dev = h.device
+    rows = torch.empty((blocks * BLOCK, W), dtype=h.dtype, device=dev)
+    if not h.is_cuda:
+        rows.zero_()
+        slot = torch.empty((T, r.top), dtype=torch.int32)
+        block_expert, at = [], 0
+        for e in range(r.experts):
+            t, k = (c.expert == e).nonzero(as_tuple=True)
+            if len(t):
+                slot[t, k] = torch.arange(at, at + len(t), dtype=torch.int32)
+                rows[at:at + len(t)] = h[t]
+                n = (len(t) + BLOCK - 1) // BLOCK
+                block_expert += [e] * n
+                at += n * BLOCK
+        block_expert += [-1] * (blocks - len(block_expert))
+        return Sorted(rows, slot, torch.tensor(block_expert, dtype=torch.int32))
+    slot = torch.empty((T, r.top), dtype=torch.int32, device=dev)
+    block_expert = torch.empty(blocks, dtype=torch.int32, device=dev)
+    base = torch.empty_like(c.counts)
+    rc = _lib.serving_lib().cb_moe_sort(
+        _p(h), h.stride(0), _p(c.expert), _p(c.rank), _p(c.counts), T, r.experts, r.top, c.per_block,
+        c.counts.shape[0], _p(base), _p(slot), _p(block_expert), blocks, _p(rows), W,
+        int(h.dtype == torch.float32), _p(_lib.status_buffer(dev)), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_moe_sort", launches=2)
+    return Sorted(rows, slot, block_expert)
+
+
+def grouped_linear(x: torch.Tensor, w: torch.Tensor, block_expert: torch.Tensor, out: torch.Tensor, *,
+                   glu: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+    """``out[block] = x[block] @ w[block_expert[block]]^T`` for every block of ``BLOCK`` rows (``w [experts, N,
+    K]``); blocks of no expert are left alone.  ``glu = (slope, limit)``: see :func:`coeus_b200.ops.gemm.linear`."""
+    E, N, K = w.shape
+    M = x.shape[0]
+    if x.shape[1] != K or M != block_expert.shape[0] * BLOCK or out.shape != (M, N // 2 if glu else N):
+        raise ValueError(f"grouped_linear: shapes {tuple(x.shape)} {tuple(w.shape)} {tuple(out.shape)}")
+    if not x.is_cuda:
+        for b, e in enumerate(block_expert.tolist()):
+            if e >= 0:
+                s = slice(b * BLOCK, (b + 1) * BLOCK)
+                z = x[s].float() @ w[e].float().t()
+                out[s] = (clamped_glu(z, *glu) if glu else z).to(out.dtype)
+        return out
+    slope, limit = glu or (0.0, 0.0)
+    lib, st = _lib.serving_lib(), _p(_lib.status_buffer(x.device))
+    if x.dtype == torch.float32:
+        rc = lib.cb_linear_f32_grouped(
+            _p(x), x.stride(0), _p(w), w.stride(1), _p(block_expert), _p(out), out.stride(0), M, N, K,
+            int(glu is not None), _F(slope), _F(limit), _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_linear_f32_grouped")
+        return out
+    rc = lib.cb_gemm_bf16_blocks(
+        _p(x), _p(w), _p(out), M, N, K, E, x.stride(0), w.stride(1), out.stride(0), _p(block_expert),
+        int(glu is not None), _F(slope), _F(limit), st, _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_gemm_bf16_blocks")
+    return out
+
+
+def experts_few(h: torch.Tensor, c: Choice, r: Routing, w_in: torch.Tensor, w_down: torch.Tensor,
+                limit: float, s_in: Optional[torch.Tensor], s_down: Optional[torch.Tensor],
+                s_limit: float, slope: float) -> torch.Tensor:
+    """All experts of up to ``FEW`` bf16 rows and the shared one: fp32 ``[tokens, W]``."""
+    T, W = h.shape
+    n, ns = w_down.shape[2], s_down.shape[1] if s_down is not None else 0
+    live = min(r.experts, T * r.top)
+    act = torch.empty((T, live * n + ns), dtype=h.dtype, device=h.device)
+    y = torch.empty((T, W), dtype=torch.float32, device=h.device)
+    rc = _lib.serving_lib().cb_moe_few(
+        _p(h), h.stride(0), T, W, r.experts, r.top, _p(c.expert), _p(c.weight), _p(w_in), _p(w_down), n,
+        _F(limit), _p(s_in), _p(s_down), ns, _F(s_limit), _F(slope), _p(act), act.stride(0), _p(y),
+        y.stride(0), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_moe_few", launches=2)
+    return y

@@ -140,8 +140,8 @@ def gather_rows(cache: torch.Tensor, page_table: torch.Tensor, where: torch.Tens
     """``n`` cached rows, the ``i``-th that of slot ``where[2 i]`` at position ``where[2 i + 1]``."""
     row_p = cache.shape[-1]
     rc = _lib.serving_lib().cb_kv_gather(
-        _p(cache), _p(cache), 1, row_p, row_p, _p(page_table), page_table.shape[1], cache.shape[0],
-        _p(where), n, _p(out), None, row_p, _p(_lib.status_buffer(out.device)), _lib.stream_ptr())
+        _p(cache), _p(cache), 1, 1, row_p, row_p, _p(page_table), page_table.shape[1], cache.shape[0],
+        _p(where), n, _p(out), None, row_p, row_p, _p(_lib.status_buffer(out.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_kv_gather")
 
 
@@ -155,7 +155,7 @@ def piece_attention(q: torch.Tensor, kv: torch.Tensor, batch: RaggedBatch, plan:
     T, heads, P = q.shape
     rc = _lib.serving_lib().cb_attn_fwd_pieces(
         _p(q), _p(kv), _p(kv[:, heads * P:]), _p(out), T, kv.shape[0], _p(pieces), n_pieces, longest,
-        heads, heads, P, vdim, q.stride(0), kv.stride(0), kv.stride(0), out.stride(0), _F(scale), None,
-        _p(gate), gate.stride(0) if gate is not None else 0, 1, plan.window or 0,
-        _p(_lib.status_buffer(q.device)), _lib.stream_ptr())
+        heads, heads, P, P, vdim, q.stride(0), kv.stride(0), kv.stride(0), out.stride(0), _F(scale), None,
+        _p(gate), gate.stride(0) if gate is not None else 0, 1, plan.window or 0, _F(0.0), 1, None, _F(1.0),
+        _F(0.0), _p(_lib.status_buffer(q.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_attn_fwd_pieces")

@@ -51,11 +51,13 @@ class AttnPlan:
 
     Under a sliding ``window`` a piece is a run of at most ``WINDOW_PIECE`` rows together with the
     keys its first row sees before it; an entry that continues a sequence gathers its own keys and
-    those of the window before it."""
+    those of the window before it.  Where sizes do not allow pieces, ``tiles`` says whether long entries
+    go in tiles instead."""
 
     chunk: Optional[int]
     pieces: bool              # whether the layer's sizes allow the piece kernel
     window: Optional[int] = None
+    tiles: bool = False
 
 
 SCAN_MIN = 16         # entries of more tokens than this take the chunked recurrence
@@ -86,6 +88,52 @@ def _segments(plan: ScanPlan, long: List[int], lens: List[int]):
     return segs, runs
 
 
+def head_prep(raw: torch.Tensor, koff: int, voff: int, heads: int, kv_heads: int, dim: int, vdim: int,
+              batch: "RaggedBatch", rope: Optional[torch.Tensor], k_cache: torch.Tensor,
+              v_cache: torch.Tensor, page_table: torch.Tensor, *, interleaved: bool = False,
+              unit_eps: Optional[float] = None, q_head: Optional[int] = None,
+              k_rows: Optional[torch.Tensor] = None, v_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """What stands between the projections ``raw`` (queries at column 0, keys at ``koff``, values at
+    ``voff``) and the scores: rotation of the first ``2 * rope.shape[1]`` entries of the q and k heads (pairs
+    half a rotation apart, or with ``interleaved`` neighbours), division of q and k by their root mean
+    square over ``dim`` (``unit_eps`` inside the root; None: not), the write of k and v into the cache pages
+    (and row by row into the first rows of ``k_rows [.., kv_heads, P]`` and ``v_rows``, zeros behind a
+    head).  Returns ``q [rows, heads, q_head]``, zeros behind ``dim``.  ``heads`` and ``kv_heads`` count the
+    heads of q and k; v has ``v_cache.shape[2]``."""
+    T, v_heads = raw.shape[0], v_cache.shape[2]
+    half = rope.shape[1] if rope is not None else 0
+    Q = q_head or (dim + 7) // 8 * 8
+    q = torch.empty((T, heads, Q), dtype=raw.dtype, device=raw.device)
+    if not raw.is_cuda:
+        def rotated(x):
+            if half:
+                c, s = rope[:, None, :, 0], rope[:, None, :, 1]
+                a, b = (x[..., 0:2 * half:2], x[..., 1:2 * half:2]) if interleaved else \
+                    (x[..., :half], x[..., half:2 * half])
+                y = (a * c - b * s, b * c + a * s)
+                y = torch.stack(y, -1).flatten(-2) if interleaved else torch.cat(y, -1)
+                x = torch.cat([y, x[..., 2 * half:]], -1)
+            if unit_eps is not None:
+                x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + unit_eps)
+            return x
+        q.zero_()
+        q[..., :dim] = rotated(raw[:, :heads * dim].float().view(T, heads, dim)).to(q.dtype)
+        k = rotated(raw[:, koff:koff + kv_heads * dim].float().view(T, kv_heads, dim))
+        page, at = _cells(page_table, batch)
+        k_cache[page, at, :, :dim] = k.to(k_cache.dtype)
+        v_cache[page, at, :, :vdim] = raw[:, voff:voff + v_heads * vdim].view(T, v_heads, vdim)
+        return q
+    rc = _lib.serving_lib().cb_head_prep(
+        _p(raw), raw.stride(0), koff, voff, heads, kv_heads, v_heads, dim, vdim, half, _p(rope),
+        int(interleaved), int(unit_eps is not None), _F(unit_eps or 0.0), _p(q), Q, _p(k_cache),
+        _p(v_cache), k_cache.shape[-1], v_cache.shape[-1], _p(k_rows), _p(v_rows),
+        k_rows.shape[2] if k_rows is not None else 0, v_rows.shape[2] if v_rows is not None else 0,
+        _p(page_table), page_table.shape[1], k_cache.shape[0], _p(batch.row_slot), _p(batch.pos), T,
+        int(raw.dtype == torch.float32), _p(_lib.status_buffer(raw.device)), _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_head_prep")
+    return q
+
+
 def pieces_allowed(dim: int, vdim: int, chunk: Optional[int], scale: float) -> bool:
     return max(dim, vdim) <= 128 and scale > 0 and (chunk is None or chunk >= MIN_PIECE)
 
@@ -93,6 +141,13 @@ def pieces_allowed(dim: int, vdim: int, chunk: Optional[int], scale: float) -> b
 def row_head(dim: int, vdim: int) -> int:
     """Distance of the heads in the row-wise q, k and v of the piece kernel."""
     return 64 if max(dim, vdim) <= 64 else 128
+
+
+def row_heads(dim: int, vdim: int, maps: int) -> Tuple[int, int]:
+    """Distance of the heads in q and k, and in v, of the piece kernel without a convolution: with one
+    map they are the same."""
+    p = row_head(dim, vdim)
+    return (p, p) if maps == 1 else (row_head(dim, 0), p)
 
 
 def _cut(plan: AttnPlan, pos0: int, n: int):
@@ -156,6 +211,8 @@ class RaggedBatch:
                 p0, r0 = entries[i].pos0, int(row0[i])
                 if plan.window is not None:
                     if not plan.pieces:
+                        if plan.tiles:
+                            tiles += [(i, o, min(ATTN_TILE, lens[i] - o)) for o in range(0, lens[i], ATTN_TILE)]
                         continue
                     ahead = min(p0, plan.window - 1)
                     first = r0                             # key row of the entry's first token
@@ -264,20 +321,33 @@ def rms_rows(x: torch.Tensor, w1: torch.Tensor, width: int, eps: float, dtype: t
     return y1, y2
 
 
+@dataclass
+class Spread:
+    """A sublayer's result in pieces: row ``t`` is the sum over ``k`` of ``weight[t, k] * rows[slot[t, k]]``
+    (``slot`` int32 and ``weight`` fp32 ``[tokens, top]``, ``rows`` in the activation type)."""
+
+    rows: torch.Tensor
+    slot: torch.Tensor
+    weight: torch.Tensor
+
+
 def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dtype, *,
              y: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
              post: Optional[torch.Tensor] = None, gain: Optional[torch.Tensor] = None,
              shift: Optional[torch.Tensor] = None, before: Optional[torch.Tensor] = None,
              batch: Optional["RaggedBatch"] = None, rows: Optional[torch.Tensor] = None,
-             keep: bool = True, casts: Sequence[torch.Tensor] = ()
+             keep: bool = True, casts: Sequence[torch.Tensor] = (),
+             spread: Optional["Spread"] = None
              ) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
-    """One pass between two sublayers, ``(x', h)``: ``v = y + bias``, RMS-normed with gain ``post`` when
+    """One pass between two sublayers, ``(x', h)``: ``v = y + bias`` (plus the weighted rows of ``spread``,
+    which may also stand alone), RMS-normed with gain ``post`` when
     given; ``x' = x + v`` in fp32 (``v`` alone without ``x``, ``x`` itself without ``y``); ``h`` the RMS
     norm of ``x'`` with ``gain`` in the activation type, shifted by ``h + (h_before - h) * shift`` with
     the previous token's h (``before [slots, ld]`` at an entry's start, which is advanced).  Gains are
     one number or a vector.  ``rows`` restricts the pass to some rows (``x'`` is not returned then),
     ``keep=False`` drops ``x'``; ``casts`` are up to two views that get ``x'`` in the activation type."""
     src = x if x is not None else y
+    added = y is not None or spread is not None
     ld, n = src.shape[1], src.shape[0] if rows is None else rows.shape[0]
     if rows is not None:
         keep = False
@@ -287,8 +357,11 @@ def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dty
         def norm(v, g):
             return v * torch.rsqrt((v[:, :width] ** 2).mean(-1, keepdim=True) + eps) * g
         out = None if x is None else pick(x)
-        if y is not None:
-            v = pick(y).float()
+        if added:
+            v = pick(y).float() if y is not None else torch.zeros_like(out)
+            if spread is not None:
+                for k in range(spread.weight.shape[1]):
+                    v = v + pick(spread.rows[spread.slot[:, k].long()].float() * spread.weight[:, k, None])
             v = v if bias is None else v + bias
             v = v if post is None else norm(v, post)
             out = v if out is None else out + v
@@ -309,18 +382,20 @@ def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dty
             h = h.to(dtype)
         return (out if keep else None), h
     x_out = torch.empty((n, ld), dtype=torch.float32, device=src.device) \
-        if keep and (y is not None or x is None) else None
+        if keep and (added or x is None) else None
     h = torch.empty((n, ld), dtype=dtype, device=src.device) if gain is not None else None
     shifted = shift is not None
     none = (None,) * 6
     ents = (*batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off)) if shifted else none
     cast = list(casts) + [None] * (2 - len(casts))
+    sp = (None, 0, None, None, 0) if spread is None else (
+        _p(spread.rows), spread.rows.stride(0), _p(spread.slot), _p(spread.weight), spread.slot.shape[1])
     rc = _lib.serving_lib().cb_add_norm(
         _p(x), _p(y), _p(bias), _p(post), int(post is not None and post.numel() > 1), _p(x_out), ld,
         y.stride(0) if y is not None else 0, _p(gain), int(gain is not None and gain.numel() > 1), _p(h),
         ld, _p(cast[0]), _p(cast[1]), casts[0].stride(0) if casts else 0, _p(shift), _p(before),
         _p(rows), *ents, batch.n_conv if shifted else n, width, _F(eps), int(dtype == torch.float32),
-        int(y is not None and y.dtype == torch.float32), _lib.stream_ptr())
+        int(y is not None and y.dtype == torch.float32), *sp, _lib.stream_ptr())
     _lib.check_rc(rc, "cb_add_norm")
     return (x_out if x_out is not None else (x if keep else None)), h
 
@@ -500,20 +575,31 @@ def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, e
 def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                      page_table: torch.Tensor, batch: RaggedBatch, heads: int, kv_heads: int,
                      dim: int, vdim: int, scale: float, out: torch.Tensor, *,
-                     chunk: Optional[int] = None, sink: Optional[torch.Tensor] = None,
-                     gate: Optional[torch.Tensor] = None, max_ctx: Optional[int] = None,
+                     chunk: Optional[int] = None, window: Optional[int] = None,
+                     softcap: Optional[float] = None, maps: int = 1,
+                     map_weight: Optional[torch.Tensor] = None, map_factor: float = 1.0,
+                     eps: float = 0.0, sink: Optional[torch.Tensor] = None,
+                     gate: Optional[torch.Tensor] = None, gate_wide: bool = False,
+                     max_ctx: Optional[int] = None,
                      k_rows: Optional[torch.Tensor] = None,
                      v_rows: Optional[torch.Tensor] = None,
                      plan: Optional[AttnPlan] = None) -> torch.Tensor:
     """Causal attention of every query row over the cached keys of its own sequence, restricted to
-    the row's chunk (positions with the same ``pos // chunk``) when ``chunk`` is given.  ``sink``
-    (fp32 ``[heads]``) is a logit that enters the softmax denominator only; ``gate`` (a view whose
-    column ``h`` belongs to head ``h``) multiplies head ``h``'s output by its sigmoid.  Query head
-    ``h`` reads key/value head ``h // (heads // kv_heads)``.  ``q`` is ``[rows, heads, Q >= dim]``, ``out`` a ``[rows, heads * vdim]``
+    the row's chunk (positions with the same ``pos // chunk``) when ``chunk`` is given, or to itself and
+    the ``window - 1`` positions before it.  Scores ``s`` become ``softcap * tanh(s / softcap)``.  ``sink``
+    (fp32 ``[heads]``) is a logit that enters the softmax denominator only; ``gate`` multiplies by its
+    sigmoid: a view whose column ``h`` belongs to head ``h``, or (``gate_wide``) a view like ``out``.  Query
+    head ``h`` reads key/value head ``h // (heads // kv_heads)``.  ``q`` is ``[rows, heads, Q >= dim]``,
+    ``out`` a ``[rows, heads * vdim]``
     view; ``max_ctx`` bounds the keys of any row (it only chooses how many CTAs share a row).  With
     row-wise ``k_rows`` and ``v_rows`` at hand (:meth:`RaggedBatch.kv_rows` rows of ``[kv_heads, P]``,
-    this step's filled in; q then has the same head distance P), the pieces of ``plan`` go through
-    the tcgen05 kernel; the default plan has pieces when the buffers are given."""
+    this step's filled in; q then has the keys' head distance), the pieces of ``plan`` go through
+    the tcgen05 kernel; the default plan has pieces when the buffers are given.
+
+    With two ``maps`` a head has two queries and its key head two keys (``q [rows, heads * 2, Q]``,
+    ``k_cache [pages, PAGE, kv_heads * 2, dim_p]``, map 0 first) over the same values; with their outputs
+    ``a0`` and ``a1`` the head's output is ``a0 - map_weight * a1`` (``map_weight`` one fp32 number on the
+    device) divided by its root mean square (``eps`` inside the root), times ``map_factor``."""
     T = q.shape[0]
     if not q.is_cuda:
         per = heads // kv_heads
@@ -522,12 +608,15 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             pos = batch.pos[r:r + m].long()
             n = int(pos[-1]) + 1
             pages = page_table[batch.slots_host[i], :(n + PAGE - 1) // PAGE].long()
-            K = k_cache[pages].reshape(-1, kv_heads, k_cache.shape[-1])[:n, :, :dim].float()
+            K = k_cache[pages].reshape(-1, kv_heads, maps, k_cache.shape[-1])[:n, ..., :dim].float()
             V = v_cache[pages].reshape(-1, kv_heads, v_cache.shape[-1])[:n, :, :vdim].float()
-            K, V = K.repeat_interleave(per, 1), V.repeat_interleave(per, 1)
-            s = torch.einsum("thd,nhd->htn", q[r:r + m].float(), K) * scale
+            K, V = K.repeat_interleave(per, 1).flatten(1, 2), V.repeat_interleave(per * maps, 1)
+            s = torch.einsum("thd,nhd->htn", q[r:r + m, :, :dim].float(), K) * scale
+            if softcap is not None:
+                s = softcap * torch.tanh(s / softcap)
             j = torch.arange(n)
             lo = pos // chunk * chunk if chunk else torch.zeros_like(pos)
+            lo = torch.clamp(pos + 1 - window, min=0) if window else lo
             ok = (j[None] <= pos[:, None]) & (j[None] >= lo[:, None])
             s = s.masked_fill(~ok, float("-inf"))
             top = s.amax(-1, keepdim=True)
@@ -538,51 +627,65 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             if sink is not None:
                 den = den + torch.exp(sink.view(-1, 1, 1) - top)
             o = torch.einsum("htn,nhd->thd", w / den, V)
+            if maps == 2:
+                o = o[:, 0::2] - map_weight * o[:, 1::2]
+                o = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps) * map_factor
             if gate is not None:
-                o = o * torch.sigmoid(gate[r:r + m, :heads].float())[:, :, None]
+                g = torch.sigmoid(gate[r:r + m].float())
+                o = o * (g[:, :heads * vdim].view(m, heads, vdim) if gate_wide else g[:, :heads, None])
             out[r:r + m] = o.reshape(m, -1).to(out.dtype)
             r += m
         return out
     st = _p(_lib.status_buffer(q.device))
     lib = _lib.serving_lib()
+    spec = _AttnSpec(heads, kv_heads, dim, vdim, k_cache.shape[-1], v_cache.shape[-1], chunk or 0,
+                     window or 0, maps, int(gate_wide), scale, softcap or 0.0, map_factor, eps)
     common = (_p(q), q.shape[2], _p(k_cache), _p(v_cache), _p(page_table), page_table.shape[1],
-              k_cache.shape[0], heads, kv_heads, dim, vdim, k_cache.shape[-1], v_cache.shape[-1],
-              chunk or 0, _F(scale), _p(sink), _p(gate), gate.stride(0) if gate is not None else 0,
-              _p(out), out.stride(0))
+              k_cache.shape[0], ctypes.byref(spec), _p(sink), _p(gate),
+              gate.stride(0) if gate is not None else 0, _p(map_weight), _p(out), out.stride(0))
     if batch.n_big:
         n_tiles, n_pieces, longest, extra, pieces, where, t_entry, t_off, t_len = batch.plan(
-            plan or AttnPlan(chunk, k_rows is not None))
+            plan or AttnPlan(chunk, k_rows is not None, window))
         if n_tiles:
             rc = lib.cb_ragged_attn_tiles(*common, *batch.entry_args(), _p(t_entry), _p(t_off),
                                           _p(t_len), n_tiles, st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_ragged_attn_tiles")
         if extra:
-            rc = lib.cb_kv_gather(_p(k_cache), _p(v_cache), kv_heads, k_cache.shape[-1],
+            rc = lib.cb_kv_gather(_p(k_cache), _p(v_cache), kv_heads * maps, kv_heads, k_cache.shape[-1],
                                   v_cache.shape[-1], _p(page_table), page_table.shape[1],
                                   k_cache.shape[0], _p(where), extra, _p(k_rows[T:]), _p(v_rows[T:]),
-                                  k_rows.shape[2], st, _lib.stream_ptr())
+                                  k_rows.shape[2], v_rows.shape[2], st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_kv_gather")
         if n_pieces:
             rc = lib.cb_attn_fwd_pieces(
                 _p(q), _p(k_rows), _p(v_rows), _p(out), T, k_rows.shape[0], _p(pieces), n_pieces,
-                longest, heads, kv_heads, k_rows.shape[2], vdim, q.stride(0), k_rows.stride(0),
-                v_rows.stride(0), out.stride(0), _F(scale), _p(sink), _p(gate),
-                gate.stride(0) if gate is not None else 0, 0, 0, st, _lib.stream_ptr())
+                longest, heads, kv_heads, k_rows.shape[2], v_rows.shape[2], vdim, q.stride(0),
+                k_rows.stride(0), v_rows.stride(0), out.stride(0), _F(scale), _p(sink), _p(gate),
+                gate.stride(0) if gate is not None else 0, int(gate_wide), window or 0,
+                _F(softcap or 0.0), maps, _p(map_weight), _F(map_factor), _F(eps), st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_attn_fwd_pieces")
     n = batch.n_rows
     if n:
-        per = heads // kv_heads
+        per = heads // kv_heads * maps
         ctas = n * kv_heads * ((per + 15) // 16)
         ctx = max_ctx or batch.max_ctx
-        ctx = min(ctx, chunk) if chunk else ctx
+        ctx = min([ctx] + [c for c in (chunk, window) if c])
         # a CTA takes 128 keys at a time
         splits = max(1, min(16, (2 * 148 + ctas - 1) // ctas, (ctx + 127) // 128))
         part_o = part_ml = None
-        if splits > 1:
-            part_o = torch.empty((n, heads, splits, vdim), dtype=torch.float32, device=q.device)
-            part_ml = torch.empty((n, heads, splits, 2), dtype=torch.float32, device=q.device)
+        if splits > 1 or maps > 1:
+            part_o = torch.empty((n, heads * maps, splits, vdim), dtype=torch.float32, device=q.device)
+            part_ml = torch.empty((n, heads * maps, splits, 2), dtype=torch.float32, device=q.device)
         rc = lib.cb_ragged_attn_rows(*common, _p(batch.rows), _p(batch.row_slot), _p(batch.pos), n,
                                      splits, _p(part_o), _p(part_ml), int(q.dtype == torch.float32),
                                      st, _lib.stream_ptr())
-        _lib.check_rc(rc, "cb_ragged_attn_rows", launches=2 if splits > 1 else 1)
+        _lib.check_rc(rc, "cb_ragged_attn_rows", launches=2 if part_o is not None else 1)
     return out
+
+
+class _AttnSpec(ctypes.Structure):
+    """``RaggedSpec`` of ``csrc/ragged_attn.cu``."""
+
+    _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "dim", "vdim", "dim_p", "vdim_p", "chunk",
+                                            "window", "maps", "gate_wide")] + \
+               [(n, ctypes.c_float) for n in ("scale", "softcap", "map_factor", "eps")]
