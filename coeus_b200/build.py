@@ -41,7 +41,7 @@ NVCC_FLAGS = [
 
 SERVING_SOURCES = ("gemm", "ragged_rows", "residual", "shortconv", "delta_scan", "ssd", "ssd_chunk", "mingru",
                    "linear_f32", "linear_skinny", "linear_heads", "ragged_attn", "latent_attn",
-                   "attention_fwd")
+                   "attention_fwd", "head_prep", "experts")
 
 
 def _nvcc() -> str:

@@ -20,6 +20,13 @@
 // by more than 2^8); optionally a quarter of the exponentials is evaluated as a cubic polynomial
 // on the FMA pipe, because the exponential unit (16 results per clock per SM) bounds dh = 64.
 // Grouped-query attention: query head h reads K/V head h / (nh / nkv).
+//
+// Two variants serve prompts of unequal length (PIECES) only.  CAP: scores s become cap * tanh(s / cap).
+// DIFF: a head has two maps, each with queries and keys of its own over the same values; an item is ONE
+// query tile of a head, tiles A and B of the step are its two maps, every step has its own key tile and
+// every pair of steps its value tile.  At the end each warpgroup takes half of the columns of
+// o = a0 - w a1, and the two meet at two barriers: one when both results are complete, one for the sum of
+// squares of o, which is divided by its root mean square.
 // Every wait is bounded; a wait that runs out records a status code and the CTA leaves.
 #include "common.cuh"
 #include "ptx.cuh"
@@ -57,6 +64,9 @@ struct AttnFwdArgs {
   int ldg;                     // of head h, or (gate_wide) column h * vdim + d for its column d
   int gate_wide;
   int window;                  // 0: no window
+  float cap_log2, cap_in;      // CAP: the cap in units of log2, and what takes a product to the tanh
+  const float* map_weight;     // DIFF: weight of the second map, factor and eps of the norm
+  float map_factor, map_eps;
 };
 
 // Optional device timeline of CTA 0 (clock64 stamps; see cb_attn_fwd_set_trace): softmax warp 0
@@ -66,27 +76,32 @@ struct AttnFwdArgs {
 __device__ long long* g_attn_fwd_trace = nullptr;
 __device__ int g_attn_fwd_trace_cta = 0;   // which CTA writes the step timeline
 
-template <int DH>
+template <int DQ, int DV, bool DIFF = false>
 struct AFCfg {
   static constexpr int BKV = 128;                       // keys per step
-  static constexpr int NBUF = (DH == 64) ? 3 : 2;       // score buffers in tensor memory
-  static constexpr int Q_BYTES = AF_BM * DH * 2;        // one query tile
-  static constexpr int KV_BYTES = BKV * DH * 2;         // one K (or V) tile
-  static constexpr int KST = (DH == 64) ? 3 : 2;        // ring depth of K and of V
+  static constexpr int NBUF = (DV == 64) ? 3 : 2;       // score buffers in tensor memory
+  static constexpr int Q_BYTES = AF_BM * DQ * 2;        // one query tile
+  static constexpr int K_BYTES = BKV * DQ * 2;          // one K tile
+  static constexpr int V_BYTES = BKV * DV * 2;          // one V tile
+  static constexpr int KST = DIFF ? (DQ == 64 ? 4 : 2) : (DQ == 64 ? 3 : 2);   // ring depth of K
+  static constexpr int VST = (DV == 64) ? 3 : 2;                               // and of V
   static constexpr int OFF_Q = 0;
   static constexpr int OFF_K = 2 * Q_BYTES;
-  static constexpr int OFF_V = OFF_K + KST * KV_BYTES;
-  static constexpr int OFF_BAR = OFF_V + KST * KV_BYTES;
-  static constexpr int SMEM_BYTES = OFF_BAR + 512;
+  static constexpr int OFF_V = OFF_K + KST * K_BYTES;
+  static constexpr int OFF_BAR = OFF_V + VST * V_BYTES;
+  static constexpr int OFF_X = OFF_BAR + 512;           // DIFF: two numbers per row and warpgroup
+  static constexpr int SMEM_BYTES = OFF_X + (DIFF ? 4 * AF_BM * 4 : 0);
   static constexpr int TMEM_COLS = 512;
-  static constexpr int O_COL0 = 0;            // O_t (fp32, DH columns each)
-  static constexpr int S_COL0 = 2 * DH;       // NBUF score buffers of BKV fp32 columns; P (bf16)
+  static constexpr int O_COL0 = 0;            // O_t (fp32, DV columns each)
+  static constexpr int S_COL0 = 2 * DV;       // NBUF score buffers of BKV fp32 columns; P (bf16)
                                               // takes the first BKV / 2 columns of its buffer
   static_assert(S_COL0 + NBUF * BKV <= TMEM_COLS, "tensor memory budget");
+  static_assert(SMEM_BYTES <= 227 * 1024, "shared memory budget");
   // barrier indices
   static constexpr int B_QF = 0, B_QE = 2, B_SF = 4, B_PR = B_SF + NBUF, B_BF = B_PR + NBUF,
                        B_KF = B_BF + NBUF, B_KE = B_KF + KST, B_VF = B_KE + KST,
-                       B_VE = B_VF + KST, N_BARS = B_VE + KST;
+                       B_VE = B_VF + VST, B_X = B_VE + VST, N_BARS = B_X + 2;
+  static_assert(N_BARS * 8 + 16 <= 512, "barrier area");
 };
 
 // 2^x for x <= ~8 without the special-function unit and without conversion instructions (which
@@ -109,7 +124,7 @@ __device__ __forceinline__ float exp2_poly(float x) {
 // item of every wave of gridDim.x items, counted from the front of even waves and from the back
 // of odd ones, so that the heavy and the light ends of the sorted list meet in one CTA), within
 // an item key tile by key tile, tile A before tile B.
-template <bool PIECES>
+template <bool PIECES, bool DIFF = false>
 struct AFWalk {
   // problem
   int n_items, n_bh, n_pairs, n_q_tiles, n_kv_tiles, nh, causal, bkv, n_waves;
@@ -125,12 +140,13 @@ struct AFWalk {
   __device__ int first_row(const AttnFwdArgs& p) const { return PIECES ? piece.x : b * p.S; }
   __device__ int first_key(const AttnFwdArgs& p) const { return PIECES ? piece.z : b * p.S; }
   __device__ int rows(const AttnFwdArgs& p) const { return PIECES ? piece.y : p.S; }
+  __device__ int tile() const { return DIFF ? qa : qa + t; }           // query tile of this step
   __device__ int keys_ahead() const { return PIECES ? piece.w : 0; }   // keys before query 0's own
   __device__ void init(const AttnFwdArgs& p, int bkv_) {
     bkv = bkv_;
     n_q_tiles = (p.S + AF_BM - 1) / AF_BM;
     n_kv_tiles = (p.S + bkv - 1) / bkv;
-    n_pairs = (n_q_tiles + 1) / 2;
+    n_pairs = DIFF ? n_q_tiles : (n_q_tiles + 1) / 2;
     nh = p.nh;
     n_bh = p.B * p.nh;
     n_items = n_pairs * n_bh;
@@ -154,7 +170,7 @@ struct AFWalk {
       const int pair = n_pairs - 1 - i / n_bh;     // pairs with the most key tiles first
       b = bh / nh;
       h = bh % nh;
-      qa = 2 * pair;
+      qa = DIFF ? pair : 2 * pair;
       if constexpr (PIECES) {
         piece = pieces[b];
         n_q_tiles = (piece.y + AF_BM - 1) / AF_BM;
@@ -163,7 +179,8 @@ struct AFWalk {
       }
       const int ahead = keys_ahead();
       n0 = causal ? min(n_kv_tiles, (ahead + (qa + 1) * AF_BM + bkv - 1) / bkv) : n_kv_tiles;
-      n1 = qa + 1 >= n_q_tiles ? 0
+      n1 = DIFF ? n0
+           : qa + 1 >= n_q_tiles ? 0
            : (causal ? min(n_kv_tiles, (ahead + (qa + 2) * AF_BM + bkv - 1) / bkv) : n_kv_tiles);
       nmax = max(n0, n1);
       j = 0;
@@ -186,12 +203,16 @@ struct AFWalk {
   __device__ bool last_of_tile() const { return j == (t ? n1 : n0) - 1; }
 };
 
-template <int DH, bool POLY, bool DROP, bool PIECES>
+template <int DQ, int DV, bool POLY, bool DROP, bool PIECES, bool CAP, bool DIFF>
 __global__ void __launch_bounds__(AF_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const AttnFwdArgs p) {
-  using Cfg = AFCfg<DH>;
-  constexpr int KST = Cfg::KST, NBUF = Cfg::NBUF, BKV = Cfg::BKV;
+  static_assert(PIECES || (!CAP && !DIFF), "the variants of pieces");
+  static_assert(!CAP || !DIFF, "no kernel has both");
+  using Cfg = AFCfg<DQ, DV, DIFF>;
+  using Walk = AFWalk<PIECES, DIFF>;
+  constexpr int KST = Cfg::KST, VST = Cfg::VST, NBUF = Cfg::NBUF, BKV = Cfg::BKV;
+  constexpr int MAPS = DIFF ? 2 : 1;
   extern __shared__ __align__(1024) uint8_t smem[];
   const uint32_t sbase = smem_u32(smem);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Cfg::OFF_BAR);
@@ -220,9 +241,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     for (int s = 0; s < KST; ++s) {
       mbar_init(bar(Cfg::B_KF + s), 1);
       mbar_init(bar(Cfg::B_KE + s), 1);
+    }
+    for (int s = 0; s < VST; ++s) {
       mbar_init(bar(Cfg::B_VF + s), 1);
       mbar_init(bar(Cfg::B_VE + s), 1);
     }
+    for (int s = 0; s < 2; ++s) mbar_init(bar(Cfg::B_X + s), 8);   // one arrival per softmax warp
     *abort_flag = 0;
     seen[0] = 0;
     seen[1] = 0;
@@ -240,8 +264,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   auto sQ = [&](int t) { return sbase + Cfg::OFF_Q + t * Cfg::Q_BYTES; };
-  auto sK = [&](int s) { return sbase + Cfg::OFF_K + s * Cfg::KV_BYTES; };
-  auto sV = [&](int s) { return sbase + Cfg::OFF_V + s * Cfg::KV_BYTES; };
+  auto sK = [&](int s) { return sbase + Cfg::OFF_K + s * Cfg::K_BYTES; };
+  auto sV = [&](int s) { return sbase + Cfg::OFF_V + s * Cfg::V_BYTES; };
 
   // The kernel starts with 168 registers per thread (384 threads); the first warpgroup (producer
   // and MMA issue: little state) hands registers to the two softmax warpgroups, whose step keeps a
@@ -256,7 +280,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       uint32_t qcnt[2] = {0u, 0u};     // uses of each query buffer so far
       uint32_t kcnt = 0, vcnt = 0;     // K / V tiles loaded so far
       bool ok = true;
-      AFWalk<PIECES> w;
+      Walk w;
       w.init(p, BKV);
       while (w.valid && ok) {
         const int row0 = w.first_row(p), kv_row0 = w.first_key(p);
@@ -271,45 +295,48 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           }
           mbar_arrive_expect_tx(bar(Cfg::B_QF + t), Cfg::Q_BYTES);
 #pragma unroll
-          for (int c = 0; c < DH / 64; ++c)
-            tma_load_2d(sQ(t) + c * (AF_BM * 128), &tmQ, bar(Cfg::B_QF + t), h * DH + c * 64,
-                        row0 + (qa + t) * AF_BM);
+          for (int c = 0; c < DQ / 64; ++c)
+            tma_load_2d(sQ(t) + c * (AF_BM * 128), &tmQ, bar(Cfg::B_QF + t),
+                        (h * MAPS + (DIFF ? t : 0)) * DQ + c * 64,
+                        row0 + (DIFF ? qa : qa + t) * AF_BM);
           ++qcnt[t];
         };
-        auto load_k = [&](int j) {
+        auto load_k = [&](int j, int map) {
           const int s = kcnt % KST;
           if (!mbar_wait(bar(Cfg::B_KE + s), ((kcnt / KST) & 1u) ^ 1u, abort_flag)) {
             record_status(p.status, ST_WAIT_TIMEOUT, 952);
             ok = false;
             return;
           }
-          mbar_arrive_expect_tx(bar(Cfg::B_KF + s), Cfg::KV_BYTES);
+          mbar_arrive_expect_tx(bar(Cfg::B_KF + s), Cfg::K_BYTES);
 #pragma unroll
-          for (int c = 0; c < DH / 64; ++c)
-            tma_load_2d(sK(s) + c * (BKV * 128), &tmK, bar(Cfg::B_KF + s), hk * DH + c * 64,
+          for (int c = 0; c < DQ / 64; ++c)
+            tma_load_2d(sK(s) + c * (BKV * 128), &tmK, bar(Cfg::B_KF + s), (hk * MAPS + map) * DQ + c * 64,
                         kv_row0 + j * BKV);
           ++kcnt;
         };
         auto load_v = [&](int j) {
-          const int s = vcnt % KST;
-          if (!mbar_wait(bar(Cfg::B_VE + s), ((vcnt / KST) & 1u) ^ 1u, abort_flag)) {
+          const int s = vcnt % VST;
+          if (!mbar_wait(bar(Cfg::B_VE + s), ((vcnt / VST) & 1u) ^ 1u, abort_flag)) {
             record_status(p.status, ST_WAIT_TIMEOUT, 953);
             ok = false;
             return;
           }
-          mbar_arrive_expect_tx(bar(Cfg::B_VF + s), Cfg::KV_BYTES);
+          mbar_arrive_expect_tx(bar(Cfg::B_VF + s), Cfg::V_BYTES);
 #pragma unroll
-          for (int c = 0; c < DH / 64; ++c)
-            tma_load_2d(sV(s) + c * (BKV * 128), &tmV, bar(Cfg::B_VF + s), hk * DH + c * 64,
+          for (int c = 0; c < DV / 64; ++c)
+            tma_load_2d(sV(s) + c * (BKV * 128), &tmV, bar(Cfg::B_VF + s), hk * DV + c * 64,
                         kv_row0 + j * BKV);
           ++vcnt;
         };
         load_q(0);
-        if (ok) load_k(0);
+        if (ok) load_k(0, 0);
         if (ok) load_q(1);
+        if (DIFF && ok) load_k(0, 1);
         if (ok) load_v(0);
         for (int j = 1; j < nmax && ok; ++j) {
-          load_k(j);
+          load_k(j, 0);
+          if (DIFF && ok) load_k(j, 1);
           if (ok) load_v(j);
         }
         w.next_item();
@@ -326,7 +353,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           }
         };
         drain(Cfg::B_KF, kcnt, KST);
-        drain(Cfg::B_VF, vcnt, KST);
+        drain(Cfg::B_VF, vcnt, VST);
         for (int t = 0; t < 2; ++t)
           if (qcnt[t] > 0) drain(Cfg::B_QF + t, qcnt[t], 1);
       }
@@ -340,19 +367,19 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     // issuing (measured ~35 clocks per MMA against ~60-100 from a divergent single lane), and
     // build their descriptors once; a step only adds constants to the address field.
     {
-      constexpr uint32_t idesc_o = umma_idesc_bf16(AF_BM, DH, 0, 1);
+      constexpr uint32_t idesc_o = umma_idesc_bf16(AF_BM, DV, 0, 1);
       const uint64_t dV0 = umma_desc_sw128(sV(0), BKV * 128, 1024);
       const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem_base, 0);
       bool ok = true;
       int v_waited = -1;
-      AFWalk<PIECES> wp;
+      Walk wp;
       wp.init(p, BKV);
       for (uint32_t gp = 0; wp.valid && ok; wp.advance(), ++gp) {
         const uint32_t buf = gp % NBUF;
         const int t = wp.t;
-        const int vs = wp.kv_seq % KST;
+        const int vs = wp.kv_seq % VST;
         if (v_waited != wp.kv_seq) {
-          if (!mbar_wait(bar(Cfg::B_VF + vs), (wp.kv_seq / KST) & 1u, abort_flag)) {
+          if (!mbar_wait(bar(Cfg::B_VF + vs), (wp.kv_seq / VST) & 1u, abort_flag)) {
             record_status(p.status, ST_WAIT_TIMEOUT, 962);
             break;
           }
@@ -365,8 +392,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         long long* tr = (blockIdx.x == g_attn_fwd_trace_cta && gp < 120 && lane == 0) ? g_attn_fwd_trace : nullptr;
         if (tr) tr[2048 + gp * 8] = clock64();
         tc_fence_after();
-        const uint64_t bd0 = dV0 + static_cast<uint64_t>((vs * Cfg::KV_BYTES) >> 4);
-        const uint32_t d_addr = tmem_u + Cfg::O_COL0 + t * DH;
+        const uint64_t bd0 = dV0 + static_cast<uint64_t>((vs * Cfg::V_BYTES) >> 4);
+        const uint32_t d_addr = tmem_u + Cfg::O_COL0 + t * DV;
         const uint32_t a_addr = tmem_u + Cfg::S_COL0 + buf * BKV;
         const uint32_t acc0 = wp.j > 0 ? 1u : 0u;
         const bool last_kv = wp.last_of_kv();
@@ -400,7 +427,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
         return ok;
       };
-      AFWalk<PIECES> ws;
+      Walk ws;
       ws.init(p, BKV);
       for (uint32_t gs = 0; ws.valid && ok; ws.advance(), ++gs) {
         const int t = ws.t;
@@ -411,21 +438,22 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           if (!wait1(Cfg::B_QF + t, (t ? qc1 : qc0) & 1u, 960)) break;
           if (t) ++qc1; else ++qc0;
         }
-        const int ks = ws.kv_seq % KST;
-        if (k_waited != ws.kv_seq) {
-          if (!wait1(Cfg::B_KF + ks, (ws.kv_seq / KST) & 1u, 961)) break;
-          k_waited = ws.kv_seq;
+        const int k_seq = DIFF ? static_cast<int>(gs) : ws.kv_seq;    // K tiles that came before
+        const int ks = k_seq % KST;
+        if (k_waited != k_seq) {
+          if (!wait1(Cfg::B_KF + ks, (k_seq / KST) & 1u, 961)) break;
+          k_waited = k_seq;
         }
         long long* tr = (blockIdx.x == g_attn_fwd_trace_cta && gs < 120 && lane == 0) ? g_attn_fwd_trace : nullptr;
         if (tr) tr[2048 + gs * 8 + 2] = clock64();
         tc_fence_after();
         const uint64_t ad0 = dQ0 + static_cast<uint64_t>((t * Cfg::Q_BYTES) >> 4);
-        const uint64_t bd0 = dK0 + static_cast<uint64_t>((ks * Cfg::KV_BYTES) >> 4);
+        const uint64_t bd0 = dK0 + static_cast<uint64_t>((ks * Cfg::K_BYTES) >> 4);
         const uint32_t d_addr = tmem_u + Cfg::S_COL0 + buf * BKV;
-        const bool last_tile = ws.last_of_tile(), last_kv = ws.last_of_kv();
+        const bool last_tile = ws.last_of_tile(), last_kv = DIFF || ws.last_of_kv();
         if (elect_one()) {
 #pragma unroll
-          for (int kk = 0; kk < DH / 16; ++kk) {
+          for (int kk = 0; kk < DQ / 16; ++kk) {
             const uint64_t a_off = static_cast<uint64_t>(((kk / 4) * (AF_BM * 128) + (kk % 4) * 32) >> 4);
             const uint64_t b_off = static_cast<uint64_t>(((kk / 4) * (BKV * 128) + (kk % 4) * 32) >> 4);
             umma_bf16_ss(d_addr, ad0 + a_off, bd0 + b_off, idesc_s, kk > 0 ? 1u : 0u);
@@ -447,17 +475,18 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const int quarter = warp & 3;
     const int r = quarter * 32 + lane;         // query row within the tile = TMEM lane
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
-    const uint32_t o_addr = lane_addr + Cfg::O_COL0 + t * DH;
+    const uint32_t o_addr = lane_addr + Cfg::O_COL0 + t * DV;
+    uint32_t items = 0;                          // DIFF: items finished
     uint32_t g = 0, g_prev = 0, mine = 0, own_seen = 0;
     bool ok = true;
     float m_used = -INFINITY;
     float l[4] = {0.f, 0.f, 0.f, 0.f};           // the row sum is kept as four partial sums
-    AFWalk<PIECES> w;
+    Walk w;
     w.init(p, BKV);
     for (; w.valid && ok; w.advance(), ++g) {
       if (w.t != t) continue;
       const int j = w.j;
-      const int q0 = (w.qa + t) * AF_BM;
+      const int q0 = w.tile() * AF_BM;
       const int q_idx = q0 + r;
       if (j == 0) {
         m_used = -INFINITY;
@@ -523,6 +552,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       for (int c = 0; c < BKV / 32; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v + c * 32);
       tmem_ld_wait();
       if (tr) tr[tri + 1] = clock64();
+      if constexpr (CAP) {
+#pragma unroll
+        for (int e = 0; e < BKV; ++e)
+          v[e] = __float_as_uint(p.cap_log2 * tanh_exp(__uint_as_float(v[e]) * p.cap_in));
+      }
       if (need_mask) {
         // hidden keys get a score of -inf, after which the step takes the common path (their
         // exponential is an exact zero); with causal masking every row sees at least key 0, with
@@ -544,7 +578,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
         mx = fmaxf(fmaxf(m0, m1), fmaxf(m2, m3));
       }
-      mx *= p.scale_log2;  // scale > 0, so max commutes with it
+      if constexpr (!CAP) mx *= p.scale_log2;  // scale > 0, so max commutes with it
       const float m_new = fmaxf(m_used, mx);
       const bool grow = (m_new - m_used) > 8.0f;  // also true for the first step (m_used = -inf)
       if (j > 0 && __any_sync(0xffffffffu, grow)) {
@@ -560,7 +594,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         tc_fence_after();
         const float f = grow ? fast_exp2(m_used - m_new) : 1.0f;
 #pragma unroll 1
-        for (int c = 0; c < DH / 16; ++c) {
+        for (int c = 0; c < DV / 16; ++c) {
           uint32_t o[16];
           tmem_ld_32x32b_x16(o_addr + c * 16, o);
           tmem_ld_wait();
@@ -576,7 +610,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (grow) m_used = (m_new == -INFINITY) ? 0.f : m_new;
       else if (PIECES && m_used == -INFINITY) m_used = -1e30f;
       // P = exp2(s * scale - m) as packed bf16 over the first half of the score buffer; row sum
-      const float sc = p.scale_log2, nm = -m_used;
+      const float sc = CAP ? 1.0f : p.scale_log2, nm = -m_used;
       if (tr) tr[tri + 2] = clock64();
       if constexpr (DROP) {
         // four consecutive keys share one hash; the index of this row's first key of the tile is
@@ -645,15 +679,78 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       float inv_l = lsum > 0.f ? 1.0f / lsum : 0.f;
       const bool row_ok = q_idx < w.rows(p);
       const size_t out_row = static_cast<size_t>(w.first_row(p)) + q_idx;
+      if constexpr (DIFF) {
+        float* x_norm = reinterpret_cast<float*>(smem + Cfg::OFF_X);      // [2][AF_BM] 1 / row sums
+        float* x_sum = x_norm + 2 * AF_BM;                                // [2][AF_BM] sums of squares
+        auto meet = [&](int which) {
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(bar(Cfg::B_X + which));
+          const bool got = mbar_wait(bar(Cfg::B_X + which), items & 1u, abort_flag);
+          if (!__all_sync(0xffffffffu, got)) {
+            if (lane == 0) record_status(p.status, ST_WAIT_TIMEOUT, 974 + which);
+            return false;
+          }
+          tc_fence_after();
+          return true;
+        };
+        x_norm[t * AF_BM + r] = inv_l;
+        ok = meet(0);
+        if (!ok) break;
+        const float n0 = x_norm[r], n1 = -*p.map_weight * x_norm[AF_BM + r];
+        constexpr int HALF = DV / 2;
+        const uint32_t half_addr = lane_addr + Cfg::O_COL0 + t * HALF;
+        float y[HALF], ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < HALF / 16; ++c) {
+          uint32_t a[16], b[16];
+          tmem_ld_32x32b_x16(half_addr + c * 16, a);
+          tmem_ld_32x32b_x16(half_addr + DV + c * 16, b);
+          tmem_ld_wait();
+#pragma unroll
+          for (int e = 0; e < 16; ++e) {
+            const float o = __uint_as_float(a[e]) * n0 + __uint_as_float(b[e]) * n1;
+            y[c * 16 + e] = o;
+            ss += o * o;
+          }
+        }
+        x_sum[t * AF_BM + r] = ss;
+        ok = meet(1);           // both have read both results: the next item may overwrite them
+        if (!ok) break;
+        ++items;
+        if (!row_ok) continue;
+        const float f = p.map_factor / sqrtf((x_sum[r] + x_sum[AF_BM + r]) / p.vdim + p.map_eps);
+        __nv_bfloat16* dst = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * p.vdim + t * HALF;
+        const int left = p.vdim - t * HALF;
+        const bool vec = (p.vdim & 7) == 0;
+#pragma unroll
+        for (int gq = 0; gq < HALF / 8; ++gq) {
+          if (vec) {
+            if (gq * 8 < left) {
+              uint4 wv;
+              wv.x = pack_bf16x2(y[8 * gq + 0] * f, y[8 * gq + 1] * f);
+              wv.y = pack_bf16x2(y[8 * gq + 2] * f, y[8 * gq + 3] * f);
+              wv.z = pack_bf16x2(y[8 * gq + 4] * f, y[8 * gq + 5] * f);
+              wv.w = pack_bf16x2(y[8 * gq + 6] * f, y[8 * gq + 7] * f);
+              *reinterpret_cast<uint4*>(dst + gq * 8) = wv;
+            }
+          } else {
+#pragma unroll
+            for (int x = 0; x < 8; ++x)
+              if (gq * 8 + x < left) dst[gq * 8 + x] = __float2bfloat16(y[8 * gq + x] * f);
+          }
+        }
+        continue;
+      }
       if constexpr (PIECES) {
         if (p.sink != nullptr)
           inv_l = 1.0f / (lsum + exp2f(p.sink[w.h] * 1.4426950408889634f - m_used));
         if (p.gate != nullptr && row_ok && !p.gate_wide)
           inv_l /= 1.0f + expf(-__bfloat162float(p.gate[out_row * p.ldg + w.h]));
       }
-      __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * (PIECES ? p.vdim : DH);
+      __nv_bfloat16* orow = p.O + out_row * p.ldo + static_cast<size_t>(w.h) * (PIECES ? p.vdim : DV);
 #pragma unroll 1
-      for (int c = 0; c < DH / 32; ++c) {
+      for (int c = 0; c < DV / 32; ++c) {
         uint32_t o[32];
         tmem_ld_32x32b_x32(o_addr + c * 32, o);
         tmem_ld_wait();
@@ -714,23 +811,23 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
-template <int DH, bool POLY, bool DROP = false, bool PIECES = false>
+template <int DQ, int DV, bool POLY, bool DROP = false, bool PIECES = false, bool CAP = false, bool DIFF = false>
 static int launch_attn_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
                               const AttnFwdArgs& a, int max_ctas, cudaStream_t st) {
-  using Cfg = AFCfg<DH>;
+  using Cfg = AFCfg<DQ, DV, DIFF>;
   static bool configured = false;
+  auto kern = attn_fwd_kernel<DQ, DV, POLY, DROP, PIECES, CAP, DIFF>;
   if (!configured) {
-    if (cudaFuncSetAttribute(attn_fwd_kernel<DH, POLY, DROP, PIECES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             Cfg::SMEM_BYTES) != cudaSuccess)
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES) != cudaSuccess)
       return -10;
     configured = true;
   }
   const int n_q_tiles = (a.S + AF_BM - 1) / AF_BM;
-  const int items = ((n_q_tiles + 1) / 2) * a.B * a.nh;
+  const int items = (DIFF ? n_q_tiles : (n_q_tiles + 1) / 2) * a.B * a.nh;
   int grid = sm_count();
   if (max_ctas > 0 && max_ctas < grid) grid = max_ctas;
   if (items < grid) grid = items;
-  attn_fwd_kernel<DH, POLY, DROP, PIECES><<<grid, AF_THREADS, Cfg::SMEM_BYTES, st>>>(tq, tk, tv, a);
+  kern<<<grid, AF_THREADS, Cfg::SMEM_BYTES, st>>>(tq, tk, tv, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
 }
 
@@ -759,7 +856,7 @@ extern "C" int cb_attn_fwd_dropout(const void* q, const void* k, const void* v, 
   if (drop_thr < 0 || drop_thr > 255 || (drop_thr > 0 && (S % 4) != 0)) return -6;
   CUtensorMap tq, tk, tv;
   const uint64_t rows = static_cast<uint64_t>(B) * S;
-  const uint32_t bkv = dh == 64 ? AFCfg<64>::BKV : AFCfg<128>::BKV;
+  const uint32_t bkv = AFCfg<64, 64>::BKV;
   if (make_tmap_bf16_2d(&tq, q, static_cast<uint64_t>(nh) * dh, rows, ldq, 64, AF_BM) != 0) return -3;
   if (make_tmap_bf16_2d(&tk, k, static_cast<uint64_t>(nkv) * dh, rows, ldk, 64, bkv) != 0) return -4;
   if (make_tmap_bf16_2d(&tv, v, static_cast<uint64_t>(nkv) * dh, rows, ldv, 64, bkv) != 0) return -5;
@@ -783,13 +880,13 @@ extern "C" int cb_attn_fwd_dropout(const void* q, const void* k, const void* v, 
   a.drop_scale = 256.0f / static_cast<float>(256 - drop_thr);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (drop_thr > 0)
-    return dh == 64 ? launch_attn_fwd<64, false, true>(tq, tk, tv, a, max_ctas, st)
-                    : launch_attn_fwd<128, false, true>(tq, tk, tv, a, max_ctas, st);
+    return dh == 64 ? launch_attn_fwd<64, 64, false, true>(tq, tk, tv, a, max_ctas, st)
+                    : launch_attn_fwd<128, 128, false, true>(tq, tk, tv, a, max_ctas, st);
   if (poly)
-    return dh == 64 ? launch_attn_fwd<64, true>(tq, tk, tv, a, max_ctas, st)
-                    : launch_attn_fwd<128, true>(tq, tk, tv, a, max_ctas, st);
-  return dh == 64 ? launch_attn_fwd<64, false>(tq, tk, tv, a, max_ctas, st)
-                  : launch_attn_fwd<128, false>(tq, tk, tv, a, max_ctas, st);
+    return dh == 64 ? launch_attn_fwd<64, 64, true>(tq, tk, tv, a, max_ctas, st)
+                    : launch_attn_fwd<128, 128, true>(tq, tk, tv, a, max_ctas, st);
+  return dh == 64 ? launch_attn_fwd<64, 64, false>(tq, tk, tv, a, max_ctas, st)
+                  : launch_attn_fwd<128, 128, false>(tq, tk, tv, a, max_ctas, st);
 }
 
 extern "C" int cb_attn_fwd(const void* q, const void* k, const void* v, void* o, float* lse,
@@ -801,28 +898,34 @@ extern "C" int cb_attn_fwd(const void* q, const void* k, const void* v, void* o,
 }
 
 // Causal attention of a ragged batch in pieces (see AttnFwdArgs): n_pieces quadruples over `rows`
-// query rows and `kv_rows` key rows, none with more than max_len queries.  Heads of q, k and v are
-// dh apart (64 or 128, padded with zeros), heads of o vdim <= dh.  sink (fp32 [nh]) is a logit per head
-// that enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view, or with
+// query rows and `kv_rows` key rows, none with more than max_len queries.  Heads of q and k are dq
+// apart, heads of v dv (64 or 128, padded with zeros), heads of o vdim <= dv.  sink (fp32 [nh]) is a logit
+// per head that enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view, or with
 // gate_wide column h * vdim + d) multiplies head h's output by its sigmoid; both may be null.  A
-// query sees the last `window` of its keys (0: all).  scale > 0.
+// query sees the last `window` of its keys (0: all).  scale > 0.  Scores are capped by softcap (0: not).
+// With two maps q and k have two heads per head (map 0 first), and the output is the weighted difference
+// divided by its root mean square, times map_factor; it has neither sink, gate nor cap.
 extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, void* o, int rows,
                                   int kv_rows, const void* pieces, int n_pieces, int max_len, int nh,
-                                  int nkv, int dh, int vdim, int ldq, int ldk, int ldv, int ldo,
+                                  int nkv, int dq, int dv, int vdim, int ldq, int ldk, int ldv, int ldo,
                                   float scale, const float* sink, const void* gate, int ldg,
-                                  int gate_wide, int window, int* status, void* stream) {
+                                  int gate_wide, int window, float softcap, int maps,
+                                  const float* map_weight, float map_factor, float map_eps, int* status,
+                                  void* stream) {
   using namespace cb;
-  if (dh != 64 && dh != 128) return -1;
+  if (!(dq == 64 && dv == 64) && !(dq == 128 && dv == 128) && !(dq == 64 && dv == 128 && maps == 2)) return -1;
   if (gate_wide && vdim % 8 == 0 && ((reinterpret_cast<uintptr_t>(gate) & 15u) || ldg % 8)) return -6;
-  if (window < 0) return -2;
+  if (window < 0 || softcap < 0.f || (maps != 1 && maps != 2)) return -2;
+  if (maps == 2 && (sink != nullptr || gate != nullptr || softcap > 0.f || map_weight == nullptr)) return -7;
+  if (softcap > 0.f && sink != nullptr) return -7;
   if (rows <= 0 || kv_rows <= 0 || n_pieces <= 0 || max_len <= 0 || nh <= 0 || nkv <= 0 ||
-      (nh % nkv) != 0 || (ldo % 8) != 0 || vdim < 1 || vdim > dh || !(scale > 0.f))
+      (nh % nkv) != 0 || (ldo % 8) != 0 || vdim < 1 || vdim > dv || !(scale > 0.f))
     return -2;
   CUtensorMap tq, tk, tv;
-  const uint32_t bkv = dh == 64 ? AFCfg<64>::BKV : AFCfg<128>::BKV;
-  if (make_tmap_bf16_2d(&tq, q, static_cast<uint64_t>(nh) * dh, rows, ldq, 64, AF_BM) != 0) return -3;
-  if (make_tmap_bf16_2d(&tk, k, static_cast<uint64_t>(nkv) * dh, kv_rows, ldk, 64, bkv) != 0) return -4;
-  if (make_tmap_bf16_2d(&tv, v, static_cast<uint64_t>(nkv) * dh, kv_rows, ldv, 64, bkv) != 0) return -5;
+  const uint32_t bkv = AFCfg<64, 64>::BKV;
+  if (make_tmap_bf16_2d(&tq, q, static_cast<uint64_t>(nh) * maps * dq, rows, ldq, 64, AF_BM) != 0) return -3;
+  if (make_tmap_bf16_2d(&tk, k, static_cast<uint64_t>(nkv) * maps * dq, kv_rows, ldk, 64, bkv) != 0) return -4;
+  if (make_tmap_bf16_2d(&tv, v, static_cast<uint64_t>(nkv) * dv, kv_rows, ldv, 64, bkv) != 0) return -5;
   AttnFwdArgs a = {};
   a.B = n_pieces; a.S = max_len; a.nh = nh; a.nkv = nkv;
   a.O = static_cast<__nv_bfloat16*>(o);
@@ -838,7 +941,21 @@ extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, v
   a.ldg = ldg;
   a.gate_wide = gate_wide;
   a.window = window;
+  a.map_weight = map_weight;
+  a.map_factor = map_factor;
+  a.map_eps = map_eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return dh == 64 ? launch_attn_fwd<64, false, false, true>(tq, tk, tv, a, 0, st)
-                  : launch_attn_fwd<128, false, false, true>(tq, tk, tv, a, 0, st);
+  if (maps == 2) {
+    if (dv == 64) return launch_attn_fwd<64, 64, false, false, true, false, true>(tq, tk, tv, a, 0, st);
+    return dq == 64 ? launch_attn_fwd<64, 128, false, false, true, false, true>(tq, tk, tv, a, 0, st)
+                    : launch_attn_fwd<128, 128, false, false, true, false, true>(tq, tk, tv, a, 0, st);
+  }
+  if (softcap > 0.f) {
+    a.cap_log2 = softcap * 1.4426950408889634f;
+    a.cap_in = scale / softcap;
+    return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, true>(tq, tk, tv, a, 0, st)
+                    : launch_attn_fwd<128, 128, false, false, true, true>(tq, tk, tv, a, 0, st);
+  }
+  return dv == 64 ? launch_attn_fwd<64, 64, false, false, true>(tq, tk, tv, a, 0, st)
+                  : launch_attn_fwd<128, 128, false, false, true>(tq, tk, tv, a, 0, st);
 }

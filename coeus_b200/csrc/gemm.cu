@@ -12,8 +12,10 @@
 //   dgrad    dX[M,K] = dY[M,N]  . W[K,N]^T    A K-major,  B K-major
 //   wgrad    dW[K,N] = X[M,K]^T . dY[M,N]     A MN-major, B MN-major (split along tokens,
 //                                             fp32 atomic accumulation)
+// Blocks of 128 rows of A may each have a weight of their own (experts whose rows are sorted).
 // Fused epilogues: alpha scale, +bias[N], GELU(tanh) with the pre-activation kept, dGELU, squared
-// ReLU, GELU(erf), +residual, bf16 / fp32 / fp32-atomic-add output.
+// ReLU, GELU(erf), +residual, bounded gated unit over alternating columns, bf16 / fp32 /
+// fp32-atomic-add output.
 #include <cudaTypedefs.h>
 
 #include <cstring>
@@ -31,7 +33,7 @@ constexpr int MAX_TP = 8;
 enum : int { COMM_NONE = 0, COMM_AG = 1, COMM_RS = 2 };
 
 enum : int { EPI_NONE = 0, EPI_GELU = 1, EPI_DGELU = 2, EPI_SWIGLU_BWD = 3, EPI_RELU2 = 4,
-             EPI_GELU_ERF = 6 };
+             EPI_GELU_ERF = 6, EPI_GLU = 7 };
 enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_F32_ATOMIC = 2, OUT_DISCARD = 3 };
 
 struct GemmArgs {
@@ -57,6 +59,8 @@ struct GemmArgs {
   int group_m;                  // output rows per group; 0 = one group.  Group g of a tile adds
   int g_am, g_ak;               // g * g_am to A's m coordinate, g * g_ak to its k coordinate,
   int g_bn, g_bk;               // g * g_bn to B's n coordinate, g * g_bk to its k coordinate
+  const int* block_group;       // group of every GEMM_BM rows instead (-1: none from here on), or null
+  float glu_slope, glu_limit;   // EPI_GLU: columns alternate g, u; the output has half as many
   // ---- fused collectives over peer memory (COMM template parameter)
   int tp, rank;                 // ranks of the tensor-parallel group, this rank
   int tiles_per_shard;          // 128-row tiles per rank's sequence shard
@@ -301,6 +305,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     else return (mi + p.rank * p.tiles_per_shard) % tiles_m;
   };
 
+  // Group of an m-block; negative: no work from here on.
+  auto group_of = [&](int m_blk) {
+    if constexpr (COMM == COMM_NONE && !CTA2)
+      if (p.block_group != nullptr) return p.block_group[m_blk];
+    return p.group_m > 0 ? (m_blk * TILE_M) / p.group_m : 0;
+  };
+
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
@@ -317,7 +328,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         const int kb0 = split * kb_per;
         const int kb1 = min(kblocks, kb0 + kb_per);
         // grouped GEMM: the tile's group shifts where its operands start
-        const int grp = p.group_m > 0 ? (m_blk * TILE_M) / p.group_m : 0;
+        const int grp = group_of(m_blk);
+        if (grp < 0) break;
         const int am0 = m0 + grp * p.g_am, ak0 = grp * p.g_ak;
         const int bn_off = grp * p.g_bn, bk0 = grp * p.g_bk;
         if constexpr (COMM == COMM_AG) {
@@ -433,6 +445,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         return ok;
       };
       for (int w = first_tile; w < total && ok; w += tile_step, ++it) {
+        if (group_of(m_block_of(w / p.ksplit)) < 0) break;
         const int split = w % p.ksplit;
         const int kb0 = split * kb_per;
         const int kb1 = min(kblocks, kb0 + kb_per);
@@ -594,6 +607,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     for (int w = first_tile; w < total; w += tile_step, ++it) {
       const int tile = w / p.ksplit;
       const int m_blk = m_block_of(tile);
+      if (group_of(m_blk) < 0) break;
       const int m0 = m_blk * TILE_M + static_cast<int>(cta_rank) * GEMM_BM;
       const int n0 = (tile % tiles_n) * BN;
       const int acc = it & 1;
@@ -611,7 +625,38 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       const int row = m0 + r_in_tile;
       const bool row_ok = row < p.M;
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + acc * BN;
-      if (p.tma_store) {
+      if (p.epi == EPI_GLU) {
+        // 128 columns of the accumulator make one 64-column store tile
+#pragma unroll 1
+        for (int qs = 0; qs < BN / 128; ++qs) {
+          if (n0 + qs * 128 >= p.N) break;
+          const uint32_t s_out = s_staging + (step & 1u) * 16384;
+          if (leader) asm volatile("cp.async.bulk.wait_group.read 1;" ::: "memory");
+          asm volatile("bar.sync 1, 128;" ::: "memory");
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            float v[32];
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+              uint32_t r[32];
+              tmem_ld_32x32b_x32(taddr + qs * 128 + h * 64 + half * 32, r);
+              tmem_ld_wait();
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                v[half * 16 + j] = clamped_glu(__uint_as_float(r[2 * j]), __uint_as_float(r[2 * j + 1]),
+                                               p.glu_slope, p.glu_limit);
+            }
+            stage_row(s_out, r_in_tile, h, v);
+          }
+          fence_proxy_async_smem();
+          asm volatile("bar.sync 1, 128;" ::: "memory");
+          if (leader && m0 < p.M) {
+            tma_store_2d(&tmD, s_out, n0 / 2 + qs * 64, m0);
+            tma_store_commit();
+          }
+          ++step;
+        }
+      } else if (p.tma_store) {
 #pragma unroll 1
         for (int qs = 0; qs < BN / 64; ++qs) {
           const int colq = n0 + qs * 64;
@@ -1023,6 +1068,45 @@ extern "C" int cb_gemm_bf16_grouped(const void* A, const void* B, void* D, int g
   return gemm_bf16_impl(A, B, D, M, N, K, lda, ldb, ldd, a_mn, b_mn, nullptr, nullptr, 0, nullptr,
                         nullptr, 0, cb::EPI_NONE, out_mode, alpha, ksplit, bn, status, max_ctas,
                         stream, groups);
+}
+
+// D[rows of block b] = epilogue(A[rows of block b] . B[block_expert[b]]^T), blocks of 128 rows: A [M, K],
+// B [experts, N, K] (pitch ldb), D [M, N] or with glu (a bounded gated unit over alternating columns)
+// [M, N / 2], all bf16.  A negative entry says that this block and all behind it have no work; their
+// rows of D are left alone.  block_expert null: one weight, any M.
+extern "C" int cb_gemm_bf16_blocks(const void* A, const void* B, void* D, int M, int N, int K, int experts,
+                                   int lda, int ldb, int ldd, const int* block_expert, int glu,
+                                   float slope, float limit, int* status, void* stream) {
+  using namespace cb;
+  const int cols = glu ? N / 2 : N;
+  if (M <= 0 || N <= 0 || K <= 0 || experts < 1 || N % 8 || cols % 8 || K % 8 || ldd % 8) return -21;
+  if (block_expert != nullptr && M % GEMM_BM) return -24;
+  if (reinterpret_cast<uintptr_t>(D) & 15u) return -21;
+  const bool pairs = block_expert == nullptr && M >= 256 && N > 128;
+  const long long wide = static_cast<long long>((M + GEMM_BM - 1) / GEMM_BM) * ((N + 255) / 256);
+  const int bn = pairs || (N > 128 && wide >= 4 * sm_count()) ? 256 : 128;
+  CUtensorMap ta, tb, td;
+  if (make_tmap_bf16_2d(&ta, A, K, M, lda, 64, GEMM_BM) != 0) return -30;
+  if (make_tmap_bf16_2d(&tb, B, K, static_cast<uint64_t>(experts) * N, ldb, 64, pairs ? 128 : bn) != 0) return -40;
+  if (make_tmap_bf16_2d(&td, D, cols, M, ldd, 64, GEMM_BM) != 0) return -45;
+  GemmArgs g;
+  std::memset(&g, 0, sizeof(g));
+  g.tma_store = 1;
+  g.tp = 1;
+  g.tiles_per_shard = 1;
+  g.M = M; g.N = N; g.K = K;
+  g.D = D; g.ldd = ldd;
+  g.epi = glu ? EPI_GLU : EPI_NONE;
+  g.out_mode = OUT_BF16; g.alpha = 1.0f; g.ksplit = 1; g.status = status;
+  g.drop_scale = 1.0f;
+  g.block_group = block_expert;
+  g.g_bn = N;
+  g.glu_slope = slope;
+  g.glu_limit = limit;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (pairs) return launch_gemm_pair<false, false>(ta, tb, td, td, g, 0, st);
+  return bn == 256 ? launch_gemm<256, false, false>(ta, tb, td, td, g, 0, st)
+                   : launch_gemm<128, false, false>(ta, tb, td, td, g, 0, st);
 }
 
 // ------------------------------------------------------------------------------------------

@@ -1,8 +1,14 @@
 // Attention of a ragged batch over the paged cache: every query row sits at its own position of
-// its own sequence and sees the cached keys of its chunk up to itself (chunk = 0: all of them).
-// The softmax may have a sink per head (a logit in the denominator only) and the head's output a
-// gate (a sigmoid of a projected number).  Query head h reads key/value head h / (heads / kv_heads);
-// query/key width and value width are independent.
+// its own sequence and sees the cached keys of its chunk or its sliding window up to itself (both 0: all
+// of them).  Scores may be capped (s -> cap tanh(s / cap)), the softmax may have a sink per head (a logit
+// in the denominator only) and the head's output a gate (a sigmoid of a projected number, one per head or
+// one per number).  Query head h reads key/value head h / (heads / kv_heads); query/key width and value
+// width are independent.
+//
+// With two maps a head has two queries and a key head two keys over the same values, and the head's
+// output is (a0 - w a1) / rms * factor of the two results.  A cached key is then the keys of both maps
+// side by side; a query of one map is zero at the other's places, so that both maps of a group share
+// every load, and two maps are twice as many query heads on a key twice as wide.
 //
 //   rows kernel    one CTA per (query row, key/value head, split): the query heads of the group
 //                  share every key and value that is loaded.  Everything in fp32, and decoding
@@ -17,35 +23,60 @@ namespace cb {
 
 constexpr float LOG2E = 1.4426950408889634f;
 
+struct RaggedSpec {        // as the host gives it
+  int heads, kv_heads, dim, vdim, dim_p, vdim_p, chunk, window, maps, gate_wide;
+  float scale, softcap, map_factor, eps;
+};
+
 struct RaggedAttn {
   const void* q;           // [rows, heads, q_head]
   int q_head;
-  const void* k_cache;     // [pages, PAGE, kv_heads, dim_p]
+  const void* k_cache;     // [pages, PAGE, kv_heads, kdim]
   const void* v_cache;     // [pages, PAGE, kv_heads, vdim_p]
   const int* page_table;   // [slots, max_pages]
   int max_pages, num_pages;
-  int heads, kv_heads, dim, vdim, dim_p, vdim_p;
-  int chunk;
-  float scale;
+  int heads, kv_heads, dim, vdim, dim_p, vdim_p;    // heads: of all maps
+  int maps, kdim;          // kdim = maps * dim_p
+  int chunk, window;
+  float scale;             // products to units of log2, or with a cap to the tanh's argument
+  float cap;               // 0, or the cap in units of log2
   const float* sink;       // [heads] or null
-  const void* gate;        // [rows, ldg] or null: column h gates head h
-  int ldg;
+  const void* gate;        // [rows, ldg] or null: column h gates head h, or (gate_wide) h * vdim + d
+  int ldg, gate_wide;
+  const float* map_weight; // two maps: weight of the second
+  float map_factor, eps;
   void* out;               // [rows, ldo]
   int ldo;
   int* status;
 };
 
-__device__ __forceinline__ int chunk_start(int pos, int chunk) {
-  return chunk > 0 ? pos / chunk * chunk : 0;
+// First position that position pos sees; it does not fall as pos grows.
+__device__ __forceinline__ int first_seen(const RaggedAttn& p, int pos) {
+  if (p.window > 0) return max(0, pos + 1 - p.window);
+  return p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
 }
 template <typename T>
 __device__ __forceinline__ float exp2_t(float x) {
   if constexpr (sizeof(T) == 4) return exp2f(x);
   else return fast_exp2(x);
 }
+// A product of a query and a key (times p.scale) to a score in units of log2.
+template <typename T>
+__device__ __forceinline__ float score_of(const RaggedAttn& p, float s) {
+  if (p.cap == 0.f) return s;
+  if constexpr (sizeof(T) == 4) return p.cap * tanhf(s);
+  else return p.cap * tanh_exp(s);
+}
+// Column of the key's row where the query of head h starts.
+__device__ __forceinline__ int map_off(const RaggedAttn& p, int h) { return p.maps == 2 ? (h & 1) * p.dim_p : 0; }
+template <typename T>
+__device__ __forceinline__ float gate_wide_of(const RaggedAttn& p, int row, int col) {
+  if (p.gate == nullptr || !p.gate_wide) return 1.f;
+  return sigmoidf_(to_f32(static_cast<const T*>(p.gate)[static_cast<size_t>(row) * p.ldg + col]));
+}
 template <typename T>
 __device__ __forceinline__ float gate_of(const RaggedAttn& p, int row, int h) {
-  if (p.gate == nullptr) return 1.f;
+  if (p.gate == nullptr || p.gate_wide) return 1.f;
   return sigmoidf_(to_f32(static_cast<const T*>(p.gate)[static_cast<size_t>(row) * p.ldg + h]));
 }
 // Softmax denominator with the sink, in units of 2^m.
@@ -86,10 +117,11 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
   const T* qp = static_cast<const T*>(p.q) + static_cast<size_t>(row) * p.heads * p.q_head;
   for (int j = threadIdx.x; j < GM * DC; j += RA_WARPS * 32) {
     const int g = j / DC, d = j % DC;
-    sq[g][d] = (g < ng && d < p.dim) ? to_f32(qp[(h0 + g) * p.q_head + d]) * (p.scale * LOG2E) : 0.f;
+    const int c = d - map_off(p, h0 + g);
+    sq[g][d] = (g < ng && c >= 0 && c < p.dim) ? to_f32(qp[(h0 + g) * p.q_head + c]) * p.scale : 0.f;
   }
   __syncthreads();
-  const int lo = chunk_start(pos, p.chunk), n = pos + 1 - lo;
+  const int lo = first_seen(p, pos), n = pos + 1 - lo;
   const int piece = (n + ra.splits - 1) / ra.splits;
   const int t0 = lo + split * piece, t1 = min(pos + 1, t0 + piece);
   const T* kc = static_cast<const T*>(p.k_cache);
@@ -124,11 +156,11 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
 #pragma unroll
       for (int g = 0; g < GM; ++g) s[g] = 0.f;
       if (t < t1) {
-        const T* kp = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + t % RAGGED_PAGE) * p.kv_heads + hk) * p.dim_p;
+        const T* kp = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + t % RAGGED_PAGE) * p.kv_heads + hk) * p.kdim;
 #pragma unroll
         for (int c = 0; c < KIT; ++c) {
           const int d = ((lane & 7) + 8 * c) * 8;
-          if (d < p.dim_p) {
+          if (d < p.kdim) {
             float f[8];
             load_vec<8>(kp + d, f);
 #pragma unroll
@@ -153,7 +185,7 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
     // weights: one key per lane
 #pragma unroll
     for (int g = 0; g < GM; ++g) {
-      const float s = my_t < t1 ? sp[warp][lane][g] : -INFINITY;
+      const float s = my_t < t1 ? score_of<T>(p, sp[warp][lane][g]) : -INFINITY;
       const float mn = fmaxf(m[g], warp_max(s));          // finite: the block has a key
       const float c = exp2_t<T>(m[g] - mn), w = exp2_t<T>(s - mn);
       m[g] = mn;
@@ -209,16 +241,18 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
     }
     __syncthreads();
     const int h = h0 + g;
-    const float dn = ra.splits == 1 ? gate_of<T>(p, row, h) / denom<T>(p, h, gm, gl) : 1.f;
+    const bool direct = ra.part_o == nullptr;
+    const float dn = direct ? gate_of<T>(p, row, h) / denom<T>(p, h, gm, gl) : 1.f;
     for (int d = threadIdx.x; d < p.vdim; d += RA_WARPS * 32) {
       float o = 0.f;
       for (int w = 0; w < parts; ++w) o += red[w * p.vdim_p + d];
-      if (ra.splits == 1)
-        static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] = from_f32<T>(o * dn);
+      if (direct)
+        static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] =
+            from_f32<T>(o * dn * gate_wide_of<T>(p, row, h * p.vdim + d));
       else
         ra.part_o[((static_cast<size_t>(i) * p.heads + h) * ra.splits + split) * p.vdim + d] = o;
     }
-    if (ra.splits > 1 && threadIdx.x == 0) {
+    if (!direct && threadIdx.x == 0) {
       float* ml = ra.part_ml + ((static_cast<size_t>(i) * p.heads + h) * ra.splits + split) * 2;
       ml[0] = gm;
       ml[1] = gl;
@@ -246,7 +280,58 @@ __global__ void __launch_bounds__(64) ragged_attn_merge_kernel(const RowsArgs ra
       const float ms = ra.part_ml[(base + s) * 2];
       if (ms != -INFINITY) o += ra.part_o[(base + s) * p.vdim + d] * exp2_t<T>(ms - gm);
     }
-    static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] = from_f32<T>(o * dn);
+    static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] =
+        from_f32<T>(o * dn * gate_wide_of<T>(p, row, h * p.vdim + d));
+  }
+}
+
+// Two maps: merges the splits of both and takes their difference.  At most 256 columns.
+template <typename T>
+__global__ void __launch_bounds__(128) ragged_attn_difference_kernel(const RowsArgs ra) {
+  const RaggedAttn& p = ra.a;
+  __shared__ float red[32];
+  const int i = blockIdx.x, h = blockIdx.y;
+  const int row = ra.rows != nullptr ? ra.rows[i] : i;
+  const float w = *p.map_weight;
+  float o[2] = {0.f, 0.f};
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const size_t base = (static_cast<size_t>(i) * p.heads + h * 2 + m) * ra.splits;
+    float gm = -INFINITY, gl = 0.f;
+    for (int s = 0; s < ra.splits; ++s) gm = fmaxf(gm, ra.part_ml[(base + s) * 2]);
+    for (int s = 0; s < ra.splits; ++s) {
+      const float ms = ra.part_ml[(base + s) * 2];
+      gl += ms == -INFINITY ? 0.f : ra.part_ml[(base + s) * 2 + 1] * exp2_t<T>(ms - gm);
+    }
+    const float dn = (m == 0 ? 1.f : -w) / denom<T>(p, h * 2 + m, gm, gl);
+    for (int s = 0; s < ra.splits; ++s) {
+      const float ms = ra.part_ml[(base + s) * 2];
+      if (ms == -INFINITY) continue;
+      const float c = exp2_t<T>(ms - gm) * dn;
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int d = threadIdx.x + 128 * x;
+        if (d < p.vdim) o[x] += ra.part_o[(base + s) * p.vdim + d] * c;
+      }
+    }
+  }
+  const float ss = block_sum(o[0] * o[0] + o[1] * o[1], red);
+  const float rs = p.map_factor / sqrtf(ss / p.vdim + p.eps) * gate_of<T>(p, row, h);
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int d = threadIdx.x + 128 * x;
+    if (d < p.vdim)
+      static_cast<T*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] =
+          from_f32<T>(o[x] * rs * gate_wide_of<T>(p, row, h * p.vdim + d));
+  }
+}
+
+template <typename T>
+static void launch_merge(const RowsArgs& a, int n, cudaStream_t st) {
+  if (a.a.maps == 2) {
+    ragged_attn_difference_kernel<T><<<dim3(n, a.a.heads / 2), 128, 0, st>>>(a);
+  } else if (a.part_o != nullptr) {
+    ragged_attn_merge_kernel<T><<<dim3(n, a.a.heads), 64, 0, st>>>(a);
   }
 }
 
@@ -262,31 +347,37 @@ struct TilesArgs {
   const int* tile_len;     // [tiles] its tokens, at most TA_ROWS
 };
 
-template <int DC, int VC>   // dim <= DC, vdim <= VC, multiples of 32
-__global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const TilesArgs ta) {
+// dim <= DC, vdim <= VC, multiples of 32.  With two maps the block has warps for both: they share the
+// values, and the second map's results cross to the first map's warps through shared memory.
+template <int DC, int VC, int MAPS>
+__global__ void __launch_bounds__(MAPS * TA_WARPS * 32) ragged_attn_tiles_kernel(const TilesArgs ta) {
   using bf16 = __nv_bfloat16;
   const RaggedAttn& p = ta.a;
-  constexpr int KS = DC + 8, VS = VC + 8;       // padded rows (elements): conflict-free ldmatrix
+  constexpr int KS = MAPS * DC + 8, VS = VC + 8;       // padded rows (elements): conflict-free ldmatrix
+  constexpr int NT = MAPS * TA_WARPS * 32;
   extern __shared__ __align__(16) unsigned char smem[];
   bf16* sK = reinterpret_cast<bf16*>(smem);                      // [2][PAGE][KS]
   bf16* sV = sK + 2 * RAGGED_PAGE * KS;                          // [2][PAGE][VS]
   bf16* sQ = sV + 2 * RAGGED_PAGE * VS;                          // [TA_ROWS][KS]
   const int e = ta.tile_entry[blockIdx.x], off = ta.tile_off[blockIdx.x], h = blockIdx.y;
-  const int hk = h / (p.heads / p.kv_heads);
+  const int hk = h / (p.heads / MAPS / p.kv_heads);
   const int row0 = ta.e.row0[e] + off, len = min(TA_ROWS, ta.tile_len[blockIdx.x]);
   const int pos0 = ta.e.pos0[e] + off, slot = ta.e.slot[e];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int warp = (tid >> 5) % TA_WARPS, map = tid / (TA_WARPS * 32);
   const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
   const bf16* q = static_cast<const bf16*>(p.q);
   const bf16* kc = static_cast<const bf16*>(p.k_cache);
   const bf16* vc = static_cast<const bf16*>(p.v_cache);
   // padding columns of the rings are zero once and for all
-  for (int i = tid; i < 2 * RAGGED_PAGE * (KS - p.dim_p); i += TA_WARPS * 32)
-    sK[(i / (KS - p.dim_p)) * KS + p.dim_p + i % (KS - p.dim_p)] = __float2bfloat16(0.f);
-  for (int i = tid; i < 2 * RAGGED_PAGE * (VS - p.vdim_p); i += TA_WARPS * 32)
+#pragma unroll
+  for (int m = 0; m < MAPS; ++m)
+    for (int i = tid; i < 2 * RAGGED_PAGE * (DC - p.dim_p); i += NT)
+      sK[(i / (DC - p.dim_p)) * KS + m * DC + p.dim_p + i % (DC - p.dim_p)] = __float2bfloat16(0.f);
+  for (int i = tid; i < 2 * RAGGED_PAGE * (VS - p.vdim_p); i += NT)
     sV[(i / (VS - p.vdim_p)) * VS + p.vdim_p + i % (VS - p.vdim_p)] = __float2bfloat16(0.f);
   const int last = pos0 + len - 1;
-  const int pg0 = chunk_start(pos0, p.chunk) / RAGGED_PAGE, pg1 = last / RAGGED_PAGE;
+  const int pg0 = first_seen(p, pos0) / RAGGED_PAGE, pg1 = last / RAGGED_PAGE;
   auto fetch = [&](int pg, int st) {
     int page = pg < p.max_pages ? pt[pg] : -1;
     if (page < 0 || page >= p.num_pages) {
@@ -295,12 +386,13 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
     }
     const int base = pg * RAGGED_PAGE;
     const int kch = p.dim_p / 8, vch = p.vdim_p / 8;
-    for (int i = tid; i < RAGGED_PAGE * kch; i += TA_WARPS * 32) {
-      const int t = i / kch, c = i % kch;
-      const bf16* src = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + t) * p.kv_heads + hk) * p.dim_p + c * 8;
-      cp_async16_zfill(smem_u32(sK + (st * RAGGED_PAGE + t) * KS + c * 8), src, base + t <= last ? 16 : 0);
+    for (int i = tid; i < RAGGED_PAGE * MAPS * kch; i += NT) {
+      const int t = i / (MAPS * kch), c = i % (MAPS * kch), m = c / kch;
+      const bf16* src = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + t) * p.kv_heads + hk) * p.kdim + c * 8;
+      cp_async16_zfill(smem_u32(sK + (st * RAGGED_PAGE + t) * KS + m * DC + (c - m * kch) * 8), src,
+                       base + t <= last ? 16 : 0);
     }
-    for (int i = tid; i < RAGGED_PAGE * vch; i += TA_WARPS * 32) {
+    for (int i = tid; i < RAGGED_PAGE * vch; i += NT) {
       const int t = i / vch, c = i % vch;
       const bf16* src = vc + ((static_cast<size_t>(page) * RAGGED_PAGE + t) * p.kv_heads + hk) * p.vdim_p + c * 8;
       cp_async16_zfill(smem_u32(sV + (st * RAGGED_PAGE + t) * VS + c * 8), src, base + t <= last ? 16 : 0);
@@ -309,18 +401,18 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
   };
   fetch(pg0, 0);
   if (p.dim % 8 == 0 && p.q_head % 8 == 0) {
-    for (int i = tid; i < TA_ROWS * (DC / 8); i += TA_WARPS * 32) {
-      const int t = i / (DC / 8), c = (i % (DC / 8)) * 8;
+    for (int i = tid; i < TA_ROWS * MAPS * (DC / 8); i += NT) {
+      const int t = i / (MAPS * (DC / 8)), x = i % (MAPS * (DC / 8)), m = x / (DC / 8), c = x % (DC / 8) * 8;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (t < len && c < p.dim)
-        v = *reinterpret_cast<const uint4*>(q + (static_cast<size_t>(row0 + t) * p.heads + h) * p.q_head + c);
-      *reinterpret_cast<uint4*>(sQ + t * KS + c) = v;
+        v = *reinterpret_cast<const uint4*>(q + (static_cast<size_t>(row0 + t) * p.heads + h * MAPS + m) * p.q_head + c);
+      *reinterpret_cast<uint4*>(sQ + t * KS + m * DC + c) = v;
     }
   } else {
-    for (int i = tid; i < TA_ROWS * DC; i += TA_WARPS * 32) {
-      const int t = i / DC, c = i % DC;
-      sQ[t * KS + c] = (t < len && c < p.dim)
-                           ? q[(static_cast<size_t>(row0 + t) * p.heads + h) * p.q_head + c]
+    for (int i = tid; i < TA_ROWS * MAPS * DC; i += NT) {
+      const int t = i / (MAPS * DC), x = i % (MAPS * DC), m = x / DC, c = x % DC;
+      sQ[t * KS + x] = (t < len && c < p.dim)
+                           ? q[(static_cast<size_t>(row0 + t) * p.heads + h * MAPS + m) * p.q_head + c]
                            : __float2bfloat16(0.f);
     }
   }
@@ -328,7 +420,7 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
   uint32_t qf[DC / 16][4];
 #pragma unroll
   for (int k = 0; k < DC / 16; ++k)
-    ldsm4(qf[k], smem_u32(sQ + (warp * 16 + (lane & 15)) * KS + k * 16 + (lane >> 4) * 8));
+    ldsm4(qf[k], smem_u32(sQ + (warp * 16 + (lane & 15)) * KS + map * DC + k * 16 + (lane >> 4) * 8));
   float o[VC / 8][4];
 #pragma unroll
   for (int i = 0; i < VC / 8; ++i)
@@ -337,8 +429,7 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const int r0 = warp * 16 + (lane >> 2);
   const int qpos[2] = {pos0 + r0, pos0 + r0 + 8};
-  const int qlo[2] = {chunk_start(qpos[0], p.chunk), chunk_start(qpos[1], p.chunk)};
-  const float sl2 = p.scale * LOG2E;
+  const int qlo[2] = {first_seen(p, qpos[0]), first_seen(p, qpos[1])};
   const int w_first = pos0 + warp * 16, w_last = min(w_first + 15, last);
   for (int pg = pg0; pg <= pg1; ++pg) {
     const int st = (pg - pg0) & 1, base = pg * RAGGED_PAGE;
@@ -350,7 +441,7 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
     }
     __syncthreads();
     // skip pages that no row of this warp sees
-    if (w_first <= last && base <= w_last && base + RAGGED_PAGE > chunk_start(w_first, p.chunk)) {
+    if (w_first <= last && base <= w_last && base + RAGGED_PAGE > first_seen(p, w_first)) {
       float s[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i)
@@ -362,19 +453,19 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
 #pragma unroll
         for (int i = 0; i < 4; ++i) {       // 16 keys: two n-tiles
           uint32_t b[4];
-          ldsm4(b, smem_u32(kb + (i * 16 + (lane & 7) + (lane >> 4) * 8) * KS + k * 16 + ((lane >> 3) & 1) * 8));
+          ldsm4(b, smem_u32(kb + (i * 16 + (lane & 7) + (lane >> 4) * 8) * KS + map * DC + k * 16 + ((lane >> 3) & 1) * 8));
           mma_bf16(s[2 * i], qf[k], b[0], b[1]);
           mma_bf16(s[2 * i + 1], qf[k], b[2], b[3]);
         }
       }
-      const bool full = base >= chunk_start(w_last, p.chunk) && base + RAGGED_PAGE - 1 <= w_first;
+      const bool full = base >= first_seen(p, w_last) && base + RAGGED_PAGE - 1 <= w_first;
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int i = 0; i < 8; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int r = j >> 1, t = base + i * 8 + (lane & 3) * 2 + (j & 1);
-          s[i][j] = (full || (t <= qpos[r] && t >= qlo[r])) ? s[i][j] * sl2 : -INFINITY;
+          s[i][j] = (full || (t <= qpos[r] && t >= qlo[r])) ? score_of<bf16>(p, s[i][j] * p.scale) : -INFINITY;
           mx[r] = fmaxf(mx[r], s[i][j]);
         }
       float c[2], sum[2] = {0.f, 0.f};
@@ -432,15 +523,63 @@ __global__ void __launch_bounds__(TA_WARPS * 32) ragged_attn_tiles_kernel(const 
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
     const int t = r0 + r * 8;
+    const float dn = t < len ? 1.f / denom<bf16>(p, h * MAPS + map, m[r], l[r]) : 0.f;
+#pragma unroll
+    for (int i = 0; i < VC / 8; ++i) {
+      o[i][2 * r] *= dn;
+      o[i][2 * r + 1] *= dn;
+    }
+  }
+  if constexpr (MAPS == 2) {
+    float* other = reinterpret_cast<float*>(smem);         // [TA_ROWS][VC + 8]: the rings are free
+    constexpr int OS = VC + 8;
+    if (map == 1) {
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+#pragma unroll
+        for (int i = 0; i < VC / 8; ++i)
+          *reinterpret_cast<float2*>(other + (r0 + r * 8) * OS + i * 8 + (lane & 3) * 2) =
+              make_float2(o[i][2 * r], o[i][2 * r + 1]);
+    }
+    __syncthreads();
+    if (map == 1) return;
+    const float w = *p.map_weight;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < VC / 8; ++i) {
+        const float2 b = *reinterpret_cast<const float2*>(other + (r0 + r * 8) * OS + i * 8 + (lane & 3) * 2);
+        o[i][2 * r] -= w * b.x;
+        o[i][2 * r + 1] -= w * b.y;
+        ss += o[i][2 * r] * o[i][2 * r] + o[i][2 * r + 1] * o[i][2 * r + 1];
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      const float f = p.map_factor / sqrtf(ss / p.vdim + p.eps);
+#pragma unroll
+      for (int i = 0; i < VC / 8; ++i) {
+        o[i][2 * r] *= f;
+        o[i][2 * r + 1] *= f;
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int t = r0 + r * 8;
     if (t >= len) continue;
     const int row = row0 + t;
-    const float dn = gate_of<bf16>(p, row, h) / denom<bf16>(p, h, m[r], l[r]);
+    const float dn = gate_of<bf16>(p, row, h);
     bf16* dst = static_cast<bf16*>(p.out) + static_cast<size_t>(row) * p.ldo + h * p.vdim;
     const bool pairs = (p.vdim & 1) == 0 && (p.ldo & 1) == 0;
 #pragma unroll
     for (int i = 0; i < VC / 8; ++i) {
       const int d = i * 8 + (lane & 3) * 2;
-      const float u = o[i][r * 2] * dn, w = o[i][r * 2 + 1] * dn;
+      float u = o[i][r * 2] * dn, w = o[i][r * 2 + 1] * dn;
+      if (p.gate_wide) {
+        if (d < p.vdim) u *= gate_wide_of<bf16>(p, row, h * p.vdim + d);
+        if (d + 1 < p.vdim) w *= gate_wide_of<bf16>(p, row, h * p.vdim + d + 1);
+      }
       if (pairs) {
         if (d < p.vdim) *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(u, w);
       } else {
@@ -475,13 +614,13 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
   const int row = ra.rows != nullptr ? ra.rows[i] : i;
   const int slot = ra.row_slot[row], pos = ra.row_pos[row];
   const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
-  const bf16* kc = static_cast<const bf16*>(p.k_cache) + hk * p.dim_p;
+  const bf16* kc = static_cast<const bf16*>(p.k_cache) + hk * p.kdim;
   const bf16* vc = static_cast<const bf16*>(p.v_cache) + hk * p.vdim_p;
-  const int lo = chunk_start(pos, p.chunk), n = pos + 1 - lo;
+  const int lo = first_seen(p, pos), n = pos + 1 - lo;
   const int piece = (n + ra.splits - 1) / ra.splits;
   const int t0 = lo + split * piece, t1 = min(pos + 1, t0 + piece);
   bf16* mine = ring + warp * 2 * STAGE;
-  const int kch = p.dim_p / 8, vch = p.vdim_p / 8;
+  const int kch = p.kdim / 8, vch = p.vdim_p / 8;
   auto fetch = [&](int tb, int st) {                    // keys tb .. tb + 31 into a stage
     const int t = tb + lane;
     int page = 0;
@@ -499,7 +638,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
       const int key = x / kch, c = x % kch;
       const int pg = __shfl_sync(0xffffffffu, page, key);
       const size_t cell = static_cast<size_t>(pg) * RAGGED_PAGE + (tb + key) % RAGGED_PAGE;
-      cp_async16_zfill(smem_u32(kd + key * KS + c * 8), kc + cell * p.kv_heads * p.dim_p + c * 8,
+      cp_async16_zfill(smem_u32(kd + key * KS + c * 8), kc + cell * p.kv_heads * p.kdim + c * 8,
                        tb + key < t1 ? 16 : 0);
     }
     for (int x = lane; x < GA_KEYS * vch; x += 32) {
@@ -512,8 +651,8 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
     cp_async_commit();
   };
   // zero the padding columns of this warp's ring, then start loading
-  for (int x = lane; x < 2 * GA_KEYS * (DC - p.dim_p); x += 32) {
-    const int r = x / (DC - p.dim_p), c = p.dim_p + x % (DC - p.dim_p);
+  for (int x = lane; x < 2 * GA_KEYS * (DC - p.kdim); x += 32) {
+    const int r = x / (DC - p.kdim), c = p.kdim + x % (DC - p.kdim);
     mine[(r / GA_KEYS) * STAGE + (r % GA_KEYS) * KS + c] = __float2bfloat16(0.f);
   }
   for (int x = lane; x < 2 * GA_KEYS * (VC - p.vdim_p); x += 32) {
@@ -525,7 +664,8 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
   const bf16* q = static_cast<const bf16*>(p.q) + (static_cast<size_t>(row) * p.heads + h0) * p.q_head;
   for (int x = tid; x < 16 * DC; x += GA_WARPS * 32) {
     const int g = x / DC, d = x % DC;
-    sQ[g * KS + d] = g < ng && d < p.dim ? q[g * p.q_head + d] : __float2bfloat16(0.f);
+    const int c = d - map_off(p, h0 + g);
+    sQ[g * KS + d] = g < ng && c >= 0 && c < p.dim ? q[g * p.q_head + c] : __float2bfloat16(0.f);
   }
   __syncthreads();
   uint32_t qf[DC / 16][4];
@@ -537,7 +677,6 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
   for (int x = 0; x < VC / 8; ++x)
 #pragma unroll
     for (int j = 0; j < 4; ++j) o[x][j] = 0.f;
-  const float sl2 = p.scale * LOG2E;
   for (int st = 0; tb < t1; tb += GA_WARPS * GA_KEYS, st ^= 1) {
     if (tb + GA_WARPS * GA_KEYS < t1) {
       fetch(tb + GA_WARPS * GA_KEYS, st ^ 1);
@@ -568,7 +707,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int t = tb + x * 8 + (lane & 3) * 2 + (j & 1);
-        s[x][j] = t < t1 ? s[x][j] * sl2 : -INFINITY;
+        s[x][j] = t < t1 ? score_of<bf16>(p, s[x][j] * p.scale) : -INFINITY;
         mx[j >> 1] = fmaxf(mx[j >> 1], s[x][j]);
       }
 #pragma unroll
@@ -647,17 +786,19 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
     for (int w = 0; w < GA_WARPS; ++w)
       gl += sm_m[w][g] == -INFINITY ? 0.f : sm_l[w][g] * fast_exp2(sm_m[w][g] - gm);
     const size_t part = (static_cast<size_t>(i) * p.heads + h) * ra.splits + split;
-    const float dn = ra.splits == 1 ? gate_of<bf16>(p, row, h) / denom<bf16>(p, h, gm, gl) : 1.f;
+    const bool direct = ra.part_o == nullptr;
+    const float dn = direct ? gate_of<bf16>(p, row, h) / denom<bf16>(p, h, gm, gl) : 1.f;
     for (int d = lane; d < p.vdim; d += 32) {
       float v = 0.f;
 #pragma unroll
       for (int w = 0; w < GA_WARPS; ++w) v += red[(w * 16 + g) * VC + d];
-      if (ra.splits == 1)
-        static_cast<bf16*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] = __float2bfloat16(v * dn);
+      if (direct)
+        static_cast<bf16*>(p.out)[static_cast<size_t>(row) * p.ldo + h * p.vdim + d] =
+            __float2bfloat16(v * dn * gate_wide_of<bf16>(p, row, h * p.vdim + d));
       else
         ra.part_o[part * p.vdim + d] = v;
     }
-    if (ra.splits > 1 && lane == 0) {
+    if (!direct && lane == 0) {
       ra.part_ml[part * 2] = gm;
       ra.part_ml[part * 2 + 1] = gl;
     }
@@ -679,10 +820,7 @@ static int launch_group(const RowsArgs& a, int n, cudaStream_t st) {
   const int per = a.a.heads / a.a.kv_heads;
   dim3 grid(n, a.a.kv_heads * ((per + 15) / 16), a.splits);
   ragged_attn_group_kernel<DC, VC><<<grid, GA_WARPS * 32, smem, st>>>(a);
-  if (a.splits > 1) {
-    dim3 g2(n, a.a.heads);
-    ragged_attn_merge_kernel<__nv_bfloat16><<<g2, 64, 0, st>>>(a);
-  }
+  launch_merge<__nv_bfloat16>(a, n, st);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 template <int DC>
@@ -691,25 +829,27 @@ static int launch_group_v(const RowsArgs& a, int n, cudaStream_t st) {
   return launch_group<DC, 128>(a, n, st);
 }
 
-template <int DC, int VC>
+template <int DC, int VC, int MAPS>
 static int launch_tiles(const TilesArgs& a, int tiles, cudaStream_t st) {
-  const int smem = (2 * RAGGED_PAGE * (DC + 8) + 2 * RAGGED_PAGE * (VC + 8) + TA_ROWS * (DC + 8)) * 2;
+  const int ring = (2 * RAGGED_PAGE * (MAPS * DC + 8) + 2 * RAGGED_PAGE * (VC + 8) + TA_ROWS * (MAPS * DC + 8)) * 2;
+  const int other = MAPS == 2 ? TA_ROWS * (VC + 8) * 4 : 0;
+  const int smem = ring > other ? ring : other;
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(ragged_attn_tiles_kernel<DC, VC>,
+    if (cudaFuncSetAttribute(ragged_attn_tiles_kernel<DC, VC, MAPS>,
                              cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
       return -4;
     set = true;
   }
-  dim3 grid(tiles, a.a.heads);
-  ragged_attn_tiles_kernel<DC, VC><<<grid, TA_WARPS * 32, smem, st>>>(a);
+  dim3 grid(tiles, a.a.heads / MAPS);
+  ragged_attn_tiles_kernel<DC, VC, MAPS><<<grid, MAPS * TA_WARPS * 32, smem, st>>>(a);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
-template <int DC>
+template <int DC, int MAPS>
 static int launch_tiles_v(const TilesArgs& a, int tiles, cudaStream_t st) {
-  if (a.a.vdim <= 64) return launch_tiles<DC, 64>(a, tiles, st);
-  if (a.a.vdim <= 128) return launch_tiles<DC, 128>(a, tiles, st);
-  return launch_tiles<DC, 256>(a, tiles, st);
+  if (a.a.vdim <= 64) return launch_tiles<DC, 64, MAPS>(a, tiles, st);
+  if (a.a.vdim <= 128) return launch_tiles<DC, 128, MAPS>(a, tiles, st);
+  return launch_tiles<DC, 256, MAPS>(a, tiles, st);
 }
 
 template <typename T, int KIT>
@@ -725,17 +865,15 @@ static int launch_rows(const RowsArgs& a, int n, cudaStream_t st) {
   else if (per <= 4) CB_ROWS(4);
   else CB_ROWS(8);
 #undef CB_ROWS
-  if (a.splits > 1) {
-    dim3 g2(n, a.a.heads);
-    ragged_attn_merge_kernel<T><<<g2, 64, 0, st>>>(a);
-  }
+  launch_merge<T>(a, n, st);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 template <typename T>
 static int launch_rows_d(const RowsArgs& a, int n, cudaStream_t st) {
-  if (a.a.dim <= 64) return launch_rows<T, 1>(a, n, st);
-  if (a.a.dim <= 128) return launch_rows<T, 2>(a, n, st);
-  return launch_rows<T, 4>(a, n, st);
+  if (a.a.kdim <= 64) return launch_rows<T, 1>(a, n, st);
+  if (a.a.kdim <= 128) return launch_rows<T, 2>(a, n, st);
+  if (a.a.kdim <= 256) return launch_rows<T, 4>(a, n, st);
+  return launch_rows<T, 8>(a, n, st);
 }
 
 }  // namespace cb
@@ -743,57 +881,74 @@ static int launch_rows_d(const RowsArgs& a, int n, cudaStream_t st) {
 using namespace cb;
 
 static int fill_attn(RaggedAttn& p, const void* q, int q_head, const void* k_cache, const void* v_cache,
-                     const int* page_table, int max_pages, int num_pages, int heads, int kv_heads,
-                     int dim, int vdim, int dim_p, int vdim_p, int chunk, float scale,
-                     const float* sink, const void* gate, int ldg, void* out, int ldo, int* status) {
-  if (kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || dim > 256 || vdim > 256) return -1;
-  if (dim_p % 8 != 0 || vdim_p % 8 != 0 || dim_p < dim || vdim_p < vdim || dim_p > 256 || vdim_p > 256)
+                     const int* page_table, int max_pages, int num_pages, const RaggedSpec& c,
+                     const float* sink, const void* gate, int ldg, const float* map_weight, void* out,
+                     int ldo, int* status) {
+  if (c.kv_heads < 1 || c.heads % c.kv_heads != 0 || c.dim < 1 || c.vdim < 1 || c.dim > 256 || c.vdim > 256)
+    return -1;
+  if (c.dim_p % 8 != 0 || c.vdim_p % 8 != 0 || c.dim_p < c.dim || c.vdim_p < c.vdim || c.dim_p > 256 ||
+      c.vdim_p > 256)
+    return -2;
+  if (c.maps == 2 && sink != nullptr) return -2;
+  if ((c.maps != 1 && c.maps != 2) || (c.maps == 2 && map_weight == nullptr) || c.window < 0 || c.chunk < 0 ||
+      (c.window > 0 && c.chunk > 0) || c.softcap < 0.f)
     return -2;
   p.q = q; p.q_head = q_head; p.k_cache = k_cache; p.v_cache = v_cache; p.page_table = page_table;
-  p.max_pages = max_pages; p.num_pages = num_pages; p.heads = heads; p.kv_heads = kv_heads;
-  p.dim = dim; p.vdim = vdim; p.dim_p = dim_p; p.vdim_p = vdim_p; p.chunk = chunk; p.scale = scale;
-  p.sink = sink; p.gate = gate; p.ldg = ldg; p.out = out; p.ldo = ldo; p.status = status;
+  p.max_pages = max_pages; p.num_pages = num_pages; p.heads = c.heads * c.maps; p.kv_heads = c.kv_heads;
+  p.dim = c.dim; p.vdim = c.vdim; p.dim_p = c.dim_p; p.vdim_p = c.vdim_p; p.maps = c.maps;
+  p.kdim = c.maps * c.dim_p; p.chunk = c.chunk; p.window = c.window;
+  p.scale = c.softcap > 0.f ? c.scale / c.softcap : c.scale * LOG2E;
+  p.cap = c.softcap * LOG2E;
+  p.sink = sink; p.gate = gate; p.ldg = ldg; p.gate_wide = c.gate_wide; p.map_weight = map_weight;
+  p.map_factor = c.map_factor; p.eps = c.eps; p.out = out; p.ldo = ldo; p.status = status;
   return 0;
 }
 
 extern "C" int cb_ragged_attn_tile() { return TA_ROWS; }
 
 extern "C" int cb_ragged_attn_rows(const void* q, int q_head, const void* k_cache, const void* v_cache,
-                                   const int* page_table, int max_pages, int num_pages, int heads,
-                                   int kv_heads, int dim, int vdim, int dim_p, int vdim_p, int chunk,
-                                   float scale, const float* sink, const void* gate, int ldg,
-                                   void* out, int ldo, const int* rows, const int* row_slot,
-                                   const int* row_pos, int n, int splits, float* part_o,
-                                   float* part_ml, int f32, int* status, void* stream) {
+                                   const int* page_table, int max_pages, int num_pages,
+                                   const RaggedSpec* spec, const float* sink, const void* gate, int ldg,
+                                   const float* map_weight, void* out, int ldo, const int* rows,
+                                   const int* row_slot, const int* row_pos, int n, int splits,
+                                   float* part_o, float* part_ml, int f32, int* status, void* stream) {
   RowsArgs a;
-  const int rc = fill_attn(a.a, q, q_head, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
-                           dim, vdim, dim_p, vdim_p, chunk, scale, sink, gate, ldg, out, ldo, status);
+  const int rc = fill_attn(a.a, q, q_head, k_cache, v_cache, page_table, max_pages, num_pages, *spec, sink,
+                           gate, ldg, map_weight, out, ldo, status);
   if (rc != 0) return rc;
-  if (n <= 0 || splits < 1 || (splits > 1 && (part_o == nullptr || part_ml == nullptr))) return -5;
+  if (n <= 0 || splits < 1 || ((splits > 1 || spec->maps == 2) && (part_o == nullptr || part_ml == nullptr)))
+    return -5;
   a.rows = rows; a.row_slot = row_slot; a.row_pos = row_pos; a.splits = splits;
   a.part_o = part_o; a.part_ml = part_ml;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32) return launch_rows_d<float>(a, n, st);
-  if (dim > 128 || vdim > 128) return launch_rows<__nv_bfloat16, 4>(a, n, st);
-  return dim <= 64 ? launch_group_v<64>(a, n, st) : launch_group_v<128>(a, n, st);
+  if (a.a.kdim > 256) return launch_rows<__nv_bfloat16, 8>(a, n, st);
+  if (a.a.kdim > 128 || a.a.vdim > 128) return launch_rows<__nv_bfloat16, 4>(a, n, st);
+  return a.a.kdim <= 64 ? launch_group_v<64>(a, n, st) : launch_group_v<128>(a, n, st);
 }
 
 extern "C" int cb_ragged_attn_tiles(const void* q, int q_head, const void* k_cache, const void* v_cache,
-                                    const int* page_table, int max_pages, int num_pages, int heads,
-                                    int kv_heads, int dim, int vdim, int dim_p, int vdim_p, int chunk,
-                                    float scale, const float* sink, const void* gate, int ldg,
-                                    void* out, int ldo, const int* slot, const int* row0,
-                                    const int* len, const int* pos0, const int* tile_entry,
-                                    const int* tile_off, const int* tile_len, int tiles, int* status, void* stream) {
+                                    const int* page_table, int max_pages, int num_pages,
+                                    const RaggedSpec* spec, const float* sink, const void* gate, int ldg,
+                                    const float* map_weight, void* out, int ldo, const int* slot,
+                                    const int* row0, const int* len, const int* pos0,
+                                    const int* tile_entry, const int* tile_off, const int* tile_len,
+                                    int tiles, int* status, void* stream) {
   TilesArgs a;
-  const int rc = fill_attn(a.a, q, q_head, k_cache, v_cache, page_table, max_pages, num_pages, heads, kv_heads,
-                           dim, vdim, dim_p, vdim_p, chunk, scale, sink, gate, ldg, out, ldo, status);
+  const int rc = fill_attn(a.a, q, q_head, k_cache, v_cache, page_table, max_pages, num_pages, *spec, sink,
+                           gate, ldg, map_weight, out, ldo, status);
   if (rc != 0) return rc;
   if (tiles <= 0) return -5;
   a.e.slot = slot; a.e.row0 = row0; a.e.len = len; a.e.pos0 = pos0;
   a.tile_entry = tile_entry; a.tile_off = tile_off; a.tile_len = tile_len;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dim <= 64) return launch_tiles_v<64>(a, tiles, st);
-  if (dim <= 128) return launch_tiles_v<128>(a, tiles, st);
-  return launch_tiles_v<256>(a, tiles, st);
+  const int dim = a.a.dim;
+  if (spec->maps == 2) {
+    if (dim <= 64) return launch_tiles_v<64, 2>(a, tiles, st);
+    if (dim <= 128) return launch_tiles_v<128, 2>(a, tiles, st);
+    return -6;
+  }
+  if (dim <= 64) return launch_tiles_v<64, 1>(a, tiles, st);
+  if (dim <= 128) return launch_tiles_v<128, 1>(a, tiles, st);
+  return launch_tiles_v<256, 1>(a, tiles, st);
 }

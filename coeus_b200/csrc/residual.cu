@@ -4,7 +4,8 @@
 //   x = x + v                                     (written to another buffer than it is read from)
 //   h = x / rms(x) * gain                         (what the next sublayer reads, in T)
 //   h = h + (h_before - h) * shift                (token shift: h_before is the previous token's h)
-// Gains are one number or a vector.  x can also be written in T to one or two places (operands of a
+// y may also be, or get added, a sum of weighted rows of another buffer: the results of the experts a
+// token uses.  Gains are one number or a vector.  x can also be written in T to one or two places (operands of a
 // product over [x | x0]).
 //
 // Without a shift a block takes one row.  With it a block takes a tile of consecutive tokens of one
@@ -38,6 +39,10 @@ struct AddNorm {
   Entries e;
   const int* tile_entry;
   const int* tile_off;
+  const void* spread;      // rows in T, pitch lds, or null: y + sum_k weight[row, k] * spread[slot[row, k]]
+  int lds, top;
+  const int* spread_slot;  // [rows, top]
+  const float* spread_weight;
   int width;
   float eps;
 };
@@ -49,13 +54,30 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const AddNorm p) {
   // x of one row after the sublayer's result is added (f), and its normalised form (f again)
   auto stream = [&](int row, float (*f)[8], bool store) {
     float s = 0.f;
-    if (p.y != nullptr) {
+    const bool added = p.y != nullptr || p.spread != nullptr;
+    if (added) {
       const Y* yp = static_cast<const Y*>(p.y) + static_cast<size_t>(row) * p.ldy;
 #pragma unroll
       for (int i = 0; i < KEEP; ++i) {
         const int v = threadIdx.x + i * blockDim.x;
         if (v >= nv) continue;
-        load_vec<8>(yp + v * 8, f[i]);
+        if (p.y != nullptr) {
+          load_vec<8>(yp + v * 8, f[i]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[i][e] = 0.f;
+        }
+        if (p.spread != nullptr) {
+#pragma unroll 4
+          for (int k = 0; k < p.top; ++k) {
+            const size_t at = static_cast<size_t>(row) * p.top + k;
+            const float w = p.spread_weight[at];
+            float g[8];
+            load_vec<8>(static_cast<const T*>(p.spread) + static_cast<size_t>(p.spread_slot[at]) * p.lds + v * 8, g);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[i][e] += w * g[e];
+          }
+        }
         if (p.bias != nullptr) {
           float b[8];
           load_vec<8>(p.bias + v * 8, b);
@@ -76,7 +98,7 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const AddNorm p) {
         for (int e = 0; e < 8; ++e) xs[i][e] = 0.f;
     }
     float rs = 1.f;
-    if (p.y != nullptr && p.post != nullptr) {
+    if (added && p.post != nullptr) {
       s = block_sum(s, red);
       rs = 1.0f / sqrtf(s / p.width + p.eps);
       if (!p.post_vec) rs *= *p.post;
@@ -85,7 +107,7 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const AddNorm p) {
     for (int i = 0; i < KEEP; ++i) {
       const int v = threadIdx.x + i * blockDim.x;
       if (v >= nv) continue;
-      if (p.y == nullptr) {
+      if (!added) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) f[i][e] = xs[i][e];
       } else {
@@ -215,14 +237,18 @@ extern "C" int cb_add_norm(const float* x, const void* y, const float* bias, con
                            const float* shift, float* before, const int* rows, const int* slot,
                            const int* row0, const int* len, const int* pos0, const int* tile_entry,
                            const int* tile_off, int blocks, int width, float eps, int f32, int y_f32,
-                           void* stream) {
+                           const void* spread, int lds, const int* spread_slot,
+                           const float* spread_weight, int top, void* stream) {
   if (blocks <= 0 || ld % 8 || width > ld || ld > 16384) return -1;
   if (y != nullptr && (ldy % 8 || ldy < ld)) return -2;
   if (gain != nullptr && (h == nullptr || ldh % 8 || ldh < ld)) return -2;
   if ((cast0 != nullptr || cast1 != nullptr) && (ldc % 8 || ldc < ld)) return -2;
   if (shift != nullptr && (gain == nullptr || before == nullptr || rows != nullptr)) return -2;
   if (shift != nullptr && x != nullptr && x == x_out) return -2;     // the row in front is read late
+  if (spread != nullptr && (lds % 8 || lds < ld || top < 1 || spread_slot == nullptr || spread_weight == nullptr))
+    return -2;
   AddNorm p;
+  p.spread = spread; p.lds = lds; p.spread_slot = spread_slot; p.spread_weight = spread_weight; p.top = top;
   p.x = x; p.y = y; p.bias = bias; p.post = post; p.post_vec = post_vec; p.x_out = x_out;
   p.ld = ld; p.ldy = ldy; p.gain = gain; p.gain_vec = gain_vec; p.h = h; p.ldh = ldh;
   p.cast[0] = cast0; p.cast[1] = cast1; p.ldc = ldc; p.shift = shift; p.before = before;

@@ -748,10 +748,10 @@ static int launch_conv_act(const ConvAct& p, int tiles, cudaStream_t st) {
 
 // One block per row, vectors of eight bf16; the padding of a head is zero.  v may be absent.
 __global__ void kv_gather_kernel(const uint4* __restrict__ k_cache, const uint4* __restrict__ v_cache,
-                                 int kv_heads, int kw, int vw, const int* __restrict__ page_table,
+                                 int k_heads, int v_heads, int kw, int vw, const int* __restrict__ page_table,
                                  int max_pages, int num_pages, const int2* __restrict__ where,
-                                 uint4* __restrict__ k_rows, uint4* __restrict__ v_rows, int row_w,
-                                 int* status) {
+                                 uint4* __restrict__ k_rows, uint4* __restrict__ v_rows, int krow_w,
+                                 int vrow_w, int* status) {
   const int2 at = where[blockIdx.x];
   const int lp = at.y / RAGGED_PAGE;
   int page = lp < max_pages ? page_table[static_cast<size_t>(at.x) * max_pages + lp] : -1;
@@ -761,11 +761,16 @@ __global__ void kv_gather_kernel(const uint4* __restrict__ k_cache, const uint4*
   }
   const size_t cell = static_cast<size_t>(page) * RAGGED_PAGE + at.y % RAGGED_PAGE;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-  for (int i = threadIdx.x; i < kv_heads * row_w; i += blockDim.x) {
-    const int g = i / row_w, c = i % row_w;
-    const size_t dst = static_cast<size_t>(blockIdx.x) * kv_heads * row_w + i;
-    k_rows[dst] = c < kw ? k_cache[(cell * kv_heads + g) * kw + c] : zero;
-    if (v_rows != nullptr) v_rows[dst] = c < vw ? v_cache[(cell * kv_heads + g) * vw + c] : zero;
+  for (int i = threadIdx.x; i < k_heads * krow_w; i += blockDim.x) {
+    const int g = i / krow_w, c = i % krow_w;
+    k_rows[static_cast<size_t>(blockIdx.x) * k_heads * krow_w + i] =
+        c < kw ? k_cache[(cell * k_heads + g) * kw + c] : zero;
+  }
+  if (v_rows == nullptr) return;
+  for (int i = threadIdx.x; i < v_heads * vrow_w; i += blockDim.x) {
+    const int g = i / vrow_w, c = i % vrow_w;
+    v_rows[static_cast<size_t>(blockIdx.x) * v_heads * vrow_w + i] =
+        c < vw ? v_cache[(cell * v_heads + g) * vw + c] : zero;
   }
 }
 
@@ -876,17 +881,18 @@ extern "C" int cb_shortconv_attn(const void* raw, int ld, int koff, int voff, co
              : launch_conv_attn<__nv_bfloat16>(p, grid, vec, st);
 }
 
-// Rows gathered from the cache pages: row i of k_rows / v_rows ([n, kv_heads, row_head]) is the token
-// at position where[2 i + 1] of slot where[2 i].
-extern "C" int cb_kv_gather(const void* k_cache, const void* v_cache, int kv_heads, int dim_p,
+// Rows gathered from the cache pages: row i of k_rows [n, k_heads, kr_head] and v_rows [n, v_heads,
+// vr_head] is the token at position where[2 i + 1] of slot where[2 i].
+extern "C" int cb_kv_gather(const void* k_cache, const void* v_cache, int k_heads, int v_heads, int dim_p,
                             int vdim_p, const int* page_table, int max_pages, int num_pages,
-                            const void* where, int n, void* k_rows, void* v_rows, int row_head,
-                            int* status, void* stream) {
-  if (n <= 0 || dim_p % 8 || vdim_p % 8 || row_head % 8 || dim_p > row_head || vdim_p > row_head) return -1;
+                            const void* where, int n, void* k_rows, void* v_rows, int kr_head,
+                            int vr_head, int* status, void* stream) {
+  if (n <= 0 || dim_p % 8 || vdim_p % 8 || kr_head % 8 || vr_head % 8 || dim_p > kr_head || vdim_p > vr_head)
+    return -1;
   kv_gather_kernel<<<n, 128, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const uint4*>(k_cache), static_cast<const uint4*>(v_cache), kv_heads, dim_p / 8,
+      static_cast<const uint4*>(k_cache), static_cast<const uint4*>(v_cache), k_heads, v_heads, dim_p / 8,
       vdim_p / 8, page_table, max_pages, num_pages, static_cast<const int2*>(where),
-      static_cast<uint4*>(k_rows), static_cast<uint4*>(v_rows), row_head / 8, status);
+      static_cast<uint4*>(k_rows), static_cast<uint4*>(v_rows), kr_head / 8, vr_head / 8, status);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 

@@ -60,10 +60,11 @@ class HybridEngine(InferenceEngine):
         if isinstance(a, AttentionSpec):
             return R.AttnPlan(a.chunk, self._tiles and R.pieces_allowed(a.dim, a.vdim, a.chunk, a.scale))
         if isinstance(a, HeadAttentionSpec):
-            return R.AttnPlan(None, self._tiles and R.pieces_allowed(a.dim, a.vdim, None, a.scale), a.window,
-                              tiles=True)
+            plain = a.maps == 1 or (a.softcap is None and not a.gated)
+            return R.AttnPlan(None, self._tiles and plain and R.pieces_allowed(a.dim, a.vdim, None, a.scale),
+                              a.window, tiles=a.maps * a.dim <= 256)
         return R.AttnPlan(None, self._tiles and L.pieces_allowed(a.dim + a.rot_dim, a.vdim, a.scale),
-                          a.window or 1 << 30)
+                          a.window or 1 << 30, tiles=False)
 
     def _batch(self, entries: List[Entry], into: Optional[R.RaggedBatch] = None) -> R.RaggedBatch:
         return R.RaggedBatch(entries, self.m.device, tile_rows=self._tiles, into=into,

@@ -51,13 +51,12 @@ class AttnPlan:
 
     Under a sliding ``window`` a piece is a run of at most ``WINDOW_PIECE`` rows together with the
     keys its first row sees before it; an entry that continues a sequence gathers its own keys and
-    those of the window before it.  Where sizes do not allow pieces, ``tiles`` says whether long entries
-    go in tiles instead."""
+    those of the window before it.  Without ``tiles``, what is no piece goes row by row."""
 
     chunk: Optional[int]
     pieces: bool              # whether the layer's sizes allow the piece kernel
     window: Optional[int] = None
-    tiles: bool = False
+    tiles: bool = True
 
 
 SCAN_MIN = 16         # entries of more tokens than this take the chunked recurrence
@@ -231,7 +230,7 @@ class RaggedBatch:
                     where.append(np.stack([np.full_like(keys, entries[i].slot), keys], 1))
                     pieces.append((r0, head, self.T + extra, ahead))
                     extra += len(keys)
-                else:
+                elif plan.tiles:
                     tiles += [(i, o, min(ATTN_TILE, head - o)) for o in range(0, head, ATTN_TILE)]
                 pieces += [(r0 + o, m, r0 + o, 0) for o, m in ps]
             tiles.sort(key=lambda t: -(entries[t[0]].pos0 + t[1]))     # the most keys first
@@ -643,9 +642,12 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     common = (_p(q), q.shape[2], _p(k_cache), _p(v_cache), _p(page_table), page_table.shape[1],
               k_cache.shape[0], ctypes.byref(spec), _p(sink), _p(gate),
               gate.stride(0) if gate is not None else 0, _p(map_weight), _p(out), out.stride(0))
+    n, rows = batch.n_rows, batch.rows
     if batch.n_big:
         n_tiles, n_pieces, longest, extra, pieces, where, t_entry, t_off, t_len = batch.plan(
             plan or AttnPlan(chunk, k_rows is not None, window))
+        if not n_tiles and not n_pieces:       # sizes that neither kernel takes
+            n, rows = T, batch.every_row
         if n_tiles:
             rc = lib.cb_ragged_attn_tiles(*common, *batch.entry_args(), _p(t_entry), _p(t_off),
                                           _p(t_len), n_tiles, st, _lib.stream_ptr())
@@ -664,7 +666,6 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                 gate.stride(0) if gate is not None else 0, int(gate_wide), window or 0,
                 _F(softcap or 0.0), maps, _p(map_weight), _F(map_factor), _F(eps), st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_attn_fwd_pieces")
-    n = batch.n_rows
     if n:
         per = heads // kv_heads * maps
         ctas = n * kv_heads * ((per + 15) // 16)
@@ -676,7 +677,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         if splits > 1 or maps > 1:
             part_o = torch.empty((n, heads * maps, splits, vdim), dtype=torch.float32, device=q.device)
             part_ml = torch.empty((n, heads * maps, splits, 2), dtype=torch.float32, device=q.device)
-        rc = lib.cb_ragged_attn_rows(*common, _p(batch.rows), _p(batch.row_slot), _p(batch.pos), n,
+        rc = lib.cb_ragged_attn_rows(*common, _p(rows), _p(batch.row_slot), _p(batch.pos), n,
                                      splits, _p(part_o), _p(part_ml), int(q.dtype == torch.float32),
                                      st, _lib.stream_ptr())
         _lib.check_rc(rc, "cb_ragged_attn_rows", launches=2 if part_o is not None else 1)
