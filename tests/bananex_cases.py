@@ -9,8 +9,7 @@ from coeus_b200.models import hybrid as H
 from coeus_b200.ops import gemm as G
 from coeus_b200.ops import latent as LT
 from coeus_b200.ops import ragged as R
-from coeus_b200.ops.decode import PAGE
-from hybrid_checks import MODEL_CHECKS, agrees, rel, rnd, tokens  # noqa: F401
+from hybrid_checks import CUTS, MODEL_CHECKS, agrees, drive, rel, rnd, single_mixer, tokens  # noqa: F401
 
 A, S, U, M, L = H.LatentAttentionSpec, H.Mamba2Spec, H.MinGruSpec, H.MlpSpec, H.LayerSpec
 
@@ -163,38 +162,8 @@ def check_linear_heads(device, dtype, tol):
         assert float((y[rest].float() - 5.0).abs().max()) == 0
 
 
-def _mixer(spec, device, dtype, seed, scale=1.0):
-    """One layer of a single mixer with its engine, random projected inputs and their segments."""
-    cfg = H.HybridConfig(16, 16, (L(spec, None),), 1e-4, architecture="Bananex")
-    w = H.random_state(cfg, seed, dtype=torch.float32)
-    w = {n: t.bfloat16().float() for n, t in w.items()}
-    lm = H.HybridLM(cfg, w, device, dtype)
-    return lm, {n[7:]: t.double() for n, t in w.items() if n.startswith("l0.mix.")}
-
-
-CUTS = (((1, 40), (2, 1), (1, 1), (70, 2), (127, 1), (9, 165)), ((3, 130), (5, 6), (202, 74)))
-
-
-def _drive(lm, raws, cuts, run):
-    """Two sequences through ``run(engine, layer, raw, out, batch, rope)``, cut at several places, in slots
-    whose state holds something else; the mixer's outputs of each."""
-    eng = lm.make_engine(max_batch=3)
-    eng.open_slots(3, 512)
-    for t in eng.state.tensors.values():
-        t.fill_(9.0)
-    layer, outs, at = lm.layers[0], [[], []], [0, 0]
-    for s in (1, 2, 0, 2, 1):         # pages in an order that is not ascending
-        eng.cache.reserve(s, min(eng.cache.page_table.shape[1], len(eng.cache.owned.get(s, [])) + 3) * PAGE)
-    for cut in cuts:
-        b = eng._batch([R.Entry(slot, at[s], [0] * cut[s]) for s, slot in ((0, 2), (1, 0))])
-        raw = torch.cat([raws[s][at[s]:at[s] + cut[s]] for s in (0, 1)])
-        out = torch.full((b.T, layer.act_off), 5.0, dtype=lm.dtype, device=lm.device)
-        rope = {k: R.rope_table(b.pos, f) for k, f in lm.inv_freq.items()}
-        run(eng, layer, raw, out, b, rope)
-        outs[0].append(out[:cut[0]])
-        outs[1].append(out[cut[0]:])
-        at = [at[0] + cut[0], at[1] + cut[1]]
-    return [torch.cat(o)[:, :layer.out_dim] for o in outs], eng
+def _mixer(spec, device, dtype, seed):
+    return single_mixer(spec, "Bananex", device, dtype, seed)
 
 
 def check_latent_attention(device, dtype, tol):
@@ -231,7 +200,7 @@ def check_latent_attention(device, dtype, tol):
             raws.append(raw.to(dtype).to(device))
             wants.append(o.reshape(T, -1) * g)
         for cuts in CUTS[:1] if rank > 400 else CUTS + (((T, T),),):
-            got, _ = _drive(lm, raws, cuts, lambda e, layer, raw, out, b, rope: e._latent(
+            got, _ = drive(lm, raws, cuts, lambda e, layer, raw, out, b, rope: e._latent(
                 0, layer, raw, out, b, rope, b.max_ctx))
             for y, want in zip(got, wants):
                 err = (y.double().cpu() - want).abs().amax(1) / want.abs().max()
@@ -254,7 +223,7 @@ def check_mamba2(device, dtype, tol):
             for n, m in (("x", H_ * P), ("B", Gr * N), ("C", Gr * N)):     # segments are padded with zeros
                 raw[:, seg[n] + m:seg[n] + (m + 7) // 8 * 8] = 0
         for cuts in CUTS:
-            got, eng = _drive(lm, raws, cuts, lambda e, layer, raw, out, b, rope: e._mamba2(
+            got, eng = drive(lm, raws, cuts, lambda e, layer, raw, out, b, rope: e._mamba2(
                 0, layer, raw, out, b))
             for s, slot in ((0, 2), (1, 0)):
                 r = raws[s].cpu().double()
@@ -285,7 +254,7 @@ def check_mingru(device, dtype, tol):
             for n in ("z", "x", "g"):
                 raw[:, seg[n] + width:seg[n] + (width + 7) // 8 * 8] = 0
         for cuts in CUTS:
-            got, eng = _drive(lm, raws, cuts, lambda e, layer, raw, out, b, rope: e._mingru(
+            got, eng = drive(lm, raws, cuts, lambda e, layer, raw, out, b, rope: e._mingru(
                 0, layer, raw, out, b))
             for s, slot in ((0, 2), (1, 0)):
                 z, u, g = (raws[s][:, seg[n]:seg[n] + width].cpu().double() for n in ("z", "x", "g"))

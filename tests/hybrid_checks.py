@@ -190,3 +190,38 @@ def check_batcher(b):
 
 MODEL_CHECKS = [check_whole_prompt, check_token_by_token, check_portions, check_mixed_batches,
                 check_reuse, check_long_decode, check_generate, check_batcher]
+
+
+# ----------------------------------------------------------------------- one mixer on its own
+CUTS = (((1, 40), (2, 1), (1, 1), (70, 2), (127, 1), (9, 165)), ((3, 130), (5, 6), (202, 74)))
+
+
+def single_mixer(spec, architecture, device, dtype, seed):
+    """A model of one layer with this mixer alone, and the mixer's weights."""
+    cfg = H.HybridConfig(16, 16, (H.LayerSpec(spec, None),), 1e-4, architecture=architecture)
+    w = H.random_state(cfg, seed, dtype=torch.float32)
+    w = {n: t.bfloat16().float() for n, t in w.items()}
+    lm = H.HybridLM(cfg, w, device, dtype)
+    return lm, {n[7:]: t.double() for n, t in w.items() if n.startswith("l0.mix.")}
+
+
+def drive(lm, raws, cuts, run):
+    """Two sequences through ``run(engine, layer, raw, out, batch, rope)``, cut at several places, in slots
+    whose state holds something else; the mixer's outputs of each."""
+    eng = lm.make_engine(max_batch=3)
+    eng.open_slots(3, 512)
+    for t in eng.state.tensors.values():
+        t.fill_(9.0)
+    layer, outs, at = lm.layers[0], [[], []], [0, 0]
+    for s in (1, 2, 0, 2, 1):         # pages in an order that is not ascending
+        eng.cache.reserve(s, min(eng.cache.page_table.shape[1], len(eng.cache.owned.get(s, [])) + 3) * PAGE)
+    for cut in cuts:
+        b = eng._batch([R.Entry(slot, at[s], [0] * cut[s]) for s, slot in ((0, 2), (1, 0))])
+        raw = torch.cat([raws[s][at[s]:at[s] + cut[s]] for s in (0, 1)])
+        out = torch.full((b.T, layer.act_off), 5.0, dtype=lm.dtype, device=lm.device)
+        rope = {k: R.rope_table(b.pos, f) for k, f in lm.inv_freq.items()}
+        run(eng, layer, raw, out, b, rope)
+        outs[0].append(out[:cut[0]])
+        outs[1].append(out[cut[0]:])
+        at = [at[0] + cut[0], at[1] + cut[1]]
+    return [torch.cat(o)[:, :layer.out_dim] for o in outs], eng

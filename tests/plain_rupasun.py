@@ -5,6 +5,7 @@ the framework with it; it shares no code with the framework.
 Notation: ``x [T, width]`` is one sequence's residual stream, ``w`` a mapping from tensor name to
 tensor (linear weights ``[out, in]``), ``cfg`` the configuration as a plain dictionary.
 """
+import functools
 import math
 
 import torch
@@ -20,11 +21,8 @@ def rms_norm(x, gain, eps):
 
 
 def _angles(T, dims, base):
-    a = torch.empty(T, dims // 2, dtype=torch.float64)
-    for t in range(T):
-        for i in range(dims // 2):
-            a[t, i] = t * base ** (-2.0 * i / dims)
-    return a[:, None]
+    f = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
+    return torch.arange(T, dtype=torch.float64)[:, None, None] * f
 
 
 def rotate_halves(x, dims, base):
@@ -53,6 +51,7 @@ def visible(i, j, size=None):
     return j <= i and (size is None or i - j < size)
 
 
+@functools.lru_cache(maxsize=None)
 def visibility(T, size=None):
     return torch.tensor([[visible(i, j, size) for j in range(T)] for i in range(T)])
 
@@ -150,7 +149,7 @@ def experts(h, w, p, m):
     for t in range(h.shape[0]):
         for e, c in zip(*choose(z[t], r["top"], r["groups"]["count"], r["groups"]["keep"], r["scale"])):
             out[t] += c * expert(h[t], w, f"{p}e{e}.", m["expert"]["limit"])
-    return out + expert(h, w, p + "shared.", m["shared"]["limit"])
+    return out + expert(h, w, p + "shared.", m["shared"]["limit"]) if m.get("shared") else out
 
 
 MIXERS = {"attention": diff_attention, "attention_2": capped_attention}
