@@ -1,10 +1,11 @@
 """Serving throughput of a design of mixed layers beside the framework's closest model at equal size,
-and its kernels one by one against the roofline (``python bench.py --serving sapasun|bananex
-[--kernels]``; the kernels of Bananex are in :mod:`coeus_b200.utils.bananex_bench`).
+and its kernels one by one against the roofline (``python bench.py --serving sapasun|bananex|rupasun
+[--kernels]``; the kernels of Bananex are in :mod:`coeus_b200.utils.bananex_bench`, those of Rupasun in
+:mod:`coeus_b200.utils.rupasun_bench`).
 
 The closest model is the RMSNorm / SwiGLU / rotary decoder with grouped-query attention: same
 width, depth, heads and vocabulary, the feed-forward as wide as gives the same parameters per
-layer (three matrices of 8/3 width against two of 4 width).  Weights are random.  Times are CUDA
+layer (three matrices of 8/3 width against two of 4 width; for a mixture of experts: per token).  Weights are random.  Times are CUDA
 events around whole engine calls (prompt batches, decode steps), after warm-up; every call streams
 weights and caches far above the L2 cache.  The kernel table flushes L2 between launches.
 """
@@ -244,12 +245,21 @@ def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> Li
     return rows
 
 
+DESIGNS = ("sapasun", "bananex", "rupasun")
+
+
+def bench_of(design: str):
+    """``(config, kernel_table)`` of a design."""
+    from . import bananex_bench, rupasun_bench
+    return {"sapasun": (sapasun_config, kernel_table),
+            "bananex": (bananex_bench.config, bananex_bench.kernel_table),
+            "rupasun": (rupasun_bench.config, rupasun_bench.kernel_table)}[design]
+
+
 def run(design: str, steps: int = 20, warmup: int = 3, kernels: bool = False, sampler=None) -> None:
     """One JSON line per size and model, then (``kernels``) one per kernel."""
     from ..ops import _lib
-    from . import bananex_bench
-    config, table = {"sapasun": (sapasun_config, kernel_table),
-                     "bananex": (bananex_bench.config, bananex_bench.kernel_table)}[design]
+    config, table = bench_of(design)
     for name, size in SIZES.items():
         for which in (design, "closest"):
             if which == design:
@@ -287,14 +297,12 @@ def main(argv=None) -> int:
     rows whose ``name, phase`` contains the text (with ``--iters 1`` a small case for a profiler)."""
     import argparse
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default="sapasun", choices=["sapasun", "bananex"])
+    ap.add_argument("--design", default="sapasun", choices=DESIGNS)
     ap.add_argument("--size", default="1b-layers", choices=list(SIZES))
     ap.add_argument("--kernel", default="")
     ap.add_argument("--iters", type=int, default=10)
     a = ap.parse_args(argv)
-    from . import bananex_bench
-    table = kernel_table if a.design == "sapasun" else bananex_bench.kernel_table
-    for row in table(a.size, a.kernel, a.iters):
+    for row in bench_of(a.design)[1](a.size, a.kernel, a.iters):
         print(json.dumps(row), flush=True)
     return 0
 
