@@ -21,8 +21,9 @@
 // on the FMA pipe, because the exponential unit (16 results per clock per SM) bounds dh = 64.
 // Grouped-query attention: query head h reads K/V head h / (nh / nkv).
 //
-// Two variants serve prompts of unequal length (PIECES) only.  CAP: scores s become cap * tanh(s / cap).
-// DIFF: a head has two maps, each with queries and keys of its own over the same values; an item is ONE
+// Two variants serve prompts of unequal length (PIECES) only.  CAP: scores s become cap * tanh(s / cap),
+// from the exponential unit (1) or, where the argument is known not to leave [-1, 1], as a polynomial on
+// the FMA pipe (2).  DIFF: a head has two maps, each with queries and keys of its own over the same values; an item is ONE
 // query tile of a head, tiles A and B of the step are its two maps, every step has its own key tile and
 // every pair of steps its value tile.  At the end each warpgroup takes half of the columns of
 // o = a0 - w a1, and the two meet at two barriers: one when both results are complete, one for the sum of
@@ -65,6 +66,7 @@ struct AttnFwdArgs {
   int gate_wide;
   int window;                  // 0: no window
   float cap_log2, cap_in;      // CAP: the cap in units of log2, and what takes a product to the tanh
+  float cap_poly[7];           // CAP 2: score / product as a polynomial in the product's square
   const float* map_weight;     // DIFF: weight of the second map, factor and eps of the norm
   float map_factor, map_eps;
 };
@@ -203,7 +205,7 @@ struct AFWalk {
   __device__ bool last_of_tile() const { return j == (t ? n1 : n0) - 1; }
 };
 
-template <int DQ, int DV, bool POLY, bool DROP, bool PIECES, bool CAP, bool DIFF>
+template <int DQ, int DV, bool POLY, bool DROP, bool PIECES, int CAP, bool DIFF>
 __global__ void __launch_bounds__(AF_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const AttnFwdArgs p) {
@@ -552,7 +554,19 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       for (int c = 0; c < BKV / 32; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v + c * 32);
       tmem_ld_wait();
       if (tr) tr[tri + 1] = clock64();
-      if constexpr (CAP) {
+      if constexpr (CAP == 2) {
+#pragma unroll
+        for (int e = 0; e < BKV; e += 2) {
+          const float a = __uint_as_float(v[e]), b = __uint_as_float(v[e + 1]);
+          float wa, wb, ra = p.cap_poly[6], rb = ra;
+          fma2(wa, wb, a, b, a, b, 0.f, 0.f);
+#pragma unroll
+          for (int i = 5; i >= 0; --i) fma2(ra, rb, ra, rb, wa, wb, p.cap_poly[i], p.cap_poly[i]);
+          fma2(ra, rb, ra, rb, a, b, 0.f, 0.f);
+          v[e] = __float_as_uint(ra);
+          v[e + 1] = __float_as_uint(rb);
+        }
+      } else if constexpr (CAP == 1) {
 #pragma unroll
         for (int e = 0; e < BKV; ++e)
           v[e] = __float_as_uint(p.cap_log2 * tanh_exp(__uint_as_float(v[e]) * p.cap_in));
@@ -811,7 +825,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
-template <int DQ, int DV, bool POLY, bool DROP = false, bool PIECES = false, bool CAP = false, bool DIFF = false>
+template <int DQ, int DV, bool POLY, bool DROP = false, bool PIECES = false, int CAP = 0, bool DIFF = false>
 static int launch_attn_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
                               const AttnFwdArgs& a, int max_ctas, cudaStream_t st) {
   using Cfg = AFCfg<DQ, DV, DIFF>;
@@ -903,13 +917,14 @@ extern "C" int cb_attn_fwd(const void* q, const void* k, const void* v, void* o,
 // per head that enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view, or with
 // gate_wide column h * vdim + d) multiplies head h's output by its sigmoid; both may be null.  A
 // query sees the last `window` of its keys (0: all).  scale > 0.  Scores are capped by softcap (0: not).
+// score_max bounds |q . k| * scale where the caller knows it (0: not known).
 // With two maps q and k have two heads per head (map 0 first), and the output is the weighted difference
 // divided by its root mean square, times map_factor; it has neither sink, gate nor cap.
 extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, void* o, int rows,
                                   int kv_rows, const void* pieces, int n_pieces, int max_len, int nh,
                                   int nkv, int dq, int dv, int vdim, int ldq, int ldk, int ldv, int ldo,
                                   float scale, const float* sink, const void* gate, int ldg,
-                                  int gate_wide, int window, float softcap, int maps,
+                                  int gate_wide, int window, float softcap, float score_max, int maps,
                                   const float* map_weight, float map_factor, float map_eps, int* status,
                                   void* stream) {
   using namespace cb;
@@ -946,15 +961,25 @@ extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, v
   a.map_eps = map_eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (maps == 2) {
-    if (dv == 64) return launch_attn_fwd<64, 64, false, false, true, false, true>(tq, tk, tv, a, 0, st);
-    return dq == 64 ? launch_attn_fwd<64, 128, false, false, true, false, true>(tq, tk, tv, a, 0, st)
-                    : launch_attn_fwd<128, 128, false, false, true, false, true>(tq, tk, tv, a, 0, st);
+    if (dv == 64) return launch_attn_fwd<64, 64, false, false, true, 0, true>(tq, tk, tv, a, 0, st);
+    return dq == 64 ? launch_attn_fwd<64, 128, false, false, true, 0, true>(tq, tk, tv, a, 0, st)
+                    : launch_attn_fwd<128, 128, false, false, true, 0, true>(tq, tk, tv, a, 0, st);
   }
   if (softcap > 0.f) {
     a.cap_log2 = softcap * 1.4426950408889634f;
     a.cap_in = scale / softcap;
-    return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, true>(tq, tk, tv, a, 0, st)
-                    : launch_attn_fwd<128, 128, false, false, true, true>(tq, tk, tv, a, 0, st);
+    if (score_max > 0.f && score_max <= softcap) {
+      // tanh(x) / x on [0, 1] as a polynomial in x^2: interpolated at Chebyshev nodes, |error| of tanh < 1e-7
+      const double t[7] = {0.99999994, -0.33332828, 0.13325076, -0.05345165, 0.02027971, -0.0061943247,
+                           0.0010380251};
+      double f = static_cast<double>(a.cap_log2) * a.cap_in;
+      for (int i = 0; i < 7; ++i, f *= static_cast<double>(a.cap_in) * a.cap_in)
+        a.cap_poly[i] = static_cast<float>(t[i] * f);
+      return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, 2>(tq, tk, tv, a, 0, st)
+                      : launch_attn_fwd<128, 128, false, false, true, 2>(tq, tk, tv, a, 0, st);
+    }
+    return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, 1>(tq, tk, tv, a, 0, st)
+                    : launch_attn_fwd<128, 128, false, false, true, 1>(tq, tk, tv, a, 0, st);
   }
   return dv == 64 ? launch_attn_fwd<64, 64, false, false, true>(tq, tk, tv, a, 0, st)
                   : launch_attn_fwd<128, 128, false, false, true>(tq, tk, tv, a, 0, st);

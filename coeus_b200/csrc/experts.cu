@@ -4,7 +4,7 @@
 //                computes the router's product as well.  More: the logits are given, a block takes
 //                CHOOSE_TOKENS tokens and counts its pairs per expert.
 //   moe_place    one block: where every block's pairs of an expert go in a buffer sorted by expert, whose
-//                experts start at multiples of MOE_BLOCK rows, and the expert of every MOE_BLOCK rows
+//                experts start at multiples of a block of rows, and the expert of every block
 //   moe_gather   rows into that buffer
 //   moe_few_in / moe_few_down   up to 16 rows: the weights of the chosen experts and of the shared one are
 //                streamed straight into mma fragments.  The activations of all live experts lie side by
@@ -17,7 +17,6 @@ namespace cb {
 constexpr int CHOOSE_TOKENS = 32;
 constexpr int CHOOSE_WARPS = 8;
 constexpr int MOE_E = 256, MOE_K = 16;
-constexpr int MOE_BLOCK = 128;
 constexpr unsigned FULL = 0xffffffffu;
 
 struct Choose {
@@ -167,8 +166,8 @@ __global__ void __launch_bounds__(512) moe_choose_few_kernel(const Choose p) {
 
 __global__ void __launch_bounds__(1024)
 moe_place_kernel(const int* __restrict__ counts, int blocks, int E, int* __restrict__ base,
-                 int* __restrict__ block_expert, int n_tiles) {
-  __shared__ int total[MOE_E], start[MOE_E + 1];        // start: in tiles of MOE_BLOCK rows
+                 int* __restrict__ block_expert, int n_tiles, int tile_rows) {
+  __shared__ int total[MOE_E], start[MOE_E + 1];        // start: in tiles
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int e = warp; e < E; e += 32) {
     int n = 0;
@@ -181,7 +180,7 @@ moe_place_kernel(const int* __restrict__ counts, int blocks, int E, int* __restr
   if (warp == 0) {
     int run = 0;
     for (int e0 = 0; e0 < E; e0 += 32) {
-      const int n = e0 + lane < E ? (total[e0 + lane] + MOE_BLOCK - 1) / MOE_BLOCK : 0;
+      const int n = e0 + lane < E ? (total[e0 + lane] + tile_rows - 1) / tile_rows : 0;
       int incl = n;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
@@ -198,7 +197,7 @@ moe_place_kernel(const int* __restrict__ counts, int blocks, int E, int* __restr
   for (int e = warp; e < E; e += 32) {
     for (int i = start[e] + lane; i < start[e + 1]; i += 32)
       if (i < n_tiles) block_expert[i] = e;
-    int run = start[e] * MOE_BLOCK;
+    int run = start[e] * tile_rows;
     for (int b0 = 0; b0 < blocks; b0 += 32) {
       const int b = b0 + lane;
       const int n = b < blocks ? counts[static_cast<size_t>(b) * E + e] : 0;
@@ -479,22 +478,22 @@ extern "C" int cb_moe_choose(const float* logits, int ldl, const void* h, int ld
   return CB_RC();
 }
 
-// rows [n_tiles * 128, W]; base has the shape of counts [blocks, E].
+// rows [n_tiles * tile_rows, W]; base has the shape of counts [blocks, E].
 extern "C" int cb_moe_sort(const void* h, int ldh, const int* expert, const int* rank, const int* counts,
                            int T, int E, int top, int per_block, int blocks, int* base, int* slot,
-                           int* block_expert, int n_tiles, void* rows, int W, int f32, int* status,
+                           int* block_expert, int n_tiles, int tile_rows, void* rows, int W, int f32, int* status,
                            void* stream) {
   const int v = f32 ? 4 : 8;
   if (T <= 0 || E < 1 || E > MOE_E || top < 1 || top > MOE_K || W % v || ldh % v || per_block < 1) return -1;
-  if (blocks != (T + per_block - 1) / per_block) return -1;
-  if (static_cast<long long>(n_tiles) < static_cast<long long>(T) * top / MOE_BLOCK + (T * top < E ? T * top : E))
+  if (blocks != (T + per_block - 1) / per_block || tile_rows < 1) return -1;
+  if (static_cast<long long>(n_tiles) < static_cast<long long>(T) * top / tile_rows + (T * top < E ? T * top : E))
     return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  moe_place_kernel<<<1, 1024, 0, st>>>(counts, blocks, E, base, block_expert, n_tiles);
+  moe_place_kernel<<<1, 1024, 0, st>>>(counts, blocks, E, base, block_expert, n_tiles, tile_rows);
   const int nv = W / v, threads = nv >= 256 ? 256 : (nv + 31) / 32 * 32;
   moe_gather_kernel<<<T, threads, 0, st>>>(static_cast<const uint4*>(h), ldh / v, expert, rank, base, E, top,
                                            per_block, slot, static_cast<uint4*>(rows), nv,
-                                           n_tiles * MOE_BLOCK, status);
+                                           n_tiles * tile_rows, status);
   return CB_RC();
 }
 

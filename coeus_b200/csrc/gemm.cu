@@ -12,7 +12,7 @@
 //   dgrad    dX[M,K] = dY[M,N]  . W[K,N]^T    A K-major,  B K-major
 //   wgrad    dW[K,N] = X[M,K]^T . dY[M,N]     A MN-major, B MN-major (split along tokens,
 //                                             fp32 atomic accumulation)
-// Blocks of 128 rows of A may each have a weight of their own (experts whose rows are sorted).
+// Blocks of rows of A (one tile high) may each have a weight of their own (experts whose rows are sorted).
 // Fused epilogues: alpha scale, +bias[N], GELU(tanh) with the pre-activation kept, dGELU, squared
 // ReLU, GELU(erf), +residual, bounded gated unit over alternating columns, bf16 / fp32 /
 // fp32-atomic-add output.
@@ -59,7 +59,7 @@ struct GemmArgs {
   int group_m;                  // output rows per group; 0 = one group.  Group g of a tile adds
   int g_am, g_ak;               // g * g_am to A's m coordinate, g * g_ak to its k coordinate,
   int g_bn, g_bk;               // g * g_bn to B's n coordinate, g * g_bk to its k coordinate
-  const int* block_group;       // group of every GEMM_BM rows instead (-1: none from here on), or null
+  const int* block_group;       // group of every tile of rows instead (-1: none from here on), or null
   float glu_slope, glu_limit;   // EPI_GLU: columns alternate g, u; the output has half as many
   // ---- fused collectives over peer memory (COMM template parameter)
   int tp, rank;                 // ranks of the tensor-parallel group, this rank
@@ -307,7 +307,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 
   // Group of an m-block; negative: no work from here on.
   auto group_of = [&](int m_blk) {
-    if constexpr (COMM == COMM_NONE && !CTA2)
+    if constexpr (COMM == COMM_NONE)
       if (p.block_group != nullptr) return p.block_group[m_blk];
     return p.group_m > 0 ? (m_blk * TILE_M) / p.group_m : 0;
   };
@@ -1070,19 +1070,21 @@ extern "C" int cb_gemm_bf16_grouped(const void* A, const void* B, void* D, int g
                         stream, groups);
 }
 
-// D[rows of block b] = epilogue(A[rows of block b] . B[block_expert[b]]^T), blocks of 128 rows: A [M, K],
+// D[rows of block b] = epilogue(A[rows of block b] . B[block_expert[b]]^T), blocks of 128 or 256 rows: A [M, K],
 // B [experts, N, K] (pitch ldb), D [M, N] or with glu (a bounded gated unit over alternating columns)
 // [M, N / 2], all bf16.  A negative entry says that this block and all behind it have no work; their
 // rows of D are left alone.  block_expert null: one weight, any M.
 extern "C" int cb_gemm_bf16_blocks(const void* A, const void* B, void* D, int M, int N, int K, int experts,
-                                   int lda, int ldb, int ldd, const int* block_expert, int glu,
-                                   float slope, float limit, int* status, void* stream) {
+                                   int lda, int ldb, int ldd, const int* block_expert, int block_rows,
+                                   int glu, float slope, float limit, int* status, void* stream) {
   using namespace cb;
   const int cols = glu ? N / 2 : N;
   if (M <= 0 || N <= 0 || K <= 0 || experts < 1 || N % 8 || cols % 8 || K % 8 || ldd % 8) return -21;
-  if (block_expert != nullptr && M % GEMM_BM) return -24;
+  if (block_rows != GEMM_BM && block_rows != 2 * GEMM_BM) return -24;
+  if (block_expert != nullptr && M % block_rows) return -24;
   if (reinterpret_cast<uintptr_t>(D) & 15u) return -21;
-  const bool pairs = block_expert == nullptr && M >= 256 && N > 128;
+  // CTA pairs work on 256 rows at a time, which have to be of one expert
+  const bool pairs = block_expert == nullptr ? M >= 256 && N > 128 : block_rows == 2 * GEMM_BM;
   const long long wide = static_cast<long long>((M + GEMM_BM - 1) / GEMM_BM) * ((N + 255) / 256);
   const int bn = pairs || (N > 128 && wide >= 4 * sm_count()) ? 256 : 128;
   CUtensorMap ta, tb, td;

@@ -3,7 +3,8 @@
 // by their root mean square, and the write of k and v into the cache pages and, for the kernel that
 // works on pieces of prompts, row by row.
 //
-// One block per row; a group of L lanes takes one head, eight consecutive numbers per lane.
+// One block per row; a group of L lanes takes one head of q or k, eight consecutive numbers per lane, or
+// as many of a head of v.
 #include "ragged.cuh"
 
 namespace cb {
@@ -52,7 +53,7 @@ __device__ __forceinline__ void head_load(const T* src, int d, int n, float* f) 
 // VEC: head sizes (and, for pairs half a rotation apart, half) are multiples of eight.
 template <typename T, int L, bool VEC>
 __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p) {
-  const int row = blockIdx.x, d = (threadIdx.x % L) * 8;
+  const int row = blockIdx.x, d0 = (threadIdx.x % L) * 8;
   const int pos = p.row_pos[row], lp = pos / RAGGED_PAGE;
   int page = lp < p.max_pages ? p.page_table[static_cast<size_t>(p.row_slot[row]) * p.max_pages + lp] : -1;
   if (page < 0 || page >= p.num_pages) {
@@ -62,12 +63,15 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
   const size_t cell = static_cast<size_t>(page) * RAGGED_PAGE + pos % RAGGED_PAGE;
   const T* raw = static_cast<const T*>(p.raw) + static_cast<size_t>(row) * p.ld;
   const float2* rope = p.rope + static_cast<size_t>(row) * p.half;
-  const int units = p.heads + p.kv_heads + p.v_heads;
+  const int v_units = (max(p.vdim_p, p.vr_head) + 8 * L - 1) / (8 * L);     // per head
+  const int units = p.heads + p.kv_heads + p.v_heads * v_units;
   for (int u = threadIdx.x / L; u < (units + HP_THREADS / L - 1) / (HP_THREADS / L) * (HP_THREADS / L);
        u += HP_THREADS / L) {                     // whole groups: the lanes of a warp stay together
     const bool live = u < units, is_q = u < p.heads, is_v = u >= p.heads + p.kv_heads;
     const int n = is_v ? p.vdim : p.dim;
-    const int h = is_q ? u : (is_v ? u - p.heads - p.kv_heads : u - p.heads);
+    const int uv = u - p.heads - p.kv_heads;
+    const int h = is_q ? u : (is_v ? uv / v_units : u - p.heads);
+    const int d = is_v ? d0 + uv % v_units * 8 * L : d0;
     const T* src = raw + (is_q ? 0 : (is_v ? p.voff : p.koff)) + static_cast<size_t>(h) * n;
     float f[8];
 #pragma unroll
@@ -86,13 +90,13 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
         }
       } else if constexpr (VEC) {                 // the other numbers lie half further or half before
         const bool low = d < p.half;
-        const int d0 = low ? d : d - p.half;
+        const int first = low ? d : d - p.half;
         float o[8];
-        load_vec<8>(src + (low ? d + p.half : d0), o);
+        load_vec<8>(src + (low ? d + p.half : first), o);
         const float sign = low ? -1.f : 1.f;
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-          const float2 cs = rope[d0 + i];
+          const float2 cs = rope[first + i];
           f[i] = f[i] * cs.x + sign * o[i] * cs.y;
         }
       } else {
@@ -168,8 +172,8 @@ extern "C" int cb_head_prep(const void* raw, int ld, int koff, int voff, int hea
   if (k_rows != nullptr && (v_rows == nullptr || kr_head % 8 || vr_head % 8 || kr_head < dim || vr_head < vdim))
     return -2;
   int widest = q_head;
-  for (int w : {dim_p, vdim_p, kr_head, vr_head}) widest = w > widest ? w : widest;
-  if (widest > 256) return -2;
+  for (int w : {dim_p, kr_head}) widest = w > widest ? w : widest;
+  if (widest > 256 || vdim_p > 256 || vr_head > 256) return -2;
   HeadPrep p;
   p.raw = raw; p.ld = ld; p.koff = koff; p.voff = voff; p.heads = heads; p.kv_heads = kv_heads;
   p.v_heads = v_heads; p.dim = dim; p.vdim = vdim; p.half = half; p.rope = static_cast<const float2*>(rope);

@@ -1,23 +1,22 @@
 // fp32 linear layer Y[M, N] = act(X[M, K] . W[N, K]^T + bias[N]) on the FMA units, for serving a model in
 // full 32-bit precision: 64 x 64 tiles, 4 x 4 outputs per thread, operands staged in shared memory.
-// Grouped: the rows of x come in blocks of 128 of which each has a weight of its own (experts).
+// Grouped: the rows of x come in blocks of which each has a weight of its own (experts).
 #include "ragged.cuh"
 
 namespace cb {
 
 constexpr int LT = 64, LK = 16;
 enum : int { ACT_NONE = 0, ACT_RELU2 = 4, ACT_SOFTCAP = 5, ACT_GELU_ERF = 6, ACT_GLU = 7 };
-constexpr int GROUP_ROWS = 128;
 
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw,
                   const float* __restrict__ bias, float* __restrict__ y, int ldy, int M, int N,
                   int K, int act, float act_arg, float limit, int accumulate,
-                  const int* __restrict__ block_expert) {
+                  const int* __restrict__ block_expert, int block_rows) {
   __shared__ float sx[LK][LT + 4], sw[LK][LT + 4];
   const int m0 = blockIdx.y * LT, n0 = blockIdx.x * LT;
   if (block_expert != nullptr) {
-    const int e = block_expert[m0 / GROUP_ROWS];
+    const int e = block_expert[m0 / block_rows];
     if (e < 0) return;
     w += static_cast<size_t>(e) * N * ldw;
   }
@@ -88,20 +87,21 @@ extern "C" int cb_linear_f32(const float* x, int ldx, const float* w, int ldw,
   dim3 grid((N + cb::LT - 1) / cb::LT, (M + cb::LT - 1) / cb::LT);
   if (grid.y > 65535) return -1;
   cb::linear_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      x, ldx, w, ldw, bias, y, ldy, M, N, K, act, act_arg, 0.f, accumulate, nullptr);
+      x, ldx, w, ldw, bias, y, ldy, M, N, K, act, act_arg, 0.f, accumulate, nullptr, 0);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-// block_expert[b]: which of the weights [experts, N, K] the rows 128 b .. 128 b + 127 take (-1: none, they
-// are left alone); null: one weight.  glu: alternating columns g, u make one (clamped_glu).
+// block_expert[b]: which of the weights [experts, N, K] block b of block_rows (a multiple of 64) rows takes
+// (-1: none, they are left alone); null: one weight.  glu: alternating columns g, u make one (clamped_glu).
 extern "C" int cb_linear_f32_grouped(const float* x, int ldx, const float* w, int ldw,
-                                     const int* block_expert, float* y, int ldy, int M, int N, int K,
+                                     const int* block_expert, int block_rows, float* y, int ldy, int M, int N, int K,
                                      int glu, float slope, float limit, void* stream) {
   if (M <= 0 || N <= 0 || K <= 0 || K % 4 || ldx % 4 || ldw % 4 || (glu && N % 2)) return -1;
-  if (block_expert != nullptr && M % cb::GROUP_ROWS) return -1;
+  if (block_expert != nullptr && (block_rows < cb::LT || block_rows % cb::LT || M % block_rows)) return -1;
   dim3 grid((N + cb::LT - 1) / cb::LT, (M + cb::LT - 1) / cb::LT);
   if (grid.y > 65535) return -1;
   cb::linear_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      x, ldx, w, ldw, nullptr, y, ldy, M, N, K, glu ? cb::ACT_GLU : cb::ACT_NONE, slope, limit, 0, block_expert);
+      x, ldx, w, ldw, nullptr, y, ldy, M, N, K, glu ? cb::ACT_GLU : cb::ACT_NONE, slope, limit, 0, block_expert,
+      block_rows);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

@@ -181,7 +181,7 @@ class HybridEngine(InferenceEngine):
                         unit_eps=eps if s.unit_qk else None, q_head=q_head, k_rows=k_rows, v_rows=v_rows)
         R.ragged_attention(
             q, c.k[i], c.v[i], c.page_table, b, s.heads, s.kv_heads, s.dim, s.vdim, s.scale,
-            out[:, :layer.out_dim], window=s.window, softcap=s.softcap, maps=s.maps,
+            out[:, :layer.out_dim], window=s.window, softcap=s.softcap, score_max=s.score_max, maps=s.maps,
             map_weight=layer.map_weight, map_factor=1.0 - s.diff if s.maps == 2 else 1.0, eps=eps,
             gate=raw[:, layer.seg["g"]:] if s.gated else None, gate_wide=True, max_ctx=max_ctx,
             k_rows=k_rows, v_rows=v_rows, plan=plan)

@@ -376,6 +376,11 @@ class HeadAttentionSpec:
         return out
 
     @property
+    def score_max(self) -> float:
+        """A bound on scores before the cap, with room for the rounding of q and k to bf16; 0: none."""
+        return 1.02 * self.dim * abs(self.scale) if self.unit_qk else 0.0
+
+    @property
     def out_dim(self) -> int:
         return self.heads * self.vdim
 

@@ -2,7 +2,7 @@
 groups, without a capacity (every chosen expert runs), and experts whose gated unit is bounded.
 
 Few rows stream the weights of the chosen experts (:func:`experts_few`).  Larger batches are sorted by
-expert into a buffer whose experts start at multiples of ``BLOCK`` rows, and the experts' products are one
+expert into a buffer whose experts start at multiples of a block of rows, and the experts' products are one
 grouped launch each (:func:`route`, :func:`sort_rows`, :func:`grouped_linear`); the results leave through
 :class:`coeus_b200.ops.ragged.Spread`.
 
@@ -19,7 +19,7 @@ import torch
 from . import _lib
 from .gemm import clamped_glu
 
-BLOCK = 128           # rows of one expert's tile
+BLOCKS = (128, 256)   # rows of one expert's tile: 256 where experts have many
 FEW = 16              # rows up to which the experts' weights are streamed
 ROUTE_FEW = 128       # rows up to which the router's product and the choice are one launch
 ROUTE_TOKENS = 32     # tokens per block of the choice otherwise
@@ -90,7 +90,7 @@ def route(h: torch.Tensor, router: torch.Tensor, r: Routing) -> Choice:
 
 @dataclass
 class Sorted:
-    """``rows [blocks * BLOCK, W]``: every token's row once per expert it uses, sorted by expert;
+    """``rows [blocks * 128 or 256, W]``: every token's row once per expert it uses, sorted by expert;
     ``slot [tokens, top]`` says where; ``block_expert [blocks]`` is the expert of a block of rows, -1 behind
     the last one."""
 
@@ -102,9 +102,10 @@ class Sorted:
 def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
     T, W = h.shape
     pairs = T * r.top
-    blocks = pairs // BLOCK + min(r.experts, pairs)
+    block = BLOCKS[1] if pairs >= 1024 * r.experts else BLOCKS[0]
+    blocks = pairs // block + min(r.experts, pairs)
     dev = h.device
-    rows = torch.empty((blocks * BLOCK, W), dtype=h.dtype, device=dev)
+    rows = torch.empty((blocks * block, W), dtype=h.dtype, device=dev)
     if not h.is_cuda:
         rows.zero_()
         slot = torch.empty((T, r.top), dtype=torch.int32)
@@ -114,9 +115,9 @@ def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
             if len(t):
                 slot[t, k] = torch.arange(at, at + len(t), dtype=torch.int32)
                 rows[at:at + len(t)] = h[t]
-                n = (len(t) + BLOCK - 1) // BLOCK
+                n = (len(t) + block - 1) // block
                 block_expert += [e] * n
-                at += n * BLOCK
+                at += n * block
         block_expert += [-1] * (blocks - len(block_expert))
         return Sorted(rows, slot, torch.tensor(block_expert, dtype=torch.int32))
     slot = torch.empty((T, r.top), dtype=torch.int32, device=dev)
@@ -124,7 +125,7 @@ def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
     base = torch.empty_like(c.counts)
     rc = _lib.serving_lib().cb_moe_sort(
         _p(h), h.stride(0), _p(c.expert), _p(c.rank), _p(c.counts), T, r.experts, r.top, c.per_block,
-        c.counts.shape[0], _p(base), _p(slot), _p(block_expert), blocks, _p(rows), W,
+        c.counts.shape[0], _p(base), _p(slot), _p(block_expert), blocks, block, _p(rows), W,
         int(h.dtype == torch.float32), _p(_lib.status_buffer(dev)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_moe_sort", launches=2)
     return Sorted(rows, slot, block_expert)
@@ -132,16 +133,17 @@ def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
 
 def grouped_linear(x: torch.Tensor, w: torch.Tensor, block_expert: torch.Tensor, out: torch.Tensor, *,
                    glu: Optional[Tuple[float, float]] = None) -> torch.Tensor:
-    """``out[block] = x[block] @ w[block_expert[block]]^T`` for every block of ``BLOCK`` rows (``w [experts, N,
-    K]``); blocks of no expert are left alone.  ``glu = (slope, limit)``: see :func:`coeus_b200.ops.gemm.linear`."""
+    """``out[block] = x[block] @ w[block_expert[block]]^T`` for every block of rows (``w [experts, N, K]``, as
+    many blocks as ``block_expert`` has entries, of 128 or 256 rows); blocks of no expert are left alone.  ``glu = (slope, limit)``: see :func:`coeus_b200.ops.gemm.linear`."""
     E, N, K = w.shape
     M = x.shape[0]
-    if x.shape[1] != K or M != block_expert.shape[0] * BLOCK or out.shape != (M, N // 2 if glu else N):
+    block = M // block_expert.shape[0]
+    if x.shape[1] != K or block not in BLOCKS or M != block_expert.shape[0] * block or out.shape != (M, N // 2 if glu else N):
         raise ValueError(f"grouped_linear: shapes {tuple(x.shape)} {tuple(w.shape)} {tuple(out.shape)}")
     if not x.is_cuda:
         for b, e in enumerate(block_expert.tolist()):
             if e >= 0:
-                s = slice(b * BLOCK, (b + 1) * BLOCK)
+                s = slice(b * block, (b + 1) * block)
                 z = x[s].float() @ w[e].float().t()
                 out[s] = (clamped_glu(z, *glu) if glu else z).to(out.dtype)
         return out
@@ -149,12 +151,12 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, block_expert: torch.Tensor,
     lib, st = _lib.serving_lib(), _p(_lib.status_buffer(x.device))
     if x.dtype == torch.float32:
         rc = lib.cb_linear_f32_grouped(
-            _p(x), x.stride(0), _p(w), w.stride(1), _p(block_expert), _p(out), out.stride(0), M, N, K,
+            _p(x), x.stride(0), _p(w), w.stride(1), _p(block_expert), block, _p(out), out.stride(0), M, N, K,
             int(glu is not None), _F(slope), _F(limit), _lib.stream_ptr())
         _lib.check_rc(rc, "cb_linear_f32_grouped")
         return out
     rc = lib.cb_gemm_bf16_blocks(
-        _p(x), _p(w), _p(out), M, N, K, E, x.stride(0), w.stride(1), out.stride(0), _p(block_expert),
+        _p(x), _p(w), _p(out), M, N, K, E, x.stride(0), w.stride(1), out.stride(0), _p(block_expert), block,
         int(glu is not None), _F(slope), _F(limit), st, _lib.stream_ptr())
     _lib.check_rc(rc, "cb_gemm_bf16_blocks")
     return out

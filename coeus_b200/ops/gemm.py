@@ -336,12 +336,12 @@ def _linear_glu(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, slope: floa
         return out.copy_(clamped_glu(x.float() @ w.float().t(), slope, limit).to(out.dtype))
     lib, F = _lib.serving_lib(), ctypes.c_float
     if x.dtype == torch.float32:
-        rc = lib.cb_linear_f32_grouped(_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), None, _lib.ptr(out),
+        rc = lib.cb_linear_f32_grouped(_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), None, 128, _lib.ptr(out),
                                        out.stride(0), M, N, K, 1, F(slope), F(limit), _lib.stream_ptr())
         _lib.check_rc(rc, "cb_linear_f32_grouped")
         return out
     rc = lib.cb_gemm_bf16_blocks(_lib.ptr(x), _lib.ptr(w), _lib.ptr(out), M, N, K, 1, x.stride(0), w.stride(0),
-                                 out.stride(0), None, 1, F(slope), F(limit),
+                                 out.stride(0), None, 128, 1, F(slope), F(limit),
                                  _lib.ptr(_lib.status_buffer(x.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_gemm_bf16_blocks")
     return out

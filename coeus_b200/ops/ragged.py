@@ -575,7 +575,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      page_table: torch.Tensor, batch: RaggedBatch, heads: int, kv_heads: int,
                      dim: int, vdim: int, scale: float, out: torch.Tensor, *,
                      chunk: Optional[int] = None, window: Optional[int] = None,
-                     softcap: Optional[float] = None, maps: int = 1,
+                     softcap: Optional[float] = None, score_max: float = 0.0, maps: int = 1,
                      map_weight: Optional[torch.Tensor] = None, map_factor: float = 1.0,
                      eps: float = 0.0, sink: Optional[torch.Tensor] = None,
                      gate: Optional[torch.Tensor] = None, gate_wide: bool = False,
@@ -585,7 +585,8 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      plan: Optional[AttnPlan] = None) -> torch.Tensor:
     """Causal attention of every query row over the cached keys of its own sequence, restricted to
     the row's chunk (positions with the same ``pos // chunk``) when ``chunk`` is given, or to itself and
-    the ``window - 1`` positions before it.  Scores ``s`` become ``softcap * tanh(s / softcap)``.  ``sink``
+    the ``window - 1`` positions before it.  Scores ``s`` become ``softcap * tanh(s / softcap)``
+    (``score_max`` bounds ``|s|``, 0 where no bound is known).  ``sink``
     (fp32 ``[heads]``) is a logit that enters the softmax denominator only; ``gate`` multiplies by its
     sigmoid: a view whose column ``h`` belongs to head ``h``, or (``gate_wide``) a view like ``out``.  Query
     head ``h`` reads key/value head ``h // (heads // kv_heads)``.  ``q`` is ``[rows, heads, Q >= dim]``,
@@ -664,7 +665,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                 longest, heads, kv_heads, k_rows.shape[2], v_rows.shape[2], vdim, q.stride(0),
                 k_rows.stride(0), v_rows.stride(0), out.stride(0), _F(scale), _p(sink), _p(gate),
                 gate.stride(0) if gate is not None else 0, int(gate_wide), window or 0,
-                _F(softcap or 0.0), maps, _p(map_weight), _F(map_factor), _F(eps), st, _lib.stream_ptr())
+                _F(softcap or 0.0), _F(score_max), maps, _p(map_weight), _F(map_factor), _F(eps), st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_attn_fwd_pieces")
     if n:
         per = heads // kv_heads * maps

@@ -94,7 +94,7 @@ def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> Li
             q, out = prep(), torch.empty((T, nh * s.vdim), dtype=bf, device=dev)
             attn = lambda: R.ragged_attention(                                       # noqa: E731
                 q, c.k[i], c.v[i], c.page_table, batch, nh, kv, s.dim, s.vdim, s.scale, out, window=s.window,
-                softcap=s.softcap, maps=s.maps, map_weight=layer.map_weight,
+                softcap=s.softcap, score_max=s.score_max, maps=s.maps, map_weight=layer.map_weight,
                 map_factor=1.0 - s.diff if s.maps == 2 else 1.0, eps=eps,
                 gate=raw[:, layer.seg["g"]:] if s.gated else None, gate_wide=True, k_rows=k_rows, v_rows=v_rows,
                 plan=plan)

@@ -137,7 +137,7 @@ def check_spread(device, dtype, tol):
 ROUTERS = (H.MoeSpec(6, 3, E(13, 0.8), 1.7, 3, 2, E(21, 1.5)), H.MoeSpec(16, 4, E(40, 1.0), 2.5, 4, 2, E(72, 3.0)),
            H.MoeSpec(5, 1, E(9, 0.5), 1.0, 1, 1, None), H.MoeSpec(1, 1, E(16, 1.0), 3.0, 1, 1, E(8, 0.2)),
            H.MoeSpec(40, 12, E(24, 1.1), 0.5, 40, 20, None), H.MoeSpec(96, 6, E(8, 1.0), 1.0, 8, 3, E(136, 1.0)),
-           H.MoeSpec(12, 4, E(64, 1.0), 1.0, 6, 2, E(64, 1.0)))
+           H.MoeSpec(12, 4, E(64, 1.0), 1.0, 6, 2, E(64, 1.0)), H.MoeSpec(2, 1, E(136, 1.0), 1.0, 1, 1, None))
 
 
 def check_route(device, dtype, tol):
@@ -179,7 +179,7 @@ def check_experts(device, dtype, tol):
         eng, layer = lm.make_engine(max_batch=1), lm.layers[0]
         d = {n: t.double() for n, t in w.items()}
         g = torch.Generator().manual_seed(i)
-        for T in (1, 5, 16, 40, 150, 300) if i == 1 else (3, 17, 131):
+        for T in (1, 5, 16, 40, 150, 300) if i == 1 else (3, 17, 131) if m.experts > 2 else (2, 2100):
             h = torch.randn(T, W, generator=g)
             for t in range(T):
                 h[t, :m.experts] = levels(m, g)
@@ -263,9 +263,9 @@ def check_capped_attention(device, dtype, tol):
     page's border, or one somewhere in between."""
     T = 210
     for spec, seed in ((C(6, 3, 10, 14, 2.0, 6, 300.0, 9, 30.0), 1), (C(4, 2, 64, 40, 0.4, 64, 1e4, 64, 25.0), 2),
-                       (C(18, 1, 128, 128, 0.2, 32, 1e5, 100, 40.0), 3), (C(2, 2, 24, 64, 1.0, 24, 50.0, 1, 9.0), 4),
+                       (C(18, 1, 128, 128, 0.2, 32, 1e5, 100, 20.0), 3), (C(2, 2, 24, 64, 1.0, 24, 50.0, 1, 9.0), 4),
                        (C(2, 1, 160, 16, 0.15, 160, 1e3, 130, 60.0), 5), (C(4, 2, 8, 200, 2.5, 8, 1e4, 65, 30.0), 6),
-                       (C(3, 3, 40, 32, 0.6, 0, 1.0, 300, 50.0), 7)):
+                       (C(3, 3, 40, 72, 0.6, 0, 1.0, 300, 50.0), 7)):
         lm, w = single_mixer(spec, "Rupasun", device, dtype, seed)
         layer, H_, Gr, d, dv, size = lm.layers[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.window
         seg, m = layer.seg, dict(scale=spec.scale, mask=dict(size=size), softcap=spec.softcap)
