@@ -22,13 +22,15 @@
 // Grouped-query attention: query head h reads K/V head h / (nh / nkv).
 //
 // Two variants serve prompts of unequal length (PIECES) only.  CAP: scores s become cap * tanh(s / cap),
-// from the exponential unit (1) or, where the argument is known not to leave [-1, 1], as a polynomial on
-// the FMA pipe (2).  DIFF: a head has two maps, each with queries and keys of its own over the same values; an item is ONE
+// from the exponential unit (1) or, where the argument is known not to leave [-1, 1] or [-1/2, 1/2], as
+// an odd polynomial on the FMA pipe (2, 3).  DIFF: a head has two maps, each with queries and keys of its own over the same values; an item is ONE
 // query tile of a head, tiles A and B of the step are its two maps, every step has its own key tile and
 // every pair of steps its value tile.  At the end each warpgroup takes half of the columns of
 // o = a0 - w a1, and the two meet at two barriers: one when both results are complete, one for the sum of
 // squares of o, which is divided by its root mean square.
 // Every wait is bounded; a wait that runs out records a status code and the CTA leaves.
+#include <cmath>
+
 #include "common.cuh"
 #include "ptx.cuh"
 
@@ -66,7 +68,8 @@ struct AttnFwdArgs {
   int gate_wide;
   int window;                  // 0: no window
   float cap_log2, cap_in;      // CAP: the cap in units of log2, and what takes a product to the tanh
-  float cap_poly[7];           // CAP 2: score / product as a polynomial in the product's square
+  float cap_poly[7];           // CAP 2, 3: score / product as a polynomial in the product's square, of
+                               // degree 6 or 3
   const float* map_weight;     // DIFF: weight of the second map, factor and eps of the norm
   float map_factor, map_eps;
 };
@@ -136,6 +139,7 @@ struct AFWalk {
   int4 piece;            // PIECES: the entry of AttnFwdArgs::pieces
   const int4* pieces;
   int n0, n1, nmax;      // key tiles of tile A / B (0: the tile does not exist)
+  int lo0, lo1, window;  // first key tile of A / B that a row's window reaches
   int kv_seq;            // how many (item, j) groups came before this one: the K/V ring position
   bool valid;
 
@@ -153,6 +157,7 @@ struct AFWalk {
     n_bh = p.B * p.nh;
     n_items = n_pairs * n_bh;
     causal = p.causal;
+    window = p.window;
     pieces = p.pieces;
     n_waves = (n_items + gridDim.x - 1) / gridDim.x;
     wave = -1;
@@ -185,14 +190,22 @@ struct AFWalk {
            : qa + 1 >= n_q_tiles ? 0
            : (causal ? min(n_kv_tiles, (ahead + (qa + 2) * AF_BM + bkv - 1) / bkv) : n_kv_tiles);
       nmax = max(n0, n1);
-      j = 0;
+      lo0 = lo1 = 0;
+      if constexpr (PIECES) {
+        if (window > 0) {
+          const int low = ahead + qa * AF_BM + 1 - window;     // first key of the tile's first row
+          lo0 = max(0, low) / bkv;
+          lo1 = DIFF ? lo0 : max(0, low + AF_BM) / bkv;
+        }
+      }
+      j = lo0;
       t = 0;
       ++kv_seq;
       return;
     }
   }
   __device__ void advance() {
-    if (t == 0 && j < n1) { t = 1; return; }
+    if (t == 0 && j < n1 && j >= lo1) { t = 1; return; }
     ++j;
     if (j < nmax) {
       ++kv_seq;
@@ -201,7 +214,8 @@ struct AFWalk {
     }
     next_item();
   }
-  __device__ bool last_of_kv() const { return t == 1 || j >= n1; }   // last tile using K_j / V_j
+  __device__ bool last_of_kv() const { return t == 1 || j >= n1 || j < lo1; }   // last tile using K_j / V_j
+  __device__ bool first_of_tile() const { return j == (t ? lo1 : lo0); }
   __device__ bool last_of_tile() const { return j == (t ? n1 : n0) - 1; }
 };
 
@@ -287,7 +301,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       while (w.valid && ok) {
         const int row0 = w.first_row(p), kv_row0 = w.first_key(p);
         const int h = w.h, hk = w.h / group, qa = w.qa;
-        const int n0 = w.n0, n1 = w.n1, nmax = w.nmax;
+        const int n0 = w.n0, n1 = w.n1, nmax = w.nmax, lo = w.lo0;
         auto load_q = [&](int t) {
           if ((t == 0 ? n0 : n1) == 0) return;
           if (!mbar_wait(bar(Cfg::B_QE + t), (qcnt[t] & 1u) ^ 1u, abort_flag)) {
@@ -332,11 +346,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           ++vcnt;
         };
         load_q(0);
-        if (ok) load_k(0, 0);
+        if (ok) load_k(lo, 0);
         if (ok) load_q(1);
-        if (DIFF && ok) load_k(0, 1);
-        if (ok) load_v(0);
-        for (int j = 1; j < nmax && ok; ++j) {
+        if (DIFF && ok) load_k(lo, 1);
+        if (ok) load_v(lo);
+        for (int j = lo + 1; j < nmax && ok; ++j) {
           load_k(j, 0);
           if (DIFF && ok) load_k(j, 1);
           if (ok) load_v(j);
@@ -397,7 +411,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         const uint64_t bd0 = dV0 + static_cast<uint64_t>((vs * Cfg::V_BYTES) >> 4);
         const uint32_t d_addr = tmem_u + Cfg::O_COL0 + t * DV;
         const uint32_t a_addr = tmem_u + Cfg::S_COL0 + buf * BKV;
-        const uint32_t acc0 = wp.j > 0 ? 1u : 0u;
+        const uint32_t acc0 = wp.first_of_tile() ? 0u : 1u;
         const bool last_kv = wp.last_of_kv();
         if (elect_one()) {
 #pragma unroll
@@ -436,7 +450,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         const uint32_t buf = gs % NBUF;
         // the buffer is free once P.V of the step that used it last has completed
         if (gs >= NBUF && !wait1(Cfg::B_BF + buf, ((gs / NBUF) - 1u) & 1u, 963)) break;
-        if (ws.j == 0) {
+        if (ws.first_of_tile()) {
           if (!wait1(Cfg::B_QF + t, (t ? qc1 : qc0) & 1u, 960)) break;
           if (t) ++qc1; else ++qc0;
         }
@@ -490,7 +504,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       const int j = w.j;
       const int q0 = w.tile() * AF_BM;
       const int q_idx = q0 + r;
-      if (j == 0) {
+      const bool first = w.first_of_tile();
+      if (first) {
         m_used = -INFINITY;
         l[0] = l[1] = l[2] = l[3] = 0.f;
       }
@@ -554,14 +569,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       for (int c = 0; c < BKV / 32; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v + c * 32);
       tmem_ld_wait();
       if (tr) tr[tri + 1] = clock64();
-      if constexpr (CAP == 2) {
+      if constexpr (CAP >= 2) {
+        constexpr int DEG = CAP == 2 ? 6 : 3;
 #pragma unroll
         for (int e = 0; e < BKV; e += 2) {
           const float a = __uint_as_float(v[e]), b = __uint_as_float(v[e + 1]);
-          float wa, wb, ra = p.cap_poly[6], rb = ra;
+          float wa, wb, ra = p.cap_poly[DEG], rb = ra;
           fma2(wa, wb, a, b, a, b, 0.f, 0.f);
 #pragma unroll
-          for (int i = 5; i >= 0; --i) fma2(ra, rb, ra, rb, wa, wb, p.cap_poly[i], p.cap_poly[i]);
+          for (int i = DEG - 1; i >= 0; --i) fma2(ra, rb, ra, rb, wa, wb, p.cap_poly[i], p.cap_poly[i]);
           fma2(ra, rb, ra, rb, a, b, 0.f, 0.f);
           v[e] = __float_as_uint(ra);
           v[e + 1] = __float_as_uint(rb);
@@ -595,7 +611,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if constexpr (!CAP) mx *= p.scale_log2;  // scale > 0, so max commutes with it
       const float m_new = fmaxf(m_used, mx);
       const bool grow = (m_new - m_used) > 8.0f;  // also true for the first step (m_used = -inf)
-      if (j > 0 && __any_sync(0xffffffffu, grow)) {
+      if (!first && __any_sync(0xffffffffu, grow)) {
         // O_t may be rescaled once P.V of the previous step of this tile has completed.  (The
         // wait is skipped when no row needs rescaling: the barrier of that buffer cannot advance
         // a second time before this step hands over its P, so no phase is missed.)
@@ -911,6 +927,24 @@ extern "C" int cb_attn_fwd(const void* q, const void* k, const void* v, void* o,
                              poly, 0, 0u, status, max_ctas, stream);
 }
 
+// Coefficients c[0 .. n] of the polynomial in u = x * x that meets tanh(x) / x at the n + 1 Chebyshev nodes
+// of u in [0, bound^2] (Newton's divided differences, multiplied out).  x times it is within 3e-7 of
+// tanh(x) for n = 6, bound = 1 and for n = 3, bound = 1/2.
+static void tanh_ratio(double bound, int n, double* c) {
+  double u[8], d[8];
+  for (int i = 0; i <= n; ++i) {
+    u[i] = 0.5 * bound * bound * (1.0 + std::cos(3.14159265358979323846 * (i + 0.5) / (n + 1)));
+    d[i] = std::tanh(std::sqrt(u[i])) / std::sqrt(u[i]);
+  }
+  for (int k = 1; k <= n; ++k)
+    for (int i = n; i >= k; --i) d[i] = (d[i] - d[i - 1]) / (u[i] - u[i - k]);
+  for (int i = 0; i <= n; ++i) c[i] = 0.0;
+  for (int k = n; k >= 0; --k) {                 // c <- c * (x - u[k]) + d[k]
+    for (int i = n; i > 0; --i) c[i] = c[i - 1] - u[k] * c[i];
+    c[0] = d[k] - u[k] * c[0];
+  }
+}
+
 // Causal attention of a ragged batch in pieces (see AttnFwdArgs): n_pieces quadruples over `rows`
 // query rows and `kv_rows` key rows, none with more than max_len queries.  Heads of q and k are dq
 // apart, heads of v dv (64 or 128, padded with zeros), heads of o vdim <= dv.  sink (fp32 [nh]) is a logit
@@ -969,12 +1003,15 @@ extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, v
     a.cap_log2 = softcap * 1.4426950408889634f;
     a.cap_in = scale / softcap;
     if (score_max > 0.f && score_max <= softcap) {
-      // tanh(x) / x on [0, 1] as a polynomial in x^2: interpolated at Chebyshev nodes, |error| of tanh < 1e-7
-      const double t[7] = {0.99999994, -0.33332828, 0.13325076, -0.05345165, 0.02027971, -0.0061943247,
-                           0.0010380251};
+      const bool narrow = score_max <= 0.5f * softcap;
+      double t[7];
+      tanh_ratio(narrow ? 0.5 : 1.0, narrow ? 3 : 6, t);
       double f = static_cast<double>(a.cap_log2) * a.cap_in;
-      for (int i = 0; i < 7; ++i, f *= static_cast<double>(a.cap_in) * a.cap_in)
+      for (int i = 0; i <= (narrow ? 3 : 6); ++i, f *= static_cast<double>(a.cap_in) * a.cap_in)
         a.cap_poly[i] = static_cast<float>(t[i] * f);
+      if (narrow)
+        return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, 3>(tq, tk, tv, a, 0, st)
+                        : launch_attn_fwd<128, 128, false, false, true, 3>(tq, tk, tv, a, 0, st);
       return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, 2>(tq, tk, tv, a, 0, st)
                       : launch_attn_fwd<128, 128, false, false, true, 2>(tq, tk, tv, a, 0, st);
     }

@@ -621,33 +621,39 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
   const int t0 = lo + split * piece, t1 = min(pos + 1, t0 + piece);
   bf16* mine = ring + warp * 2 * STAGE;
   const int kch = p.kdim / 8, vch = p.vdim_p / 8;
+  // rows of nch vectors of eight, one per key (cell), to shared memory
+  auto copy = [&](const bf16* src, size_t stride, int nch, uint32_t dst, int pitch, int cell, int left) {
+    if ((nch & (nch - 1)) == 0 && nch <= 32) {          // a lane keeps its column
+      const int sh = __ffs(nch) - 1, c = lane & (nch - 1);
+      src += c * 8;
+      dst += c * 16;
+#pragma unroll 4
+      for (int key = lane >> sh; key < GA_KEYS; key += 32 >> sh)
+        cp_async16_zfill(dst + key * pitch * 2, src + __shfl_sync(0xffffffffu, cell, key) * stride,
+                         key < left ? 16 : 0);
+      return;
+    }
+    for (int x = lane; x < GA_KEYS * nch; x += 32) {
+      const int key = x / nch, c = x % nch;
+      cp_async16_zfill(dst + (key * pitch + c * 8) * 2, src + __shfl_sync(0xffffffffu, cell, key) * stride + c * 8,
+                       key < left ? 16 : 0);
+    }
+  };
   auto fetch = [&](int tb, int st) {                    // keys tb .. tb + 31 into a stage
     const int t = tb + lane;
-    int page = 0;
+    int cell = 0;
     if (t < t1) {
       const int lp = t / RAGGED_PAGE;
-      page = lp < p.max_pages ? pt[lp] : -1;
+      int page = lp < p.max_pages ? pt[lp] : -1;
       if (page < 0 || page >= p.num_pages) {
         record_status(p.status, ST_BOUNDS, row);
         page = 0;
       }
+      cell = page * RAGGED_PAGE + t % RAGGED_PAGE;
     }
-    bf16* kd = mine + st * STAGE;
-    bf16* vd = kd + GA_KEYS * KS;
-    for (int x = lane; x < GA_KEYS * kch; x += 32) {
-      const int key = x / kch, c = x % kch;
-      const int pg = __shfl_sync(0xffffffffu, page, key);
-      const size_t cell = static_cast<size_t>(pg) * RAGGED_PAGE + (tb + key) % RAGGED_PAGE;
-      cp_async16_zfill(smem_u32(kd + key * KS + c * 8), kc + cell * p.kv_heads * p.kdim + c * 8,
-                       tb + key < t1 ? 16 : 0);
-    }
-    for (int x = lane; x < GA_KEYS * vch; x += 32) {
-      const int key = x / vch, c = x % vch;
-      const int pg = __shfl_sync(0xffffffffu, page, key);
-      const size_t cell = static_cast<size_t>(pg) * RAGGED_PAGE + (tb + key) % RAGGED_PAGE;
-      cp_async16_zfill(smem_u32(vd + key * VS + c * 8), vc + cell * p.kv_heads * p.vdim_p + c * 8,
-                       tb + key < t1 ? 16 : 0);
-    }
+    const uint32_t kd = smem_u32(mine + st * STAGE);
+    copy(kc, static_cast<size_t>(p.kv_heads) * p.kdim, kch, kd, KS, cell, t1 - tb);
+    copy(vc, static_cast<size_t>(p.kv_heads) * p.vdim_p, vch, kd + GA_KEYS * KS * 2, VS, cell, t1 - tb);
     cp_async_commit();
   };
   // zero the padding columns of this warp's ring, then start loading

@@ -265,7 +265,8 @@ def check_capped_attention(device, dtype, tol):
     for spec, seed in ((C(6, 3, 10, 14, 2.0, 6, 300.0, 9, 30.0), 1), (C(4, 2, 64, 40, 0.4, 64, 1e4, 64, 25.0), 2),
                        (C(18, 1, 128, 128, 0.2, 32, 1e5, 100, 20.0), 3), (C(2, 2, 24, 64, 1.0, 24, 50.0, 1, 9.0), 4),
                        (C(2, 1, 160, 16, 0.15, 160, 1e3, 130, 60.0), 5), (C(4, 2, 8, 200, 2.5, 8, 1e4, 65, 30.0), 6),
-                       (C(3, 3, 40, 72, 0.6, 0, 1.0, 300, 50.0), 7)):
+                       (C(3, 3, 40, 72, 0.6, 0, 1.0, 300, 50.0), 7), (C(2, 2, 96, 80, 0.25, 96, 1e4, 64, 25.0), 8),
+                       (C(2, 1, 56, 48, 0.4, 8, 1e2, 128, 30.0), 9), (C(2, 1, 20, 20, 1.2, 20, 1e3, 5, 60.0), 10)):
         lm, w = single_mixer(spec, "Rupasun", device, dtype, seed)
         layer, H_, Gr, d, dv, size = lm.layers[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.window
         seg, m = layer.seg, dict(scale=spec.scale, mask=dict(size=size), softcap=spec.softcap)
