@@ -30,7 +30,8 @@ struct Choose {
   int* expert;             // [T, top]
   float* weight;           // [T, top]
   int* rank;               // [T, top] among the block's earlier pairs of the same expert
-  int* counts;             // [blocks, E]
+  int* counts;             // [E, blocks]
+  int blocks;
 };
 
 // (value, index) of the largest of v over the warp, the lowest index among equals.
@@ -122,45 +123,48 @@ __global__ void __launch_bounds__(CHOOSE_WARPS * 32) moe_choose_kernel(const Cho
     p.rank[static_cast<size_t>(t0) * p.top + i] = r;
   }
   for (int e = threadIdx.x; e < p.E; e += CHOOSE_WARPS * 32)
-    p.counts[static_cast<size_t>(blockIdx.x) * p.E + e] = hist[e];
+    p.counts[static_cast<size_t>(e) * p.blocks + blockIdx.x] = hist[e];
 }
 
-// One token per block, with the router's product: four experts per warp at a time.
+// One token per block, with the router's product: two experts per warp at a time.
 template <typename T>
 __global__ void __launch_bounds__(512) moe_choose_few_kernel(const Choose p) {
   __shared__ float s[MOE_E + 4], gv[MOE_E];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x, nw = blockDim.x >> 5;
   const T* h = static_cast<const T*>(p.h) + static_cast<size_t>(t) * p.ldh;
   const T* r = static_cast<const T*>(p.router);
-  for (int e0 = warp * 4; e0 < p.E; e0 += nw * 4) {
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 2
+  for (int e0 = warp * 2; e0 < p.E; e0 += nw * 2) {
+    const T* r0 = r + static_cast<size_t>(e0) * p.ldr;
+    const T* r1 = r + static_cast<size_t>(min(e0 + 1, p.E - 1)) * p.ldr;
+    float a = 0.f, b = 0.f;
+#pragma unroll 4
     for (int c = lane * 8; c < p.W; c += 256) {
-      float x[8];
+      float x[8], u[8], v[8];
       load_vec<8>(h + c, x);
+      load_vec<8>(r0 + c, u);
+      load_vec<8>(r1 + c, v);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        float w[8];
-        load_vec<8>(r + static_cast<size_t>(min(e0 + i, p.E - 1)) * p.ldr + c, w);
-#pragma unroll
-        for (int k = 0; k < 8; ++k) acc[i] += x[k] * w[k];
+      for (int k = 0; k < 8; ++k) {
+        a += x[k] * u[k];
+        b += x[k] * v[k];
       }
     }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      acc[i] = warp_sum(acc[i]);
-      if (lane == 0) s[e0 + i] = acc[i];
+    a = warp_sum(a);
+    b = warp_sum(b);
+    if (lane == 0) {
+      s[e0] = a;
+      s[e0 + 1] = b;
     }
   }
   __syncthreads();
   if (warp != 0) return;
   choose_token(p, t, s, gv);
-  for (int e = lane; e < p.E; e += 32) p.counts[static_cast<size_t>(t) * p.E + e] = 0;
+  for (int e = lane; e < p.E; e += 32) p.counts[static_cast<size_t>(e) * p.blocks + t] = 0;
   __syncwarp();
   if (lane < p.top) {
     const size_t at = static_cast<size_t>(t) * p.top + lane;
     p.rank[at] = 0;
-    p.counts[static_cast<size_t>(t) * p.E + p.expert[at]] = 1;
+    p.counts[static_cast<size_t>(p.expert[at]) * p.blocks + t] = 1;
   }
 }
 
@@ -171,7 +175,8 @@ moe_place_kernel(const int* __restrict__ counts, int blocks, int E, int* __restr
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int e = warp; e < E; e += 32) {
     int n = 0;
-    for (int b = lane; b < blocks; b += 32) n += counts[static_cast<size_t>(b) * E + e];
+#pragma unroll 8
+    for (int b = lane; b < blocks; b += 32) n += counts[static_cast<size_t>(e) * blocks + b];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) n += __shfl_xor_sync(FULL, n, o);
     if (lane == 0) total[e] = n;
@@ -198,16 +203,28 @@ moe_place_kernel(const int* __restrict__ counts, int blocks, int E, int* __restr
     for (int i = start[e] + lane; i < start[e + 1]; i += 32)
       if (i < n_tiles) block_expert[i] = e;
     int run = start[e] * tile_rows;
-    for (int b0 = 0; b0 < blocks; b0 += 32) {
-      const int b = b0 + lane;
-      const int n = b < blocks ? counts[static_cast<size_t>(b) * E + e] : 0;
-      int incl = n;
+    const size_t at = static_cast<size_t>(e) * blocks;
+    for (int b0 = 0; b0 < blocks; b0 += 256) {       // a lane sums up eight blocks
+      int n[8], sum = 0;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int b = b0 + lane * 8 + i;
+        n[i] = b < blocks ? counts[at + b] : 0;
+        sum += n[i];
+      }
+      int incl = sum;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const int v = __shfl_up_sync(FULL, incl, o);
         if (lane >= o) incl += v;
       }
-      if (b < blocks) base[static_cast<size_t>(b) * E + e] = run + incl - n;
+      int before = run + incl - sum;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int b = b0 + lane * 8 + i;
+        if (b < blocks) base[at + b] = before;
+        before += n[i];
+      }
       run += __shfl_sync(FULL, incl, 31);
     }
   }
@@ -216,14 +233,14 @@ moe_place_kernel(const int* __restrict__ counts, int blocks, int E, int* __restr
 // One block per token: its row (nv vectors of 16 bytes) once per expert.
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(const uint4* __restrict__ h, int ldh, const int* __restrict__ expert,
-                  const int* __restrict__ rank, const int* __restrict__ base, int E, int top,
+                  const int* __restrict__ rank, const int* __restrict__ base, int blocks, int top,
                   int per_block, int* __restrict__ slot, uint4* __restrict__ rows, int nv, int n_rows,
                   int* status) {
   __shared__ int to[MOE_K];
   const int t = blockIdx.x;
   if (threadIdx.x < top) {
     const size_t i = static_cast<size_t>(t) * top + threadIdx.x;
-    int at = base[static_cast<size_t>(t / per_block) * E + expert[i]] + rank[i];
+    int at = base[static_cast<size_t>(expert[i]) * blocks + t / per_block] + rank[i];
     if (at < 0 || at >= n_rows) {
       record_status(status, ST_BOUNDS, t);
       at = 0;
@@ -468,9 +485,10 @@ extern "C" int cb_moe_choose(const float* logits, int ldl, const void* h, int ld
   p.logits = logits; p.ldl = ldl; p.h = h; p.ldh = ldh; p.router = router; p.ldr = ldr; p.W = W;
   p.T = T; p.E = E; p.top = top; p.groups = groups; p.keep = keep; p.scale = scale; p.expert = expert;
   p.weight = weight; p.rank = rank; p.counts = counts;
+  p.blocks = logits != nullptr ? (T + CHOOSE_TOKENS - 1) / CHOOSE_TOKENS : T;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (logits != nullptr)
-    moe_choose_kernel<<<(T + CHOOSE_TOKENS - 1) / CHOOSE_TOKENS, CHOOSE_WARPS * 32, 0, st>>>(p);
+    moe_choose_kernel<<<p.blocks, CHOOSE_WARPS * 32, 0, st>>>(p);
   else if (f32)
     moe_choose_few_kernel<float><<<T, 512, 0, st>>>(p);
   else
@@ -478,7 +496,7 @@ extern "C" int cb_moe_choose(const float* logits, int ldl, const void* h, int ld
   return CB_RC();
 }
 
-// rows [n_tiles * tile_rows, W]; base has the shape of counts [blocks, E].
+// rows [n_tiles * tile_rows, W]; base has the shape of counts [E, blocks].
 extern "C" int cb_moe_sort(const void* h, int ldh, const int* expert, const int* rank, const int* counts,
                            int T, int E, int top, int per_block, int blocks, int* base, int* slot,
                            int* block_expert, int n_tiles, int tile_rows, void* rows, int W, int f32, int* status,
@@ -491,7 +509,7 @@ extern "C" int cb_moe_sort(const void* h, int ldh, const int* expert, const int*
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   moe_place_kernel<<<1, 1024, 0, st>>>(counts, blocks, E, base, block_expert, n_tiles, tile_rows);
   const int nv = W / v, threads = nv >= 256 ? 256 : (nv + 31) / 32 * 32;
-  moe_gather_kernel<<<T, threads, 0, st>>>(static_cast<const uint4*>(h), ldh / v, expert, rank, base, E, top,
+  moe_gather_kernel<<<T, threads, 0, st>>>(static_cast<const uint4*>(h), ldh / v, expert, rank, base, blocks, top,
                                            per_block, slot, static_cast<uint4*>(rows), nv,
                                            n_tiles * tile_rows, status);
   return CB_RC();

@@ -286,32 +286,42 @@ __global__ void __launch_bounds__(64) ragged_attn_merge_kernel(const RowsArgs ra
 }
 
 // Two maps: merges the splits of both and takes their difference.  At most 256 columns.
+constexpr int RA_SPLITS = 16;
 template <typename T>
 __global__ void __launch_bounds__(128) ragged_attn_difference_kernel(const RowsArgs ra) {
   const RaggedAttn& p = ra.a;
   __shared__ float red[32];
-  const int i = blockIdx.x, h = blockIdx.y;
+  __shared__ float part[2 * RA_SPLITS];          // factor of every split's sum
+  const int i = blockIdx.x, h = blockIdx.y, n = ra.splits;
   const int row = ra.rows != nullptr ? ra.rows[i] : i;
-  const float w = *p.map_weight;
+  const size_t base = (static_cast<size_t>(i) * p.heads + h * 2) * n;      // the second map's follow
+  if (threadIdx.x < 32) {
+    // lanes 0 .. 15: the first map's splits, 16 .. 31: the second's
+    const int m = threadIdx.x / RA_SPLITS, k = threadIdx.x % RA_SPLITS;
+    const bool in = k < n;
+    const float mk = in ? ra.part_ml[(base + m * n + k) * 2] : -INFINITY;
+    const float lk = in ? ra.part_ml[(base + m * n + k) * 2 + 1] : 0.f;
+    float gm = mk;
+#pragma unroll
+    for (int o = RA_SPLITS / 2; o > 0; o >>= 1) gm = fmaxf(gm, __shfl_xor_sync(0xffffffffu, gm, o));
+    const float c = mk == -INFINITY ? 0.f : exp2_t<T>(mk - gm);
+    float gl = lk * c;
+#pragma unroll
+    for (int o = RA_SPLITS / 2; o > 0; o >>= 1) gl += __shfl_xor_sync(0xffffffffu, gl, o);
+    part[threadIdx.x] = (m == 0 ? c : -*p.map_weight * c) / gl;
+  }
+  __syncthreads();
   float o[2] = {0.f, 0.f};
 #pragma unroll
   for (int m = 0; m < 2; ++m) {
-    const size_t base = (static_cast<size_t>(i) * p.heads + h * 2 + m) * ra.splits;
-    float gm = -INFINITY, gl = 0.f;
-    for (int s = 0; s < ra.splits; ++s) gm = fmaxf(gm, ra.part_ml[(base + s) * 2]);
-    for (int s = 0; s < ra.splits; ++s) {
-      const float ms = ra.part_ml[(base + s) * 2];
-      gl += ms == -INFINITY ? 0.f : ra.part_ml[(base + s) * 2 + 1] * exp2_t<T>(ms - gm);
-    }
-    const float dn = (m == 0 ? 1.f : -w) / denom<T>(p, h * 2 + m, gm, gl);
-    for (int s = 0; s < ra.splits; ++s) {
-      const float ms = ra.part_ml[(base + s) * 2];
-      if (ms == -INFINITY) continue;
-      const float c = exp2_t<T>(ms - gm) * dn;
+#pragma unroll 8
+    for (int k = 0; k < n; ++k) {
+      const float c = part[m * RA_SPLITS + k];
+      const float* src = ra.part_o + (base + m * n + k) * p.vdim;
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         const int d = threadIdx.x + 128 * x;
-        if (d < p.vdim) o[x] += ra.part_o[(base + s) * p.vdim + d] * c;
+        if (d < p.vdim) o[x] += c != 0.f ? src[d] * c : 0.f;     // a split without keys has no sum
       }
     }
   }
@@ -922,7 +932,7 @@ extern "C" int cb_ragged_attn_rows(const void* q, int q_head, const void* k_cach
   const int rc = fill_attn(a.a, q, q_head, k_cache, v_cache, page_table, max_pages, num_pages, *spec, sink,
                            gate, ldg, map_weight, out, ldo, status);
   if (rc != 0) return rc;
-  if (n <= 0 || splits < 1 || ((splits > 1 || spec->maps == 2) && (part_o == nullptr || part_ml == nullptr)))
+  if (n <= 0 || splits < 1 || (spec->maps == 2 && splits > RA_SPLITS) || ((splits > 1 || spec->maps == 2) && (part_o == nullptr || part_ml == nullptr)))
     return -5;
   a.rows = rows; a.row_slot = row_slot; a.row_pos = row_pos; a.splits = splits;
   a.part_o = part_o; a.part_ml = part_ml;

@@ -79,7 +79,7 @@ def route(h: torch.Tensor, router: torch.Tensor, r: Routing) -> Choice:
     blocks = (T + per - 1) // per
     expert, rank = (torch.empty((T, r.top), dtype=torch.int32, device=dev) for _ in range(2))
     weight = torch.empty((T, r.top), dtype=torch.float32, device=dev)
-    counts = torch.empty((blocks, r.experts), dtype=torch.int32, device=dev)
+    counts = torch.empty((r.experts, blocks), dtype=torch.int32, device=dev)
     rc = _lib.serving_lib().cb_moe_choose(
         _p(logits), logits.stride(0) if logits is not None else 0, _p(h), h.stride(0), _p(router),
         router.stride(0), W, T, r.experts, r.top, r.groups, r.keep, _F(r.scale), _p(expert), _p(weight),
@@ -125,7 +125,7 @@ def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
     base = torch.empty_like(c.counts)
     rc = _lib.serving_lib().cb_moe_sort(
         _p(h), h.stride(0), _p(c.expert), _p(c.rank), _p(c.counts), T, r.experts, r.top, c.per_block,
-        c.counts.shape[0], _p(base), _p(slot), _p(block_expert), blocks, block, _p(rows), W,
+        c.counts.shape[1], _p(base), _p(slot), _p(block_expert), blocks, block, _p(rows), W,
         int(h.dtype == torch.float32), _p(_lib.status_buffer(dev)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_moe_sort", launches=2)
     return Sorted(rows, slot, block_expert)
