@@ -256,7 +256,7 @@ moe_gather_kernel(const uint4* __restrict__ h, int ldh, const int* __restrict__ 
 }
 
 // ------------------------------------------------------------------------------- few rows
-constexpr int FEW_WARPS = 8;
+constexpr int FEW_WARPS = 8, DOWN_WARPS = 16;    // the second product has few blocks and long sums
 
 struct Few {
   const __nv_bfloat16* h;        // [M, ldh]
@@ -321,11 +321,11 @@ __device__ __forceinline__ void few_mma(float (*acc)[4], const uint4 (*a)[2], co
 }
 
 // Adds the warps' 16 x (NT * 8) results; the sum of row c, token m is red[m * 17 + c] of warp 0's part.
-template <int NT>
+template <int NT, int WARPS>
 __device__ __forceinline__ float few_sum(const float* red, int m, int c) {
   float v = 0.f;
 #pragma unroll
-  for (int w = 0; w < FEW_WARPS; ++w) v += red[(w * NT * 8 + m) * 17 + c];
+  for (int w = 0; w < WARPS; ++w) v += red[(w * NT * 8 + m) * 17 + c];
   return v;
 }
 template <int NT>
@@ -411,14 +411,14 @@ __global__ void __launch_bounds__(FEW_WARPS * 32) moe_few_in_kernel(const Few p)
     if (2 * ch >= rows) continue;
     float v = 0.f;
     if (wt[m] != 0.f)
-      v = wt[m] * clamped_glu(few_sum<NT>(red, m, 2 * c), few_sum<NT>(red, m, 2 * c + 1), p.slope, limit);
+      v = wt[m] * clamped_glu(few_sum<NT, FEW_WARPS>(red, m, 2 * c), few_sum<NT, FEW_WARPS>(red, m, 2 * c + 1), p.slope, limit);
     p.act[static_cast<size_t>(m) * p.lda + col0 + ch] = __float2bfloat16(v);
   }
 }
 
 template <int NT>
-__global__ void __launch_bounds__(FEW_WARPS * 32) moe_few_down_kernel(const Few p) {
-  __shared__ float red[FEW_WARPS * NT * 8 * 17];
+__global__ void __launch_bounds__(DOWN_WARPS * 32) moe_few_down_kernel(const Few p) {
+  __shared__ float red[DOWN_WARPS * NT * 8 * 17];
   __shared__ int list[MOE_E], count;
   __shared__ uint32_t bits[MOE_E / 32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n0 = blockIdx.x * 16;
@@ -436,11 +436,11 @@ __global__ void __launch_bounds__(FEW_WARPS * 32) moe_few_down_kernel(const Few 
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   const int per = (p.n + 63) / 64, chunks = live * per + (p.ns + 63) / 64;
   constexpr int U = NT == 1 ? 4 : 2;
-  for (int c0 = warp; c0 < chunks; c0 += FEW_WARPS * U) {
+  for (int c0 = warp; c0 < chunks; c0 += DOWN_WARPS * U) {
     uint4 x[U][2][2], b[U][NT][2];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      const int c = c0 + u * FEW_WARPS;
+      const int c = c0 + u * DOWN_WARPS;
       const bool in = c < chunks, sh = c >= live * per;
       const int a = sh ? 0 : c / per, k0 = (sh ? c - live * per : c % per) * 64 + q;
       const int n = sh ? p.ns : p.n;
@@ -462,9 +462,9 @@ __global__ void __launch_bounds__(FEW_WARPS * 32) moe_few_down_kernel(const Few 
   }
   few_store<NT>(red, warp, lane, acc);
   __syncthreads();
-  for (int i = threadIdx.x; i < p.M * 16; i += FEW_WARPS * 32) {
+  for (int i = threadIdx.x; i < p.M * 16; i += DOWN_WARPS * 32) {
     const int m = i >> 4, c = i & 15;
-    if (n0 + c < p.W) p.y[static_cast<size_t>(m) * p.ldy + n0 + c] = few_sum<NT>(red, m, c);
+    if (n0 + c < p.W) p.y[static_cast<size_t>(m) * p.ldy + n0 + c] = few_sum<NT, DOWN_WARPS>(red, m, c);
   }
 }
 
@@ -536,10 +536,10 @@ extern "C" int cb_moe_few(const void* h, int ldh, int M, int W, int E, int top, 
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (M <= 8) {
     moe_few_in_kernel<1><<<in_blocks, FEW_WARPS * 32, 0, st>>>(p);
-    moe_few_down_kernel<1><<<down_blocks, FEW_WARPS * 32, 0, st>>>(p);
+    moe_few_down_kernel<1><<<down_blocks, DOWN_WARPS * 32, 0, st>>>(p);
   } else {
     moe_few_in_kernel<2><<<in_blocks, FEW_WARPS * 32, 0, st>>>(p);
-    moe_few_down_kernel<2><<<down_blocks, FEW_WARPS * 32, 0, st>>>(p);
+    moe_few_down_kernel<2><<<down_blocks, DOWN_WARPS * 32, 0, st>>>(p);
   }
   return CB_RC();
 }
