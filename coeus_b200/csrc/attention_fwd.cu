@@ -27,7 +27,8 @@
 // query tile of a head, tiles A and B of the step are its two maps, every step has its own key tile and
 // every pair of steps its value tile.  At the end each warpgroup takes half of the columns of
 // o = a0 - w a1, and the two meet at two barriers: one when both results are complete, one for the sum of
-// squares of o, which is divided by its root mean square.
+// squares of o, which is divided by its root mean square.  KEPT (with a window): the first positions of the
+// sequence stay visible behind the window; their keys are tiles of their own in front of an item's others.
 // Every wait is bounded; a wait that runs out records a status code and the CTA leaves.
 #include <cmath>
 
@@ -59,7 +60,9 @@ struct AttnFwdArgs {
   float drop_scale;
   // Pieces of unequal length instead of B sequences of S rows.  Piece b has y = pieces[b].y query
   // rows (at most S) from row pieces[b].x on and w + y keys from row pieces[b].z of K and V on; its
-  // query i sees the first w + i + 1 of them (causal), or of those the last `window`.  null: none
+  // query i sees the first w + i + 1 of them (causal), or of those the last `window`.  Two quadruples per
+  // piece: with KEPT the second one says that positions 0 .. y - 1 of the sequence, keys from row x on,
+  // stay visible, and that z positions lie before the piece's first key.  null: none
   const int4* pieces;
   int vdim;                    // columns of a head that are stored, vdim apart in O
   const float* sink;           // [nh] logits that enter the denominator only, or null
@@ -132,7 +135,7 @@ __device__ __forceinline__ float exp2_poly(float x) {
 // item of every wave of gridDim.x items, counted from the front of even waves and from the back
 // of odd ones, so that the heavy and the light ends of the sorted list meet in one CTA), within
 // an item key tile by key tile, tile A before tile B.
-template <bool PIECES, bool DIFF = false>
+template <bool PIECES, bool DIFF = false, bool KEPT = false>
 struct AFWalk {
   // problem
   int n_items, n_bh, n_pairs, n_q_tiles, n_kv_tiles, nh, causal, bkv, n_waves;
@@ -145,12 +148,22 @@ struct AFWalk {
   int lo0, lo1, window;  // first key tile of A / B that a row's window reaches
   int kv_seq;            // how many (item, j) groups came before this one: the K/V ring position
   bool valid;
+  int4 kept;             // KEPT: the piece's second quadruple; its kt tiles are j = -kt .. -1
+  int kt;
 
   __device__ int first_row(const AttnFwdArgs& p) const { return PIECES ? piece.x : b * p.S; }
   __device__ int first_key(const AttnFwdArgs& p) const { return PIECES ? piece.z : b * p.S; }
   __device__ int rows(const AttnFwdArgs& p) const { return PIECES ? piece.y : p.S; }
   __device__ int tile() const { return DIFF ? qa : qa + t; }           // query tile of this step
   __device__ int keys_ahead() const { return PIECES ? piece.w : 0; }   // keys before query 0's own
+  // KEPT: first position in the window of query q
+  __device__ int low_position(int q) const { return kept.z + max(0, piece.w + q + 1 - window); }
+  __device__ int first_tile() const { return KEPT && kt > 0 ? -kt : lo0; }
+  __device__ int next_tile(int i) const { return KEPT && i == -1 ? lo0 : i + 1; }
+  __device__ int tile_row(const AttnFwdArgs& p, int i) const {
+    return KEPT && i < 0 ? kept.x + (i + kt) * bkv : first_key(p) + i * bkv;
+  }
+  __device__ bool b_has(int i) const { return KEPT && i < 0 ? n1 > 0 : i < n1 && i >= lo1; }
   __device__ void init(const AttnFwdArgs& p, int bkv_) {
     bkv = bkv_;
     n_q_tiles = (p.S + AF_BM - 1) / AF_BM;
@@ -182,7 +195,8 @@ struct AFWalk {
       h = bh % nh;
       qa = DIFF ? pair : 2 * pair;
       if constexpr (PIECES) {
-        piece = pieces[b];
+        piece = pieces[2 * b];
+        if constexpr (KEPT) kept = pieces[2 * b + 1];
         n_q_tiles = (piece.y + AF_BM - 1) / AF_BM;
         n_kv_tiles = (piece.w + piece.y + bkv - 1) / bkv;
         if (qa >= n_q_tiles) continue;             // a shorter piece ends before this pair
@@ -201,15 +215,19 @@ struct AFWalk {
           lo1 = DIFF ? lo0 : max(0, low + AF_BM) / bkv;
         }
       }
-      j = lo0;
+      if constexpr (KEPT) {
+        const int low = low_position(min(piece.y, (qa + 2) * AF_BM) - 1);
+        kt = (min(kept.y, low) + bkv - 1) / bkv;
+      }
+      j = first_tile();
       t = 0;
       ++kv_seq;
       return;
     }
   }
   __device__ void advance() {
-    if (t == 0 && j < n1 && j >= lo1) { t = 1; return; }
-    ++j;
+    if (t == 0 && b_has(j)) { t = 1; return; }
+    j = next_tile(j);
     if (j < nmax) {
       ++kv_seq;
       t = j < n0 ? 0 : 1;
@@ -217,19 +235,19 @@ struct AFWalk {
     }
     next_item();
   }
-  __device__ bool last_of_kv() const { return t == 1 || j >= n1 || j < lo1; }   // last tile using K_j / V_j
-  __device__ bool first_of_tile() const { return j == (t ? lo1 : lo0); }
+  __device__ bool last_of_kv() const { return t == 1 || !b_has(j); }   // last tile using K_j / V_j
+  __device__ bool first_of_tile() const { return j == (KEPT && kt > 0 ? -kt : t ? lo1 : lo0); }
   __device__ bool last_of_tile() const { return j == (t ? n1 : n0) - 1; }
 };
 
-template <int DQ, int DV, bool POLY, bool DROP, bool PIECES, int CAP, bool DIFF>
+template <int DQ, int DV, bool POLY, bool DROP, bool PIECES, int CAP, bool DIFF, bool KEPT>
 __global__ void __launch_bounds__(AF_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const AttnFwdArgs p) {
-  static_assert(PIECES || (!CAP && !DIFF), "the variants of pieces");
+  static_assert(PIECES || (!CAP && !DIFF && !KEPT), "the variants of pieces");
   static_assert(!CAP || !DIFF, "no kernel has both");
   using Cfg = AFCfg<DQ, DV, DIFF>;
-  using Walk = AFWalk<PIECES, DIFF>;
+  using Walk = AFWalk<PIECES, DIFF, KEPT>;
   constexpr int KST = Cfg::KST, VST = Cfg::VST, NBUF = Cfg::NBUF, BKV = Cfg::BKV;
   constexpr int MAPS = DIFF ? 2 : 1;
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -302,9 +320,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       Walk w;
       w.init(p, BKV);
       while (w.valid && ok) {
-        const int row0 = w.first_row(p), kv_row0 = w.first_key(p);
+        const int row0 = w.first_row(p);
         const int h = w.h, hk = w.h / group, qa = w.qa;
-        const int n0 = w.n0, n1 = w.n1, nmax = w.nmax, lo = w.lo0;
+        const int n0 = w.n0, n1 = w.n1, nmax = w.nmax, lo = w.first_tile();
         auto load_q = [&](int t) {
           if ((t == 0 ? n0 : n1) == 0) return;
           if (!mbar_wait(bar(Cfg::B_QE + t), (qcnt[t] & 1u) ^ 1u, abort_flag)) {
@@ -331,7 +349,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int c = 0; c < DQ / 64; ++c)
             tma_load_2d(sK(s) + c * (BKV * 128), &tmK, bar(Cfg::B_KF + s), (hk * MAPS + map) * DQ + c * 64,
-                        kv_row0 + j * BKV);
+                        w.tile_row(p, j));
           ++kcnt;
         };
         auto load_v = [&](int j) {
@@ -345,7 +363,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int c = 0; c < DV / 64; ++c)
             tma_load_2d(sV(s) + c * (BKV * 128), &tmV, bar(Cfg::B_VF + s), hk * DV + c * 64,
-                        kv_row0 + j * BKV);
+                        w.tile_row(p, j));
           ++vcnt;
         };
         load_q(0);
@@ -353,7 +371,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         if (ok) load_q(1);
         if (DIFF && ok) load_k(lo, 1);
         if (ok) load_v(lo);
-        for (int j = lo + 1; j < nmax && ok; ++j) {
+        for (int j = w.next_tile(lo); j < nmax && ok; j = w.next_tile(j)) {
           load_k(j, 0);
           if (DIFF && ok) load_k(j, 1);
           if (ok) load_v(j);
@@ -561,12 +579,21 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       ++mine;
       if (tr) tr[tri] = clock64();
       tc_fence_after();
-      const int kv0 = j * BKV;
+      int kv0 = j * BKV;
       const bool below = PIECES && p.window > 0;
-      const bool need_mask = (p.causal && kv0 + BKV - 1 > q0 + w.keys_ahead()) ||
+      bool need_mask = (p.causal && kv0 + BKV - 1 > q0 + w.keys_ahead()) ||
                              (kv0 + BKV > w.keys_ahead() + w.rows(p)) ||
                              (below && kv0 < q0 + AF_BM + w.keys_ahead() - p.window);
-      const int kv_limit = w.keys_ahead() + (p.causal ? min(q_idx, w.rows(p) - 1) : (w.rows(p) - 1));  // last visible key
+      int kv_limit = w.keys_ahead() + (p.causal ? min(q_idx, w.rows(p) - 1) : (w.rows(p) - 1));  // last visible key
+      int kv_low = below ? kv_limit - p.window : -1;                                             // last one hidden below
+      if constexpr (KEPT) {
+        if (j < 0) {          // kept positions that lie below the row's window
+          kv0 = (j + w.kt) * BKV;
+          kv_limit = min(w.kept.y, w.low_position(min(q_idx, w.rows(p) - 1))) - 1;
+          kv_low = -1;
+          need_mask = true;
+        }
+      }
       uint32_t v[BKV];
 #pragma unroll
       for (int c = 0; c < BKV / 32; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v + c * 32);
@@ -594,7 +621,6 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         // hidden keys get a score of -inf, after which the step takes the common path (their
         // exponential is an exact zero); with causal masking every row sees at least key 0, with
         // a window at least its own key
-        const int kv_low = below ? kv_limit - p.window : -1;
 #pragma unroll
         for (int e = 0; e < BKV; ++e)
           if (kv0 + e > kv_limit || (PIECES && kv0 + e <= kv_low)) v[e] = 0xff800000u;
@@ -844,12 +870,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
-template <int DQ, int DV, bool POLY, bool DROP = false, bool PIECES = false, int CAP = 0, bool DIFF = false>
+template <int DQ, int DV, bool POLY, bool DROP = false, bool PIECES = false, int CAP = 0, bool DIFF = false,
+          bool KEPT = false>
 static int launch_attn_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
                               const AttnFwdArgs& a, int max_ctas, cudaStream_t st) {
   using Cfg = AFCfg<DQ, DV, DIFF>;
   static bool configured = false;
-  auto kern = attn_fwd_kernel<DQ, DV, POLY, DROP, PIECES, CAP, DIFF>;
+  auto kern = attn_fwd_kernel<DQ, DV, POLY, DROP, PIECES, CAP, DIFF, KEPT>;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES) != cudaSuccess)
       return -10;
@@ -948,12 +975,13 @@ static void tanh_ratio(double bound, int n, double* c) {
   }
 }
 
-// Causal attention of a ragged batch in pieces (see AttnFwdArgs): n_pieces quadruples over `rows`
+// Causal attention of a ragged batch in pieces (see AttnFwdArgs): n_pieces pairs of quadruples over `rows`
 // query rows and `kv_rows` key rows, none with more than max_len queries.  Heads of q and k are dq
 // apart, heads of v dv (64 or 128, padded with zeros), heads of o vdim <= dv.  sink (fp32 [nh]) is a logit
 // per head that enters the softmax denominator only; gate (bf16, column h of a pitch-ldg view, or with
 // gate_wide column h * vdim + d) multiplies head h's output by its sigmoid; both may be null.  A
-// query sees the last `window` of its keys (0: all).  scale > 0.  Scores are capped by softcap (0: not).
+// query sees the last `window` of its keys (0: all), with keep > 0 also the first positions that the pieces
+// name.  scale > 0.  Scores are capped by softcap (0: not).
 // score_max bounds |q . k| * scale where the caller knows it (0: not known).
 // With two maps q and k have two heads per head (map 0 first), and the output is the weighted difference
 // divided by its root mean square, times map_factor; it has neither sink, gate nor cap.
@@ -961,13 +989,14 @@ extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, v
                                   int kv_rows, const void* pieces, int n_pieces, int max_len, int nh,
                                   int nkv, int dq, int dv, int vdim, int ldq, int ldk, int ldv, int ldo,
                                   float scale, const float* sink, const void* gate, int ldg,
-                                  int gate_wide, int window, float softcap, float score_max, int maps,
+                                  int gate_wide, int window, int keep, float softcap, float score_max, int maps,
                                   const float* map_weight, float map_factor, float map_eps, int* status,
                                   void* stream) {
   using namespace cb;
   if (!(dq == 64 && dv == 64) && !(dq == 128 && dv == 128) && !(dq == 64 && dv == 128 && maps == 2)) return -1;
   if (gate_wide && vdim % 8 == 0 && ((reinterpret_cast<uintptr_t>(gate) & 15u) || ldg % 8)) return -6;
-  if (window < 0 || softcap < 0.f || (maps != 1 && maps != 2)) return -2;
+  if (window < 0 || keep < 0 || softcap < 0.f || (maps != 1 && maps != 2)) return -2;
+  if (keep > 0 && (window == 0 || maps == 2 || softcap > 0.f)) return -7;
   if (maps == 2 && (sink != nullptr || gate != nullptr || softcap > 0.f || map_weight == nullptr)) return -7;
   if (softcap > 0.f && sink != nullptr) return -7;
   if (rows <= 0 || kv_rows <= 0 || n_pieces <= 0 || max_len <= 0 || nh <= 0 || nkv <= 0 ||
@@ -1021,6 +1050,9 @@ extern "C" int cb_attn_fwd_pieces(const void* q, const void* k, const void* v, v
     return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, 1>(tq, tk, tv, a, 0, st)
                     : launch_attn_fwd<128, 128, false, false, true, 1>(tq, tk, tv, a, 0, st);
   }
+  if (keep > 0)
+    return dv == 64 ? launch_attn_fwd<64, 64, false, false, true, 0, false, true>(tq, tk, tv, a, 0, st)
+                    : launch_attn_fwd<128, 128, false, false, true, 0, false, true>(tq, tk, tv, a, 0, st);
   return dv == 64 ? launch_attn_fwd<64, 64, false, false, true>(tq, tk, tv, a, 0, st)
                   : launch_attn_fwd<128, 128, false, false, true>(tq, tk, tv, a, 0, st);
 }

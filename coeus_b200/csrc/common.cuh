@@ -96,10 +96,10 @@ __device__ __forceinline__ float dropout_factor(uint32_t bits, int lane, int thr
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 
 // The gated unit of an expert: g bounded above, u on both sides, g * sigmoid(slope * g) * (u + 1).
-__device__ __forceinline__ float clamped_glu(float g, float u, float slope, float limit) {
+__device__ __forceinline__ float clamped_glu(float g, float u, float slope, float limit, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return __fdividef(g * (u + 1.0f), 1.0f + __expf(-slope * g));
+  return __fdividef(g * (u + shift), 1.0f + __expf(-slope * g));
 }
 // tanh from the fast exponential, absolute error below 3e-7
 __device__ __forceinline__ float tanh_exp(float x) {

@@ -1,8 +1,10 @@
 // Mixture of experts of the serving step: no capacity, every chosen expert runs.
-//   moe_choose   sigmoid scores, the best groups (by the sum of a group's two largest scores), the top
-//                experts in them, weights = scores / their sum * scale.  Few tokens: one block per token
+//   moe_choose   sigmoid or softmax scores, the best groups (by the sum of a group's largest scores, two or
+//                one), the top experts in them, weights = scores (over their sum) * scale.  A correction per
+//                expert can be added to the scores for the choice.  Few tokens: one block per token
 //                computes the router's product as well.  More: the logits are given, a block takes
-//                CHOOSE_TOKENS tokens and counts its pairs per expert.
+//                CHOOSE_TOKENS tokens and counts its pairs per expert.  One more logit can be the gate of the
+//                shared expert.  The last experts can be identities: they get no rows and no weights.
 //   moe_place    one block: where every block's pairs of an expert go in a buffer sorted by expert, whose
 //                experts start at multiples of a block of rows, and the expert of every block
 //   moe_gather   rows into that buffer
@@ -27,6 +29,9 @@ struct Choose {
   int ldh, ldr, W;
   int T, E, top, groups, keep;
   float scale;
+  int softmax, group_best, normalise;
+  const float* correction; // [E] or null
+  float* shared;           // [T] or null: sigmoid of logit E
   int* expert;             // [T, top]
   float* weight;           // [T, top]
   int* rank;               // [T, top] among the block's earlier pairs of the same expert
@@ -44,57 +49,95 @@ __device__ __forceinline__ void warp_best(float& v, int& i) {
   }
 }
 
-// One warp, one token: s[E] holds the logits and becomes the scores; gv is scratch for the groups.
+// One warp, one token: s[E] holds the logits and becomes the scores that are compared; gv is scratch for the
+// groups.
 __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, float* gv) {
   const int lane = threadIdx.x & 31, n = p.E / p.groups;
-  for (int e = lane; e < p.E; e += 32) s[e] = sigmoidf_(s[e]);
+  float score[MOE_E / 32];                       // of this lane's experts lane, lane + 32, ...
+  float total = 1.f, top = 0.f;
+  if (p.softmax) {
+    top = -INFINITY;
+    for (int e = lane; e < p.E; e += 32) top = fmaxf(top, s[e]);
+    top = warp_max(top);
+    total = 0.f;
+    for (int e = lane; e < p.E; e += 32) total += expf(s[e] - top);
+    total = warp_sum(total);
+  }
+#pragma unroll
+  for (int i = 0; i < MOE_E / 32; ++i) {
+    const int e = lane + 32 * i;
+    score[i] = 0.f;
+    if (e < p.E) {
+      score[i] = p.softmax ? expf(s[e] - top) / total : sigmoidf_(s[e]);
+      s[e] = p.correction != nullptr ? score[i] + p.correction[e] : score[i];
+    }
+  }
   __syncwarp();
+  uint32_t open[MOE_E / 32];                     // kept groups
+#pragma unroll
+  for (int i = 0; i < MOE_E / 32; ++i) open[i] = 0xffffffffu;
   if (p.keep < p.groups) {
+#pragma unroll
+    for (int i = 0; i < MOE_E / 32; ++i) open[i] = 0u;
     for (int g = lane; g < p.groups; g += 32) {
-      float a = 0.f, b = 0.f;                    // scores are not negative
+      float a = -INFINITY, b = -INFINITY;
       for (int i = 0; i < n; ++i) {
         const float v = s[g * n + i];
         b = fmaxf(b, fminf(a, v));
         a = fmaxf(a, v);
       }
-      gv[g] = a + b;
+      gv[g] = p.group_best == 2 && n > 1 ? a + b : a;
     }
     __syncwarp();
     for (int k = 0; k < p.keep; ++k) {
-      float v = -1.f;
-      int at = 0x7fffffff;
+      float v = -INFINITY;
+      int at = p.groups - 1;                     // of scores that are no numbers, any
       for (int g = lane; g < p.groups; g += 32)
         if (gv[g] > v) { v = gv[g]; at = g; }
       warp_best(v, at);
       __syncwarp();
-      if (lane == 0) gv[at] = -2.f;              // kept
+      if (lane == 0) gv[at] = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < MOE_E / 32; ++i)
+        if (i == at >> 5) open[i] |= 1u << (at & 31);
       __syncwarp();
     }
   }
-  float left[MOE_E / 32];                        // this lane's experts lane, lane + 32, ...
+  float left[MOE_E / 32];
 #pragma unroll
   for (int i = 0; i < MOE_E / 32; ++i) {
     const int e = lane + 32 * i;
-    left[i] = e < p.E && (p.keep == p.groups || gv[e / n] == -2.f) ? s[e] : -1.f;
+    left[i] = -INFINITY;
+    if (e < p.E) {
+      const int g = e / n;
+      uint32_t bits = 0u;
+#pragma unroll
+      for (int x = 0; x < MOE_E / 32; ++x)
+        if (x == g >> 5) bits = open[x];
+      if (bits >> (g & 31) & 1u) left[i] = s[e];
+    }
   }
   float mine = 0.f, sum = 0.f;
   int chosen = 0;
   for (int k = 0; k < p.top; ++k) {
-    float v = -2.f;
-    int at = 0x7fffffff;
+    float v = -INFINITY, w = 0.f;
+    int at = p.E - 1;
 #pragma unroll
     for (int i = 0; i < MOE_E / 32; ++i)
       if (left[i] > v) { v = left[i]; at = lane + 32 * i; }
     warp_best(v, at);
 #pragma unroll
-    for (int i = 0; i < MOE_E / 32; ++i)
-      if (at == lane + 32 * i) left[i] = -3.f;
-    sum += v;
-    if (lane == k) { mine = v; chosen = at; }
+    for (int i = 0; i < MOE_E / 32; ++i) {
+      if (i == at >> 5) w = score[i];
+      if (at == lane + 32 * i) left[i] = -INFINITY;
+    }
+    w = __shfl_sync(FULL, w, at & 31);
+    sum += w;
+    if (lane == k) { mine = w; chosen = at; }
   }
   if (lane < p.top) {
     p.expert[static_cast<size_t>(t) * p.top + lane] = chosen;
-    p.weight[static_cast<size_t>(t) * p.top + lane] = mine / (sum + 1e-20f) * p.scale;
+    p.weight[static_cast<size_t>(t) * p.top + lane] = (p.normalise ? mine / (sum + 1e-20f) : mine) * p.scale;
   }
   __syncwarp();
 }
@@ -107,6 +150,8 @@ __global__ void __launch_bounds__(CHOOSE_WARPS * 32) moe_choose_kernel(const Cho
   for (int t = warp; t < nt; t += CHOOSE_WARPS) {
     for (int e = lane; e < p.E; e += 32) s[warp][e] = p.logits[static_cast<size_t>(t0 + t) * p.ldl + e];
     __syncwarp();
+    if (p.shared != nullptr && lane == 0)
+      p.shared[t0 + t] = sigmoidf_(p.logits[static_cast<size_t>(t0 + t) * p.ldl + p.E]);
     choose_token(p, t0 + t, s[warp], gv[warp]);
   }
   for (int e = threadIdx.x; e < p.E; e += CHOOSE_WARPS * 32) hist[e] = 0;
@@ -133,9 +178,10 @@ __global__ void __launch_bounds__(512) moe_choose_few_kernel(const Choose p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x, nw = blockDim.x >> 5;
   const T* h = static_cast<const T*>(p.h) + static_cast<size_t>(t) * p.ldh;
   const T* r = static_cast<const T*>(p.router);
-  for (int e0 = warp * 2; e0 < p.E; e0 += nw * 2) {
+  const int outputs = p.E + (p.shared != nullptr);
+  for (int e0 = warp * 2; e0 < outputs; e0 += nw * 2) {
     const T* r0 = r + static_cast<size_t>(e0) * p.ldr;
-    const T* r1 = r + static_cast<size_t>(min(e0 + 1, p.E - 1)) * p.ldr;
+    const T* r1 = r + static_cast<size_t>(min(e0 + 1, outputs - 1)) * p.ldr;
     float a = 0.f, b = 0.f;
 #pragma unroll 4
     for (int c = lane * 8; c < p.W; c += 256) {
@@ -158,6 +204,7 @@ __global__ void __launch_bounds__(512) moe_choose_few_kernel(const Choose p) {
   }
   __syncthreads();
   if (warp != 0) return;
+  if (p.shared != nullptr && lane == 0) p.shared[t] = sigmoidf_(s[p.E]);
   choose_token(p, t, s, gv);
   for (int e = lane; e < p.E; e += 32) p.counts[static_cast<size_t>(e) * p.blocks + t] = 0;
   __syncwarp();
@@ -234,16 +281,19 @@ moe_place_kernel(const int* __restrict__ counts, int blocks, int E, int* __restr
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(const uint4* __restrict__ h, int ldh, const int* __restrict__ expert,
                   const int* __restrict__ rank, const int* __restrict__ base, int blocks, int top,
-                  int per_block, int* __restrict__ slot, uint4* __restrict__ rows, int nv, int n_rows,
+                  int per_block, int* __restrict__ slot, uint4* __restrict__ rows, int nv, int n_rows, int E,
                   int* status) {
   __shared__ int to[MOE_K];
   const int t = blockIdx.x;
   if (threadIdx.x < top) {
     const size_t i = static_cast<size_t>(t) * top + threadIdx.x;
-    int at = base[static_cast<size_t>(expert[i]) * blocks + t / per_block] + rank[i];
-    if (at < 0 || at >= n_rows) {
-      record_status(status, ST_BOUNDS, t);
-      at = 0;
+    int at = -1;                                 // an identity expert
+    if (expert[i] < E) {
+      at = base[static_cast<size_t>(expert[i]) * blocks + t / per_block] + rank[i];
+      if (at < 0 || at >= n_rows) {
+        record_status(status, ST_BOUNDS, t);
+        at = 0;
+      }
     }
     to[threadIdx.x] = at;
     slot[i] = at;
@@ -251,7 +301,8 @@ moe_gather_kernel(const uint4* __restrict__ h, int ldh, const int* __restrict__ 
   __syncthreads();
   for (int c = threadIdx.x; c < nv; c += blockDim.x) {
     const uint4 v = h[static_cast<size_t>(t) * ldh + c];
-    for (int k = 0; k < top; ++k) rows[static_cast<size_t>(to[k]) * nv + c] = v;
+    for (int k = 0; k < top; ++k)
+      if (to[k] >= 0) rows[static_cast<size_t>(to[k]) * nv + c] = v;
   }
 }
 
@@ -260,15 +311,16 @@ constexpr int FEW_WARPS = 8, DOWN_WARPS = 16;    // the second product has few b
 
 struct Few {
   const __nv_bfloat16* h;        // [M, ldh]
-  int ldh, M, W, E, top;         // W: multiple of 8
+  int ldh, M, W, E, top;         // W: multiple of 8; experts from E on are identities
   const int* expert;             // [M, top]
   const float* weight;
+  const float* s_weight;         // [M] of the shared expert, or null: 1
   const __nv_bfloat16* w_in;     // [E, 2 n, W], gate and up rows alternate
   const __nv_bfloat16* w_down;   // [E, W, n]
   const __nv_bfloat16* s_in;     // [2 ns, W] or null
   const __nv_bfloat16* s_down;   // [W, ns]
   int n, ns, live;               // live: most experts that can be in use
-  float limit, s_limit, slope;
+  float limit, s_limit, slope, shift;
   __nv_bfloat16* act;            // [M, lda]: live * n columns of experts, then ns
   int lda;
   float* y;                      // [M, ldy]
@@ -280,7 +332,7 @@ __device__ __forceinline__ int live_experts(const Few& p, int* list, uint32_t* b
   if (threadIdx.x < MOE_E / 32) bits[threadIdx.x] = 0;
   __syncthreads();
   for (int i = threadIdx.x; i < p.M * p.top; i += blockDim.x)
-    atomicOr(&bits[p.expert[i] >> 5], 1u << (p.expert[i] & 31));
+    if (p.expert[i] < p.E) atomicOr(&bits[p.expert[i] >> 5], 1u << (p.expert[i] & 31));
   __syncthreads();
   if (threadIdx.x < 32) {
     const uint32_t b = threadIdx.x < MOE_E / 32 ? bits[threadIdx.x] : 0u;
@@ -363,7 +415,7 @@ __global__ void __launch_bounds__(FEW_WARPS * 32) moe_few_in_kernel(const Few p)
       wt[threadIdx.x] = v;
     }
   } else if (threadIdx.x < 16) {
-    wt[threadIdx.x] = 1.f;
+    wt[threadIdx.x] = p.s_weight != nullptr && static_cast<int>(threadIdx.x) < p.M ? p.s_weight[threadIdx.x] : 1.f;
   }
   const int r = lane >> 2, q = (lane & 3) * 16;
   const __nv_bfloat16* wp[2];
@@ -411,7 +463,8 @@ __global__ void __launch_bounds__(FEW_WARPS * 32) moe_few_in_kernel(const Few p)
     if (2 * ch >= rows) continue;
     float v = 0.f;
     if (wt[m] != 0.f)
-      v = wt[m] * clamped_glu(few_sum<NT, FEW_WARPS>(red, m, 2 * c), few_sum<NT, FEW_WARPS>(red, m, 2 * c + 1), p.slope, limit);
+      v = wt[m] * clamped_glu(few_sum<NT, FEW_WARPS>(red, m, 2 * c), few_sum<NT, FEW_WARPS>(red, m, 2 * c + 1), p.slope, limit,
+                              p.shift);
     p.act[static_cast<size_t>(m) * p.lda + col0 + ch] = __float2bfloat16(v);
   }
 }
@@ -464,7 +517,12 @@ __global__ void __launch_bounds__(DOWN_WARPS * 32) moe_few_down_kernel(const Few
   __syncthreads();
   for (int i = threadIdx.x; i < p.M * 16; i += DOWN_WARPS * 32) {
     const int m = i >> 4, c = i & 15;
-    if (n0 + c < p.W) p.y[static_cast<size_t>(m) * p.ldy + n0 + c] = few_sum<NT, DOWN_WARPS>(red, m, c);
+    if (n0 + c >= p.W) continue;
+    float v = few_sum<NT, DOWN_WARPS>(red, m, c);
+    for (int k = 0; k < p.top; ++k)
+      if (p.expert[m * p.top + k] >= p.E)
+        v += p.weight[m * p.top + k] * __bfloat162float(p.h[static_cast<size_t>(m) * p.ldh + n0 + c]);
+    p.y[static_cast<size_t>(m) * p.ldy + n0 + c] = v;
   }
 }
 
@@ -473,16 +531,21 @@ __global__ void __launch_bounds__(DOWN_WARPS * 32) moe_few_down_kernel(const Few
 using namespace cb;
 #define CB_RC() (cudaGetLastError() == cudaSuccess ? 0 : -3)
 
-// logits null: computed here, one block (of the counts) per token; else blocks of CHOOSE_TOKENS tokens.
+// logits null: computed here, one block (of the counts) per token; else blocks of CHOOSE_TOKENS tokens.  E
+// counts the identity experts too; shared (or null) gets the sigmoid of logit E.
 extern "C" int cb_moe_choose(const float* logits, int ldl, const void* h, int ldh, const void* router,
                              int ldr, int W, int T, int E, int top, int groups, int keep, float scale,
+                             int softmax, int group_best, int normalise, const float* correction, float* shared,
                              int* expert, float* weight, int* rank, int* counts, int f32, void* stream) {
   if (T <= 0 || E < 1 || E > MOE_E || top < 1 || top > MOE_K || groups < 1 || E % groups || keep < 1 ||
-      keep > groups || top > keep * (E / groups))
+      keep > groups || top > keep * (E / groups) || group_best < 1 || group_best > 2)
     return -1;
+  if (logits != nullptr && ldl < E + (shared != nullptr)) return -2;
   if (logits == nullptr && (h == nullptr || W % 8 || ldh % 8 || ldr % 8 || ldh < W || ldr < W)) return -2;
   Choose p;
   p.logits = logits; p.ldl = ldl; p.h = h; p.ldh = ldh; p.router = router; p.ldr = ldr; p.W = W;
+  p.softmax = softmax; p.group_best = group_best; p.normalise = normalise; p.correction = correction;
+  p.shared = shared;
   p.T = T; p.E = E; p.top = top; p.groups = groups; p.keep = keep; p.scale = scale; p.expert = expert;
   p.weight = weight; p.rank = rank; p.counts = counts;
   p.blocks = logits != nullptr ? (T + CHOOSE_TOKENS - 1) / CHOOSE_TOKENS : T;
@@ -496,7 +559,8 @@ extern "C" int cb_moe_choose(const float* logits, int ldl, const void* h, int ld
   return CB_RC();
 }
 
-// rows [n_tiles * tile_rows, W]; base has the shape of counts [E, blocks].
+// rows [n_tiles * tile_rows, W]; base has the shape of counts [E, blocks].  Pairs of experts from E on have no
+// row, their slot is -1.
 extern "C" int cb_moe_sort(const void* h, int ldh, const int* expert, const int* rank, const int* counts,
                            int T, int E, int top, int per_block, int blocks, int* base, int* slot,
                            int* block_expert, int n_tiles, int tile_rows, void* rows, int W, int f32, int* status,
@@ -511,15 +575,15 @@ extern "C" int cb_moe_sort(const void* h, int ldh, const int* expert, const int*
   const int nv = W / v, threads = nv >= 256 ? 256 : (nv + 31) / 32 * 32;
   moe_gather_kernel<<<T, threads, 0, st>>>(static_cast<const uint4*>(h), ldh / v, expert, rank, base, blocks, top,
                                            per_block, slot, static_cast<uint4*>(rows), nv,
-                                           n_tiles * tile_rows, status);
+                                           n_tiles * tile_rows, E, status);
   return CB_RC();
 }
 
 // All experts of up to 16 bf16 rows and the shared one (s_in null: none), complete in y (fp32).
 extern "C" int cb_moe_few(const void* h, int ldh, int M, int W, int E, int top, const int* expert,
-                          const float* weight, const void* w_in, const void* w_down, int n, float limit,
+                          const float* weight, const float* s_weight, const void* w_in, const void* w_down, int n, float limit,
                           const void* s_in, const void* s_down, int ns, float s_limit, float slope,
-                          void* act, int lda, float* y, int ldy, void* stream) {
+                          float shift, void* act, int lda, float* y, int ldy, void* stream) {
   if (M < 1 || M > 16 || E < 1 || E > MOE_E || top < 1 || top > MOE_K || W % 8 || ldh % 8 || n % 8 || n < 1 ||
       ns % 8 || (s_in == nullptr) != (ns == 0) || ldh < W || ldy < W)
     return -1;
@@ -530,7 +594,7 @@ extern "C" int cb_moe_few(const void* h, int ldh, int M, int W, int E, int top, 
   p.expert = expert; p.weight = weight; p.w_in = static_cast<const __nv_bfloat16*>(w_in);
   p.w_down = static_cast<const __nv_bfloat16*>(w_down); p.s_in = static_cast<const __nv_bfloat16*>(s_in);
   p.s_down = static_cast<const __nv_bfloat16*>(s_down); p.n = n; p.ns = ns; p.limit = limit;
-  p.s_limit = s_limit; p.slope = slope; p.act = static_cast<__nv_bfloat16*>(act); p.lda = lda; p.y = y;
+  p.s_limit = s_limit; p.slope = slope; p.shift = shift; p.s_weight = s_weight; p.act = static_cast<__nv_bfloat16*>(act); p.lda = lda; p.y = y;
   p.ldy = ldy;
   const int in_blocks = p.live * ((2 * n + 15) / 16) + (2 * ns + 15) / 16, down_blocks = (W + 15) / 16;
   cudaStream_t st = static_cast<cudaStream_t>(stream);

@@ -60,7 +60,7 @@ struct GemmArgs {
   int g_am, g_ak;               // g * g_am to A's m coordinate, g * g_ak to its k coordinate,
   int g_bn, g_bk;               // g * g_bn to B's n coordinate, g * g_bk to its k coordinate
   const int* block_group;       // group of every tile of rows instead (-1: none from here on), or null
-  float glu_slope, glu_limit;   // EPI_GLU: columns alternate g, u; the output has half as many
+  float glu_slope, glu_limit, glu_shift;   // EPI_GLU: columns alternate g, u; the output has half as many
   // ---- fused collectives over peer memory (COMM template parameter)
   int tp, rank;                 // ranks of the tensor-parallel group, this rank
   int tiles_per_shard;          // 128-row tiles per rank's sequence shard
@@ -641,10 +641,21 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               uint32_t r[32];
               tmem_ld_32x32b_x32(taddr + qs * 128 + h * 64 + half * 32, r);
               tmem_ld_wait();
+              if (p.bias != nullptr) {
+                const int col0 = n0 + qs * 128 + h * 64 + half * 32;
+#pragma unroll
+                for (int g = 0; g < 4; ++g)
+                  if (col0 + g * 8 < p.N) {
+                    float b[8];
+                    load8(p.bias + col0 + g * 8, b);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) r[g * 8 + j] = __float_as_uint(__uint_as_float(r[g * 8 + j]) + b[j]);
+                  }
+              }
 #pragma unroll
               for (int j = 0; j < 16; ++j)
                 v[half * 16 + j] = clamped_glu(__uint_as_float(r[2 * j]), __uint_as_float(r[2 * j + 1]),
-                                               p.glu_slope, p.glu_limit);
+                                               p.glu_slope, p.glu_limit, p.glu_shift);
             }
             stage_row(s_out, r_in_tile, h, v);
           }
@@ -1070,19 +1081,19 @@ extern "C" int cb_gemm_bf16_grouped(const void* A, const void* B, void* D, int g
                         stream, groups);
 }
 
-// D[rows of block b] = epilogue(A[rows of block b] . B[block_expert[b]]^T), blocks of 128 or 256 rows: A [M, K],
-// B [experts, N, K] (pitch ldb), D [M, N] or with glu (a bounded gated unit over alternating columns)
-// [M, N / 2], all bf16.  A negative entry says that this block and all behind it have no work; their
+// D[rows of block b] = epilogue(A[rows of block b] . B[block_expert[b]]^T + bias), blocks of 128 or 256 rows: A
+// [M, K], B [experts, N, K] (pitch ldb), bias [N] or null, D [M, N] or with glu (a gated unit over alternating
+// columns, see clamped_glu) [M, N / 2], all bf16.  A negative entry says that this block and all behind it have no work; their
 // rows of D are left alone.  block_expert null: one weight, any M.
-extern "C" int cb_gemm_bf16_blocks(const void* A, const void* B, void* D, int M, int N, int K, int experts,
+extern "C" int cb_gemm_bf16_blocks(const void* A, const void* B, const void* bias, void* D, int M, int N, int K, int experts,
                                    int lda, int ldb, int ldd, const int* block_expert, int block_rows,
-                                   int glu, float slope, float limit, int* status, void* stream) {
+                                   int glu, float slope, float limit, float shift, int* status, void* stream) {
   using namespace cb;
   const int cols = glu ? N / 2 : N;
   if (M <= 0 || N <= 0 || K <= 0 || experts < 1 || N % 8 || cols % 8 || K % 8 || ldd % 8) return -21;
   if (block_rows != GEMM_BM && block_rows != 2 * GEMM_BM) return -24;
   if (block_expert != nullptr && M % block_rows) return -24;
-  if (reinterpret_cast<uintptr_t>(D) & 15u) return -21;
+  if ((reinterpret_cast<uintptr_t>(D) & 15u) || (reinterpret_cast<uintptr_t>(bias) & 15u)) return -21;
   // CTA pairs work on 256 rows at a time, which have to be of one expert
   const bool pairs = block_expert == nullptr ? M >= 256 && N > 128 : block_rows == 2 * GEMM_BM;
   const long long wide = static_cast<long long>((M + GEMM_BM - 1) / GEMM_BM) * ((N + 255) / 256);
@@ -1105,6 +1116,8 @@ extern "C" int cb_gemm_bf16_blocks(const void* A, const void* B, void* D, int M,
   g.g_bn = N;
   g.glu_slope = slope;
   g.glu_limit = limit;
+  g.glu_shift = shift;
+  g.bias = static_cast<const __nv_bfloat16*>(bias);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (pairs) return launch_gemm_pair<false, false>(ta, tb, td, td, g, 0, st);
   return bn == 256 ? launch_gemm<256, false, false>(ta, tb, td, td, g, 0, st)

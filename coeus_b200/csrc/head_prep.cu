@@ -1,10 +1,11 @@
 // Between the projections and the scores of an attention layer without a convolution, for a ragged
-// batch: rotary embedding of q and k (pairs half a rotation apart, or neighbours), division of q and k
-// by their root mean square, and the write of k and v into the cache pages and, for the kernel that
+// batch: RMS norms of q and of k over all heads at once, rotary embedding of q and k (pairs half a rotation
+// apart, or neighbours), division of the heads of q and k, or of v, by their root mean square, a factor per
+// query head, and the write of k and v into the cache pages and, for the kernel that
 // works on pieces of prompts, row by row.
 //
 // One block per row; a group of L lanes takes one head of q or k, eight consecutive numbers per lane, or
-// as many of a head of v.
+// as many of a head of v.  Without key/value heads only q is made.
 #include "ragged.cuh"
 
 namespace cb {
@@ -17,8 +18,11 @@ struct HeadPrep {
   int heads, kv_heads, v_heads, dim, vdim;
   int half;                // rotated pairs per head (0: none)
   const float2* rope;      // [rows, half] (cos, sin)
-  int interleaved, unit;
+  int interleaved, unit, unit_v;
   float eps;
+  const float* q_norm;     // [heads * dim] or null
+  const float* k_norm;
+  const float* q_factor;   // [heads] or null
   void* q;                 // [rows, heads, q_head]
   int q_head;
   void* k_cache;           // [pages, PAGE, kv_heads, dim_p]
@@ -50,6 +54,19 @@ __device__ __forceinline__ void head_load(const T* src, int d, int n, float* f) 
   }
 }
 
+// Sum of squares of n numbers, this thread's share.
+template <typename T, bool VEC>
+__device__ __forceinline__ float row_squares(const T* src, int n) {
+  float s = 0.f;
+  for (int c = threadIdx.x * 8; c < n; c += HP_THREADS * 8) {
+    float f[8];
+    head_load<T, VEC>(src + c, 0, n - c, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) s += f[i] * f[i];
+  }
+  return s;
+}
+
 // VEC: head sizes (and, for pairs half a rotation apart, half) are multiples of eight.
 template <typename T, int L, bool VEC>
 __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p) {
@@ -63,6 +80,14 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
   const size_t cell = static_cast<size_t>(page) * RAGGED_PAGE + pos % RAGGED_PAGE;
   const T* raw = static_cast<const T*>(p.raw) + static_cast<size_t>(row) * p.ld;
   const float2* rope = p.rope + static_cast<size_t>(row) * p.half;
+  float q_rs = 1.f, k_rs = 1.f;
+  if (p.q_norm != nullptr) {
+    __shared__ float red[32];
+    q_rs = 1.0f / sqrtf(block_sum(row_squares<T, VEC>(raw, p.heads * p.dim), red) / (p.heads * p.dim) + p.eps);
+    if (p.kv_heads > 0)
+      k_rs = 1.0f / sqrtf(block_sum(row_squares<T, VEC>(raw + p.koff, p.kv_heads * p.dim), red) /
+                              (p.kv_heads * p.dim) + p.eps);
+  }
   const int v_units = (max(p.vdim_p, p.vr_head) + 8 * L - 1) / (8 * L);     // per head
   const int units = p.heads + p.kv_heads + p.v_heads * v_units;
   for (int u = threadIdx.x / L; u < (units + HP_THREADS / L - 1) / (HP_THREADS / L) * (HP_THREADS / L);
@@ -77,6 +102,14 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
 #pragma unroll
     for (int i = 0; i < 8; ++i) f[i] = 0.f;
     if (live) head_load<T, VEC>(src, d, n, f);
+    const float* gain = is_v || p.q_norm == nullptr ? nullptr : (is_q ? p.q_norm : p.k_norm) + static_cast<size_t>(h) * n;
+    const float row_rs = is_q ? q_rs : k_rs;
+    if (live && gain != nullptr) {
+      float g[8];
+      head_load<float, VEC>(gain, d, n, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] *= row_rs * g[i];
+    }
     if (live && !is_v && d < 2 * p.half) {
       if (p.interleaved) {                        // both numbers of a pair are this lane's
 #pragma unroll
@@ -93,6 +126,12 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
         const int first = low ? d : d - p.half;
         float o[8];
         load_vec<8>(src + (low ? d + p.half : first), o);
+        if (gain != nullptr) {
+          float g[8];
+          load_vec<8>(gain + (low ? d + p.half : first), g);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) o[i] *= row_rs * g[i];
+        }
         const float sign = low ? -1.f : 1.f;
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
@@ -106,19 +145,20 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
           if (c < 2 * p.half) {
             const bool low = c < p.half;
             const float2 cs = rope[low ? c : c - p.half];
-            const float o = to_f32(src[low ? c + p.half : c - p.half]);
+            const int other = low ? c + p.half : c - p.half;
+            const float o = to_f32(src[other]) * (gain != nullptr ? row_rs * gain[other] : 1.f);
             f[i] = f[i] * cs.x + (low ? -o : o) * cs.y;
           }
         }
       }
     }
-    if (p.unit) {
+    if (p.unit || p.unit_v) {
       float s = 0.f;
 #pragma unroll
       for (int i = 0; i < 8; ++i) s += f[i] * f[i];
 #pragma unroll
       for (int o = L / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-      if (!is_v) {
+      if (is_v ? p.unit_v : p.unit) {
         const float r = 1.0f / sqrtf(s / n + p.eps);
 #pragma unroll
         for (int i = 0; i < 8; ++i) f[i] *= r;
@@ -126,6 +166,11 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
     }
     if (!live) continue;
     if (is_q) {
+      if (p.q_factor != nullptr) {
+        const float c = p.q_factor[h];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] *= c;
+      }
       if (d < p.q_head)
         store_vec<8>(static_cast<T*>(p.q) + (static_cast<size_t>(row) * p.heads + h) * p.q_head + d, f);
       continue;
@@ -159,13 +204,14 @@ static int head_prep(const HeadPrep& p, int rows, int widest, cudaStream_t st) {
 
 extern "C" int cb_head_prep(const void* raw, int ld, int koff, int voff, int heads, int kv_heads,
                             int v_heads, int dim, int vdim, int half, const void* rope,
-                            int interleaved, int unit, float eps, void* q, int q_head, void* k_cache,
+                            int interleaved, int unit, float eps, const float* q_norm, const float* k_norm,
+                            int unit_v, const float* q_factor, void* q, int q_head, void* k_cache,
                             void* v_cache, int dim_p, int vdim_p, void* k_rows, void* v_rows,
                             int kr_head, int vr_head, const int* page_table, int max_pages,
                             int num_pages, const int* row_slot, const int* row_pos, int rows, int f32,
                             int* status, void* stream) {
   using namespace cb;
-  if (rows <= 0 || heads < 1 || kv_heads < 1 || v_heads < 1 || dim < 1 || vdim < 1 || half < 0 || 2 * half > dim)
+  if (rows <= 0 || heads < 1 || kv_heads < 0 || (v_heads < 1) != (kv_heads < 1) || dim < 1 || vdim < 1 || half < 0 || 2 * half > dim)
     return -1;
   if (half > 0 && rope == nullptr) return -1;
   if (q_head % 8 || dim_p % 8 || vdim_p % 8 || q_head < dim || dim_p < dim || vdim_p < vdim) return -2;
@@ -174,10 +220,14 @@ extern "C" int cb_head_prep(const void* raw, int ld, int koff, int voff, int hea
   int widest = q_head;
   for (int w : {dim_p, kr_head}) widest = w > widest ? w : widest;
   if (widest > 256 || vdim_p > 256 || vr_head > 256) return -2;
+  if (q_norm != nullptr && kv_heads > 0 && k_norm == nullptr) return -2;
+  if (kv_heads > 0 && unit_v)              // a head of v by one group of lanes
+    for (int w : {vdim_p, vr_head}) widest = w > widest ? w : widest;
   HeadPrep p;
   p.raw = raw; p.ld = ld; p.koff = koff; p.voff = voff; p.heads = heads; p.kv_heads = kv_heads;
   p.v_heads = v_heads; p.dim = dim; p.vdim = vdim; p.half = half; p.rope = static_cast<const float2*>(rope);
-  p.interleaved = interleaved; p.unit = unit; p.eps = eps; p.q = q; p.q_head = q_head; p.k_cache = k_cache;
+  p.interleaved = interleaved; p.unit = unit; p.eps = eps; p.q_norm = q_norm; p.k_norm = k_norm;
+  p.unit_v = kv_heads > 0 && unit_v; p.q_factor = q_factor; p.q = q; p.q_head = q_head; p.k_cache = k_cache;
   p.v_cache = v_cache; p.dim_p = dim_p; p.vdim_p = vdim_p; p.k_rows = k_rows; p.v_rows = v_rows;
   p.kr_head = kr_head; p.vr_head = vr_head; p.page_table = page_table; p.max_pages = max_pages;
   p.num_pages = num_pages; p.row_slot = row_slot; p.row_pos = row_pos; p.status = status;

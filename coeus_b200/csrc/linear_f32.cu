@@ -11,7 +11,7 @@ enum : int { ACT_NONE = 0, ACT_RELU2 = 4, ACT_SOFTCAP = 5, ACT_GELU_ERF = 6, ACT
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw,
                   const float* __restrict__ bias, float* __restrict__ y, int ldy, int M, int N,
-                  int K, int act, float act_arg, float limit, int accumulate,
+                  int K, int act, float act_arg, float limit, float shift, int accumulate,
                   const int* __restrict__ block_expert, int block_rows) {
   __shared__ float sx[LK][LT + 4], sw[LK][LT + 4];
   const int m0 = blockIdx.y * LT, n0 = blockIdx.x * LT;
@@ -53,8 +53,9 @@ linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict_
       for (int j = 0; j < 4; j += 2) {
         const int n = n0 + tx * 4 + j;
         if (n >= N) continue;
-        const float g = fminf(acc[i][j], limit), u = fminf(fmaxf(acc[i][j + 1], -limit), limit);
-        y[static_cast<size_t>(m) * ldy + n / 2] = g * (u + 1.0f) / (1.0f + expf(-act_arg * g));
+        const float g = fminf(acc[i][j] + (bias != nullptr ? bias[n] : 0.f), limit);
+        const float u = fminf(fmaxf(acc[i][j + 1] + (bias != nullptr ? bias[n + 1] : 0.f), -limit), limit);
+        y[static_cast<size_t>(m) * ldy + n / 2] = g * (u + shift) / (1.0f + expf(-act_arg * g));
       }
       continue;
     }
@@ -87,21 +88,21 @@ extern "C" int cb_linear_f32(const float* x, int ldx, const float* w, int ldw,
   dim3 grid((N + cb::LT - 1) / cb::LT, (M + cb::LT - 1) / cb::LT);
   if (grid.y > 65535) return -1;
   cb::linear_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      x, ldx, w, ldw, bias, y, ldy, M, N, K, act, act_arg, 0.f, accumulate, nullptr, 0);
+      x, ldx, w, ldw, bias, y, ldy, M, N, K, act, act_arg, 0.f, 0.f, accumulate, nullptr, 0);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
 // block_expert[b]: which of the weights [experts, N, K] block b of block_rows (a multiple of 64) rows takes
 // (-1: none, they are left alone); null: one weight.  glu: alternating columns g, u make one (clamped_glu).
-extern "C" int cb_linear_f32_grouped(const float* x, int ldx, const float* w, int ldw,
+extern "C" int cb_linear_f32_grouped(const float* x, int ldx, const float* w, int ldw, const float* bias,
                                      const int* block_expert, int block_rows, float* y, int ldy, int M, int N, int K,
-                                     int glu, float slope, float limit, void* stream) {
+                                     int glu, float slope, float limit, float shift, void* stream) {
   if (M <= 0 || N <= 0 || K <= 0 || K % 4 || ldx % 4 || ldw % 4 || (glu && N % 2)) return -1;
   if (block_expert != nullptr && (block_rows < cb::LT || block_rows % cb::LT || M % block_rows)) return -1;
   dim3 grid((N + cb::LT - 1) / cb::LT, (M + cb::LT - 1) / cb::LT);
   if (grid.y > 65535) return -1;
   cb::linear_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      x, ldx, w, ldw, nullptr, y, ldy, M, N, K, glu ? cb::ACT_GLU : cb::ACT_NONE, slope, limit, 0, block_expert,
+      x, ldx, w, ldw, bias, y, ldy, M, N, K, glu ? cb::ACT_GLU : cb::ACT_NONE, slope, limit, shift, 0, block_expert,
       block_rows);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

@@ -9,7 +9,7 @@
 
 namespace cb {
 
-enum : int { SK_NONE = 0, SK_RELU2 = 4, SK_SOFTCAP = 5, SK_GELU_ERF = 6 };
+enum : int { SK_NONE = 0, SK_RELU2 = 4, SK_SOFTCAP = 5, SK_GELU_ERF = 6, SK_GLU = 7 };
 
 struct SkinnyProblem {
   const __nv_bfloat16* x;   // [M, ldx]
@@ -17,7 +17,8 @@ struct SkinnyProblem {
   const __nv_bfloat16* bias;   // [N] or null
   void* y;                  // [M, ldy] bf16 or fp32
   int ldx, ldw, ldy, N, K, act, f32, accumulate;
-  float act_arg;
+  float act_arg;            // the cap, or of a gated unit the slope
+  float limit, shift;       // SK_GLU: rows of w alternate, y [M, N / 2] (clamped_glu)
 };
 struct SkinnyArgs {
   SkinnyProblem p[2];
@@ -112,6 +113,25 @@ __global__ void __launch_bounds__(WARPS * 32) linear_skinny_kernel(const SkinnyA
       for (int k = 0; k < 4; ++k)
         mine[(j * 8 + t * 2 + (k & 1)) * LD + i * 16 + r + (k >> 1) * 8] = acc[i][j][k];
   __syncthreads();
+  if (p.act == SK_GLU) {
+    for (int i = threadIdx.x; i < args.M * MW * 8; i += WARPS * 32) {
+      const int m = i / (MW * 8), c = i % (MW * 8) * 2, n = n0 + c;
+      if (n >= p.N) continue;
+      float g = 0.f, u = 0.f;
+#pragma unroll
+      for (int w = 0; w < WARPS; ++w) {
+        g += red[(w * NT * 8 + m) * LD + c];
+        u += red[(w * NT * 8 + m) * LD + c + 1];
+      }
+      if (p.bias != nullptr) {
+        g += __bfloat162float(p.bias[n]);
+        u += __bfloat162float(p.bias[n + 1]);
+      }
+      static_cast<__nv_bfloat16*>(p.y)[static_cast<size_t>(m) * p.ldy + n / 2] =
+          __float2bfloat16(clamped_glu(g, u, p.act_arg, p.limit, p.shift));
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < args.M * MW * 16; i += WARPS * 32) {
     const int m = i / (MW * 16), c = i % (MW * 16), n = n0 + c;
     if (n >= p.N) continue;
@@ -169,6 +189,26 @@ static int skinny_problem(SkinnyProblem& p, const void* x, int ldx, const void* 
   return 0;
 }
 
+static int launch_skinny_m(const SkinnyArgs& a, int count, int K, cudaStream_t st) {
+  const bool deep = K >= 4096 && count == 1;
+  if (a.M <= 8) return deep ? launch_skinny<1, 1, 16>(a, count, st) : launch_skinny<1, 1, 8>(a, count, st);
+  return deep ? launch_skinny<1, 2, 16>(a, count, st) : launch_skinny<1, 2, 8>(a, count, st);
+}
+
+// y [M, N / 2]: a gated unit (see clamped_glu) over alternating rows of w, after the bias [N] (null: none).
+extern "C" int cb_linear_skinny_glu(const void* x, int ldx, const void* w, int ldw, const void* bias, void* y,
+                                    int ldy, int N, int K, float slope, float limit, float shift, int M,
+                                    void* stream) {
+  if (M <= 0 || M > 16 || N % 2) return -1;
+  SkinnyArgs a = {};
+  a.M = M;
+  const int rc = skinny_problem(a.p[0], x, ldx, w, ldw, bias, y, ldy, N, K, SK_GLU, slope, 0, 0);
+  if (rc != 0) return rc;
+  a.p[0].limit = limit;
+  a.p[0].shift = shift;
+  return launch_skinny_m(a, 1, K, static_cast<cudaStream_t>(stream));
+}
+
 // The second problem is skipped when x1 is null.
 extern "C" int cb_linear_skinny(const void* x0, int ldx0, const void* w0, int ldw0,
                                 const void* b0, void* y0, int ldy0, int N0, int K0, int act0, float arg0, int f32_0, int acc0,
@@ -186,8 +226,5 @@ extern "C" int cb_linear_skinny(const void* x0, int ldx0, const void* w0, int ld
     if (rc != 0) return rc;
     count = 2;
   }
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool deep = K0 >= 4096 && count == 1;
-  if (M <= 8) return deep ? launch_skinny<1, 1, 16>(a, count, st) : launch_skinny<1, 1, 8>(a, count, st);
-  return deep ? launch_skinny<1, 2, 16>(a, count, st) : launch_skinny<1, 2, 8>(a, count, st);
+  return launch_skinny_m(a, count, K0, static_cast<cudaStream_t>(stream));
 }

@@ -1,6 +1,6 @@
 // Attention of a ragged batch over the paged cache: every query row sits at its own position of
 // its own sequence and sees the cached keys of its chunk or its sliding window up to itself (both 0: all
-// of them).  Scores may be capped (s -> cap tanh(s / cap)), the softmax may have a sink per head (a logit
+// of them), and with a window the sequence's first `keep` positions.  Scores may be capped (s -> cap tanh(s / cap)), the softmax may have a sink per head (a logit
 // in the denominator only) and the head's output a gate (a sigmoid of a projected number, one per head or
 // one per number).  Query head h reads key/value head h / (heads / kv_heads); query/key width and value
 // width are independent.
@@ -24,7 +24,7 @@ namespace cb {
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct RaggedSpec {        // as the host gives it
-  int heads, kv_heads, dim, vdim, dim_p, vdim_p, chunk, window, maps, gate_wide;
+  int heads, kv_heads, dim, vdim, dim_p, vdim_p, chunk, window, keep, maps, gate_wide;
   float scale, softcap, map_factor, eps;
 };
 
@@ -37,7 +37,7 @@ struct RaggedAttn {
   int max_pages, num_pages;
   int heads, kv_heads, dim, vdim, dim_p, vdim_p;    // heads: of all maps
   int maps, kdim;          // kdim = maps * dim_p
-  int chunk, window;
+  int chunk, window, keep;
   float scale;             // products to units of log2, or with a cap to the tanh's argument
   float cap;               // 0, or the cap in units of log2
   const float* sink;       // [heads] or null
@@ -55,6 +55,13 @@ __device__ __forceinline__ int first_seen(const RaggedAttn& p, int pos) {
   if (p.window > 0) return max(0, pos + 1 - p.window);
   return p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
 }
+// The keys that position pos sees, counted 0 .. n - 1: the kept positions below its window, then the window.
+struct Seen {
+  int lo, kept, n;
+  __device__ __forceinline__ Seen(const RaggedAttn& p, int pos)
+      : lo(first_seen(p, pos)), kept(min(p.keep, lo)), n(pos + 1 - lo + kept) {}
+  __device__ __forceinline__ int place(int i) const { return i < kept ? i : i - kept + lo; }
+};
 template <typename T>
 __device__ __forceinline__ float exp2_t(float x) {
   if constexpr (sizeof(T) == 4) return exp2f(x);
@@ -121,9 +128,9 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
     sq[g][d] = (g < ng && c >= 0 && c < p.dim) ? to_f32(qp[(h0 + g) * p.q_head + c]) * p.scale : 0.f;
   }
   __syncthreads();
-  const int lo = first_seen(p, pos), n = pos + 1 - lo;
-  const int piece = (n + ra.splits - 1) / ra.splits;
-  const int t0 = lo + split * piece, t1 = min(pos + 1, t0 + piece);
+  const Seen seen(p, pos);
+  const int piece = (seen.n + ra.splits - 1) / ra.splits;
+  const int t0 = split * piece, t1 = min(seen.n, t0 + piece);
   const T* kc = static_cast<const T*>(p.k_cache);
   const T* vc = static_cast<const T*>(p.v_cache);
   const int nchunk = p.vdim_p / 8, ngroups = 32 / nchunk;
@@ -141,7 +148,7 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
     const int my_t = tb + lane;
     int my_page = 0;
     if (my_t < t1) {
-      const int lp = my_t / RAGGED_PAGE;
+      const int lp = seen.place(my_t) / RAGGED_PAGE;
       my_page = lp < p.max_pages ? pt[lp] : -1;
       if (my_page < 0 || my_page >= p.num_pages) {
         record_status(p.status, ST_BOUNDS, row);
@@ -156,7 +163,7 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
 #pragma unroll
       for (int g = 0; g < GM; ++g) s[g] = 0.f;
       if (t < t1) {
-        const T* kp = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + t % RAGGED_PAGE) * p.kv_heads + hk) * p.kdim;
+        const T* kp = kc + ((static_cast<size_t>(page) * RAGGED_PAGE + seen.place(t) % RAGGED_PAGE) * p.kv_heads + hk) * p.kdim;
 #pragma unroll
         for (int c = 0; c < KIT; ++c) {
           const int d = ((lane & 7) + 8 * c) * 8;
@@ -202,7 +209,7 @@ __global__ void __launch_bounds__(RA_WARPS * 32) ragged_attn_rows_kernel(const R
       const int key = k0 + kg, t = tb + key;
       const int page = __shfl_sync(0xffffffffu, my_page, key & 31);
       if (kg < ngroups && key < nk) {
-        const T* vp = vc + ((static_cast<size_t>(page) * RAGGED_PAGE + t % RAGGED_PAGE) * p.kv_heads + hk) * p.vdim_p;
+        const T* vp = vc + ((static_cast<size_t>(page) * RAGGED_PAGE + seen.place(t) % RAGGED_PAGE) * p.kv_heads + hk) * p.vdim_p;
         float f[8];
         load_vec<8>(vp + vch * 8, f);
 #pragma unroll
@@ -387,7 +394,10 @@ __global__ void __launch_bounds__(MAPS * TA_WARPS * 32) ragged_attn_tiles_kernel
   for (int i = tid; i < 2 * RAGGED_PAGE * (VS - p.vdim_p); i += NT)
     sV[(i / (VS - p.vdim_p)) * VS + p.vdim_p + i % (VS - p.vdim_p)] = __float2bfloat16(0.f);
   const int last = pos0 + len - 1;
+  // pages of kept positions, then those from the first row's window on
   const int pg0 = first_seen(p, pos0) / RAGGED_PAGE, pg1 = last / RAGGED_PAGE;
+  const int kp = min(pg0, (p.keep + RAGGED_PAGE - 1) / RAGGED_PAGE), n_pages = kp + pg1 - pg0 + 1;
+  auto page_at = [&](int i) { return i < kp ? i : pg0 + i - kp; };
   auto fetch = [&](int pg, int st) {
     int page = pg < p.max_pages ? pt[pg] : -1;
     if (page < 0 || page >= p.num_pages) {
@@ -409,7 +419,7 @@ __global__ void __launch_bounds__(MAPS * TA_WARPS * 32) ragged_attn_tiles_kernel
     }
     cp_async_commit();
   };
-  fetch(pg0, 0);
+  fetch(page_at(0), 0);
   if (p.dim % 8 == 0 && p.q_head % 8 == 0) {
     for (int i = tid; i < TA_ROWS * MAPS * (DC / 8); i += NT) {
       const int t = i / (MAPS * (DC / 8)), x = i % (MAPS * (DC / 8)), m = x / (DC / 8), c = x % (DC / 8) * 8;
@@ -441,17 +451,18 @@ __global__ void __launch_bounds__(MAPS * TA_WARPS * 32) ragged_attn_tiles_kernel
   const int qpos[2] = {pos0 + r0, pos0 + r0 + 8};
   const int qlo[2] = {first_seen(p, qpos[0]), first_seen(p, qpos[1])};
   const int w_first = pos0 + warp * 16, w_last = min(w_first + 15, last);
-  for (int pg = pg0; pg <= pg1; ++pg) {
-    const int st = (pg - pg0) & 1, base = pg * RAGGED_PAGE;
-    if (pg < pg1) {
-      fetch(pg + 1, st ^ 1);
+  for (int i_pg = 0; i_pg < n_pages; ++i_pg) {
+    const int st = i_pg & 1, base = page_at(i_pg) * RAGGED_PAGE;
+    if (i_pg + 1 < n_pages) {
+      fetch(page_at(i_pg + 1), st ^ 1);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
     __syncthreads();
     // skip pages that no row of this warp sees
-    if (w_first <= last && base <= w_last && base + RAGGED_PAGE > first_seen(p, w_first)) {
+    if (w_first <= last && base <= w_last &&
+        (base + RAGGED_PAGE > first_seen(p, w_first) || base < p.keep)) {
       float s[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i)
@@ -468,14 +479,15 @@ __global__ void __launch_bounds__(MAPS * TA_WARPS * 32) ragged_attn_tiles_kernel
           mma_bf16(s[2 * i + 1], qf[k], b[2], b[3]);
         }
       }
-      const bool full = base >= first_seen(p, w_last) && base + RAGGED_PAGE - 1 <= w_first;
+      const bool full = (base >= first_seen(p, w_last) || base + RAGGED_PAGE <= p.keep) &&
+                        base + RAGGED_PAGE - 1 <= w_first;
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int i = 0; i < 8; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int r = j >> 1, t = base + i * 8 + (lane & 3) * 2 + (j & 1);
-          s[i][j] = (full || (t <= qpos[r] && t >= qlo[r])) ? score_of<bf16>(p, s[i][j] * p.scale) : -INFINITY;
+          s[i][j] = (full || (t <= qpos[r] && (t >= qlo[r] || t < p.keep))) ? score_of<bf16>(p, s[i][j] * p.scale) : -INFINITY;
           mx[r] = fmaxf(mx[r], s[i][j]);
         }
       float c[2], sum[2] = {0.f, 0.f};
@@ -626,9 +638,9 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
   const int* pt = p.page_table + static_cast<size_t>(slot) * p.max_pages;
   const bf16* kc = static_cast<const bf16*>(p.k_cache) + hk * p.kdim;
   const bf16* vc = static_cast<const bf16*>(p.v_cache) + hk * p.vdim_p;
-  const int lo = first_seen(p, pos), n = pos + 1 - lo;
-  const int piece = (n + ra.splits - 1) / ra.splits;
-  const int t0 = lo + split * piece, t1 = min(pos + 1, t0 + piece);
+  const Seen seen(p, pos);
+  const int piece = (seen.n + ra.splits - 1) / ra.splits;
+  const int t0 = split * piece, t1 = min(seen.n, t0 + piece);
   bf16* mine = ring + warp * 2 * STAGE;
   const int kch = p.kdim / 8, vch = p.vdim_p / 8;
   // rows of nch vectors of eight, one per key (cell), to shared memory
@@ -650,10 +662,9 @@ __global__ void __launch_bounds__(GA_WARPS * 32) ragged_attn_group_kernel(const 
     }
   };
   auto fetch = [&](int tb, int st) {                    // keys tb .. tb + 31 into a stage
-    const int t = tb + lane;
     int cell = 0;
-    if (t < t1) {
-      const int lp = t / RAGGED_PAGE;
+    if (tb + lane < t1) {
+      const int t = seen.place(tb + lane), lp = t / RAGGED_PAGE;
       int page = lp < p.max_pages ? pt[lp] : -1;
       if (page < 0 || page >= p.num_pages) {
         record_status(p.status, ST_BOUNDS, row);
@@ -906,13 +917,13 @@ static int fill_attn(RaggedAttn& p, const void* q, int q_head, const void* k_cac
       c.vdim_p > 256)
     return -2;
   if (c.maps == 2 && sink != nullptr) return -2;
-  if ((c.maps != 1 && c.maps != 2) || (c.maps == 2 && map_weight == nullptr) || c.window < 0 || c.chunk < 0 ||
+  if ((c.maps != 1 && c.maps != 2) || (c.maps == 2 && map_weight == nullptr) || c.window < 0 || c.chunk < 0 || c.keep < 0 ||
       (c.window > 0 && c.chunk > 0) || c.softcap < 0.f)
     return -2;
   p.q = q; p.q_head = q_head; p.k_cache = k_cache; p.v_cache = v_cache; p.page_table = page_table;
   p.max_pages = max_pages; p.num_pages = num_pages; p.heads = c.heads * c.maps; p.kv_heads = c.kv_heads;
   p.dim = c.dim; p.vdim = c.vdim; p.dim_p = c.dim_p; p.vdim_p = c.vdim_p; p.maps = c.maps;
-  p.kdim = c.maps * c.dim_p; p.chunk = c.chunk; p.window = c.window;
+  p.kdim = c.maps * c.dim_p; p.chunk = c.chunk; p.window = c.window; p.keep = c.window > 0 ? c.keep : 0;
   p.scale = c.softcap > 0.f ? c.scale / c.softcap : c.scale * LOG2E;
   p.cap = c.softcap * LOG2E;
   p.sink = sink; p.gate = gate; p.ldg = ldg; p.gate_wide = c.gate_wide; p.map_weight = map_weight;

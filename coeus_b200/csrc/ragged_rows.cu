@@ -8,11 +8,11 @@ namespace cb {
 
 constexpr int ROW_THREADS = 256;
 
-// out row r: rms_norm(embed[tokens[r]]) * w, fp32; columns width .. ld-1 are zero.
+// out row r: rms_norm(embed[tokens[r]]) * w * scale (without w: embed[tokens[r]] * scale), fp32; columns width .. ld-1 are zero.
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS)
 embed_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ embed, int lde, int vocab,
-                  const float* __restrict__ w, float* __restrict__ x, int ld, int width, float eps,
+                  const float* __restrict__ w, float* __restrict__ x, int ld, int width, float eps, float scale,
                   int* status) {
   __shared__ float red[32];
   const int r = blockIdx.x;
@@ -34,7 +34,7 @@ embed_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ embed, i
     float v = 0.f;
     if (c < width) {
       v = to_f32(src[c]);
-      v = w != nullptr ? v * rs * w[c] : v;
+      v = (w != nullptr ? v * rs * w[c] : v) * scale;
     }
     dst[c] = v;
   }
@@ -196,16 +196,16 @@ using namespace cb;
 #define CB_RC() (cudaGetLastError() == cudaSuccess ? 0 : -3)
 
 extern "C" int cb_embed_norm(const int* tokens, const void* embed, int lde, int vocab,
-                             const float* w, float* x, int ld, int rows, int width, float eps,
+                             const float* w, float* x, int ld, int rows, int width, float eps, float scale,
                              int f32, int* status, void* stream) {
   if (rows <= 0 || width > ld || width > lde) return -1;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     embed_norm_kernel<float><<<rows, ROW_THREADS, 0, st>>>(
-        tokens, static_cast<const float*>(embed), lde, vocab, w, x, ld, width, eps, status);
+        tokens, static_cast<const float*>(embed), lde, vocab, w, x, ld, width, eps, scale, status);
   else
     embed_norm_kernel<__nv_bfloat16><<<rows, ROW_THREADS, 0, st>>>(
-        tokens, static_cast<const __nv_bfloat16*>(embed), lde, vocab, w, x, ld, width, eps, status);
+        tokens, static_cast<const __nv_bfloat16*>(embed), lde, vocab, w, x, ld, width, eps, scale, status);
   return CB_RC();
 }
 

@@ -10,6 +10,7 @@ are kept on top of it.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Dict, List, Optional
 
 import numpy as np
@@ -34,6 +35,16 @@ def _up8(n: int) -> int:
     return (n + 7) // 8 * 8
 
 
+@dataclass
+class _KvRows:
+    """Row-wise keys and values of a layer in one step: the step's rows, then cached ones gathered for the
+    pieces of one plan."""
+
+    k: Optional[torch.Tensor] = None
+    v: Optional[torch.Tensor] = None
+    gathered: Optional[R.AttnPlan] = None
+
+
 class HybridEngine(InferenceEngine):
     ragged = True
     prefill_tokens = 16384       # rows of one step when a prompt batch is cut by generate()
@@ -51,6 +62,10 @@ class HybridEngine(InferenceEngine):
         self._graphs: Dict[int, tuple] = {}
         self._tiles = model.device.type == "cuda" and model.dtype == torch.bfloat16
         self._runs = self.cfg.runs()
+        self._shared: Dict[int, List[int]] = {}     # layer -> the later layers that use its keys and values
+        for i, layer in enumerate(self.cfg.layers):
+            if getattr(layer.mixer, "kv_from", None) is not None:
+                self._shared.setdefault(layer.mixer.kv_from, []).append(i)
         self._plans = [self._plan(layer.mixer) for layer in self.cfg.layers
                        if isinstance(layer.mixer, CACHED)]
         self._plans += [RC.ssd_plan(a.heads, a.vdim, a.state) for a in
@@ -61,8 +76,9 @@ class HybridEngine(InferenceEngine):
             return R.AttnPlan(a.chunk, self._tiles and R.pieces_allowed(a.dim, a.vdim, a.chunk, a.scale))
         if isinstance(a, HeadAttentionSpec):
             plain = a.maps == 1 or (a.softcap is None and not a.gated)
+            plain &= not a.keep_first or (a.maps == 1 and a.softcap is None)
             return R.AttnPlan(None, self._tiles and plain and R.pieces_allowed(a.dim, a.vdim, None, a.scale),
-                              a.window, tiles=a.maps * a.dim <= 256)
+                              a.window, tiles=a.maps * a.dim <= 256, keep=a.keep_first)
         return R.AttnPlan(None, self._tiles and L.pieces_allowed(a.dim + a.rot_dim, a.vdim, a.scale),
                           a.window or 1 << 30, tiles=False)
 
@@ -82,7 +98,9 @@ class HybridEngine(InferenceEngine):
         self._cache_index: Dict[int, int] = {}
         for n, run in enumerate(self._runs):
             a = m.layers[run.layer].spec.mixer
-            if isinstance(a, CACHED):
+            if getattr(a, "kv_from", None) is not None:        # without a loop runs are layers
+                self._cache_index[n] = self._cache_index[a.kv_from]
+            elif isinstance(a, CACHED):
                 self._cache_index[n] = len(dims)
                 if isinstance(a, LatentAttentionSpec):
                     dims.append((1, _up8(a.latent), 0))
@@ -105,6 +123,8 @@ class HybridEngine(InferenceEngine):
                 self.state.add(n, "gru", (_up8(s.width),), torch.float32)
             if layer.shift is not None:
                 self.state.add(n, "before", (self.cfg.width_padded,), torch.float32)
+            if layer.taps is not None:
+                self.state.add(n, "before", (layer.taps.shape[0] - 1, self.cfg.width_padded), torch.float32)
         self._graphs.clear()
         return self.cache
 
@@ -171,42 +191,57 @@ class HybridEngine(InferenceEngine):
                max_ctx: int) -> None:
         s, c, i = layer.spec.mixer, self.cache, self._cache_index[n]
         eps, plan, kh = self.cfg.norm_eps, self._plan(s), s.kv_heads * s.maps
-        key_rows, k_rows, v_rows, q_head = b.kv_rows(plan), None, None, None
-        if key_rows:        # the heads' distance in the row-wise buffers of the piece kernel
-            q_head, v_head = R.row_heads(s.dim, s.vdim, s.maps)
-            k_rows, v_rows = (torch.empty((key_rows, h, p), dtype=raw.dtype, device=raw.device)
-                              for h, p in ((kh, q_head), (s.kv_heads, v_head)))
-        q = R.head_prep(raw, layer.seg["k"], layer.seg["v"], s.heads * s.maps, kh, s.dim, s.vdim, b,
-                        rope.get(layer.rope_key), c.k[i], c.v[i], c.page_table, interleaved=s.interleaved,
-                        unit_eps=eps if s.unit_qk else None, q_head=q_head, k_rows=k_rows, v_rows=v_rows)
+        own, rows = s.kv_from is None, _KvRows()
+        if not own:
+            rows = b.kept[s.kv_from]
+        else:       # row-wise keys and values for the piece kernel, of this layer and those that use them too
+            users = [plan] + [self._plan(self.cfg.layers[j].mixer) for j in self._shared.get(n, ())]
+            size = max(b.kv_rows(p) for p in users)
+            if size:        # heads at the distance that the piece kernel has
+                q_head, v_head = R.row_heads(s.dim, s.vdim, s.maps)
+                rows = _KvRows(*(torch.empty((size, h, p), dtype=raw.dtype, device=raw.device)
+                                 for h, p in ((kh, q_head), (s.kv_heads, v_head))))
+            if n in self._shared:
+                b.kept[n] = rows
+        pieces = b.kv_rows(plan) > 0
+        q = R.head_prep(raw, layer.seg.get("k", 0), layer.seg.get("v", 0), s.heads * s.maps, kh if own else 0,
+                        s.dim, s.vdim, b, rope.get(layer.rope_key), c.k[i], c.v[i], c.page_table,
+                        interleaved=s.interleaved, unit_eps=eps if s.unit_qk else None,
+                        q_head=rows.k.shape[2] if pieces else None, k_rows=rows.k if own else None,
+                        v_rows=rows.v if own else None, eps=eps, q_norm=layer.q_norm, k_norm=layer.k_norm,
+                        unit_v=s.unit_v, q_factor=layer.temp)
         R.ragged_attention(
             q, c.k[i], c.v[i], c.page_table, b, s.heads, s.kv_heads, s.dim, s.vdim, s.scale,
-            out[:, :layer.out_dim], window=s.window, softcap=s.softcap, score_max=s.score_max, maps=s.maps,
-            map_weight=layer.map_weight, map_factor=1.0 - s.diff if s.maps == 2 else 1.0, eps=eps,
-            gate=raw[:, layer.seg["g"]:] if s.gated else None, gate_wide=True, max_ctx=max_ctx,
-            k_rows=k_rows, v_rows=v_rows, plan=plan)
+            out[:, :layer.out_dim], window=s.window, keep=s.keep_first, softcap=s.softcap, score_max=s.score_max,
+            maps=s.maps, map_weight=layer.map_weight, map_factor=1.0 - s.diff if s.maps == 2 else 1.0, eps=eps,
+            sink=layer.sink, gate=raw[:, layer.seg["g"]:] if s.gated else None, gate_wide=True, max_ctx=max_ctx,
+            k_rows=rows.k if pieces else None, v_rows=rows.v if pieces else None, plan=plan,
+            gathered=rows.gathered == plan)
+        if pieces:
+            rows.gathered = plan
 
     def _experts(self, layer, h: torch.Tensor) -> dict:
         """The mixture of experts of ``h``, as what the next pass over the stream adds."""
         e, m = layer.experts, layer.experts.spec
-        r = X.Routing(m.experts, m.top, m.groups, m.keep, m.scale)
-        c = X.route(h, e.router, r)
+        r = e.routing
+        c = X.route(h, e.router, r, e.correction)
         shared = m.shared is not None
         if h.is_cuda and h.dtype == torch.bfloat16 and h.shape[0] <= X.FEW:
             return dict(y=X.experts_few(h, c, r, e.w_in, e.w_down, m.expert.limit, e.s_in, e.s_down,
-                                        m.shared.limit if shared else 0.0, e.slope))
+                                        m.shared.limit if shared else 0.0, e.slope, e.shift))
 
         def rows(n, w):
             return torch.empty((n, w), dtype=h.dtype, device=h.device)
         s = X.sort_rows(h, c, r)
         n = s.rows.shape[0]
         act = X.grouped_linear(s.rows, e.w_in, s.block_expert, rows(n, e.w_in.shape[1] // 2),
-                               glu=(e.slope, m.expert.limit))
+                               glu=(e.slope, m.expert.limit, e.shift))
         res = X.grouped_linear(act, e.w_down, s.block_expert, rows(n, e.wp))
-        add = dict(spread=R.Spread(res, s.slot, c.weight))
+        add = dict(spread=R.Spread(res, s.slot, c.weight, h if m.identity else None))
         if shared:
-            act = G.linear(h, e.s_in, rows(h.shape[0], e.s_in.shape[0] // 2), glu=(e.slope, m.shared.limit))
-            add["y"] = self._product(act, e.s_down)
+            act = G.linear(h, e.s_in, rows(h.shape[0], e.s_in.shape[0] // 2),
+                           glu=(e.slope, m.shared.limit, e.shift))
+            add.update(y=self._product(act, e.s_down), y_weight=c.shared)
         return add
 
     def _latent(self, n: int, layer, raw: torch.Tensor, out: torch.Tensor, b: R.RaggedBatch,
@@ -268,7 +303,7 @@ class HybridEngine(InferenceEngine):
         m, cfg = self.m, self.cfg
         rope = {k: R.rope_table(b.pos, f) for k, f in m.inv_freq.items()}
         x = torch.empty((b.T, cfg.width_padded), dtype=torch.float32, device=m.device)
-        R.embed_norm(b.tokens, m.embed, m.embed_norm, cfg.hidden_dim, cfg.norm_eps, x)
+        R.embed_norm(b.tokens, m.embed, m.embed_norm, cfg.hidden_dim, cfg.norm_eps, x, cfg.embed_scale)
         blocks = self._parallel if cfg.design.parallel else self._sequential
         xf = blocks(x, b, rope, max_ctx, layer_out)
         if xf is None:
@@ -312,9 +347,10 @@ class HybridEngine(InferenceEngine):
             if run.starts is not None:
                 R.add_norm(x, W, eps, dt, casts=[both[:, :wp]], keep=False, **add)
                 x, add = None, dict(y=self._product(both, m.loop_in), bias=m.loop_step[run.starts])
-            shift = {} if layer.shift is None else dict(shift=layer.shift, before=self.state[n, "before"],
-                                                        batch=b)
-            x, h = R.add_norm(x, W, eps, dt, gain=layer.norm1, **shift, **add)
+            back = {}                      # what the mixer reads of earlier tokens' h
+            if layer.shift is not None or layer.taps is not None:
+                back = dict(shift=layer.shift, taps=layer.taps, before=self.state[n, "before"], batch=b)
+            x, h = R.add_norm(x, W, eps, dt, gain=layer.norm1, center=layer.center1, **back, **add)
             raw = torch.empty((b.T, layer.w_in.shape[0]), dtype=dt, device=m.device)
             G.linear(h, layer.w_in, raw, bias=layer.b_in)
             out = torch.empty((b.T, layer.act_off), dtype=dt, device=m.device)
@@ -325,21 +361,22 @@ class HybridEngine(InferenceEngine):
                 mix(n, layer, raw, out, b, rope, max_ctx)
             else:
                 {"mamba2": self._mamba2, "mingru": self._mingru}[layer.spec.mixer.kind](n, layer, raw, out, b)
-            add = dict(y=self._product(out, layer.w_out), post=layer.norm1b)
+            add = dict(y=self._product(out, layer.w_out), post=layer.norm1b, scale=layer.scale1)
+            if layer.norm2 is not None:
+                x, h = R.add_norm(x, W, eps, dt, gain=layer.norm2, center=layer.center2, **add)
             if layer.experts is not None:
-                x, h = R.add_norm(x, W, eps, dt, gain=layer.norm2, **add)
-                add = dict(post=layer.norm2b, **self._experts(layer, h))
+                add = dict(post=layer.norm2b, scale=layer.scale2, **self._experts(layer, h))
             elif layer.w_up is not None:
-                x, h = R.add_norm(x, W, eps, dt, gain=layer.norm2, **add)
                 act = torch.empty((b.T, layer.ff_padded), dtype=dt, device=m.device)
-                G.linear(h, layer.w_up, act, epi=cfg.design.act, bias=layer.b_up)
-                add = dict(y=self._product(act, layer.w_down), bias=layer.b_down, post=layer.norm2b)
+                G.linear(h, layer.w_up, act, epi=cfg.design.act, bias=layer.b_up, glu=layer.glu)
+                add = dict(y=self._product(act, layer.w_down), bias=layer.b_down, post=layer.norm2b,
+                           scale=layer.scale2)
             if layer_out is not None:
                 x, add = R.add_norm(x, W, eps, dt, **add)[0], {}
                 layer_out.append(x[:, :W].clone())
         if not b.n_want:
             return None
-        return R.add_norm(x, W, eps, dt, gain=m.final_gain, rows=b.want, **add)[1]
+        return R.add_norm(x, W, eps, dt, gain=m.final_gain, center=m.final_center, rows=b.want, **add)[1]
 
     def step(self, entries: List[Entry], layer_out: Optional[list] = None
              ) -> Optional[torch.Tensor]:

@@ -16,9 +16,14 @@ What a design fixes for all its models is a :class:`Design`; the mixers are open
 * Rupasun: norms before and after each sublayer, differential attention over the whole context,
   attention under a sliding window with normalised queries and keys, capped scores and an output
   gate, and feed-forwards that are dense or a mixture of experts with a shared one.
+* Dogilorn: layer norms in front of each sublayer and layer scales behind it, a short convolution in
+  front of every mixer, attention under a sliding window that keeps the first tokens, whose keys and
+  values layers can share, and feed-forwards that are a bounded gated unit or a mixture of experts among
+  which some pass their input on.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Any, ClassVar, Dict, List, Mapping, NamedTuple, Optional, Tuple, Union
 
@@ -30,6 +35,7 @@ MAX_HEAD_DIM = 256           # the attention and recurrence kernels' limit per h
 MAX_LATENT = 640             # and per cached latent row
 MAX_TAPS = 17                # and of the convolution kernels
 MAX_WIDTH = 16384            # and of the pass between two sublayers
+MAX_HISTORY = 52 * 1024      # numbers of earlier tokens that this pass keeps for its convolution
 MAX_EXPERTS, MAX_TOP = 256, 16   # and of the routing kernels
 DEFAULT_MAX_SEQ_LEN = 8192   # serving default; the designs themselves have no length limit
 
@@ -49,9 +55,13 @@ class Design:
     token_shift: bool
     act: str                 # of the dense feed-forward
     mlp_bias: bool
-    mlps: Tuple[str, ...] = ("dense",)
-    glu_slope: float = 1.0   # of the sigmoid in the experts' gated unit
+    mlps: Mapping[str, str] = field(default_factory=lambda: _same("dense"))   # name in a file -> kind
     scaled_logits: bool = False
+    layer_norms: bool = False     # norms of the stream subtract the mean and have a bias
+    layer_scale: bool = False     # sublayer results times a vector
+    input_conv: bool = False      # a mixer reads h + conv(h)
+    scaled_embed: bool = False
+    tied_head: bool = False       # the logits' matrix is the embedding table
 
 
 def _same(*kinds: str) -> Dict[str, str]:
@@ -66,7 +76,11 @@ DESIGNS = {d.name: d for d in (
            scaled_logits=True),
     Design("Rupasun", {"attention": "diff_attention", "attention_2": "capped_attention"}, parallel=False,
            post_norms=True, scalar_norms=False, embed_norm=False, token_shift=False, act="relu2",
-           mlp_bias=False, mlps=("dense", "moe"), glu_slope=1.702),
+           mlp_bias=False, mlps=_same("dense", "moe")),
+    Design("Dogilorn", {"attention": "kept_window_attention"}, parallel=False, post_norms=False,
+           scalar_norms=False, embed_norm=False, token_shift=False, act="none", mlp_bias=True,
+           mlps={"dense": "glu", "moe": "softmax_moe"}, layer_norms=True, layer_scale=True, input_conv=True,
+           scaled_embed=True, tied_head=True),
 )}
 ARCHITECTURES = tuple(DESIGNS)
 
@@ -317,6 +331,10 @@ class HeadAttentionSpec:
     interleaved: ClassVar[bool] = False  # rotated pairs are neighbours, else half a rotation apart
     unit_qk: ClassVar[bool] = False     # rotated queries and keys are divided by their root mean square
     gated: ClassVar[bool] = False       # the output times the sigmoid of a projection, number by number
+    row_norms: ClassVar[bool] = False   # RMS norms of q and of k over all heads at once, before the rotation
+    unit_v: ClassVar[bool] = False      # each head's value is divided by its root mean square
+    tempered: ClassVar[bool] = False    # a head's scores times a number of its own
+    beside_one: ClassVar[bool] = False  # one more term exp(0) in the softmax's denominator
 
     heads: int
     kv_heads: int
@@ -328,6 +346,8 @@ class HeadAttentionSpec:
     window: Optional[int] = None        # a position sees itself and window - 1 before it
     softcap: Optional[float] = None     # scores s become softcap * tanh(s / softcap)
     diff: Optional[float] = None        # two maps: what their weights add to
+    keep_first: int = 0                 # positions that stay visible when the window has passed them
+    kv_from: Optional[int] = None       # the layer whose keys and values this one uses
 
     @classmethod
     def read(cls, m: Mapping[str, Any], shapes: Mapping[str, Any], p: str) -> "HeadAttentionSpec":
@@ -337,7 +357,9 @@ class HeadAttentionSpec:
                    rot_base=float(rot["base"]) if rot else 1.0,
                    window=int(mask["size"]) if mask else None,
                    softcap=None if cap is None else float(cap),
-                   diff=float(m["diff"]) if cls.maps == 2 else None)
+                   diff=float(m["diff"]) if cls.maps == 2 else None,
+                   keep_first=int(mask.get("keep_first") or 0) if mask else 0,
+                   kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
 
     def to_json(self) -> Dict[str, Any]:
         out: Dict[str, Any] = dict(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim,
@@ -346,6 +368,10 @@ class HeadAttentionSpec:
             out["rot"] = {"base": self.rot_base, "dims": self.rot_dims}
         if self.window is not None:
             out["mask"] = {"size": self.window}
+            if self.keep_first:
+                out["mask"]["keep_first"] = self.keep_first
+        if self.kv_from is not None:
+            out["kv_from"] = self.kv_from
         if self.softcap is not None:
             out["softcap"] = self.softcap
         if self.diff is not None:
@@ -361,14 +387,21 @@ class HeadAttentionSpec:
             _refuse(where, self.rot_dims, "Rotated dimensions must be even and fit the head")
         if self.window is not None and self.window < 1:
             _refuse(where, self.window, "A window has at least one position")
+        if self.keep_first < 0 or (self.keep_first and self.window is None):
+            _refuse(where, self.keep_first, "Only a window keeps first positions")
         if self.softcap is not None and not self.softcap > 0:
             _refuse(where, self.softcap, "A cap of scores is positive")
         if (self.diff is not None) != (self.maps == 2):
             _refuse(where, self.diff, "Two maps, and only two, need the constant of their difference")
 
     def tensors(self, W: int) -> Shapes:
-        out: Shapes = {"q": (self.heads * self.maps * self.dim, W),
-                       "k": (self.kv_heads * self.maps * self.dim, W), "v": (self.kv_heads * self.vdim, W)}
+        out: Shapes = {"q": (self.heads * self.maps * self.dim, W)}
+        if self.kv_from is None:
+            out.update({"k": (self.kv_heads * self.maps * self.dim, W), "v": (self.kv_heads * self.vdim, W)})
+        if self.row_norms:
+            out.update({n + ".norm": out[n][:1] for n in "qk" if n in out})
+        if self.tempered:
+            out["temp"] = (self.heads,)
         if self.maps == 2:
             out.update({n: (self.dim,) for n in MAP_VECTORS})
         if self.gated:
@@ -405,10 +438,22 @@ class CappedAttentionSpec(HeadAttentionSpec):
     gated: ClassVar[bool] = True
 
 
+@dataclass(frozen=True)
+class KeptWindowAttentionSpec(HeadAttentionSpec):
+    """A sliding window beside which the first positions stay visible."""
+
+    kind: ClassVar[str] = "kept_window_attention"
+    interleaved: ClassVar[bool] = True
+    row_norms: ClassVar[bool] = True
+    unit_v: ClassVar[bool] = True
+    tempered: ClassVar[bool] = True
+    beside_one: ClassVar[bool] = True
+
+
 MixerSpec = Union[AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, Mamba2Spec, MinGruSpec,
                   HeadAttentionSpec]
 MIXERS = {c.kind: c for c in (AttentionSpec, ChannelDeltaSpec, LatentAttentionSpec, Mamba2Spec,
-                              MinGruSpec, DiffAttentionSpec, CappedAttentionSpec)}
+                              MinGruSpec, DiffAttentionSpec, CappedAttentionSpec, KeptWindowAttentionSpec)}
 # mixers that look back through the paged cache
 CACHED = (AttentionSpec, LatentAttentionSpec, HeadAttentionSpec)
 
@@ -425,7 +470,7 @@ class MlpSpec:
         return cls(ff=int(m["ff"]))
 
     def to_json(self) -> Dict[str, Any]:
-        return dict(kind=self.kind, ff=self.ff)
+        return dict(ff=self.ff)
 
     def check(self, where: str) -> None:
         if self.ff < 1:
@@ -439,16 +484,47 @@ class MlpSpec:
 
 
 @dataclass(frozen=True)
-class GluSpec:
-    """An expert: ``down(g * sigmoid(slope * g) * (u + 1))``, ``g`` bounded by ``limit`` above and ``u``
-    on both sides."""
+class GluMlpSpec:
+    """``down(g * sigmoid(slope * g) * (u + shift))``, ``g`` (of ``gate``) bounded by ``limit`` above and ``u``
+    (of ``up``) on both sides."""
 
+    kind: ClassVar[str] = "glu"
+    slope: ClassVar[float] = 1.702
+    shift: ClassVar[float] = 1.0
     ff: int
     limit: float
 
     @classmethod
-    def read(cls, m: Mapping[str, Any]) -> "GluSpec":
+    def read(cls, m: Mapping[str, Any]) -> "GluMlpSpec":
         return cls(ff=int(m["ff"]), limit=float(m["limit"]))
+
+    def to_json(self) -> Dict[str, Any]:
+        return dict(ff=self.ff, limit=self.limit)
+
+    def check(self, where: str) -> None:
+        if self.ff < 1 or not self.limit > 0:
+            _refuse(where, f"{self.ff}/{self.limit}", "A feed-forward has a channel and a positive limit")
+
+    def tensors(self, W: int, bias: bool) -> Shapes:
+        out: Shapes = {"gate": (self.ff, W), "up": (self.ff, W), "down": (W, self.ff)}
+        if bias:
+            out.update({n + ".b": out[n][:1] for n in ("gate", "up", "down")})
+        return out
+
+
+@dataclass(frozen=True)
+class GluSpec:
+    """An expert: the same unit without biases, bounded or (``limit`` infinite) not."""
+
+    ff: int
+    limit: float = math.inf
+
+    @classmethod
+    def read(cls, m: Mapping[str, Any], bounded: bool = True) -> "GluSpec":
+        return cls(ff=int(m["ff"]), limit=float(m["limit"]) if bounded else math.inf)
+
+    def to_json(self) -> Dict[str, Any]:
+        return dict(ff=self.ff) if math.isinf(self.limit) else dict(ff=self.ff, limit=self.limit)
 
     def tensors(self, W: int, p: str) -> Shapes:
         return {p + "gate": (self.ff, W), p + "up": (self.ff, W), p + "down": (W, self.ff)}
@@ -456,11 +532,20 @@ class GluSpec:
 
 @dataclass(frozen=True)
 class MoeSpec:
-    """Every token uses the ``top`` of ``experts`` with the largest sigmoid scores among the ``keep`` best
-    of ``groups`` equal groups of neighbours (a group counts the sum of its two largest), weighted by
-    their scores over the scores' sum, times ``scale``; and the shared expert, if there is one."""
+    """Every token uses the ``top`` of ``experts`` with the largest scores among the ``keep`` best of
+    ``groups`` equal groups of neighbours, weighted by their scores times ``scale``; and the shared expert,
+    if there is one.  Class attributes are what a kind fixes."""
 
     kind: ClassVar[str] = "moe"
+    softmax: ClassVar[bool] = False      # scores are a softmax over all experts, else sigmoids
+    corrected: ClassVar[bool] = False    # a number per expert is added to its score for the choice only
+    group_best: ClassVar[int] = 2        # a group counts the sum of so many of its largest scores
+    normalised: ClassVar[bool] = True    # weights are divided by their sum
+    shared_gate: ClassVar[bool] = False  # the shared expert times the sigmoid of a projection
+    slope: ClassVar[float] = 1.702       # of the experts' gated unit
+    shift: ClassVar[float] = 1.0
+    bounded: ClassVar[bool] = True
+
     experts: int
     top: int
     expert: GluSpec
@@ -468,49 +553,79 @@ class MoeSpec:
     groups: int = 1
     keep: int = 1
     shared: Optional[GluSpec] = None
+    identity: int = 0                    # experts behind the others whose result is their input
 
     @classmethod
     def read(cls, m: Mapping[str, Any]) -> "MoeSpec":
         r = m["router"]
         groups = r.get("groups") or {"count": 1, "keep": 1}
-        return cls(experts=int(r["experts"]), top=int(r["top"]), expert=GluSpec.read(m["expert"]),
+        return cls(experts=int(r["experts"]), top=int(r["top"]), expert=GluSpec.read(m["expert"], cls.bounded),
                    scale=float(r.get("scale", 1.0)), groups=int(groups["count"]), keep=int(groups["keep"]),
-                   shared=GluSpec.read(m["shared"]) if m.get("shared") else None)
+                   shared=GluSpec.read(m["shared"], cls.bounded) if m.get("shared") else None,
+                   identity=int(r.get("identity") or 0))
 
     def to_json(self) -> Dict[str, Any]:
-        def glu(g: GluSpec) -> Dict[str, Any]:
-            return dict(ff=g.ff, limit=g.limit)
-        out: Dict[str, Any] = dict(
-            kind=self.kind, expert=glu(self.expert),
-            router=dict(experts=self.experts, top=self.top, scale=self.scale,
-                        groups=dict(count=self.groups, keep=self.keep)))
+        router: Dict[str, Any] = dict(experts=self.experts, top=self.top,
+                                      groups=dict(count=self.groups, keep=self.keep))
+        if self.normalised or self.scale != 1.0:
+            router["scale"] = self.scale
+        if self.identity:
+            router["identity"] = self.identity
+        out: Dict[str, Any] = dict(expert=self.expert.to_json(), router=router)
         if self.shared is not None:
-            out["shared"] = glu(self.shared)
+            out["shared"] = self.shared.to_json()
         return out
 
     def check(self, where: str) -> None:
-        if not 1 <= self.experts <= MAX_EXPERTS or not 1 <= self.top <= MAX_TOP:
-            _refuse(where, f"{self.top} of {self.experts}",
+        if self.experts < 1 or self.identity < 0 or self.outputs > MAX_EXPERTS or not 1 <= self.top <= MAX_TOP:
+            _refuse(where, f"{self.top} of {self.outputs}",
                     f"Up to {MAX_TOP} of up to {MAX_EXPERTS} experts are chosen")
-        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
+        if self.groups < 1 or self.outputs % self.groups or not 1 <= self.keep <= self.groups:
             _refuse(where, f"{self.keep} of {self.groups}", "Groups must be equal, and one of them kept")
-        if self.top > self.keep * (self.experts // self.groups):
+        if self.top > self.keep * (self.outputs // self.groups):
             _refuse(where, self.top, "The kept groups must hold enough experts")
         for g in (self.expert, self.shared):
             if g is not None and (g.ff < 1 or not g.limit > 0):
                 _refuse(where, f"{g.ff}/{g.limit}", "An expert has a channel and a positive limit")
 
+    @property
+    def outputs(self) -> int:
+        """Of the router."""
+        return self.experts + self.identity
+
+    def routing(self):
+        from ..ops.experts import Routing
+        return Routing(self.experts, self.top, self.groups, self.keep, self.scale, self.identity, self.softmax,
+                       self.group_best, self.normalised, self.shared_gate and self.shared is not None)
+
     def tensors(self, W: int, bias: bool) -> Shapes:
-        out: Shapes = {"router": (self.experts, W)}
+        out: Shapes = {"router": (self.outputs, W)}
+        if self.corrected:
+            out["correction"] = (self.outputs,)
         for e in range(self.experts):
             out.update(self.expert.tensors(W, f"e{e}."))
         if self.shared is not None:
             out.update(self.shared.tensors(W, "shared."))
+            if self.shared_gate:
+                out["shared.sg"] = (1, W)
         return out
 
 
-FeedForwardSpec = Union[MlpSpec, MoeSpec]
-MLPS = {c.kind: c for c in (MlpSpec, MoeSpec)}
+@dataclass(frozen=True)
+class SoftmaxMoeSpec(MoeSpec):
+    kind: ClassVar[str] = "softmax_moe"
+    softmax: ClassVar[bool] = True
+    corrected: ClassVar[bool] = True
+    group_best: ClassVar[int] = 1
+    normalised: ClassVar[bool] = False
+    shared_gate: ClassVar[bool] = True
+    slope: ClassVar[float] = 1.0
+    shift: ClassVar[float] = 0.0
+    bounded: ClassVar[bool] = False
+
+
+FeedForwardSpec = Union[MlpSpec, GluMlpSpec, MoeSpec]
+MLPS = {c.kind: c for c in (MlpSpec, GluMlpSpec, MoeSpec, SoftmaxMoeSpec)}
 
 
 @dataclass(frozen=True)
@@ -546,6 +661,8 @@ class HybridConfig:
     max_seq_len: int = DEFAULT_MAX_SEQ_LEN
     logit_scale: float = 1.0
     loop: Optional[LoopSpec] = None
+    embed_scale: float = 1.0
+    conv_taps: int = 0       # of the convolution in front of the mixers
     pos: str = field(default="rope", init=False)   # positions need no table of trained rows
 
     @property
@@ -591,16 +708,32 @@ class HybridConfig:
                     _refuse(where, size, "Layers that mix values must agree in their size")
                 mixing = size
             if layer.mlp is not None:
-                if layer.mlp.kind not in self.design.mlps:
+                if layer.mlp.kind not in self.design.mlps.values():
                     _refuse(f"layers[{i}].mlp", layer.mlp.kind,
-                            f"Feed-forwards of {self.architecture}: {', '.join(self.design.mlps)}")
+                            f"Feed-forwards of {self.architecture}: {', '.join(self.design.mlps.values())}")
                 layer.mlp.check(f"layers[{i}].mlp")
+            if getattr(m, "kv_from", None) is not None:
+                self._check_shared(i, m)
+        if self.design.input_conv:
+            _taps_ok("conv_taps", self.conv_taps)
+            if (self.conv_taps - 1) * self.width_padded > MAX_HISTORY:
+                _refuse("conv_taps", self.conv_taps, f"Taps times width must not exceed {MAX_HISTORY}")
         if self.loop is not None:
             lo = self.loop
             if self.design.parallel:
                 _refuse("loop", lo, f"{self.architecture} has no loop")
             if not 0 <= lo.start < lo.stop <= self.num_layers or lo.times < 1:
                 _refuse("loop", f"{lo.start}..{lo.stop} x {lo.times}", "The loop must be a run of layers")
+
+    def _check_shared(self, i: int, m: "HeadAttentionSpec") -> None:
+        where = f"layers[{i}].mixer.kv_from"
+        if not 0 <= m.kv_from < i or self.loop is not None:
+            _refuse(where, m.kv_from, "Keys and values come from an earlier layer")
+        s = self.layers[m.kv_from].mixer
+        if s.kind != m.kind or s.kv_from is not None:
+            _refuse(where, m.kv_from, "Keys and values come from a layer that makes them")
+        if (s.kv_heads, s.dim, s.vdim) != (m.kv_heads, m.dim, m.vdim):
+            _refuse(where, m.kv_from, "Layers that share keys and values have the same key/value heads")
 
     def to_dict(self) -> Dict[str, Any]:
         return config_to_json(self)
@@ -623,21 +756,24 @@ def config_from_json(config: Mapping[str, Any], shapes: Mapping[str, Any]) -> Hy
     architecture = str(config.get("architecture", "Sapasun"))
     if architecture not in DESIGNS:
         raise ProcessingError.unsupported(f"architecture '{architecture}'", ", ".join(DESIGNS))
-    kinds = DESIGNS[architecture].mixers
+    design = DESIGNS[architecture]
+    kinds = design.mixers
     for i, entry in enumerate(config["layers"]):
         if entry["type"] not in kinds:
             raise ProcessingError.unsupported(f"mixer type '{entry['type']}'", ", ".join(kinds))
         mixer = MIXERS[kinds[entry["type"]]].read(entry["mixer"], shapes, f"l{i}.mix.")
         mlp = entry.get("mlp")
-        if mlp and mlp["kind"] not in MLPS:
-            raise ProcessingError.unsupported(f"feed-forward '{mlp['kind']}'", ", ".join(MLPS))
-        layers.append(LayerSpec(mixer, MLPS[mlp["kind"]].read(mlp) if mlp else None))
+        if mlp and mlp["kind"] not in design.mlps:
+            raise ProcessingError.unsupported(f"feed-forward '{mlp['kind']}'", ", ".join(design.mlps))
+        layers.append(LayerSpec(mixer, MLPS[design.mlps[mlp["kind"]]].read(mlp) if mlp else None))
     cap, loop = config.get("logit_softcap"), config.get("loop")
     cfg = HybridConfig(
         vocab_size=int(config["vocab"]), hidden_dim=int(config["width"]), layers=tuple(layers),
         norm_eps=float(config["norm"]["eps"]), logit_softcap=None if cap is None else float(cap),
         architecture=architecture,
-        logit_scale=float(config.get("logit_scale", 1.0)) if DESIGNS[architecture].scaled_logits else 1.0,
+        logit_scale=float(config.get("logit_scale", 1.0)) if design.scaled_logits else 1.0,
+        embed_scale=float(config["embedding"]["scale"]) if design.scaled_embed else 1.0,
+        conv_taps=int(config["canon"]["taps"]) if design.input_conv else 0,
         loop=None if not loop else LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"])))
     cfg.validate()
     return cfg
@@ -645,14 +781,20 @@ def config_from_json(config: Mapping[str, Any], shapes: Mapping[str, Any]) -> Hy
 
 def config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
     types = {kind: name for name, kind in cfg.design.mixers.items()}
+    mlps = {kind: name for name, kind in cfg.design.mlps.items()}
     layers = [{"type": types[layer.mixer.kind], "mixer": layer.mixer.to_json(),
-               "mlp": None if layer.mlp is None else layer.mlp.to_json()} for layer in cfg.layers]
+               "mlp": None if layer.mlp is None else dict(kind=mlps[layer.mlp.kind], **layer.mlp.to_json())}
+              for layer in cfg.layers]
     out = {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_dim,
            "norm": {"eps": cfg.norm_eps}, "layers": layers}
     if cfg.design.parallel:
         out["logit_softcap"] = cfg.logit_softcap
     elif cfg.design.scaled_logits:
         out["logit_scale"] = cfg.logit_scale
+    if cfg.design.scaled_embed:
+        out["embedding"] = {"scale": cfg.embed_scale}
+    if cfg.design.input_conv:
+        out["canon"] = {"taps": cfg.conv_taps}
     if cfg.loop is not None:
         out["loop"] = {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times}
     return out
@@ -673,13 +815,23 @@ def tensor_shapes(cfg: HybridConfig) -> Shapes:
             out[p + n] = norm
             if d.post_norms:
                 out[p + n + "b"] = norm
+            if d.layer_norms:
+                out[p + n + ".b"] = norm
+            if d.layer_scale:
+                out[p + "ls" + n[4:]] = (W,)
         if d.token_shift:
             out[p + "shift"] = (W,)
+        if d.input_conv:
+            out[p + "canon1"] = (W, cfg.conv_taps)
         out.update({f"{p}mix.{n}": s for n, s in layer.mixer.tensors(W).items()})
         out[p + "mix.o"] = (W, layer.mixer.out_dim)
         if layer.mlp is not None:
             out.update({f"{p}mlp.{n}": s for n, s in layer.mlp.tensors(W, d.mlp_bias).items()})
-    out.update({"final.norm": norm, "head": (V, W)})
+    out["final.norm"] = norm
+    if d.layer_norms:
+        out["final.norm.b"] = norm
+    if not d.tied_head:
+        out["head"] = (V, W)
     return out
 
 
@@ -694,8 +846,14 @@ def random_state(cfg: HybridConfig, seed: int = 0, device="cpu",
     out = {}
     for name, shape in tensor_shapes(cfg).items():
         leaf = name.split(".")[-1]
-        if leaf.startswith("norm"):
+        if leaf.startswith("norm") or leaf in ("ls1", "ls2", "temp"):
             t = 1.0 + normal(shape, 0.1)
+        elif leaf == "canon1":
+            t = normal(shape, 0.3)
+        elif leaf == "embed" and cfg.design.tied_head:
+            t = normal(shape, shape[-1] ** -0.5)
+        elif leaf == "correction":
+            t = normal(shape, 0.1)
         elif leaf == "conv":
             t = normal(shape, 0.3)
             t[:, -1] += 1.0
@@ -719,26 +877,39 @@ def _pad(t: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
     return out
 
 
+def _alternate(a: torch.Tensor, b: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
+    """Rows of ``a`` and ``b`` in turn, each padded to ``rows x cols``."""
+    return torch.stack([_pad(a, rows, cols), _pad(b, rows, cols)], 1).view(2 * rows, cols)
+
+
 class Experts:
     """Device weights of a mixture of experts.  Rows of gate and up alternate (``w_in [experts, 2 ff, W]``),
     so that a tile of the product has both numbers of a channel; ``w_down [experts, W, ff]``; the shared
     expert's ``s_in`` and ``s_down`` likewise."""
 
-    def __init__(self, spec: MoeSpec, slope: float, mat, wp: int) -> None:
-        self.spec, self.slope, self.wp = spec, slope, wp
-        self.router = _pad(mat("mlp.router"), _up8(spec.experts), wp)
+    def __init__(self, spec: MoeSpec, mat, vec, wp: int) -> None:
+        self.spec, self.wp = spec, wp
+        self.slope, self.shift = spec.slope, spec.shift
+        self.routing = spec.routing()
+        router = mat("mlp.router")
+        if self.routing.shared_gate:          # one more output of the same product
+            router = torch.cat([router, mat("mlp.shared.sg")])
+        self.router = _pad(router, _up8(router.shape[0]), wp)
+        self.correction = vec("mlp.correction") if spec.corrected else None
 
         def pair(p: str, g: GluSpec):
-            n = _up8(g.ff)
-            w = torch.stack([_pad(mat(p + "gate"), n, wp), _pad(mat(p + "up"), n, wp)], 1)
-            return w.view(2 * n, wp), _pad(mat(p + "down"), wp, n)
+            return _alternate(mat(p + "gate"), mat(p + "up"), _up8(g.ff), wp), _pad(mat(p + "down"), wp, _up8(g.ff))
         ws = [pair(f"mlp.e{e}.", spec.expert) for e in range(spec.experts)]
         self.w_in, self.w_down = (torch.stack(t).contiguous() for t in zip(*ws))
         self.s_in, self.s_down = pair("mlp.shared.", spec.shared) if spec.shared else (None, None)
 
     def tensors(self, W: int) -> Dict[str, torch.Tensor]:
         s = self.spec
-        out = {"router": self.router[:s.experts, :W]}
+        out = {"router": self.router[:s.outputs, :W]}
+        if self.correction is not None:
+            out["correction"] = self.correction
+        if self.routing.shared_gate:
+            out["shared.sg"] = self.router[s.outputs:s.outputs + 1, :W]
 
         def apart(p: str, w_in: torch.Tensor, down: torch.Tensor, ff: int) -> None:
             out.update({p + "gate": w_in[0:2 * ff:2, :W], p + "up": w_in[1:2 * ff:2, :W],
@@ -757,7 +928,8 @@ class HybridLayer:
     projection and the feed-forward's down projection side by side: both are added to the same
     stream, so they are one product over ``[mixer output | activation]``, the activation starting at
     column ``act_off``.  Otherwise ``w_out`` is the mixer's output projection and ``w_down`` the
-    feed-forward's."""
+    feed-forward's.  A feed-forward with a gated unit has the rows of its gate and up projections in
+    turn in ``w_up`` (and their biases in ``b_up``)."""
 
     def __init__(self, spec: LayerSpec, design: Design, w_get, width: int, dtype: torch.dtype) -> None:
         self.spec, self.dtype = spec, dtype
@@ -765,11 +937,18 @@ class HybridLayer:
         self.wp = _up8(width)
         self.norm1 = self._gain("norm1", design)
         self.norm1b = self._gain("norm1b", design) if design.post_norms else None
+        self.center1 = self._vec("norm1.b", self.wp) if design.layer_norms else None
+        self.scale1 = self._vec("ls1", self.wp) if design.layer_scale else None
+        self.center2 = self.scale2 = self.taps = None
+        if design.input_conv:         # taps-major
+            t = w_get("canon1").float()
+            self.taps = _pad(t.t(), t.shape[1], self.wp)
         self.shift = self._vec("shift", self.wp) if design.token_shift else None
         self.seg: Dict[str, int] = {}
         {"attention": self._attention, "channel_delta": self._channel_delta,
          "latent_attention": self._latent, "mamba2": self._mamba2, "mingru": self._mingru,
-         "diff_attention": self._heads, "capped_attention": self._heads}[spec.mixer.kind](spec.mixer)
+         "diff_attention": self._heads, "capped_attention": self._heads,
+         "kept_window_attention": self._heads}[spec.mixer.kind](spec.mixer)
         self.out_dim = spec.mixer.out_dim
         self.act_off = _up8(self.out_dim)
         outs = [_pad(self._mat("mix.o"), self.wp, self.act_off)]
@@ -779,11 +958,18 @@ class HybridLayer:
         if spec.mlp is not None:
             self.norm2 = self._gain("norm2", design)
             self.norm2b = self._gain("norm2b", design) if design.post_norms else None
+            self.center2 = self._vec("norm2.b", self.wp) if design.layer_norms else None
+            self.scale2 = self._vec("ls2", self.wp) if design.layer_scale else None
+        self.glu: Optional[Tuple[float, float, float]] = None
         if isinstance(spec.mlp, MoeSpec):
-            self.experts = Experts(spec.mlp, design.glu_slope, self._mat, self.wp)
+            self.experts = Experts(spec.mlp, self._mat, self._vec, self.wp)
         elif spec.mlp is not None:
             self.ff, self.ff_padded = spec.mlp.ff, _up8(spec.mlp.ff)
-            self.w_up = _pad(self._mat("mlp.up"), self.ff_padded, self.wp)
+            if isinstance(spec.mlp, GluMlpSpec):
+                self.glu = (spec.mlp.slope, spec.mlp.limit, spec.mlp.shift)
+                self.w_up = _alternate(self._mat("mlp.gate"), self._mat("mlp.up"), self.ff_padded, self.wp)
+            else:
+                self.w_up = _pad(self._mat("mlp.up"), self.ff_padded, self.wp)
             down = _pad(self._mat("mlp.down"), self.wp, self.ff_padded)
             if design.parallel:
                 outs.append(down)
@@ -791,6 +977,9 @@ class HybridLayer:
                 self.w_down = down
             if design.mlp_bias:
                 self.b_up = self._vec("mlp.up.b", self.ff_padded).to(dtype)
+                if self.glu is not None:
+                    self.b_up = torch.stack([self._vec("mlp.gate.b", self.ff_padded).to(dtype), self.b_up],
+                                            1).flatten()
                 self.b_down = self._vec("mlp.down.b", self.wp)
         self.w_out = torch.cat(outs, 1).contiguous()
         del self._get
@@ -878,7 +1067,12 @@ class HybridLayer:
                     {n: self._get(f"mix.{n}.b") for n in ("z", "x")})
 
     def _heads(self, m: HeadAttentionSpec) -> None:
-        self._stack({n: self._mat("mix." + n) for n in (("q", "k", "v", "g") if m.gated else ("q", "k", "v"))})
+        shapes = m.tensors(self.wp)
+        self._stack({n: self._mat("mix." + n) for n in "qkvg" if n in shapes})
+        self.q_norm, self.k_norm = (self._vec(f"mix.{n}.norm") if n + ".norm" in shapes else None for n in "qk")
+        self.temp = self._vec("mix.temp") if m.tempered else None
+        # a term exp(0) in the softmax's denominator is a sink of score 0
+        self.sink = torch.zeros(m.heads, device=self.w_in.device) if m.beside_one else None
         self.rope_key = (m.rot_base, m.rot_dims) if m.rot_dims else None
         self.map_vectors = self.map_weight = None
         if m.maps == 2:
@@ -928,22 +1122,31 @@ class HybridLayer:
                         "mix.norm": self.out_norm})
         elif isinstance(m, HeadAttentionSpec):
             stacked(n for n in ("q", "k", "v", "g") if n in shapes)
+            out.update({"mix." + n: t for n, t in (("q.norm", self.q_norm), ("k.norm", self.k_norm),
+                                                   ("temp", self.temp)) if t is not None})
             out.update({"mix." + n: t for n, t in (self.map_vectors or {}).items()})
         else:
             stacked(("z", "x", "g"))
             for n in ("z", "x"):
                 out[f"mix.{n}.b"] = self.b_in[self.seg[n]:self.seg[n] + m.width]
-        for n in ("norm1b", "norm2", "norm2b", "shift"):
-            if getattr(self, n) is not None:
-                out[n] = getattr(self, n)
+        for n, t in (("norm1b", self.norm1b), ("norm2", self.norm2), ("norm2b", self.norm2b), ("shift", self.shift),
+                     ("norm1.b", self.center1), ("norm2.b", self.center2), ("ls1", self.scale1), ("ls2", self.scale2)):
+            if t is not None:
+                out[n] = t
+        if self.taps is not None:
+            out["canon1"] = self.taps[:, :W].t()
         if self.experts is not None:
             out.update({"mlp." + n: t for n, t in self.experts.tensors(W).items()})
         if self.w_up is not None:
             out["mlp.up"] = self.w_up[:self.ff, :W]
+            if self.glu is not None:
+                out["mlp.gate"], out["mlp.up"] = (self.w_up[i:2 * self.ff:2, :W] for i in (0, 1))
             out["mlp.down"] = self.w_out[:W, self.act_off:self.act_off + self.ff] \
                 if self.w_down is None else self.w_down[:W, :self.ff]
             if self.b_up is not None:
                 out["mlp.up.b"], out["mlp.down.b"] = self.b_up[:self.ff], self.b_down[:W]
+                if self.glu is not None:
+                    out["mlp.gate.b"], out["mlp.up.b"] = (self.b_up[i:2 * self.ff:2] for i in (0, 1))
         return out
 
 
@@ -974,7 +1177,7 @@ class HybridLM:
             t = get(name).float()
             return t.reshape(1) if design.scalar_norms else \
                 torch.nn.functional.pad(t, (0, wp - W)).contiguous()
-        self.embed = _pad(get("embed").to(self.dtype), cfg.vocab_size, wp)
+        self.embed = _pad(get("embed").to(self.dtype), cfg.vocab_padded if design.tied_head else cfg.vocab_size, wp)
         self.embed_norm = gain("embed.norm") if design.embed_norm else None
         self.loop_in = self.loop_step = None
         if cfg.loop is not None:       # [W, 2 W] with the padding of each half behind it
@@ -986,7 +1189,8 @@ class HybridLM:
         self.final_norm = gain("final.norm")
         # the logits' factor rides on the last norm's gain
         self.final_gain = self.final_norm * cfg.logit_scale
-        self.head = _pad(get("head").to(self.dtype), cfg.vocab_padded, wp)
+        self.final_center = gain("final.norm.b") * cfg.logit_scale if design.layer_norms else None
+        self.head = self.embed if design.tied_head else _pad(get("head").to(self.dtype), cfg.vocab_padded, wp)
         # rotary frequencies base^(-2i/dims), one table per distinct (base, dims)
         self.inv_freq: Dict[Tuple[float, int], torch.Tensor] = {}
         for layer in self.layers:
@@ -1012,8 +1216,11 @@ class HybridLM:
     def state_dict(self) -> Dict[str, torch.Tensor]:
         """The checkpoint's tensors, taken apart again."""
         cfg, W = self.cfg, self.cfg.hidden_dim
-        out = {"embed": self.embed[:, :W], "final.norm": self.final_norm[:W],
-               "head": self.head[:cfg.vocab_size, :W]}
+        out = {"embed": self.embed[:cfg.vocab_size, :W], "final.norm": self.final_norm[:W]}
+        if not cfg.design.tied_head:
+            out["head"] = self.head[:cfg.vocab_size, :W]
+        if self.final_center is not None:
+            out["final.norm.b"] = self.final_center[:W] / cfg.logit_scale
         if self.embed_norm is not None:
             out["embed.norm"] = self.embed_norm[:W]
         if self.loop_in is not None:

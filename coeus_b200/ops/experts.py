@@ -1,5 +1,6 @@
-"""Mixture of experts of the serving step (``csrc/experts.cu``): routing by sigmoid scores among the best
-groups, without a capacity (every chosen expert runs), and experts whose gated unit is bounded.
+"""Mixture of experts of the serving step (``csrc/experts.cu``): routing by sigmoid or softmax scores among
+the best groups, without a capacity (every chosen expert runs), experts with a gated unit, and identity
+experts, whose result is their input.
 
 Few rows stream the weights of the chosen experts (:func:`experts_few`).  Larger batches are sorted by
 expert into a buffer whose experts start at multiples of a block of rows, and the experts' products are one
@@ -37,39 +38,55 @@ class Routing:
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
+    identity: int = 0         # experts ``experts ..`` that pass their input on
+    softmax: bool = False     # scores: softmax over all of them, else sigmoids
+    group_best: int = 2       # a group counts the sum of its one or two largest scores
+    normalise: bool = True    # weights are divided by their sum
+    shared_gate: bool = False   # the router's next output is the logit of the shared expert's gate
+
+    @property
+    def outputs(self) -> int:
+        return self.experts + self.identity
 
 
 @dataclass
 class Choice:
-    """``expert`` (int32) and ``weight`` (fp32) ``[tokens, top]``; on the GPU also what sorting needs: the
-    tokens of a block, the rank of a pair among its block's of the same expert, the blocks' counts."""
+    """``expert`` (int32) and ``weight`` (fp32) ``[tokens, top]``, ``shared`` (fp32 ``[tokens]``) the shared
+    expert's weight where it has one; on the GPU also what sorting needs: the tokens of a block, the rank of
+    a pair among its block's of the same expert, the blocks' counts."""
 
     expert: torch.Tensor
     weight: torch.Tensor
+    shared: Optional[torch.Tensor] = None
     per_block: int = 0
     rank: Optional[torch.Tensor] = None
     counts: Optional[torch.Tensor] = None
 
 
-def choose(z: torch.Tensor, r: Routing) -> Tuple[torch.Tensor, torch.Tensor]:
-    """The choice in PyTorch, from the router's logits ``z [tokens, experts]``; ties go to the lower index."""
-    s = torch.sigmoid(z.float())
-    T, n = s.shape[0], r.experts // r.groups
-    value = s.view(T, r.groups, n).topk(min(2, n), -1).values.sum(-1)
+def choose(z: torch.Tensor, r: Routing, correction: Optional[torch.Tensor] = None
+           ) -> Tuple[torch.Tensor, torch.Tensor]:
+    """The choice in PyTorch, from the router's logits ``z [tokens, outputs]``; ties go to the lower index.
+    ``correction`` is added to the scores that are compared, not to the weights."""
+    s = torch.softmax(z.float(), -1) if r.softmax else torch.sigmoid(z.float())
+    rated = s if correction is None else s + correction
+    T, n = s.shape[0], r.outputs // r.groups
+    value = rated.view(T, r.groups, n).topk(min(r.group_best, n), -1).values.sum(-1)
     kept = torch.sort(value, dim=-1, descending=True, stable=True).indices[:, :r.keep]
     ok = torch.zeros(T, r.groups, dtype=torch.bool, device=z.device).scatter_(1, kept, True)
-    masked = s.masked_fill(~ok.repeat_interleave(n, 1), -1.0)
+    masked = rated.masked_fill(~ok.repeat_interleave(n, 1), float("-inf"))
     expert = torch.sort(masked, dim=-1, descending=True, stable=True).indices[:, :r.top]
     w = s.gather(1, expert)
-    return expert.to(torch.int32), w / (w.sum(-1, keepdim=True) + 1e-20) * r.scale
+    return expert.to(torch.int32), (w / (w.sum(-1, keepdim=True) + 1e-20) if r.normalise else w) * r.scale
 
 
-def route(h: torch.Tensor, router: torch.Tensor, r: Routing) -> Choice:
-    """The experts of every row of ``h [tokens, W]`` by the logits ``h @ router^T`` (``router [experts
-    rounded up to 8, W]``), which are fp32."""
+def route(h: torch.Tensor, router: torch.Tensor, r: Routing, correction: Optional[torch.Tensor] = None) -> Choice:
+    """The experts of every row of ``h [tokens, W]`` by the logits ``h @ router^T`` (``router [outputs, and
+    the shared expert's gate, rounded up to 8, W]``), which are fp32."""
     T, W = h.shape
     if not h.is_cuda:
-        return Choice(*choose(h.float() @ router[:r.experts].float().t(), r))
+        z = h.float() @ router.float().t()
+        return Choice(*choose(z[:, :r.outputs], r, correction),
+                      torch.sigmoid(z[:, r.outputs]) if r.shared_gate else None)
     from .gemm import linear
     few, dev = T <= ROUTE_FEW, h.device
     logits = None
@@ -79,20 +96,22 @@ def route(h: torch.Tensor, router: torch.Tensor, r: Routing) -> Choice:
     blocks = (T + per - 1) // per
     expert, rank = (torch.empty((T, r.top), dtype=torch.int32, device=dev) for _ in range(2))
     weight = torch.empty((T, r.top), dtype=torch.float32, device=dev)
-    counts = torch.empty((r.experts, blocks), dtype=torch.int32, device=dev)
+    counts = torch.empty((r.outputs, blocks), dtype=torch.int32, device=dev)
+    shared = torch.empty(T, dtype=torch.float32, device=dev) if r.shared_gate else None
     rc = _lib.serving_lib().cb_moe_choose(
         _p(logits), logits.stride(0) if logits is not None else 0, _p(h), h.stride(0), _p(router),
-        router.stride(0), W, T, r.experts, r.top, r.groups, r.keep, _F(r.scale), _p(expert), _p(weight),
+        router.stride(0), W, T, r.outputs, r.top, r.groups, r.keep, _F(r.scale), int(r.softmax), r.group_best,
+        int(r.normalise), _p(correction), _p(shared), _p(expert), _p(weight),
         _p(rank), _p(counts), int(h.dtype == torch.float32), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_moe_choose")
-    return Choice(expert, weight, per, rank, counts)
+    return Choice(expert, weight, shared, per, rank, counts)
 
 
 @dataclass
 class Sorted:
     """``rows [blocks * 128 or 256, W]``: every token's row once per expert it uses, sorted by expert;
-    ``slot [tokens, top]`` says where; ``block_expert [blocks]`` is the expert of a block of rows, -1 behind
-    the last one."""
+    ``slot [tokens, top]`` says where (-1: nowhere, an identity expert); ``block_expert [blocks]`` is the expert
+    of a block of rows, -1 behind the last one."""
 
     rows: torch.Tensor
     slot: torch.Tensor
@@ -108,7 +127,7 @@ def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
     rows = torch.empty((blocks * block, W), dtype=h.dtype, device=dev)
     if not h.is_cuda:
         rows.zero_()
-        slot = torch.empty((T, r.top), dtype=torch.int32)
+        slot = torch.full((T, r.top), -1, dtype=torch.int32)
         block_expert, at = [], 0
         for e in range(r.experts):
             t, k = (c.expert == e).nonzero(as_tuple=True)
@@ -132,9 +151,9 @@ def sort_rows(h: torch.Tensor, c: Choice, r: Routing) -> Sorted:
 
 
 def grouped_linear(x: torch.Tensor, w: torch.Tensor, block_expert: torch.Tensor, out: torch.Tensor, *,
-                   glu: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+                   glu: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
     """``out[block] = x[block] @ w[block_expert[block]]^T`` for every block of rows (``w [experts, N, K]``, as
-    many blocks as ``block_expert`` has entries, of 128 or 256 rows); blocks of no expert are left alone.  ``glu = (slope, limit)``: see :func:`coeus_b200.ops.gemm.linear`."""
+    many blocks as ``block_expert`` has entries, of 128 or 256 rows); blocks of no expert are left alone.  ``glu = (slope, limit, shift)``: see :func:`coeus_b200.ops.gemm.linear`."""
     E, N, K = w.shape
     M = x.shape[0]
     block = M // block_expert.shape[0]
@@ -147,24 +166,24 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, block_expert: torch.Tensor,
                 z = x[s].float() @ w[e].float().t()
                 out[s] = (clamped_glu(z, *glu) if glu else z).to(out.dtype)
         return out
-    slope, limit = glu or (0.0, 0.0)
+    slope, limit, shift = glu or (0.0, 0.0, 0.0)
     lib, st = _lib.serving_lib(), _p(_lib.status_buffer(x.device))
     if x.dtype == torch.float32:
         rc = lib.cb_linear_f32_grouped(
-            _p(x), x.stride(0), _p(w), w.stride(1), _p(block_expert), block, _p(out), out.stride(0), M, N, K,
-            int(glu is not None), _F(slope), _F(limit), _lib.stream_ptr())
+            _p(x), x.stride(0), _p(w), w.stride(1), None, _p(block_expert), block, _p(out), out.stride(0), M, N, K,
+            int(glu is not None), _F(slope), _F(limit), _F(shift), _lib.stream_ptr())
         _lib.check_rc(rc, "cb_linear_f32_grouped")
         return out
     rc = lib.cb_gemm_bf16_blocks(
-        _p(x), _p(w), _p(out), M, N, K, E, x.stride(0), w.stride(1), out.stride(0), _p(block_expert), block,
-        int(glu is not None), _F(slope), _F(limit), st, _lib.stream_ptr())
+        _p(x), _p(w), None, _p(out), M, N, K, E, x.stride(0), w.stride(1), out.stride(0), _p(block_expert), block,
+        int(glu is not None), _F(slope), _F(limit), _F(shift), st, _lib.stream_ptr())
     _lib.check_rc(rc, "cb_gemm_bf16_blocks")
     return out
 
 
 def experts_few(h: torch.Tensor, c: Choice, r: Routing, w_in: torch.Tensor, w_down: torch.Tensor,
                 limit: float, s_in: Optional[torch.Tensor], s_down: Optional[torch.Tensor],
-                s_limit: float, slope: float) -> torch.Tensor:
+                s_limit: float, slope: float, shift: float = 1.0) -> torch.Tensor:
     """All experts of up to ``FEW`` bf16 rows and the shared one: fp32 ``[tokens, W]``."""
     T, W = h.shape
     n, ns = w_down.shape[2], s_down.shape[1] if s_down is not None else 0
@@ -172,8 +191,8 @@ def experts_few(h: torch.Tensor, c: Choice, r: Routing, w_in: torch.Tensor, w_do
     act = torch.empty((T, live * n + ns), dtype=h.dtype, device=h.device)
     y = torch.empty((T, W), dtype=torch.float32, device=h.device)
     rc = _lib.serving_lib().cb_moe_few(
-        _p(h), h.stride(0), T, W, r.experts, r.top, _p(c.expert), _p(c.weight), _p(w_in), _p(w_down), n,
-        _F(limit), _p(s_in), _p(s_down), ns, _F(s_limit), _F(slope), _p(act), act.stride(0), _p(y),
+        _p(h), h.stride(0), T, W, r.experts, r.top, _p(c.expert), _p(c.weight), _p(c.shared),
+        _p(w_in), _p(w_down), n, _F(limit), _p(s_in), _p(s_down), ns, _F(s_limit), _F(slope), _F(shift), _p(act), act.stride(0), _p(y),
         y.stride(0), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_moe_few", launches=2)
     return y

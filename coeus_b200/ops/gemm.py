@@ -26,11 +26,11 @@ def _gelu_ref(x: torch.Tensor) -> torch.Tensor:
     return 0.5 * x * (1.0 + torch.tanh(0.7978845608028654 * x * (1.0 + 0.044715 * x * x)))
 
 
-def clamped_glu(z: torch.Tensor, slope: float, limit: float) -> torch.Tensor:
-    """``g * sigmoid(slope * g) * (u + 1)`` of alternating columns g and u, g bounded by ``limit`` above and
-    u on both sides."""
+def clamped_glu(z: torch.Tensor, slope: float, limit: float, shift: float = 1.0) -> torch.Tensor:
+    """``g * sigmoid(slope * g) * (u + shift)`` of alternating columns g and u, g bounded by ``limit`` above
+    and u on both sides (infinite: not)."""
     g, u = z[..., 0::2].clamp(max=limit), z[..., 1::2].clamp(-limit, limit)
-    return g * torch.sigmoid(slope * g) * (u + 1)
+    return g * torch.sigmoid(slope * g) * (u + shift)
 
 
 def _gelu_grad_ref(x: torch.Tensor) -> torch.Tensor:
@@ -274,14 +274,16 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
     operands run on the tensor cores
     with a bf16 or fp32 ``out``; fp32 operands are multiplied in full fp32 (``cb_linear_f32``).
     ``accumulate`` adds into an fp32 ``out`` (the residual stream); ``softcap`` maps the result
-    ``z`` to ``softcap * tanh(z / softcap)`` (fp32 ``out``).  ``glu = (slope, limit)`` makes one column of
-    every two (:func:`clamped_glu`), in the type of the operands."""
+    ``z`` to ``softcap * tanh(z / softcap)`` (fp32 ``out``).  ``glu = (slope, limit[, shift])`` makes one column of
+    every two after the bias (:func:`clamped_glu`), in the type of the operands."""
     M, K = x.shape
     N = w.shape[0]
     if glu is not None:
-        if bias is not None or accumulate or softcap is not None or epi != "none" or out.dtype != x.dtype:
-            raise ValueError("linear: a gated unit has no bias, cap, accumulation or other activation")
-        return _linear_glu(x, w, out, *glu)
+        if accumulate or softcap is not None or epi != "none" or out.dtype != x.dtype:
+            raise ValueError("linear: a gated unit has no cap, accumulation or other activation")
+        if bias is not None and (bias.dtype != w.dtype or bias.shape != (N,)):
+            raise ValueError("linear: the bias needs the weight's type, one entry per row of the weight")
+        return _linear_glu(x, w, out, bias, *glu)
     if w.shape[1] != K or out.shape[0] != M or out.shape[1] != N:
         raise ValueError(f"linear: shapes {tuple(x.shape)} {tuple(w.shape)} {tuple(out.shape)}")
     if bias is not None and (bias.dtype != w.dtype or bias.shape != (N,) or accumulate):
@@ -327,21 +329,29 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, epi: str = "n
     return out
 
 
-def _linear_glu(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, slope: float, limit: float
-                ) -> torch.Tensor:
+def _linear_glu(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor],
+                slope: float, limit: float, shift: float = 1.0) -> torch.Tensor:
     (M, K), N = x.shape, w.shape[0]
     if w.shape[1] != K or tuple(out.shape) != (M, N // 2):
         raise ValueError(f"linear: shapes {tuple(x.shape)} {tuple(w.shape)} {tuple(out.shape)}")
     if not x.is_cuda:
-        return out.copy_(clamped_glu(x.float() @ w.float().t(), slope, limit).to(out.dtype))
+        z = x.float() @ w.float().t()
+        z = z if bias is None else z + bias.float()
+        return out.copy_(clamped_glu(z, slope, limit, shift).to(out.dtype))
     lib, F = _lib.serving_lib(), ctypes.c_float
+    unit = (F(slope), F(limit), F(shift))
     if x.dtype == torch.float32:
-        rc = lib.cb_linear_f32_grouped(_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), None, 128, _lib.ptr(out),
-                                       out.stride(0), M, N, K, 1, F(slope), F(limit), _lib.stream_ptr())
+        rc = lib.cb_linear_f32_grouped(_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(bias), None, 128,
+                                       _lib.ptr(out), out.stride(0), M, N, K, 1, *unit, _lib.stream_ptr())
         _lib.check_rc(rc, "cb_linear_f32_grouped")
         return out
-    rc = lib.cb_gemm_bf16_blocks(_lib.ptr(x), _lib.ptr(w), _lib.ptr(out), M, N, K, 1, x.stride(0), w.stride(0),
-                                 out.stride(0), None, 128, 1, F(slope), F(limit),
+    if M <= SKINNY_MAX:
+        rc = lib.cb_linear_skinny_glu(_lib.ptr(x), x.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(bias),
+                                      _lib.ptr(out), out.stride(0), N, K, *unit, M, _lib.stream_ptr())
+        _lib.check_rc(rc, "cb_linear_skinny_glu")
+        return out
+    rc = lib.cb_gemm_bf16_blocks(_lib.ptr(x), _lib.ptr(w), _lib.ptr(bias), _lib.ptr(out), M, N, K, 1, x.stride(0),
+                                 w.stride(0), out.stride(0), None, 128, 1, *unit,
                                  _lib.ptr(_lib.status_buffer(x.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_gemm_bf16_blocks")
     return out

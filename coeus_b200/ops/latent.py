@@ -156,6 +156,6 @@ def piece_attention(q: torch.Tensor, kv: torch.Tensor, batch: RaggedBatch, plan:
     rc = _lib.serving_lib().cb_attn_fwd_pieces(
         _p(q), _p(kv), _p(kv[:, heads * P:]), _p(out), T, kv.shape[0], _p(pieces), n_pieces, longest,
         heads, heads, P, P, vdim, q.stride(0), kv.stride(0), kv.stride(0), out.stride(0), _F(scale), None,
-        _p(gate), gate.stride(0) if gate is not None else 0, 1, plan.window or 0, _F(0.0), _F(0.0), 1, None, _F(1.0),
+        _p(gate), gate.stride(0) if gate is not None else 0, 1, plan.window or 0, 0, _F(0.0), _F(0.0), 1, None, _F(1.0),
         _F(0.0), _p(_lib.status_buffer(q.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_attn_fwd_pieces")

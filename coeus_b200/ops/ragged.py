@@ -51,12 +51,14 @@ class AttnPlan:
 
     Under a sliding ``window`` a piece is a run of at most ``WINDOW_PIECE`` rows together with the
     keys its first row sees before it; an entry that continues a sequence gathers its own keys and
-    those of the window before it.  Without ``tiles``, what is no piece goes row by row."""
+    those of the window before it.  The first ``keep`` positions that the window has passed are a run of
+    keys of their own.  Without ``tiles``, what is no piece goes row by row."""
 
     chunk: Optional[int]
     pieces: bool              # whether the layer's sizes allow the piece kernel
     window: Optional[int] = None
     tiles: bool = True
+    keep: int = 0
 
 
 SCAN_MIN = 16         # entries of more tokens than this take the chunked recurrence
@@ -91,15 +93,21 @@ def head_prep(raw: torch.Tensor, koff: int, voff: int, heads: int, kv_heads: int
               batch: "RaggedBatch", rope: Optional[torch.Tensor], k_cache: torch.Tensor,
               v_cache: torch.Tensor, page_table: torch.Tensor, *, interleaved: bool = False,
               unit_eps: Optional[float] = None, q_head: Optional[int] = None,
-              k_rows: Optional[torch.Tensor] = None, v_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+              k_rows: Optional[torch.Tensor] = None, v_rows: Optional[torch.Tensor] = None,
+              eps: float = 0.0, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None,
+              unit_v: bool = False, q_factor: Optional[torch.Tensor] = None) -> torch.Tensor:
     """What stands between the projections ``raw`` (queries at column 0, keys at ``koff``, values at
     ``voff``) and the scores: rotation of the first ``2 * rope.shape[1]`` entries of the q and k heads (pairs
     half a rotation apart, or with ``interleaved`` neighbours), division of q and k by their root mean
     square over ``dim`` (``unit_eps`` inside the root; None: not), the write of k and v into the cache pages
     (and row by row into the first rows of ``k_rows [.., kv_heads, P]`` and ``v_rows``, zeros behind a
     head).  Returns ``q [rows, heads, q_head]``, zeros behind ``dim``.  ``heads`` and ``kv_heads`` count the
-    heads of q and k; v has ``v_cache.shape[2]``."""
-    T, v_heads = raw.shape[0], v_cache.shape[2]
+    heads of q and k; v has ``v_cache.shape[2]``.  ``kv_heads`` 0: queries alone, the cache is left alone.
+
+    With ``q_norm [heads * dim]`` (and ``k_norm``) q and k are RMS-normed over all heads at once in front of
+    the rotation; ``unit_v`` divides each head of v by its root mean square (both with ``eps``); ``q_factor
+    [heads]`` multiplies the queries of a head at the end."""
+    T, v_heads = raw.shape[0], v_cache.shape[2] if kv_heads else 0
     half = rope.shape[1] if rope is not None else 0
     Q = q_head or (dim + 7) // 8 * 8
     q = torch.empty((T, heads, Q), dtype=raw.dtype, device=raw.device)
@@ -115,16 +123,26 @@ def head_prep(raw: torch.Tensor, koff: int, voff: int, heads: int, kv_heads: int
             if unit_eps is not None:
                 x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + unit_eps)
             return x
+        def unit(x):
+            return x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)
+
+        def heads_of(at, n, gain):
+            x = raw[:, at:at + n * dim].float()
+            x = x if gain is None else unit(x) * gain
+            return rotated(x.view(T, n, dim))
         q.zero_()
-        q[..., :dim] = rotated(raw[:, :heads * dim].float().view(T, heads, dim)).to(q.dtype)
-        k = rotated(raw[:, koff:koff + kv_heads * dim].float().view(T, kv_heads, dim))
-        page, at = _cells(page_table, batch)
-        k_cache[page, at, :, :dim] = k.to(k_cache.dtype)
-        v_cache[page, at, :, :vdim] = raw[:, voff:voff + v_heads * vdim].view(T, v_heads, vdim)
+        x = heads_of(0, heads, q_norm)
+        q[..., :dim] = (x if q_factor is None else x * q_factor[:, None]).to(q.dtype)
+        if kv_heads:
+            page, at = _cells(page_table, batch)
+            k_cache[page, at, :, :dim] = heads_of(koff, kv_heads, k_norm).to(k_cache.dtype)
+            v = raw[:, voff:voff + v_heads * vdim].float().view(T, v_heads, vdim)
+            v_cache[page, at, :, :vdim] = (unit(v) if unit_v else v).to(v_cache.dtype)
         return q
     rc = _lib.serving_lib().cb_head_prep(
         _p(raw), raw.stride(0), koff, voff, heads, kv_heads, v_heads, dim, vdim, half, _p(rope),
-        int(interleaved), int(unit_eps is not None), _F(unit_eps or 0.0), _p(q), Q, _p(k_cache),
+        int(interleaved), int(unit_eps is not None), _F(eps if unit_eps is None else unit_eps), _p(q_norm),
+        _p(k_norm), int(unit_v), _p(q_factor), _p(q), Q, _p(k_cache),
         _p(v_cache), k_cache.shape[-1], v_cache.shape[-1], _p(k_rows), _p(v_rows),
         k_rows.shape[2] if k_rows is not None else 0, v_rows.shape[2] if v_rows is not None else 0,
         _p(page_table), page_table.shape[1], k_cache.shape[0], _p(batch.row_slot), _p(batch.pos), T,
@@ -173,6 +191,7 @@ class RaggedBatch:
         if not n or min(lens) < 1:
             raise ValueError("a step needs entries of at least one token")
         self.n, self.T, self.lens = n, sum(lens), lens
+        self.kept: dict = {}         # what a layer leaves for later layers of the same step
         self.pos0_host = [e.pos0 for e in entries]
         self.slots_host = [e.slot for e in entries]
         self.max_ctx = max(e.pos0 + m for e, m in zip(entries, lens))
@@ -215,24 +234,31 @@ class RaggedBatch:
                         continue
                     ahead = min(p0, plan.window - 1)
                     first = r0                             # key row of the entry's first token
+                    kept = min(plan.keep, p0 + lens[i])    # positions 0 .. kept - 1 from this key row on
+                    kept0 = r0
                     if p0:
                         keys = np.arange(p0 - ahead, p0 + lens[i], dtype=np.int32)
+                        if p0 > ahead:
+                            keys = np.concatenate([np.arange(min(kept, p0 - ahead), dtype=np.int32), keys])
                         where.append(np.stack([np.full_like(keys, entries[i].slot), keys], 1))
-                        first = self.T + extra + ahead
+                        kept0 = self.T + extra
                         extra += len(keys)
+                        first = self.T + extra - lens[i]
                     for o in range(0, lens[i], WINDOW_PIECE):
                         before = min(ahead + o, plan.window - 1)
-                        pieces.append((r0 + o, min(WINDOW_PIECE, lens[i] - o), first + o - before, before))
+                        size, unseen = min(WINDOW_PIECE, lens[i] - o), p0 + o - before
+                        pieces.append((r0 + o, size, first + o - before, before, kept0,
+                                       kept if unseen + before + size > plan.window else 0, unseen, 0))
                     continue
                 head, ahead, ps = _cut(plan, p0, lens[i]) if plan.pieces else (lens[i], 0, [])
                 if plan.pieces and head > MIN_PIECE:
                     keys = np.arange(p0 - ahead, p0 + head, dtype=np.int32)
                     where.append(np.stack([np.full_like(keys, entries[i].slot), keys], 1))
-                    pieces.append((r0, head, self.T + extra, ahead))
+                    pieces.append((r0, head, self.T + extra, ahead, 0, 0, 0, 0))
                     extra += len(keys)
                 elif plan.tiles:
                     tiles += [(i, o, min(ATTN_TILE, head - o)) for o in range(0, head, ATTN_TILE)]
-                pieces += [(r0 + o, m, r0 + o, 0) for o, m in ps]
+                pieces += [(r0 + o, m, r0 + o, 0, 0, 0, 0, 0) for o, m in ps]
             tiles.sort(key=lambda t: -(entries[t[0]].pos0 + t[1]))     # the most keys first
             pieces.sort(key=lambda t: -t[1] * (t[1] + 2 * t[3]))
             if pieces:
@@ -283,19 +309,19 @@ class RaggedBatch:
 
 
 def embed_norm(tokens: torch.Tensor, embed: torch.Tensor, weight: Optional[torch.Tensor],
-               width: int, eps: float, out: torch.Tensor) -> torch.Tensor:
-    """Rows of ``embed`` (RMS-normalised with ``weight`` when given) as the fp32 residual stream;
-    columns ``width ..`` of ``out`` are zero."""
+               width: int, eps: float, out: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+    """Rows of ``embed`` (RMS-normalised with ``weight`` when given) times ``scale`` as the fp32 residual
+    stream; columns ``width ..`` of ``out`` are zero."""
     if not out.is_cuda:
         x = embed[tokens.long(), :width].float()
         if weight is not None:
             x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * weight[:width]
         out.zero_()
-        out[:, :width] = x
+        out[:, :width] = x * scale
         return out
     rc = _lib.serving_lib().cb_embed_norm(
         _p(tokens), _p(embed), embed.stride(0), embed.shape[0], _p(weight), _p(out), out.stride(0),
-        out.shape[0], width, _F(eps), int(embed.dtype == torch.float32),
+        out.shape[0], width, _F(eps), _F(scale), int(embed.dtype == torch.float32),
         _p(_lib.status_buffer(out.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "cb_embed_norm")
     return out
@@ -323,11 +349,22 @@ def rms_rows(x: torch.Tensor, w1: torch.Tensor, width: int, eps: float, dtype: t
 @dataclass
 class Spread:
     """A sublayer's result in pieces: row ``t`` is the sum over ``k`` of ``weight[t, k] * rows[slot[t, k]]``
-    (``slot`` int32 and ``weight`` fp32 ``[tokens, top]``, ``rows`` in the activation type)."""
+    (``slot`` int32 and ``weight`` fp32 ``[tokens, top]``, ``rows`` in the activation type); where the slot is
+    negative, row ``t`` of ``own`` stands for it."""
 
     rows: torch.Tensor
     slot: torch.Tensor
     weight: torch.Tensor
+    own: Optional[torch.Tensor] = None
+
+    def sum(self) -> torch.Tensor:
+        v = 0
+        for k in range(self.weight.shape[1]):
+            r = self.rows[self.slot[:, k].clamp_min(0).long()].float()
+            if self.own is not None:
+                r = torch.where(self.slot[:, k, None] < 0, self.own.float(), r)
+            v = v + r * self.weight[:, k, None]
+        return v
 
 
 def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dtype, *,
@@ -336,14 +373,20 @@ def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dty
              shift: Optional[torch.Tensor] = None, before: Optional[torch.Tensor] = None,
              batch: Optional["RaggedBatch"] = None, rows: Optional[torch.Tensor] = None,
              keep: bool = True, casts: Sequence[torch.Tensor] = (),
-             spread: Optional["Spread"] = None
+             spread: Optional["Spread"] = None, y_weight: Optional[torch.Tensor] = None,
+             scale: Optional[torch.Tensor] = None, center: Optional[torch.Tensor] = None,
+             taps: Optional[torch.Tensor] = None
              ) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
     """One pass between two sublayers, ``(x', h)``: ``v = y + bias`` (plus the weighted rows of ``spread``,
     which may also stand alone), RMS-normed with gain ``post`` when
     given; ``x' = x + v`` in fp32 (``v`` alone without ``x``, ``x`` itself without ``y``); ``h`` the RMS
     norm of ``x'`` with ``gain`` in the activation type, shifted by ``h + (h_before - h) * shift`` with
     the previous token's h (``before [slots, ld]`` at an entry's start, which is advanced).  Gains are
-    one number or a vector.  ``rows`` restricts the pass to some rows (``x'`` is not returned then),
+    one number or a vector.  ``y_weight [rows]`` multiplies a row of y before anything is added to it,
+    ``scale`` (a vector) multiplies v; with ``center`` the norm of ``x'`` is a layer norm and this vector is
+    added to it.  With ``taps [n, ld]`` h becomes ``h + conv(h)``, the causal convolution over time of every
+    channel (the last tap for the token itself), whose earlier inputs at an entry's start are ``before
+    [slots, n - 1, ld]`` (advanced too).  ``rows`` restricts the pass to some rows (``x'`` is not returned then),
     ``keep=False`` drops ``x'``; ``casts`` are up to two views that get ``x'`` in the activation type."""
     src = x if x is not None else y
     added = y is not None or spread is not None
@@ -353,22 +396,27 @@ def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dty
     if not src.is_cuda:
         pick = (lambda t: t) if rows is None else (lambda t: t[rows.long()])
 
-        def norm(v, g):
-            return v * torch.rsqrt((v[:, :width] ** 2).mean(-1, keepdim=True) + eps) * g
+        def norm(v, g, c=None):
+            if c is not None:
+                v = v - v[:, :width].mean(-1, keepdim=True)
+            v = v * torch.rsqrt((v[:, :width] ** 2).mean(-1, keepdim=True) + eps) * g
+            return v if c is None else v + c
         out = None if x is None else pick(x)
         if added:
             v = pick(y).float() if y is not None else torch.zeros_like(out)
-            if spread is not None:
-                for k in range(spread.weight.shape[1]):
-                    v = v + pick(spread.rows[spread.slot[:, k].long()].float() * spread.weight[:, k, None])
+            v = v if y_weight is None else v * pick(y_weight)[:, None]
+            v = v if spread is None else v + pick(spread.sum())
             v = v if bias is None else v + bias
             v = v if post is None else norm(v, post)
+            v = v if scale is None else v * scale
             out = v if out is None else out + v
         for c in casts:
             c.copy_(out.to(c.dtype))
         h = None
         if gain is not None:
-            h = norm(out, gain)
+            h = norm(out, gain, center)
+            if taps is not None:
+                h = h + _conv_ref(h, taps, before, batch)
             if shift is not None:
                 prev, r = torch.zeros_like(h), 0
                 prev[1:] = h[:-1]
@@ -383,18 +431,20 @@ def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dty
     x_out = torch.empty((n, ld), dtype=torch.float32, device=src.device) \
         if keep and (added or x is None) else None
     h = torch.empty((n, ld), dtype=dtype, device=src.device) if gain is not None else None
-    shifted = shift is not None
+    shifted = shift is not None or taps is not None
     none = (None,) * 6
     ents = (*batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off)) if shifted else none
     cast = list(casts) + [None] * (2 - len(casts))
-    sp = (None, 0, None, None, 0) if spread is None else (
-        _p(spread.rows), spread.rows.stride(0), _p(spread.slot), _p(spread.weight), spread.slot.shape[1])
+    sp = (None, 0, None, None, 0, None, 0) if spread is None else (
+        _p(spread.rows), spread.rows.stride(0), _p(spread.slot), _p(spread.weight), spread.slot.shape[1],
+        _p(spread.own), spread.own.stride(0) if spread.own is not None else 0)
     rc = _lib.serving_lib().cb_add_norm(
         _p(x), _p(y), _p(bias), _p(post), int(post is not None and post.numel() > 1), _p(x_out), ld,
         y.stride(0) if y is not None else 0, _p(gain), int(gain is not None and gain.numel() > 1), _p(h),
         ld, _p(cast[0]), _p(cast[1]), casts[0].stride(0) if casts else 0, _p(shift), _p(before),
         _p(rows), *ents, batch.n_conv if shifted else n, width, _F(eps), int(dtype == torch.float32),
-        int(y is not None and y.dtype == torch.float32), *sp, _lib.stream_ptr())
+        int(y is not None and y.dtype == torch.float32), *sp, _p(y_weight), _p(scale), _p(center), _p(taps),
+        taps.shape[0] if taps is not None else 0, _lib.stream_ptr())
     _lib.check_rc(rc, "cb_add_norm")
     return (x_out if x_out is not None else (x if keep else None)), h
 
@@ -574,7 +624,7 @@ def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, e
 def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                      page_table: torch.Tensor, batch: RaggedBatch, heads: int, kv_heads: int,
                      dim: int, vdim: int, scale: float, out: torch.Tensor, *,
-                     chunk: Optional[int] = None, window: Optional[int] = None,
+                     chunk: Optional[int] = None, window: Optional[int] = None, keep: int = 0,
                      softcap: Optional[float] = None, score_max: float = 0.0, maps: int = 1,
                      map_weight: Optional[torch.Tensor] = None, map_factor: float = 1.0,
                      eps: float = 0.0, sink: Optional[torch.Tensor] = None,
@@ -582,10 +632,10 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      max_ctx: Optional[int] = None,
                      k_rows: Optional[torch.Tensor] = None,
                      v_rows: Optional[torch.Tensor] = None,
-                     plan: Optional[AttnPlan] = None) -> torch.Tensor:
+                     plan: Optional[AttnPlan] = None, gathered: bool = False) -> torch.Tensor:
     """Causal attention of every query row over the cached keys of its own sequence, restricted to
     the row's chunk (positions with the same ``pos // chunk``) when ``chunk`` is given, or to itself and
-    the ``window - 1`` positions before it.  Scores ``s`` become ``softcap * tanh(s / softcap)``
+    the ``window - 1`` positions before it (and the sequence's first ``keep`` positions).  Scores ``s`` become ``softcap * tanh(s / softcap)``
     (``score_max`` bounds ``|s|``, 0 where no bound is known).  ``sink``
     (fp32 ``[heads]``) is a logit that enters the softmax denominator only; ``gate`` multiplies by its
     sigmoid: a view whose column ``h`` belongs to head ``h``, or (``gate_wide``) a view like ``out``.  Query
@@ -594,7 +644,8 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     view; ``max_ctx`` bounds the keys of any row (it only chooses how many CTAs share a row).  With
     row-wise ``k_rows`` and ``v_rows`` at hand (:meth:`RaggedBatch.kv_rows` rows of ``[kv_heads, P]``,
     this step's filled in; q then has the keys' head distance), the pieces of ``plan`` go through
-    the tcgen05 kernel; the default plan has pieces when the buffers are given.
+    the tcgen05 kernel; the default plan has pieces when the buffers are given (``gathered``: so are the
+    cached rows behind this step's).
 
     With two ``maps`` a head has two queries and its key head two keys (``q [rows, heads * 2, Q]``,
     ``k_cache [pages, PAGE, kv_heads * 2, dim_p]``, map 0 first) over the same values; with their outputs
@@ -617,7 +668,7 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             j = torch.arange(n)
             lo = pos // chunk * chunk if chunk else torch.zeros_like(pos)
             lo = torch.clamp(pos + 1 - window, min=0) if window else lo
-            ok = (j[None] <= pos[:, None]) & (j[None] >= lo[:, None])
+            ok = (j[None] <= pos[:, None]) & ((j[None] >= lo[:, None]) | (j[None] < keep))
             s = s.masked_fill(~ok, float("-inf"))
             top = s.amax(-1, keepdim=True)
             if sink is not None:
@@ -639,21 +690,21 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     st = _p(_lib.status_buffer(q.device))
     lib = _lib.serving_lib()
     spec = _AttnSpec(heads, kv_heads, dim, vdim, k_cache.shape[-1], v_cache.shape[-1], chunk or 0,
-                     window or 0, maps, int(gate_wide), scale, softcap or 0.0, map_factor, eps)
+                     window or 0, keep, maps, int(gate_wide), scale, softcap or 0.0, map_factor, eps)
     common = (_p(q), q.shape[2], _p(k_cache), _p(v_cache), _p(page_table), page_table.shape[1],
               k_cache.shape[0], ctypes.byref(spec), _p(sink), _p(gate),
               gate.stride(0) if gate is not None else 0, _p(map_weight), _p(out), out.stride(0))
     n, rows = batch.n_rows, batch.rows
     if batch.n_big:
         n_tiles, n_pieces, longest, extra, pieces, where, t_entry, t_off, t_len = batch.plan(
-            plan or AttnPlan(chunk, k_rows is not None, window))
+            plan or AttnPlan(chunk, k_rows is not None, window, keep=keep))
         if not n_tiles and not n_pieces:       # sizes that neither kernel takes
             n, rows = T, batch.every_row
         if n_tiles:
             rc = lib.cb_ragged_attn_tiles(*common, *batch.entry_args(), _p(t_entry), _p(t_off),
                                           _p(t_len), n_tiles, st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_ragged_attn_tiles")
-        if extra:
+        if extra and not gathered:
             rc = lib.cb_kv_gather(_p(k_cache), _p(v_cache), kv_heads * maps, kv_heads, k_cache.shape[-1],
                                   v_cache.shape[-1], _p(page_table), page_table.shape[1],
                                   k_cache.shape[0], _p(where), extra, _p(k_rows[T:]), _p(v_rows[T:]),
@@ -664,14 +715,14 @@ def ragged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                 _p(q), _p(k_rows), _p(v_rows), _p(out), T, k_rows.shape[0], _p(pieces), n_pieces,
                 longest, heads, kv_heads, k_rows.shape[2], v_rows.shape[2], vdim, q.stride(0),
                 k_rows.stride(0), v_rows.stride(0), out.stride(0), _F(scale), _p(sink), _p(gate),
-                gate.stride(0) if gate is not None else 0, int(gate_wide), window or 0,
+                gate.stride(0) if gate is not None else 0, int(gate_wide), window or 0, keep,
                 _F(softcap or 0.0), _F(score_max), maps, _p(map_weight), _F(map_factor), _F(eps), st, _lib.stream_ptr())
             _lib.check_rc(rc, "cb_attn_fwd_pieces")
     if n:
         per = heads // kv_heads * maps
         ctas = n * kv_heads * ((per + 15) // 16)
         ctx = max_ctx or batch.max_ctx
-        ctx = min([ctx] + [c for c in (chunk, window) if c])
+        ctx = min([ctx] + [c + keep for c in (chunk, window) if c])
         # a CTA takes 128 keys at a time
         splits = max(1, min(16, (2 * 148 + ctas - 1) // ctas, (ctx + 127) // 128))
         part_o = part_ml = None
@@ -689,5 +740,5 @@ class _AttnSpec(ctypes.Structure):
     """``RaggedSpec`` of ``csrc/ragged_attn.cu``."""
 
     _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "dim", "vdim", "dim_p", "vdim_p", "chunk",
-                                            "window", "maps", "gate_wide")] + \
+                                            "window", "keep", "maps", "gate_wide")] + \
                [(n, ctypes.c_float) for n in ("scale", "softcap", "map_factor", "eps")]
