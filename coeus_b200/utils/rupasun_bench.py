@@ -47,7 +47,7 @@ def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> Li
     lm = H.HybridLM.random(config(W, 3, nh, kv))
     dense, lc = lm.layers[0], lm.layers[2]
     ex, moe = lc.experts, lc.experts.spec
-    r = X.Routing(moe.experts, moe.top, moe.groups, moe.keep, moe.scale)
+    r = ex.routing
     ff, fs = moe.expert.ff, moe.shared.ff
     for phase, B, S, at in (("prefill 8x2048", 8, 2048, 0), ("decode 64", 64, 1, CONTEXT),
                             ("decode 16", 16, 1, CONTEXT)):

@@ -196,9 +196,9 @@ MODEL_CHECKS = [check_whole_prompt, check_token_by_token, check_portions, check_
 CUTS = (((1, 40), (2, 1), (1, 1), (70, 2), (127, 1), (9, 165)), ((3, 130), (5, 6), (202, 74)))
 
 
-def single_mixer(spec, architecture, device, dtype, seed):
+def single_mixer(spec, architecture, device, dtype, seed, **kw):
     """A model of one layer with this mixer alone, and the mixer's weights."""
-    cfg = H.HybridConfig(16, 16, (H.LayerSpec(spec, None),), 1e-4, architecture=architecture)
+    cfg = H.HybridConfig(16, 16, (H.LayerSpec(spec, None),), 1e-4, architecture=architecture, **kw)
     w = H.random_state(cfg, seed, dtype=torch.float32)
     w = {n: t.bfloat16().float() for n, t in w.items()}
     lm = H.HybridLM(cfg, w, device, dtype)
@@ -215,6 +215,8 @@ def drive(lm, raws, cuts, run):
     layer, outs, at = lm.layers[0], [[], []], [0, 0]
     for s in (1, 2, 0, 2, 1):         # pages in an order that is not ascending
         eng.cache.reserve(s, min(eng.cache.page_table.shape[1], len(eng.cache.owned.get(s, [])) + 3) * PAGE)
+    for s, raw in ((2, raws[0]), (0, raws[1])):
+        eng.cache.reserve(s, raw.shape[0])
     for cut in cuts:
         b = eng._batch([R.Entry(slot, at[s], [0] * cut[s]) for s, slot in ((0, 2), (1, 0))])
         raw = torch.cat([raws[s][at[s]:at[s] + cut[s]] for s in (0, 1)])

@@ -26,10 +26,9 @@ def conv_in(h, taps):
     position itself."""
     T, n = h.shape[0], taps.shape[1]
     out = h.clone()
-    for t in range(T):
-        for j in range(n):
-            if t - n + 1 + j >= 0:
-                out[t] = out[t] + taps[:, j] * h[t - n + 1 + j]
+    for j in range(n):
+        back = n - 1 - j
+        out[back:] = out[back:] + taps[:, j] * h[:max(T - back, 0)]
     return out
 
 
@@ -48,12 +47,13 @@ def rotate_pairs(x, dims, base):
 def visible(i, j, size=None, keep=0):
     """Whether position ``i`` sees position ``j``, under a sliding window of ``size`` positions beside which the
     first ``keep`` positions stay visible."""
-    return j <= i and (size is None or i - j < size or j < keep)
+    return (j <= i) & ((i - j < (size or math.inf)) | (j < keep))
 
 
 @functools.lru_cache(maxsize=None)
 def visibility(T, size=None, keep=0):
-    return torch.tensor([[visible(i, j, size, keep) for j in range(T)] for i in range(T)])
+    i = torch.arange(T)
+    return visible(i[:, None], i[None], size, keep)
 
 
 def weights_beside_one(s):

@@ -153,7 +153,7 @@ def check_route(device, dtype, tol):
             router = torch.zeros(m.experts + -m.experts % 8, W)
             router[:m.experts, 3:3 + m.experts] = torch.eye(m.experts)
             h, router = h.to(dtype).to(device), router.to(dtype).to(device)
-            c = X.route(h, router, X.Routing(m.experts, m.top, m.groups, m.keep, m.scale))
+            c = X.route(h, router, m.routing())
             z = h.double().cpu()[:, 3:3 + m.experts]
             for t in range(T):
                 want, weight = plain.choose(z[t], m.top, m.groups, m.keep, m.scale)
