@@ -203,7 +203,7 @@ class HybridEngine(InferenceEngine):
                                  for h, p in ((kh, q_head), (s.kv_heads, v_head))))
             if n in self._shared:
                 b.kept[n] = rows
-        pieces = b.kv_rows(plan) > 0
+        pieces = b.kv_rows(plan)       # later rows of the buffers may hold nothing: they stay out of sight
         q = R.head_prep(raw, layer.seg.get("k", 0), layer.seg.get("v", 0), s.heads * s.maps, kh if own else 0,
                         s.dim, s.vdim, b, rope.get(layer.rope_key), c.k[i], c.v[i], c.page_table,
                         interleaved=s.interleaved, unit_eps=eps if s.unit_qk else None,
@@ -215,7 +215,7 @@ class HybridEngine(InferenceEngine):
             out[:, :layer.out_dim], window=s.window, keep=s.keep_first, softcap=s.softcap, score_max=s.score_max,
             maps=s.maps, map_weight=layer.map_weight, map_factor=1.0 - s.diff if s.maps == 2 else 1.0, eps=eps,
             sink=layer.sink, gate=raw[:, layer.seg["g"]:] if s.gated else None, gate_wide=True, max_ctx=max_ctx,
-            k_rows=rows.k if pieces else None, v_rows=rows.v if pieces else None, plan=plan,
+            k_rows=rows.k[:pieces] if pieces else None, v_rows=rows.v[:pieces] if pieces else None, plan=plan,
             gathered=rows.gathered == plan)
         if pieces:
             rows.gathered = plan

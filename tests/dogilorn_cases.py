@@ -68,7 +68,7 @@ def levels(m, correction, g, scales=(1.0,), margin=None):
     margin = margin or 0.05 / m.outputs
     for _ in range(5000):
         z = torch.linspace(-1.5, 1.5, m.outputs)[torch.randperm(m.outputs, generator=g)]
-        z = z + 0.3 / m.outputs * torch.randn(m.outputs, generator=g)
+        z = (z + 0.3 / m.outputs * torch.randn(m.outputs, generator=g)).bfloat16().float()
         if all(sure(c * z, correction, m, margin) for c in scales):
             return z
     raise AssertionError("no logits with a clear choice")
@@ -227,15 +227,11 @@ def check_route(device, dtype, tol):
             h, router = h.to(dtype).to(device), router.to(dtype).to(device)
             c = X.route(h, router, r, corr.to(device))
             z = h.double().cpu()[:, 3:3 + n]
-            clear = 0
             for t in range(T):
                 want, weight = plain.choose(z[t], corr.double(), m.top, m.groups, m.keep)
                 got = dict(zip(c.expert[t].tolist(), c.weight[t].tolist()))
-                if sure(z[t], corr.double(), m, 1e-5):
-                    clear += 1
-                    assert set(got) == set(want), (i, t)
-                    assert all(abs(got[e] - float(x)) < 2e-6 for e, x in zip(want, weight)), (i, t)
-            assert clear > 0.8 * T
+                assert set(got) == set(want), (i, t)
+                assert all(abs(got[e] - float(x)) < 2e-6 for e, x in zip(want, weight)), (i, t)
             if r.shared_gate:
                 gate = torch.sigmoid(h.double().cpu() @ router[n].double().cpu())
                 assert float((c.shared.double().cpu() - gate).abs().max()) < 2e-5
@@ -266,12 +262,10 @@ def check_experts(device, dtype, tol):
             for t in range(T):
                 h[t, :n] = levels(m, corr.float(), g, margin=2e-3 / n)
             h = h.to(dtype)
-            clear = torch.tensor([sure(h[t, :n].double(), corr, m, 1e-5) for t in range(T)])
             want = plain.experts(h.double(), d, "l0.mlp.", spec)
             hp = torch.nn.functional.pad(h, (0, layer.wp - W)).to(device)
             got = R.add_norm(torch.zeros((T, layer.wp), device=device), W, 1e-4, dtype, **eng._experts(layer, hp))[0]
-            assert clear.double().mean() > 0.8
-            assert rel(got[:, :W].cpu()[clear], want[clear]) < tol, (i, T, rel(got[:, :W], want))
+            assert rel(got[:, :W], want) < tol, (i, T, rel(got[:, :W], want))
 
 
 def check_linear_glu(device, dtype, tol):
