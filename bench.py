@@ -4,7 +4,7 @@
     python bench.py --gpus N --steps K --warmup W            # this framework
     python bench.py --impl reference ...                     # the unmodified reference
     python bench.py --impl torch ...                         # same model on stock PyTorch
-    python bench.py --serving rupasun [--kernels]            # serving throughput of that design
+    python bench.py --serving dogilorn [--kernels]           # serving throughput of that design
 
 Metric: train tokens/s (device-timed with CUDA events, max over ranks), whole-job aggregate.
 Config: decoder-only, vocab 32000, d_model 1024, 16 layers, 16 heads, FFN 4096, sequences of
@@ -200,7 +200,7 @@ def main() -> int:
     ap.add_argument("--no-compare", action="store_true",
                     help="skip the stock-PyTorch comparator that the coeus arm times afterwards "
                          "in the same process to fill vs_baseline")
-    ap.add_argument("--serving", choices=["sapasun", "bananex", "rupasun"], default=None,
+    ap.add_argument("--serving", choices=["sapasun", "bananex", "rupasun", "dogilorn"], default=None,
                     help="instead of the training benchmark: prefill and decode throughput of this "
                          "design beside the closest decoder of equal size (one GPU)")
     ap.add_argument("--kernels", action="store_true",

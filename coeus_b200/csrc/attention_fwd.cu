@@ -28,7 +28,9 @@
 // every pair of steps its value tile.  At the end each warpgroup takes half of the columns of
 // o = a0 - w a1, and the two meet at two barriers: one when both results are complete, one for the sum of
 // squares of o, which is divided by its root mean square.  KEPT (with a window): the first positions of the
-// sequence stay visible behind the window; their keys are tiles of their own in front of an item's others.
+// sequence stay visible behind the window; their keys are tiles of their own.  They come right before the
+// first key tile of B: from there on A and B take turns, so that no tile sits out while a buffer that its
+// last step used goes round (the wait before rescaling O counts on that).
 // Every wait is bounded; a wait that runs out records a status code and the CTA leaves.
 #include <cmath>
 
@@ -148,7 +150,8 @@ struct AFWalk {
   int lo0, lo1, window;  // first key tile of A / B that a row's window reaches
   int kv_seq;            // how many (item, j) groups came before this one: the K/V ring position
   bool valid;
-  int4 kept;             // KEPT: the piece's second quadruple; its kt tiles are j = -kt .. -1
+  int4 kept;             // KEPT: the piece's second quadruple; its kt tiles are j = -kt .. -1, between
+                         // lo1 - 1 and lo1
   int kt;
 
   __device__ int first_row(const AttnFwdArgs& p) const { return PIECES ? piece.x : b * p.S; }
@@ -158,8 +161,11 @@ struct AFWalk {
   __device__ int keys_ahead() const { return PIECES ? piece.w : 0; }   // keys before query 0's own
   // KEPT: first position in the window of query q
   __device__ int low_position(int q) const { return kept.z + max(0, piece.w + q + 1 - window); }
-  __device__ int first_tile() const { return KEPT && kt > 0 ? -kt : lo0; }
-  __device__ int next_tile(int i) const { return KEPT && i == -1 ? lo0 : i + 1; }
+  __device__ int first_tile() const { return KEPT && kt > 0 && lo0 >= lo1 ? -kt : lo0; }
+  __device__ int next_tile(int i) const {
+    if (KEPT && i == -1) return lo1;
+    return KEPT && kt > 0 && i + 1 == lo1 && i >= 0 ? -kt : i + 1;
+  }
   __device__ int tile_row(const AttnFwdArgs& p, int i) const {
     return KEPT && i < 0 ? kept.x + (i + kt) * bkv : first_key(p) + i * bkv;
   }
@@ -236,8 +242,10 @@ struct AFWalk {
     next_item();
   }
   __device__ bool last_of_kv() const { return t == 1 || !b_has(j); }   // last tile using K_j / V_j
-  __device__ bool first_of_tile() const { return j == (KEPT && kt > 0 ? -kt : t ? lo1 : lo0); }
-  __device__ bool last_of_tile() const { return j == (t ? n1 : n0) - 1; }
+  __device__ bool first_of_tile() const { return j == (t == 0 ? first_tile() : KEPT && kt > 0 ? -kt : lo1); }
+  __device__ bool last_of_tile() const {
+    return j == (t ? n1 : KEPT && kt > 0 && n0 <= lo1 ? 0 : n0) - 1;     // tile A may end with kept keys
+  }
 };
 
 template <int DQ, int DV, bool POLY, bool DROP, bool PIECES, int CAP, bool DIFF, bool KEPT>

@@ -1,11 +1,12 @@
 """Serving throughput of a design of mixed layers beside the framework's closest model at equal size,
-and its kernels one by one against the roofline (``python bench.py --serving sapasun|bananex|rupasun
-[--kernels]``; the kernels of Bananex are in :mod:`coeus_b200.utils.bananex_bench`, those of Rupasun in
-:mod:`coeus_b200.utils.rupasun_bench`).
+and its kernels one by one against the roofline (``python bench.py --serving
+sapasun|bananex|rupasun|dogilorn [--kernels]``; designs behind the first are in :mod:`coeus_b200.utils.bananex_bench`,
+:mod:`coeus_b200.utils.rupasun_bench` and :mod:`coeus_b200.utils.dogilorn_bench`).
 
 The closest model is the RMSNorm / SwiGLU / rotary decoder with grouped-query attention: same
 width, depth, heads and vocabulary, the feed-forward as wide as gives the same parameters per
-layer (three matrices of 8/3 width against two of 4 width; for a mixture of experts: per token).  Weights are random.  Times are CUDA
+layer (three matrices of 8/3 width against two of 4 width; for a mixture of experts: per token).  Dogilorn
+also runs beside a Rupasun model of the same window and experts.  Weights are random.  Times are CUDA
 events around whole engine calls (prompt batches, decode steps), after warm-up; every call streams
 weights and caches far above the L2 cache.  The kernel table flushes L2 between launches.
 """
@@ -104,7 +105,8 @@ def recorder(rows: List[Dict], only: str, iters: int) -> Callable:
     return rec
 
 
-def closest_kernels(rec, phase: str, B: int, S: int, at: int, W: int, nh: int, kv: int, c) -> None:
+def closest_kernels(rec, phase: str, B: int, S: int, at: int, W: int, nh: int, kv: int, c,
+                    label: str = "closest: ") -> None:
     """The closest model's kernels at width ``W``; ``c`` is a cache of ``kv`` heads of ``HEAD``."""
     from ..ops import attention as A
     from ..ops import decode as D
@@ -118,30 +120,30 @@ def closest_kernels(rec, phase: str, B: int, S: int, at: int, W: int, nh: int, k
         return torch.randn(shape, device=dev, dtype=torch.float32).to(torch.bfloat16)
     q = t(T, nh, d)
     hx, wn = t(T, W), t(W)
-    rec("closest: norm_fwd", phase, lambda: N.norm_fwd(hx, wn, None, 1e-5, True), bytes_=T * W * 4)
+    rec(label + "norm_fwd", phase, lambda: N.norm_fwd(hx, wn, None, 1e-5, True), bytes_=T * W * 4)
     w1 = t(W, qkv)
     if S > 1:
-        rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), flops=2 * T * W * qkv)
+        rec(label + "linear qkv", phase, lambda: G.linear_fwd(hx, w1), flops=2 * T * W * qkv)
         kk, vv = t(T, kv * d), t(T, kv * d)
-        rec("closest: attention", phase, lambda: A.attention_fwd(q.view(T, -1), kk, vv, B, S, nh, d, causal=True),
+        rec(label + "attention", phase, lambda: A.attention_fwd(q.view(T, -1), kk, vv, B, S, nh, d, causal=True),
             flops=4 * B * S * S / 2 * nh * d)
     else:
-        rec("closest: linear qkv", phase, lambda: G.linear_fwd(hx, w1), bytes_=W * qkv * 2)
+        rec(label + "linear qkv", phase, lambda: G.linear_fwd(hx, w1), bytes_=W * qkv * 2)
         ctx = torch.full((B,), CONTEXT, dtype=torch.int32, device=dev)
         pages = (CONTEXT + 63) // 64
         kc, vc = t(B * pages, 64, kv, d), t(B * pages, 64, kv, d)
         pt = torch.arange(B * pages, dtype=torch.int32, device=dev).view(B, pages)
-        rec("closest: attention", phase, lambda: D.decode_attention(q.view(T, -1), kc, vc, pt, ctx, nh, d, nkv=kv),
+        rec(label + "attention", phase, lambda: D.decode_attention(q.view(T, -1), kc, vc, pt, ctx, nh, d, nkv=kv),
             bytes_=B * CONTEXT * kv * d * 2 * 2)
     buf = t(T, qkv)
     pos = torch.full((B,), at, dtype=torch.int32, device=dev)
-    rec("closest: rope", phase, lambda: E.rope_(buf, nh + kv, d, S, pos_dev=pos if S == 1 else None),
+    rec(label + "rope", phase, lambda: E.rope_(buf, nh + kv, d, S, pos_dev=pos if S == 1 else None),
         bytes_=T * (nh + kv) * d * 4)
-    rec("closest: kv_write", phase, lambda: D.kv_write(
+    rec(label + "kv_write", phase, lambda: D.kv_write(
         buf[:, nh * d:(nh + kv) * d], buf[:, (nh + kv) * d:], c.k[0], c.v[0], c.page_table, pos, S,
         kv, d), bytes_=T * kv * d * 2 * 4)
     gu = t(T, 2 * (8 * W // 3 // 128 * 128))
-    rec("closest: swiglu", phase, lambda: E.swiglu_fwd(gu), bytes_=gu.numel() * 3)
+    rec(label + "swiglu", phase, lambda: E.swiglu_fwd(gu), bytes_=gu.numel() * 3)
 
 
 def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> List[Dict]:
@@ -245,29 +247,30 @@ def kernel_table(size: str = "1b-layers", only: str = "", iters: int = 10) -> Li
     return rows
 
 
-DESIGNS = ("sapasun", "bananex", "rupasun")
+DESIGNS = ("sapasun", "bananex", "rupasun", "dogilorn")
 
 
 def bench_of(design: str):
     """``(config, kernel_table)`` of a design."""
-    from . import bananex_bench, rupasun_bench
+    from . import bananex_bench, dogilorn_bench, rupasun_bench
     return {"sapasun": (sapasun_config, kernel_table),
             "bananex": (bananex_bench.config, bananex_bench.kernel_table),
-            "rupasun": (rupasun_bench.config, rupasun_bench.kernel_table)}[design]
+            "rupasun": (rupasun_bench.config, rupasun_bench.kernel_table),
+            "dogilorn": (dogilorn_bench.config, dogilorn_bench.kernel_table)}[design]
 
 
 def run(design: str, steps: int = 20, warmup: int = 3, kernels: bool = False, sampler=None) -> None:
     """One JSON line per size and model, then (``kernels``) one per kernel."""
     from ..ops import _lib
+    from .dogilorn_bench import closest_config as closest_hybrid
     config, table = bench_of(design)
+    models = {design: lambda size: H.HybridLM.random(config(*size))}
+    if design == "dogilorn":
+        models["closest: rupasun"] = lambda size: H.HybridLM.random(closest_hybrid(*size))
+    models["closest"] = lambda size: DecoderLM(closest_config(*size), "cuda", training=False)
     for name, size in SIZES.items():
-        for which in (design, "closest"):
-            if which == design:
-                cfg = config(*size)
-                model = H.HybridLM.random(cfg)
-            else:
-                cfg = closest_config(*size)
-                model = DecoderLM(cfg, "cuda", training=False)
+        for which, make in models.items():
+            model = make(size)
             s = sampler() if sampler is not None else None
             if s is not None:
                 s.start()

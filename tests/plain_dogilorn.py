@@ -71,7 +71,7 @@ def attend(q, k, v, scale, temp, size=None, keep=0):
     out = []
     for h in range(H):
         s = (q[:, h] @ k[:, h // per].T) * scale * temp[h]
-        s = s.masked_fill(~visibility(T, size, keep), -math.inf)
+        s = s.masked_fill(~visibility(T, size, keep).to(s.device), -math.inf)
         out.append(weights_beside_one(s) @ v[:, h // per])
     return torch.stack(out, 1)
 
