@@ -16,14 +16,13 @@
 // sequence's start.  The block of an entry's first tile alone reads the state, and replaces it at
 // its end.
 //
-// With a convolution a block takes such a tile too, in two phases: its warps take the rows, and leave x and
-// the rows' statistics; then its threads take the columns, walk along the rows and keep the last h in
-// registers.  The rows in front of the tile go through shared memory.
+// With a convolution a first pass over rows leaves x and the rows' statistics; a second one takes columns of
+// such a tile, walks along its rows and keeps the last h in registers.  When every entry is one token, one
+// pass does, which finds the earlier h in the state.
 #include "ragged.cuh"
 
 namespace cb {
 
-constexpr int CN_SMEM = 208 * 1024;
 constexpr int SHIFT_TILE = 16;     // tokens per block with a shift (the convolutions' tile)
 
 struct AddNorm {
@@ -55,8 +54,10 @@ struct AddNorm {
   const float* y_weight;   // [rows] or null
   const float* scale;      // [ld] or null
   const float* center;     // [ld] or null
-  const float* taps;       // [n_taps, ld] or null; before is then [slots, n_taps - 1, ld]
+  const float* taps;       // [n_taps, ld] or null; before is then [slots, n_taps - 1, ld], and without
+                           // tile_entry every entry is one token
   int n_taps;
+  float2* stats;           // [rows] mean and 1 / deviation, between the two passes of a convolution
   int width;
   float eps;
 };
@@ -108,7 +109,11 @@ __device__ __forceinline__ float squares_about(const float* f, float mean, int c
   return s;
 }
 
-template <typename T, typename Y, int KEEP>
+// A row per block; a tile with a shift; a row, with the convolution of entries of one token; rows whose
+// statistics stand for h.
+enum : int { AN_ROWS = 0, AN_SHIFT = 1, AN_TOKEN = 2, AN_STATS = 3 };
+
+template <typename T, typename Y, int KEEP, int MODE>
 __global__ void __launch_bounds__(512) add_norm_kernel(const AddNorm p) {
   __shared__ float red[32];
   const int nv = p.ld / 8;
@@ -193,6 +198,10 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const AddNorm p) {
     }
     s = block_sum(s, red);
     rs = 1.0f / sqrtf(s / p.width + p.eps);
+    if constexpr (MODE == AN_STATS) {
+      if (threadIdx.x == 0) p.stats[row] = make_float2(mean, rs);
+      return;
+    }
     if (!p.gain_vec) rs *= *p.gain;
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
@@ -218,18 +227,46 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const AddNorm p) {
   };
 
   float f[KEEP][8];
-  if (p.shift == nullptr) {
+  if constexpr (MODE != AN_SHIFT) {
     const int row = p.rows != nullptr ? p.rows[blockIdx.x] : blockIdx.x;
     stream(row, f, true);
-    if (p.gain == nullptr) return;
+    if (MODE == AN_STATS || p.gain == nullptr) return;
+    if constexpr (MODE == AN_TOKEN) {
+      const int back = p.n_taps - 1;
+      const bool has = p.e.pos0[row] > 0;
+      float* state = p.before + static_cast<size_t>(p.e.slot[row]) * back * p.ld;
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        if (v >= nv) continue;
+        float w[8], o[8], prev[8];
+        load_vec<8>(p.taps + static_cast<size_t>(back) * p.ld + v * 8, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = f[i][e] + w[e] * f[i][e];
+        for (int k = 0; k < back; ++k) {                 // oldest first; each moves one place
+          if (has) {
+            load_vec<8>(state + static_cast<size_t>(k) * p.ld + v * 8, prev);
+          } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) prev[e] = 0.f;
+          }
+          load_vec<8>(p.taps + static_cast<size_t>(k) * p.ld + v * 8, w);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) o[e] += w[e] * prev[e];
+          if (k > 0) store_vec<8>(state + static_cast<size_t>(k - 1) * p.ld + v * 8, prev);
+        }
+        if (back > 0) store_vec<8>(state + static_cast<size_t>(back - 1) * p.ld + v * 8, f[i]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[i][e] = o[e];
+      }
+    }
     T* dst = static_cast<T*>(p.h) + static_cast<size_t>(blockIdx.x) * p.ldh;
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
       const int v = threadIdx.x + i * blockDim.x;
       if (v < nv) store_vec<8>(dst + v * 8, f[i]);
     }
-    return;
-  }
+  } else {
   const int e = p.tile_entry[blockIdx.x], off = p.tile_off[blockIdx.x];
   const int row0 = p.e.row0[e], len = p.e.len[e], slot = p.e.slot[e];
   float* state = p.before + static_cast<size_t>(slot) * p.ld;
@@ -272,137 +309,58 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const AddNorm p) {
     const int v = threadIdx.x + i * blockDim.x;
     if (v < nv) store_vec<8>(state + v * 8, prev[i]);
   }
+  }
 }
 
-// ------------------------------------------------------------------------- with a convolution
-constexpr int CN_THREADS = 256;
-constexpr int CN_KEEP = 8;         // vectors of eight that a lane keeps of a row
+// ------------------------------------------------------------------------------- the convolution
+constexpr int CN_THREADS = 128;    // columns / 8 of a block
+constexpr int CN_AHEAD = 4;        // rows loaded ahead
 
-struct RowStats {
-  float mean, rs;
-};
-
-// One warp, one row: x with the sublayer's result to dst (not when the stream itself is the source and the
-// same), and the row's statistics.
-template <typename T, typename Y>
-__device__ __forceinline__ RowStats conv_row(const AddNorm& p, int row, float* dst) {
-  const int lane = threadIdx.x & 31, nv = p.ld / 8;
-  const bool added = p.y != nullptr || p.spread != nullptr;
-  const float* src = p.x + static_cast<size_t>(row) * p.ld;
-  auto make = [&](int v, float* f) {
-    if (added) {
-      sublayer_result<T, Y>(p, row, v, f);
-      if (p.scale != nullptr) {
-        float c[8];
-        load_vec<8>(p.scale + v * 8, c);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) f[e] *= c[e];
-      }
-    } else {
-#pragma unroll
-      for (int e = 0; e < 8; ++e) f[e] = 0.f;
-    }
-    if (p.x != nullptr) {
-      float a[8];
-      load_vec<8>(src + v * 8, a);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) f[e] += a[e];
-    }
-    if (dst != nullptr) store_vec<8>(dst + v * 8, f);
-  };
-  float f[CN_KEEP][8], s = 0.f;
-#pragma unroll
-  for (int i = 0; i < CN_KEEP; ++i) {
-    const int v = lane + 32 * i;
-    if (v >= nv) continue;
-    make(v, f[i]);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) s += f[i][e];
-  }
-  for (int v = lane + 32 * CN_KEEP; v < nv; v += 32) {
-    float g[8];
-    make(v, g);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) s += g[e];
-  }
-  RowStats r = {0.f, 0.f};
-  if (p.center != nullptr) r.mean = warp_sum(s) / p.width;
-  s = 0.f;
-#pragma unroll
-  for (int i = 0; i < CN_KEEP; ++i) {
-    const int v = lane + 32 * i;
-    if (v < nv) s += squares_about(f[i], r.mean, v * 8, p.width);
-  }
-  const float* again = dst != nullptr ? dst : src;      // this lane's own writes
-  for (int v = lane + 32 * CN_KEEP; v < nv; v += 32) {
-    float g[8];
-    load_vec<8>(again + v * 8, g);
-    s += squares_about(g, r.mean, v * 8, p.width);
-  }
-  r.rs = 1.0f / sqrtf(warp_sum(s) / p.width + p.eps);
-  return r;
-}
-
-// Columns of the norm's gain and center.
-__device__ __forceinline__ void norm_vectors(const AddNorm& p, int v, float* g, float* c) {
+// One thread: eight columns of a tile of tokens of one entry, from x and the rows' statistics.  HIST > 0: the
+// last HIST >= n_taps - 1 tokens' h stay in registers; 0: they are read again.
+template <typename T, int HIST>
+__global__ void __launch_bounds__(CN_THREADS) conv_pass_kernel(const AddNorm p) {
+  const int v = blockIdx.y * CN_THREADS + threadIdx.x;
+  if (v >= p.ld / 8) return;
+  const int back = p.n_taps - 1;
+  const int e = p.tile_entry[blockIdx.x], off = p.tile_off[blockIdx.x];
+  const int row0 = p.e.row0[e], len = p.e.len[e], t1 = min(off + SHIFT_TILE, len);
+  const bool has = p.e.pos0[e] > 0;
+  const float* src = (p.x_out != nullptr ? p.x_out : p.x) + static_cast<size_t>(row0) * p.ld + v * 8;
+  const float2* stats = p.stats + row0;
+  float* state = p.before + static_cast<size_t>(p.e.slot[e]) * back * p.ld + v * 8;
+  T* dst = static_cast<T*>(p.h) + static_cast<size_t>(row0) * p.ldh + v * 8;
+  float g[8], c[8];
   if (p.gain_vec) {
     load_vec<8>(p.gain + v * 8, g);
   } else {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) g[e] = *p.gain;
+    for (int k = 0; k < 8; ++k) g[k] = *p.gain;
   }
   if (p.center != nullptr) {
     load_vec<8>(p.center + v * 8, c);
   } else {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) c[e] = 0.f;
+    for (int k = 0; k < 8; ++k) c[k] = 0.f;
   }
-}
-
-// One warp, one row whose x was just left at f: its h instead.
-__device__ __forceinline__ void norm_in_place(const AddNorm& p, float* row, RowStats r) {
-  for (int v = threadIdx.x & 31; v < p.ld / 8; v += 32) {
-    float f[8], g[8], c[8];
-    load_vec<8>(row + v * 8, f);
-    norm_vectors(p, v, g, c);
+  auto norm = [&](int t, float* f) {
+    const float2 r = stats[t];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) f[e] = (f[e] - r.mean) * r.rs * g[e] + c[e];
-    store_vec<8>(row + v * 8, f);
-  }
-}
-
-template <typename T, typename Y, int HIST>     // n_taps - 1 <= HIST
-__global__ void __launch_bounds__(CN_THREADS) add_norm_conv_kernel(const AddNorm p) {
-  extern __shared__ __align__(16) float halo[];          // [n_taps - 1, ld]: h in front of the tile
-  __shared__ RowStats stats[SHIFT_TILE];
-  const int back = p.n_taps - 1, nv = p.ld / 8;
-  const int e = p.tile_entry[blockIdx.x], off = p.tile_off[blockIdx.x];
-  const int row0 = p.e.row0[e], len = p.e.len[e];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n = min(SHIFT_TILE, len - off);
-  float* state = p.before + static_cast<size_t>(p.e.slot[e]) * back * p.ld;
-  if (off == 0) {
-    const bool has = p.e.pos0[e] > 0;
-    for (int i = threadIdx.x; i < back * p.ld / 4; i += CN_THREADS)
-      reinterpret_cast<float4*>(halo)[i] = has ? reinterpret_cast<const float4*>(state)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  for (int i = warp - (off > 0 ? back : 0); i < n; i += CN_THREADS / 32) {
-    const int row = row0 + off + i;
-    if (i < 0) {
-      float* dst = halo + (back + i) * p.ld;
-      norm_in_place(p, dst, conv_row<T, Y>(p, row, dst));
+    for (int k = 0; k < 8; ++k) f[k] = (f[k] - r.x) * r.y * g[k] + c[k];
+  };
+  auto h_of = [&](int t, float* f) {             // of the entry's token t; negative: of the step before
+    if (t >= 0) {
+      load_vec<8>(src + static_cast<size_t>(t) * p.ld, f);
+      norm(t, f);
+    } else if (has) {
+      load_vec<8>(state + static_cast<size_t>(back + t) * p.ld, f);
     } else {
-      const RowStats r = conv_row<T, Y>(p, row, p.x_out != nullptr ? p.x_out + static_cast<size_t>(row) * p.ld : nullptr);
-      if (lane == 0) stats[i] = r;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) f[k] = 0.f;
     }
-  }
-  __syncthreads();
-  const float* src = (p.x_out != nullptr ? p.x_out : p.x) + static_cast<size_t>(row0 + off) * p.ld;
-  T* dst = static_cast<T*>(p.h) + static_cast<size_t>(row0 + off) * p.ldh;
-  const bool all = off == 0 && n == len;                 // the state is what this tile leaves
-  for (int v = threadIdx.x; v < nv; v += CN_THREADS) {
-    float w[HIST + 1][8], prev[HIST][8], g[8], c[8];     // [d]: d tokens back; prev[d - 1]
-    norm_vectors(p, v, g, c);
+  };
+  if constexpr (HIST > 0) {
+    float w[HIST + 1][8], prev[HIST][8];         // [d]: d tokens back; prev[d - 1]
 #pragma unroll
     for (int d = 0; d <= HIST; ++d) {
 #pragma unroll
@@ -412,77 +370,90 @@ __global__ void __launch_bounds__(CN_THREADS) add_norm_conv_kernel(const AddNorm
       }
       if (d <= back) {
         load_vec<8>(p.taps + static_cast<size_t>(back - d) * p.ld + v * 8, w[d]);
-        if (d > 0) load_vec<8>(halo + (back - d) * p.ld + v * 8, prev[d > 0 ? d - 1 : 0]);
+        if (d > 0) h_of(off - d, prev[d > 0 ? d - 1 : 0]);
       }
     }
-    if (all)                                             // tokens that stay in the state, moved on
-      for (int k = 0; k < back - n; ++k) {
-        float f[8];
-        load_vec<8>(halo + (n + k) * p.ld + v * 8, f);
-        store_vec<8>(state + static_cast<size_t>(k) * p.ld + v * 8, f);
+    for (int t0 = off; t0 < t1; t0 += CN_AHEAD) {
+      float x[CN_AHEAD][8];
+#pragma unroll
+      for (int i = 0; i < CN_AHEAD; ++i)
+        if (t0 + i < t1) load_vec<8>(src + static_cast<size_t>(t0 + i) * p.ld, x[i]);
+#pragma unroll
+      for (int i = 0; i < CN_AHEAD; ++i) {
+        if (t0 + i >= t1) break;
+        norm(t0 + i, x[i]);
+        float o[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          float a = w[0][k] * x[i][k];
+#pragma unroll
+          for (int d = 1; d <= HIST; ++d) a += w[d][k] * prev[d - 1][k];
+          o[k] = x[i][k] + a;
+#pragma unroll
+          for (int d = HIST - 1; d > 0; --d) prev[d][k] = prev[d - 1][k];
+          prev[0][k] = x[i][k];
+        }
+        store_vec<8>(dst + static_cast<size_t>(t0 + i) * p.ldh, o);
       }
-#pragma unroll 4
-    for (int t = 0; t < n; ++t) {
-      float f[8], o[8];
-      load_vec<8>(src + static_cast<size_t>(t) * p.ld + v * 8, f);
-      const RowStats r = stats[t];
+    }
+  } else {
+    for (int t = off; t < t1; ++t) {
+      float f[8], o[8], w[8];
+      h_of(t, f);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        f[k] = (f[k] - r.mean) * r.rs * g[k] + c[k];
-        float a = w[0][k] * f[k];
+      for (int k = 0; k < 8; ++k) o[k] = f[k];
+      for (int d = 0; d <= back; ++d) {
+        if (d > 0) h_of(t - d, f);
+        load_vec<8>(p.taps + static_cast<size_t>(back - d) * p.ld + v * 8, w);
 #pragma unroll
-        for (int d = 1; d <= HIST; ++d) a += w[d][k] * prev[d - 1][k];
-        o[k] = f[k] + a;
-#pragma unroll
-        for (int d = HIST - 1; d > 0; --d) prev[d][k] = prev[d - 1][k];
-        prev[0][k] = f[k];
+        for (int k = 0; k < 8; ++k) o[k] += w[k] * f[k];
       }
-      store_vec<8>(dst + static_cast<size_t>(t) * p.ldh + v * 8, o);
-      if (all && t >= n - back) store_vec<8>(state + static_cast<size_t>(t - n + back) * p.ld + v * 8, f);
+      store_vec<8>(dst + static_cast<size_t>(t) * p.ldh, o);
     }
   }
-  if (off > 0 || all) return;
-  __syncthreads();                                       // the state has been read
-  for (int k = warp; k < back; k += CN_THREADS / 32) {   // a longer entry's last tokens
-    float* row = state + static_cast<size_t>(k) * p.ld;
-    norm_in_place(p, row, conv_row<T, Y>(p, row0 + len - back + k, row));
+  if (off > 0) return;
+  for (int k = 0; k < back; ++k) {               // the entry's last tokens; what is read lies behind k
+    float f[8];
+    h_of(len - back + k, f);
+    store_vec<8>(state + static_cast<size_t>(k) * p.ld, f);
   }
 }
 
-template <typename T, typename Y, int HIST>
-static int launch_add_norm_conv(const AddNorm& p, int blocks, cudaStream_t st) {
-  const int smem = (p.n_taps - 1) * p.ld * 4;
-  static int set = 48 * 1024;
-  if (smem > set) {
-    if (cudaFuncSetAttribute(add_norm_conv_kernel<T, Y, HIST>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             CN_SMEM) != cudaSuccess)
-      return -4;
-    set = CN_SMEM;
-  }
-  add_norm_conv_kernel<T, Y, HIST><<<blocks, CN_THREADS, smem, st>>>(p);
-  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+template <typename T>
+static void launch_conv_pass(const AddNorm& p, int tiles, cudaStream_t st) {
+  const dim3 grid(tiles, (p.ld / 8 + CN_THREADS - 1) / CN_THREADS);
+  if (p.n_taps <= 4) conv_pass_kernel<T, 3><<<grid, CN_THREADS, 0, st>>>(p);
+  else conv_pass_kernel<T, 0><<<grid, CN_THREADS, 0, st>>>(p);
 }
 
-template <typename T, typename Y>
+template <typename T, typename Y, int MODE>
 static int launch_add_norm(const AddNorm& p, int blocks, cudaStream_t st) {
-  if (p.taps != nullptr)
-    return p.n_taps <= 4 ? launch_add_norm_conv<T, Y, 3>(p, blocks, st) : launch_add_norm_conv<T, Y, 16>(p, blocks, st);
   const int nv = p.ld / 8;
   if (nv <= 512) {
-    add_norm_kernel<T, Y, 1><<<blocks, (nv + 31) / 32 * 32, 0, st>>>(p);
+    add_norm_kernel<T, Y, 1, MODE><<<blocks, (nv + 31) / 32 * 32, 0, st>>>(p);
   } else if (nv <= 1024) {
-    add_norm_kernel<T, Y, 2><<<blocks, 512, 0, st>>>(p);
+    add_norm_kernel<T, Y, 2, MODE><<<blocks, 512, 0, st>>>(p);
   } else {
-    add_norm_kernel<T, Y, 4><<<blocks, 512, 0, st>>>(p);
+    add_norm_kernel<T, Y, 4, MODE><<<blocks, 512, 0, st>>>(p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+template <typename T, typename Y>
+static int launch_add_norm_mode(const AddNorm& p, int blocks, int rows, cudaStream_t st) {
+  if (p.shift != nullptr) return launch_add_norm<T, Y, AN_SHIFT>(p, blocks, st);
+  if (p.taps == nullptr) return launch_add_norm<T, Y, AN_ROWS>(p, blocks, st);
+  if (p.tile_entry == nullptr) return launch_add_norm<T, Y, AN_TOKEN>(p, blocks, st);
+  const int rc = launch_add_norm<T, Y, AN_STATS>(p, rows, st);
+  if (rc == 0) launch_conv_pass<T>(p, blocks, st);
+  return rc == 0 && cudaGetLastError() != cudaSuccess ? -3 : rc;
 }
 
 }  // namespace cb
 
 using namespace cb;
 
-// blocks: rows (without a shift or a convolution) or tiles.  y_f32: y is fp32 although T is bf16.
+// blocks: rows (without a shift or a convolution) or tiles, with rows_all rows in all and a convolution's stats
+// [rows_all, 2].  y_f32: y is fp32 although T is bf16.
 extern "C" int cb_add_norm(const float* x, const void* y, const float* bias, const float* post,
                            int post_vec, float* x_out, int ld, int ldy, const float* gain,
                            int gain_vec, void* h, int ldh, void* cast0, void* cast1, int ldc,
@@ -492,7 +463,7 @@ extern "C" int cb_add_norm(const float* x, const void* y, const float* bias, con
                            const void* spread, int lds, const int* spread_slot,
                            const float* spread_weight, int top, const void* own, int ldo, const float* y_weight,
                            const float* scale, const float* center, const float* taps, int n_taps,
-                           void* stream) {
+                           float* stats, int rows_all, void* stream) {
   if (blocks <= 0 || ld % 8 || width > ld || ld > 16384) return -1;
   if (y != nullptr && (ldy % 8 || ldy < ld)) return -2;
   if (gain != nullptr && (h == nullptr || ldh % 8 || ldh < ld)) return -2;
@@ -504,14 +475,15 @@ extern "C" int cb_add_norm(const float* x, const void* y, const float* bias, con
   if (own != nullptr && (ldo % 8 || ldo < ld)) return -2;
   if (taps != nullptr) {
     if (gain == nullptr || shift != nullptr || rows != nullptr || post != nullptr || cast0 != nullptr ||
-        cast1 != nullptr || tile_entry == nullptr || tile_off == nullptr)
+        cast1 != nullptr || (tile_entry == nullptr) != (tile_off == nullptr) || slot == nullptr || pos0 == nullptr)
       return -2;
-    if (n_taps < 1 || n_taps > 17 || (n_taps > 1 && before == nullptr) || (n_taps - 1) * ld * 4 > CN_SMEM) return -2;
+    if (n_taps < 1 || n_taps > SHIFT_TILE + 1 || (n_taps > 1 && before == nullptr)) return -2;
+    if (tile_entry != nullptr && (stats == nullptr || rows_all < 1)) return -2;
     if (x_out != nullptr ? x == x_out : (x == nullptr || y != nullptr || spread != nullptr)) return -2;
   }
   AddNorm p;
   p.own = own; p.ldo = ldo; p.y_weight = y_weight; p.scale = scale; p.center = center; p.taps = taps;
-  p.n_taps = n_taps;
+  p.n_taps = n_taps; p.stats = reinterpret_cast<float2*>(stats);
   p.spread = spread; p.lds = lds; p.spread_slot = spread_slot; p.spread_weight = spread_weight; p.top = top;
   p.x = x; p.y = y; p.bias = bias; p.post = post; p.post_vec = post_vec; p.x_out = x_out;
   p.ld = ld; p.ldy = ldy; p.gain = gain; p.gain_vec = gain_vec; p.h = h; p.ldh = ldh;
@@ -519,7 +491,7 @@ extern "C" int cb_add_norm(const float* x, const void* y, const float* bias, con
   p.rows = rows; p.e.slot = slot; p.e.row0 = row0; p.e.len = len; p.e.pos0 = pos0;
   p.tile_entry = tile_entry; p.tile_off = tile_off; p.width = width; p.eps = eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) return launch_add_norm<float, float>(p, blocks, st);
-  return y_f32 ? launch_add_norm<__nv_bfloat16, float>(p, blocks, st)
-               : launch_add_norm<__nv_bfloat16, __nv_bfloat16>(p, blocks, st);
+  if (f32) return launch_add_norm_mode<float, float>(p, blocks, rows_all, st);
+  return y_f32 ? launch_add_norm_mode<__nv_bfloat16, float>(p, blocks, rows_all, st)
+               : launch_add_norm_mode<__nv_bfloat16, __nv_bfloat16>(p, blocks, rows_all, st);
 }

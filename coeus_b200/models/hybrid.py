@@ -35,7 +35,6 @@ MAX_HEAD_DIM = 256           # the attention and recurrence kernels' limit per h
 MAX_LATENT = 640             # and per cached latent row
 MAX_TAPS = 17                # and of the convolution kernels
 MAX_WIDTH = 16384            # and of the pass between two sublayers
-MAX_HISTORY = 52 * 1024      # numbers of earlier tokens that this pass keeps for its convolution
 MAX_EXPERTS, MAX_TOP = 256, 16   # and of the routing kernels
 DEFAULT_MAX_SEQ_LEN = 8192   # serving default; the designs themselves have no length limit
 
@@ -716,8 +715,6 @@ class HybridConfig:
                 self._check_shared(i, m)
         if self.design.input_conv:
             _taps_ok("conv_taps", self.conv_taps)
-            if (self.conv_taps - 1) * self.width_padded > MAX_HISTORY:
-                _refuse("conv_taps", self.conv_taps, f"Taps times width must not exceed {MAX_HISTORY}")
         if self.loop is not None:
             lo = self.loop
             if self.design.parallel:

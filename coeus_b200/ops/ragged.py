@@ -433,7 +433,10 @@ def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dty
     h = torch.empty((n, ld), dtype=dtype, device=src.device) if gain is not None else None
     shifted = shift is not None or taps is not None
     none = (None,) * 6
-    ents = (*batch.entry_args(), _p(batch.conv_entry), _p(batch.conv_off)) if shifted else none
+    tiles = shifted and not (taps is not None and batch.T == batch.n)      # else every entry is one token
+    ents = none if not shifted else (*batch.entry_args(), *((_p(batch.conv_entry), _p(batch.conv_off)) if tiles
+                                                            else (None, None)))
+    stats = torch.empty((n, 2), dtype=torch.float32, device=src.device) if tiles and taps is not None else None
     cast = list(casts) + [None] * (2 - len(casts))
     sp = (None, 0, None, None, 0, None, 0) if spread is None else (
         _p(spread.rows), spread.rows.stride(0), _p(spread.slot), _p(spread.weight), spread.slot.shape[1],
@@ -442,10 +445,10 @@ def add_norm(x: Optional[torch.Tensor], width: int, eps: float, dtype: torch.dty
         _p(x), _p(y), _p(bias), _p(post), int(post is not None and post.numel() > 1), _p(x_out), ld,
         y.stride(0) if y is not None else 0, _p(gain), int(gain is not None and gain.numel() > 1), _p(h),
         ld, _p(cast[0]), _p(cast[1]), casts[0].stride(0) if casts else 0, _p(shift), _p(before),
-        _p(rows), *ents, batch.n_conv if shifted else n, width, _F(eps), int(dtype == torch.float32),
+        _p(rows), *ents, batch.n_conv if tiles else n, width, _F(eps), int(dtype == torch.float32),
         int(y is not None and y.dtype == torch.float32), *sp, _p(y_weight), _p(scale), _p(center), _p(taps),
-        taps.shape[0] if taps is not None else 0, _lib.stream_ptr())
-    _lib.check_rc(rc, "cb_add_norm")
+        taps.shape[0] if taps is not None else 0, _p(stats), n, _lib.stream_ptr())
+    _lib.check_rc(rc, "cb_add_norm", launches=1 if stats is None else 2)
     return (x_out if x_out is not None else (x if keep else None)), h
 
 

@@ -170,7 +170,7 @@ def check_input_convolution(device, dtype, tol):
     eps, T = 1e-4, 75
     cuts = (((1, 30), (2, 1), (1, 2), (17, 1), (16, 33), (18, 1), (20, 7)), ((75, 3), (0, 72)), ((40, 16), (35, 59)))
     for W, ld, taps in ((44, 48, 3), (50, 56, 1), (96, 96, 4), (40, 40, 2), (24, 24, 17), (72, 72, 6), (2100, 2104, 4),
-                        (4200, 4200, 2)):
+                        (4200, 4200, 2), (4096, 4096, 4)):
         def vec(s, base=0.0):
             return torch.nn.functional.pad(base + 0.3 * rnd((W,), s, device), (0, ld - W))
         w = torch.nn.functional.pad(rnd((taps, W), 3, device), (0, ld - W))
