@@ -73,12 +73,7 @@ __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, f
     }
   }
   __syncwarp();
-  uint32_t open[MOE_E / 32];                     // kept groups
-#pragma unroll
-  for (int i = 0; i < MOE_E / 32; ++i) open[i] = 0xffffffffu;
   if (p.keep < p.groups) {
-#pragma unroll
-    for (int i = 0; i < MOE_E / 32; ++i) open[i] = 0u;
     for (int g = lane; g < p.groups; g += 32) {
       float a = -INFINITY, b = -INFINITY;
       for (int i = 0; i < n; ++i) {
@@ -96,10 +91,7 @@ __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, f
         if (gv[g] > v) { v = gv[g]; at = g; }
       warp_best(v, at);
       __syncwarp();
-      if (lane == 0) gv[at] = -INFINITY;
-#pragma unroll
-      for (int i = 0; i < MOE_E / 32; ++i)
-        if (i == at >> 5) open[i] |= 1u << (at & 31);
+      if (lane == 0) gv[at] = -INFINITY;         // kept
       __syncwarp();
     }
   }
@@ -107,31 +99,23 @@ __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, f
 #pragma unroll
   for (int i = 0; i < MOE_E / 32; ++i) {
     const int e = lane + 32 * i;
-    left[i] = -INFINITY;
-    if (e < p.E) {
-      const int g = e / n;
-      uint32_t bits = 0u;
-#pragma unroll
-      for (int x = 0; x < MOE_E / 32; ++x)
-        if (x == g >> 5) bits = open[x];
-      if (bits >> (g & 31) & 1u) left[i] = s[e];
-    }
+    left[i] = e < p.E && (p.keep == p.groups || gv[e / n] == -INFINITY) ? s[e] : -INFINITY;
+    if (e < p.E) s[e] = score[i];
   }
+  __syncwarp();
   float mine = 0.f, sum = 0.f;
   int chosen = 0;
   for (int k = 0; k < p.top; ++k) {
-    float v = -INFINITY, w = 0.f;
+    float v = -INFINITY;
     int at = p.E - 1;
 #pragma unroll
     for (int i = 0; i < MOE_E / 32; ++i)
       if (left[i] > v) { v = left[i]; at = lane + 32 * i; }
     warp_best(v, at);
 #pragma unroll
-    for (int i = 0; i < MOE_E / 32; ++i) {
-      if (i == at >> 5) w = score[i];
+    for (int i = 0; i < MOE_E / 32; ++i)
       if (at == lane + 32 * i) left[i] = -INFINITY;
-    }
-    w = __shfl_sync(FULL, w, at & 31);
+    const float w = s[at];
     sum += w;
     if (lane == k) { mine = w; chosen = at; }
   }

@@ -58,6 +58,7 @@ __device__ __forceinline__ void head_load(const T* src, int d, int n, float* f) 
 template <typename T, bool VEC>
 __device__ __forceinline__ float row_squares(const T* src, int n) {
   float s = 0.f;
+#pragma unroll 2
   for (int c = threadIdx.x * 8; c < n; c += HP_THREADS * 8) {
     float f[8];
     head_load<T, VEC>(src + c, 0, n - c, f);
@@ -82,11 +83,24 @@ __global__ void __launch_bounds__(HP_THREADS) head_prep_kernel(const HeadPrep p)
   const float2* rope = p.rope + static_cast<size_t>(row) * p.half;
   float q_rs = 1.f, k_rs = 1.f;
   if (p.q_norm != nullptr) {
-    __shared__ float red[32];
-    q_rs = 1.0f / sqrtf(block_sum(row_squares<T, VEC>(raw, p.heads * p.dim), red) / (p.heads * p.dim) + p.eps);
-    if (p.kv_heads > 0)
-      k_rs = 1.0f / sqrtf(block_sum(row_squares<T, VEC>(raw + p.koff, p.kv_heads * p.dim), red) /
-                              (p.kv_heads * p.dim) + p.eps);
+    __shared__ float red[2][HP_THREADS / 32];
+    const int nq = p.heads * p.dim, nk = p.kv_heads * p.dim;
+    float sq = row_squares<T, VEC>(raw, nq), sk = row_squares<T, VEC>(raw + p.koff, nk);
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) {
+      red[0][threadIdx.x >> 5] = sq;
+      red[1][threadIdx.x >> 5] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < HP_THREADS / 32; ++i) {
+      sq += red[0][i];
+      sk += red[1][i];
+    }
+    q_rs = 1.0f / sqrtf(sq / nq + p.eps);
+    if (nk > 0) k_rs = 1.0f / sqrtf(sk / nk + p.eps);
   }
   const int v_units = (max(p.vdim_p, p.vr_head) + 8 * L - 1) / (8 * L);     // per head
   const int units = p.heads + p.kv_heads + p.v_heads * v_units;
