@@ -50,10 +50,11 @@ __device__ __forceinline__ void warp_best(float& v, int& i) {
 }
 
 // One warp, one token: s[E] holds the logits and becomes the scores that are compared; gv is scratch for the
-// groups.
+// groups.  NI: experts per lane.
+template <int NI>
 __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, float* gv) {
   const int lane = threadIdx.x & 31, n = p.E / p.groups;
-  float score[MOE_E / 32];                       // of this lane's experts lane, lane + 32, ...
+  float score[NI];                       // of this lane's experts lane, lane + 32, ...
   float total = 1.f, top = 0.f;
   if (p.softmax) {
     top = -INFINITY;
@@ -64,7 +65,7 @@ __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, f
     total = warp_sum(total);
   }
 #pragma unroll
-  for (int i = 0; i < MOE_E / 32; ++i) {
+  for (int i = 0; i < NI; ++i) {
     const int e = lane + 32 * i;
     score[i] = 0.f;
     if (e < p.E) {
@@ -95,9 +96,9 @@ __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, f
       __syncwarp();
     }
   }
-  float left[MOE_E / 32];
+  float left[NI];
 #pragma unroll
-  for (int i = 0; i < MOE_E / 32; ++i) {
+  for (int i = 0; i < NI; ++i) {
     const int e = lane + 32 * i;
     left[i] = e < p.E && (p.keep == p.groups || gv[e / n] == -INFINITY) ? s[e] : -INFINITY;
     if (e < p.E) s[e] = score[i];
@@ -109,11 +110,11 @@ __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, f
     float v = -INFINITY;
     int at = p.E - 1;
 #pragma unroll
-    for (int i = 0; i < MOE_E / 32; ++i)
+    for (int i = 0; i < NI; ++i)
       if (left[i] > v) { v = left[i]; at = lane + 32 * i; }
     warp_best(v, at);
 #pragma unroll
-    for (int i = 0; i < MOE_E / 32; ++i)
+    for (int i = 0; i < NI; ++i)
       if (at == lane + 32 * i) left[i] = -INFINITY;
     const float w = s[at];
     sum += w;
@@ -126,6 +127,7 @@ __device__ __forceinline__ void choose_token(const Choose& p, int t, float* s, f
   __syncwarp();
 }
 
+template <int NI>
 __global__ void __launch_bounds__(CHOOSE_WARPS * 32) moe_choose_kernel(const Choose p) {
   __shared__ float s[CHOOSE_WARPS][MOE_E], gv[CHOOSE_WARPS][MOE_E];
   __shared__ int pair[CHOOSE_TOKENS * MOE_K], hist[MOE_E];
@@ -136,7 +138,7 @@ __global__ void __launch_bounds__(CHOOSE_WARPS * 32) moe_choose_kernel(const Cho
     __syncwarp();
     if (p.shared != nullptr && lane == 0)
       p.shared[t0 + t] = sigmoidf_(p.logits[static_cast<size_t>(t0 + t) * p.ldl + p.E]);
-    choose_token(p, t0 + t, s[warp], gv[warp]);
+    choose_token<NI>(p, t0 + t, s[warp], gv[warp]);
   }
   for (int e = threadIdx.x; e < p.E; e += CHOOSE_WARPS * 32) hist[e] = 0;
   __syncthreads();
@@ -156,7 +158,7 @@ __global__ void __launch_bounds__(CHOOSE_WARPS * 32) moe_choose_kernel(const Cho
 }
 
 // One token per block, with the router's product: two experts per warp at a time.
-template <typename T>
+template <typename T, int NI>
 __global__ void __launch_bounds__(512) moe_choose_few_kernel(const Choose p) {
   __shared__ float s[MOE_E + 4], gv[MOE_E];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x, nw = blockDim.x >> 5;
@@ -189,7 +191,7 @@ __global__ void __launch_bounds__(512) moe_choose_few_kernel(const Choose p) {
   __syncthreads();
   if (warp != 0) return;
   if (p.shared != nullptr && lane == 0) p.shared[t] = sigmoidf_(s[p.E]);
-  choose_token(p, t, s, gv);
+  choose_token<NI>(p, t, s, gv);
   for (int e = lane; e < p.E; e += 32) p.counts[static_cast<size_t>(e) * p.blocks + t] = 0;
   __syncwarp();
   if (lane < p.top) {
@@ -515,6 +517,13 @@ __global__ void __launch_bounds__(DOWN_WARPS * 32) moe_few_down_kernel(const Few
 using namespace cb;
 #define CB_RC() (cudaGetLastError() == cudaSuccess ? 0 : -3)
 
+template <int NI>
+static void launch_choose(const Choose& p, int f32, cudaStream_t st) {
+  if (p.logits != nullptr) moe_choose_kernel<NI><<<p.blocks, CHOOSE_WARPS * 32, 0, st>>>(p);
+  else if (f32) moe_choose_few_kernel<float, NI><<<p.T, 512, 0, st>>>(p);
+  else moe_choose_few_kernel<__nv_bfloat16, NI><<<p.T, 512, 0, st>>>(p);
+}
+
 // logits null: computed here, one block (of the counts) per token; else blocks of CHOOSE_TOKENS tokens.  E
 // counts the identity experts too; shared (or null) gets the sigmoid of logit E.
 extern "C" int cb_moe_choose(const float* logits, int ldl, const void* h, int ldh, const void* router,
@@ -534,12 +543,8 @@ extern "C" int cb_moe_choose(const float* logits, int ldl, const void* h, int ld
   p.weight = weight; p.rank = rank; p.counts = counts;
   p.blocks = logits != nullptr ? (T + CHOOSE_TOKENS - 1) / CHOOSE_TOKENS : T;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (logits != nullptr)
-    moe_choose_kernel<<<p.blocks, CHOOSE_WARPS * 32, 0, st>>>(p);
-  else if (f32)
-    moe_choose_few_kernel<float><<<T, 512, 0, st>>>(p);
-  else
-    moe_choose_few_kernel<__nv_bfloat16><<<T, 512, 0, st>>>(p);
+  if (E <= 32) launch_choose<1>(p, f32, st);
+  else launch_choose<MOE_E / 32>(p, f32, st);
   return CB_RC();
 }
 
